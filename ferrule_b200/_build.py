@@ -34,6 +34,9 @@ CUDA_SOURCES = [
     "data_movers.cu",
     "quant.cu",
     "v4_ops.cu",
+    "layered_ops.cu",
+    "delta_rule.cu",
+    "gemm_f32.cu",
     "ep_moe.cu",
     "expert_table.cu",
     "comm.cu",

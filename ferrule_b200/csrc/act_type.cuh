@@ -1,0 +1,55 @@
+// Element access for kernels that exist in bf16 (served models) and fp32 (full 32-bit runs): every value is computed
+// in fp32, `T` is only the storage type of activations.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stdint.h>
+
+namespace fb {
+
+__device__ __forceinline__ float act_load(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float act_load(const float* p) { return *p; }
+__device__ __forceinline__ void act_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ void act_store(float* p, float v) { *p = v; }
+
+// eight consecutive elements, 16-byte aligned
+__device__ __forceinline__ void act_load8(const __nv_bfloat16* p, float (&v)[8]) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&a);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) v[j] = __bfloat162float(e[j]);
+}
+__device__ __forceinline__ void act_load8(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void act_store8(__nv_bfloat16* p, const float (&v)[8]) {
+  uint4 a;
+  __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&a);
+#pragma unroll
+  for (int j = 0; j < 8; ++j) e[j] = __float2bfloat16_rn(v[j]);
+  *reinterpret_cast<uint4*>(p) = a;
+}
+__device__ __forceinline__ void act_store8(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+// sum over a block of `blockDim.x` threads (a multiple of 32, at most 1024); `red` holds 32 floats
+__device__ __forceinline__ float cta_sum(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < nw ? red[lane] : 0.f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+  return t;
+}
+
+}  // namespace fb

@@ -1,0 +1,535 @@
+// Gated delta rule with one decay per key channel, short causal convolutions in front, gated per-head output norm.
+//
+// Per head, S [dim, vdim] in fp32, rows of key channels:
+//     S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+// with q, k the unit vectors (q also times dim^-1/2) of silu(conv(W x)), v = silu(conv(W_v x)),
+// g = exp(a_neg * softplus(decay + dt_bias)), beta = sigmoid(b).
+//
+// State of a sequence: one S per head and the last taps - 1 projected inputs of every convolved channel.  A slot of
+// the state pool has several buffers; a step reads buffer `state_in[seq]` (-1: a new sequence, all zeros) and writes
+// buffer `state_out[seq]` (-1: nothing is kept), so a step that is rolled back leaves the committed state untouched.
+//
+//   fb_delta_decode   one row per sequence, everything in one launch: one CTA per (sequence, head), the state slice in
+//                     registers (16 bytes per thread and row)
+//   fb_delta_prefill  any mix of row counts: prepare (convolutions, unit norms, decays; one CTA per row) -> scan (the
+//                     recurrence, state in registers, eight lanes per value column) -> output norm and gate
+//
+// S^T q after the write equals S^T q before it plus (q . k) u, so both dot products of a token are taken in one pass
+// over the decayed state.
+#include "act_type.cuh"
+#include "common.cuh"
+#include "ferrule_b200.h"
+#include "launch.cuh"
+
+namespace fb {
+
+template <typename T>
+struct DeltaParams {
+  const T* proj;              // [rows, ldp]: pre-convolution q | k | v at off_q / off_k / off_v, beta logits at off_b
+  long long ldp;
+  int off_q, off_k, off_v, off_b;
+  const float* ag;            // [rows, ldag]: decay pre-activation at 0, output gate pre-activation at off_gate
+  long long ldag;
+  int off_gate;
+  const float* conv;          // [channels, taps], channels = q | k | v
+  const float* a_neg;         // [heads]
+  const float* dt_bias;       // [heads * dim]
+  const float* norm_w;        // [vdim]
+  float eps;
+  float* state;               // [n_states, heads, dim, vdim]
+  T* tail;                    // [n_states, taps - 1, channels]
+  int n_states;
+  const int* row_seq;
+  const int* seq_start;       // [n_seqs + 1]
+  const int* state_in;
+  const int* state_out;
+  int rows, n_seqs, heads, kv_heads, dim, vdim, taps;
+  float *qn, *kn, *v, *decay, *beta, *qk, *o;      // scratch of the prefill form
+  T* out;                     // [rows, ldo]
+  long long ldo;
+  DeviceStatus* status;
+  __device__ int channels() const { return 2 * kv_heads * dim + heads * vdim; }
+  // column of channel c in a projected row
+  __device__ int col(int c) const {
+    const int nk = kv_heads * dim;
+    return c < nk ? off_q + c : (c < 2 * nk ? off_k + c - nk : off_v + c - 2 * nk);
+  }
+};
+
+// silu(conv) of channel c at local row i of the sequence whose rows start at r0
+template <typename T>
+__device__ __forceinline__ float conv_silu(const DeltaParams<T>& p, int c, int r0, int i, int sin, int channels) {
+  const int col = p.col(c), taps = p.taps;
+  float acc = 0.f;
+  for (int j = 0; j < taps; ++j) {
+    const int idx = i - (taps - 1) + j;
+    float x = 0.f;
+    if (idx >= 0) x = act_load(p.proj + (r0 + idx) * p.ldp + col);
+    else if (sin >= 0) x = act_load(p.tail + (static_cast<long long>(sin) * (taps - 1) + idx + taps - 1) * channels + c);
+    acc = fmaf(p.conv[c * taps + j], x, acc);
+  }
+  return acc / (1.f + expf(-acc));
+}
+
+// The convolution inputs the next step needs: entry j of the tail is the input `taps - 1 - j` tokens before the end.
+// Called for local row i of n: that row's own entry, and by row 0 the entries that still come from the old tail.
+template <typename T>
+__device__ __forceinline__ void store_tail(const DeltaParams<T>& p, int c, int r0, int i, int n, int sin, int sout,
+                                           int channels) {
+  const int keep = p.taps - 1;
+  if (sout < 0 || keep <= 0) return;
+  T* dst = p.tail + static_cast<long long>(sout) * keep * channels + c;
+  const int j = i - (n - keep);
+  if (j >= 0) dst[static_cast<long long>(j) * channels] = p.proj[(r0 + i) * p.ldp + p.col(c)];
+  if (i == 0) {
+    for (int q = 0; q < keep - n; ++q) {
+      T x{};
+      if (sin >= 0) x = p.tail[(static_cast<long long>(sin) * keep + q + n) * channels + c];
+      else act_store(&x, 0.f);
+      dst[static_cast<long long>(q) * channels] = x;
+    }
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ bool seq_states(const DeltaParams<T>& p, int seq, int& sin, int& sout) {
+  sin = p.state_in[seq];
+  sout = p.state_out[seq];
+  if (sin >= p.n_states || sout >= p.n_states || (sin >= 0 && sin == sout)) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xC00, seq, sout);
+    return false;
+  }
+  return true;
+}
+
+// ---------------------------------------------------------------------------------
+// prepare: one CTA per row
+// ---------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_prepare_kernel(const DeltaParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float qk_s[];                 // [2 * kv_heads * dim]
+  const int r = blockIdx.x;
+  const int seq = p.row_seq[r];
+  if (seq < 0 || seq >= p.n_seqs) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xC01, r, seq);
+    return;
+  }
+  const int r0 = p.seq_start[seq], n = p.seq_start[seq + 1] - r0, i = r - r0;
+  if (r0 < 0 || i < 0 || i >= n || r0 + n > p.rows) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xC02, r, r0);
+    return;
+  }
+  int sin, sout;
+  if (!seq_states(p, seq, sin, sout)) return;
+  const int nk = p.kv_heads * p.dim, nv = p.heads * p.vdim, channels = p.channels();
+  for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+    const float y = conv_silu(p, c, r0, i, sin, channels);
+    if (c < 2 * nk) qk_s[c] = y;
+    else p.v[static_cast<long long>(r) * nv + c - 2 * nk] = y;
+    store_tail(p, c, r0, i, n, sin, sout, channels);
+  }
+  for (int c = threadIdx.x; c < p.heads * p.dim; c += blockDim.x)
+    p.decay[static_cast<long long>(r) * p.heads * p.dim + c] =
+        expf(p.a_neg[c / p.dim] * softplus_f(p.ag[r * p.ldag + c] + p.dt_bias[c]));
+  for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
+    p.beta[static_cast<long long>(r) * p.heads + h] = sigmoid_f(act_load(p.proj + r * p.ldp + p.off_b + h));
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  for (int h = warp; h < p.kv_heads; h += nw) {
+    const float* q = qk_s + h * p.dim;
+    const float* k = qk_s + nk + h * p.dim;
+    float sq = 0.f, sk = 0.f, dot = 0.f;
+    for (int d = lane; d < p.dim; d += 32) {
+      sq = fmaf(q[d], q[d], sq);
+      sk = fmaf(k[d], k[d], sk);
+      dot = fmaf(q[d], k[d], dot);
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    dot = warp_sum(dot);
+    const float fq = 1.f / sqrtf(sq + 1e-6f) / sqrtf(static_cast<float>(p.dim)), fk = 1.f / sqrtf(sk + 1e-6f);
+    const long long base = static_cast<long long>(r) * nk + h * p.dim;
+    for (int d = lane; d < p.dim; d += 32) {
+      p.qn[base + d] = q[d] * fq;
+      p.kn[base + d] = k[d] * fk;
+    }
+    if (lane == 0) p.qk[static_cast<long long>(r) * p.kv_heads + h] = dot * fq * fk;
+  }
+}
+
+__device__ __forceinline__ void cp_async4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+
+// ---------------------------------------------------------------------------------
+// scan: CTA = (head, 16 value columns) x sequence; eight lanes per column, lane l holds the key channels
+// 32 * (j / 4) + 4 * l + j % 4.  Tokens are staged sixteen at a time, double buffered.
+// ---------------------------------------------------------------------------------
+constexpr int kScanStep = 16, kScanCols = 16;
+
+template <typename T, int RPT>
+__global__ void __launch_bounds__(128)
+delta_scan_kernel(const DeltaParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int DP = RPT * 8;                                   // padded key dimension
+  extern __shared__ float sm[];
+  // per buffer: k, q, g [kScanStep][DP], v [kScanStep][kScanCols], beta, qk [kScanStep]
+  constexpr int kBuf = kScanStep * (3 * DP + kScanCols + 2);
+  const int seq = blockIdx.y;
+  const int vtiles = (p.vdim + kScanCols - 1) / kScanCols;
+  const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * kScanCols;
+  const int hk = h / (p.heads / p.kv_heads);
+  const int r0 = p.seq_start[seq], n = p.seq_start[seq + 1] - r0;
+  if (r0 < 0 || n <= 0 || r0 + n > p.rows) return;              // reported by the prepare kernel
+  int sin, sout;
+  if (!seq_states(p, seq, sin, sout)) return;
+  const int tid = threadIdx.x, l8 = tid & 7;
+  const int vc = tid >> 3, v = v0 + vc;
+  const bool vok = v < p.vdim;
+  for (int i = tid; i < 2 * kBuf; i += 128) sm[i] = 0.f;        // padding channels stay zero
+
+  float S[RPT];
+  const long long sbase = static_cast<long long>(h) * p.dim * p.vdim + v;
+  const long long per_state = static_cast<long long>(p.heads) * p.dim * p.vdim;
+#pragma unroll
+  for (int j = 0; j < RPT; ++j) {
+    const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
+    S[j] = (sin >= 0 && vok && d < p.dim) ? p.state[sin * per_state + sbase + static_cast<long long>(d) * p.vdim] : 0.f;
+  }
+  __syncthreads();
+  const long long ldk = static_cast<long long>(p.kv_heads) * p.dim, ldg = static_cast<long long>(p.heads) * p.dim,
+                  ldv = static_cast<long long>(p.heads) * p.vdim;
+  auto stage = [&](int t0, int b) {
+    float* base = sm + b * kBuf;
+    const int cnt = min(kScanStep, n - t0);
+    if ((p.dim & 3) == 0) {
+      const int q4 = p.dim >> 2;
+      for (int i = tid; i < cnt * q4; i += 128) {
+        const int t = i / q4, d = (i - t * q4) * 4;
+        const long long r = r0 + t0 + t;
+        cp_async16(base + t * DP + d, p.kn + r * ldk + hk * p.dim + d);
+        cp_async16(base + kScanStep * DP + t * DP + d, p.qn + r * ldk + hk * p.dim + d);
+        cp_async16(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
+      }
+    } else {
+      for (int i = tid; i < cnt * p.dim; i += 128) {
+        const int t = i / p.dim, d = i - t * p.dim;
+        const long long r = r0 + t0 + t;
+        cp_async4(base + t * DP + d, p.kn + r * ldk + hk * p.dim + d);
+        cp_async4(base + kScanStep * DP + t * DP + d, p.qn + r * ldk + hk * p.dim + d);
+        cp_async4(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
+      }
+    }
+    float* vb = base + 3 * kScanStep * DP;
+    for (int i = tid; i < cnt * kScanCols; i += 128) {
+      const int t = i / kScanCols, c = i - t * kScanCols;
+      if (v0 + c < p.vdim) cp_async4(vb + i, p.v + (r0 + t0 + t) * ldv + h * p.vdim + v0 + c);
+    }
+    if (tid < cnt) {
+      cp_async4(vb + kScanStep * kScanCols + tid, p.beta + static_cast<long long>(r0 + t0 + tid) * p.heads + h);
+      cp_async4(vb + kScanStep * kScanCols + kScanStep + tid,
+                p.qk + static_cast<long long>(r0 + t0 + tid) * p.kv_heads + hk);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  stage(0, 0);
+  int b = 0;
+  for (int t0 = 0; t0 < n; t0 += kScanStep, b ^= 1) {
+    if (t0 + kScanStep < n) {
+      stage(t0 + kScanStep, b ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const float* base = sm + b * kBuf;
+    const float* vb = base + 3 * kScanStep * DP;
+    const int cnt = min(kScanStep, n - t0);
+    for (int t = 0; t < cnt; ++t) {
+      float k[RPT];
+      float sk0 = 0.f, sk1 = 0.f, sq0 = 0.f, sq1 = 0.f;
+#pragma unroll
+      for (int c = 0; c < RPT / 4; ++c) {
+        const int off = t * DP + c * 32 + l8 * 4;
+        const float4 k4 = *reinterpret_cast<const float4*>(base + off);
+        const float4 q4 = *reinterpret_cast<const float4*>(base + kScanStep * DP + off);
+        const float4 g4 = *reinterpret_cast<const float4*>(base + 2 * kScanStep * DP + off);
+        k[4 * c] = k4.x; k[4 * c + 1] = k4.y; k[4 * c + 2] = k4.z; k[4 * c + 3] = k4.w;
+        S[4 * c] *= g4.x; S[4 * c + 1] *= g4.y; S[4 * c + 2] *= g4.z; S[4 * c + 3] *= g4.w;
+        sk0 = fmaf(S[4 * c], k4.x, sk0); sk1 = fmaf(S[4 * c + 1], k4.y, sk1);
+        sq0 = fmaf(S[4 * c], q4.x, sq0); sq1 = fmaf(S[4 * c + 1], q4.y, sq1);
+        sk0 = fmaf(S[4 * c + 2], k4.z, sk0); sk1 = fmaf(S[4 * c + 3], k4.w, sk1);
+        sq0 = fmaf(S[4 * c + 2], q4.z, sq0); sq1 = fmaf(S[4 * c + 3], q4.w, sq1);
+      }
+      float sk = sk0 + sk1, sq = sq0 + sq1;
+#pragma unroll
+      for (int o = 1; o < 8; o <<= 1) {
+        sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+      }
+      const float u = vb[kScanStep * kScanCols + t] * (vb[t * kScanCols + vc] - sk);
+      if (l8 == 0 && vok)
+        p.o[(r0 + t0 + t) * ldv + h * p.vdim + v] = fmaf(vb[kScanStep * kScanCols + kScanStep + t], u, sq);
+#pragma unroll
+      for (int j = 0; j < RPT; ++j) S[j] = fmaf(k[j], u, S[j]);
+    }
+    __syncthreads();
+  }
+  if (sout >= 0 && vok) {
+#pragma unroll
+    for (int j = 0; j < RPT; ++j) {
+      const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
+      if (d < p.dim) p.state[sout * per_state + sbase + static_cast<long long>(d) * p.vdim] = S[j];
+    }
+  }
+}
+
+// output norm and gate: one warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(128)
+delta_output_kernel(const DeltaParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long i = static_cast<long long>(blockIdx.x) * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (i >= static_cast<long long>(p.rows) * p.heads) return;
+  const long long r = i / p.heads;
+  const int h = static_cast<int>(i - r * p.heads);
+  const float* o = p.o + i * p.vdim;
+  float ss = 0.f;
+  for (int v = lane; v < p.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
+  ss = warp_sum(ss);
+  const float inv = 1.f / sqrtf(ss / p.vdim + p.eps);
+  const float* g = p.ag + r * p.ldag + p.off_gate + h * p.vdim;
+  for (int v = lane; v < p.vdim; v += 32)
+    act_store(p.out + r * p.ldo + h * p.vdim + v, o[v] * inv * p.norm_w[v] * sigmoid_f(g[v]));
+}
+
+// ---------------------------------------------------------------------------------
+// decode: CTA = (sequence, head), 8 warps; lane l holds the value columns 4l .. 4l + 3, warp w the key channels
+// w, w + 8, ...  Needs vdim <= 128, vdim % 4 == 0, dim <= 8 * RW.
+// ---------------------------------------------------------------------------------
+template <typename T, int RW>
+__global__ void __launch_bounds__(256)
+delta_decode_kernel(const DeltaParams<T> p) {
+  pdl_launch_dependents();
+  __shared__ float s_q[8 * RW], s_k[8 * RW], s_g[8 * RW], s_v[128], s_red[2][8][128];
+  const int seq = blockIdx.x, h = blockIdx.y;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int hk = h / (p.heads / p.kv_heads);
+  // the state binding and the sequence's state precede the running step: their loads go out before the dependency wait
+  int sin, sout;
+  const bool ok = seq_states(p, seq, sin, sout);
+  const long long per_state = static_cast<long long>(p.heads) * p.dim * p.vdim;
+  const int vcol = lane * 4;
+  const bool vok = vcol < p.vdim;
+  float4 S[RW];
+#pragma unroll
+  for (int j = 0; j < RW; ++j) {
+    const int d = warp + 8 * j;
+    S[j] = (ok && sin >= 0 && vok && d < p.dim)
+               ? *reinterpret_cast<const float4*>(p.state + sin * per_state +
+                                                  (static_cast<long long>(h) * p.dim + d) * p.vdim + vcol)
+               : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  if (!ok) return;
+  const int r = p.seq_start[seq];
+  if (r < 0 || r >= p.rows || p.seq_start[seq + 1] != r + 1) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xC03, seq, r);
+    return;
+  }
+  const int nk = p.kv_heads * p.dim, channels = p.channels();
+  const int first = h % (p.heads / p.kv_heads) == 0;         // this CTA also keeps the shared q / k inputs
+  for (int d = tid; d < 8 * RW; d += 256) {
+    float q = 0.f, k = 0.f, g = 0.f;
+    if (d < p.dim) {
+      const int cq = hk * p.dim + d, ck = nk + cq;
+      q = conv_silu(p, cq, r, 0, sin, channels);
+      k = conv_silu(p, ck, r, 0, sin, channels);
+      if (first) {
+        store_tail(p, cq, r, 0, 1, sin, sout, channels);
+        store_tail(p, ck, r, 0, 1, sin, sout, channels);
+      }
+      const int c = h * p.dim + d;
+      g = expf(p.a_neg[h] * softplus_f(p.ag[r * p.ldag + c] + p.dt_bias[c]));
+    }
+    s_q[d] = q;
+    s_k[d] = k;
+    s_g[d] = g;
+  }
+  for (int v = tid; v < 128; v += 256) {
+    float y = 0.f;
+    if (v < p.vdim) {
+      const int c = 2 * nk + h * p.vdim + v;
+      y = conv_silu(p, c, r, 0, sin, channels);
+      store_tail(p, c, r, 0, 1, sin, sout, channels);
+    }
+    s_v[v] = y;
+  }
+  __syncthreads();
+  // norms of q and k, their product: every warp computes them for itself
+  float nq = 0.f, nkk = 0.f, dot = 0.f;
+#pragma unroll
+  for (int d = lane; d < 8 * RW; d += 32) {
+    nq = fmaf(s_q[d], s_q[d], nq);
+    nkk = fmaf(s_k[d], s_k[d], nkk);
+    dot = fmaf(s_q[d], s_k[d], dot);
+  }
+  nq = warp_sum(nq);
+  nkk = warp_sum(nkk);
+  dot = warp_sum(dot);
+  const float fq = 1.f / sqrtf(nq + 1e-6f) / sqrtf(static_cast<float>(p.dim)), fk = 1.f / sqrtf(nkk + 1e-6f);
+  float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
+#pragma unroll
+  for (int j = 0; j < RW; ++j) {
+    const int d = warp + 8 * j;
+    const float g = s_g[d], k = s_k[d] * fk, q = s_q[d] * fq;
+    S[j].x *= g; S[j].y *= g; S[j].z *= g; S[j].w *= g;
+    ak.x = fmaf(S[j].x, k, ak.x); ak.y = fmaf(S[j].y, k, ak.y); ak.z = fmaf(S[j].z, k, ak.z); ak.w = fmaf(S[j].w, k, ak.w);
+    aq.x = fmaf(S[j].x, q, aq.x); aq.y = fmaf(S[j].y, q, aq.y); aq.z = fmaf(S[j].z, q, aq.z); aq.w = fmaf(S[j].w, q, aq.w);
+  }
+  *reinterpret_cast<float4*>(&s_red[0][warp][vcol]) = ak;
+  *reinterpret_cast<float4*>(&s_red[1][warp][vcol]) = aq;
+  __syncthreads();
+  float sk[4] = {}, sq[4] = {};
+#pragma unroll
+  for (int w = 0; w < 8; ++w) {
+    const float4 a = *reinterpret_cast<const float4*>(&s_red[0][w][vcol]);
+    const float4 c = *reinterpret_cast<const float4*>(&s_red[1][w][vcol]);
+    sk[0] += a.x; sk[1] += a.y; sk[2] += a.z; sk[3] += a.w;
+    sq[0] += c.x; sq[1] += c.y; sq[2] += c.z; sq[3] += c.w;
+  }
+  const float beta = sigmoid_f(act_load(p.proj + r * p.ldp + p.off_b + h));
+  const float qk = dot * fq * fk;
+  float u[4], o[4], ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    u[e] = vok ? beta * (s_v[vcol + e] - sk[e]) : 0.f;
+    o[e] = vok ? fmaf(qk, u[e], sq[e]) : 0.f;
+    ss = fmaf(o[e], o[e], ss);
+  }
+  if (sout >= 0 && vok) {
+#pragma unroll
+    for (int j = 0; j < RW; ++j) {
+      const int d = warp + 8 * j;
+      if (d < p.dim) {
+        const float k = s_k[d] * fk;
+        *reinterpret_cast<float4*>(p.state + sout * per_state + (static_cast<long long>(h) * p.dim + d) * p.vdim + vcol) =
+            make_float4(fmaf(k, u[0], S[j].x), fmaf(k, u[1], S[j].y), fmaf(k, u[2], S[j].z), fmaf(k, u[3], S[j].w));
+      }
+    }
+  }
+  if (warp == 0) {
+    ss = warp_sum(ss);
+    const float inv = 1.f / sqrtf(ss / p.vdim + p.eps);
+    if (vok) {
+      const float* g = p.ag + r * p.ldag + p.off_gate + h * p.vdim + vcol;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        act_store(p.out + r * p.ldo + h * p.vdim + vcol + e, o[e] * inv * p.norm_w[vcol + e] * sigmoid_f(g[e]));
+    }
+  }
+}
+
+template <typename T>
+static int fill(const FbDeltaArgs* a, DeltaParams<T>& p) {
+  if (!a || !a->proj || !a->ag || !a->conv || !a->a_neg || !a->dt_bias || !a->norm_w || !a->state || !a->seq_start ||
+      !a->state_in || !a->state_out || !a->out)
+    return FB_ERR_SHAPE;
+  if (a->rows <= 0 || a->n_seqs <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 ||
+      a->vdim <= 0 || a->taps <= 0 || a->n_states <= 0 || (a->taps > 1 && !a->tail))
+    return FB_ERR_SHAPE;
+  if (a->ldo < static_cast<long long>(a->heads) * a->vdim) return FB_ERR_SHAPE;
+  p.proj = static_cast<const T*>(a->proj); p.ldp = a->ldp;
+  p.off_q = a->off_q; p.off_k = a->off_k; p.off_v = a->off_v; p.off_b = a->off_b;
+  p.ag = a->ag; p.ldag = a->ldag; p.off_gate = a->off_gate;
+  p.conv = a->conv; p.a_neg = a->a_neg; p.dt_bias = a->dt_bias; p.norm_w = a->norm_w; p.eps = a->eps;
+  p.state = a->state; p.tail = static_cast<T*>(a->tail); p.n_states = a->n_states;
+  p.row_seq = a->row_seq; p.seq_start = a->seq_start; p.state_in = a->state_in; p.state_out = a->state_out;
+  p.rows = a->rows; p.n_seqs = a->n_seqs; p.heads = a->heads; p.kv_heads = a->kv_heads; p.dim = a->dim; p.vdim = a->vdim;
+  p.taps = a->taps;
+  p.qn = a->qn; p.kn = a->kn; p.v = a->v; p.decay = a->decay; p.beta = a->beta; p.qk = a->qk; p.o = a->o;
+  p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
+  p.status = static_cast<DeviceStatus*>(a->status);
+  return FB_OK;
+}
+
+static int launched() { return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH; }
+
+template <typename T>
+static int run_decode(const FbDeltaArgs* a, cudaStream_t s) {
+  DeltaParams<T> p{};
+  const int rc = fill<T>(a, p);
+  if (rc != FB_OK) return rc;
+  if (p.vdim > 128 || p.vdim % 4 || p.dim > 128 || p.heads > 65535) return FB_ERR_SHAPE;
+  const dim3 grid(p.n_seqs, p.heads);
+  if (p.dim <= 64) launch_pdl(delta_decode_kernel<T, 8>, grid, dim3(256), 0, s, p);
+  else launch_pdl(delta_decode_kernel<T, 16>, grid, dim3(256), 0, s, p);
+  return launched();
+}
+
+template <typename T, int RPT>
+static int launch_scan(const DeltaParams<T>& p, cudaStream_t s) {
+  constexpr int smem = 2 * kScanStep * (3 * RPT * 8 + kScanCols + 2) * static_cast<int>(sizeof(float));
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  const dim3 grid(p.heads * ((p.vdim + kScanCols - 1) / kScanCols), p.n_seqs);
+  launch_pdl(delta_scan_kernel<T, RPT>, grid, dim3(128), smem, s, p);
+  return launched();
+}
+
+template <typename T>
+static int run_prefill(const FbDeltaArgs* a, cudaStream_t s) {
+  DeltaParams<T> p{};
+  int rc = fill<T>(a, p);
+  if (rc != FB_OK) return rc;
+  if (!p.row_seq || !p.qn || !p.kn || !p.v || !p.decay || !p.beta || !p.qk || !p.o) return FB_ERR_SHAPE;
+  if (p.dim > 256 || p.n_seqs > 65535) return FB_ERR_SHAPE;
+  const size_t smem = 2ull * p.kv_heads * p.dim * sizeof(float);
+  if (smem > 200 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(delta_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
+        cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(delta_prepare_kernel<T>, dim3(p.rows), dim3(256), smem, s, p);
+  if ((rc = launched()) != FB_OK) return rc;
+  if (p.dim <= 32) rc = launch_scan<T, 4>(p, s);
+  else if (p.dim <= 64) rc = launch_scan<T, 8>(p, s);
+  else if (p.dim <= 128) rc = launch_scan<T, 16>(p, s);
+  else rc = launch_scan<T, 32>(p, s);
+  if (rc != FB_OK) return rc;
+  const long long items = static_cast<long long>(p.rows) * p.heads;
+  launch_pdl(delta_output_kernel<T>, dim3(static_cast<unsigned>((items + 3) / 4)), dim3(128), 0, s, p);
+  return launched();
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_delta_decode(const FbDeltaArgs* a, void* stream) {
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (!a) return FB_ERR_SHAPE;
+  return a->fp32 ? run_decode<float>(a, s) : run_decode<__nv_bfloat16>(a, s);
+}
+
+extern "C" int fb_delta_prefill(const FbDeltaArgs* a, void* stream) {
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (!a) return FB_ERR_SHAPE;
+  return a->fp32 ? run_prefill<float>(a, s) : run_prefill<__nv_bfloat16>(a, s);
+}

@@ -271,12 +271,12 @@ __device__ __forceinline__ void route_one_token(const float* lr, int warp, int l
       wsum += val;
       if (lane == k) { mine = val; oi[k] = e; }
     }
-    if (lane < topk) ow[lane] = (normalize ? mine / wsum : mine) * route_scale;
+    if (lane < topk) ow[lane] = ((normalize & 1) ? mine / wsum : mine) * route_scale;
     return;
   }
 
-  // group-limited selection (sigmoid family): keep the topk_groups groups with the largest
-  // sum of their two best selection values, mask the rest.
+  // group-limited selection: keep the topk_groups groups with the largest score - the sum of their two best selection
+  // values (sigmoid family), or their best one (normalize bit 1) - and mask the rest.
   if (n_groups > 1 && topk_groups < n_groups) {
     const int per_group = experts / n_groups;
     float gscore_mine = -INFINITY;  // lane g holds group g's score
@@ -297,7 +297,7 @@ __device__ __forceinline__ void route_one_token(const float* lr, int warp, int l
         const float n2 = fmaxf(fminf(b1, o1), fmaxf(b2, o2));
         b1 = n1; b2 = n2;
       }
-      if (lane == g) gscore_mine = b1 + b2;
+      if (lane == g) gscore_mine = (normalize & 2) ? b1 : b1 + b2;
     }
     // pick topk_groups groups (ties -> lower group id)
     uint32_t keep = 0;
@@ -345,7 +345,7 @@ __device__ __forceinline__ void route_one_token(const float* lr, int warp, int l
     wsum += val;
     if (lane == k) { mine = val; oi[k] = idx; }
   }
-  if (lane < topk) ow[lane] = (normalize ? mine / (wsum + 1e-20f) : mine) * route_scale;
+  if (lane < topk) ow[lane] = ((normalize & 1) ? mine / (wsum + 1e-20f) : mine) * route_scale;
 }
 
 __global__ void __launch_bounds__(128)
@@ -1356,7 +1356,7 @@ extern "C" int fb_router_plan_fused(const void* x, long long ldx, const void* w,
                                     void* done_ctr, void* status, void* stream) {
   if (rows <= 0 || experts <= 0 || experts > 256 || topk <= 0 || topk > 32 || topk > experts)
     return FB_ERR_SHAPE;
-  if (hidden % 256 != 0 || hidden > 8192 || (ldx % 8) != 0) return FB_ERR_SHAPE;
+  if (hidden % 8 != 0 || hidden > 8192 || (ldx % 8) != 0) return FB_ERR_SHAPE;
   if (n_groups > 32 || (n_groups > 1 && experts % n_groups != 0)) return FB_ERR_SHAPE;
   if (e_hi <= e_lo || e_hi - e_lo > 256 || ntok <= 0 || !done_ctr) return FB_ERR_SHAPE;
   PlanOut o{src_token, dst_row, row_scale, tile_group, tile_row0, tile_rows, max_tiles, counts, meta};
@@ -1406,7 +1406,7 @@ extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delt
                                   const void* s_src, long long lds, void* xg_q, long long ldxgq, void* xg_s,
                                   long long ldxgs, int s_cols, void* status, void* stream) {
   if (rows <= 0 || experts <= 0 || experts > 256 || topk <= 0 || topk > 32 || topk > experts) return FB_ERR_SHAPE;
-  if (hidden % 256 != 0 || hidden > 8192 || (ldx % 8) != 0 || (ldxg % 8) != 0) return FB_ERR_SHAPE;
+  if (hidden % 8 != 0 || hidden > 8192 || (ldx % 8) != 0 || (ldxg % 8) != 0) return FB_ERR_SHAPE;
   if (slot_rows < rows || e_hi <= e_lo || !cnt || !src_token || !dst_row || !row_scale) return FB_ERR_SHAPE;
   if (q_src == nullptr && !xg) return FB_ERR_SHAPE;
   if (q_src != nullptr && (!s_src || !xg_q || !xg_s || s_cols <= 0 || (ldq % 16) != 0 || (ldxgq % 16) != 0 ||

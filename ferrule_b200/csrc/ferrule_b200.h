@@ -78,6 +78,9 @@ typedef struct FbGemmArgs {
 
 int fb_gemm_bf16(const FbGemmArgs* args, void* stream);
 
+// fp32 tensors, full 32-bit arithmetic (FMA units); same argument block (epilogues 0..2, act_limit 0, no collectives)
+int fb_gemm_f32(const FbGemmArgs* args, void* stream);
+
 // ---- block-scaled FP8 GEMM ---------------------------------------------------------------
 typedef struct FbGemmFp8Args {
   const void* w;            // e4m3 [groups, w_rows_per_group, k]
@@ -149,14 +152,19 @@ typedef struct FbAttnArgs {
   void* trace;              // optional uint64 [32]: globaltimer stamps of CTA (0,0,0) (profiling)
   int decode_only;          // the caller asserts: every sequence has exactly one query row in this launch and its
                             // KV rows below row_pos were written before the running step began (plain decode)
+  const void* gate;         // optional [rows, ldg] (element type of q): head h's output is multiplied by sigmoid(gate[row][h])
+  long long ldg;
 } FbAttnArgs;
 
 int fb_mla_attention(const FbAttnArgs* args, void* stream);
+// the same attention in 32-bit arithmetic on the FMA units (rope_dim 0, kv_lora <= 1024; no splits, sink or selection);
+// fp32: q / kv / gate / out are fp32 instead of bf16
+int fb_latent_attention(const FbAttnArgs* args, int fp32, void* stream);
 
 // ---- prefill attention on tcgen05 (128-row tiles of (position, head) pairs of one sequence) ----
 typedef struct FbPrefillAttnArgs {
-  const void* q;            // bf16 [rows, heads, 576] contiguous (ldq == heads * 576)
-  const void* kv;           // bf16 [pool_rows, 576] (one layer of the pool)
+  const void* q;            // bf16 [rows, heads, 512 + rope_dim] contiguous (ldq == heads * (512 + rope_dim))
+  const void* kv;           // bf16 [pool_rows, 512 + rope_dim] (one layer of the pool)
   void* out;                // bf16 [rows, heads, 512]
   const int* tiles;         // [n_tiles, 4]: sequence, first query row, query rows (<= 128 / heads, consecutive
                             //   positions of that sequence), position of the first row; 16-byte aligned
@@ -170,14 +178,87 @@ typedef struct FbPrefillAttnArgs {
   int rows;
   int heads;                // must divide 128
   int kv_lora;              // 512
-  int rope_dim;             // 64
+  int rope_dim;             // 64, or 0: keys and values are the same 512 features
   int num_seqs;
   int max_blocks;
   int page_size;            // power of two >= 8
   float softmax_scale;
+  const void* gate;         // optional bf16 [rows, ldg]: head h's output is multiplied by sigmoid(gate[row][h])
+  long long ldg;
 } FbPrefillAttnArgs;
 
 int fb_mla_prefill_tc(const FbPrefillAttnArgs* args, void* stream);
+
+// ---- layer-list models: row operators (act tensors bf16, or fp32 with fp32 = 1) ---------------------------
+// x = table[ids] (fp32), h = RMSNorm(x) * norm_w; norm_stride 0: norm_w is one number.  dim_pad: row width rounded up
+// to 8, padding columns are zero
+int fb_embed_norm(const int* ids, const void* table, long long ldt, int vocab, float* x, long long ldx,
+                  const float* norm_w, int norm_stride, void* h, long long ldh, int rows, int dim, int dim_pad, float eps,
+                  int fp32, void* status, void* stream);
+// x += sigmoid(gate1 + bias1) * mix + sigmoid(gate2 + bias2) * sum_{s < topk} ffn[row * slots + s];
+// h = RMSNorm(x) * norm_w.  mix / ffn / gates may be null
+typedef struct FbLayerTailArgs {
+  float* x;
+  long long ldx;
+  const void* mix;
+  long long ldm;
+  const void* gate1;
+  long long ldg1;
+  const float* bias1;
+  const void* ffn;
+  long long ldf;
+  int slots;
+  int topk;
+  const void* gate2;
+  long long ldg2;
+  const float* bias2;
+  const float* norm_w;
+  int norm_stride;
+  int rows;
+  void* h;
+  long long ldh;
+  int dim;
+  int dim_pad;
+  float eps;
+  int fp32;
+} FbLayerTailArgs;
+int fb_gated_residual_norm(const FbLayerTailArgs* args, void* stream);
+// pool[write_slot[r]] = RMSNorm(src[r, :rank]) * norm_w, zero-padded to row_dim
+int fb_latent_append(const void* src, long long lds, int rank, int row_dim, const float* norm_w, float eps,
+                     const long long* write_slot, void* pool, long long pool_rows, int rows, int fp32, void* status,
+                     void* stream);
+int fb_softcap(float* logits, long long ldl, int rows, int vocab, float cap, void* stream);
+int fb_state_rotate(int* state_in, int* state_out, int n, int buffers, void* stream);
+
+// ---- gated delta rule (see delta_rule.cu) ------------------------------------------------------------------
+typedef struct FbDeltaArgs {
+  const void* proj;         // [rows, ldp] projected rows: q | k | v inputs of the convolutions, beta logits
+  long long ldp;
+  int off_q, off_k, off_v, off_b;
+  const float* ag;          // [rows, ldag]: decay pre-activation [heads * dim] at 0, output gate [heads * vdim] at off_gate
+  long long ldag;
+  int off_gate;
+  int fp32;                 // activations (proj, tail, out) are fp32 instead of bf16
+  const float* conv;        // [2 * kv_heads * dim + heads * vdim, taps]
+  const float* a_neg;       // [heads] = -exp(A_log)
+  const float* dt_bias;     // [heads * dim]
+  const float* norm_w;      // [vdim]
+  float* state;             // [n_states, heads, dim, vdim]
+  void* tail;               // [n_states, taps - 1, channels]
+  const int* row_seq;       // [rows] (prefill form)
+  const int* seq_start;     // [n_seqs + 1] first row of every sequence
+  const int* state_in;      // [n_seqs] state index read, -1: zeros
+  const int* state_out;     // [n_seqs] state index written (never the one read), -1: none
+  float *qn, *kn, *v, *decay, *beta, *qk, *o;   // scratch (prefill form): [rows, kv_heads * dim] x 2,
+                            // [rows, heads * vdim], [rows, heads * dim], [rows, heads], [rows, kv_heads], [rows, heads * vdim]
+  void* out;                // [rows, ldo], heads * vdim columns
+  long long ldo;
+  void* status;
+  int n_states, rows, n_seqs, heads, kv_heads, dim, vdim, taps;
+  float eps;
+} FbDeltaArgs;
+int fb_delta_decode(const FbDeltaArgs* args, void* stream);    // one row per sequence; dim, vdim <= 128, vdim % 4 == 0
+int fb_delta_prefill(const FbDeltaArgs* args, void* stream);   // dim <= 256
 
 // ---- small fused operators ------------------------------------------------------------
 int fb_embedding(const int* ids, const void* table, void* out, int rows, int dim, int vocab,
@@ -197,6 +278,8 @@ int fb_mla_prep(const void* q, long long ldq, int q_head_dim, const void* ckv, l
                 const float* sin_t, int max_pos, const int* positions, const long long* write_slot,
                 void* kv_pool, long long pool_rows, void* q_out, long long ldq_out, int rows,
                 void* status, void* stream);
+// `normalize` of the routers: bit 0 = weights sum to one; bit 1 = a group's score is its best selection value instead
+// of the sum of its two best
 int fb_router_topk(const float* logits, long long ldl, const float* bias,
                    const long long* hash_table, const int* token_ids, int rows, int experts,
                    int topk, int score_fn, int n_groups, int topk_groups, int normalize,

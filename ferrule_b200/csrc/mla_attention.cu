@@ -59,6 +59,8 @@ struct AttnParams {
   int prefetch_old;         // one query row per sequence (plain decode step): every KV row below the row's own
                             // position was written by an earlier step, so the first tile may be requested before
                             // the dependency wait
+  const __nv_bfloat16* gate;  // optional [rows, ldg]: head output times sigmoid(gate[row][head])
+  long long ldg;
   unsigned long long* trace;  // optional: CTA (0,0,0) writes globaltimer stamps of its milestones
 };
 
@@ -99,6 +101,11 @@ __device__ __forceinline__ void bulk_copy_g2s_stream(void* dst, const void* src,
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
+}
+
+__device__ __forceinline__ float head_gate(const AttnParams& p, int row, int head) {
+  if (p.gate == nullptr) return 1.f;
+  return 1.f / (1.f + __expf(-__bfloat162float(p.gate[row * p.ldg + head])));
 }
 
 template <int DL, int DR>
@@ -446,7 +453,9 @@ mla_attention_kernel(const AttnParams p) {
       const int lane_base = lane & ~7;
 #pragma unroll
       for (int cc = 0; cc < 8; ++cc) L += __shfl_sync(0xffffffffu, lv * w, lane_base + cc);
-      const float inv = L > 0.f ? 1.f / L : 0.f;
+      float inv = L > 0.f ? 1.f / L : 0.f;
+      const int qr = qrow0 + r / Hb;
+      if (r / Hb < G && qr < p.rows && h < p.heads) inv *= head_gate(p, qr, h);
       wsm[r * 8 + c] = w * inv;
     }
     __syncthreads();
@@ -503,7 +512,7 @@ mla_attention_kernel(const AttnParams p) {
 #pragma unroll
         for (int i = 0; i < kNT; ++i) { o_acc[i][half * 2] *= a; o_acc[i][half * 2 + 1] *= a; }
       }
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      const float inv = (l > 0.f ? 1.f / l : 0.f) * head_gate(p, qr, h);
       __nv_bfloat16* o = p.out + qr * p.ldo + static_cast<long long>(h) * DL + warp * kDimsPerWarp + t4 * 2;
 #pragma unroll
       for (int i = 0; i < kNT; ++i)
@@ -560,7 +569,7 @@ mla_attention_kernel(const AttnParams p) {
         wts[r * p.splits + s2] = w;
         L += l * w;
       }
-      const float inv = L > 0.f ? 1.f / L : 0.f;
+      const float inv = (L > 0.f ? 1.f / L : 0.f) * head_gate(p, qr, h);
       for (int s2 = 0; s2 < p.splits; ++s2) wts[r * p.splits + s2] *= inv;
     }
   }
@@ -685,6 +694,8 @@ extern "C" int fb_mla_attention(const FbAttnArgs* a, void* stream_) {
   const bool cluster_merge = a->splits > 1 && !a->part_o;
   if (cluster_merge && a->splits != 2 && a->splits != 4 && a->splits != 8) return FB_ERR_SHAPE;
   if (a->splits > 1 && !cluster_merge && !a->part_ml) return FB_ERR_SHAPE;
+  // the gate is applied where the softmax sum is divided out: in this kernel, not in the separate merge kernel
+  if (a->gate && ((a->splits > 1 && !cluster_merge && !a->merge_ctr) || a->ldg < a->heads)) return FB_ERR_SHAPE;
   if ((a->ldq % 8) != 0 || (a->ldo % 2) != 0) return FB_ERR_ALIGN;
   if ((reinterpret_cast<uintptr_t>(a->kv) & 15) || (reinterpret_cast<uintptr_t>(a->q) & 15)) return FB_ERR_ALIGN;
   AttnParams p{};
@@ -715,6 +726,8 @@ extern "C" int fb_mla_attention(const FbAttnArgs* a, void* stream_) {
   p.sel_width = a->sel_width;
   p.status = static_cast<DeviceStatus*>(a->status);
   p.trace = static_cast<unsigned long long*>(a->trace);
+  p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+  p.ldg = a->ldg;
   p.prefetch_old = (a->decode_only && a->group_rows == 1 && a->selection == nullptr) ? 1 : 0;
   {
     static const bool enabled = [] {
@@ -730,5 +743,12 @@ extern "C" int fb_mla_attention(const FbAttnArgs* a, void* stream_) {
   // single shared K = V head (DeepSeek-V4): scores and values both span the whole row
   if (a->kv_lora == 512 && a->rope_dim == 0) return launch_attn<512, 0>(p, stream);
   if (a->kv_lora == 64 && a->rope_dim == 0) return launch_attn<64, 0>(p, stream);
+  // latent attention without positions: the cache row is the latent alone, padded to a multiple of 64
+  if (a->kv_lora == 128 && a->rope_dim == 0) return launch_attn<128, 0>(p, stream);
+  if (a->kv_lora == 192 && a->rope_dim == 0) return launch_attn<192, 0>(p, stream);
+  if (a->kv_lora == 256 && a->rope_dim == 0) return launch_attn<256, 0>(p, stream);
+  if (a->kv_lora == 320 && a->rope_dim == 0) return launch_attn<320, 0>(p, stream);
+  if (a->kv_lora == 384 && a->rope_dim == 0) return launch_attn<384, 0>(p, stream);
+  if (a->kv_lora == 448 && a->rope_dim == 0) return launch_attn<448, 0>(p, stream);
   return FB_ERR_SHAPE;
 }

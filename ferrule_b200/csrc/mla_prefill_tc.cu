@@ -7,7 +7,7 @@
 // scores of the tile (QK^T is repeated, PV is split), and they share nothing.
 //
 //   TMA producer (warp 0): the query slab once (9 blocks of 128 rows x 64 features, 128-byte swizzle), then per
-//     64-token KV tile the 9 feature blocks of the pages that hold it (box = 64 features x min(page, 64) rows,
+//     64-token KV tile the 9 (8 without a rotated part) feature blocks of the pages that hold it (box = 64 features x min(page, 64) rows,
 //     straight from the paged pool, zero-filled past the sequence).
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T with both operands K-major from shared memory (36 tcgen05.mma of
 //     K = 16), then O[128 x 256] += P V with P read from TMEM as the A operand and the same shared-memory KV
@@ -42,12 +42,13 @@ namespace fb {
 constexpr int kTcThreads = 192;
 constexpr int kTcM = 128;                 // (position, head) rows per tile
 constexpr int kTcKv = 64;                 // tokens per KV tile
-constexpr int kTcBlocks = 9;              // 64-feature blocks of a 576-wide row (8 latent + 1 rope)
 constexpr int kTcLat = 512;
 constexpr int kTcHalf = 256;              // latent features per CTA
 constexpr int kTcQBlockBytes = kTcM * 128;
 constexpr int kTcKvBlockBytes = kTcKv * 128;
-constexpr int kTcSmem = kTcBlocks * (kTcQBlockBytes + kTcKvBlockBytes) + 1024 /*alignment*/ + 256 /*barriers*/;
+// 64-feature blocks of a cache row: 8 latent, and 1 rope block unless the model has no rotated part
+template <int BLOCKS>
+constexpr int tc_smem() { return BLOCKS * (kTcQBlockBytes + kTcKvBlockBytes) + 1024 /*alignment*/ + 256 /*barriers*/; }
 // TMEM columns: O 0..255, S0 256..319, S1 320..383, P 384..415
 constexpr uint32_t kColO = 0, kColS = 256, kColP = 384, kTmemCols = 512;
 
@@ -67,6 +68,8 @@ struct TcParams {
   int page_size;
   int box_rows;              // min(page_size, 64)
   float scale_log2;
+  const __nv_bfloat16* gate; // optional [rows, ldg]: head output times sigmoid(gate[row][head])
+  long long ldg;
 };
 
 __device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc,
@@ -104,9 +107,12 @@ __device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr, uint32_t
   return d;
 }
 
+template <int BLOCKS>
 __global__ void __launch_bounds__(kTcThreads, 1)
 mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                       const TcParams p) {
+  static_assert(BLOCKS == 8 || BLOCKS == 9, "512 latent features, with or without a rope block");
+  constexpr int kTcBlocks = BLOCKS, kSetA = BLOCKS - 4;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* q_s = smem;
@@ -187,9 +193,9 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         }
         if (j > 0) ok = mbar_wait(kva_free, (j - 1) & 1, abort_flag, p.status, 0xA10);
         if (!ok) break;
-        mbar_arrive_expect_tx(kva_full, 5 * kTcKvBlockBytes);
+        mbar_arrive_expect_tx(kva_full, kSetA * kTcKvBlockBytes);
         for (int s = 0; s < subs; ++s) {
-          for (int i = 0; i < 5; ++i) {
+          for (int i = 0; i < kSetA; ++i) {
             const int b = i < 4 ? a_lo + i : 8;
             tma_load_2d(kv_s + b * kTcKvBlockBytes + s * p.box_rows * 128, &map_kv, kva_full, b * 64, rowc[s]);
           }
@@ -211,7 +217,7 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       constexpr uint32_t idesc_pv = umma_idesc(kTcM, kTcHalf, 1, 1) | (1u << 16);     // B is MN-major
       auto qk_blocks = [&](int j, bool set_b) {
         const uint32_t s_t = tmem + kColS + (j & 1) * kTcKv;
-        const int n = set_b ? 4 : 5;
+        const int n = set_b ? 4 : kSetA;
         for (int i = 0; i < n; ++i) {
           const int b = set_b ? b_lo + i : (i < 4 ? a_lo + i : 8);
 #pragma unroll
@@ -343,7 +349,9 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         // the accumulator is scaled by 2^-m_ref: bring the sink term to the same reference
         l_tot += exp2f(sk - ((m_ref == -INFINITY) ? sk : m_ref));
       }
-      const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+      float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
+      if (p.gate != nullptr && valid)
+        inv /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<long long>(row0 + g) * p.ldg + head]));
       __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + g) * p.ldo + static_cast<long long>(head) * kTcLat +
                            half * kTcHalf;
 #pragma unroll 1
@@ -395,13 +403,13 @@ static TcEncodeFn tc_encoder() {
   return fn;
 }
 
-// bf16 [rows, 576] matrix, box 64 features x box_rows rows, 128-byte swizzle, zeros outside
-static int tc_map(CUtensorMap* map, const void* base, uint64_t rows, uint32_t box_rows) {
+// bf16 [rows, width] matrix, box 64 features x box_rows rows, 128-byte swizzle, zeros outside
+static int tc_map(CUtensorMap* map, const void* base, int width, uint64_t rows, uint32_t box_rows) {
   TcEncodeFn fn = tc_encoder();
   if (!fn) return FB_ERR_DRIVER;
   if (reinterpret_cast<uintptr_t>(base) & 15) return FB_ERR_ALIGN;
-  cuuint64_t dims[2] = {576, rows};
-  cuuint64_t strides[1] = {576 * 2};
+  cuuint64_t dims[2] = {static_cast<cuuint64_t>(width), rows};
+  cuuint64_t strides[1] = {static_cast<cuuint64_t>(width) * 2};
   cuuint32_t box[2] = {64, box_rows};
   cuuint32_t estr[2] = {1, 1};
   CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
@@ -410,26 +418,38 @@ static int tc_map(CUtensorMap* map, const void* base, uint64_t rows, uint32_t bo
   return r == CUDA_SUCCESS ? FB_OK : FB_ERR_DRIVER;
 }
 
+template <int BLOCKS>
+static int launch_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const TcParams& p, cudaStream_t stream) {
+  if (cudaFuncSetAttribute(mla_prefill_tc_kernel<BLOCKS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                           tc_smem<BLOCKS>()) != cudaSuccess)
+    return FB_ERR_LAUNCH;
+  if (launch_pdl(mla_prefill_tc_kernel<BLOCKS>, dim3(p.n_tiles, 2), dim3(kTcThreads), tc_smem<BLOCKS>(), stream, mq, mkv,
+                 p) != cudaSuccess)
+    return FB_ERR_LAUNCH;
+  return FB_OK;
+}
+
 }  // namespace fb
 
 using namespace fb;
 
 extern "C" int fb_mla_prefill_tc(const FbPrefillAttnArgs* a, void* stream_) {
   if (!a || !a->q || !a->kv || !a->out || !a->tiles || !a->block_table) return FB_ERR_SHAPE;
-  if (a->kv_lora != kTcLat || a->rope_dim != 64) return FB_ERR_SHAPE;
+  if (a->kv_lora != kTcLat || (a->rope_dim != 64 && a->rope_dim != 0)) return FB_ERR_SHAPE;
+  const int width = a->kv_lora + a->rope_dim;
   if (a->heads <= 0 || a->heads > kTcM || (kTcM % a->heads) != 0) return FB_ERR_SHAPE;
   if (a->rows <= 0 || a->n_tiles <= 0 || a->num_seqs <= 0 || a->max_blocks <= 0) return FB_ERR_SHAPE;
   if (a->page_size < 8 || (a->page_size & (a->page_size - 1)) != 0) return FB_ERR_SHAPE;
-  if (a->ldq != static_cast<long long>(a->heads) * 576) return FB_ERR_SHAPE;      // (row, head) pairs form one matrix
+  if (a->ldq != static_cast<long long>(a->heads) * width) return FB_ERR_SHAPE;      // (row, head) pairs form one matrix
   if ((a->ldo % 8) != 0 || (reinterpret_cast<uintptr_t>(a->out) & 15)) return FB_ERR_ALIGN;
   if (a->pool_rows <= 0 || a->pool_rows > 0x7fffffffLL || (a->pool_rows % a->page_size) != 0) return FB_ERR_SHAPE;
   if (reinterpret_cast<uintptr_t>(a->tiles) & 15) return FB_ERR_ALIGN;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   const int box_rows = a->page_size < kTcKv ? a->page_size : kTcKv;
   CUtensorMap mq, mkv;
-  int rc = tc_map(&mq, a->q, static_cast<uint64_t>(a->rows) * a->heads, kTcM);
+  int rc = tc_map(&mq, a->q, width, static_cast<uint64_t>(a->rows) * a->heads, kTcM);
   if (rc != FB_OK) return rc;
-  rc = tc_map(&mkv, a->kv, static_cast<uint64_t>(a->pool_rows), box_rows);
+  rc = tc_map(&mkv, a->kv, width, static_cast<uint64_t>(a->pool_rows), box_rows);
   if (rc != FB_OK) return rc;
   TcParams p{};
   p.tiles = a->tiles;
@@ -447,10 +467,8 @@ extern "C" int fb_mla_prefill_tc(const FbPrefillAttnArgs* a, void* stream_) {
   p.page_size = a->page_size;
   p.box_rows = box_rows;
   p.scale_log2 = a->softmax_scale * 1.4426950408889634f;
-  if (cudaFuncSetAttribute(mla_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kTcSmem) != cudaSuccess)
-    return FB_ERR_LAUNCH;
-  if (launch_pdl(mla_prefill_tc_kernel, dim3(a->n_tiles, 2), dim3(kTcThreads), kTcSmem, stream, mq, mkv, p) !=
-      cudaSuccess)
-    return FB_ERR_LAUNCH;
-  return FB_OK;
+  if (a->gate && a->ldg < a->heads) return FB_ERR_SHAPE;
+  p.gate = static_cast<const __nv_bfloat16*>(a->gate);
+  p.ldg = a->ldg;
+  return a->rope_dim ? launch_tc<9>(mq, mkv, p, stream) : launch_tc<8>(mq, mkv, p, stream);
 }

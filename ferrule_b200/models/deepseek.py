@@ -48,6 +48,11 @@ class DeviceBatch:
     tc_tiles: Optional[torch.Tensor] = None     # [cap, 4] int32 tiles of the tensor-core prefill attention kernel
     n_tc_tiles: int = 0
     rest_ranges: Optional[list] = None          # (first row, end row) ranges the tiles do not cover
+    # models with recurrent state (models/state_pool.py)
+    seq_start: Optional[torch.Tensor] = None    # [>= n_seqs + 1] int32 first row of every sequence of the batch
+    state_in: Optional[torch.Tensor] = None     # [>= n_seqs] int32 state index read (-1: a new sequence)
+    state_out: Optional[torch.Tensor] = None    # [>= n_seqs] int32 state index written (-1: none)
+    n_seqs: int = 0
 
 
 class KvPool:

@@ -1,0 +1,406 @@
+"""Forward pass of layer-list models over a packed ragged batch (paged latent pool + recurrent-state pool).
+
+    x = embed[token]                                             (residual stream, fp32)
+    per layer:  h = RMSNorm(x) * g
+                x += sigmoid(rg1 h + b1) * mixer(h) + sigmoid(rg2 h + b2) * ff(h)
+    logits = softcap(head . RMSNorm(x) * g_final)
+
+* `LayeredReference` - plain PyTorch; the execution path of a CPU runner.
+* `LayeredCuda`      - the sm_100a kernel pipeline, allocation-free over a preallocated workspace, so a decode step can be
+  captured in a CUDA graph.  With fp32 weights the same pipeline runs in full 32 bits.
+
+Kernels of a latent layer: input projection (one GEMM for q, latent, gates) -> latent append -> W_uk absorption ->
+attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o.  Of a delta layer: input projection -> second
+low-rank halves -> delta rule -> W_o.  The feed-forward branch reads the same h and runs on a second stream beside
+the mixer: router (+ row reservation) -> grouped SwiGLU GEMM -> grouped scatter GEMM.  One kernel joins both branches:
+gated residual additions, expert reduction, next layer's norm.
+"""
+from __future__ import annotations
+
+from typing import Dict, Optional
+
+import torch
+
+from ..ops import reference as ref
+from .config import SCORE_SOFTMAX
+from .deepseek import DeviceBatch, KvPool, _pow2_at_least
+from .layered_config import LatentMixer, pad_to
+from .layered_weights import LayerImage, LayeredWeights, MixerImage
+from .state_pool import RecurrentStatePool
+
+
+# ======================================================================================
+# reference forward (PyTorch)
+# ======================================================================================
+class LayeredReference:
+    def __init__(self, weights: LayeredWeights, pool: KvPool, states: RecurrentStatePool):
+        self.w, self.cfg, self.pool, self.states = weights, weights.cfg, pool, states
+        self.latent_index = {l: i for i, l in enumerate(self.cfg.latent_layers)}
+        self.prof = self.tap = None
+
+    def _norm(self, x: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
+        W = self.cfg.width
+        inv = torch.rsqrt(x[:, :W].pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps)
+        return x * inv * g
+
+    def _latent(self, layer: int, mx: MixerImage, m: LatentMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        T, DL = proj.shape[0], self.cfg.kv_row_dim
+        o = mx.off
+        dp, vp = pad_to(m.dim, 8), pad_to(m.vdim, 8)
+        q = proj[:, o["q"]:o["q"] + m.heads * dp].view(T, m.heads, dp)
+        c = proj[:, o["dkv"]:o["dkv"] + m.kv_rank]
+        c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps) * mx.kv_norm[:m.kv_rank]
+        pool = self.pool.layer(self.latent_index[layer]).view(-1, DL)
+        slots = b.write_slot[:T]
+        ok = slots >= 0
+        pool[slots[ok], :m.kv_rank] = c[ok].to(pool.dtype)
+        pool[slots[ok], m.kv_rank:] = 0
+        q_lat = torch.einsum("thk,hnk->thn", q, mx.w_uk_t.float())
+        lat = ref.mla_paged_attention(q_lat, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, DL,
+                                      m.scale)
+        v = torch.einsum("thn,hvn->thv", lat, mx.w_uv.float())
+        gate = torch.sigmoid(proj[:, o["g"]:o["g"] + m.heads])
+        return (v * gate[:, :, None]).reshape(T, m.heads * vp) @ mx.w_o.float().T
+
+    def _delta(self, layer: int, mx: MixerImage, m, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        T, o = proj.shape[0], mx.off
+        H, KV, D, V = m.heads, m.kv_heads, m.dim, m.vdim
+        nk, nv, keep = KV * D, H * V, m.taps - 1
+        low = proj[:, o["a1"]:o["a1"] + mx.w_ag.shape[1]]
+        ag = low @ mx.w_ag.float().T
+        raw = torch.cat([proj[:, o["q"]:o["q"] + nk], proj[:, o["k"]:o["k"] + nk], proj[:, o["v"]:o["v"] + nv]], 1)
+        decay = torch.exp(mx.a_neg[:, None] * torch.nn.functional.softplus(ag[:, :H * D] + mx.dt_bias).view(T, H, D))
+        beta = torch.sigmoid(proj[:, o["b"]:o["b"] + H])
+        state, tail = self.states.state[layer], self.states.tail[layer]
+        out = torch.zeros(T, mx.w_o.shape[1])
+        for s in range(b.n_seqs):
+            r0, r1 = int(b.seq_start[s]), int(b.seq_start[s + 1])
+            sin, sout = int(b.state_in[s]), int(b.state_out[s])
+            old = tail[sin, :keep].float() if (sin >= 0 and keep) else torch.zeros(keep, m.channels)
+            S = state[sin].clone() if sin >= 0 else torch.zeros(H, D, V)
+            x = torch.cat([old, raw[r0:r1]], 0)
+            n = r1 - r0
+            y = sum(x[j:j + n] * mx.conv[:, j] for j in range(m.taps))
+            y = torch.nn.functional.silu(y)
+            q, k, v = y[:, :nk].view(n, KV, D), y[:, nk:2 * nk].view(n, KV, D), y[:, 2 * nk:].view(n, H, V)
+            unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+            q = (unit(q) * D ** -0.5).repeat_interleave(H // KV, 1)
+            k = unit(k).repeat_interleave(H // KV, 1)
+            for i in range(n):
+                S = S * decay[r0 + i][:, :, None]
+                u = beta[r0 + i][:, None] * (v[i] - torch.einsum("hdv,hd->hv", S, k[i]))
+                S = S + k[i][:, :, None] * u[:, None, :]
+                oi = torch.einsum("hdv,hd->hv", S, q[i])
+                oi = oi * torch.rsqrt(oi.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps) * mx.o_norm
+                out[r0 + i, :nv] = (oi * torch.sigmoid(ag[r0 + i, mx.off_gate:].view(H, V))).reshape(-1)
+            if sout >= 0:
+                state[sout] = S
+                if keep:
+                    tail[sout, :keep] = x[-keep:].to(tail.dtype)
+        return out @ mx.w_o.float().T
+
+    def _moe(self, lw: LayerImage, h: torch.Tensor) -> torch.Tensor:
+        s = lw.spec.mlp
+        idx, wts = ref.route(h @ lw.router_w.float().T, s.top, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep,
+                             group_top=1)
+        out = torch.zeros_like(h)
+        fp = lw.e_w2.shape[2]
+        for e in range(s.experts):
+            hit = idx == e
+            rows = hit.any(-1).nonzero().flatten()
+            if rows.numel() == 0:
+                continue
+            y = h[rows] @ lw.e_w13[e].float().T
+            y = (torch.nn.functional.silu(y[:, :fp]) * y[:, fp:]) @ lw.e_w2[e].float().T
+            out[rows] += y * (wts * hit)[rows].sum(-1, keepdim=True)
+        return out
+
+    def hidden_states(self, b: DeviceBatch, allreduce=None, start_layer: int = 0, h0=None) -> torch.Tensor:
+        """Residual stream after the last layer [rows, width_pad]."""
+        Wp = self.cfg.width_pad
+        x = self.w.embed[b.token_ids[:b.n_rows].long()].float()
+        for i, lw in enumerate(self.w.layers):
+            if self.prof is not None:
+                self.prof.mark(i, "layer")
+            mx = lw.mixer
+            h = self._norm(x, lw.norm)
+            proj = h @ mx.w_in.float().T
+            m = lw.spec.mixer
+            y = (self._latent if isinstance(m, LatentMixer) else self._delta)(i, mx, m, proj, b)
+            y = y * torch.sigmoid(proj[:, mx.off["rg1"]:mx.off["rg1"] + Wp] + lw.rg1_b)
+            if lw.spec.mlp is not None:
+                y = y + self._moe(lw, h) * torch.sigmoid(proj[:, mx.off["rg2"]:mx.off["rg2"] + Wp] + lw.rg2_b)
+            x = x + y
+            if self.tap is not None:
+                self.tap.write(i, "layer_out", x)
+        return x
+
+    def logits_from_hidden(self, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        logits = self._norm(x[b.logit_rows[:b.n_logit].long()], self.w.final_norm) @ self.w.lm_head.float().T
+        cap = self.cfg.logit_softcap
+        return cap * torch.tanh(logits / cap) if cap else logits
+
+
+# ======================================================================================
+# CUDA forward (sm_100a kernels)
+# ======================================================================================
+class LayeredWorkspace:
+    """Preallocated activations for up to `max_rows` packed rows."""
+
+    def __init__(self, w: LayeredWeights, max_rows: int, max_logit_rows: int, device):
+        from ..ops import layered as KL
+        from ..ops.kernels import ArgmaxScratch, MoePlan, static_plan
+        cfg = w.cfg
+        dt = w.embed.dtype
+        act = dict(dtype=dt, device=device)
+        f32 = dict(dtype=torch.float32, device=device)
+        i32 = dict(dtype=torch.int32, device=device)
+        R, Wp, DL = max_rows, cfg.width_pad, cfg.kv_row_dim
+        self.max_rows, self.max_logit_rows = R, max_logit_rows
+        self.x = torch.zeros(R, Wp, **f32)
+        self.h = torch.zeros(R, Wp, **act)
+        self.proj = torch.zeros(R * max(l.mixer.w_in.shape[0] for l in w.layers), **act)
+        self.mix_in = torch.zeros(R * max(l.mixer.w_o.shape[1] for l in w.layers), **act)
+        self.mix = torch.zeros(R, Wp, **act)
+        latent = [cfg.layers[i].mixer for i in cfg.latent_layers]
+        delta = [cfg.layers[i].mixer for i in cfg.delta_layers]
+        if latent:
+            n = max(m.heads for m in latent) * DL
+            self.q_lat = torch.zeros(R * n, **act)
+            self.o_lat = torch.zeros(R * n, **act)
+        if delta:
+            self.ag = torch.zeros(R * max(w.layers[i].mixer.w_ag.shape[0] for i in cfg.delta_layers), **f32)
+            self.delta = KL.DeltaScratch(R, delta, device)
+        moes = [(i, l.mlp) for i, l in enumerate(cfg.layers) if l.mlp is not None]
+        self.plans: Dict[tuple, MoePlan] = {}
+        self.static_plans: Dict[tuple, MoePlan] = {}
+        self.static_rows = (16, 32, 64)
+        if moes:
+            kmax, emax = max(s.top for _, s in moes), max(s.experts for _, s in moes)
+            self.router_logits = torch.zeros(R * emax, **f32)
+            self.topk_idx = torch.zeros(R * kmax, **i32)
+            self.topk_w = torch.zeros(R * kmax, **f32)
+            xrows = max(R * kmax, emax * self.static_rows[-1])
+            self.xg = torch.zeros(xrows, Wp, **act)
+            self.hmid = torch.zeros(xrows * max(l.e_w2.shape[2] for l in w.layers if l.e_w2 is not None), **act)
+            self.route_out = torch.zeros(R * kmax, Wp, **act)
+            self.route_cnt = torch.zeros(cfg.n_layers, emax, **i32)
+            for E, k in sorted({(s.experts, s.top) for _, s in moes}):
+                for ntok in (16, 32, 64, 128):
+                    self.plans[E, k, ntok] = MoePlan.allocate(R * k, E, ntok, device)
+                self.plans[E, k, 256] = None                        # tile table of the scatter GEMM, built on first use
+            base: Dict[tuple, MoePlan] = {}
+            for i, s in moes:
+                for nt in self.static_rows:
+                    p = static_plan(nt, s.experts, self.route_cnt[i][:s.experts], base.get((s.experts, nt)))
+                    base.setdefault((s.experts, nt), p)
+                    self.static_plans[i, nt] = p
+        L = max_logit_rows
+        self.hn_last = torch.zeros(L, Wp, **act)
+        self.logits = torch.zeros(L, cfg.vocab_size, **f32)
+        self.out_buf = torch.zeros(2 * L, **i32)          # greedy result: [ids | fp32 value bits]
+        self.next_id = self.out_buf[:L]
+        self.next_val = self.out_buf[L:].view(torch.float32)
+        self.argmax_scratch = ArgmaxScratch.allocate(max(L, 1), device)
+
+
+class LayeredCuda:
+    def __init__(self, weights: LayeredWeights, pool: KvPool, states: RecurrentStatePool, max_rows: int = 4096,
+                 max_logit_rows: int = 256, decode_rows: int = 64, max_seq_len: int = 4096, attn_splits: int = 8):
+        from ..ops import kernels as K
+        from ..ops import layered as KL
+        from ..ops import movers as M
+        self.K, self.KL, self.M = K, KL, M
+        self.w, self.cfg, self.pool, self.states = weights, weights.cfg, pool, states
+        self.device = weights.embed.device
+        self.fp32 = weights.embed.dtype == torch.float32
+        self.decode_rows = decode_rows
+        self.attn_splits = attn_splits
+        self.split_tokens = max(64, pad_to((max_seq_len + attn_splits - 1) // attn_splits, 64))
+        self.ws = LayeredWorkspace(weights, max_rows, max_logit_rows, self.device)
+        self.latent_index = {l: i for i, l in enumerate(self.cfg.latent_layers)}
+        # the tensor-core attention kernels take latents up to 512 features
+        self.mma_attention = not self.fp32 and self.cfg.kv_row_dim <= 512
+        self.static_moe = not self.fp32 and self.cfg.width_pad <= 8192
+        self.side_stream = torch.cuda.Stream(device=self.device)      # the feed-forward runs beside the mixer
+        self.launches = 0
+        self.last_hidden = None
+        self.prof = self.tap = None
+        for i in self.cfg.delta_layers:
+            if self.cfg.layers[i].mixer.dim > 256:
+                raise ValueError("delta mixers wider than 256 key channels per head are not supported")
+        for l in self.cfg.layers:
+            if l.mlp is not None and (l.mlp.experts > 256 or l.mlp.top > 32 or l.mlp.groups > 32):
+                raise ValueError("the router takes at most 256 experts, top 32, 32 groups")
+
+    @staticmethod
+    def _view(buf: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
+        return buf[:rows * cols].view(rows, cols)
+
+    # -- mixers ---------------------------------------------------------------------------
+    def _latent(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+        mx, m = lw.mixer, lw.spec.mixer
+        DL, dp, vp = cfg.kv_row_dim, pad_to(m.dim, 8), pad_to(m.vdim, 8)
+        pool = self.pool.layer(self.latent_index[layer])
+        KL.latent_append(proj[:, mx.off["dkv"]:], m.kv_rank, mx.kv_norm, cfg.norm_eps, b.write_slot[:T], pool)
+        q = proj[:, mx.off["q"]:mx.off["q"] + m.heads * dp]
+        q_lat = self._view(ws.q_lat, T, m.heads * DL)
+        K.gemm(q, mx.w_uk_t, out=q_lat, x_group_koff=dp, out_group_coff=DL, k=dp)
+        o_lat = self._view(ws.o_lat, T, m.heads * DL)
+        q3, o3 = q_lat.view(T, m.heads, DL), o_lat.view(T, m.heads, DL)
+        gate = proj[:, mx.off["g"]:]
+        if not self.mma_attention:
+            KL.latent_attention(q3, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, m.scale, o3,
+                                gate=gate)
+        else:
+            ranges = [(0, T)]
+            if b.n_tc_tiles:
+                # sequences with many rows: 128-row tiles on tcgen05; the other rows keep the row-tile kernel
+                K.mla_prefill_tc(q3, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, self.pool.page_size, DL, 0, m.scale,
+                                 o3, gate=gate)
+                ranges = b.rest_ranges
+            for r0, r1 in ranges:
+                split = self.attn_splits > 1 and r1 - r0 <= 4 * self.decode_rows
+                K.mla_attention(q3[r0:r1], pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], self.pool.page_size, DL,
+                                0, m.scale, o3[r0:r1], splits=self.attn_splits if split else 1,
+                                split_tokens=self.split_tokens if split else (1 << 30) // 64 * 64,
+                                decode_only=b.decode_only, gate=gate[r0:r1])
+        out = self._view(ws.mix_in, T, m.heads * vp)
+        K.gemm(o_lat, mx.w_uv, out=out, x_group_koff=DL, out_group_coff=vp)
+        return out
+
+    def _delta(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        K, KL, ws = self.K, self.KL, self.ws
+        mx, m = lw.mixer, lw.spec.mixer
+        ag = self._view(ws.ag, T, mx.w_ag.shape[0])
+        a0 = mx.off["a1"]
+        K.gemm(proj[:, a0:a0 + mx.w_ag.shape[1]], mx.w_ag, out=ag)
+        out = self._view(ws.mix_in, T, mx.w_o.shape[1])
+        decode = b.n_seqs == T and KL.delta_decode_supported(m)
+        KL.delta_rule(proj, mx.off, ag, mx, m, self.cfg.norm_eps, self.states.state[layer], self.states.tail[layer],
+                      b.seq_start, b.state_in, b.state_out, b.n_seqs, out, row_seq=b.row_seq[:T], scratch=ws.delta,
+                      decode=decode)
+        return out
+
+    # -- feed-forward ------------------------------------------------------------------------
+    def _moe(self, layer: int, lw: LayerImage, h: torch.Tensor, T: int) -> torch.Tensor:
+        """Routed experts -> [T, top, width_pad] weighted expert rows."""
+        K, ws, s = self.K, self.ws, lw.spec.mlp
+        k, E, Wp = s.top, s.experts, self.cfg.width_pad
+        fp = lw.e_w2.shape[2]
+        idx, wts = self._view(ws.topk_idx, T, k), self._view(ws.topk_w, T, k)
+        route_out = ws.route_out[:T * k]
+        static = next((nt for nt in ws.static_rows if T <= nt), 0) if self.static_moe else 0
+        if static:
+            plan = ws.static_plans[layer, static]
+            K.router_append(h, lw.router_w, k, SCORE_SOFTMAX, plan, 0, E, idx, wts, ws.xg, n_groups=s.groups,
+                            topk_groups=s.keep, group_top=1, dst_slots=k)
+            rows = plan.cap_rows
+            scatter_plan = plan
+        else:
+            logits = self._view(ws.router_logits, T, E)
+            K.gemm(h, lw.router_w, out=logits, ntok=32 if (T >= 1024 and not self.fp32) else None)
+            K.router_topk(logits, k, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep, group_top=1, out_idx=idx,
+                          out_w=wts)
+            ntok = _pow2_at_least(2 * T * k / E, 16, 128)
+            plan = ws.plans[E, k, ntok]
+            K.moe_plan(idx, wts, plan, 0, E, dst_slots=k)
+            rows = T * k
+            if self.fp32:       # a row copy: two bf16 elements per fp32 element
+                K.gather_rows(h.view(torch.bfloat16), plan, ws.xg.view(torch.bfloat16), cap_rows=rows)
+            else:
+                K.gather_rows(h, plan, ws.xg, cap_rows=rows)
+            scatter_plan = plan
+            if not self.fp32 and ntok == 128 and rows >= 160 * E:
+                # prefill-sized expert loads: the scatter GEMM keeps one accumulator and takes 256-row tiles
+                scatter_plan = ws.plans[E, k, 256] = K.moe_retile(plan, 256, ws.plans[E, k, 256])
+        hmid = self._view(ws.hmid, rows, fp)
+        K.gemm(ws.xg[:rows], lw.e_w13, out=hmid, epilogue=K.EPI_SWIGLU, plan=plan)
+        K.gemm(hmid, lw.e_w2, out=route_out, epilogue=K.EPI_SCATTER, plan=scatter_plan, scatter_rows=T * k)
+        return route_out.view(T, k, Wp)
+
+    # -- whole model ---------------------------------------------------------------------
+    def hidden_states(self, b: DeviceBatch, T: int) -> torch.Tensor:
+        """Runs the layers; returns the normalised rows the head reads (`ws.h`); `ws.x` holds the residual stream."""
+        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+        layers = self.w.layers
+        x, h = ws.x[:T], ws.h[:T]
+        if self.static_moe and T <= ws.static_rows[-1] and ws.static_plans:
+            self.M.fill_(ws.route_cnt, 0)
+        KL.embed_norm(b.token_ids[:T], self.w.embed, x, layers[0].norm, h, cfg.width, cfg.norm_eps)
+        prof = self.prof
+        for i, lw in enumerate(layers):
+            mx = lw.mixer
+            ffn = None
+            if lw.spec.mlp is not None:
+                main = torch.cuda.current_stream()
+                self.side_stream.wait_stream(main)
+                with torch.cuda.stream(self.side_stream):
+                    ffn = self._moe(i, lw, h, T)
+            if prof is not None:
+                prof.mark(i, "proj")
+            proj = self._view(ws.proj, T, mx.w_in.shape[0])
+            K.gemm(h, mx.w_in, out=proj)
+            if prof is not None:
+                prof.mark(i, "mixer")
+            mixer = self._latent if isinstance(lw.spec.mixer, LatentMixer) else self._delta
+            a = mixer(i, lw, proj, b, T)
+            if prof is not None:
+                prof.mark(i, "mixer.out")
+            K.gemm(a, mx.w_o, out=ws.mix[:T])
+            if ffn is not None:
+                torch.cuda.current_stream().wait_stream(self.side_stream)
+            if prof is not None:
+                prof.mark(i, "tail")
+            nxt = layers[i + 1].norm if i + 1 < len(layers) else self.w.final_norm
+            KL.gated_residual_norm(
+                x, nxt, h, cfg.width, cfg.norm_eps, mix=ws.mix[:T], gate1=proj[:, mx.off["rg1"]:], bias1=lw.rg1_b,
+                ffn=ffn, topk=lw.spec.mlp.top if ffn is not None else 0,
+                gate2=proj[:, mx.off["rg2"]:] if ffn is not None else None, bias2=lw.rg2_b)
+            if self.tap is not None and self.tap.wants(i, "layer_out"):
+                self.tap.write(i, "layer_out", x)
+        if prof is not None:
+            prof.mark(len(layers), None)
+        return h
+
+    def head(self, h: torch.Tensor, logit_rows: torch.Tensor, L: int):
+        """Logits and greedy tokens of `L` rows -> (next_id, next_val, logits), views of the workspace."""
+        K, ws = self.K, self.ws
+        hn = ws.hn_last[:L]
+        self.M.gather_rows(h, logit_rows[:L], hn)
+        logits = ws.logits[:L]
+        K.gemm(hn, self.w.lm_head, out=logits)
+        if self.cfg.logit_softcap:
+            self.KL.softcap_(logits, self.cfg.logit_softcap)
+        K.argmax_chunked(logits, ws.argmax_scratch, ws.next_id[:L], ws.next_val[:L])
+        return ws.next_id[:L], ws.next_val[:L], logits
+
+    def forward(self, b: DeviceBatch, want_logits: bool = False, start_layer: int = 0, h0=None):
+        """Runs the batch; returns (next_id [n_logit] int32, next_val, logits or None)."""
+        T = b.token_ids.shape[0]
+        assert T <= self.ws.max_rows and b.n_logit <= self.ws.max_logit_rows and start_layer == 0 and h0 is None
+        from ..ops import _lib
+        start = _lib.LAUNCHES[0]
+        h = self.hidden_states(b, T)
+        self.last_hidden = h
+        out = (None, None, None)
+        if b.n_logit:
+            ids, vals, logits = self.head(h, b.logit_rows, b.n_logit)
+            out = (ids, vals, logits if want_logits else None)
+        self.launches = _lib.LAUNCHES[0] - start
+        return out
+
+    def forward_rows(self, b: DeviceBatch, consume) -> None:
+        """Runs the batch and hands the logits of the wanted rows to `consume(first, logits)`, in pieces of at most
+        `max_logit_rows` rows."""
+        T = b.token_ids.shape[0]
+        assert T <= self.ws.max_rows
+        from ..ops import _lib
+        start = _lib.LAUNCHES[0]
+        h = self.hidden_states(b, T)
+        self.last_hidden = h
+        for lo in range(0, b.n_logit, self.ws.max_logit_rows):
+            n = min(self.ws.max_logit_rows, b.n_logit - lo)
+            consume(lo, self.head(h, b.logit_rows[lo:], n)[2])
+        self.launches = _lib.LAUNCHES[0] - start

@@ -40,15 +40,23 @@ class BatchStaging:
     tensor-core prefill attention kernel (128 / tc_heads positions x all heads); the other rows - decode rows,
     verification rows, short chunk tails - stay with the row-tile kernel, whose split boundaries make a
     verification row bit-equal to the decode row of the same position.
+
+    state_slots: models with recurrent state - the buffer also carries the first row of every sequence and the state
+    indices its step reads and writes (seq_start seqs + 1 | state_in seqs | state_out seqs); the runner fills the latter
+    two from its state pool (`fill_states`).
     """
 
-    def __init__(self, rows: int, seqs: int, max_blocks: int, device, tc_heads: int = 0, tc_min_rows: int = 16):
+    def __init__(self, rows: int, seqs: int, max_blocks: int, device, tc_heads: int = 0, tc_min_rows: int = 16,
+                 state_slots: bool = False):
         self.rows, self.seqs, self.max_blocks = rows, seqs, max_blocks
         R = rows
         self.tc_heads, self.tc_min_rows = tc_heads, tc_min_rows
         self.tile_cap = (R // (128 // tc_heads) + seqs + 1) if tc_heads else 0
         self.tile_off = (7 * R + seqs * max_blocks + 3) // 4 * 4          # 16-byte aligned
-        self.words = self.tile_off + 4 * self.tile_cap
+        self.state_slots = state_slots
+        self.state_off = self.tile_off + 4 * self.tile_cap
+        self.words = self.state_off + (3 * seqs + 1 if state_slots else 0)
+        self.n_seqs = 0
         self.n_tiles, self.rest_ranges = 0, None
         cuda = torch.device(device).type == "cuda"
         self.host = torch.zeros(self.words, dtype=torch.int32)
@@ -69,6 +77,16 @@ class BatchStaging:
         self.d_tiles = d[self.tile_off:self.tile_off + 4 * self.tile_cap].view(self.tile_cap, 4)
         self.cuda = cuda
         self._arange = np.arange(R, dtype=np.int32)
+        if state_slots:
+            a = self.state_off
+            parts = ((a, a + seqs + 1), (a + seqs + 1, a + 2 * seqs + 1), (a + 2 * seqs + 1, a + 3 * seqs + 1))
+            self.np_start, self.np_state_in, self.np_state_out = (self.np[lo:hi] for lo, hi in parts)
+            self.d_start, self.d_state_in, self.d_state_out = (d[lo:hi] for lo, hi in parts)
+            # until a batch is filled in: one row per sequence, no state read or kept
+            self.np_start[:] = np.arange(seqs + 1)
+            self.np_state_in[:] = -1
+            self.np_state_out[:] = -1
+            self.n_seqs = seqs
 
     def fill(self, b: ExecutionBatch, pad_rows: int = 0):
         T = b.rows
@@ -86,7 +104,7 @@ class BatchStaging:
             self.np_slot[T:R] = -1
             self.np_seq[T:R] = 0
         seqs = b.sequences
-        n = len(seqs)
+        n = self.n_seqs = len(seqs)
         L = seqs[0].block_len
         if (n == T and L <= self.max_blocks and len(b.block_ids) == n * L
                 and all(s.block_len == L and s.block_start == i * L for i, s in enumerate(seqs))):
@@ -112,6 +130,14 @@ class BatchStaging:
                 self.n_tiles, self.rest_ranges = len(tiles), rest
         return T, R, lrows
 
+    def fill_states(self, bindings) -> None:
+        """(state read, state written) of every sequence of the batch just filled in, and its first rows."""
+        n = self.n_seqs
+        self.np_state_in[:n] = [r for r, _, _ in bindings]
+        self.np_state_out[:n] = [w for _, w, _ in bindings]
+        self.np_start[0] = 0
+        np.cumsum([rows for _, _, rows in bindings], out=self.np_start[1:n + 1])
+
     def upload(self) -> int:
         if self.cuda:
             self.dev.copy_(self.host, non_blocking=True)
@@ -122,6 +148,8 @@ class BatchStaging:
                          self.d_bt, self.d_lrows, R, n_logit)
         if self.n_tiles:
             db.tc_tiles, db.n_tc_tiles, db.rest_ranges = self.d_tiles, self.n_tiles, self.rest_ranges
+        if self.state_slots:
+            db.seq_start, db.state_in, db.state_out, db.n_seqs = self.d_start, self.d_state_in, self.d_state_out, self.n_seqs
         return db
 
 
@@ -163,8 +191,7 @@ class DeepSeekRunner(ModelRunner):
         self.vocab_size, self.eos_token_id = self.cfg.vocab_size, self.cfg.eos_token_id
         self.page_size, self.max_rows, self.max_seqs, self.max_seq_len = page_size, max_rows, max_seqs, max_seq_len
         self.max_blocks = (max_seq_len + page_size - 1) // page_size
-        self.pool = KvPool(self.cfg, n_pages, page_size, self.device,
-                           dtype=torch.bfloat16 if self.is_cuda else weights.embed.dtype)
+        self.pool = self._make_pool(n_pages)
         self.tp = tp
         # pipeline parallelism (parallel.pp.PipelineParallel): `weights` is this stage's share; every step runs
         # through all stages, the last one's greedy tokens are broadcast, so all ranks' engines stay in step
@@ -197,17 +224,11 @@ class DeepSeekRunner(ModelRunner):
             use_graphs = False
         self.use_graphs = use_graphs and self.is_cuda
         self.stats = RunnerStats()
-        tc_heads = 0
-        if self.is_cuda and pp is None and os.environ.get("FERRULE_PREFILL_TC", "1") != "0":
-            from ..ops.kernels import prefill_tc_supported
-            if prefill_tc_supported(weights.heads_local, self.cfg.kv_lora_rank, self.cfg.qk_rope_dim, page_size):
-                tc_heads = weights.heads_local
-        self.staging = BatchStaging(max_rows, max_seqs, self.max_blocks, self.device, tc_heads=tc_heads)
+        self.staging = self._make_staging(max_rows, max_seqs, prefill=True)
+        # a verification batch asks for logits on the anchor and on every draft row of each sequence
+        self.fwd = self._make_forward(max(max_seqs, 1) * (1 + (max_draft if weights.mtp and enable_mtp else 0)), attn_splits,
+                                      emulate_bf16)
         if self.is_cuda:
-            # a verification batch asks for logits on the anchor and on every draft row of each sequence
-            logit_rows = max(max_seqs, 1) * (1 + (max_draft if weights.mtp and enable_mtp else 0))
-            self.fwd = CudaForward(weights, self.pool, max_rows=max_rows, max_logit_rows=logit_rows,
-                                   decode_rows=max_seqs, max_seq_len=max_seq_len, attn_splits=attn_splits, tp=tp)
             self.fwd.arena = self.arena
             if self.arena is not None:
                 from ..utils.telemetry import ExpertTelemetry
@@ -216,8 +237,6 @@ class DeepSeekRunner(ModelRunner):
                 self.telemetry = self.fwd.telemetry
             L = self.fwd.ws.max_logit_rows
             self.out_host = torch.zeros(2 * L, dtype=torch.int32).pin_memory()
-        else:
-            self.fwd = ReferenceForward(weights, self.pool, emulate_bf16=emulate_bf16)
         self.graphs: Dict[int, tuple] = {}
         # captured decode graphs and their staging, one per row count (exact-key reuse, build on first use)
         from ..runtime.arena import PersistentArenaPool
@@ -267,6 +286,31 @@ class DeepSeekRunner(ModelRunner):
         # candidates does not pay for the observations (tens of microseconds per streamed layer pass)
         self.predictor = None
 
+    # ------------------------------------------------------------------ parts another model family replaces
+    def _make_pool(self, n_pages: int) -> KvPool:
+        return KvPool(self.cfg, n_pages, self.page_size, self.device,
+                      dtype=torch.bfloat16 if self.is_cuda else self.w.embed.dtype)
+
+    def _prefill_tc_heads(self) -> int:
+        """Heads per tile row block of the tensor-core prefill attention kernel, 0 when it does not serve the model."""
+        from ..ops.kernels import prefill_tc_supported
+        ok = prefill_tc_supported(self.w.heads_local, self.cfg.kv_lora_rank, self.cfg.qk_rope_dim, self.page_size)
+        return self.w.heads_local if ok else 0
+
+    def _make_staging(self, rows: int, seqs: int, prefill: bool = False) -> BatchStaging:
+        tc = prefill and self.is_cuda and self.pp is None and os.environ.get("FERRULE_PREFILL_TC", "1") != "0"
+        return BatchStaging(rows, seqs, self.max_blocks, self.device, tc_heads=self._prefill_tc_heads() if tc else 0)
+
+    def _make_forward(self, logit_rows: int, attn_splits: int, emulate_bf16: bool):
+        if not self.is_cuda:
+            return ReferenceForward(self.w, self.pool, emulate_bf16=emulate_bf16)
+        return CudaForward(self.w, self.pool, max_rows=self.max_rows, max_logit_rows=logit_rows, decode_rows=self.max_seqs,
+                           max_seq_len=self.max_seq_len, attn_splits=attn_splits, tp=self.tp)
+
+    def _stage(self, st: BatchStaging, b: ExecutionBatch, ahead: bool = False):
+        """Lower a batch into its staging buffer; `ahead`: it follows a step that is not published yet."""
+        return st.fill(b)
+
     # ------------------------------------------------------------------ contract
     def capabilities(self) -> ExecutionCapabilities:
         return ExecutionCapabilities(max_batch_rows=self.max_rows, max_sequences=self.max_seqs, max_topk=40,
@@ -289,7 +333,7 @@ class DeepSeekRunner(ModelRunner):
         g = self.graphs.get(rows)
         if g is None:
             def build():
-                st = BatchStaging(rows, rows, self.max_blocks, self.device)
+                st = self._make_staging(rows, rows)
                 st.np_rpos[:] = -1
                 st.np_slot[:] = -1
                 st.np_lrows[:] = np.arange(rows)
@@ -568,7 +612,7 @@ class DeepSeekRunner(ModelRunner):
             ahead[2].synchronize()      # mispredicted step: its input staging and result buffer are reused below
         if graph_step:
             st, graph = self._graph_for(b.rows)
-            T, R, lrows = st.fill(b)
+            T, R, lrows = self._stage(st, b)
             self.stats.h2d_bytes += st.upload()
             graph.replay()
             self._last_hidden = graph.hidden
@@ -578,7 +622,7 @@ class DeepSeekRunner(ModelRunner):
             want_topk = False
         else:
             st = self.staging
-            T, R, lrows = st.fill(b)
+            T, R, lrows = self._stage(st, b)
             self.stats.h2d_bytes += st.upload()
             L = len(lrows)
             if L > fwd.ws.max_logit_rows:
@@ -648,7 +692,7 @@ class DeepSeekRunner(ModelRunner):
             return
         fwd = self.fwd
         st, graph = self._graph_for(pred.rows)
-        st.fill(pred)
+        self._stage(st, pred, ahead=True)
         self.stats.h2d_bytes += st.upload()
         # the ids just uploaded equal the ones on the device; taking them from there keeps the step independent
         # of the host copy and is what lets it start before the host has looked at them
@@ -664,7 +708,7 @@ class DeepSeekRunner(ModelRunner):
 
     def _execute_reference(self, b: ExecutionBatch, start_layer: int = 0, h0=None) -> ExecutionOutput:
         st = self.staging
-        T, R, lrows = st.fill(b)
+        T, R, lrows = self._stage(st, b)
         L = len(lrows)
         db = st.device_batch(T, L)
         rows: List[RowOutput] = []

@@ -68,6 +68,7 @@ class AttnArgs(C.Structure):
         ("softmax_scale", C.c_float), ("merge_ctr", C.c_void_p),
         ("selection", C.c_void_p), ("sel_width", C.c_int), ("trace", C.c_void_p),
         ("decode_only", C.c_int),
+        ("gate", C.c_void_p), ("ldg", C.c_longlong),
     ]
 
 
@@ -78,6 +79,35 @@ class PrefillAttnArgs(C.Structure):
         ("ldq", C.c_longlong), ("ldo", C.c_longlong), ("pool_rows", C.c_longlong),
         ("n_tiles", C.c_int), ("rows", C.c_int), ("heads", C.c_int), ("kv_lora", C.c_int), ("rope_dim", C.c_int),
         ("num_seqs", C.c_int), ("max_blocks", C.c_int), ("page_size", C.c_int), ("softmax_scale", C.c_float),
+        ("gate", C.c_void_p), ("ldg", C.c_longlong),
+    ]
+
+
+class LayerTailArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("ldx", C.c_longlong), ("mix", C.c_void_p), ("ldm", C.c_longlong),
+        ("gate1", C.c_void_p), ("ldg1", C.c_longlong), ("bias1", C.c_void_p),
+        ("ffn", C.c_void_p), ("ldf", C.c_longlong), ("slots", C.c_int), ("topk", C.c_int),
+        ("gate2", C.c_void_p), ("ldg2", C.c_longlong), ("bias2", C.c_void_p),
+        ("norm_w", C.c_void_p), ("norm_stride", C.c_int), ("rows", C.c_int),
+        ("h", C.c_void_p), ("ldh", C.c_longlong), ("dim", C.c_int), ("dim_pad", C.c_int), ("eps", C.c_float),
+        ("fp32", C.c_int),
+    ]
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = [
+        ("proj", C.c_void_p), ("ldp", C.c_longlong),
+        ("off_q", C.c_int), ("off_k", C.c_int), ("off_v", C.c_int), ("off_b", C.c_int),
+        ("ag", C.c_void_p), ("ldag", C.c_longlong), ("off_gate", C.c_int), ("fp32", C.c_int),
+        ("conv", C.c_void_p), ("a_neg", C.c_void_p), ("dt_bias", C.c_void_p), ("norm_w", C.c_void_p),
+        ("state", C.c_void_p), ("tail", C.c_void_p), ("row_seq", C.c_void_p), ("seq_start", C.c_void_p),
+        ("state_in", C.c_void_p), ("state_out", C.c_void_p),
+        ("qn", C.c_void_p), ("kn", C.c_void_p), ("v", C.c_void_p), ("decay", C.c_void_p), ("beta", C.c_void_p),
+        ("qk", C.c_void_p), ("o", C.c_void_p),
+        ("out", C.c_void_p), ("ldo", C.c_longlong), ("status", C.c_void_p),
+        ("n_states", C.c_int), ("rows", C.c_int), ("n_seqs", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int),
+        ("dim", C.c_int), ("vdim", C.c_int), ("taps", C.c_int), ("eps", C.c_float),
     ]
 
 

@@ -64,6 +64,16 @@ def declare(lib) -> None:
         # expert_table.cu
         "fb_expert_table_apply": ([vp, vp, vp, vp, i, i, i, vp, vp], i),
         "fb_expert_table_resolve": ([vp, vp, vp, i, vp, i, vp, vp], i),
+        # gemm_f32.cu, layered_ops.cu, delta_rule.cu (argument blocks by reference)
+        "fb_gemm_f32": ([vp, vp], i),
+        "fb_embed_norm": ([vp, vp, ll, i, vp, ll, vp, i, vp, ll, i, i, i, f, i, vp, vp], i),
+        "fb_gated_residual_norm": ([vp, vp], i),
+        "fb_latent_append": ([vp, ll, i, i, vp, f, vp, vp, ll, i, i, vp, vp], i),
+        "fb_softcap": ([vp, ll, i, i, f, vp], i),
+        "fb_state_rotate": ([vp, vp, i, i, vp], i),
+        "fb_latent_attention": ([vp, i, vp], i),
+        "fb_delta_decode": ([vp, vp], i),
+        "fb_delta_prefill": ([vp, vp], i),
         # v4_ops.cu
         "fb_hc_pre": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, vp], i),
         "fb_hc_pre_split": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, i, vp, vp, vp], i),

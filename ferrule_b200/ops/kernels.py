@@ -62,7 +62,7 @@ def _w3(w: torch.Tensor):
     """weights as [groups, rows, k] -> (groups, rows, k, ldw, group_stride)."""
     if w.dim() == 2:
         w = w.unsqueeze(0)
-    assert w.dim() == 3 and w.dtype == torch.bfloat16 and w.stride(2) == 1
+    assert w.dim() == 3 and w.dtype in (torch.bfloat16, torch.float32) and w.stride(2) == 1
     return w, w.shape[0], w.shape[1], w.shape[2], w.stride(1), (w.stride(0) if w.shape[0] > 1 else w.shape[1] * w.stride(1))
 
 
@@ -73,7 +73,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
          x_group_koff: int = 0, out_group_coff: int = 0, k: Optional[int] = None,
          comm=None, residual: Optional[torch.Tensor] = None, split_k: int = 0,
          trace: Optional[torch.Tensor] = None, ep_combine=None) -> torch.Tensor:
-    """out = x @ w^T on the tcgen05 path.
+    """out = x @ w^T on the tcgen05 path (bf16 operands), or in full 32 bits on the FMA units (fp32 operands).
 
     x [rows, K] bf16 (row stride arbitrary multiple of 8), w [N, K] or [groups, N, K] bf16.
     plan        : grouped mode, x rows are in expert-major order.
@@ -86,7 +86,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
                   (expert-parallel combine over peer memory); `out` is then unused.
     """
     lib = get_lib(True)
-    assert x.dtype == torch.bfloat16 and x.dim() == 2 and x.stride(1) == 1
+    assert x.dtype in (torch.bfloat16, torch.float32) and x.dtype == w.dtype and x.dim() == 2 and x.stride(1) == 1
+    fp32 = x.dtype == torch.float32
     w, groups, w_rows, wk, ldw, gstride = _w3(w)
     K = wk if k is None else k
     rows = x.shape[0]
@@ -101,8 +102,8 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     if out is None:
         cols = n_out * groups if batched else n_out
         orow = scatter_rows if (epilogue == EPI_SCATTER and scatter_rows) else rows
-        out = torch.empty(orow, cols, dtype=out_dtype, device=x.device)
-    assert out.stride(-1) == 1
+        out = torch.empty(orow, cols, dtype=torch.float32 if fp32 else out_dtype, device=x.device)
+    assert out.stride(-1) == 1 and (not fp32 or out.dtype == torch.float32)
     a = GemmArgs()
     a.w, a.x, a.out = w.data_ptr(), x.data_ptr(), out.data_ptr()
     a.ldw, a.w_group_stride, a.ldx, a.ldo = ldw, gstride, x.stride(0), out.stride(0)
@@ -135,6 +136,9 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
         a.remap_rank, a.remap_row = remap_rank.data_ptr(), remap_row.data_ptr()
         a.ldo = pitch
     a.status = status_tensor(x.device).data_ptr()
+    if fp32:
+        check(lib.fb_gemm_f32(C.byref(a), stream_ptr()), "fb_gemm_f32")
+        return out
     check(lib.fb_gemm_bf16(C.byref(a), stream_ptr()), "fb_gemm_bf16")
     return out
 
@@ -198,11 +202,17 @@ def mla_prep(q: torch.Tensor, q_head_dim: int, ckv: torch.Tensor, heads: int, kv
                           status_tensor(q.device).data_ptr(), stream_ptr()), "fb_mla_prep")
 
 
+def _norm_bits(normalize: bool, group_top: int) -> int:
+    assert group_top in (1, 2)
+    return (1 if normalize else 0) | (2 if group_top == 1 else 0)
+
+
 def router_topk(logits: torch.Tensor, topk: int, score_fn: int, bias: Optional[torch.Tensor] = None,
                 n_groups: int = 1, topk_groups: int = 1, normalize: bool = False,
                 route_scale: float = 1.0, hash_table: Optional[torch.Tensor] = None,
                 token_ids: Optional[torch.Tensor] = None, out_idx: Optional[torch.Tensor] = None,
-                out_w: Optional[torch.Tensor] = None):
+                out_w: Optional[torch.Tensor] = None, group_top: int = 2):
+    """group_top: a group's score is the sum of its two best selection values (2) or its best one (1)."""
     lib = get_lib(True)
     rows, experts = logits.shape
     assert logits.dtype == torch.float32
@@ -212,7 +222,7 @@ def router_topk(logits: torch.Tensor, topk: int, score_fn: int, bias: Optional[t
         out_w = torch.empty(rows, topk, dtype=torch.float32, device=logits.device)
     check(lib.fb_router_topk(logits.data_ptr(), logits.stride(0), ptr(bias), ptr(hash_table),
                              ptr(token_ids), rows, experts, topk, score_fn, n_groups, topk_groups,
-                             1 if normalize else 0, route_scale, out_idx.data_ptr(), out_w.data_ptr(),
+                             _norm_bits(normalize, group_top), route_scale, out_idx.data_ptr(), out_w.data_ptr(),
                              stream_ptr()), "fb_router_topk")
     return out_idx, out_w
 
@@ -375,7 +385,7 @@ def router_append(x: torch.Tensor, w: torch.Tensor, topk: int, score_fn: int, pl
                   token_ids: Optional[torch.Tensor] = None, dst_slots: int = 0,
                   norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, delta: Optional[torch.Tensor] = None,
                   res_out: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
-                  quant_rows=None) -> None:
+                  quant_rows=None, group_top: int = 2) -> None:
     """Router + top-k + row reservation in a static plan + activation gather, one launch (one CTA per token).
     `plan.counts` must be zero on entry.  With `norm_w` the kernel first forms the row itself: `x` is then the
     residual stream, res_out = bf16(x + delta), norm_out = RMSNorm(res_out) * norm_w (bit-equal to `add_rmsnorm`),
@@ -393,7 +403,7 @@ def router_append(x: torch.Tensor, w: torch.Tensor, topk: int, score_fn: int, pl
                                      ptr(norm_out), norm_out.stride(0) if norm_out is not None else 0, eps,
                                      w.data_ptr(), hidden, ptr(bias), ptr(hash_table),
                                      ptr(token_ids), rows, w.shape[0], topk, score_fn, n_groups, topk_groups,
-                                     1 if normalize else 0, route_scale, out_idx.data_ptr(), out_w.data_ptr(), e_lo,
+                                     _norm_bits(normalize, group_top), route_scale, out_idx.data_ptr(), out_w.data_ptr(), e_lo,
                                      e_hi, plan.ntok, dst_slots, plan.counts.data_ptr(), plan.src_token.data_ptr(),
                                      plan.dst_row.data_ptr(), plan.row_scale.data_ptr(), None, 8,
                                      q.data_ptr(), q.stride(0), sc.data_ptr(), sc.stride(0), xgq.data_ptr(),
@@ -406,7 +416,7 @@ def router_append(x: torch.Tensor, w: torch.Tensor, topk: int, score_fn: int, pl
                                     ptr(norm_out), norm_out.stride(0) if norm_out is not None else 0, eps,
                                     w.data_ptr(), hidden, ptr(bias), ptr(hash_table),
                                     ptr(token_ids), rows, w.shape[0], topk, score_fn, n_groups, topk_groups,
-                                    1 if normalize else 0, route_scale, out_idx.data_ptr(), out_w.data_ptr(), e_lo, e_hi,
+                                    _norm_bits(normalize, group_top), route_scale, out_idx.data_ptr(), out_w.data_ptr(), e_lo, e_hi,
                                     plan.ntok, dst_slots, plan.counts.data_ptr(), plan.src_token.data_ptr(),
                                     plan.dst_row.data_ptr(), plan.row_scale.data_ptr(), xg.data_ptr(), xg.stride(0),
                                     status_tensor(x.device).data_ptr(), stream_ptr()), "fb_norm_router_append")
@@ -477,14 +487,14 @@ def prefill_tiles(segments, heads: int, min_rows: int = 1):
 
 
 def prefill_tc_supported(heads: int, kv_lora: int, rope_dim: int, page_size: int) -> bool:
-    return (kv_lora == 512 and rope_dim == 64 and 0 < heads <= 128 and 128 % heads == 0
+    return (kv_lora == 512 and rope_dim in (0, 64) and 0 < heads <= 128 and 128 % heads == 0
             and page_size >= 8 and page_size & (page_size - 1) == 0)
 
 
 def mla_prefill_tc(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor,
                    n_tiles: int, page_size: int, kv_lora: int, rope_dim: int, scale: float, out: torch.Tensor,
-                   sink: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Prefill attention on tcgen05: q [rows, heads, 576] bf16 contiguous, tiles [>= n_tiles, 4] int32 on the
+                   sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Prefill attention on tcgen05: q [rows, heads, 512 + rope_dim] bf16 contiguous, tiles [>= n_tiles, 4] int32 on the
     device (see `prefill_tiles`); rows that no tile covers are left untouched in `out` [rows, heads, 512]."""
     lib = get_lib(True)
     rows, heads, D = q.shape
@@ -498,6 +508,8 @@ def mla_prefill_tc(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.T
     a.n_tiles, a.rows, a.heads, a.kv_lora, a.rope_dim = n_tiles, rows, heads, kv_lora, rope_dim
     a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
     a.softmax_scale = scale
+    if gate is not None:
+        a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
     check(lib.fb_mla_prefill_tc(C.byref(a), stream_ptr()), "fb_mla_prefill_tc")
     return out
 
@@ -507,10 +519,12 @@ def mla_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Te
                   rope_dim: int, scale: float, out: torch.Tensor, *, splits: int = 1,
                   split_tokens: int = 1 << 20, ws: Optional[AttnWorkspace] = None,
                   sink: Optional[torch.Tensor] = None, group_rows: int = 1,
-                  trace: Optional[torch.Tensor] = None, decode_only: bool = False) -> torch.Tensor:
+                  trace: Optional[torch.Tensor] = None, decode_only: bool = False,
+                  gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q [rows, heads, D] bf16; kv_layer [..., D] bf16 (any leading shape, contiguous rows).
     decode_only: one query row per sequence, and every KV row below its position predates the running step
-    (the kernel then requests its first KV tile before waiting for the preceding kernel)."""
+    (the kernel then requests its first KV tile before waiting for the preceding kernel).
+    gate: bf16 [rows, >= heads], the output of a head is multiplied by the sigmoid of its entry."""
     lib = get_lib(True)
     rows, heads, D = q.shape
     assert D == kv_lora + rope_dim and q.stride(2) == 1 and q.stride(1) == D
@@ -531,5 +545,7 @@ def mla_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Te
     a.softmax_scale = scale
     a.trace = ptr(trace)
     a.decode_only = 1 if (decode_only and group_rows == 1) else 0
+    if gate is not None:
+        a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
     check(lib.fb_mla_attention(C.byref(a), stream_ptr()), "fb_mla_attention")
     return out

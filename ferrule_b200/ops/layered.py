@@ -1,0 +1,151 @@
+"""Launchers of the layer-list model kernels (csrc/layered_ops.cu, csrc/delta_rule.cu).
+
+Activations are bf16, or fp32 for models that run in full 32 bits: the launcher follows the tensors' dtype.
+"""
+from __future__ import annotations
+
+import ctypes as C
+from typing import Optional
+
+import torch
+
+from . import _lib
+from ._lib import AttnArgs, DeltaArgs, LayerTailArgs, check, get_lib, ptr, status_tensor, stream_ptr
+
+
+def _fp32(t: torch.Tensor) -> int:
+    assert t.dtype in (torch.bfloat16, torch.float32)
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, norm_w: torch.Tensor, h: torch.Tensor, dim: int,
+               eps: float) -> None:
+    """x = table[ids] (fp32), h = RMSNorm(x) * norm_w (one number, or a vector over `dim`)."""
+    assert x.dtype == torch.float32 and table.dtype == h.dtype and norm_w.dtype == torch.float32
+    check(get_lib(True).fb_embed_norm(ids.data_ptr(), table.data_ptr(), table.stride(0), table.shape[0], x.data_ptr(),
+                                      x.stride(0), norm_w.data_ptr(), 0 if norm_w.numel() == 1 else 1, h.data_ptr(),
+                                      h.stride(0), ids.shape[0], dim, table.shape[1], eps, _fp32(h),
+                                      status_tensor(x.device).data_ptr(), stream_ptr()), "fb_embed_norm")
+
+
+def gated_residual_norm(x: torch.Tensor, norm_w: torch.Tensor, h: torch.Tensor, dim: int, eps: float, *,
+                        mix: Optional[torch.Tensor] = None, gate1: Optional[torch.Tensor] = None,
+                        bias1: Optional[torch.Tensor] = None, ffn: Optional[torch.Tensor] = None, topk: int = 0,
+                        gate2: Optional[torch.Tensor] = None, bias2: Optional[torch.Tensor] = None) -> None:
+    """x += sigmoid(gate1 + bias1) * mix + sigmoid(gate2 + bias2) * sum(ffn rows of the token); h = RMSNorm(x) * norm_w.
+    ffn: [rows, slots, width], of which the first `topk` slots are summed."""
+    a = LayerTailArgs()
+    a.x, a.ldx, a.rows, a.dim, a.dim_pad, a.eps, a.fp32 = x.data_ptr(), x.stride(0), x.shape[0], dim, h.shape[1], eps, _fp32(h)
+    a.norm_w, a.norm_stride = norm_w.data_ptr(), 0 if norm_w.numel() == 1 else 1
+    a.h, a.ldh = h.data_ptr(), h.stride(0)
+    if mix is not None:
+        assert mix.dtype == h.dtype
+        a.mix, a.ldm = mix.data_ptr(), mix.stride(0)
+    if gate1 is not None:
+        a.gate1, a.ldg1, a.bias1 = gate1.data_ptr(), gate1.stride(0), bias1.data_ptr()
+    if ffn is not None:
+        assert ffn.dtype == h.dtype and ffn.dim() == 3 and ffn.is_contiguous() and topk <= ffn.shape[1]
+        a.ffn, a.ldf, a.slots, a.topk = ffn.data_ptr(), ffn.stride(1), ffn.shape[1], topk
+    if gate2 is not None:
+        a.gate2, a.ldg2, a.bias2 = gate2.data_ptr(), gate2.stride(0), bias2.data_ptr()
+    check(get_lib(True).fb_gated_residual_norm(C.byref(a), stream_ptr()), "fb_gated_residual_norm")
+
+
+def latent_append(src: torch.Tensor, rank: int, norm_w: torch.Tensor, eps: float, write_slot: torch.Tensor,
+                  pool_layer: torch.Tensor) -> None:
+    """pool row of every token <- RMSNorm(src[:, :rank]) * norm_w, padded with zeros to the pool's row width."""
+    rows, row_dim = src.shape[0], pool_layer.shape[-1]
+    assert pool_layer.is_contiguous() and pool_layer.dtype == src.dtype and norm_w.numel() == row_dim
+    check(get_lib(True).fb_latent_append(src.data_ptr(), src.stride(0), rank, row_dim, norm_w.data_ptr(), eps,
+                                         write_slot.data_ptr(), pool_layer.data_ptr(), pool_layer.numel() // row_dim, rows,
+                                         _fp32(src), status_tensor(src.device).data_ptr(), stream_ptr()),
+          "fb_latent_append")
+
+
+def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """logits <- cap * tanh(logits / cap) (fp32)."""
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    check(get_lib(True).fb_softcap(logits.data_ptr(), logits.stride(0), logits.shape[0], logits.shape[1], cap,
+                                   stream_ptr()), "fb_softcap")
+    return logits
+
+
+def state_rotate(state_in: torch.Tensor, state_out: torch.Tensor, buffers: int) -> None:
+    """The next step reads what this one wrote: state_in <- state_out <- the slot's next buffer."""
+    check(get_lib(True).fb_state_rotate(state_in.data_ptr(), state_out.data_ptr(), state_in.numel(), buffers,
+                                        stream_ptr()), "fb_state_rotate")
+
+
+def latent_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
+                     row_pos: torch.Tensor, page_size: int, scale: float, out: torch.Tensor,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention over a latent cache in 32-bit arithmetic: q / out [rows, heads, row_dim]."""
+    rows, heads, D = q.shape
+    assert q.stride(1) == D and out.stride(1) == D and kv_layer.shape[-1] == D and kv_layer.dtype == q.dtype
+    a = AttnArgs()
+    a.q, a.kv, a.out = q.data_ptr(), kv_layer.data_ptr(), out.data_ptr()
+    a.block_table, a.row_seq, a.row_pos = block_table.data_ptr(), row_seq.data_ptr(), row_pos.data_ptr()
+    a.status = status_tensor(q.device).data_ptr()
+    a.ldq, a.ldo, a.pool_rows = q.stride(0), out.stride(0), kv_layer.numel() // D
+    a.rows, a.heads, a.kv_lora = rows, heads, D
+    a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
+    a.softmax_scale = scale
+    if gate is not None:
+        a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
+    check(get_lib(True).fb_latent_attention(C.byref(a), _fp32(q), stream_ptr()), "fb_latent_attention")
+    return out
+
+
+class DeltaScratch:
+    """Intermediate rows of the prefill form of the delta rule, for mixers up to the given sizes."""
+
+    def __init__(self, rows: int, mixers, device):
+        f32 = dict(dtype=torch.float32, device=device)
+        big = lambda f: max(f(m) for m in mixers)
+        self.rows = rows
+        self.qn = torch.empty(rows * big(lambda m: m.kv_heads * m.dim), **f32)
+        self.kn = torch.empty_like(self.qn)
+        self.decay = torch.empty(rows * big(lambda m: m.heads * m.dim), **f32)
+        self.v = torch.empty(rows * big(lambda m: m.heads * m.vdim), **f32)
+        self.o = torch.empty_like(self.v)
+        self.beta = torch.empty(rows * big(lambda m: m.heads), **f32)
+        self.qk = torch.empty(rows * big(lambda m: m.kv_heads), **f32)
+
+
+def delta_decode_supported(mixer) -> bool:
+    return mixer.vdim <= 128 and mixer.vdim % 4 == 0 and mixer.dim <= 128
+
+
+def delta_rule(proj: torch.Tensor, off, ag: torch.Tensor, img, mixer, eps: float, state: torch.Tensor,
+               tail: torch.Tensor, seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int,
+               out: torch.Tensor, *, row_seq: Optional[torch.Tensor] = None, scratch: Optional[DeltaScratch] = None,
+               decode: bool = False) -> torch.Tensor:
+    """Convolutions, recurrence and gated output norm of a delta mixer over the rows of a packed batch.
+    proj: rows of the layer's input projection, `off` its block offsets; ag: fp32 rows of the second low-rank halves;
+    decode: one row per sequence, a single launch."""
+    assert ag.dtype == torch.float32 and state.dtype == torch.float32 and state.is_contiguous() and tail.is_contiguous()
+    assert tail.dtype == proj.dtype == out.dtype
+    a = DeltaArgs()
+    a.proj, a.ldp = proj.data_ptr(), proj.stride(0)
+    a.off_q, a.off_k, a.off_v, a.off_b = off["q"], off["k"], off["v"], off["b"]
+    a.ag, a.ldag, a.off_gate, a.fp32 = ag.data_ptr(), ag.stride(0), img.off_gate, _fp32(proj)
+    a.conv, a.a_neg, a.dt_bias, a.norm_w = (img.conv.data_ptr(), img.a_neg.data_ptr(), img.dt_bias.data_ptr(),
+                                            img.o_norm.data_ptr())
+    a.state, a.tail, a.n_states = state.data_ptr(), tail.data_ptr(), state.shape[0]
+    a.row_seq, a.seq_start = ptr(row_seq), seq_start.data_ptr()
+    a.state_in, a.state_out = state_in.data_ptr(), state_out.data_ptr()
+    a.rows, a.n_seqs = proj.shape[0], n_seqs
+    a.heads, a.kv_heads, a.dim, a.vdim, a.taps = mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim, mixer.taps
+    a.out, a.ldo, a.eps = out.data_ptr(), out.stride(0), eps
+    a.status = status_tensor(proj.device).data_ptr()
+    if decode:
+        assert n_seqs == proj.shape[0]
+        check(get_lib(True).fb_delta_decode(C.byref(a), stream_ptr()), "fb_delta_decode")
+        return out
+    assert scratch is not None and scratch.rows >= proj.shape[0]
+    a.qn, a.kn, a.v, a.decay = (scratch.qn.data_ptr(), scratch.kn.data_ptr(), scratch.v.data_ptr(),
+                                scratch.decay.data_ptr())
+    a.beta, a.qk, a.o = scratch.beta.data_ptr(), scratch.qk.data_ptr(), scratch.o.data_ptr()
+    check(get_lib(True).fb_delta_prefill(C.byref(a), stream_ptr()), "fb_delta_prefill")
+    _lib.LAUNCHES[0] += 2                    # prepare, scan, output
+    return out

@@ -91,8 +91,8 @@ def route(logits: torch.Tensor, topk: int, score_fn: int = SCORE_SOFTMAX,
           bias: Optional[torch.Tensor] = None, n_groups: int = 1, topk_groups: int = 1,
           normalize: bool = False, route_scale: float = 1.0,
           hash_table: Optional[torch.Tensor] = None,
-          token_ids: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
-    """-> (expert ids [T,k] int32, weights [T,k] fp32)."""
+          token_ids: Optional[torch.Tensor] = None, group_top: int = 2) -> Tuple[torch.Tensor, torch.Tensor]:
+    """-> (expert ids [T,k] int32, weights [T,k] fp32).  group_top: how many of a group's best values its score sums."""
     lf = logits.float()
     if score_fn == SCORE_SOFTMAX:
         score = torch.softmax(lf, dim=-1)
@@ -108,7 +108,7 @@ def route(logits: torch.Tensor, topk: int, score_fn: int = SCORE_SOFTMAX,
         if n_groups > 1 and topk_groups < n_groups:
             T, E = sel.shape
             grp = sel.view(T, n_groups, E // n_groups)
-            gscore = stable_topk(grp, 2)[0].sum(-1)
+            gscore = stable_topk(grp, group_top)[0].sum(-1)
             _, gidx = stable_topk(gscore, topk_groups)
             mask = torch.zeros(T, n_groups, dtype=torch.bool, device=sel.device)
             mask.scatter_(1, gidx, True)

@@ -16,6 +16,8 @@ from dataclasses import dataclass, field
 from enum import Enum
 from typing import Dict, List, Optional, Sequence, Tuple
 
+import numpy as np
+
 
 class ExecutionError(ValueError):
     pass
@@ -247,7 +249,7 @@ class ExecutionOutput:
                         raise ExecutionError(f"row {ro.input_row}: candidates not sorted by logit")
                     if ro.logits[a] == ro.logits[a - 1] and ro.token_ids[a] <= ro.token_ids[a - 1]:
                         raise ExecutionError(f"row {ro.input_row}: tied candidates not in token order")
-            if ro.full_logits is not None and any(not math.isfinite(v) for v in ro.full_logits):
+            if ro.full_logits is not None and not np.isfinite(np.asarray(ro.full_logits)).all():
                 raise ExecutionError(f"row {ro.input_row}: non-finite full logits")
 
     def by_row(self) -> Dict[int, RowOutput]:
