@@ -10,6 +10,7 @@
   bench-interactive    multi-turn timing report (JSON) with engine, KV and speculative statistics
   bench-serve          synthetic serving sweep against a running server (Poisson arrivals, shared prefixes)
   expert-stream-smoke  stream routed experts of a checkpoint through the materialization stack
+  trace-run            replay given token streams step by step and write logits (the same program as bin/trace_run)
 
 Counterpart of crates/ferrule-cli/src/args.rs:34-230, commands/serve.rs:20-168,
 commands/bench_interactive.rs:57-235 and scripts/bench_vllm_serve.sh, dsv4_synthetic_fixture.py.
@@ -117,7 +118,11 @@ def build_engine(args, layout=None):
     dev = args.device or ("cuda" if torch.cuda.is_available() else "cpu")
     if getattr(args, "model", None) and not args.model_dir:
         args.model_dir = args.model
-    if args.model_dir and _is_v4_dir(args.model_dir):
+    from ..models import layered_config as LC
+    arch = _architecture(args.model_dir)
+    if arch == "gitozen" or (not args.model_dir and args.preset in LC.PRESETS):
+        return _build_layered_engine(args, dev, args.model_dir, layout)
+    if arch == "deepseek_v4":
         return _build_v4_engine(args, dev, args.model_dir)
     if args.model_dir:
         from ..io.checkpoint import load_deepseek_hf
@@ -187,12 +192,23 @@ def build_engine(args, layout=None):
     return eng, load_tokenizer(args.model_dir), name
 
 
-def _is_v4_dir(model_dir: str) -> bool:
-    try:
-        with open(os.path.join(model_dir, "config.json")) as f:
-            return json.load(f).get("model_type") == "deepseek_v4"
-    except OSError:
-        return False
+def _architecture(model_dir: Optional[str]) -> Optional[str]:
+    """Registry name of a checkpoint directory's architecture, None without a directory."""
+    if not model_dir:
+        return None
+    from ..models.registry import architecture_of
+    return architecture_of(model_dir).name
+
+
+def _engine_sizes(args, max_position: int):
+    """(context tokens, pages per sequence, scheduler configuration) from the command line's limits."""
+    from ..runtime.scheduler import SchedulerConfig
+    pages_per_seq = (min(args.ctx_size, max_position) + args.page_size - 1) // args.page_size
+    ctx = pages_per_seq * args.page_size
+    return ctx, pages_per_seq, SchedulerConfig(
+        max_active_sequences=args.max_seqs, max_decode_batch=args.max_seqs, max_batch_tokens=args.max_batch_tokens,
+        prefill_chunk_size=args.prefill_chunk, decode_cohort_target=getattr(args, "decode_cohort_target", 1),
+        decode_cohort_max_deferrals=getattr(args, "decode_cohort_max_deferrals", 0), ctx_size=ctx)
 
 
 def _chat_template(args):
@@ -212,6 +228,47 @@ def _expert_plan(args):
     return {int(l): [int(e) for e in o] for l, o in doc.get("plan", doc).items()}
 
 
+def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=None):
+    """A layer-list model (Gitozen) behind the engine: a checkpoint directory, or a random-init preset."""
+    import torch
+
+    from ..models.layered_config import PRESETS
+    from ..models.layered_weights import random_weights
+    from ..models.registry import ARCHITECTURES, RunnerLimits
+    from ..runtime.engine import Engine, EngineConfig
+    from ..utils.tokenizer import load_tokenizer
+    if args.speculative and args.speculative != "auto":
+        raise SystemExit("--speculative: recurrent state cannot drop rejected rows, and the architecture has no proposal stages")
+    if layout is not None:
+        raise SystemExit("layer-list models run on one rank")
+    for flag in ("expert_residency", "moe_hotset_experts", "prefix_cache_tokens", "async_streaming", "expert_plan"):
+        if getattr(args, flag, None):
+            raise SystemExit(f"--{flag.replace('_', '-')} is not available for layer-list models")
+    if getattr(args, "weight_format", "bf16") != "bf16":
+        raise SystemExit("--weight-format: layer-list models run bf16 weights")
+    args.speculative = False
+    arch = ARCHITECTURES["gitozen"]
+    dtype = torch.bfloat16 if dev != "cpu" else torch.float32
+    if model_dir:
+        weights = arch.load(model_dir, dev, dtype, max_layers=getattr(args, "layers", 0))
+        name = os.path.basename(os.path.normpath(model_dir))
+    else:
+        cfg = PRESETS[args.preset]()
+        if getattr(args, "layers", 0):
+            cfg = cfg.with_(layers=tuple(cfg.layers[i % cfg.n_layers] for i in range(args.layers)))
+        weights = random_weights(cfg, device=dev, dtype=dtype, seed=args.seed)
+        name = args.preset
+    cfg = weights.cfg
+    ctx, pages_per_seq, sched = _engine_sizes(args, cfg.max_position)
+    n_pages = args.max_seqs * pages_per_seq + 8
+    if args.kv_cache_mb:
+        per_page = max(len(cfg.latent_layers), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
+        n_pages = max(args.kv_cache_mb * (1 << 20) // per_page, pages_per_seq + 1)
+    runner = arch.runner(weights, RunnerLimits(n_pages, args.page_size, args.max_batch_tokens, args.max_seqs, ctx), device=dev)
+    eng = Engine(runner, EngineConfig(scheduler=sched, kv_pages=n_pages, page_size=args.page_size))
+    return eng, load_tokenizer(model_dir), name
+
+
 def _build_v4_engine(args, dev, model_dir: Optional[str] = None):
     """DeepSeek-V4 family model behind the engine (slot-bound state): a checkpoint directory, or the random-init
     tiny shape."""
@@ -220,7 +277,6 @@ def _build_v4_engine(args, dev, model_dir: Optional[str] = None):
     from ..models.v4_model import random_v4_weights, tiny_v4
     from ..models.v4_runner import V4Runner
     from ..runtime.engine import Engine, EngineConfig
-    from ..runtime.scheduler import SchedulerConfig
     from ..utils.tokenizer import load_tokenizer
     if model_dir:
         from ..io.v4_checkpoint import load_v4_hf
@@ -236,16 +292,10 @@ def _build_v4_engine(args, dev, model_dir: Optional[str] = None):
         args.speculative = weights.proposal is not None
     if args.speculative and weights.proposal is None:
         raise SystemExit("--speculative: this DeepSeek-V4 checkpoint has no `mtp.*` proposal stages")
-    ctx = min(args.ctx_size, cfg.max_position)
-    pages_per_seq = (ctx + args.page_size - 1) // args.page_size
+    ctx, pages_per_seq, sched = _engine_sizes(args, cfg.max_position)
     n_pages = args.max_seqs * pages_per_seq + 8
-    runner = V4Runner(weights, n_pages=n_pages, page_size=args.page_size, max_seqs=args.max_seqs,
-                      max_seq_len=pages_per_seq * args.page_size, max_rows=args.max_batch_tokens)
-    sched = SchedulerConfig(max_active_sequences=args.max_seqs, max_decode_batch=args.max_seqs,
-                            max_batch_tokens=args.max_batch_tokens, prefill_chunk_size=args.prefill_chunk,
-                            decode_cohort_target=getattr(args, "decode_cohort_target", 1),
-                            decode_cohort_max_deferrals=getattr(args, "decode_cohort_max_deferrals", 0),
-                            ctx_size=pages_per_seq * args.page_size)
+    runner = V4Runner(weights, n_pages=n_pages, page_size=args.page_size, max_seqs=args.max_seqs, max_seq_len=ctx,
+                      max_rows=args.max_batch_tokens)
     # the block drafter proposes `proposal_block_size` tokens at once: --max-draft above 1 caps it, the default
     # takes the whole block
     draft = cfg.proposal_block_size if args.max_draft <= 1 else min(args.max_draft, cfg.proposal_block_size)
@@ -264,6 +314,7 @@ def cmd_info(args) -> int:
 
     from .. import __version__, _build
     from ..models import config as C
+    from ..models import layered_config as LC
     out = {"version": __version__, "torch": torch.__version__, "cuda_available": torch.cuda.is_available(),
            "native_library": str(_build.LIB_PATH), "native_library_built": _build.LIB_PATH.exists(),
            "native_library_current": _build.is_current()}
@@ -284,7 +335,19 @@ def cmd_info(args) -> int:
                 "missing": [{"area": m.area, "reason": m.reason} for m in plan.missing],
                 "policies": {k: enc(getattr(ps, k)) for k in ("attention", "router", "expert", "quant", "kv", "residency",
                                                              "parallelism", "speculation")}}
-    if args.model_dir and _is_v4_dir(args.model_dir):
+    arch = _architecture(args.model_dir)
+    if arch == "gitozen":
+        from ..io.layered_checkpoint import bind_config
+        from ..io.safetensors import ShardedCheckpoint
+        from ..models.families import detect_family, layout_summary
+        from ..models.layered_config import from_layer_list
+        ck = ShardedCheckpoint(args.model_dir)
+        lcfg = bind_config(from_layer_list(args.model_dir), ck)
+        fam = detect_family(ck.names())
+        out["checkpoint"] = {"family": fam.value, "tensors": len(ck.names()), "shards": len(set(ck.weight_map.values())),
+                             "roles": layout_summary(ck.names(), fam, lcfg.n_layers), "config": lcfg.to_dict()}
+        out["engine_plan"] = plan_of(lcfg)
+    elif arch == "deepseek_v4":
         from dataclasses import asdict
         from ..io.safetensors import ShardedCheckpoint
         from ..io.v4_checkpoint import v4_config_from_hf
@@ -307,7 +370,8 @@ def cmd_info(args) -> int:
             out["engine_plan"] = plan_of(cfg)
     else:
         out["presets"] = {k: {"params_b": round(f().param_count() / 1e9, 3), "layers": f().n_layers,
-                              "hidden": f().hidden, "engine_plan": plan_of(f())["status"]} for k, f in C.PRESETS.items()}
+                              "hidden": f().hidden, "engine_plan": plan_of(f())["status"]}
+                          for k, f in {**C.PRESETS, **LC.PRESETS}.items()}
     print(json.dumps(out, indent=1))
     return 0
 
@@ -381,6 +445,18 @@ def cmd_make_fixture(args) -> int:
         export_v4_hf(w, args.out, dense_format=dense, expert_format=expert, shard_bytes=args.shard_mb << 20)
         print(json.dumps({"written": args.out, "family": "deepseek_v4", "layers": cfg.n_layers,
                           "proposal_stages": cfg.n_proposal_stages, "dense_format": dense, "expert_format": expert}))
+        return 0
+    if args.family == "gitozen":
+        from ..io.layered_checkpoint import export_layered
+        from ..models.layered_config import PRESETS
+        from ..models.layered_weights import RandomTensors
+        lcfg = PRESETS[args.preset if args.preset in PRESETS else "tiny-gitozen"]()
+        if args.layers:
+            lcfg = lcfg.with_(layers=tuple(lcfg.layers[i % lcfg.n_layers] for i in range(args.layers)))
+        if args.dense_format != "plain" or args.expert_format != "plain":
+            raise SystemExit("--family gitozen: checkpoints are stored in BF16")
+        export_layered(lcfg, RandomTensors(lcfg, args.seed, gain=0.0 if args.zeros else 1.0), args.out, args.shard_mb << 20)
+        print(json.dumps({"written": args.out, "family": "gitozen", "params": lcfg.param_count(), "layers": lcfg.n_layers}))
         return 0
     cfg = C.PRESETS[args.preset]()
     if args.layers:
@@ -811,8 +887,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--zeros", action="store_true"); p.add_argument("--shard-mb", type=int, default=1024)
     p.add_argument("--dense-format", default="plain", choices=["plain", "fp8_block"])
     p.add_argument("--expert-format", default="plain", choices=["plain", "fp8_block", "mxfp4"])
-    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4"],
-                   help="v4: a DeepSeek-V4 directory (tiny shape; FP8 dense + packed FP4 experts unless --plain)")
+    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", "gitozen"],
+                   help="v4: a DeepSeek-V4 directory (tiny shape; FP8 dense + packed FP4 experts unless --plain); "
+                        "gitozen: a layer-list directory (--preset tiny-gitozen unless another of its presets is named)")
     p.add_argument("--plain", action="store_true", help="--family v4: keep every linear in BF16")
     p.add_argument("--proposal-stages", type=int, default=0,
                    help="--family v4: also write this many `mtp.*` proposal stages with their prediction heads")
@@ -852,6 +929,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--chunks", type=int, nargs="+", default=[64, 128, 256, 512]); p.add_argument("--requests", type=int, default=4)
     p.add_argument("--prompt-len", type=int, default=256); p.add_argument("--max-tokens", type=int, default=8)
     p.set_defaults(fn=cmd_chunk_sweep)
+    sub.add_parser("trace-run", add_help=False, help="replay token streams and write logits (see trace-run --help)")
     p = sub.add_parser("bench-serve")
     p.add_argument("--url", default="http://127.0.0.1:8000"); p.add_argument("--model", default="")
     p.add_argument("--concurrency", type=int, nargs="+", default=[1, 8, 32]); p.add_argument("--requests", type=int, default=64)
@@ -865,6 +943,11 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--slabs", type=int, default=8); p.add_argument("--threads", type=int, default=4)
     p.add_argument("--host-cache-mb", type=int, default=256); p.add_argument("--timeout", type=float, default=120.0)
     p.set_defaults(fn=cmd_expert_stream_smoke)
+    if argv is None:
+        argv = sys.argv[1:]
+    if argv and argv[0] == "trace-run":
+        from .trace_run import main as trace_main
+        return trace_main(argv[1:])
     args = ap.parse_args(argv)
     from ..io.safetensors import CheckpointError
     try:

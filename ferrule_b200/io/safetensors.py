@@ -153,7 +153,7 @@ def save_file(tensors: Dict[str, torch.Tensor], path, dtype_names: Optional[Dict
         dname = (dtype_names or {}).get(name) or _REV.get(t.dtype)
         if dname is None:
             raise CheckpointError(f"cannot store dtype {t.dtype}")
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         pad = (-len(raw)) % 8
         header[name] = {"dtype": dname, "shape": list(t.shape), "data_offsets": [off, off + len(raw)]}
         chunks.append(raw + b"\0" * pad)

@@ -3,8 +3,9 @@
 Roles tell the loader what a tensor is (attention projection, norm, router, routed / shared expert
 weight, scale, MTP part ...) independent of the naming scheme.  Families: DeepSeek (HuggingFace
 V2/V3 names: `model.layers.N.self_attn.q_a_proj.weight`), DeepSeek-V4 (the reference's flat names:
-`layers.N.attn.wq_a.weight`, `ffn.experts.E.w1.weight`, `mtp.M.*`), Qwen3 and generic
-Llama-style.  Only the DeepSeek family executes; the others are classified for inspection.
+`layers.N.attn.wq_a.weight`, `ffn.experts.E.w1.weight`, `mtp.M.*`), Gitozen (layer-list names:
+`lN.mix.q`, `lN.mlp.eE.gate`), Qwen3 and generic Llama-style.  The DeepSeek families and Gitozen execute; the others
+are classified for inspection.
 
 Counterpart of crates/ferrule-model/src/families/mod.rs:20-115, families/deepseek_v4.rs:9-300 and
 support/*.rs (TensorRole / ModelLayout).
@@ -51,6 +52,13 @@ class TensorRole(Enum):
     DENSE_GATE = "dense_gate"
     DENSE_UP = "dense_up"
     DENSE_DOWN = "dense_down"
+    ATTN_GATE = "attn_gate"
+    RESIDUAL_GATE = "residual_gate"
+    DELTA_CONV = "delta_conv"
+    DELTA_DECAY = "delta_decay"
+    DELTA_BETA = "delta_beta"
+    DELTA_GATE = "delta_gate"
+    DELTA_NORM = "delta_norm"
     MTP = "mtp"
     SCALE = "scale"
     UNKNOWN = "unknown"
@@ -68,6 +76,7 @@ class TensorClass:
 class Family(Enum):
     DEEPSEEK_HF = "deepseek_hf"
     DEEPSEEK_V4 = "deepseek_v4"
+    GITOZEN = "gitozen"
     QWEN3 = "qwen3"
     LLAMA = "llama"
 
@@ -86,6 +95,38 @@ _V4_ATTN = {"wq_a": TensorRole.ATTN_Q_A, "wq_b": TensorRole.ATTN_Q_B, "wkv": Ten
 _V4_FFN = {"w1": 0, "w3": 1, "w2": 2}
 
 
+_LAYERED_MIX = {"q": TensorRole.ATTN_Q, "k": TensorRole.ATTN_K, "v": TensorRole.ATTN_V, "o": TensorRole.ATTN_OUT,
+                "dkv": TensorRole.ATTN_KV_A, "dkv.norm": TensorRole.ATTN_KV_NORM, "uk": TensorRole.ATTN_KV_B,
+                "uv": TensorRole.ATTN_KV_B, "g": TensorRole.ATTN_GATE, "q.conv": TensorRole.DELTA_CONV,
+                "k.conv": TensorRole.DELTA_CONV, "v.conv": TensorRole.DELTA_CONV, "b": TensorRole.DELTA_BETA,
+                "A_log": TensorRole.DELTA_DECAY, "a1": TensorRole.DELTA_DECAY, "a2": TensorRole.DELTA_DECAY,
+                "dt_bias": TensorRole.DELTA_DECAY, "g1": TensorRole.DELTA_GATE, "g2": TensorRole.DELTA_GATE,
+                "norm": TensorRole.DELTA_NORM}
+_LAYERED_FFN = {"gate": 0, "up": 1, "down": 2}
+
+
+def _classify_layered(name: str) -> "TensorClass":
+    top = {"embed": TensorRole.EMBEDDING, "final.norm": TensorRole.FINAL_NORM, "head": TensorRole.OUTPUT_HEAD}
+    if name in top:
+        return TensorClass(top[name])
+    m = re.match(r"l(\d+)\.(.*)", name)
+    if not m:
+        return TensorClass(TensorRole.UNKNOWN)
+    layer, rest = int(m.group(1)), m.group(2)
+    if rest == "norm1":
+        return TensorClass(TensorRole.ATTN_NORM, layer)
+    if re.fullmatch(r"rg[12](\.b)?", rest):
+        return TensorClass(TensorRole.RESIDUAL_GATE, layer)
+    if rest == "mlp.router":
+        return TensorClass(TensorRole.ROUTER, layer)
+    m2 = re.fullmatch(r"mlp\.e(\d+)\.(gate|up|down)", rest)
+    if m2:
+        return TensorClass(_ffn_role("expert", _LAYERED_FFN[m2.group(2)]), layer, int(m2.group(1)))
+    if rest.startswith("mix."):
+        return TensorClass(_LAYERED_MIX.get(rest[4:], TensorRole.UNKNOWN), layer)
+    return TensorClass(TensorRole.UNKNOWN, layer)
+
+
 def _ffn_role(kind: str, idx: int) -> TensorRole:
     table = {"expert": (TensorRole.EXPERT_GATE, TensorRole.EXPERT_UP, TensorRole.EXPERT_DOWN),
              "shared": (TensorRole.SHARED_GATE, TensorRole.SHARED_UP, TensorRole.SHARED_DOWN),
@@ -94,6 +135,8 @@ def _ffn_role(kind: str, idx: int) -> TensorRole:
 
 
 def classify(name: str, family: Family, n_layers: Optional[int] = None) -> TensorClass:
+    if family == Family.GITOZEN:
+        return _classify_layered(name)
     is_scale = name.endswith(_SCALE_SUFFIX)
     base = name
     for s in _SCALE_SUFFIX + (".weight", ".bias"):
@@ -188,6 +231,8 @@ def classify(name: str, family: Family, n_layers: Optional[int] = None) -> Tenso
 
 def detect_family(names: Iterable[str], model_type: str = "") -> Family:
     names = list(names)
+    if "l0.norm1" in names or model_type.lower() == "gitozen":
+        return Family.GITOZEN
     if any(n.startswith("layers.") and ".attn.wq_a" in n for n in names) or any(n.startswith("mtp.") for n in names):
         return Family.DEEPSEEK_V4
     mt = model_type.lower()

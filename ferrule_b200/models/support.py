@@ -18,16 +18,19 @@ from enum import Enum
 from typing import List, Optional, Tuple
 
 from .config import SCORE_SIGMOID, SCORE_SOFTMAX, ModelConfig
+from .layered_config import LayeredConfig
 
 
 class AttentionKind(Enum):
     MLA = "mla"                       # latent KV, weight-absorbed (DeepSeek-V2 / V3)
     HYBRID_SPARSE_MLA = "hybrid_mla"  # single latent head + window + compressed selection (DeepSeek-V4)
+    LATENT_DELTA = "latent_delta"     # per layer: latent attention without positions, or gated delta rule (Gitozen)
 
 
 class RouterKind(Enum):
     NONE = "none"
     SOFTMAX_TOPK = "softmax_topk"
+    SOFTMAX_GROUP_TOPK = "softmax_group_topk"
     SIGMOID_GROUP_TOPK = "sigmoid_group_topk"
     SQRT_SOFTPLUS_TOPK = "sqrt_softplus_topk"
     HASH = "hash"
@@ -125,15 +128,23 @@ class PolicySet:
     speculation: SpeculationPolicy
     tokenizer: TokenizerPolicy
     validation: ValidationPolicy
-    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4"
+    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4" | "gitozen"
 
     @staticmethod
     def from_config(cfg, weight_format: str = "bf16", parallelism: Optional[ParallelismPlan] = None,
                     page_size: int = 64, resident_fraction: float = 1.0, chat_template: bool = True,
                     tokenizer_files: bool = False) -> "PolicySet":
         par = parallelism or ParallelismPlan()
-        v4 = not isinstance(cfg, ModelConfig)          # models.v4_model.V4Config
-        if v4:
+        if isinstance(cfg, LayeredConfig):
+            moes = [l.mlp for l in cfg.layers if l.mlp is not None]
+            groups = max(((m.groups, m.keep) for m in moes), default=(1, 1))
+            att = AttentionPolicy(AttentionKind.LATENT_DELTA, cfg.kv_row_dim, cfg.n_heads, False)
+            router = RouterPolicy(RouterKind.NONE if not moes else (RouterKind.SOFTMAX_GROUP_TOPK if groups[0] > 1
+                                                                    else RouterKind.SOFTMAX_TOPK), cfg.topk, groups)
+            expert = ExpertPolicy(cfg.n_routed_experts, 0, cfg.n_layers - len(moes))
+            planes = (("latent_kv",) if cfg.latent_layers else ()) + (("recurrent_state",) if cfg.delta_layers else ())
+            spec, sem = SpeculationPolicy(SpeculationMode.NONE, 0), "gitozen"
+        elif not isinstance(cfg, ModelConfig):         # models.v4_model.V4Config
             att = AttentionPolicy(AttentionKind.HYBRID_SPARSE_MLA, cfg.head_dim, cfg.n_heads, True)
             router = RouterPolicy(RouterKind.HASH if cfg.n_hash_layers >= cfg.n_layers else RouterKind.SQRT_SOFTPLUS_TOPK,
                                   cfg.topk, (1, 1))
@@ -214,6 +225,13 @@ class EnginePlan:
                                              "dequantised at load time)"))
             if par.tensor_parallel > 1 or par.pipeline_parallel > 1:
                 missing.append(MissingPolicy("parallelism", "the V4 runner is single-GPU"))
+        if p.semantics == "gitozen":
+            if p.quant.weight_format != "bf16":
+                missing.append(MissingPolicy("quantization", "layer-list models run bf16 (or fp32) weights"))
+            if par.tensor_parallel > 1 or par.pipeline_parallel > 1 or par.expert_parallel > 1:
+                missing.append(MissingPolicy("parallelism", "the layer-list runner is single-GPU"))
+            if p.residency.resident_fraction < 1.0:
+                missing.append(MissingPolicy("residency", "layer-list models keep every expert resident"))
         if p.residency.resident_fraction < 1.0 and p.quant.weight_format != "bf16" and p.semantics != "deepseek-v4":
             pass        # quantised experts stream through the same arena (frames hold the packed form)
         status = EnginePlanStatus.EXECUTABLE if not missing else EnginePlanStatus.METADATA_ONLY
