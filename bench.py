@@ -101,7 +101,9 @@ def main() -> None:
     ap.add_argument("--impl", default="ours")
     ap.add_argument("--batch", type=int, default=32)
     ap.add_argument("--prompt-len", type=int, default=512)
-    ap.add_argument("--model", default="deepseek-v2-lite")
+    ap.add_argument("--model", default="deepseek-v2-lite",
+                    help="deepseek-v2-lite is the headline configuration; gitozen-lite and gitozen-latent-lite are layer-list "
+                         "models of the same widths (one GPU), reported without a baseline")
     ap.add_argument("--weight-format", default="bf16", choices=["bf16", "fp8_block", "fp8_mxfp4"],
                     help="bf16 is the headline configuration; the FP8 formats are reported with their own dtype")
     ap.add_argument("--shard-as", type=int, default=0,
@@ -157,13 +159,17 @@ def main() -> None:
                              fused=not args.no_fused, collective=args.collective, multicast_push=args.mc_push)
         tp, pp = lay.tp, lay.pp
 
-    cfg = C.PRESETS[args.model]()
+    from ferrule_b200.models import layered_config as LC
+    layered = args.model in LC.PRESETS
+    if layered and (world > 1 or args.weight_format != "bf16"):
+        raise SystemExit(f"--model {args.model} runs on one GPU with bf16 weights")
+    cfg = (LC.PRESETS if layered else C.PRESETS)[args.model]()
     if cfg.n_mtp_layers:
         # plain greedy decoding: the multi-token-prediction module only serves speculative decoding and is not
         # instantiated (its weights are not part of the decode step's traffic either way)
         cfg = cfg.with_(n_mtp_layers=0)
     if args.layers:
-        cfg = cfg.with_(n_layers=args.layers)
+        cfg = cfg.with_(layers=cfg.layers[:args.layers]) if layered else cfg.with_(n_layers=args.layers)
     B, P, K, Wm = args.batch, args.prompt_len, args.steps, args.warmup
     page = 64
     margin = 64                      # sequences that finish prefill early decode ahead of the others
@@ -172,15 +178,21 @@ def main() -> None:
     pages_per_seq = (max_seq + page - 1) // page
     tp_world = lay.tp_size if lay else 1
     from ferrule_b200.parallel.pp import stage_range, stage_weights
-    weights = W.random_weights(cfg, device=dev, seed=0, tp_rank=lay.tp_rank if lay else 0, tp_world=args.shard_as or tp_world,
-                               fast_device_init=True, weight_format=args.weight_format,
-                               replicate_shared=(tp_world > 1 and args.moe == "dispatch"), router_zipf=args.router_zipf,
-                               layer_range=stage_range(cfg.n_layers, lay.pp_rank, lay.pp_size) if pp is not None else None)
+    if layered:
+        from ferrule_b200.models.layered_runner import LayeredRunner
+        from ferrule_b200.models.layered_weights import random_weights as layered_weights
+        from ferrule_b200.ops import layered as KL
+        weights = layered_weights(cfg, device=dev, seed=0)
+    else:
+        weights = W.random_weights(cfg, device=dev, seed=0, tp_rank=lay.tp_rank if lay else 0, tp_world=args.shard_as or tp_world,
+                                   fast_device_init=True, weight_format=args.weight_format,
+                                   replicate_shared=(tp_world > 1 and args.moe == "dispatch"), router_zipf=args.router_zipf,
+                                   layer_range=stage_range(cfg.n_layers, lay.pp_rank, lay.pp_size) if pp is not None else None)
     if pp is not None:
         weights = stage_weights(weights, lay.pp_rank, lay.pp_size)
-    runner = DeepSeekRunner(weights, n_pages=B * pages_per_seq + 8, page_size=page, max_rows=2048, max_seqs=B,
-                            max_seq_len=pages_per_seq * page, device=dev, tp=tp, pp=pp,
-                            enable_mtp=False)
+    sizes = dict(n_pages=B * pages_per_seq + 8, page_size=page, max_rows=2048, max_seqs=B, max_seq_len=pages_per_seq * page,
+                 device=dev)
+    runner = LayeredRunner(weights, **sizes) if layered else DeepSeekRunner(weights, **sizes, tp=tp, pp=pp, enable_mtp=False)
     if tp is not None:
         tp.attach(runner.fwd)
         if args.moe == "dispatch":
@@ -294,12 +306,16 @@ def main() -> None:
             for i, pg in enumerate(pages):
                 st.np_bt[i, :len(pg)] = pg
                 st.np_slot[i] = pg[start_pos[i] // page] * page + start_pos[i] % page
+            if layered:
+                st.fill_states([(*runner.states.bind(s.slot, False), 1) for s in seqs0])
             st.upload()
 
         def device_steps(n: int) -> None:
             for _ in range(n):
                 graph.replay()
                 KK.decode_advance(runner.fwd.ws.next_id[:B], graph.batch, cfg.vocab_size, page, True)
+                if layered:
+                    KL.state_rotate(st.d_state_in[:B], st.d_state_out[:B], runner.states.buffers)
 
         rewind()
         device_steps(3)
@@ -336,7 +352,7 @@ def main() -> None:
             "metric": "decode tokens/s (whole job, max over ranks)",
             "value": round(value, 1), "unit": "tokens/s", "n_gpus": world, "steps": K, "warmup": Wm,
             "ms_per_step": round(dev_ms / K, 4), "higher_is_better": True, "scaling": "strong",
-            "vs_baseline": round(value / BASELINE_TOK_S, 1), "dtype": {"bf16": "bf16", "fp8_block": "fp8 e4m3 weights (128x128 scales) + fp8 activations (1x128), bf16 elsewhere", "fp8_mxfp4": "mxfp4 experts + fp8 dense, bf16 elsewhere"}[args.weight_format],
+            "vs_baseline": None if layered else round(value / BASELINE_TOK_S, 1), "dtype": {"bf16": "bf16", "fp8_block": "fp8 e4m3 weights (128x128 scales) + fp8 activations (1x128), bf16 elsewhere", "fp8_mxfp4": "mxfp4 experts + fp8 dense, bf16 elsewhere"}[args.weight_format],
             "data": "synthetic (uniform-random token ids, random-init N(0,0.02) weights)",
             "config": {"model": cfg.name, "global_batch": B, "seq_len": P,
                        "decode_context": "%d..%d (grows one token per step, in both numbers)"
@@ -366,6 +382,8 @@ def main() -> None:
             "device_status": list(status),
             "impl": "ours",
         }
+        if layered:
+            line["config"]["state_bytes_per_sequence"] = runner.states.nbytes // (B * runner.states.buffers)
         if args.layers:
             line["invalid"] = "debug run with a reduced layer count"
         if args.shard_as:
