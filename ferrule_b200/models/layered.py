@@ -197,7 +197,7 @@ class LayeredWorkspace:
                     self.static_plans[i, nt] = p
         L = max_logit_rows
         self.hn_last = torch.zeros(L, Wp, **act)
-        self.logits = torch.zeros(L, cfg.vocab_size, **f32)
+        self.logits = torch.zeros(L, pad_to(cfg.vocab_size, 4), **f32)[:, :cfg.vocab_size]     # 16-byte aligned rows
         self.out_buf = torch.zeros(2 * L, **i32)          # greedy result: [ids | fp32 value bits]
         self.next_id = self.out_buf[:L]
         self.next_val = self.out_buf[L:].view(torch.float32)

@@ -84,6 +84,7 @@ class BatchStaging:
             self.d_start, self.d_state_in, self.d_state_out = (d[lo:hi] for lo, hi in parts)
             # until a batch is filled in: one row per sequence, no state read or kept
             self.np_start[:] = np.arange(seqs + 1)
+            self.np_seq[:] = np.minimum(self._arange, seqs - 1)
             self.np_state_in[:] = -1
             self.np_state_out[:] = -1
             self.n_seqs = seqs
