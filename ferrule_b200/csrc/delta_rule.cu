@@ -31,7 +31,7 @@ struct DeltaParams {
   const float* ag;            // [rows, ldag]: decay pre-activation at 0, output gate pre-activation at off_gate
   long long ldag;
   int off_gate;
-  const float* conv;          // [channels, taps], channels = q | k | v
+  const float* conv;          // [taps, channels], channels = q | k | v
   const float* a_neg;         // [heads]
   const float* dt_bias;       // [heads * dim]
   const float* norm_w;        // [vdim]
@@ -66,7 +66,7 @@ __device__ __forceinline__ float conv_silu(const DeltaParams<T>& p, int c, int r
     float x = 0.f;
     if (idx >= 0) x = act_load(p.proj + (r0 + idx) * p.ldp + col);
     else if (sin >= 0) x = act_load(p.tail + (static_cast<long long>(sin) * (taps - 1) + idx + taps - 1) * channels + c);
-    acc = fmaf(p.conv[c * taps + j], x, acc);
+    acc = fmaf(p.conv[static_cast<long long>(j) * channels + c], x, acc);
   }
   return acc / (1.f + expf(-acc));
 }
@@ -103,14 +103,61 @@ __device__ __forceinline__ bool seq_states(const DeltaParams<T>& p, int seq, int
 }
 
 // ---------------------------------------------------------------------------------
-// prepare: one CTA per row
+// prepare: one CTA per row.  VEC consecutive channels per thread (4 when every block of channels is a multiple of 4)
 // ---------------------------------------------------------------------------------
+__device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float (&v)[4]) {
+  const uint2 a = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&a);
+#pragma unroll
+  for (int j = 0; j < 4; ++j) v[j] = __bfloat162float(e[j]);
+}
+__device__ __forceinline__ void load_vec(const float* p, float (&v)[4]) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
 template <typename T>
+__device__ __forceinline__ void load_vec(const T* p, float (&v)[1]) { v[0] = act_load(p); }
+__device__ __forceinline__ void store_vec(float* p, const float (&v)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+}
+__device__ __forceinline__ void store_vec(float* p, const float (&v)[1]) { p[0] = v[0]; }
+
+// convolution and silu of channels [c0, c0 + n) of one row into `dst`, whose inputs start at column `col0`
+template <int VEC, typename T>
+__device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int n, int col0, int r, int i, int sin,
+                                           int channels, float* dst) {
+  const int keep = p.taps - 1;
+  const T* tail = p.tail + static_cast<long long>(max(sin, 0)) * keep * channels;
+  for (int c = threadIdx.x * VEC; c < n; c += blockDim.x * VEC) {
+    float acc[VEC], x[VEC], w[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+    const T* in = p.proj + r * p.ldp + col0 + c;
+    for (int j = 0; j <= keep; ++j) {
+      const int back = keep - j;                          // tokens before this one
+      load_vec(p.conv + static_cast<long long>(j) * channels + c0 + c, w);
+      if (back <= i) {
+        load_vec(in - back * p.ldp, x);
+      } else {
+        load_vec(tail + static_cast<long long>(i + j) * channels + c0 + c, x);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x[e] = sin >= 0 ? x[e] : 0.f;
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(w[e], x[e], acc[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+    store_vec(dst + c, acc);
+  }
+}
+
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(const DeltaParams<T> p) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float qk_s[];                 // [2 * kv_heads * dim]
+  extern __shared__ __align__(16) float qk_s[];   // [2 * kv_heads * dim]
   const int r = blockIdx.x;
   const int seq = p.row_seq[r];
   if (seq < 0 || seq >= p.n_seqs) {
@@ -125,19 +172,22 @@ delta_prepare_kernel(const DeltaParams<T> p) {
   int sin, sout;
   if (!seq_states(p, seq, sin, sout)) return;
   const int nk = p.kv_heads * p.dim, nv = p.heads * p.vdim, channels = p.channels();
-  for (int c = threadIdx.x; c < channels; c += blockDim.x) {
-    const float y = conv_silu(p, c, r0, i, sin, channels);
-    if (c < 2 * nk) qk_s[c] = y;
-    else p.v[static_cast<long long>(r) * nv + c - 2 * nk] = y;
-    store_tail(p, c, r0, i, n, sin, sout, channels);
+  conv_block<VEC>(p, 0, nk, p.off_q, r, i, sin, channels, qk_s);
+  conv_block<VEC>(p, nk, nk, p.off_k, r, i, sin, channels, qk_s + nk);
+  conv_block<VEC>(p, 2 * nk, nv, p.off_v, r, i, sin, channels, p.v + static_cast<long long>(r) * nv);
+  if (i == 0 || i > n - p.taps)
+    for (int c = threadIdx.x; c < channels; c += blockDim.x) store_tail(p, c, r0, i, n, sin, sout, channels);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  for (int h = warp; h < p.heads; h += nw) {
+    const float a = p.a_neg[h];
+    const float* pre = p.ag + r * p.ldag + h * p.dim;
+    const float* bias = p.dt_bias + h * p.dim;
+    float* dst = p.decay + (static_cast<long long>(r) * p.heads + h) * p.dim;
+    for (int d = lane; d < p.dim; d += 32) dst[d] = expf(a * softplus_f(pre[d] + bias[d]));
   }
-  for (int c = threadIdx.x; c < p.heads * p.dim; c += blockDim.x)
-    p.decay[static_cast<long long>(r) * p.heads * p.dim + c] =
-        expf(p.a_neg[c / p.dim] * softplus_f(p.ag[r * p.ldag + c] + p.dt_bias[c]));
   for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
     p.beta[static_cast<long long>(r) * p.heads + h] = sigmoid_f(act_load(p.proj + r * p.ldp + p.off_b + h));
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   for (int h = warp; h < p.kv_heads; h += nw) {
     const float* q = qk_s + h * p.dim;
     const float* k = qk_s + nk + h * p.dim;
@@ -168,40 +218,44 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 }
 
 // ---------------------------------------------------------------------------------
-// scan: CTA = (head, 16 value columns) x sequence; eight lanes per column, lane l holds the key channels
-// 32 * (j / 4) + 4 * l + j % 4.  Tokens are staged sixteen at a time, double buffered.
+// scan: CTA = (head, 16 * COLS value columns) x sequence; eight lanes share COLS columns, lane l holds the key channels
+// 32 * (j / 4) + 4 * l + j % 4.  Tokens are staged sixteen at a time, double buffered.  More columns per lane mean
+// fewer shared-memory reads of k, q and g per column; the launcher takes as many as still fill the GPU.
 // ---------------------------------------------------------------------------------
-constexpr int kScanStep = 16, kScanCols = 16;
+constexpr int kScanStep = 16;
 
-template <typename T, int RPT>
+template <typename T, int RPT, int COLS>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(const DeltaParams<T> p) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int DP = RPT * 8;                                   // padded key dimension
-  extern __shared__ float sm[];
-  // per buffer: k, q, g [kScanStep][DP], v [kScanStep][kScanCols], beta, qk [kScanStep]
-  constexpr int kBuf = kScanStep * (3 * DP + kScanCols + 2);
+  constexpr int kCols = 16 * COLS;
+  extern __shared__ __align__(16) float sm[];
+  // per buffer: k, q, g [kScanStep][DP], v [kScanStep][kCols], beta, qk [kScanStep]
+  constexpr int kBuf = kScanStep * (3 * DP + kCols + 2);
   const int seq = blockIdx.y;
-  const int vtiles = (p.vdim + kScanCols - 1) / kScanCols;
-  const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * kScanCols;
+  const int vtiles = (p.vdim + kCols - 1) / kCols;
+  const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * kCols;
   const int hk = h / (p.heads / p.kv_heads);
   const int r0 = p.seq_start[seq], n = p.seq_start[seq + 1] - r0;
   if (r0 < 0 || n <= 0 || r0 + n > p.rows) return;              // reported by the prepare kernel
   int sin, sout;
   if (!seq_states(p, seq, sin, sout)) return;
   const int tid = threadIdx.x, l8 = tid & 7;
-  const int vc = tid >> 3, v = v0 + vc;
-  const bool vok = v < p.vdim;
+  const int vc = (tid >> 3) * COLS;                             // first column of this lane inside the tile
   for (int i = tid; i < 2 * kBuf; i += 128) sm[i] = 0.f;        // padding channels stay zero
 
-  float S[RPT];
-  const long long sbase = static_cast<long long>(h) * p.dim * p.vdim + v;
+  float S[COLS][RPT];
   const long long per_state = static_cast<long long>(p.heads) * p.dim * p.vdim;
+  const long long sbase = static_cast<long long>(h) * p.dim * p.vdim + v0 + vc;
 #pragma unroll
   for (int j = 0; j < RPT; ++j) {
     const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
-    S[j] = (sin >= 0 && vok && d < p.dim) ? p.state[sin * per_state + sbase + static_cast<long long>(d) * p.vdim] : 0.f;
+#pragma unroll
+    for (int c = 0; c < COLS; ++c)
+      S[c][j] = (sin >= 0 && v0 + vc + c < p.vdim && d < p.dim)
+                    ? p.state[sin * per_state + sbase + static_cast<long long>(d) * p.vdim + c] : 0.f;
   }
   __syncthreads();
   const long long ldk = static_cast<long long>(p.kv_heads) * p.dim, ldg = static_cast<long long>(p.heads) * p.dim,
@@ -228,14 +282,13 @@ delta_scan_kernel(const DeltaParams<T> p) {
       }
     }
     float* vb = base + 3 * kScanStep * DP;
-    for (int i = tid; i < cnt * kScanCols; i += 128) {
-      const int t = i / kScanCols, c = i - t * kScanCols;
+    for (int i = tid; i < cnt * kCols; i += 128) {
+      const int t = i / kCols, c = i - t * kCols;
       if (v0 + c < p.vdim) cp_async4(vb + i, p.v + (r0 + t0 + t) * ldv + h * p.vdim + v0 + c);
     }
     if (tid < cnt) {
-      cp_async4(vb + kScanStep * kScanCols + tid, p.beta + static_cast<long long>(r0 + t0 + tid) * p.heads + h);
-      cp_async4(vb + kScanStep * kScanCols + kScanStep + tid,
-                p.qk + static_cast<long long>(r0 + t0 + tid) * p.kv_heads + hk);
+      cp_async4(vb + kScanStep * kCols + tid, p.beta + static_cast<long long>(r0 + t0 + tid) * p.heads + h);
+      cp_async4(vb + kScanStep * kCols + kScanStep + tid, p.qk + static_cast<long long>(r0 + t0 + tid) * p.kv_heads + hk);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -253,40 +306,53 @@ delta_scan_kernel(const DeltaParams<T> p) {
     const float* vb = base + 3 * kScanStep * DP;
     const int cnt = min(kScanStep, n - t0);
     for (int t = 0; t < cnt; ++t) {
-      float k[RPT];
-      float sk0 = 0.f, sk1 = 0.f, sq0 = 0.f, sq1 = 0.f;
+      float k[RPT], sk[COLS], sq[COLS], u[COLS];
 #pragma unroll
-      for (int c = 0; c < RPT / 4; ++c) {
-        const int off = t * DP + c * 32 + l8 * 4;
+      for (int c = 0; c < COLS; ++c) sk[c] = sq[c] = 0.f;
+#pragma unroll
+      for (int j = 0; j < RPT / 4; ++j) {
+        const int off = t * DP + j * 32 + l8 * 4;
         const float4 k4 = *reinterpret_cast<const float4*>(base + off);
         const float4 q4 = *reinterpret_cast<const float4*>(base + kScanStep * DP + off);
         const float4 g4 = *reinterpret_cast<const float4*>(base + 2 * kScanStep * DP + off);
-        k[4 * c] = k4.x; k[4 * c + 1] = k4.y; k[4 * c + 2] = k4.z; k[4 * c + 3] = k4.w;
-        S[4 * c] *= g4.x; S[4 * c + 1] *= g4.y; S[4 * c + 2] *= g4.z; S[4 * c + 3] *= g4.w;
-        sk0 = fmaf(S[4 * c], k4.x, sk0); sk1 = fmaf(S[4 * c + 1], k4.y, sk1);
-        sq0 = fmaf(S[4 * c], q4.x, sq0); sq1 = fmaf(S[4 * c + 1], q4.y, sq1);
-        sk0 = fmaf(S[4 * c + 2], k4.z, sk0); sk1 = fmaf(S[4 * c + 3], k4.w, sk1);
-        sq0 = fmaf(S[4 * c + 2], q4.z, sq0); sq1 = fmaf(S[4 * c + 3], q4.w, sq1);
-      }
-      float sk = sk0 + sk1, sq = sq0 + sq1;
+        k[4 * j] = k4.x; k[4 * j + 1] = k4.y; k[4 * j + 2] = k4.z; k[4 * j + 3] = k4.w;
 #pragma unroll
-      for (int o = 1; o < 8; o <<= 1) {
-        sk += __shfl_xor_sync(0xffffffffu, sk, o);
-        sq += __shfl_xor_sync(0xffffffffu, sq, o);
+        for (int c = 0; c < COLS; ++c) {
+          float* s = S[c] + 4 * j;
+          s[0] *= g4.x; s[1] *= g4.y; s[2] *= g4.z; s[3] *= g4.w;
+          sk[c] = fmaf(s[3], k4.w, fmaf(s[2], k4.z, fmaf(s[1], k4.y, fmaf(s[0], k4.x, sk[c]))));
+          sq[c] = fmaf(s[3], q4.w, fmaf(s[2], q4.z, fmaf(s[1], q4.y, fmaf(s[0], q4.x, sq[c]))));
+        }
       }
-      const float u = vb[kScanStep * kScanCols + t] * (vb[t * kScanCols + vc] - sk);
-      if (l8 == 0 && vok)
-        p.o[(r0 + t0 + t) * ldv + h * p.vdim + v] = fmaf(vb[kScanStep * kScanCols + kScanStep + t], u, sq);
 #pragma unroll
-      for (int j = 0; j < RPT; ++j) S[j] = fmaf(k[j], u, S[j]);
+      for (int o = 1; o < 8; o <<= 1)
+#pragma unroll
+        for (int c = 0; c < COLS; ++c) {
+          sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], o);
+          sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], o);
+        }
+      const float beta = vb[kScanStep * kCols + t], qk = vb[kScanStep * kCols + kScanStep + t];
+      float* o = p.o + (r0 + t0 + t) * ldv + h * p.vdim + v0 + vc;
+#pragma unroll
+      for (int c = 0; c < COLS; ++c) {
+        u[c] = beta * (vb[t * kCols + vc + c] - sk[c]);
+        if (l8 == c && v0 + vc + c < p.vdim) o[c] = fmaf(qk, u[c], sq[c]);
+      }
+#pragma unroll
+      for (int c = 0; c < COLS; ++c)
+#pragma unroll
+        for (int j = 0; j < RPT; ++j) S[c][j] = fmaf(k[j], u[c], S[c][j]);
     }
     __syncthreads();
   }
-  if (sout >= 0 && vok) {
+  if (sout >= 0) {
 #pragma unroll
     for (int j = 0; j < RPT; ++j) {
       const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
-      if (d < p.dim) p.state[sout * per_state + sbase + static_cast<long long>(d) * p.vdim] = S[j];
+#pragma unroll
+      for (int c = 0; c < COLS; ++c)
+        if (d < p.dim && v0 + vc + c < p.vdim)
+          p.state[sout * per_state + sbase + static_cast<long long>(d) * p.vdim + c] = S[c][j];
     }
   }
 }
@@ -476,18 +542,30 @@ static int run_decode(const FbDeltaArgs* a, cudaStream_t s) {
   return launched();
 }
 
-template <typename T, int RPT>
-static int launch_scan(const DeltaParams<T>& p, cudaStream_t s) {
-  constexpr int smem = 2 * kScanStep * (3 * RPT * 8 + kScanCols + 2) * static_cast<int>(sizeof(float));
+template <typename T, int RPT, int COLS>
+static int launch_scan_cols(const DeltaParams<T>& p, cudaStream_t s) {
+  constexpr int smem = 2 * kScanStep * (3 * RPT * 8 + 16 * COLS + 2) * static_cast<int>(sizeof(float));
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+        cudaSuccess)
       return FB_ERR_LAUNCH;
     attr = true;
   }
-  const dim3 grid(p.heads * ((p.vdim + kScanCols - 1) / kScanCols), p.n_seqs);
-  launch_pdl(delta_scan_kernel<T, RPT>, grid, dim3(128), smem, s, p);
+  const dim3 grid(p.heads * ((p.vdim + 16 * COLS - 1) / (16 * COLS)), p.n_seqs);
+  launch_pdl(delta_scan_kernel<T, RPT, COLS>, grid, dim3(128), smem, s, p);
   return launched();
+}
+
+template <typename T, int RPT>
+static int launch_scan(const DeltaParams<T>& p, cudaStream_t s) {
+  const long long per_col = static_cast<long long>(p.heads) * p.n_seqs;
+  auto ctas = [&](int cols) { return per_col * ((p.vdim + 16 * cols - 1) / (16 * cols)); };
+  if constexpr (RPT <= 16) {
+    if (ctas(4) >= 120 && p.vdim > 32) return launch_scan_cols<T, RPT, 4>(p, s);
+  }
+  if (ctas(2) >= 120 && p.vdim > 16) return launch_scan_cols<T, RPT, 2>(p, s);
+  return launch_scan_cols<T, RPT, 1>(p, s);
 }
 
 template <typename T>
@@ -499,14 +577,17 @@ static int run_prefill(const FbDeltaArgs* a, cudaStream_t s) {
   if (p.dim > 256 || p.n_seqs > 65535) return FB_ERR_SHAPE;
   const size_t smem = 2ull * p.kv_heads * p.dim * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
-  static bool attr = false;
-  if (!attr) {
-    if (cudaFuncSetAttribute(delta_prepare_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) !=
-        cudaSuccess)
+  const bool vec = (p.kv_heads * p.dim) % 4 == 0 && (p.heads * p.vdim) % 4 == 0 && p.ldp % 4 == 0 && p.off_q % 4 == 0 &&
+                   p.off_k % 4 == 0 && p.off_v % 4 == 0 && (reinterpret_cast<uintptr_t>(p.proj) & 15) == 0 &&
+                   (reinterpret_cast<uintptr_t>(p.tail) & 15) == 0;
+  auto prepare = vec ? delta_prepare_kernel<T, 4> : delta_prepare_kernel<T, 1>;
+  static bool attr[2] = {false, false};
+  if (!attr[vec]) {
+    if (cudaFuncSetAttribute(prepare, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
       return FB_ERR_LAUNCH;
-    attr = true;
+    attr[vec] = true;
   }
-  launch_pdl(delta_prepare_kernel<T>, dim3(p.rows), dim3(256), smem, s, p);
+  launch_pdl(prepare, dim3(p.rows), dim3(256), smem, s, p);
   if ((rc = launched()) != FB_OK) return rc;
   if (p.dim <= 32) rc = launch_scan<T, 4>(p, s);
   else if (p.dim <= 64) rc = launch_scan<T, 8>(p, s);

@@ -239,7 +239,7 @@ typedef struct FbDeltaArgs {
   long long ldag;
   int off_gate;
   int fp32;                 // activations (proj, tail, out) are fp32 instead of bf16
-  const float* conv;        // [2 * kv_heads * dim + heads * vdim, taps]
+  const float* conv;        // [taps, 2 * kv_heads * dim + heads * vdim]
   const float* a_neg;       // [heads] = -exp(A_log)
   const float* dt_bias;     // [heads * dim]
   const float* norm_w;      // [vdim]

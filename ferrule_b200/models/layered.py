@@ -80,7 +80,7 @@ class LayeredReference:
             S = state[sin].clone() if sin >= 0 else torch.zeros(H, D, V)
             x = torch.cat([old, raw[r0:r1]], 0)
             n = r1 - r0
-            y = sum(x[j:j + n] * mx.conv[:, j] for j in range(m.taps))
+            y = sum(x[j:j + n] * mx.conv[j] for j in range(m.taps))
             y = torch.nn.functional.silu(y)
             q, k, v = y[:, :nk].view(n, KV, D), y[:, nk:2 * nk].view(n, KV, D), y[:, 2 * nk:].view(n, H, V)
             unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)

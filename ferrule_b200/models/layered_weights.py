@@ -46,7 +46,7 @@ class MixerImage:
     # delta rule
     w_ag: Optional[torch.Tensor] = None      # [heads * dim | heads * vdim, low ranks]
     off_gate: int = 0
-    conv: Optional[torch.Tensor] = None      # fp32 [channels, taps]
+    conv: Optional[torch.Tensor] = None      # fp32 [taps, channels]
     a_neg: Optional[torch.Tensor] = None     # fp32 [heads] = -exp(A_log)
     dt_bias: Optional[torch.Tensor] = None   # fp32 [heads * dim]
     o_norm: Optional[torch.Tensor] = None    # fp32 [vdim]
@@ -123,8 +123,8 @@ def _pack_delta(m: DeltaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _B
     ag = torch.zeros(nd8 + nv, ra + rg, dtype=a2.dtype, device=a2.device)
     ag[:nd, :m.decay_rank] = a2
     ag[nd8:, ra:ra + m.gate_rank] = g2
-    conv = torch.cat([get(p + n + ".conv").view(-1, m.taps) for n in ("q", "k", "v")], 0).float().contiguous()
-    assert conv.shape[0] == m.channels and nk + nk + nv == m.channels
+    conv = torch.cat([get(p + n + ".conv").view(-1, m.taps) for n in ("q", "k", "v")], 0).float().t().contiguous()
+    assert conv.shape[1] == m.channels and nk + nk + nv == m.channels
     return MixerImage(None, b.off, _pad(get(p + "o"), Wp, pad_to(nv, 8)).contiguous(), w_ag=ag, off_gate=nd8, conv=conv,
                       a_neg=-torch.exp(get(p + "A_log").float()), dt_bias=get(p + "dt_bias").float().contiguous(),
                       o_norm=get(p + "norm").float().contiguous())

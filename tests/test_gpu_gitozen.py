@@ -240,7 +240,7 @@ def delta_case(dtype, m, lens, old, seed=0):
         at += pad(n)
     img = type("Img", (), {})()
     img.off_gate = pad(nd)
-    img.conv, img.a_neg = rnd(m.channels, m.taps, seed=seed + 1), -torch.exp(rnd(m.heads, seed=seed + 2))
+    img.conv, img.a_neg = rnd(m.taps, m.channels, seed=seed + 1), -torch.exp(rnd(m.heads, seed=seed + 2))
     img.dt_bias, img.o_norm = rnd(nd, seed=seed + 3) - 2, rnd(m.vdim, seed=seed + 4)
     n_states = 2 * len(lens) + 1
     case = dict(proj=rnd(T, at, dtype=dtype, seed=seed + 5), off=off, ag=rnd(T, img.off_gate + nv, seed=seed + 6), img=img, mixer=m,
@@ -259,7 +259,7 @@ def delta_want(case, lens, old):
     nk, nv, keep = m.kv_heads * m.dim, m.heads * m.vdim, m.taps - 1
     proj, ag = case["proj"].double().cpu(), case["ag"].double().cpu()
     raw = torch.cat([proj[:, off["q"]:off["q"] + nk], proj[:, off["k"]:off["k"] + nk], proj[:, off["v"]:off["v"] + nv]], 1)
-    conv, share = img.conv.double().cpu(), [h // (m.heads // m.kv_heads) for h in range(m.heads)]
+    conv, share = img.conv.double().cpu().T, [h // (m.heads // m.kv_heads) for h in range(m.heads)]
     outs, states, tails, at = [], [], [], 0
     for i, n in enumerate(lens):
         r = slice(at, at + n)
