@@ -102,6 +102,22 @@ __device__ __forceinline__ bool seq_states(const DeltaParams<T>& p, int seq, int
   return true;
 }
 
+// exp(a * softplus(z)) and silu(z).  bf16 models take the hardware exponential and logarithm (a few 1e-7 relative, far
+// below the rounding of z itself), fp32 models the full-precision functions.
+template <typename T>
+__device__ __forceinline__ float decay_of(float a, float z) {
+  if constexpr (sizeof(T) == 4) return expf(a * softplus_f(z));
+  const float e = __expf(-fabsf(z)), w = 1.f + e;
+  // log1p(e) = log(w) * e / (w - 1): the quotient restores what rounding w lost
+  const float l = w == 1.f ? e : __logf(w) * __fdividef(e, w - 1.f);
+  return __expf(a * (fmaxf(z, 0.f) + l));
+}
+template <typename T>
+__device__ __forceinline__ float silu_of(float z) {
+  if constexpr (sizeof(T) == 4) return z / (1.f + expf(-z));
+  return __fdividef(z, 1.f + __expf(-z));
+}
+
 // ---------------------------------------------------------------------------------
 // prepare: one CTA per row.  VEC consecutive channels per thread (4 when every block of channels is a multiple of 4)
 // ---------------------------------------------------------------------------------
@@ -133,6 +149,23 @@ __device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int 
 #pragma unroll
     for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
     const T* in = p.proj + r * p.ldp + col0 + c;
+    if (keep <= 3 && i >= keep) {
+      // every tap lies in this batch: all loads go out together
+      float xs[4][VEC], wf[4][VEC];
+#pragma unroll
+      for (int b = 0; b < 4; ++b) {
+        if (b <= keep) {
+          load_vec(in - b * p.ldp, xs[b]);
+          load_vec(p.conv + static_cast<long long>(keep - b) * channels + c0 + c, wf[b]);
+        }
+      }
+#pragma unroll
+      for (int b = 3; b >= 0; --b)
+        if (b <= keep) {
+#pragma unroll
+          for (int e = 0; e < VEC; ++e) acc[e] = fmaf(wf[b][e], xs[b][e], acc[e]);
+        }
+    } else
     for (int j = 0; j <= keep; ++j) {
       const int back = keep - j;                          // tokens before this one
       load_vec(p.conv + static_cast<long long>(j) * channels + c0 + c, w);
@@ -147,7 +180,7 @@ __device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int 
       for (int e = 0; e < VEC; ++e) acc[e] = fmaf(w[e], x[e], acc[e]);
     }
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+    for (int e = 0; e < VEC; ++e) acc[e] = silu_of<T>(acc[e]);
     store_vec(dst + c, acc);
   }
 }
@@ -155,7 +188,7 @@ __device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 delta_prepare_kernel(const DeltaParams<T> p) {
-  pdl_launch_dependents();
+  // no early release: the scan's CTAs would be packed onto the first SMs with room instead of spreading over all
   pdl_wait();
   extern __shared__ __align__(16) float qk_s[];   // [2 * kv_heads * dim]
   const int r = blockIdx.x;
@@ -183,7 +216,7 @@ delta_prepare_kernel(const DeltaParams<T> p) {
     const float* pre = p.ag + r * p.ldag + h * p.dim;
     const float* bias = p.dt_bias + h * p.dim;
     float* dst = p.decay + (static_cast<long long>(r) * p.heads + h) * p.dim;
-    for (int d = lane; d < p.dim; d += 32) dst[d] = expf(a * softplus_f(pre[d] + bias[d]));
+    for (int d = lane; d < p.dim; d += 32) dst[d] = decay_of<T>(a, pre[d] + bias[d]);
   }
   for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
     p.beta[static_cast<long long>(r) * p.heads + h] = sigmoid_f(act_load(p.proj + r * p.ldp + p.off_b + h));
@@ -224,10 +257,30 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 // ---------------------------------------------------------------------------------
 constexpr int kScanStep = 16;
 
+// two fp32 lanes in one 64-bit register: one instruction for two multiply-adds, each rounded as the scalar one
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& a, float& b) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 template <typename T, int RPT, int COLS>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(const DeltaParams<T> p) {
-  pdl_launch_dependents();
+  // the dependents are released at the end: their CTAs would only wait, on the SMs this long kernel needs
   pdl_wait();
   constexpr int DP = RPT * 8;                                   // padded key dimension
   constexpr int kCols = 16 * COLS;
@@ -246,16 +299,18 @@ delta_scan_kernel(const DeltaParams<T> p) {
   const int vc = (tid >> 3) * COLS;                             // first column of this lane inside the tile
   for (int i = tid; i < 2 * kBuf; i += 128) sm[i] = 0.f;        // padding channels stay zero
 
-  float S[COLS][RPT];
+  uint64_t S[COLS][RPT / 2];                                    // pairs of neighbouring key channels
   const long long per_state = static_cast<long long>(p.heads) * p.dim * p.vdim;
   const long long sbase = static_cast<long long>(h) * p.dim * p.vdim + v0 + vc;
 #pragma unroll
-  for (int j = 0; j < RPT; ++j) {
+  for (int j = 0; j < RPT; j += 2) {
     const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
+    const float* src = p.state + max(sin, 0) * per_state + sbase + static_cast<long long>(d) * p.vdim;
 #pragma unroll
-    for (int c = 0; c < COLS; ++c)
-      S[c][j] = (sin >= 0 && v0 + vc + c < p.vdim && d < p.dim)
-                    ? p.state[sin * per_state + sbase + static_cast<long long>(d) * p.vdim + c] : 0.f;
+    for (int c = 0; c < COLS; ++c) {
+      const bool in = sin >= 0 && v0 + vc + c < p.vdim;
+      S[c][j / 2] = pack2(in && d < p.dim ? src[c] : 0.f, in && d + 1 < p.dim ? src[p.vdim + c] : 0.f);
+    }
   }
   __syncthreads();
   const long long ldk = static_cast<long long>(p.kv_heads) * p.dim, ldg = static_cast<long long>(p.heads) * p.dim,
@@ -305,54 +360,81 @@ delta_scan_kernel(const DeltaParams<T> p) {
     const float* base = sm + b * kBuf;
     const float* vb = base + 3 * kScanStep * DP;
     const int cnt = min(kScanStep, n - t0);
-    for (int t = 0; t < cnt; ++t) {
-      float k[RPT], sk[COLS], sq[COLS], u[COLS];
-#pragma unroll
-      for (int c = 0; c < COLS; ++c) sk[c] = sq[c] = 0.f;
+    uint64_t k[RPT / 2], q[RPT / 2], g[RPT / 2];
+    auto fetch = [&](int t) {
 #pragma unroll
       for (int j = 0; j < RPT / 4; ++j) {
-        const int off = t * DP + j * 32 + l8 * 4;
-        const float4 k4 = *reinterpret_cast<const float4*>(base + off);
-        const float4 q4 = *reinterpret_cast<const float4*>(base + kScanStep * DP + off);
-        const float4 g4 = *reinterpret_cast<const float4*>(base + 2 * kScanStep * DP + off);
-        k[4 * j] = k4.x; k[4 * j + 1] = k4.y; k[4 * j + 2] = k4.z; k[4 * j + 3] = k4.w;
-#pragma unroll
-        for (int c = 0; c < COLS; ++c) {
-          float* s = S[c] + 4 * j;
-          s[0] *= g4.x; s[1] *= g4.y; s[2] *= g4.z; s[3] *= g4.w;
-          sk[c] = fmaf(s[3], k4.w, fmaf(s[2], k4.z, fmaf(s[1], k4.y, fmaf(s[0], k4.x, sk[c]))));
-          sq[c] = fmaf(s[3], q4.w, fmaf(s[2], q4.z, fmaf(s[1], q4.y, fmaf(s[0], q4.x, sq[c]))));
-        }
+        const float* row = base + t * DP + j * 32 + l8 * 4;
+        const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(row);
+        const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(row + kScanStep * DP);
+        const ulonglong2 e = *reinterpret_cast<const ulonglong2*>(row + 2 * kScanStep * DP);
+        k[2 * j] = a.x; k[2 * j + 1] = a.y;
+        q[2 * j] = c.x; q[2 * j + 1] = c.y;
+        g[2 * j] = e.x; g[2 * j + 1] = e.y;
       }
-#pragma unroll
-      for (int o = 1; o < 8; o <<= 1)
-#pragma unroll
-        for (int c = 0; c < COLS; ++c) {
-          sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], o);
-          sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], o);
-        }
+    };
+    fetch(0);
+    float* o = p.o + (r0 + t0) * ldv + h * p.vdim + v0 + vc + l8;
+    const bool writer = l8 < COLS && v0 + vc + l8 < p.vdim;
+    for (int t = 0; t < cnt; ++t, o += ldv) {
       const float beta = vb[kScanStep * kCols + t], qk = vb[kScanStep * kCols + kScanStep + t];
-      float* o = p.o + (r0 + t0 + t) * ldv + h * p.vdim + v0 + vc;
+      float sk[COLS], sq[COLS], vt[COLS], out = 0.f;
+#pragma unroll
+      for (int c = 0; c < COLS; ++c) vt[c] = vb[t * kCols + vc + c];
 #pragma unroll
       for (int c = 0; c < COLS; ++c) {
-        u[c] = beta * (vb[t * kCols + vc + c] - sk[c]);
-        if (l8 == c && v0 + vc + c < p.vdim) o[c] = fmaf(qk, u[c], sq[c]);
+        uint64_t ka = 0, kb = 0, qa = 0, qb = 0;          // two chains each
+#pragma unroll
+        for (int j = 0; j < RPT / 2; j += 2) {
+          S[c][j] = mul2(S[c][j], g[j]);
+          S[c][j + 1] = mul2(S[c][j + 1], g[j + 1]);
+          ka = fma2(S[c][j], k[j], ka);
+          kb = fma2(S[c][j + 1], k[j + 1], kb);
+          qa = fma2(S[c][j], q[j], qa);
+          qb = fma2(S[c][j + 1], q[j + 1], qb);
+        }
+        float a0, a1, b0, b1;
+        unpack2(ka, a0, a1);
+        unpack2(kb, b0, b1);
+        sk[c] = (a0 + b0) + (a1 + b1);
+        unpack2(qa, a0, a1);
+        unpack2(qb, b0, b1);
+        sq[c] = (a0 + b0) + (a1 + b1);
       }
 #pragma unroll
-      for (int c = 0; c < COLS; ++c)
+      for (int x = 1; x < 8; x <<= 1)
 #pragma unroll
-        for (int j = 0; j < RPT; ++j) S[c][j] = fmaf(k[j], u[c], S[c][j]);
+        for (int c = 0; c < COLS; ++c) {
+          sk[c] += __shfl_xor_sync(0xffffffffu, sk[c], x);
+          sq[c] += __shfl_xor_sync(0xffffffffu, sq[c], x);
+        }
+#pragma unroll
+      for (int c = 0; c < COLS; ++c) {
+        const float u = beta * (vt[c] - sk[c]);
+        if (l8 == c) out = fmaf(qk, u, sq[c]);
+        const uint64_t u2 = pack2(u, u);
+#pragma unroll
+        for (int j = 0; j < RPT / 2; ++j) S[c][j] = fma2(k[j], u2, S[c][j]);
+      }
+      fetch(min(t + 1, kScanStep - 1));
+      if (writer) *o = out;
     }
     __syncthreads();
   }
+  pdl_launch_dependents();
   if (sout >= 0) {
 #pragma unroll
-    for (int j = 0; j < RPT; ++j) {
+    for (int j = 0; j < RPT; j += 2) {
       const int d = (j / 4) * 32 + l8 * 4 + (j & 3);
+      float* dst = p.state + sout * per_state + sbase + static_cast<long long>(d) * p.vdim;
 #pragma unroll
-      for (int c = 0; c < COLS; ++c)
-        if (d < p.dim && v0 + vc + c < p.vdim)
-          p.state[sout * per_state + sbase + static_cast<long long>(d) * p.vdim + c] = S[c][j];
+      for (int c = 0; c < COLS; ++c) {
+        if (v0 + vc + c >= p.vdim) continue;
+        float a0, a1;
+        unpack2(S[c][j / 2], a0, a1);
+        if (d < p.dim) dst[c] = a0;
+        if (d + 1 < p.dim) dst[p.vdim + c] = a1;
+      }
     }
   }
 }
@@ -369,6 +451,25 @@ delta_output_kernel(const DeltaParams<T> p) {
   const long long r = i / p.heads;
   const int h = static_cast<int>(i - r * p.heads);
   const float* o = p.o + i * p.vdim;
+  if (p.vdim <= 128 && (p.vdim & 3) == 0 && (p.ldag & 3) == 0 && (p.off_gate & 3) == 0) {
+    // four columns per lane, everything requested up front
+    const int v = lane * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), g = a, w = a;
+    if (v < p.vdim) {
+      a = *reinterpret_cast<const float4*>(o + v);
+      g = *reinterpret_cast<const float4*>(p.ag + r * p.ldag + p.off_gate + h * p.vdim + v);
+      w = *reinterpret_cast<const float4*>(p.norm_w + v);
+    }
+    const float inv = 1.f / sqrtf(warp_sum(a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w) / p.vdim + p.eps);
+    if (v < p.vdim) {
+      T* dst = p.out + r * p.ldo + h * p.vdim + v;
+      act_store(dst, a.x * inv * w.x * sigmoid_f(g.x));
+      act_store(dst + 1, a.y * inv * w.y * sigmoid_f(g.y));
+      act_store(dst + 2, a.z * inv * w.z * sigmoid_f(g.z));
+      act_store(dst + 3, a.w * inv * w.w * sigmoid_f(g.w));
+    }
+    return;
+  }
   float ss = 0.f;
   for (int v = lane; v < p.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
   ss = warp_sum(ss);
