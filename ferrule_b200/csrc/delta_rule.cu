@@ -121,18 +121,19 @@ __device__ __forceinline__ float silu_of(float z) {
 // ---------------------------------------------------------------------------------
 // prepare: one CTA per row.  VEC consecutive channels per thread (4 when every block of channels is a multiple of 4)
 // ---------------------------------------------------------------------------------
+// (reads of memory the kernel never writes: independent iterations may then be in flight together)
 __device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float (&v)[4]) {
-  const uint2 a = *reinterpret_cast<const uint2*>(p);
+  const uint2 a = __ldg(reinterpret_cast<const uint2*>(p));
   const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&a);
 #pragma unroll
   for (int j = 0; j < 4; ++j) v[j] = __bfloat162float(e[j]);
 }
 __device__ __forceinline__ void load_vec(const float* p, float (&v)[4]) {
-  const float4 a = *reinterpret_cast<const float4*>(p);
+  const float4 a = __ldg(reinterpret_cast<const float4*>(p));
   v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
 }
-template <typename T>
-__device__ __forceinline__ void load_vec(const T* p, float (&v)[1]) { v[0] = act_load(p); }
+__device__ __forceinline__ void load_vec(const __nv_bfloat16* p, float (&v)[1]) { v[0] = __bfloat162float(__ldg(p)); }
+__device__ __forceinline__ void load_vec(const float* p, float (&v)[1]) { v[0] = __ldg(p); }
 __device__ __forceinline__ void store_vec(float* p, const float (&v)[4]) {
   *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
 }
@@ -144,6 +145,7 @@ __device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int 
                                            int channels, float* dst) {
   const int keep = p.taps - 1;
   const T* tail = p.tail + static_cast<long long>(max(sin, 0)) * keep * channels;
+#pragma unroll 2
   for (int c = threadIdx.x * VEC; c < n; c += blockDim.x * VEC) {
     float acc[VEC], x[VEC], w[VEC];
 #pragma unroll
@@ -172,9 +174,10 @@ __device__ __forceinline__ void conv_block(const DeltaParams<T>& p, int c0, int 
       if (back <= i) {
         load_vec(in - back * p.ldp, x);
       } else {
-        load_vec(tail + static_cast<long long>(i + j) * channels + c0 + c, x);
+        // (the tails are written by this launch: plain loads)
 #pragma unroll
-        for (int e = 0; e < VEC; ++e) x[e] = sin >= 0 ? x[e] : 0.f;
+        for (int e = 0; e < VEC; ++e)
+          x[e] = sin >= 0 ? act_load(tail + static_cast<long long>(i + j) * channels + c0 + c + e) : 0.f;
       }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) acc[e] = fmaf(w[e], x[e], acc[e]);
@@ -216,7 +219,8 @@ delta_prepare_kernel(const DeltaParams<T> p) {
     const float* pre = p.ag + r * p.ldag + h * p.dim;
     const float* bias = p.dt_bias + h * p.dim;
     float* dst = p.decay + (static_cast<long long>(r) * p.heads + h) * p.dim;
-    for (int d = lane; d < p.dim; d += 32) dst[d] = decay_of<T>(a, pre[d] + bias[d]);
+#pragma unroll 4
+    for (int d = lane; d < p.dim; d += 32) dst[d] = decay_of<T>(a, __ldg(pre + d) + __ldg(bias + d));
   }
   for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
     p.beta[static_cast<long long>(r) * p.heads + h] = sigmoid_f(act_load(p.proj + r * p.ldp + p.off_b + h));
@@ -483,6 +487,39 @@ delta_output_kernel(const DeltaParams<T> p) {
 // decode: CTA = (sequence, head), 8 warps; lane l holds the value columns 4l .. 4l + 3, warp w the key channels
 // w, w + 8, ...  Needs vdim <= 128, vdim % 4 == 0, dim <= 8 * RW.
 // ---------------------------------------------------------------------------------
+// convolution and silu of channel c for the only row of its sequence; with `keep_inputs` also the tail for the next step
+template <typename T>
+__device__ __forceinline__ float conv_step(const DeltaParams<T>& p, int c, int r, int sin, int sout, int channels,
+                                           bool keep_inputs) {
+  const int keep = p.taps - 1;
+  if (keep > 3) {
+    if (keep_inputs) store_tail(p, c, r, 0, 1, sin, sout, channels);
+    return conv_silu(p, c, r, 0, sin, channels);
+  }
+  // inputs and taps are requested together; x[keep] is the current token's input
+  float x[4], w[4], acc = 0.f;
+  const T* old = p.tail + static_cast<long long>(max(sin, 0)) * keep * channels + c;
+#pragma unroll
+  for (int b = 0; b < 4; ++b) {
+    x[b] = w[b] = 0.f;
+    if (b < keep && sin >= 0) x[b] = act_load(old + static_cast<long long>(b) * channels);
+    if (b <= keep) w[b] = p.conv[static_cast<long long>(b) * channels + c];
+  }
+  const float cur = act_load(p.proj + r * p.ldp + p.col(c));
+#pragma unroll
+  for (int b = 0; b < 4; ++b) {
+    if (b == keep) x[b] = cur;
+    if (b <= keep) acc = fmaf(w[b], x[b], acc);
+  }
+  if (keep_inputs && sout >= 0) {
+    T* dst = p.tail + static_cast<long long>(sout) * keep * channels + c;
+#pragma unroll
+    for (int b = 0; b < 3; ++b)
+      if (b < keep) act_store(dst + static_cast<long long>(b) * channels, x[b + 1]);
+  }
+  return silu_of<T>(acc);
+}
+
 template <typename T, int RW>
 __global__ void __launch_bounds__(256)
 delta_decode_kernel(const DeltaParams<T> p) {
@@ -515,31 +552,19 @@ delta_decode_kernel(const DeltaParams<T> p) {
   }
   const int nk = p.kv_heads * p.dim, channels = p.channels();
   const int first = h % (p.heads / p.kv_heads) == 0;         // this CTA also keeps the shared q / k inputs
-  for (int d = tid; d < 8 * RW; d += 256) {
-    float q = 0.f, k = 0.f, g = 0.f;
-    if (d < p.dim) {
-      const int cq = hk * p.dim + d, ck = nk + cq;
-      q = conv_silu(p, cq, r, 0, sin, channels);
-      k = conv_silu(p, ck, r, 0, sin, channels);
-      if (first) {
-        store_tail(p, cq, r, 0, 1, sin, sout, channels);
-        store_tail(p, ck, r, 0, 1, sin, sout, channels);
-      }
-      const int c = h * p.dim + d;
-      g = expf(p.a_neg[h] * softplus_f(p.ag[r * p.ldag + c] + p.dt_bias[c]));
-    }
-    s_q[d] = q;
-    s_k[d] = k;
-    s_g[d] = g;
-  }
-  for (int v = tid; v < 128; v += 256) {
+  // channels of this head: q (8 RW entries, zero past dim) | k | v, then the decays
+  for (int i = tid; i < 16 * RW + 128; i += 256) {
+    const int part = i < 8 * RW ? 0 : (i < 16 * RW ? 1 : 2), d = part == 2 ? i - 16 * RW : i - part * 8 * RW;
     float y = 0.f;
-    if (v < p.vdim) {
-      const int c = 2 * nk + h * p.vdim + v;
-      y = conv_silu(p, c, r, 0, sin, channels);
-      store_tail(p, c, r, 0, 1, sin, sout, channels);
+    if (d < (part == 2 ? p.vdim : p.dim)) {
+      const int c = part == 2 ? 2 * nk + h * p.vdim + d : part * nk + hk * p.dim + d;
+      y = conv_step(p, c, r, sin, sout, channels, part == 2 || first);
     }
-    s_v[v] = y;
+    (part == 0 ? s_q : part == 1 ? s_k : s_v)[d] = y;
+  }
+  for (int d = tid; d < 8 * RW; d += 256) {
+    const int c = h * p.dim + d;
+    s_g[d] = d < p.dim ? decay_of<T>(p.a_neg[h], p.ag[r * p.ldag + c] + p.dt_bias[c]) : 0.f;
   }
   __syncthreads();
   // norms of q and k, their product: every warp computes them for itself
