@@ -43,6 +43,12 @@ CUDA_SOURCES = [
     "comm_mm.cu",
     "no_alloc.cu",
 ]
+# Sources one program needs: a program that serves one model family from a tree without a built library compiles this
+# much instead of everything (into a library of its own; the full library is used when it is there).
+COMPONENTS = {
+    "layered": ["gemm_tcgen05.cu", "mla_attention.cu", "mla_prefill_tc.cu", "elementwise.cu", "data_movers.cu",
+                "layered_ops.cu", "delta_rule.cu", "gemm_f32.cu"],
+}
 CXX_SOURCES = [
     "host/kv_page_manager.cpp",
     "host/direct_reader.cpp",
@@ -79,24 +85,33 @@ def _digest(paths) -> str:
     return h.hexdigest()
 
 
-def sources():
-    cu = [CSRC / n for n in _existing(CUDA_SOURCES)]
-    cxx = [CSRC / n for n in _existing(CXX_SOURCES)]
+def lib_path(component: str = "") -> Path:
+    return OUT_DIR / f"libferrule_b200_{component}.so" if component else LIB_PATH
+
+
+def sources(component: str = ""):
+    cu = [CSRC / n for n in _existing(COMPONENTS[component] if component else CUDA_SOURCES)]
+    cxx = [] if component else [CSRC / n for n in _existing(CXX_SOURCES)]
     hdr = sorted(CSRC.glob("*.h")) + sorted(CSRC.glob("*.cuh")) + sorted((CSRC / "host").glob("*.h"))
     return cu, cxx, hdr
 
 
-def is_current() -> bool:
-    cu, cxx, hdr = sources()
-    stamp = OUT_DIR / "build.sha256"
-    return LIB_PATH.exists() and stamp.exists() and stamp.read_text().strip() == _digest(cu + cxx + hdr)
+def _stamp(component: str) -> Path:
+    return OUT_DIR / (f"build_{component}.sha256" if component else "build.sha256")
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile and link the native library; returns its path."""
-    cu, cxx, hdr = sources()
-    if not force and is_current():
-        return LIB_PATH
+def is_current(component: str = "") -> bool:
+    cu, cxx, hdr = sources(component)
+    stamp = _stamp(component)
+    return lib_path(component).exists() and stamp.exists() and stamp.read_text().strip() == _digest(cu + cxx + hdr)
+
+
+def build(force: bool = False, verbose: bool = False, component: str = "") -> Path:
+    """Compile and link the native library (or one component of it); returns its path."""
+    cu, cxx, hdr = sources(component)
+    path = lib_path(component)
+    if not force and is_current(component):
+        return path
     OUT_DIR.mkdir(exist_ok=True)
     obj_dir = OUT_DIR / "obj"
     obj_dir.mkdir(exist_ok=True)
@@ -118,14 +133,14 @@ def build(force: bool = False, verbose: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 2)) as ex:
         objs = list(ex.map(compile_one, cu + cxx))
-    tmp = LIB_PATH.with_suffix(".so.tmp")
+    tmp = path.with_suffix(".so.tmp")
     cmd = [nvcc, "-shared", "-o", str(tmp), *map(str, objs), "-lpthread"]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
         raise RuntimeError(f"link failed\n{r.stdout}\n{r.stderr}")
-    os.replace(tmp, LIB_PATH)
-    (OUT_DIR / "build.sha256").write_text(_digest(cu + cxx + hdr))
-    return LIB_PATH
+    os.replace(tmp, path)
+    _stamp(component).write_text(_digest(cu + cxx + hdr))
+    return path
 
 
 if __name__ == "__main__":

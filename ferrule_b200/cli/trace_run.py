@@ -40,6 +40,8 @@ def build_replay(model_dir: str, dtype: str, max_tokens: int, device: str, page_
             raise SystemExit(3)
         device = device if ":" in device else "cuda:0"
         torch.cuda.set_device(torch.device(device))
+        from ..ops import _lib
+        _lib.use_component(arch.component)
     weights = arch.load(model_dir, device, dt)
     pages = (max_tokens + page_size - 1) // page_size
     ctx = (pages + 1) * page_size

@@ -32,6 +32,7 @@ class Architecture:
     load: Callable[..., object]                                  # (directory, device, dtype, max_layers) -> weights
     runner: Callable[..., object]                                # (weights, limits, **options) -> ModelRunner
     dtypes: tuple = (torch.bfloat16,)                            # dtypes its kernel path runs in
+    component: str = ""                                          # part of the native library it needs ("": all of it)
 
 
 def _load_gitozen(directory, device, dtype, max_layers=0):
@@ -69,7 +70,7 @@ def _run_deepseek(weights, lim: RunnerLimits, **options):
 
 ARCHITECTURES: Dict[str, Architecture] = {a.name: a for a in (
     Architecture("gitozen", lambda c: c.get("architecture") == "Gitozen", _load_gitozen, _run_layered,
-                 (torch.bfloat16, torch.float32)),
+                 (torch.bfloat16, torch.float32), "layered"),
     Architecture("deepseek_v4", lambda c: c.get("model_type") == "deepseek_v4", _load_v4, _run_v4),
     # every other HuggingFace-style config.json is read as a DeepSeek-V2 / V3 model, whose loader checks it
     Architecture("deepseek", lambda c: "architecture" not in c, _load_deepseek, _run_deepseek),

@@ -114,6 +114,16 @@ class DeltaArgs(C.Structure):
 _lock = threading.Lock()
 _lib: Optional[C.CDLL] = None
 _tried = False
+_component = ""
+
+
+def use_component(name: str) -> None:
+    """For programs that need one part of the library: without a built full library, `get_lib` builds and loads this
+    component (`_build.COMPONENTS`) instead of everything.  Call before the first `get_lib`."""
+    global _component
+    if name and name not in _build.COMPONENTS:
+        raise ValueError(f"unknown library component {name!r}")
+    _component = name
 
 
 def _declare(lib: C.CDLL) -> None:
@@ -164,7 +174,7 @@ def get_lib(required: Optional[bool] = None) -> Optional[C.CDLL]:
             if not path.exists():
                 if os.environ.get("FERRULE_NO_BUILD"):
                     raise NativeLibraryError(f"{path} is missing and FERRULE_NO_BUILD is set")
-                _build.build()
+                path = _build.build(component=_component)
             lib = C.CDLL(str(path))
             _declare(lib)
             _lib = lib
