@@ -142,7 +142,7 @@ def test_gemm_in_32_bits(ops, case):
         near(out.view(T, k, 48), want, F32)
 
 
-@pytest.mark.parametrize("E,groups,keep,top", [(8, 2, 1, 3), (6, 3, 2, 2), (64, 8, 3, 6), (5, 5, 2, 2), (7, 1, 1, 3)])
+@pytest.mark.parametrize("E,groups,keep,top", [(10, 2, 1, 3), (6, 3, 2, 2), (64, 8, 3, 6), (5, 5, 2, 2), (7, 1, 1, 3)])
 def test_router_groups_by_their_best_expert(ops, E, groups, keep, top):
     K = ops[0]
     logits = rnd(40, E, scale=2.0)
@@ -279,7 +279,7 @@ def delta_want(case, lens, old):
     return torch.cat(outs), states, tails
 
 
-MIXERS = [DeltaMixer(4, 4, 64, 32, 4), DeltaMixer(4, 2, 20, 12, 3), DeltaMixer(6, 1, 8, 4, 1), DeltaMixer(2, 2, 72, 33, 5),
+MIXERS = [DeltaMixer(3, 3, 64, 48, 4), DeltaMixer(4, 2, 20, 12, 3), DeltaMixer(6, 1, 8, 4, 1), DeltaMixer(2, 2, 72, 33, 5),
           DeltaMixer(2, 1, 128, 128, 4), DeltaMixer(1, 1, 130, 100, 2), DeltaMixer(3, 3, 128, 160, 4), DeltaMixer(2, 2, 31, 64, 4)]
 
 
@@ -338,7 +338,7 @@ def test_state_rotation(ops):
 
 # ------------------------------------------------------------------ whole models
 WIDE = LayeredConfig(vocab_size=200, width=128, layers=(
-    LayerSpec(LatentMixer(16, 24, 16, 512, 0.4), MoeSpec(8, 2, 48, 2, 1)),
+    LayerSpec(LatentMixer(16, 24, 16, 512, 0.4), MoeSpec(9, 2, 48, 3, 1)),
     LayerSpec(DeltaMixer(2, 1, 128, 128, 4, 16, 16), MoeSpec(16, 4, 24, 4, 2))), logit_softcap=8.0)
 ALL = {**CONFIGS, "wide": WIDE}
 _memo = {}
