@@ -120,7 +120,7 @@ def build_engine(args, layout=None):
         args.model_dir = args.model
     from ..models import layered_config as LC
     arch = _architecture(args.model_dir)
-    if arch == "gitozen" or (not args.model_dir and args.preset in LC.PRESETS):
+    if arch in LC.ARCHITECTURES or (not args.model_dir and args.preset in LC.PRESETS):
         return _build_layered_engine(args, dev, args.model_dir, layout)
     if arch == "deepseek_v4":
         return _build_v4_engine(args, dev, args.model_dir)
@@ -229,7 +229,7 @@ def _expert_plan(args):
 
 
 def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=None):
-    """A layer-list model (Gitozen) behind the engine: a checkpoint directory, or a random-init preset."""
+    """A layer-list model (Gitozen, Supisun) behind the engine: a checkpoint directory, or a random-init preset."""
     import torch
 
     from ..models.layered_config import PRESETS
@@ -247,7 +247,7 @@ def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=Non
     if getattr(args, "weight_format", "bf16") != "bf16":
         raise SystemExit("--weight-format: layer-list models run bf16 weights")
     args.speculative = False
-    arch = ARCHITECTURES["gitozen"]
+    arch = ARCHITECTURES[_architecture(model_dir) if model_dir else ("supisun" if "supisun" in args.preset else "gitozen")]
     dtype = torch.bfloat16 if dev != "cpu" else torch.float32
     if model_dir:
         weights = arch.load(model_dir, dev, dtype, max_layers=getattr(args, "layers", 0))
@@ -262,7 +262,7 @@ def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=Non
     ctx, pages_per_seq, sched = _engine_sizes(args, cfg.max_position)
     n_pages = args.max_seqs * pages_per_seq + 8
     if args.kv_cache_mb:
-        per_page = max(len(cfg.latent_layers), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
+        per_page = max(len(cfg.cache_layers), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
         n_pages = max(args.kv_cache_mb * (1 << 20) // per_page, pages_per_seq + 1)
     runner = arch.runner(weights, RunnerLimits(n_pages, args.page_size, args.max_batch_tokens, args.max_seqs, ctx), device=dev)
     eng = Engine(runner, EngineConfig(scheduler=sched, kv_pages=n_pages, page_size=args.page_size))
@@ -336,7 +336,7 @@ def cmd_info(args) -> int:
                 "policies": {k: enc(getattr(ps, k)) for k in ("attention", "router", "expert", "quant", "kv", "residency",
                                                              "parallelism", "speculation")}}
     arch = _architecture(args.model_dir)
-    if arch == "gitozen":
+    if arch in LC.ARCHITECTURES:
         from ..io.layered_checkpoint import bind_config
         from ..io.safetensors import ShardedCheckpoint
         from ..models.families import detect_family, layout_summary
@@ -446,17 +446,17 @@ def cmd_make_fixture(args) -> int:
         print(json.dumps({"written": args.out, "family": "deepseek_v4", "layers": cfg.n_layers,
                           "proposal_stages": cfg.n_proposal_stages, "dense_format": dense, "expert_format": expert}))
         return 0
-    if args.family == "gitozen":
+    if args.family in ("gitozen", "supisun"):
         from ..io.layered_checkpoint import export_layered
         from ..models.layered_config import PRESETS
         from ..models.layered_weights import RandomTensors
-        lcfg = PRESETS[args.preset if args.preset in PRESETS else "tiny-gitozen"]()
+        lcfg = PRESETS[args.preset if args.preset in PRESETS else f"tiny-{args.family}"]()
         if args.layers:
             lcfg = lcfg.with_(layers=tuple(lcfg.layers[i % lcfg.n_layers] for i in range(args.layers)))
         if args.dense_format != "plain" or args.expert_format != "plain":
-            raise SystemExit("--family gitozen: checkpoints are stored in BF16")
+            raise SystemExit(f"--family {args.family}: checkpoints are stored in BF16")
         export_layered(lcfg, RandomTensors(lcfg, args.seed, gain=0.0 if args.zeros else 1.0), args.out, args.shard_mb << 20)
-        print(json.dumps({"written": args.out, "family": "gitozen", "params": lcfg.param_count(), "layers": lcfg.n_layers}))
+        print(json.dumps({"written": args.out, "family": args.family, "params": lcfg.param_count(), "layers": lcfg.n_layers}))
         return 0
     cfg = C.PRESETS[args.preset]()
     if args.layers:
@@ -887,9 +887,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--zeros", action="store_true"); p.add_argument("--shard-mb", type=int, default=1024)
     p.add_argument("--dense-format", default="plain", choices=["plain", "fp8_block"])
     p.add_argument("--expert-format", default="plain", choices=["plain", "fp8_block", "mxfp4"])
-    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", "gitozen"],
+    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", "gitozen", "supisun"],
                    help="v4: a DeepSeek-V4 directory (tiny shape; FP8 dense + packed FP4 experts unless --plain); "
-                        "gitozen: a layer-list directory (--preset tiny-gitozen unless another of its presets is named)")
+                        "gitozen, supisun: a layer-list directory (--preset tiny-<family> unless another of its presets is named)")
     p.add_argument("--plain", action="store_true", help="--family v4: keep every linear in BF16")
     p.add_argument("--proposal-stages", type=int, default=0,
                    help="--family v4: also write this many `mtp.*` proposal stages with their prediction heads")

@@ -1,5 +1,5 @@
-"""Checkpoint directories of layer-list models (Gitozen): `config.json` with one entry per layer, and safetensors files
-whose tensors are named `embed`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.rg1`, `final.norm`, `head`
+"""Checkpoint directories of layer-list models (Gitozen, Supisun): `config.json` with one entry per layer, and safetensors
+files whose tensors are named `embed`, `pos`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.rg1`, `final.norm`, `head`
 (`LayeredConfig.tensor_shapes` lists them).  Linear weights are stored [out, in] in BF16."""
 from __future__ import annotations
 
@@ -20,6 +20,8 @@ def bind_config(cfg: LayeredConfig, ck: ShardedCheckpoint) -> LayeredConfig:
     for i in cfg.delta_layers:
         m = layers[i].mixer
         assert isinstance(m, DeltaMixer)
+        if not m.low_rank:
+            continue
         ranks = {}
         for field, tensor in (("decay_rank", "a1"), ("gate_rank", "g1")):
             name = f"l{i}.mix.{tensor}"

@@ -4,7 +4,8 @@ Roles tell the loader what a tensor is (attention projection, norm, router, rout
 weight, scale, MTP part ...) independent of the naming scheme.  Families: DeepSeek (HuggingFace
 V2/V3 names: `model.layers.N.self_attn.q_a_proj.weight`), DeepSeek-V4 (the reference's flat names:
 `layers.N.attn.wq_a.weight`, `ffn.experts.E.w1.weight`, `mtp.M.*`), Gitozen (layer-list names:
-`lN.mix.q`, `lN.mlp.eE.gate`), Qwen3 and generic Llama-style.  The DeepSeek families and Gitozen execute; the others
+`lN.mix.q`, `lN.mlp.eE.gate`), Supisun (the same scheme), Qwen3 and generic Llama-style.  The DeepSeek families and
+the layer-list ones execute; the others
 are classified for inspection.
 
 Counterpart of crates/ferrule-model/src/families/mod.rs:20-115, families/deepseek_v4.rs:9-300 and
@@ -59,6 +60,11 @@ class TensorRole(Enum):
     DELTA_BETA = "delta_beta"
     DELTA_GATE = "delta_gate"
     DELTA_NORM = "delta_norm"
+    SCAN_IN = "scan_in"
+    SCAN_PARAM = "scan_param"
+    INPUT_CONV = "input_conv"
+    POSITION = "position"
+    VALUE_MIX = "value_mix"
     MTP = "mtp"
     SCALE = "scale"
     UNKNOWN = "unknown"
@@ -77,6 +83,7 @@ class Family(Enum):
     DEEPSEEK_HF = "deepseek_hf"
     DEEPSEEK_V4 = "deepseek_v4"
     GITOZEN = "gitozen"
+    SUPISUN = "supisun"
     QWEN3 = "qwen3"
     LLAMA = "llama"
 
@@ -101,20 +108,30 @@ _LAYERED_MIX = {"q": TensorRole.ATTN_Q, "k": TensorRole.ATTN_K, "v": TensorRole.
                 "k.conv": TensorRole.DELTA_CONV, "v.conv": TensorRole.DELTA_CONV, "b": TensorRole.DELTA_BETA,
                 "A_log": TensorRole.DELTA_DECAY, "a1": TensorRole.DELTA_DECAY, "a2": TensorRole.DELTA_DECAY,
                 "dt_bias": TensorRole.DELTA_DECAY, "g1": TensorRole.DELTA_GATE, "g2": TensorRole.DELTA_GATE,
-                "norm": TensorRole.DELTA_NORM}
+                "norm": TensorRole.DELTA_NORM, "a": TensorRole.DELTA_DECAY, "q.norm": TensorRole.ATTN_Q_NORM,
+                "k.norm": TensorRole.ATTN_KV_NORM, "vmix": TensorRole.VALUE_MIX, "in": TensorRole.SCAN_IN,
+                "conv": TensorRole.SCAN_PARAM, "conv.b": TensorRole.SCAN_PARAM, "x": TensorRole.SCAN_PARAM,
+                "dt": TensorRole.SCAN_PARAM, "dt.b": TensorRole.SCAN_PARAM, "D": TensorRole.SCAN_PARAM}
 _LAYERED_FFN = {"gate": 0, "up": 1, "down": 2}
 
 
 def _classify_layered(name: str) -> "TensorClass":
-    top = {"embed": TensorRole.EMBEDDING, "final.norm": TensorRole.FINAL_NORM, "head": TensorRole.OUTPUT_HEAD}
+    top = {"embed": TensorRole.EMBEDDING, "pos": TensorRole.POSITION, "final.norm": TensorRole.FINAL_NORM,
+           "final.norm.b": TensorRole.FINAL_NORM, "head": TensorRole.OUTPUT_HEAD}
     if name in top:
         return TensorClass(top[name])
     m = re.match(r"l(\d+)\.(.*)", name)
     if not m:
         return TensorClass(TensorRole.UNKNOWN)
     layer, rest = int(m.group(1)), m.group(2)
-    if rest == "norm1":
+    if rest in ("norm1", "norm1.b"):
         return TensorClass(TensorRole.ATTN_NORM, layer)
+    if rest in ("norm2", "norm2.b"):
+        return TensorClass(TensorRole.FFN_NORM, layer)
+    if rest == "canon1":
+        return TensorClass(TensorRole.INPUT_CONV, layer)
+    if rest in ("mlp.up", "mlp.down"):
+        return TensorClass(_ffn_role("dense", _LAYERED_FFN[rest[4:]]), layer)
     if re.fullmatch(r"rg[12](\.b)?", rest):
         return TensorClass(TensorRole.RESIDUAL_GATE, layer)
     if rest == "mlp.router":
@@ -135,7 +152,7 @@ def _ffn_role(kind: str, idx: int) -> TensorRole:
 
 
 def classify(name: str, family: Family, n_layers: Optional[int] = None) -> TensorClass:
-    if family == Family.GITOZEN:
+    if family in (Family.GITOZEN, Family.SUPISUN):
         return _classify_layered(name)
     is_scale = name.endswith(_SCALE_SUFFIX)
     base = name
@@ -231,6 +248,8 @@ def classify(name: str, family: Family, n_layers: Optional[int] = None) -> Tenso
 
 def detect_family(names: Iterable[str], model_type: str = "") -> Family:
     names = list(names)
+    if "l0.canon1" in names or model_type.lower() == "supisun":
+        return Family.SUPISUN
     if "l0.norm1" in names or model_type.lower() == "gitozen":
         return Family.GITOZEN
     if any(n.startswith("layers.") and ".attn.wq_a" in n for n in names) or any(n.startswith("mtp.") for n in names):

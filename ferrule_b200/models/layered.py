@@ -1,32 +1,54 @@
-"""Forward pass of layer-list models over a packed ragged batch (paged latent pool + recurrent-state pool).
+"""Forward pass of layer-list models over a packed ragged batch (paged pool + recurrent-state pool).
+
+Parallel gated blocks:
 
     x = embed[token]                                             (residual stream, fp32)
     per layer:  h = RMSNorm(x) * g
                 x += sigmoid(rg1 h + b1) * mixer(h) + sigmoid(rg2 h + b2) * ff(h)
     logits = softcap(head . RMSNorm(x) * g_final)
 
+Output-norm blocks:
+
+    x = embed[token] + pos[position]
+    per layer:  x += norm1(mixer(x + conv(x)))                   (conv: short causal convolution, one filter per channel)
+                x += norm2(ff(x))
+    logits = head . norm_final(x)
+
 * `LayeredReference` - plain PyTorch; the execution path of a CPU runner.
 * `LayeredCuda`      - the sm_100a kernel pipeline, allocation-free over a preallocated workspace, so a decode step can be
   captured in a CUDA graph.  With fp32 weights the same pipeline runs in full 32 bits.
 
 Kernels of a latent layer: input projection (one GEMM for q, latent, gates) -> latent append -> W_uk absorption ->
-attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o.  Of a delta layer: input projection -> second
-low-rank halves -> delta rule -> W_o.  The feed-forward branch reads the same h and runs on a second stream beside
-the mixer: router (+ row reservation) -> grouped SwiGLU GEMM -> grouped scatter GEMM.  One kernel joins both branches:
-gated residual additions, expert reduction, next layer's norm.
+attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o.  Of an attention layer: input projection (q, k,
+v) -> norms, rotation, value mixing and cache append in one launch -> attention -> W_o.  Of a delta layer: input projection
+-> second low-rank halves -> delta rule -> W_o.  Of a selective-scan layer: input projection -> convolution -> W_x -> W_dt
+-> scan (step sizes, skip and output gate inside) -> W_o.
+
+In a parallel gated block the feed-forward branch reads the same h and runs on a second stream beside the mixer: router
+(+ row reservation) -> grouped SwiGLU GEMM -> grouped scatter GEMM.  One kernel joins both branches: gated residual
+additions, expert reduction, next layer's norm.  In an output-norm block one kernel after each sublayer normalises its
+output, adds it to the stream and leaves the rows the next GEMM reads; in decode steps it also applies the next mixer's
+input convolution, whose earlier inputs are in the state pool then.
 """
 from __future__ import annotations
 
 from typing import Dict, Optional
 
 import torch
+import torch.nn.functional as F
 
 from ..ops import reference as ref
 from .config import SCORE_SOFTMAX
 from .deepseek import DeviceBatch, KvPool, _pow2_at_least
-from .layered_config import LatentMixer, pad_to
+from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, MambaMixer,
+                             MoeSpec, pad_to)
 from .layered_weights import LayerImage, LayeredWeights, MixerImage
 from .state_pool import RecurrentStatePool
+
+
+def rotation_frequencies(base: float, dims: int) -> torch.Tensor:
+    """Angle per position of every rotated pair of a head (double)."""
+    return base ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / max(dims, 1))
 
 
 # ======================================================================================
@@ -35,7 +57,7 @@ from .state_pool import RecurrentStatePool
 class LayeredReference:
     def __init__(self, weights: LayeredWeights, pool: KvPool, states: RecurrentStatePool):
         self.w, self.cfg, self.pool, self.states = weights, weights.cfg, pool, states
-        self.latent_index = {l: i for i, l in enumerate(self.cfg.latent_layers)}
+        self.cache_index = {l: i for i, l in enumerate(self.cfg.cache_layers)}
         self.prof = self.tap = None
 
     def _norm(self, x: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
@@ -50,7 +72,7 @@ class LayeredReference:
         q = proj[:, o["q"]:o["q"] + m.heads * dp].view(T, m.heads, dp)
         c = proj[:, o["dkv"]:o["dkv"] + m.kv_rank]
         c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps) * mx.kv_norm[:m.kv_rank]
-        pool = self.pool.layer(self.latent_index[layer]).view(-1, DL)
+        pool = self.pool.layer(self.cache_index[layer]).view(-1, DL)
         slots = b.write_slot[:T]
         ok = slots >= 0
         pool[slots[ok], :m.kv_rank] = c[ok].to(pool.dtype)
@@ -66,10 +88,15 @@ class LayeredReference:
         T, o = proj.shape[0], mx.off
         H, KV, D, V = m.heads, m.kv_heads, m.dim, m.vdim
         nk, nv, keep = KV * D, H * V, m.taps - 1
-        low = proj[:, o["a1"]:o["a1"] + mx.w_ag.shape[1]]
-        ag = low @ mx.w_ag.float().T
+        nd = H if m.head_decay else H * D
+        if m.low_rank:
+            ag = proj[:, o["a1"]:o["a1"] + mx.w_ag.shape[1]] @ mx.w_ag.float().T
+            pre, gate = ag[:, :nd], ag[:, mx.off_gate:mx.off_gate + nv]
+        else:
+            pre, gate = proj[:, o["a"]:o["a"] + nd], proj[:, o["g"]:o["g"] + nv]
+        gate = torch.sigmoid(gate) if m.gate == "sigmoid" else F.silu(gate)
         raw = torch.cat([proj[:, o["q"]:o["q"] + nk], proj[:, o["k"]:o["k"] + nk], proj[:, o["v"]:o["v"] + nv]], 1)
-        decay = torch.exp(mx.a_neg[:, None] * torch.nn.functional.softplus(ag[:, :H * D] + mx.dt_bias).view(T, H, D))
+        decay = torch.exp(mx.a_neg[:, None] * F.softplus(pre + mx.dt_bias).view(T, H, nd // H))
         beta = torch.sigmoid(proj[:, o["b"]:o["b"] + H])
         state, tail = self.states.state[layer], self.states.tail[layer]
         out = torch.zeros(T, mx.w_o.shape[1])
@@ -81,7 +108,7 @@ class LayeredReference:
             x = torch.cat([old, raw[r0:r1]], 0)
             n = r1 - r0
             y = sum(x[j:j + n] * mx.conv[j] for j in range(m.taps))
-            y = torch.nn.functional.silu(y)
+            y = F.silu(y)
             q, k, v = y[:, :nk].view(n, KV, D), y[:, nk:2 * nk].view(n, KV, D), y[:, 2 * nk:].view(n, H, V)
             unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
             q = (unit(q) * D ** -0.5).repeat_interleave(H // KV, 1)
@@ -92,7 +119,7 @@ class LayeredReference:
                 S = S + k[i][:, :, None] * u[:, None, :]
                 oi = torch.einsum("hdv,hd->hv", S, q[i])
                 oi = oi * torch.rsqrt(oi.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps) * mx.o_norm
-                out[r0 + i, :nv] = (oi * torch.sigmoid(ag[r0 + i, mx.off_gate:].view(H, V))).reshape(-1)
+                out[r0 + i, :nv] = (oi * gate[r0 + i].view(H, V)).reshape(-1)
             if sout >= 0:
                 state[sout] = S
                 if keep:
@@ -111,32 +138,128 @@ class LayeredReference:
             if rows.numel() == 0:
                 continue
             y = h[rows] @ lw.e_w13[e].float().T
-            y = (torch.nn.functional.silu(y[:, :fp]) * y[:, fp:]) @ lw.e_w2[e].float().T
+            y = (F.silu(y[:, :fp]) * y[:, fp:]) @ lw.e_w2[e].float().T
             out[rows] += y * (wts * hit)[rows].sum(-1, keepdim=True)
         return out
 
+    def _conv(self, x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        """Causal convolution of packed rows x [T, channels] with w [taps, channels]; inputs before a sequence's first
+        row come from its state, which is brought up to date."""
+        keep, out = w.shape[0] - 1, torch.empty_like(x)
+        for s in range(b.n_seqs):
+            r0, r1 = int(b.seq_start[s]), int(b.seq_start[s + 1])
+            sin, sout = int(b.state_in[s]), int(b.state_out[s])
+            old = tail[sin, :keep].float() if (sin >= 0 and keep) else torch.zeros(keep, x.shape[1])
+            xs = torch.cat([old, x[r0:r1]], 0)
+            out[r0:r1] = sum(xs[j:j + r1 - r0] * w[j] for j in range(keep + 1))
+            if sout >= 0 and keep:
+                tail[sout, :keep] = xs[-keep:].to(tail.dtype)
+        return out
+
+    def _attention(self, layer: int, mx: MixerImage, m: AttentionMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        T, o, eps = proj.shape[0], mx.off, self.cfg.norm_eps
+        H, G, D, V, dp, vp = m.heads, m.kv_heads, m.dim, m.vdim, m.dim_pad, m.vdim_pad
+        part = lambda name, heads, pad, d: proj[:, o[name]:o[name] + heads * pad].view(T, heads, pad)[:, :, :d]
+        rms = lambda t, dims: t * torch.rsqrt(t.pow(2).mean(dims, keepdim=True) + eps)
+        q = rms(part("q", H, dp, D), (1, 2)) * mx.q_norm.view(H, dp)[:, :D]
+        k = rms(part("k", G, dp, D), (1, 2)) * mx.k_norm.view(G, dp)[:, :D]
+        v = rms(part("v", G, vp, V), (2,))
+        half = m.rot_dims // 2
+        a = b.positions[:T].double()[:, None] * rotation_frequencies(m.rot_base, m.rot_dims)
+        c, sn = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+
+        def turn(t):
+            u, w = t[:, :, :half], t[:, :, half:2 * half]
+            return torch.cat([u * c - w * sn, w * c + u * sn, t[:, :, 2 * half:]], -1)
+
+        slots = b.write_slot[:T]
+        ok = slots >= 0
+        rows = self.pool.layer(self.cache_index[layer]).view(-1, self.cfg.kv_row_dim)
+        first = self.cfg.first_value_layer
+        if m.v_mix and layer != first:
+            fm = self.cfg.layers[first].mixer
+            fv = self.pool.layer(self.cache_index[first]).view(-1, self.cfg.kv_row_dim)[slots.clamp(min=0)]
+            fv = fv[:, fm.v_offset:fm.v_offset + G * vp].view(T, G, vp)[:, :, :V].float()
+            v = (1 - mx.v_mix) * v + mx.v_mix * fv
+        row = torch.zeros(T, rows.shape[1])
+        row[:, :m.v_offset].view(T, G, dp)[:, :, :D] = turn(k)
+        row[:, m.v_offset:m.v_offset + G * vp].view(T, G, vp)[:, :, :V] = v
+        rows[slots[ok]] = row[ok].to(rows.dtype)
+        q, out, ps = turn(q), torch.zeros(T, H, vp), self.pool.page_size
+        for r in range(T):
+            p, seq = int(b.row_pos[r]), int(b.row_seq[r])
+            t = torch.arange(max(p, 0) // m.chunk * m.chunk, p + 1)
+            if t.numel() == 0:
+                continue
+            kv = rows[b.block_table[seq, t // ps].long() * ps + t % ps].float()
+            k = kv[:, :m.v_offset].view(-1, G, dp)[:, :, :D]
+            v = kv[:, m.v_offset:m.v_offset + G * vp].view(-1, G, vp)
+            w = torch.softmax(torch.einsum("ghd,tgd->ght", q[r].view(G, H // G, D), k) * m.scale, -1)
+            out[r] = torch.einsum("ght,tgv->ghv", w, v).reshape(H, vp)
+        return out.view(T, H * vp) @ mx.w_o.float().T
+
+    def _mamba(self, layer: int, mx: MixerImage, m: MambaMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        o, Ip, N = mx.off, m.inner_pad, m.state
+        x = F.silu(self._conv(proj[:, o["x"]:o["x"] + Ip], mx.conv, self.states.tail[layer], b) + mx.conv_b)
+        low = x @ mx.w_x.float().T
+        dt = F.softplus(low[:, :mx.w_dt.shape[1]] @ mx.w_dt.float().T + mx.dt_bias)
+        B, C = low[:, mx.off_b:mx.off_b + N], low[:, mx.off_c:mx.off_c + N]
+        state, y = self.states.state[layer], torch.empty_like(x)
+        for s in range(b.n_seqs):
+            sin, sout = int(b.state_in[s]), int(b.state_out[s])
+            S = state[sin].clone() if sin >= 0 else torch.zeros(N, Ip)
+            for r in range(int(b.seq_start[s]), int(b.seq_start[s + 1])):
+                S = torch.exp2(dt[r] * mx.a_log2) * S + B[r][:, None] * (dt[r] * x[r])
+                y[r] = C[r] @ S + mx.d_skip * x[r]
+            if sout >= 0:
+                state[sout] = S
+        return (y * F.silu(proj[:, o["z"]:o["z"] + Ip])) @ mx.w_o.float().T
+
+    def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        m = lw.spec.mixer
+        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, DeltaMixer: self._delta,
+              MambaMixer: self._mamba}[type(m)]
+        return fn(layer, lw.mixer, m, proj, b)
+
+    def _gated_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        Wp, mx = self.cfg.width_pad, lw.mixer
+        h = self._norm(x, lw.norm)
+        proj = h @ mx.w_in.float().T
+        y = self._mixer(i, lw, proj, b)
+        y = y * torch.sigmoid(proj[:, mx.off["rg1"]:mx.off["rg1"] + Wp] + lw.rg1_b)
+        if lw.spec.mlp is not None:
+            y = y + self._moe(lw, h) * torch.sigmoid(proj[:, mx.off["rg2"]:mx.off["rg2"] + Wp] + lw.rg2_b)
+        return x + y
+
+    def _layer_norm(self, x: torch.Tensor, wb: torch.Tensor) -> torch.Tensor:
+        W, out = self.cfg.width, torch.zeros_like(x)
+        out[:, :W] = F.layer_norm(x[:, :W], (W,), wb[0, :W], wb[1, :W], self.cfg.norm_eps)
+        return out
+
+    def _output_norm_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        h = x + self._conv(x, lw.canon, self.states.canon[i], b) if lw.canon is not None else x
+        x = x + self._layer_norm(self._mixer(i, lw, h @ lw.mixer.w_in.float().T, b), lw.norm1)
+        if lw.spec.mlp is not None:
+            x = x + self._layer_norm(F.gelu(x @ lw.w_up.float().T) @ lw.w_down.float().T, lw.norm2)
+        return x
+
     def hidden_states(self, b: DeviceBatch, allreduce=None, start_layer: int = 0, h0=None) -> torch.Tensor:
         """Residual stream after the last layer [rows, width_pad]."""
-        Wp = self.cfg.width_pad
         x = self.w.embed[b.token_ids[:b.n_rows].long()].float()
+        if self.w.pos is not None:
+            x = x + self.w.pos[b.positions[:b.n_rows].long()].float()
+        layer = self._gated_layer if self.cfg.block == PARALLEL_GATED else self._output_norm_layer
         for i, lw in enumerate(self.w.layers):
             if self.prof is not None:
                 self.prof.mark(i, "layer")
-            mx = lw.mixer
-            h = self._norm(x, lw.norm)
-            proj = h @ mx.w_in.float().T
-            m = lw.spec.mixer
-            y = (self._latent if isinstance(m, LatentMixer) else self._delta)(i, mx, m, proj, b)
-            y = y * torch.sigmoid(proj[:, mx.off["rg1"]:mx.off["rg1"] + Wp] + lw.rg1_b)
-            if lw.spec.mlp is not None:
-                y = y + self._moe(lw, h) * torch.sigmoid(proj[:, mx.off["rg2"]:mx.off["rg2"] + Wp] + lw.rg2_b)
-            x = x + y
+            x = layer(i, lw, x, b)
             if self.tap is not None:
                 self.tap.write(i, "layer_out", x)
         return x
 
     def logits_from_hidden(self, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
-        logits = self._norm(x[b.logit_rows[:b.n_logit].long()], self.w.final_norm) @ self.w.lm_head.float().T
+        norm = self._norm if self.cfg.block == PARALLEL_GATED else self._layer_norm
+        logits = norm(x[b.logit_rows[:b.n_logit].long()], self.w.final_norm) @ self.w.lm_head.float().T
         cap = self.cfg.logit_softcap
         return cap * torch.tanh(logits / cap) if cap else logits
 
@@ -242,7 +365,7 @@ class LayeredCuda:
         K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
         mx, m = lw.mixer, lw.spec.mixer
         DL, dp, vp = cfg.kv_row_dim, pad_to(m.dim, 8), pad_to(m.vdim, 8)
-        pool = self.pool.layer(self.latent_index[layer])
+        pool = self.pool.layer(self.cache_index[layer])
         KL.latent_append(proj[:, mx.off["dkv"]:], m.kv_rank, mx.kv_norm, cfg.norm_eps, b.write_slot[:T], pool)
         q = proj[:, mx.off["q"]:mx.off["q"] + m.heads * dp]
         q_lat = self._view(ws.q_lat, T, m.heads * DL)

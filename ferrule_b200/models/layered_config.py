@@ -1,23 +1,34 @@
 """Layer-list models: every layer names its own mixer and feed-forward, with its own sizes.
 
-`LayeredConfig` is a sequence of `LayerSpec`s over one residual width.  A layer is parallel: one RMS norm feeds the
-mixer and the feed-forward, both results are gated element by element and added to a 32-bit residual stream.  Mixers:
+`LayeredConfig` is a sequence of `LayerSpec`s over one residual width (a 32-bit residual stream) and a block form:
 
-  LatentMixer   latent attention without positions: keys and values are linear images of one normalised latent row per
-                token (the only thing cached), causal softmax, one output gate per head
-  DeltaMixer    gated delta rule: short causal convolutions, unit-norm queries and keys, one decay per key channel,
-                a [dim, vdim] state per head, gated per-head output norm
+  PARALLEL_GATED  one RMS norm feeds the mixer and the feed-forward, both results are gated element by element
+  OUTPUT_NORM     the mixer, then the feed-forward, each reading the stream itself; a norm (layer norm with weight and
+                  bias) on the sublayer's output before it is added.  With `canon_taps` the mixer reads the stream plus
+                  a short causal convolution of it
 
-Feed-forward: routed experts (softmax scores, group-limited top-k) or none.
+Mixers:
 
-`from_layer_list` reads the `config.json` of the Gitozen architecture, whose checkpoints are stored this way.
+  LatentMixer     latent attention without positions: keys and values are linear images of one normalised latent row
+                  per token (the only thing cached), causal softmax, one output gate per head
+  AttentionMixer  grouped-query attention inside position-aligned chunks: query and key norm over the whole
+                  projection, partial rotation, value norm, values mixed with those of the first mixing layer
+  DeltaMixer      gated delta rule: short causal convolutions, unit-norm queries and keys, one decay per key channel
+                  or per head, a [dim, vdim] state per head, gated per-head output norm
+  MambaMixer      selective scan: short causal convolution, per-channel step sizes, an [inner, state] diagonal recurrence
+
+Feed-forward: routed experts (softmax scores, group-limited top-k), dense with GELU, or none.
+
+`from_layer_list` reads the `config.json` of the architectures whose checkpoints are stored this way: Gitozen
+(PARALLEL_GATED; latent attention, delta rule with channel decays, experts) and Supisun (OUTPUT_NORM; chunked attention,
+selective scan, delta rule with head decays, dense feed-forward, learned positions).
 """
 from __future__ import annotations
 
 import json
 from dataclasses import asdict, dataclass, replace
 from pathlib import Path
-from typing import Dict, Optional, Tuple, Union
+from typing import Callable, Dict, Optional, Tuple, Union
 
 
 def pad_to(n: int, m: int) -> int:
@@ -41,21 +52,76 @@ class LatentMixer:
 
 
 @dataclass(frozen=True)
+class AttentionMixer:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int                     # a query sees the keys of its own chunk of positions only
+    rot_base: float
+    rot_dims: int                  # leading dimensions of a head that are rotated (halves paired)
+    v_mix: bool = False
+
+    kind = "attention"
+
+    @property
+    def dim_pad(self) -> int:
+        return pad_to(self.dim, 8)
+
+    @property
+    def vdim_pad(self) -> int:
+        return pad_to(self.vdim, 8)
+
+    @property
+    def v_offset(self) -> int:
+        """First value column of a cache row: [kv_heads][dim_pad] keys | [kv_heads][vdim_pad] values."""
+        return self.kv_heads * self.dim_pad
+
+    @property
+    def row_dim(self) -> int:
+        return pad_to(self.kv_heads * (self.dim_pad + self.vdim_pad), 8)
+
+
+@dataclass(frozen=True)
 class DeltaMixer:
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     taps: int
-    decay_rank: int = 16           # inner width of the two low-rank projections (a checkpoint's tensors say which)
-    gate_rank: int = 16
+    decay_rank: int = 16           # inner width of the two low-rank projections (a checkpoint's tensors say which);
+    gate_rank: int = 16            # 0: one full projection
+    head_decay: bool = False       # one decay per head instead of one per key channel
+    gate: str = "sigmoid"          # output gate's activation: sigmoid or silu
 
-    kind = "channel_delta"
+    @property
+    def kind(self) -> str:
+        return "delta" if self.head_decay else "channel_delta"
+
+    @property
+    def low_rank(self) -> bool:
+        return self.decay_rank > 0
 
     @property
     def channels(self) -> int:
         """Convolved channels: q | k | v."""
         return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class MambaMixer:
+    inner: int
+    state: int
+    dt_rank: int
+    taps: int
+
+    kind = "mamba1"
+    heads = 1
+
+    @property
+    def inner_pad(self) -> int:
+        return pad_to(self.inner, 8)
 
 
 @dataclass(frozen=True)
@@ -67,13 +133,24 @@ class MoeSpec:
     keep: int = 1
 
 
-Mixer = Union[LatentMixer, DeltaMixer]
+@dataclass(frozen=True)
+class DenseSpec:
+    """W_down gelu(W_up x), the exact (error-function) GELU."""
+    ff: int
+
+    experts = top = 0
+
+
+Mixer = Union[LatentMixer, AttentionMixer, DeltaMixer, MambaMixer]
+
+PARALLEL_GATED = "parallel_gated"
+OUTPUT_NORM = "output_norm"
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
-    mlp: Optional[MoeSpec]
+    mlp: Union[MoeSpec, DenseSpec, None]
 
 
 @dataclass(frozen=True)
@@ -86,7 +163,10 @@ class LayeredConfig:
     name: str = "gitozen"
     eos_token_id: int = -1              # the architecture names no special tokens
     bos_token_id: int = -1
-    max_position: int = 1 << 20         # no positional encoding: the cache is the only limit
+    max_position: int = 1 << 20         # without positional encoding the cache is the only limit
+    block: str = PARALLEL_GATED
+    canon_taps: int = 0                 # OUTPUT_NORM: taps of the mixers' input convolution, 0: none
+    learned_positions: bool = False     # a table of `max_position` vectors is added to the embedding
 
     n_mtp_layers = 0
     attn_sink = False
@@ -113,9 +193,27 @@ class LayeredConfig:
         return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, DeltaMixer))
 
     @property
+    def attention_layers(self) -> Tuple[int, ...]:
+        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, AttentionMixer))
+
+    @property
+    def mamba_layers(self) -> Tuple[int, ...]:
+        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, MambaMixer))
+
+    @property
+    def cache_layers(self) -> Tuple[int, ...]:
+        """Layers with a row per token in the paged pool."""
+        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, (LatentMixer, AttentionMixer)))
+
+    @property
+    def first_value_layer(self) -> int:
+        """The layer whose values the later value-mixing layers mix in, -1: none."""
+        return next((i for i in self.attention_layers if self.layers[i].mixer.v_mix), -1)
+
+    @property
     def kv_row_dim(self) -> int:
-        """Row width of the latent pool: the widest latent of any layer."""
-        return max((self.layers[i].mixer.row_dim for i in self.latent_layers), default=64)
+        """Row width of the paged pool: the widest row of any layer."""
+        return max((self.layers[i].mixer.row_dim for i in self.cache_layers), default=64)
 
     @property
     def n_heads(self) -> int:
@@ -132,31 +230,63 @@ class LayeredConfig:
     def tensor_shapes(self) -> Dict[str, Tuple[int, ...]]:
         """Checkpoint tensor name -> shape, in storage order."""
         W = self.width
+        gated = self.block == PARALLEL_GATED
         out: Dict[str, Tuple[int, ...]] = {"embed": (self.vocab_size, W)}
+        if self.learned_positions:
+            out["pos"] = (self.max_position, W)
         for i, l in enumerate(self.layers):
             p, m = f"l{i}.", l.mixer
             x = p + "mix."
-            out[p + "norm1"] = ()
+            if gated:
+                out[p + "norm1"] = ()
+            else:
+                for n in ("norm1", "norm2")[:2 if l.mlp else 1]:
+                    out.update({p + n: (W,), p + n + ".b": (W,)})
             if isinstance(m, LatentMixer):
                 out.update({x + "q": (m.heads * m.dim, W), x + "dkv": (m.kv_rank, W), x + "dkv.norm": (m.kv_rank,),
                             x + "uk": (m.heads * m.dim, m.kv_rank), x + "uv": (m.heads * m.vdim, m.kv_rank),
                             x + "g": (m.heads, W), x + "o": (W, m.heads * m.vdim)})
+            elif isinstance(m, AttentionMixer):
+                nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+                out.update({x + "q": (nq, W), x + "k": (nk, W), x + "v": (nv, W), x + "q.norm": (nq,), x + "k.norm": (nk,)})
+                if m.v_mix:
+                    out[x + "vmix"] = ()
+                out[x + "o"] = (W, m.heads * m.vdim)
+            elif isinstance(m, MambaMixer):
+                out.update({x + "in": (2 * m.inner, W), x + "conv": (m.inner, m.taps), x + "conv.b": (m.inner,),
+                            x + "x": (m.dt_rank + 2 * m.state, m.inner), x + "dt": (m.inner, m.dt_rank),
+                            x + "dt.b": (m.inner,), x + "A_log": (m.inner, m.state), x + "D": (m.inner,),
+                            x + "o": (W, m.inner)})
             else:
                 nk, nv = m.kv_heads * m.dim, m.heads * m.vdim
                 out.update({x + "q": (nk, W), x + "q.conv": (nk, m.taps), x + "k": (nk, W), x + "k.conv": (nk, m.taps),
                             x + "v": (nv, W), x + "v.conv": (nv, m.taps), x + "b": (m.heads, W), x + "A_log": (m.heads,),
-                            x + "norm": (m.vdim,), x + "a1": (m.decay_rank, W), x + "a2": (m.heads * m.dim, m.decay_rank),
-                            x + "dt_bias": (m.heads * m.dim,), x + "g1": (m.gate_rank, W), x + "g2": (nv, m.gate_rank),
-                            x + "o": (W, nv)})
-            if l.mlp:
+                            x + "norm": (m.vdim,)})
+                decays = m.heads if m.head_decay else m.heads * m.dim
+                if m.low_rank:
+                    out.update({x + "a1": (m.decay_rank, W), x + "a2": (decays, m.decay_rank), x + "dt_bias": (decays,),
+                                x + "g1": (m.gate_rank, W), x + "g2": (nv, m.gate_rank)})
+                else:
+                    out.update({x + "a": (decays, W), x + "dt_bias": (decays,), x + "g": (nv, W)})
+                out[x + "o"] = (W, nv)
+            if isinstance(l.mlp, MoeSpec):
                 for e in range(l.mlp.experts):
                     q = f"{p}mlp.e{e}."
                     out.update({q + "gate": (l.mlp.ff, W), q + "up": (l.mlp.ff, W), q + "down": (W, l.mlp.ff)})
                 out[p + "mlp.router"] = (l.mlp.experts, W)
-            out.update({p + "rg1": (W, W), p + "rg1.b": (W,)})
-            if l.mlp:
-                out.update({p + "rg2": (W, W), p + "rg2.b": (W,)})
-        out.update({"final.norm": (), "head": (self.vocab_size, W)})
+            elif l.mlp:
+                out.update({p + "mlp.up": (l.mlp.ff, W), p + "mlp.down": (W, l.mlp.ff)})
+            if gated:
+                out.update({p + "rg1": (W, W), p + "rg1.b": (W,)})
+                if l.mlp:
+                    out.update({p + "rg2": (W, W), p + "rg2.b": (W,)})
+            if self.canon_taps:
+                out[p + "canon1"] = (W, self.canon_taps)
+        if gated:
+            out["final.norm"] = ()
+        else:
+            out.update({"final.norm": (W,), "final.norm.b": (W,)})
+        out["head"] = (self.vocab_size, W)
         return out
 
     def param_count(self) -> int:
@@ -181,25 +311,75 @@ def _positive(**kw) -> None:
             raise ValueError(f"{k} must be positive, got {v}")
 
 
-def _mixer(kind: str, m: dict) -> Mixer:
-    if kind == LatentMixer.kind:
-        x = LatentMixer(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]))
-        _positive(heads=x.heads, dim=x.dim, vdim=x.vdim, kv_rank=x.kv_rank)
-        return x
-    if kind == DeltaMixer.kind:
-        x = DeltaMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]))
-        _positive(heads=x.heads, kv_heads=x.kv_heads, dim=x.dim, vdim=x.vdim, conv=x.taps)
-        if x.heads % x.kv_heads:
-            raise ValueError("heads must be a multiple of kv_heads")
-        return x
-    raise ValueError(f"unknown mixer type {kind!r}")
+def _grouped(heads: int, kv_heads: int) -> None:
+    if heads % kv_heads:
+        raise ValueError("heads must be a multiple of kv_heads")
 
 
-def _mlp(m: Optional[dict]) -> Optional[MoeSpec]:
+def _latent(m: dict) -> LatentMixer:
+    x = LatentMixer(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]))
+    _positive(heads=x.heads, dim=x.dim, vdim=x.vdim, kv_rank=x.kv_rank)
+    return x
+
+
+def _attention(m: dict) -> AttentionMixer:
+    x = AttentionMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                       int(m["mask"]["size"]), float(m["rot"]["base"]), int(m["rot"]["dims"]), bool(m.get("v_mix", False)))
+    _positive(heads=x.heads, kv_heads=x.kv_heads, dim=x.dim, vdim=x.vdim, chunk=x.chunk, rot_base=x.rot_base)
+    _grouped(x.heads, x.kv_heads)
+    if not 0 <= x.rot_dims <= x.dim or x.rot_dims % 2:
+        raise ValueError("rot.dims must be even and at most dim")
+    return x
+
+
+def _mamba(m: dict) -> MambaMixer:
+    x = MambaMixer(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"]))
+    _positive(inner=x.inner, state=x.state, dt_rank=x.dt_rank, conv=x.taps)
+    return x
+
+
+def _delta(m: dict, **form) -> DeltaMixer:
+    x = DeltaMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), int(m["conv"]), **form)
+    _positive(heads=x.heads, kv_heads=x.kv_heads, dim=x.dim, vdim=x.vdim, conv=x.taps)
+    _grouped(x.heads, x.kv_heads)
+    return x
+
+
+HEAD_DELTA = dict(decay_rank=0, gate_rank=0, head_decay=True, gate="silu")
+
+MIXERS: Dict[str, Callable[[dict], Mixer]] = {
+    "latent_attention": _latent,
+    "channel_delta": _delta,
+    "attention": _attention,
+    "mamba1": _mamba,
+    "delta": lambda m: _delta(m, **HEAD_DELTA),
+}
+
+
+@dataclass(frozen=True)
+class Design:
+    """What an architecture's name fixes: its block form, and the mixers and feed-forwards its layers may name."""
+    name: str
+    block: str
+    mixers: Tuple[str, ...]
+    feed_forward: str
+
+
+DESIGNS = {d.name: d for d in (Design("Gitozen", PARALLEL_GATED, ("latent_attention", "channel_delta"), "moe"),
+                               Design("Supisun", OUTPUT_NORM, ("attention", "mamba1", "delta"), "dense"))}
+
+ARCHITECTURES = tuple(n.lower() for n in DESIGNS)       # registry names of the layer-list architectures
+
+
+def _mlp(m: Optional[dict], kind: str):
     if m is None:
         return None
-    if m.get("kind", "moe") != "moe":
+    if m.get("kind", kind) != kind:
         raise ValueError(f"unknown feed-forward kind {m.get('kind')!r}")
+    if kind == "dense":
+        d = DenseSpec(int(m["ff"]))
+        _positive(ff=d.ff)
+        return d
     r = m["router"]
     g = r.get("groups") or {"count": 1, "keep": 1}
     x = MoeSpec(int(r["experts"]), int(r["top"]), int(m["expert"]["ff"]), int(g["count"]), int(g["keep"]))
@@ -217,12 +397,26 @@ def from_layer_list(source) -> LayeredConfig:
     else:
         p = Path(source)
         c = json.loads((p / "config.json" if p.is_dir() else p).read_text())
-    layers = tuple(LayerSpec(_mixer(l["type"], l["mixer"]), _mlp(l.get("mlp"))) for l in c["layers"])
+    arch = str(c.get("architecture", "Gitozen"))
+    if arch not in DESIGNS:
+        raise ValueError(f"unknown layer-list architecture {arch!r}")
+    d = DESIGNS[arch]
+    layers = []
+    for l in c["layers"]:
+        if l["type"] not in d.mixers:
+            raise ValueError(f"unknown mixer type {l['type']!r}")
+        layers.append(LayerSpec(MIXERS[l["type"]](l["mixer"]), _mlp(l.get("mlp"), d.feed_forward)))
     if not layers:
         raise ValueError("a model needs at least one layer")
-    cfg = LayeredConfig(int(c["vocab"]), int(c["width"]), layers, float(c["norm"]["eps"]),
-                        float(c.get("logit_softcap") or 0.0), name=str(c.get("architecture", "gitozen")).lower())
+    cfg = LayeredConfig(int(c["vocab"]), int(c["width"]), tuple(layers), float(c["norm"]["eps"]),
+                        float(c.get("logit_softcap") or 0.0), name=arch.lower(), block=d.block)
+    if d.block == OUTPUT_NORM:
+        cfg = cfg.with_(max_position=int(c["max_positions"]), learned_positions=True, canon_taps=int(c["canon"]["taps"]))
+        _positive(max_positions=cfg.max_position, taps=cfg.canon_taps)
     _positive(vocab=cfg.vocab_size, width=cfg.width)
+    shapes = {(m.kv_heads, m.vdim) for m in (layers[i].mixer for i in cfg.attention_layers) if m.v_mix}
+    if len(shapes) > 1:
+        raise ValueError("value-mixing layers must agree on kv_heads and vdim")
     return cfg
 
 
@@ -233,16 +427,25 @@ def to_layer_list(cfg: LayeredConfig) -> dict:
         m = l.mixer
         if isinstance(m, LatentMixer):
             mx = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale}
+        elif isinstance(m, AttentionMixer):
+            mx = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                  "mask": {"size": m.chunk}, "rot": {"base": m.rot_base, "dims": m.rot_dims}, "v_mix": m.v_mix}
+        elif isinstance(m, MambaMixer):
+            mx = {"inner": m.inner, "state": m.state, "dt_rank": m.dt_rank, "conv": m.taps}
         else:
             mx = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.taps}
         ff = None
-        if l.mlp:
+        if isinstance(l.mlp, DenseSpec):
+            ff = {"kind": "dense", "ff": l.mlp.ff}
+        elif l.mlp:
             ff = {"kind": "moe", "expert": {"ff": l.mlp.ff}, "router": {"experts": l.mlp.experts, "top": l.mlp.top}}
             if l.mlp.groups > 1:
                 ff["router"]["groups"] = {"count": l.mlp.groups, "keep": l.mlp.keep}
         layers.append({"type": m.kind, "mixer": mx, "mlp": ff})
-    return {"architecture": "Gitozen", "vocab": cfg.vocab_size, "width": cfg.width, "norm": {"eps": cfg.norm_eps},
-            "logit_softcap": cfg.logit_softcap or None, "layers": layers}
+    out = {"vocab": cfg.vocab_size, "width": cfg.width, "norm": {"eps": cfg.norm_eps}, "layers": layers}
+    if cfg.block == OUTPUT_NORM:
+        return {"architecture": "Supisun", **out, "max_positions": cfg.max_position, "canon": {"taps": cfg.canon_taps}}
+    return {"architecture": "Gitozen", **out, "logit_softcap": cfg.logit_softcap or None}
 
 
 def tiny_gitozen() -> LayeredConfig:
@@ -271,4 +474,43 @@ def gitozen_latent_lite(n_layers: int = 27) -> LayeredConfig:
     return base.with_(layers=(lat,) * n_layers, name="gitozen-latent-lite")
 
 
-PRESETS = {"tiny-gitozen": tiny_gitozen, "gitozen-lite": gitozen_lite, "gitozen-latent-lite": gitozen_latent_lite}
+def _supisun(vocab: int, width: int, layers, max_position: int, taps: int = 4, eps: float = 1e-6,
+             name: str = "supisun") -> LayeredConfig:
+    return LayeredConfig(vocab_size=vocab, width=width, layers=tuple(layers), norm_eps=eps, name=name,
+                         max_position=max_position, block=OUTPUT_NORM, canon_taps=taps, learned_positions=True)
+
+
+def tiny_supisun() -> LayeredConfig:
+    """Small shape for fixtures and the command line: all three mixers, grouped heads, a layer without feed-forward."""
+    att = AttentionMixer(heads=6, kv_heads=2, dim=24, vdim=16, scale=0.2, chunk=40, rot_base=10000.0, rot_dims=16, v_mix=True)
+    mam = MambaMixer(inner=112, state=8, dt_rank=6, taps=4)
+    dlt = DeltaMixer(heads=4, kv_heads=2, dim=16, vdim=24, taps=3, **HEAD_DELTA)
+    ff = DenseSpec(160)
+    return _supisun(512, 96, (LayerSpec(att, ff), LayerSpec(mam, ff), LayerSpec(dlt, None), LayerSpec(att, ff)), 4096, taps=3)
+
+
+def _supisun_stack(name: str, width: int, heads: int, kv_heads: int, dim: int, ff: int, n_layers: int) -> LayeredConfig:
+    """Layers of a served model's size: out of eight, three attention, three selective-scan and two delta mixers."""
+    att = AttentionMixer(heads, kv_heads, dim, dim, dim ** -0.5, 8192, 500000.0, dim, True)
+    mam = MambaMixer(inner=2 * width, state=16, dt_rank=width // 16, taps=4)
+    dlt = DeltaMixer(heads, heads, dim, dim, 4, **HEAD_DELTA)
+    order = (att, mam, dlt, mam, att, mam, dlt, att)
+    return _supisun(102400, width, (LayerSpec(order[i % 8], DenseSpec(ff)) for i in range(n_layers)), 32768, name=name)
+
+
+def supisun_small(n_layers: int = 24) -> LayeredConfig:
+    return _supisun_stack("supisun-small", 1024, 8, 4, 128, 4096, n_layers)
+
+
+def supisun_lite(n_layers: int = 27) -> LayeredConfig:
+    """The widths of DeepSeek-V2-Lite (and of gitozen-lite)."""
+    return _supisun_stack("supisun-lite", 2048, 16, 4, 128, 8192, n_layers)
+
+
+def supisun_wide(n_layers: int = 32) -> LayeredConfig:
+    return _supisun_stack("supisun-wide", 4096, 32, 8, 128, 14336, n_layers)
+
+
+PRESETS = {"tiny-gitozen": tiny_gitozen, "gitozen-lite": gitozen_lite, "gitozen-latent-lite": gitozen_latent_lite,
+           "tiny-supisun": tiny_supisun, "supisun-small": supisun_small, "supisun-lite": supisun_lite,
+           "supisun-wide": supisun_wide}

@@ -1,7 +1,7 @@
 """Engine runner for layer-list models: the paged runner's transactions, graphs and look-ahead over a model that also
 carries recurrent state.
 
-Latent rows live in the engine's pages; recurrent state and convolution inputs live in the sequence's slot
+Latent rows, or keys and values, live in the engine's pages; recurrent state and convolution inputs live in the sequence's slot
 (`RecurrentStatePool`).  A transaction reads the committed buffer of a slot and writes the next one; publishing makes it
 current, rolling back needs nothing.  State cannot be cut at an earlier position, so speculation (rows that may be
 rejected) and shared prefixes (forks, prompt-prefix cache) are refused; a retained session keeps its slot, a swapped-out
@@ -43,7 +43,7 @@ class LayeredRunner(DeepSeekRunner):
     # ------------------------------------------------------------------ parts
     def _make_pool(self, n_pages: int) -> KvPool:
         return KvPool(self.cfg, n_pages, self.page_size, self.device, dtype=self.w.embed.dtype,
-                      n_layers=len(self.cfg.latent_layers))
+                      n_layers=len(self.cfg.cache_layers))
 
     def _prefill_tc_heads(self) -> int:
         from ..ops.kernels import prefill_tc_supported
@@ -75,14 +75,14 @@ class LayeredRunner(DeepSeekRunner):
                                      supports_provisional=False, supports_full_logits=True)
 
     def kv_schema(self) -> KvLayoutSchema:
-        return KvLayoutSchema((KvPlaneDescriptor("latent_kv", self.cfg.kv_row_dim, self.pool.n_layers),), self.page_size,
+        return KvLayoutSchema((KvPlaneDescriptor("latent_kv" if self.cfg.latent_layers else "kv", self.cfg.kv_row_dim, self.pool.n_layers),), self.page_size,
                               self.max_seq_len)
 
     def prepare_batch(self, txn_id: int, batch: ExecutionBatch) -> None:
         for s in batch.sequences:
             if s.cow:
                 raise RuntimeError("recurrent state is bound by slot: shared (copy-on-write) pages are not supported")
-            if s.state_slot >= self.max_seqs or s.sequence_len > self.max_seq_len:
+            if s.state_slot >= self.max_seqs or s.sequence_len > min(self.max_seq_len, self.cfg.max_position):
                 raise RuntimeError(f"sequence in slot {s.state_slot} exceeds the runner's pools")
         super().prepare_batch(txn_id, batch)
 

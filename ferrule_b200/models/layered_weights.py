@@ -1,10 +1,14 @@
 """Weight image of a layer-list model, packed once at load time into what the kernels read.
 
-Every linear that reads the layer's normalised input is one row block of a single matrix `w_in`, so a layer starts with
-one GEMM; blocks begin at multiples of 8 columns of its output:
+Every linear that reads the mixer's input is one row block of a single matrix `w_in`, so a layer starts with one GEMM;
+blocks begin at multiples of 8 columns of its output:
 
-  latent layer  q (heads x dim, each head padded to 8) | dkv | head gates | residual gate 1 | residual gate 2
-  delta layer   q | k | v | decay low rank | gate low rank | beta | residual gate 1 | residual gate 2
+  latent layer     q (heads x dim, each head padded to 8) | dkv | head gates
+  attention layer  q | k | v, each head padded to 8
+  delta layer      q | k | v | decay low rank | gate low rank | beta      (full projections: decay | gate | beta)
+  mamba layer      x | z
+
+followed, in parallel gated blocks, by residual gate 1 | residual gate 2.
 
 The second halves of the delta layer's two low-rank projections are one block-diagonal matrix `w_ag` (fp32 output:
 decay pre-activations and output-gate pre-activations).  Keys and values of a latent layer are absorbed: `w_uk_t` maps a
@@ -20,7 +24,8 @@ from typing import Callable, Dict, List, Optional
 
 import torch
 
-from .layered_config import DeltaMixer, LatentMixer, LayeredConfig, LayerSpec, MoeSpec, pad_to
+from .layered_config import (PARALLEL_GATED, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, LayeredConfig, LayerSpec,
+                             MambaMixer, MoeSpec, pad_to)
 
 GetTensor = Callable[[str], torch.Tensor]
 
@@ -48,20 +53,39 @@ class MixerImage:
     off_gate: int = 0
     conv: Optional[torch.Tensor] = None      # fp32 [taps, channels]
     a_neg: Optional[torch.Tensor] = None     # fp32 [heads] = -exp(A_log)
-    dt_bias: Optional[torch.Tensor] = None   # fp32 [heads * dim]
+    dt_bias: Optional[torch.Tensor] = None   # fp32 [heads * dim] (one decay per head: [heads]); mamba: [inner_pad]
     o_norm: Optional[torch.Tensor] = None    # fp32 [vdim]
+    # attention
+    q_norm: Optional[torch.Tensor] = None    # fp32 [heads * dim_pad]
+    k_norm: Optional[torch.Tensor] = None    # fp32 [kv_heads * dim_pad]
+    v_mix: float = 0.0                       # share of the first mixing layer's values
+    # mamba (also conv, dt_bias)
+    w_x: Optional[torch.Tensor] = None       # [dt | B | C rows, inner_pad], blocks at off_b / off_c
+    off_b: int = 0
+    off_c: int = 0
+    w_dt: Optional[torch.Tensor] = None      # [inner_pad, dt_rank padded to 8]
+    conv_b: Optional[torch.Tensor] = None    # fp32 [inner_pad]
+    a_log2: Optional[torch.Tensor] = None    # fp32 [state, inner_pad] = -exp(A_log) * log2(e)
+    d_skip: Optional[torch.Tensor] = None    # fp32 [inner_pad]
 
 
 @dataclass
 class LayerImage:
     spec: LayerSpec
-    norm: torch.Tensor                       # fp32 [1]: one number for all coordinates
     mixer: MixerImage
-    rg1_b: torch.Tensor                      # fp32 [width_pad]
+    # parallel gated block
+    norm: Optional[torch.Tensor] = None      # fp32 [1]: one number for all coordinates
+    rg1_b: Optional[torch.Tensor] = None     # fp32 [width_pad]
     rg2_b: Optional[torch.Tensor] = None
     router_w: Optional[torch.Tensor] = None  # [experts, width_pad]
     e_w13: Optional[torch.Tensor] = None     # [experts, 2 * ff_pad, width_pad]
     e_w2: Optional[torch.Tensor] = None      # [experts, width_pad, ff_pad]
+    # output-norm block: norm weights and biases of the mixer's and the feed-forward's output, input convolution
+    norm1: Optional[torch.Tensor] = None     # fp32 [2, width_pad]
+    norm2: Optional[torch.Tensor] = None     # fp32 [2, width_pad]
+    canon: Optional[torch.Tensor] = None     # fp32 [taps, width_pad]
+    w_up: Optional[torch.Tensor] = None      # [ff_pad, width_pad]
+    w_down: Optional[torch.Tensor] = None    # [width_pad, ff_pad]
 
 
 @dataclass
@@ -69,13 +93,15 @@ class LayeredWeights:
     cfg: LayeredConfig
     embed: torch.Tensor                      # [vocab, width_pad]
     layers: List[LayerImage]
-    final_norm: torch.Tensor                 # fp32 [1]
+    final_norm: torch.Tensor                 # fp32 [1], output-norm blocks: [2, width_pad]
     lm_head: torch.Tensor                    # [vocab, width_pad]
+    pos: Optional[torch.Tensor] = None       # [max_position, width_pad] learned position vectors
     mtp: list = field(default_factory=list)  # the architecture has no proposal stages
     weight_format: str = "bf16"
 
     def nbytes(self) -> int:
-        total = sum(t.numel() * t.element_size() for t in (self.embed, self.final_norm, self.lm_head))
+        total = sum(t.numel() * t.element_size() for t in (self.embed, self.final_norm, self.lm_head)
+                    + (() if self.pos is None else (self.pos,)))
         for l in self.layers:
             for holder in (l, l.mixer):
                 total += sum(t.numel() * t.element_size() for t in vars(holder).values() if isinstance(t, torch.Tensor))
@@ -113,21 +139,59 @@ def _pack_latent(m: LatentMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: 
                       kv_norm=_pad(get(p + "dkv.norm").float(), DL).contiguous())
 
 
+def _pack_attention(m: AttentionMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
+    Wp, dp, vp = cfg.width_pad, m.dim_pad, m.vdim_pad
+    for name, heads, d, pad in (("q", m.heads, m.dim, dp), ("k", m.kv_heads, m.dim, dp), ("v", m.kv_heads, m.vdim, vp)):
+        b.add(name, _pad(get(p + name).view(heads, d, cfg.width), heads, pad, Wp).reshape(heads * pad, Wp))
+    o = _pad(get(p + "o").view(cfg.width, m.heads, m.vdim), Wp, m.heads, vp)
+    norm = lambda name, heads: _pad(get(p + name).float().view(heads, m.dim), heads, dp).reshape(-1).contiguous()
+    return MixerImage(None, b.off, o.reshape(Wp, m.heads * vp).contiguous(), q_norm=norm("q.norm", m.heads),
+                      k_norm=norm("k.norm", m.kv_heads), v_mix=float(get(p + "vmix").float()) if m.v_mix else 0.0)
+
+
+def _pack_mamba(m: MambaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
+    Ip, LOG2E = m.inner_pad, 1.4426950408889634
+    w_in = get(p + "in")
+    b.add("x", w_in[:m.inner])
+    b.add("z", w_in[m.inner:])
+    low, w_x = _Blocks(Ip), get(p + "x")
+    low.add("dt", w_x[:m.dt_rank])
+    low.add("B", w_x[m.dt_rank:m.dt_rank + m.state])
+    low.add("C", w_x[m.dt_rank + m.state:])
+    vec = lambda name: _pad(get(p + name).float(), Ip).contiguous()
+    a = -torch.exp(get(p + "A_log").double()) * LOG2E
+    return MixerImage(None, b.off, _pad(get(p + "o"), cfg.width_pad, Ip).contiguous(), w_x=low.matrix(), off_b=low.off["B"],
+                      off_c=low.off["C"], w_dt=_pad(get(p + "dt"), Ip, pad_to(m.dt_rank, 8)).contiguous(),
+                      conv=_pad(get(p + "conv").float().t(), m.taps, Ip).contiguous(), conv_b=vec("conv.b"),
+                      dt_bias=vec("dt.b"), d_skip=vec("D"), a_log2=_pad(a.float().t(), m.state, Ip).contiguous())
+
+
 def _pack_delta(m: DeltaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
     Wp = cfg.width_pad
     nk, nv, nd = m.kv_heads * m.dim, m.heads * m.vdim, m.heads * m.dim
-    for name in ("q", "k", "v", "a1", "g1", "b"):
+    for name in ("q", "k", "v") + (("a1", "g1", "b") if m.low_rank else ("a", "g", "b")):
         b.add(name, get(p + name))
-    ra, rg, nd8 = pad_to(m.decay_rank, 8), pad_to(m.gate_rank, 8), pad_to(nd, 8)
-    a2, g2 = get(p + "a2"), get(p + "g2")
-    ag = torch.zeros(nd8 + nv, ra + rg, dtype=a2.dtype, device=a2.device)
-    ag[:nd, :m.decay_rank] = a2
-    ag[nd8:, ra:ra + m.gate_rank] = g2
+    ag, nd8 = None, 0
+    if m.low_rank:
+        ra, rg, nd8 = pad_to(m.decay_rank, 8), pad_to(m.gate_rank, 8), pad_to(nd, 8)
+        a2, g2 = get(p + "a2"), get(p + "g2")
+        ag = torch.zeros(nd8 + nv, ra + rg, dtype=a2.dtype, device=a2.device)
+        ag[:nd, :m.decay_rank] = a2
+        ag[nd8:, ra:ra + m.gate_rank] = g2
     conv = torch.cat([get(p + n + ".conv").view(-1, m.taps) for n in ("q", "k", "v")], 0).float().t().contiguous()
     assert conv.shape[1] == m.channels and nk + nk + nv == m.channels
     return MixerImage(None, b.off, _pad(get(p + "o"), Wp, pad_to(nv, 8)).contiguous(), w_ag=ag, off_gate=nd8, conv=conv,
                       a_neg=-torch.exp(get(p + "A_log").float()), dt_bias=get(p + "dt_bias").float().contiguous(),
                       o_norm=get(p + "norm").float().contiguous())
+
+
+_PACK = {LatentMixer: _pack_latent, AttentionMixer: _pack_attention, DeltaMixer: _pack_delta, MambaMixer: _pack_mamba}
+
+
+def _pack_dense(s: DenseSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: LayerImage) -> None:
+    Wp, fp = cfg.width_pad, pad_to(s.ff, 8)
+    img.w_up = _pad(get(p + "up"), fp, Wp).contiguous()
+    img.w_down = _pad(get(p + "down"), Wp, fp).contiguous()
 
 
 def _pack_moe(s: MoeSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: LayerImage) -> None:
@@ -146,24 +210,35 @@ def _pack_moe(s: MoeSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: Layer
 def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
     """`get(name)` returns a checkpoint tensor in the dtype and on the device the model runs with."""
     Wp = cfg.width_pad
+    gated = cfg.block == PARALLEL_GATED
+    norm = lambda name: torch.stack([_pad(get(n).float(), Wp) for n in (name, name + ".b")]).contiguous()
     layers: List[LayerImage] = []
     for i, spec in enumerate(cfg.layers):
         p = f"l{i}."
         b = _Blocks(Wp)
-        pack = _pack_latent if isinstance(spec.mixer, LatentMixer) else _pack_delta
-        mx = pack(spec.mixer, p + "mix.", get, cfg, b)
-        img = LayerImage(spec, get(p + "norm1").float().reshape(1).contiguous(), mx,
-                         _pad(get(p + "rg1.b").float(), Wp).contiguous())
-        b.add("rg1", get(p + "rg1"))
+        mx = _PACK[type(spec.mixer)](spec.mixer, p + "mix.", get, cfg, b)
+        img = LayerImage(spec, mx)
+        if gated:
+            img.norm = get(p + "norm1").float().reshape(1).contiguous()
+            img.rg1_b = _pad(get(p + "rg1.b").float(), Wp).contiguous()
+            b.add("rg1", get(p + "rg1"))
+        else:
+            img.norm1 = norm(p + "norm1")
+        if cfg.canon_taps:
+            img.canon = _pad(get(p + "canon1").float().view(cfg.width, cfg.canon_taps).t(), cfg.canon_taps, Wp).contiguous()
         if spec.mlp is not None:
-            b.add("rg2", get(p + "rg2"))
-            img.rg2_b = _pad(get(p + "rg2.b").float(), Wp).contiguous()
-            _pack_moe(spec.mlp, p + "mlp.", get, cfg, img)
+            if gated:
+                b.add("rg2", get(p + "rg2"))
+                img.rg2_b = _pad(get(p + "rg2.b").float(), Wp).contiguous()
+            else:
+                img.norm2 = norm(p + "norm2")
+            (_pack_moe if isinstance(spec.mlp, MoeSpec) else _pack_dense)(spec.mlp, p + "mlp.", get, cfg, img)
         mx.w_in = b.matrix()
         layers.append(img)
-    return LayeredWeights(cfg, _pad(get("embed"), cfg.vocab_size, Wp).contiguous(), layers,
-                          get("final.norm").float().reshape(1).contiguous(),
-                          _pad(get("head"), cfg.vocab_size, Wp).contiguous())
+    final = get("final.norm").float().reshape(1).contiguous() if gated else norm("final.norm")
+    pos = _pad(get("pos"), cfg.max_position, Wp).contiguous() if cfg.learned_positions else None
+    return LayeredWeights(cfg, _pad(get("embed"), cfg.vocab_size, Wp).contiguous(), layers, final,
+                          _pad(get("head"), cfg.vocab_size, Wp).contiguous(), pos=pos)
 
 
 class RandomTensors:
@@ -191,13 +266,21 @@ class RandomTensors:
 
         if name == "embed":
             t = normal(0.0, self.embed_std)
+        elif name == "pos":
+            t = normal(0.0, 0.5 * self.embed_std)
         elif name.endswith("A_log"):
             t = normal(-0.5, 1.0)
-        elif name.endswith("dt_bias"):
+        elif name.endswith(("dt_bias", ".dt.b")):
             t = normal(-2.5, 1.0)
         elif name.endswith(".conv"):
             t = normal(0.0, 0.4)
             t[..., -1] += 0.7
+        elif name.endswith("canon1"):
+            t = normal(0.0, 0.3)
+        elif name.endswith(("norm1.b", "norm2.b", "final.norm.b", ".conv.b")):
+            t = normal(0.0, 0.2)
+        elif name.endswith((".vmix", ".D")):
+            t = normal(0.5, 0.2)
         elif name.endswith(("rg1.b", "rg2.b")):
             t = normal(0.7, 0.5)
         elif "norm" in name:

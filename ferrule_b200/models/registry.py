@@ -35,7 +35,7 @@ class Architecture:
     component: str = ""                                          # part of the native library it needs ("": all of it)
 
 
-def _load_gitozen(directory, device, dtype, max_layers=0):
+def _load_layered(directory, device, dtype, max_layers=0):
     from ..io.layered_checkpoint import load_layered
     return load_layered(directory, device=device, dtype=dtype, max_layers=max_layers)
 
@@ -69,7 +69,9 @@ def _run_deepseek(weights, lim: RunnerLimits, **options):
 
 
 ARCHITECTURES: Dict[str, Architecture] = {a.name: a for a in (
-    Architecture("gitozen", lambda c: c.get("architecture") == "Gitozen", _load_gitozen, _run_layered,
+    Architecture("gitozen", lambda c: c.get("architecture") == "Gitozen", _load_layered, _run_layered,
+                 (torch.bfloat16, torch.float32), "layered"),
+    Architecture("supisun", lambda c: c.get("architecture") == "Supisun", _load_layered, _run_layered,
                  (torch.bfloat16, torch.float32), "layered"),
     Architecture("deepseek_v4", lambda c: c.get("model_type") == "deepseek_v4", _load_v4, _run_v4),
     # every other HuggingFace-style config.json is read as a DeepSeek-V2 / V3 model, whose loader checks it

@@ -1,7 +1,8 @@
 """Recurrent-state pool: what a sequence carries from token to token beside its paged cache.
 
-Two kinds of plane per recurrent layer: the fp32 state matrix of every head and the last inputs of the short
-convolutions.  A plane is indexed by slot (the engine's logical sequence slot) and buffer: every slot has `buffers`
+Three kinds of plane: per recurrent layer the fp32 state (a matrix per head of a delta mixer, [inner, state] of a selective
+scan) and the last inputs of the short convolutions, and per layer with an input convolution the last rows of the
+32-bit residual stream it read.  A plane is indexed by slot (the engine's logical sequence slot) and buffer: every slot has `buffers`
 copies and one of them is committed.  A step reads the committed copy and writes the next one, and only the commit of its
 transaction makes that one current - a step that fails or is rolled back leaves nothing to undo.  With decode
 look-ahead a step may already run before its predecessor has been published, so three buffers are in rotation: the
@@ -15,7 +16,7 @@ from typing import Dict, List, Tuple
 
 import torch
 
-from .layered_config import LayeredConfig
+from .layered_config import DeltaMixer, LayeredConfig, MambaMixer
 
 
 class RecurrentStatePool:
@@ -26,15 +27,23 @@ class RecurrentStatePool:
         self.n_states = n_slots * buffers
         self.state: Dict[int, torch.Tensor] = {}
         self.tail: Dict[int, torch.Tensor] = {}
-        for i in cfg.delta_layers:
-            m = cfg.layers[i].mixer
-            self.state[i] = torch.zeros(self.n_states, m.heads, m.dim, m.vdim, dtype=torch.float32, device=device)
-            self.tail[i] = torch.zeros(self.n_states, max(m.taps - 1, 1), m.channels, dtype=dtype, device=device)
+        self.canon: Dict[int, torch.Tensor] = {}
+        plane = lambda *shape, dt=torch.float32: torch.zeros(self.n_states, *shape, dtype=dt, device=device)
+        for i, l in enumerate(cfg.layers):
+            m = l.mixer
+            if isinstance(m, DeltaMixer):
+                self.state[i] = plane(m.heads, m.dim, m.vdim)
+                self.tail[i] = plane(max(m.taps - 1, 1), m.channels, dt=dtype)
+            elif isinstance(m, MambaMixer):
+                self.state[i] = plane(m.state, m.inner_pad)
+                self.tail[i] = plane(max(m.taps - 1, 1), m.inner_pad, dt=dtype)
+            if cfg.canon_taps:
+                self.canon[i] = plane(max(cfg.canon_taps - 1, 1), cfg.width_pad)
         self.current: List[int] = [-1] * n_slots         # committed buffer of every slot, -1: none yet
 
     @property
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.state, self.tail) for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.state, self.tail, self.canon) for t in d.values())
 
     def bind(self, slot: int, fresh: bool, ahead: bool = False) -> Tuple[int, int]:
         """(state index to read, state index to write) of the slot's next step.  `fresh`: the sequence starts with
