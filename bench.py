@@ -102,8 +102,9 @@ def main() -> None:
     ap.add_argument("--batch", type=int, default=32)
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--model", default="deepseek-v2-lite",
-                    help="deepseek-v2-lite is the headline configuration; gitozen-lite and gitozen-latent-lite are layer-list "
-                         "models of the same widths (one GPU), reported without a baseline")
+                    help="deepseek-v2-lite is the headline configuration; gitozen-lite, gitozen-latent-lite and supisun-lite are "
+                         "layer-list models of the same widths (one GPU), supisun-small and supisun-wide others; they are "
+                         "reported without a baseline")
     ap.add_argument("--weight-format", default="bf16", choices=["bf16", "fp8_block", "fp8_mxfp4"],
                     help="bf16 is the headline configuration; the FP8 formats are reported with their own dtype")
     ap.add_argument("--shard-as", type=int, default=0,
@@ -344,6 +345,8 @@ def main() -> None:
     streamed_bytes = weights.nbytes()
     if weights.embed.data_ptr() != weights.lm_head.data_ptr():
         streamed_bytes -= weights.embed.numel() * weights.embed.element_size()
+    if getattr(weights, "pos", None) is not None:
+        streamed_bytes -= weights.pos.numel() * weights.pos.element_size()
     if rank == 0:
         value = B * K / (dev_ms / 1e3)
         e2e_value = B * K / (e2e_ms / 1e3)

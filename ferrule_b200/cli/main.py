@@ -204,7 +204,7 @@ def _engine_sizes(args, max_position: int):
     """(context tokens, pages per sequence, scheduler configuration) from the command line's limits."""
     from ..runtime.scheduler import SchedulerConfig
     pages_per_seq = (min(args.ctx_size, max_position) + args.page_size - 1) // args.page_size
-    ctx = pages_per_seq * args.page_size
+    ctx = min(pages_per_seq * args.page_size, max_position)
     return ctx, pages_per_seq, SchedulerConfig(
         max_active_sequences=args.max_seqs, max_decode_batch=args.max_seqs, max_batch_tokens=args.max_batch_tokens,
         prefill_chunk_size=args.prefill_chunk, decode_cohort_target=getattr(args, "decode_cohort_target", 1),

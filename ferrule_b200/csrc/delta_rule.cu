@@ -1,6 +1,7 @@
-// Gated delta rule with one decay per key channel, short causal convolutions in front, gated per-head output norm.
+// Gated delta rule with one decay per key channel or per head, short causal convolutions in front, gated per-head output
+// norm (sigmoid or SiLU gate).
 //
-// Per head, S [dim, vdim] in fp32, rows of key channels:
+// Per head, S [dim, vdim] in fp32, rows of key channels (g_t one number with a decay per head):
 //     S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
 // with q, k the unit vectors (q also times dim^-1/2) of silu(conv(W x)), v = silu(conv(W_v x)),
 // g = exp(a_neg * softplus(decay + dt_bias)), beta = sigmoid(b).
@@ -31,9 +32,12 @@ struct DeltaParams {
   const float* ag;            // [rows, ldag]: decay pre-activation at 0, output gate pre-activation at off_gate
   long long ldag;
   int off_gate;
+  int off_a;                  // >= 0: one decay per head, its pre-activation in column off_a + h of a projected row
+  int off_g;                  // >= 0: output gate pre-activation in columns off_g .. of a projected row instead of `ag`
+  int gate_silu;
   const float* conv;          // [taps, channels], channels = q | k | v
   const float* a_neg;         // [heads]
-  const float* dt_bias;       // [heads * dim]
+  const float* dt_bias;       // [heads * dim], one decay per head: [heads]
   const float* norm_w;        // [vdim]
   float eps;
   float* state;               // [n_states, heads, dim, vdim]
@@ -116,6 +120,16 @@ template <typename T>
 __device__ __forceinline__ float silu_of(float z) {
   if constexpr (sizeof(T) == 4) return z / (1.f + expf(-z));
   return __fdividef(z, 1.f + __expf(-z));
+}
+
+template <typename T>
+__device__ __forceinline__ float output_gate(const DeltaParams<T>& p, float z) {
+  return p.gate_silu ? silu_of<T>(z) : sigmoid_f(z);
+}
+// pre-activation of the output gate of value column i (head * vdim + column) of row r
+template <typename T>
+__device__ __forceinline__ float gate_pre(const DeltaParams<T>& p, long long r, int i) {
+  return p.off_g >= 0 ? act_load(p.proj + r * p.ldp + p.off_g + i) : p.ag[r * p.ldag + p.off_gate + i];
 }
 
 // ---------------------------------------------------------------------------------
@@ -214,6 +228,11 @@ delta_prepare_kernel(const DeltaParams<T> p) {
   if (i == 0 || i > n - p.taps)
     for (int c = threadIdx.x; c < channels; c += blockDim.x) store_tail(p, c, r0, i, n, sin, sout, channels);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  if (p.off_a >= 0) {
+    for (int h = threadIdx.x; h < p.heads; h += blockDim.x)
+      p.decay[static_cast<long long>(r) * p.heads + h] =
+          decay_of<T>(p.a_neg[h], act_load(p.proj + r * p.ldp + p.off_a + h) + p.dt_bias[h]);
+  } else
   for (int h = warp; h < p.heads; h += nw) {
     const float a = p.a_neg[h];
     const float* pre = p.ag + r * p.ldag + h * p.dim;
@@ -281,7 +300,12 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
   return r;
 }
 
-template <typename T, int RPT, int COLS>
+// HEADG: one decay per head.  The dot products are then taken over the state before the decay and scaled, so that the
+// decay of the state runs beside them instead of ahead of them.
+template <typename T, int RPT, int COLS, bool HEADG>
+constexpr int scan_buf() { return kScanStep * ((HEADG ? 2 : 3) * RPT * 8 + 16 * COLS + 2 + (HEADG ? 1 : 0)); }
+
+template <typename T, int RPT, int COLS, bool HEADG>
 __global__ void __launch_bounds__(128)
 delta_scan_kernel(const DeltaParams<T> p) {
   // the dependents are released at the end: their CTAs would only wait, on the SMs this long kernel needs
@@ -289,8 +313,10 @@ delta_scan_kernel(const DeltaParams<T> p) {
   constexpr int DP = RPT * 8;                                   // padded key dimension
   constexpr int kCols = 16 * COLS;
   extern __shared__ __align__(16) float sm[];
-  // per buffer: k, q, g [kScanStep][DP], v [kScanStep][kCols], beta, qk [kScanStep]
-  constexpr int kBuf = kScanStep * (3 * DP + kCols + 2);
+  // per buffer: k, q, g [kScanStep][DP], v [kScanStep][kCols], beta, qk [kScanStep]; one decay per head: no g rows,
+  // g [kScanStep] at the end
+  constexpr int kBuf = scan_buf<T, RPT, COLS, HEADG>();
+  constexpr int kV = (HEADG ? 2 : 3) * kScanStep * DP;          // first float of v
   const int seq = blockIdx.y;
   const int vtiles = (p.vdim + kCols - 1) / kCols;
   const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * kCols;
@@ -329,7 +355,7 @@ delta_scan_kernel(const DeltaParams<T> p) {
         const long long r = r0 + t0 + t;
         cp_async16(base + t * DP + d, p.kn + r * ldk + hk * p.dim + d);
         cp_async16(base + kScanStep * DP + t * DP + d, p.qn + r * ldk + hk * p.dim + d);
-        cp_async16(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
+        if (!HEADG) cp_async16(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
       }
     } else {
       for (int i = tid; i < cnt * p.dim; i += 128) {
@@ -337,10 +363,10 @@ delta_scan_kernel(const DeltaParams<T> p) {
         const long long r = r0 + t0 + t;
         cp_async4(base + t * DP + d, p.kn + r * ldk + hk * p.dim + d);
         cp_async4(base + kScanStep * DP + t * DP + d, p.qn + r * ldk + hk * p.dim + d);
-        cp_async4(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
+        if (!HEADG) cp_async4(base + 2 * kScanStep * DP + t * DP + d, p.decay + r * ldg + h * p.dim + d);
       }
     }
-    float* vb = base + 3 * kScanStep * DP;
+    float* vb = base + kV;
     for (int i = tid; i < cnt * kCols; i += 128) {
       const int t = i / kCols, c = i - t * kCols;
       if (v0 + c < p.vdim) cp_async4(vb + i, p.v + (r0 + t0 + t) * ldv + h * p.vdim + v0 + c);
@@ -348,6 +374,8 @@ delta_scan_kernel(const DeltaParams<T> p) {
     if (tid < cnt) {
       cp_async4(vb + kScanStep * kCols + tid, p.beta + static_cast<long long>(r0 + t0 + tid) * p.heads + h);
       cp_async4(vb + kScanStep * kCols + kScanStep + tid, p.qk + static_cast<long long>(r0 + t0 + tid) * p.kv_heads + hk);
+      if (HEADG)
+        cp_async4(vb + kScanStep * kCols + 2 * kScanStep + tid, p.decay + static_cast<long long>(r0 + t0 + tid) * p.heads + h);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -362,7 +390,7 @@ delta_scan_kernel(const DeltaParams<T> p) {
     }
     __syncthreads();
     const float* base = sm + b * kBuf;
-    const float* vb = base + 3 * kScanStep * DP;
+    const float* vb = base + kV;
     const int cnt = min(kScanStep, n - t0);
     uint64_t k[RPT / 2], q[RPT / 2], g[RPT / 2];
     auto fetch = [&](int t) {
@@ -371,10 +399,12 @@ delta_scan_kernel(const DeltaParams<T> p) {
         const float* row = base + t * DP + j * 32 + l8 * 4;
         const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(row);
         const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(row + kScanStep * DP);
-        const ulonglong2 e = *reinterpret_cast<const ulonglong2*>(row + 2 * kScanStep * DP);
         k[2 * j] = a.x; k[2 * j + 1] = a.y;
         q[2 * j] = c.x; q[2 * j + 1] = c.y;
-        g[2 * j] = e.x; g[2 * j + 1] = e.y;
+        if (!HEADG) {
+          const ulonglong2 e = *reinterpret_cast<const ulonglong2*>(row + 2 * kScanStep * DP);
+          g[2 * j] = e.x; g[2 * j + 1] = e.y;
+        }
       }
     };
     fetch(0);
@@ -383,6 +413,8 @@ delta_scan_kernel(const DeltaParams<T> p) {
     for (int t = 0; t < cnt; ++t, o += ldv) {
       const float beta = vb[kScanStep * kCols + t], qk = vb[kScanStep * kCols + kScanStep + t];
       float sk[COLS], sq[COLS], vt[COLS], out = 0.f;
+      const float gh = HEADG ? vb[kScanStep * kCols + 2 * kScanStep + t] : 1.f;
+      const uint64_t gh2 = pack2(gh, gh);
 #pragma unroll
       for (int c = 0; c < COLS; ++c) vt[c] = vb[t * kCols + vc + c];
 #pragma unroll
@@ -390,8 +422,10 @@ delta_scan_kernel(const DeltaParams<T> p) {
         uint64_t ka = 0, kb = 0, qa = 0, qb = 0;          // two chains each
 #pragma unroll
         for (int j = 0; j < RPT / 2; j += 2) {
-          S[c][j] = mul2(S[c][j], g[j]);
-          S[c][j + 1] = mul2(S[c][j + 1], g[j + 1]);
+          if (!HEADG) {
+            S[c][j] = mul2(S[c][j], g[j]);
+            S[c][j + 1] = mul2(S[c][j + 1], g[j + 1]);
+          }
           ka = fma2(S[c][j], k[j], ka);
           kb = fma2(S[c][j + 1], k[j + 1], kb);
           qa = fma2(S[c][j], q[j], qa);
@@ -404,6 +438,10 @@ delta_scan_kernel(const DeltaParams<T> p) {
         unpack2(qa, a0, a1);
         unpack2(qb, b0, b1);
         sq[c] = (a0 + b0) + (a1 + b1);
+        if (HEADG) {
+#pragma unroll
+          for (int j = 0; j < RPT / 2; ++j) S[c][j] = mul2(S[c][j], gh2);
+        }
       }
 #pragma unroll
       for (int x = 1; x < 8; x <<= 1)
@@ -414,8 +452,8 @@ delta_scan_kernel(const DeltaParams<T> p) {
         }
 #pragma unroll
       for (int c = 0; c < COLS; ++c) {
-        const float u = beta * (vt[c] - sk[c]);
-        if (l8 == c) out = fmaf(qk, u, sq[c]);
+        const float u = beta * (HEADG ? fmaf(-gh, sk[c], vt[c]) : vt[c] - sk[c]);
+        if (l8 == c) out = fmaf(qk, u, HEADG ? gh * sq[c] : sq[c]);
         const uint64_t u2 = pack2(u, u);
 #pragma unroll
         for (int j = 0; j < RPT / 2; ++j) S[c][j] = fma2(k[j], u2, S[c][j]);
@@ -455,22 +493,25 @@ delta_output_kernel(const DeltaParams<T> p) {
   const long long r = i / p.heads;
   const int h = static_cast<int>(i - r * p.heads);
   const float* o = p.o + i * p.vdim;
-  if (p.vdim <= 128 && (p.vdim & 3) == 0 && (p.ldag & 3) == 0 && (p.off_gate & 3) == 0) {
+  const bool gate_vec = p.off_g >= 0 ? (p.off_g & 3) == 0 && (p.ldp & 3) == 0 : (p.ldag & 3) == 0 && (p.off_gate & 3) == 0;
+  if (p.vdim <= 128 && (p.vdim & 3) == 0 && gate_vec) {
     // four columns per lane, everything requested up front
     const int v = lane * 4;
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), g = a, w = a;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f), w = a;
+    float g[4] = {};
     if (v < p.vdim) {
       a = *reinterpret_cast<const float4*>(o + v);
-      g = *reinterpret_cast<const float4*>(p.ag + r * p.ldag + p.off_gate + h * p.vdim + v);
+      if (p.off_g >= 0) load_vec(p.proj + r * p.ldp + p.off_g + h * p.vdim + v, g);
+      else load_vec(p.ag + r * p.ldag + p.off_gate + h * p.vdim + v, g);
       w = *reinterpret_cast<const float4*>(p.norm_w + v);
     }
     const float inv = 1.f / sqrtf(warp_sum(a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w) / p.vdim + p.eps);
     if (v < p.vdim) {
       T* dst = p.out + r * p.ldo + h * p.vdim + v;
-      act_store(dst, a.x * inv * w.x * sigmoid_f(g.x));
-      act_store(dst + 1, a.y * inv * w.y * sigmoid_f(g.y));
-      act_store(dst + 2, a.z * inv * w.z * sigmoid_f(g.z));
-      act_store(dst + 3, a.w * inv * w.w * sigmoid_f(g.w));
+      act_store(dst, a.x * inv * w.x * output_gate(p, g[0]));
+      act_store(dst + 1, a.y * inv * w.y * output_gate(p, g[1]));
+      act_store(dst + 2, a.z * inv * w.z * output_gate(p, g[2]));
+      act_store(dst + 3, a.w * inv * w.w * output_gate(p, g[3]));
     }
     return;
   }
@@ -478,9 +519,9 @@ delta_output_kernel(const DeltaParams<T> p) {
   for (int v = lane; v < p.vdim; v += 32) ss = fmaf(o[v], o[v], ss);
   ss = warp_sum(ss);
   const float inv = 1.f / sqrtf(ss / p.vdim + p.eps);
-  const float* g = p.ag + r * p.ldag + p.off_gate + h * p.vdim;
   for (int v = lane; v < p.vdim; v += 32)
-    act_store(p.out + r * p.ldo + h * p.vdim + v, o[v] * inv * p.norm_w[v] * sigmoid_f(g[v]));
+    act_store(p.out + r * p.ldo + h * p.vdim + v,
+              o[v] * inv * p.norm_w[v] * output_gate(p, gate_pre(p, r, h * p.vdim + v)));
 }
 
 // ---------------------------------------------------------------------------------
@@ -562,9 +603,11 @@ delta_decode_kernel(const DeltaParams<T> p) {
     }
     (part == 0 ? s_q : part == 1 ? s_k : s_v)[d] = y;
   }
+  const float gh = p.off_a >= 0 ? decay_of<T>(p.a_neg[h], act_load(p.proj + r * p.ldp + p.off_a + h) + p.dt_bias[h]) : 0.f;
   for (int d = tid; d < 8 * RW; d += 256) {
     const int c = h * p.dim + d;
-    s_g[d] = d < p.dim ? decay_of<T>(p.a_neg[h], p.ag[r * p.ldag + c] + p.dt_bias[c]) : 0.f;
+    if (p.off_a >= 0) s_g[d] = d < p.dim ? gh : 0.f;
+    else s_g[d] = d < p.dim ? decay_of<T>(p.a_neg[h], p.ag[r * p.ldag + c] + p.dt_bias[c]) : 0.f;
   }
   __syncthreads();
   // norms of q and k, their product: every warp computes them for itself
@@ -623,17 +666,17 @@ delta_decode_kernel(const DeltaParams<T> p) {
     ss = warp_sum(ss);
     const float inv = 1.f / sqrtf(ss / p.vdim + p.eps);
     if (vok) {
-      const float* g = p.ag + r * p.ldag + p.off_gate + h * p.vdim + vcol;
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        act_store(p.out + r * p.ldo + h * p.vdim + vcol + e, o[e] * inv * p.norm_w[vcol + e] * sigmoid_f(g[e]));
+        act_store(p.out + r * p.ldo + h * p.vdim + vcol + e,
+                  o[e] * inv * p.norm_w[vcol + e] * output_gate(p, gate_pre(p, r, h * p.vdim + vcol + e)));
     }
   }
 }
 
 template <typename T>
 static int fill(const FbDeltaArgs* a, DeltaParams<T>& p) {
-  if (!a || !a->proj || !a->ag || !a->conv || !a->a_neg || !a->dt_bias || !a->norm_w || !a->state || !a->seq_start ||
+  if (!a || !a->proj || (!a->ag && (a->off_a < 0 || a->off_g < 0)) || !a->conv || !a->a_neg || !a->dt_bias || !a->norm_w || !a->state || !a->seq_start ||
       !a->state_in || !a->state_out || !a->out)
     return FB_ERR_SHAPE;
   if (a->rows <= 0 || a->n_seqs <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 ||
@@ -643,6 +686,7 @@ static int fill(const FbDeltaArgs* a, DeltaParams<T>& p) {
   p.proj = static_cast<const T*>(a->proj); p.ldp = a->ldp;
   p.off_q = a->off_q; p.off_k = a->off_k; p.off_v = a->off_v; p.off_b = a->off_b;
   p.ag = a->ag; p.ldag = a->ldag; p.off_gate = a->off_gate;
+  p.off_a = a->off_a; p.off_g = a->off_g; p.gate_silu = a->gate_silu;
   p.conv = a->conv; p.a_neg = a->a_neg; p.dt_bias = a->dt_bias; p.norm_w = a->norm_w; p.eps = a->eps;
   p.state = a->state; p.tail = static_cast<T*>(a->tail); p.n_states = a->n_states;
   p.row_seq = a->row_seq; p.seq_start = a->seq_start; p.state_in = a->state_in; p.state_out = a->state_out;
@@ -668,30 +712,35 @@ static int run_decode(const FbDeltaArgs* a, cudaStream_t s) {
   return launched();
 }
 
-template <typename T, int RPT, int COLS>
+template <typename T, int RPT, int COLS, bool HEADG>
 static int launch_scan_cols(const DeltaParams<T>& p, cudaStream_t s) {
-  constexpr int smem = 2 * kScanStep * (3 * RPT * 8 + 16 * COLS + 2) * static_cast<int>(sizeof(float));
+  constexpr int smem = 2 * scan_buf<T, RPT, COLS, HEADG>() * static_cast<int>(sizeof(float));
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT, COLS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT, COLS, HEADG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess)
       return FB_ERR_LAUNCH;
     attr = true;
   }
   const dim3 grid(p.heads * ((p.vdim + 16 * COLS - 1) / (16 * COLS)), p.n_seqs);
-  launch_pdl(delta_scan_kernel<T, RPT, COLS>, grid, dim3(128), smem, s, p);
+  launch_pdl(delta_scan_kernel<T, RPT, COLS, HEADG>, grid, dim3(128), smem, s, p);
   return launched();
+}
+
+template <typename T, int RPT, bool HEADG>
+static int launch_scan_form(const DeltaParams<T>& p, cudaStream_t s) {
+  const long long per_col = static_cast<long long>(p.heads) * p.n_seqs;
+  auto ctas = [&](int cols) { return per_col * ((p.vdim + 16 * cols - 1) / (16 * cols)); };
+  if constexpr (RPT <= 16) {
+    if (ctas(4) >= 120 && p.vdim > 32) return launch_scan_cols<T, RPT, 4, HEADG>(p, s);
+  }
+  if (ctas(2) >= 120 && p.vdim > 16) return launch_scan_cols<T, RPT, 2, HEADG>(p, s);
+  return launch_scan_cols<T, RPT, 1, HEADG>(p, s);
 }
 
 template <typename T, int RPT>
 static int launch_scan(const DeltaParams<T>& p, cudaStream_t s) {
-  const long long per_col = static_cast<long long>(p.heads) * p.n_seqs;
-  auto ctas = [&](int cols) { return per_col * ((p.vdim + 16 * cols - 1) / (16 * cols)); };
-  if constexpr (RPT <= 16) {
-    if (ctas(4) >= 120 && p.vdim > 32) return launch_scan_cols<T, RPT, 4>(p, s);
-  }
-  if (ctas(2) >= 120 && p.vdim > 16) return launch_scan_cols<T, RPT, 2>(p, s);
-  return launch_scan_cols<T, RPT, 1>(p, s);
+  return p.off_a >= 0 ? launch_scan_form<T, RPT, true>(p, s) : launch_scan_form<T, RPT, false>(p, s);
 }
 
 template <typename T>

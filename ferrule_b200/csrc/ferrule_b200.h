@@ -42,7 +42,7 @@ typedef struct FbGemmArgs {
   int w_rows_per_group;
   int x_rows;
   int ntok;                 // rows per tile: 16, 32, 64, 128 or 256
-  int epilogue;             // 0 store, 1 swiglu (dual weights), 2 scatter, 3 all-reduce
+  int epilogue;             // 0 store, 1 swiglu (dual weights), 2 scatter, 3 all-reduce, 4 store gelu(x)
   int dual_offset;          // row of the "up" block inside a group (epilogue 1)
   int out_fp32;
   int max_tok_tiles;        // capacity of the tile table (grouped mode)
@@ -78,7 +78,7 @@ typedef struct FbGemmArgs {
 
 int fb_gemm_bf16(const FbGemmArgs* args, void* stream);
 
-// fp32 tensors, full 32-bit arithmetic (FMA units); same argument block (epilogues 0..2, act_limit 0, no collectives)
+// fp32 tensors, full 32-bit arithmetic (FMA units); same argument block (epilogues 0..2 and 4, act_limit 0, no collectives)
 int fb_gemm_f32(const FbGemmArgs* args, void* stream);
 
 // ---- block-scaled FP8 GEMM ---------------------------------------------------------------
@@ -230,6 +230,120 @@ int fb_latent_append(const void* src, long long lds, int rank, int row_dim, cons
 int fb_softcap(float* logits, long long ldl, int rows, int vocab, float cap, void* stream);
 int fb_state_rotate(int* state_in, int* state_out, int n, int buffers, void* stream);
 
+// ---- output-norm blocks (see stream_ops.cu) ------------------------------------------------------------------
+// The residual stream is fp32; activations bf16 or fp32 (`fp32`).  Pitches are multiples of 8 elements.
+typedef struct FbStreamArgs {
+  float* x;                 // [rows, ldx] stream; read (unless `ids`) and written
+  long long ldx;
+  const int* ids;           // embedding form: x = table[ids] + pos_table[positions]
+  const int* positions;
+  const void* table;
+  const void* pos_table;    // optional
+  long long ldt;
+  int vocab, max_pos;
+  const void* y;            // sublayer form: x += norm(y)
+  long long ldy;
+  const float* norm_w;      // [dim_pad]
+  const float* norm_b;      // optional [dim_pad]
+  int rms;                  // 0: layer norm, 1: RMS norm
+  void* act;                // optional [rows, lda]: the new stream rows as activations
+  long long lda;
+  const float* conv;        // optional [taps, dim_pad]: h = x + conv(x), one row per sequence (decode steps)
+  float* tail;              // [n_states, taps - 1, dim_pad]
+  const int* state_in;
+  const int* state_out;
+  int taps, n_states;
+  void* h;                  // [rows, ldh]
+  long long ldh;
+  int rows, dim, dim_pad, fp32;
+  float eps;
+  void* status;
+} FbStreamArgs;
+int fb_stream_step(const FbStreamArgs* args, void* stream);
+// out[i] = norm(x[rows_idx[i]]) as activations
+int fb_norm_rows(const float* x, long long ldx, int x_rows, const int* rows_idx, int n, const float* norm_w,
+                 const float* norm_b, int rms, void* out, long long ldo, int dim, int dim_pad, float eps, int fp32,
+                 void* status, void* stream);
+// causal convolution over the packed rows of several sequences, one filter of `taps` per channel; inputs before a
+// sequence's first row come from its state, which is brought up to date
+typedef struct FbConvArgs {
+  const void* x;            // [rows, ldx]
+  long long ldx;
+  const float* w;           // [taps, channels]
+  const float* bias;        // optional [channels]
+  void* tail;               // [n_states, taps - 1, channels], dtype of x
+  void* out;                // [rows, ldo]
+  long long ldo;
+  const int* row_seq;
+  const int* seq_start;
+  const int* state_in;
+  const int* state_out;
+  int rows, channels, taps, n_states, n_seqs;
+  int x_fp32;               // x and tail are fp32 instead of bf16
+  int out_fp32;
+  int residual;             // out = x + conv(x)
+  int silu;                 // out = silu(conv(x) + bias)
+  void* status;
+} FbConvArgs;
+int fb_short_conv(const FbConvArgs* args, void* stream);
+
+// ---- selective scan (see selective_scan.cu) ------------------------------------------------------------------
+typedef struct FbScanArgs {
+  const void* x;            // [rows, ldx] convolved inputs
+  long long ldx;
+  const void* z;            // [rows, ldz] output gate pre-activation
+  long long ldz;
+  const void* bc;           // [rows, ldbc]: B at off_b, C at off_c
+  long long ldbc;
+  int off_b, off_c;
+  const float* dt;          // [rows, lddt] step size pre-activation without bias
+  long long lddt;
+  const float* dt_bias;     // [inner]
+  const float* a_log2;      // [state, inner]: decay exponents, base 2
+  const float* d_skip;      // [inner]
+  float* states;            // [n_states, state, inner]
+  const int* seq_start;
+  const int* state_in;
+  const int* state_out;
+  void* out;                // [rows, ldo]: (scan + D x) * silu(z)
+  long long ldo;
+  int rows, n_seqs, inner, state, n_states, fp32;
+  void* status;
+} FbScanArgs;
+int fb_selective_scan(const FbScanArgs* args, void* stream);    // state <= 128, inner % 8 == 0
+
+// ---- grouped-query attention in position chunks (see gqa_attention.cu) -----------------------------------------
+typedef struct FbGqaArgs {
+  void* q;                  // [rows, ldq]: heads x dim_pad; `fb_gqa_prep` normalises and rotates it in place
+  long long ldq;
+  const void* k;            // fb_gqa_prep: projected keys and values [rows, ldkv]
+  const void* v;
+  long long ldkv;
+  const float* q_norm;      // [heads * dim_pad]
+  const float* k_norm;      // [kv_heads * dim_pad]
+  const float* cos_t;       // [max_pos, rot_dims / 2]
+  const float* sin_t;
+  int max_pos, rot_dims;
+  const int* positions;
+  const long long* write_slot;
+  void* pool;               // [pool_rows, pool_ld]: kv_heads x dim_pad keys | kv_heads x vdim_pad values
+  long long pool_rows, pool_ld;
+  const void* first_pool;   // optional: value mixing, pool of the layer whose values are mixed in
+  long long first_off;      // its first value column
+  float v_mix;
+  const int* block_table;
+  const int* row_seq;
+  const int* row_pos;
+  int num_seqs, max_blocks, page_size, chunk;
+  float scale, eps;
+  void* out;                // [rows, ldo]: heads x vdim_pad
+  long long ldo;
+  int rows, heads, kv_heads, dim, dim_pad, vdim, vdim_pad, fp32;
+  void* status;
+} FbGqaArgs;
+int fb_gqa_prep(const FbGqaArgs* args, void* stream);
+int fb_gqa_attention(const FbGqaArgs* args, void* stream);      // dim, vdim <= 512
+
 // ---- gated delta rule (see delta_rule.cu) ------------------------------------------------------------------
 typedef struct FbDeltaArgs {
   const void* proj;         // [rows, ldp] projected rows: q | k | v inputs of the convolutions, beta logits
@@ -238,6 +352,9 @@ typedef struct FbDeltaArgs {
   const float* ag;          // [rows, ldag]: decay pre-activation [heads * dim] at 0, output gate [heads * vdim] at off_gate
   long long ldag;
   int off_gate;
+  int off_a;                // >= 0: one decay per head, pre-activation in projected columns off_a .. (dt_bias: [heads])
+  int off_g;                // >= 0: output gate pre-activation in projected columns off_g .. instead of `ag`
+  int gate_silu;            // output gate's activation: 0 sigmoid, 1 silu
   int fp32;                 // activations (proj, tail, out) are fp32 instead of bf16
   const float* conv;        // [taps, 2 * kv_heads * dim + heads * vdim]
   const float* a_neg;       // [heads] = -exp(A_log)

@@ -10,6 +10,7 @@
 // tcgen05.mma, four warps drain TMEM and run the fused epilogue:
 //
 //   kEpiStore   : out[row, n]            = acc                      (bf16 or fp32)
+//   kEpiGelu    : out[row, n]            = gelu(acc)                (exact, error-function form)
 //   kEpiSwiGLU  : out[row, n]            = silu(gate) * up          (two weight tiles per k-block)
 //   kEpiScatter : out[dst_row[row], n]   = acc * row_scale[row]     (MoE down projection)
 //   kEpiAllReduce: partial tiles are pushed into every rank's receive buffer over
@@ -34,7 +35,7 @@ constexpr int kBlockK = 64;   // bf16 elements per k-block = one 128-byte swizzl
 constexpr int kUmmaK = 16;
 constexpr int kGemmThreads = 192;
 
-enum { kEpiStore = 0, kEpiSwiGLU = 1, kEpiScatter = 2, kEpiAllReduce = 3 };
+enum { kEpiStore = 0, kEpiSwiGLU = 1, kEpiScatter = 2, kEpiAllReduce = 3, kEpiGelu = 4 };
 
 struct GemmParams {
   int n_out;          // output channels per group
@@ -412,6 +413,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
+              if (EPI == kEpiGelu) x = gelu_f(x);
               if (EPI == kEpiScatter && p.row_scale) x *= p.row_scale[row0 + r];
             }
             sb[j * 128 + ch_in_tile] = __float2bfloat16_rn(x);
@@ -450,6 +452,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
+              if (EPI == kEpiGelu) x = gelu_f(x);
               long long orow = row0 + r;
               if (EPI == kEpiScatter) {
                 if (p.row_scale) x *= p.row_scale[row0 + r];
@@ -753,7 +756,7 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (a == nullptr || a->w == nullptr || a->x == nullptr || a->out == nullptr) return FB_ERR_SHAPE;
   if (a->n_out <= 0 || a->k <= 0 || a->groups <= 0 || (a->k % 8) != 0) return FB_ERR_SHAPE;
-  if (a->epilogue < 0 || a->epilogue > 3) return FB_ERR_SHAPE;
+  if (a->epilogue < 0 || a->epilogue > 4) return FB_ERR_SHAPE;
   const bool dual = a->epilogue == kEpiSwiGLU;
   const int ntok = a->ntok;
   if (ntok != 16 && ntok != 32 && ntok != 64 && ntok != 128 && ntok != 256) return FB_ERR_SHAPE;
@@ -852,5 +855,6 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
     }
     return launch_ntok<false, kEpiScatter>(ntok, mw, mx, p, max_tiles, grouped, stream);
   }
+  if (a->epilogue == kEpiGelu) return launch_ntok<false, kEpiGelu>(ntok, mw, mx, p, max_tiles, grouped, stream);
   return launch_ntok<false, kEpiStore>(ntok, mw, mx, p, max_tiles, grouped, stream);
 }

@@ -1,0 +1,294 @@
+// Grouped-query attention inside position-aligned chunks, over paged keys and values.
+//
+// A query at position i sees the keys floor(i / chunk) * chunk .. i; query head h reads key / value head h / (H / G).  A
+// cache row holds [G][dim_pad] keys | [G][vdim_pad] values (heads padded to multiples of 8, padding is zero).
+//
+//   fb_gqa_prep       everything between the projection and the attention in one launch: query and key RMS norm over the
+//                     whole projection, rotation of the leading dimensions (halves paired), value norm per head, mixing
+//                     with the first mixing layer's values of the token (read from that layer's cache row), cache append
+//   fb_gqa_attention  attention in 32-bit arithmetic, one CTA per (query row, head): models that run in fp32, and head sizes
+//                     the tensor-core kernels do not take
+#include "act_type.cuh"
+#include "common.cuh"
+#include "ferrule_b200.h"
+#include "launch.cuh"
+
+namespace fb {
+
+template <typename T>
+struct GqaParams {
+  T* q;
+  long long ldq;
+  const T* k;
+  const T* v;
+  long long ldkv;
+  const float* q_norm;
+  const float* k_norm;
+  const float* cos_t;
+  const float* sin_t;
+  int max_pos, half;
+  const int* positions;
+  const long long* write_slot;
+  T* pool;
+  long long pool_rows, pool_ld;
+  const T* first_pool;
+  long long first_off;
+  float v_mix;
+  const int* block_table;
+  const int* row_seq;
+  const int* row_pos;
+  int num_seqs, max_blocks, page_size, chunk;
+  float scale, eps;
+  T* out;
+  long long ldo;
+  int rows, heads, kv_heads, dim, dim_pad, vdim, vdim_pad;
+  DeviceStatus* status;
+};
+
+// normalised rows of `heads` heads in shared memory -> rotated, into `dst` (8 elements per step)
+template <typename T>
+__device__ __forceinline__ void rotate_store(const float* row, int heads, const GqaParams<T>& p, const float* cs,
+                                             const float* sn, T* dst) {
+  const int vecs = p.dim_pad / 8;
+  for (int i = threadIdx.x; i < heads * vecs; i += blockDim.x) {
+    const int d0 = (i % vecs) * 8;
+    const float* h = row + (i / vecs) * p.dim_pad;
+    float o[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const int d = d0 + j;
+      if (d < p.half) o[j] = h[d] * cs[d] - h[d + p.half] * sn[d];
+      else if (d < 2 * p.half) o[j] = h[d] * cs[d - p.half] + h[d - p.half] * sn[d - p.half];
+      else o[j] = h[d];
+    }
+    act_store8(dst + static_cast<long long>(i) * 8, o);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gqa_prep_kernel(const GqaParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float sm[];
+  __shared__ float red[2][32];
+  const int nq = p.heads * p.dim_pad, nk = p.kv_heads * p.dim_pad;
+  float* sq = sm;
+  float* sk = sq + nq;
+  float* cs = sk + nk;
+  float* sn = cs + p.half;
+  const long long r = blockIdx.x;
+  int pos = p.positions[r];
+  if (pos < 0 || pos >= p.max_pos) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD60, r, pos);
+    pos = 0;
+  }
+  const long long slot = p.write_slot[r];
+  const bool keep = slot >= 0 && slot < p.pool_rows;
+  if (!keep && slot != -1 && threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD61, r, static_cast<uint32_t>(slot));
+  float ssq = 0.f, ssk = 0.f;
+  for (int i = threadIdx.x * 8; i < nq; i += blockDim.x * 8) {
+    float v[8];
+    act_load8(p.q + r * p.ldq + i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      ssq = fmaf(v[j], v[j], ssq);
+      sq[i + j] = v[j];
+    }
+  }
+  for (int i = threadIdx.x * 8; i < nk; i += blockDim.x * 8) {
+    float v[8];
+    act_load8(p.k + r * p.ldkv + i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      ssk = fmaf(v[j], v[j], ssk);
+      sk[i + j] = v[j];
+    }
+  }
+  for (int i = threadIdx.x; i < p.half; i += blockDim.x) {
+    cs[i] = p.cos_t[static_cast<long long>(pos) * p.half + i];
+    sn[i] = p.sin_t[static_cast<long long>(pos) * p.half + i];
+  }
+  ssq = cta_sum(ssq, red[0]);
+  ssk = cta_sum(ssk, red[1]);
+  const float iq = 1.f / sqrtf(ssq / (p.heads * p.dim) + p.eps), ik = 1.f / sqrtf(ssk / (p.kv_heads * p.dim) + p.eps);
+  for (int i = threadIdx.x; i < nq; i += blockDim.x) sq[i] *= iq * p.q_norm[i];
+  for (int i = threadIdx.x; i < nk; i += blockDim.x) sk[i] *= ik * p.k_norm[i];
+  __syncthreads();
+  rotate_store(sq, p.heads, p, cs, sn, p.q + r * p.ldq);
+  if (!keep) return;
+  T* row = p.pool + slot * p.pool_ld;
+  rotate_store(sk, p.kv_heads, p, cs, sn, row);
+  // values: one warp per head
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  for (int g = warp; g < p.kv_heads; g += nw) {
+    const T* v = p.v + r * p.ldkv + g * p.vdim_pad;
+    float ss = 0.f;
+    for (int d = lane; d < p.vdim; d += 32) {
+      const float x = act_load(v + d);
+      ss = fmaf(x, x, ss);
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / p.vdim + p.eps);
+    T* dst = row + nk + g * p.vdim_pad;
+    const T* first = p.first_pool ? p.first_pool + slot * p.pool_ld + p.first_off + g * p.vdim_pad : nullptr;
+    for (int d = lane; d < p.vdim_pad; d += 32) {
+      float x = d < p.vdim ? act_load(v + d) * inv : 0.f;
+      if (first) x = fmaf(p.v_mix, act_load(first + d), (1.f - p.v_mix) * x);
+      act_store(dst + d, x);
+    }
+  }
+}
+
+// DPL: query / key and value features per lane
+template <typename T, int DPL>
+__global__ void __launch_bounds__(128)
+gqa_attention_kernel(const GqaParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sm_m[4], sm_l[4];
+  __shared__ float sm_o[4][DPL * 32];
+  const int r = blockIdx.x, h = blockIdx.y, g = h / (p.heads / p.kv_heads);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int seq = p.row_seq[r], pos = p.row_pos[r];
+  int len = pos + 1;
+  if (seq < 0 || seq >= p.num_seqs) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD70, r, seq);
+    len = 0;
+  }
+  len = min(len, p.max_blocks * p.page_size);
+  const int first = pos >= 0 ? pos / p.chunk * p.chunk : 0;
+  const long long koff = static_cast<long long>(g) * p.dim_pad;
+  const long long voff = static_cast<long long>(p.kv_heads) * p.dim_pad + static_cast<long long>(g) * p.vdim_pad;
+  float q[DPL], o[DPL];
+#pragma unroll
+  for (int j = 0; j < DPL; ++j) {
+    const int d = lane + 32 * j;
+    q[j] = d < p.dim ? act_load(p.q + r * p.ldq + static_cast<long long>(h) * p.dim_pad + d) : 0.f;
+    o[j] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int t = first + warp; t < len; t += 4) {
+    const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+    const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
+    if (page < 0 || slot >= p.pool_rows) {
+      if (lane == 0) report_status(p.status, kStatusBadIndex, 0xD71, seq, t);
+      continue;
+    }
+    const T* row = p.pool + slot * p.pool_ld;
+    float s = 0.f, v[DPL];
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) {
+      const int d = lane + 32 * j;
+      s = fmaf(q[j], d < p.dim ? act_load(row + koff + d) : 0.f, s);
+      v[j] = d < p.vdim ? act_load(row + voff + d) : 0.f;
+    }
+    s = warp_sum(s) * p.scale;
+    if (s > m) {
+      const float a = expf(m - s);
+      m = s;
+      l *= a;
+#pragma unroll
+      for (int j = 0; j < DPL; ++j) o[j] *= a;
+    }
+    const float w = expf(s - m);
+    l += w;
+#pragma unroll
+    for (int j = 0; j < DPL; ++j) o[j] = fmaf(w, v[j], o[j]);
+  }
+  if (lane == 0) { sm_m[warp] = m; sm_l[warp] = l; }
+#pragma unroll
+  for (int j = 0; j < DPL; ++j) sm_o[warp][lane + 32 * j] = o[j];
+  __syncthreads();
+  const float M = fmaxf(fmaxf(sm_m[0], sm_m[1]), fmaxf(sm_m[2], sm_m[3]));
+  float w[4], L = 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    w[k] = sm_m[k] == -INFINITY ? 0.f : expf(sm_m[k] - M);
+    L += w[k] * sm_l[k];
+  }
+  const float f = L > 0.f ? 1.f / L : 0.f;
+  T* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.vdim_pad;
+  for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x)
+    act_store(dst + d, d < p.vdim ? (w[0] * sm_o[0][d] + w[1] * sm_o[1][d] + w[2] * sm_o[2][d] + w[3] * sm_o[3][d]) * f : 0.f);
+}
+
+template <typename T>
+static void fill_gqa(const FbGqaArgs* a, GqaParams<T>& p) {
+  p.q = static_cast<T*>(a->q); p.ldq = a->ldq;
+  p.k = static_cast<const T*>(a->k); p.v = static_cast<const T*>(a->v); p.ldkv = a->ldkv;
+  p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.cos_t = a->cos_t; p.sin_t = a->sin_t;
+  p.max_pos = a->max_pos; p.half = a->rot_dims / 2;
+  p.positions = a->positions; p.write_slot = a->write_slot;
+  p.pool = static_cast<T*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
+  p.first_pool = static_cast<const T*>(a->first_pool); p.first_off = a->first_off; p.v_mix = a->v_mix;
+  p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
+  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size; p.chunk = a->chunk;
+  p.scale = a->scale; p.eps = a->eps;
+  p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
+  p.rows = a->rows; p.heads = a->heads; p.kv_heads = a->kv_heads;
+  p.dim = a->dim; p.dim_pad = a->dim_pad; p.vdim = a->vdim; p.vdim_pad = a->vdim_pad;
+  p.status = static_cast<DeviceStatus*>(a->status);
+}
+
+static bool gqa_sizes_ok(const FbGqaArgs* a) {
+  return a && a->q && a->pool && a->rows > 0 && a->heads > 0 && a->heads <= 65535 && a->kv_heads > 0 &&
+         a->heads % a->kv_heads == 0 && a->dim > 0 && a->vdim > 0 && a->dim_pad >= a->dim && a->vdim_pad >= a->vdim &&
+         a->dim_pad % 8 == 0 && a->vdim_pad % 8 == 0 && a->pool_rows > 0 && a->pool_ld % 8 == 0 &&
+         a->pool_ld >= static_cast<long long>(a->kv_heads) * (a->dim_pad + a->vdim_pad) && a->ldq % 8 == 0 &&
+         a->ldq >= static_cast<long long>(a->heads) * a->dim_pad;
+}
+
+template <typename T>
+static int run_prep(const FbGqaArgs* a, cudaStream_t s) {
+  GqaParams<T> p{};
+  fill_gqa(a, p);
+  const size_t smem = (static_cast<size_t>(a->heads + a->kv_heads) * a->dim_pad + a->rot_dims) * sizeof(float);
+  if (smem > 200 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(gqa_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(gqa_prep_kernel<T>, dim3(a->rows), dim3(256), smem, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int run_attention(const FbGqaArgs* a, cudaStream_t s) {
+  GqaParams<T> p{};
+  fill_gqa(a, p);
+  const dim3 grid(a->rows, a->heads);
+  const int d = ((a->dim > a->vdim ? a->dim : a->vdim) + 31) / 32;
+  if (d <= 2) launch_pdl(gqa_attention_kernel<T, 2>, grid, dim3(128), 0, s, p);
+  else if (d <= 4) launch_pdl(gqa_attention_kernel<T, 4>, grid, dim3(128), 0, s, p);
+  else if (d <= 8) launch_pdl(gqa_attention_kernel<T, 8>, grid, dim3(128), 0, s, p);
+  else launch_pdl(gqa_attention_kernel<T, 16>, grid, dim3(128), 0, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_gqa_prep(const FbGqaArgs* a, void* stream) {
+  if (!gqa_sizes_ok(a) || !a->k || !a->v || !a->q_norm || !a->k_norm || !a->positions || !a->write_slot || a->max_pos <= 0 ||
+      a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->dim || (a->rot_dims && (!a->cos_t || !a->sin_t)))
+    return FB_ERR_SHAPE;
+  if (a->ldkv % 8 || a->first_off < 0 || a->first_off + static_cast<long long>(a->kv_heads) * a->vdim_pad > a->pool_ld)
+    return FB_ERR_SHAPE;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) |
+                         reinterpret_cast<uintptr_t>(a->pool);
+  if (bits & 15) return FB_ERR_ALIGN;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return a->fp32 ? run_prep<float>(a, s) : run_prep<__nv_bfloat16>(a, s);
+}
+
+extern "C" int fb_gqa_attention(const FbGqaArgs* a, void* stream) {
+  if (!gqa_sizes_ok(a) || !a->out || !a->block_table || !a->row_seq || !a->row_pos || a->num_seqs <= 0 || a->max_blocks <= 0 ||
+      a->page_size <= 0 || a->chunk <= 0 || a->ldo < static_cast<long long>(a->heads) * a->vdim_pad)
+    return FB_ERR_SHAPE;
+  if (a->dim > 512 || a->vdim > 512) return FB_ERR_LIMIT;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return a->fp32 ? run_attention<float>(a, s) : run_attention<__nv_bfloat16>(a, s);
+}

@@ -1,0 +1,222 @@
+// Selective scan: a diagonal recurrence per channel c and state n, with the token's own step size, input and read-out:
+//
+//     d = softplus(dt_c + bias_c);   S[c, n] <- exp(d A[c, n]) S[c, n] + d x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
+//     out_c = y_c * silu(z_c)
+//
+// One kernel serves prompts and decode steps: CTA = (128 / LPC channels) x sequence, LPC lanes share a channel and hold
+// SPL states each in registers.  Tokens are staged sixteen at a time; the next ones are requested before the staged ones
+// are worked on.  The exponentials do not depend on the state, so a token's chain is one multiply-add per state.
+//
+// State of a sequence: fp32 [state, inner], channels innermost.  Buffer `state_in[seq]` is read (-1: a new sequence,
+// zeros), buffer `state_out[seq]` written (-1: nothing is kept), never the same one.
+#include "act_type.cuh"
+#include "common.cuh"
+#include "ferrule_b200.h"
+#include "launch.cuh"
+
+namespace fb {
+
+constexpr int kScanThreads = 128;
+constexpr int kScanTokens = 16;
+
+template <typename T>
+struct ScanParams {
+  const T* x;
+  long long ldx;
+  const T* z;
+  long long ldz;
+  const T* bc;
+  long long ldbc;
+  int off_b, off_c;
+  const float* dt;
+  long long lddt;
+  const float* dt_bias;
+  const float* a_log2;
+  const float* d_skip;
+  float* states;
+  const int* seq_start;
+  const int* state_in;
+  const int* state_out;
+  T* out;
+  long long ldo;
+  int rows, n_seqs, inner, state, n_states;
+  DeviceStatus* status;
+};
+
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// bf16 models take the hardware exponential and logarithm (a few 1e-7 relative), fp32 models the full-precision functions
+template <typename T>
+__device__ __forceinline__ float scan_exp2(float x) { return sizeof(T) == 4 ? exp2f(x) : exp2_approx(x); }
+template <typename T>
+__device__ __forceinline__ float scan_softplus(float z) {
+  if constexpr (sizeof(T) == 4) return softplus_f(z);
+  const float e = __expf(-fabsf(z)), w = 1.f + e;
+  // log1p(e) = log(w) * e / (w - 1): the quotient restores what rounding w lost
+  const float l = w == 1.f ? e : __logf(w) * __fdividef(e, w - 1.f);
+  return fmaxf(z, 0.f) + l;
+}
+template <typename T>
+__device__ __forceinline__ float scan_silu(float z) {
+  if constexpr (sizeof(T) == 4) return z / (1.f + expf(-z));
+  return __fdividef(z, 1.f + __expf(-z));
+}
+
+template <typename T, int LPC, int SPL>
+__global__ void __launch_bounds__(kScanThreads)
+selective_scan_kernel(const ScanParams<T> p) {
+  constexpr int CH = kScanThreads / LPC, NP = LPC * SPL, TS = kScanTokens;
+  constexpr int kPf = TS * CH / kScanThreads;                        // staged (token, channel) pairs per thread
+  constexpr int kBc = (2 * TS * NP + kScanThreads - 1) / kScanThreads;
+  __shared__ float s_d[TS][CH], s_x[TS][CH], s_y[TS][CH];
+  __shared__ __align__(16) float s_b[TS][NP], s_c[TS][NP];
+  const int tid = threadIdx.x, l = tid % LPC, ch = tid / LPC;
+  const int seq = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
+  const int sin = p.state_in[seq], sout = p.state_out[seq];
+  const bool ok = sin < p.n_states && sout < p.n_states && !(sin >= 0 && sin == sout);
+  const bool cin = c < p.inner;
+  float a2[SPL], S[SPL];
+#pragma unroll
+  for (int j = 0; j < SPL; ++j) {
+    const int n = l * SPL + j;
+    const bool in = cin && n < p.state;
+    a2[j] = in ? p.a_log2[static_cast<long long>(n) * p.inner + c] : 0.f;
+    S[j] = in && ok && sin >= 0 ? p.states[(static_cast<long long>(sin) * p.state + n) * p.inner + c] : 0.f;
+  }
+  // staging role of this thread: channel `pc` of tokens pt, pt + 128 / CH, ...
+  const int pc = tid % CH, pt = tid / CH;
+  constexpr int kStep = kScanThreads / CH;
+  const bool pin = c0 + pc < p.inner;
+  const float bias = pin ? p.dt_bias[c0 + pc] : 0.f, skip = pin ? p.d_skip[c0 + pc] : 0.f;
+  pdl_wait();
+  if (!ok) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xD40, seq, sout);
+    return;
+  }
+  const int r0 = p.seq_start[seq], cnt_all = p.seq_start[seq + 1] - r0;
+  if (r0 < 0 || cnt_all <= 0 || r0 + cnt_all > p.rows) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xD41, seq, r0);
+    return;
+  }
+  float fd[kPf], fx[kPf], fz[kPf], fz_next[kPf], fbc[kBc];
+  auto fetch = [&](int t0) {
+    const int cnt = min(TS, cnt_all - t0);
+#pragma unroll
+    for (int k = 0; k < kPf; ++k) {
+      const int t = pt + k * kStep;
+      fd[k] = fx[k] = fz_next[k] = 0.f;
+      if (t < cnt && pin) {
+        const long long r = r0 + t0 + t;
+        fd[k] = p.dt[r * p.lddt + c0 + pc];
+        fx[k] = act_load(p.x + r * p.ldx + c0 + pc);
+        fz_next[k] = act_load(p.z + r * p.ldz + c0 + pc);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < kBc; ++k) {
+      const int i = tid + k * kScanThreads, t = i / (2 * NP), n = i % (2 * NP), m = n % NP;
+      fbc[k] = 0.f;
+      if (t < cnt && m < p.state)
+        fbc[k] = act_load(p.bc + (r0 + t0 + t) * p.ldbc + (n < NP ? p.off_b : p.off_c) + m);
+    }
+  };
+  fetch(0);
+  for (int t0 = 0; t0 < cnt_all; t0 += TS) {
+    const int cnt = min(TS, cnt_all - t0);
+#pragma unroll
+    for (int k = 0; k < kPf; ++k) {
+      const int t = pt + k * kStep;
+      s_d[t][pc] = scan_softplus<T>(fd[k] + bias);
+      s_x[t][pc] = fx[k];
+      fz[k] = fz_next[k];
+    }
+#pragma unroll
+    for (int k = 0; k < kBc; ++k) {
+      const int i = tid + k * kScanThreads, t = i / (2 * NP), n = i % (2 * NP);
+      if (t < TS) (n < NP ? s_b[t][n] : s_c[t][n - NP]) = fbc[k];
+    }
+    __syncthreads();
+    if (t0 + TS < cnt_all) fetch(t0 + TS);
+    auto token = [&](int t) {
+      const float d = s_d[t][ch], u = d * s_x[t][ch];
+      float y = 0.f;
+#pragma unroll
+      for (int j = 0; j < SPL; ++j) {
+        S[j] = fmaf(scan_exp2<T>(d * a2[j]), S[j], u * s_b[t][l * SPL + j]);
+        y = fmaf(S[j], s_c[t][l * SPL + j], y);
+      }
+#pragma unroll
+      for (int o = 1; o < LPC; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+      if (l == 0) s_y[t][ch] = y;
+    };
+    if (cnt == TS) {
+#pragma unroll 4
+      for (int t = 0; t < TS; ++t) token(t);
+    } else {
+      for (int t = 0; t < cnt; ++t) token(t);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kPf; ++k) {
+      const int t = pt + k * kStep;
+      if (t < cnt && pin)
+        act_store(p.out + (r0 + t0 + t) * p.ldo + c0 + pc, fmaf(skip, s_x[t][pc], s_y[t][pc]) * scan_silu<T>(fz[k]));
+    }
+    // the next round overwrites this thread's own s_d / s_x entries, and s_b / s_c, last read before the barrier above;
+    // s_y is written again behind the next barrier
+  }
+  pdl_launch_dependents();
+  if (sout >= 0 && cin) {
+#pragma unroll
+    for (int j = 0; j < SPL; ++j) {
+      const int n = l * SPL + j;
+      if (n < p.state) p.states[(static_cast<long long>(sout) * p.state + n) * p.inner + c] = S[j];
+    }
+  }
+}
+
+template <typename T, int LPC, int SPL>
+static int launch_scan_form(const ScanParams<T>& p, cudaStream_t s) {
+  constexpr int CH = kScanThreads / LPC;
+  launch_pdl(selective_scan_kernel<T, LPC, SPL>, dim3((p.inner + CH - 1) / CH, p.n_seqs), dim3(kScanThreads), 0, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int run_scan(const FbScanArgs* a, cudaStream_t s) {
+  ScanParams<T> p{};
+  p.x = static_cast<const T*>(a->x); p.ldx = a->ldx;
+  p.z = static_cast<const T*>(a->z); p.ldz = a->ldz;
+  p.bc = static_cast<const T*>(a->bc); p.ldbc = a->ldbc; p.off_b = a->off_b; p.off_c = a->off_c;
+  p.dt = a->dt; p.lddt = a->lddt; p.dt_bias = a->dt_bias; p.a_log2 = a->a_log2; p.d_skip = a->d_skip;
+  p.states = a->states; p.seq_start = a->seq_start; p.state_in = a->state_in; p.state_out = a->state_out;
+  p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
+  p.rows = a->rows; p.n_seqs = a->n_seqs; p.inner = a->inner; p.state = a->state; p.n_states = a->n_states;
+  p.status = static_cast<DeviceStatus*>(a->status);
+  if (p.state <= 8) return launch_scan_form<T, 4, 2>(p, s);
+  if (p.state <= 16) return launch_scan_form<T, 4, 4>(p, s);
+  if (p.state <= 32) return launch_scan_form<T, 4, 8>(p, s);
+  if (p.state <= 64) return launch_scan_form<T, 8, 8>(p, s);
+  return launch_scan_form<T, 16, 8>(p, s);
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_selective_scan(const FbScanArgs* a, void* stream) {
+  if (!a || !a->x || !a->z || !a->bc || !a->dt || !a->dt_bias || !a->a_log2 || !a->d_skip || !a->states || !a->seq_start ||
+      !a->state_in || !a->state_out || !a->out)
+    return FB_ERR_SHAPE;
+  if (a->rows <= 0 || a->n_seqs <= 0 || a->n_seqs > 65535 || a->inner <= 0 || a->state <= 0 || a->n_states <= 0)
+    return FB_ERR_SHAPE;
+  if (a->state > 128) return FB_ERR_LIMIT;
+  if (a->ldx < a->inner || a->ldz < a->inner || a->lddt < a->inner || a->ldo < a->inner || a->off_b < 0 || a->off_c < 0 ||
+      a->ldbc < a->off_b + a->state || a->ldbc < a->off_c + a->state)
+    return FB_ERR_SHAPE;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return a->fp32 ? run_scan<float>(a, s) : run_scan<__nv_bfloat16>(a, s);
+}

@@ -40,7 +40,7 @@ import torch.nn.functional as F
 from ..ops import reference as ref
 from .config import SCORE_SOFTMAX
 from .deepseek import DeviceBatch, KvPool, _pow2_at_least
-from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, MambaMixer,
+from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, AttentionMixer, DeltaMixer, LatentMixer, MambaMixer,
                              MoeSpec, pad_to)
 from .layered_weights import LayerImage, LayeredWeights, MixerImage
 from .state_pool import RecurrentStatePool
@@ -285,16 +285,25 @@ class LayeredWorkspace:
         self.proj = torch.zeros(R * max(l.mixer.w_in.shape[0] for l in w.layers), **act)
         self.mix_in = torch.zeros(R * max(l.mixer.w_o.shape[1] for l in w.layers), **act)
         self.mix = torch.zeros(R, Wp, **act)
-        latent = [cfg.layers[i].mixer for i in cfg.latent_layers]
-        delta = [cfg.layers[i].mixer for i in cfg.delta_layers]
+        latent, delta, mamba = ([cfg.layers[i].mixer for i in ids] for ids in (cfg.latent_layers, cfg.delta_layers,
+                                                                               cfg.mamba_layers))
         if latent:
             n = max(m.heads for m in latent) * DL
             self.q_lat = torch.zeros(R * n, **act)
             self.o_lat = torch.zeros(R * n, **act)
         if delta:
-            self.ag = torch.zeros(R * max(w.layers[i].mixer.w_ag.shape[0] for i in cfg.delta_layers), **f32)
+            low = [l.mixer.w_ag for l in w.layers if l.mixer.w_ag is not None]
+            self.ag = torch.zeros(R * max((t.shape[0] for t in low), default=0), **f32)
             self.delta = KL.DeltaScratch(R, delta, device)
-        moes = [(i, l.mlp) for i, l in enumerate(cfg.layers) if l.mlp is not None]
+        if mamba:
+            n = max(m.inner_pad for m in mamba)
+            self.conv_x = torch.zeros(R * n, **act)
+            self.dt = torch.zeros(R * n, **f32)
+            self.low = torch.zeros(R * max(l.mixer.w_x.shape[0] for l in w.layers if l.mixer.w_x is not None), **act)
+        if any(l.w_up is not None for l in w.layers):
+            self.ff = torch.zeros(R * max(l.w_up.shape[0] for l in w.layers if l.w_up is not None), **act)
+            self.act = torch.zeros(R, Wp, **act)
+        moes = [(i, l.mlp) for i, l in enumerate(cfg.layers) if isinstance(l.mlp, MoeSpec)]
         self.plans: Dict[tuple, MoePlan] = {}
         self.static_plans: Dict[tuple, MoePlan] = {}
         self.static_rows = (16, 32, 64)
@@ -341,7 +350,15 @@ class LayeredCuda:
         self.attn_splits = attn_splits
         self.split_tokens = max(64, pad_to((max_seq_len + attn_splits - 1) // attn_splits, 64))
         self.ws = LayeredWorkspace(weights, max_rows, max_logit_rows, self.device)
-        self.latent_index = {l: i for i, l in enumerate(self.cfg.latent_layers)}
+        self.cache_index = {l: i for i, l in enumerate(self.cfg.cache_layers)}
+        # cosines and sines of every rotation in use, computed in double
+        self.rotation: Dict[tuple, tuple] = {}
+        for i in self.cfg.attention_layers:
+            m = self.cfg.layers[i].mixer
+            if (m.rot_base, m.rot_dims) not in self.rotation:
+                a = (torch.arange(min(max_seq_len, self.cfg.max_position), dtype=torch.float64)[:, None]
+                     * rotation_frequencies(m.rot_base, m.rot_dims))
+                self.rotation[m.rot_base, m.rot_dims] = tuple(f(a).float().to(self.device) for f in (torch.cos, torch.sin))
         # the tensor-core attention kernels take latents up to 512 features
         self.mma_attention = not self.fp32 and self.cfg.kv_row_dim <= 512
         self.static_moe = not self.fp32 and self.cfg.width_pad <= 8192
@@ -349,11 +366,15 @@ class LayeredCuda:
         self.launches = 0
         self.last_hidden = None
         self.prof = self.tap = None
-        for i in self.cfg.delta_layers:
-            if self.cfg.layers[i].mixer.dim > 256:
-                raise ValueError("delta mixers wider than 256 key channels per head are not supported")
         for l in self.cfg.layers:
-            if l.mlp is not None and (l.mlp.experts > 256 or l.mlp.top > 32 or l.mlp.groups > 32):
+            m, f = l.mixer, l.mlp
+            if isinstance(m, DeltaMixer) and m.dim > 256:
+                raise ValueError("delta mixers wider than 256 key channels per head are not supported")
+            if isinstance(m, MambaMixer) and m.state > 128:
+                raise ValueError("selective scans with more than 128 states per channel are not supported")
+            if isinstance(m, AttentionMixer) and max(m.dim, m.vdim) > 512:
+                raise ValueError("attention heads wider than 512 are not supported")
+            if isinstance(f, MoeSpec) and (f.experts > 256 or f.top > 32 or f.groups > 32):
                 raise ValueError("the router takes at most 256 experts, top 32, 32 groups")
 
     @staticmethod
@@ -396,15 +417,51 @@ class LayeredCuda:
     def _delta(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         K, KL, ws = self.K, self.KL, self.ws
         mx, m = lw.mixer, lw.spec.mixer
-        ag = self._view(ws.ag, T, mx.w_ag.shape[0])
-        a0 = mx.off["a1"]
-        K.gemm(proj[:, a0:a0 + mx.w_ag.shape[1]], mx.w_ag, out=ag)
+        ag = None
+        if m.low_rank:
+            ag = self._view(ws.ag, T, mx.w_ag.shape[0])
+            a0 = mx.off["a1"]
+            K.gemm(proj[:, a0:a0 + mx.w_ag.shape[1]], mx.w_ag, out=ag)
         out = self._view(ws.mix_in, T, mx.w_o.shape[1])
         decode = b.n_seqs == T and KL.delta_decode_supported(m)
         KL.delta_rule(proj, mx.off, ag, mx, m, self.cfg.norm_eps, self.states.state[layer], self.states.tail[layer],
                       b.seq_start, b.state_in, b.state_out, b.n_seqs, out, row_seq=b.row_seq[:T], scratch=ws.delta,
                       decode=decode)
         return out
+
+    def _attention(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        KL, cfg = self.KL, self.cfg
+        mx, m = lw.mixer, lw.spec.mixer
+        pool = self.pool.layer(self.cache_index[layer])
+        q = proj[:, mx.off["q"]:mx.off["q"] + m.heads * m.dim_pad]
+        first = cfg.first_value_layer if m.v_mix else layer
+        mixed = {} if first == layer else dict(first_pool=self.pool.layer(self.cache_index[first]),
+                                               first_off=cfg.layers[first].mixer.v_offset)
+        KL.gqa_prep(q, proj[:, mx.off["k"]:], proj[:, mx.off["v"]:], m, mx, self.rotation[m.rot_base, m.rot_dims],
+                    b.positions[:T], b.write_slot[:T], pool, cfg.norm_eps, **mixed)
+        out = self._view(self.ws.mix_in, T, m.heads * m.vdim_pad)
+        return KL.gqa_attention(q, m, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, out)
+
+    def _mamba(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        K, KL, ws = self.K, self.KL, self.ws
+        mx, m = lw.mixer, lw.spec.mixer
+        Ip = m.inner_pad
+        seqs = (b.seq_start, b.state_in, b.state_out, b.n_seqs)
+        x = self._view(ws.conv_x, T, Ip)
+        KL.short_conv(proj[:, mx.off["x"]:mx.off["x"] + Ip], mx.conv, self.states.tail[layer], x, b.row_seq[:T], *seqs,
+                      bias=mx.conv_b, silu=True)
+        low = self._view(ws.low, T, mx.w_x.shape[0])
+        K.gemm(x, mx.w_x, out=low)
+        dt = self._view(ws.dt, T, Ip)
+        K.gemm(low[:, :mx.w_dt.shape[1]], mx.w_dt, out=dt)
+        out = self._view(ws.mix_in, T, Ip)
+        return KL.selective_scan(x, proj[:, mx.off["z"]:mx.off["z"] + Ip], low, mx.off_b, mx.off_c, dt, mx,
+                                 self.states.state[layer], *seqs, out)
+
+    def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, DeltaMixer: self._delta,
+              MambaMixer: self._mamba}[type(lw.spec.mixer)]
+        return fn(layer, lw, proj, b, T)
 
     # -- feed-forward ------------------------------------------------------------------------
     def _moe(self, layer: int, lw: LayerImage, h: torch.Tensor, T: int) -> torch.Tensor:
@@ -443,16 +500,32 @@ class LayeredCuda:
         K.gemm(hmid, lw.e_w2, out=route_out, epilogue=K.EPI_SCATTER, plan=scatter_plan, scatter_rows=T * k)
         return route_out.view(T, k, Wp)
 
-    # -- whole model ---------------------------------------------------------------------
-    def hidden_states(self, b: DeviceBatch, T: int) -> torch.Tensor:
-        """Runs the layers; returns the normalised rows the head reads (`ws.h`); `ws.x` holds the residual stream."""
-        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+    # -- blocks ----------------------------------------------------------------------------
+    def _mix(self, i: int, lw: LayerImage, h: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        """Input projection, mixer and output projection (into `ws.mix`); returns the projected rows."""
+        K, ws, mx, prof = self.K, self.ws, lw.mixer, self.prof
+        if prof is not None:
+            prof.mark(i, "proj")
+        proj = self._view(ws.proj, T, mx.w_in.shape[0])
+        K.gemm(h, mx.w_in, out=proj)
+        if prof is not None:
+            prof.mark(i, "mixer")
+        a = self._mixer(i, lw, proj, b, T)
+        if prof is not None:
+            prof.mark(i, "mixer.out")
+        K.gemm(a, mx.w_o, out=ws.mix[:T])
+        return proj
+
+    def _tapped(self, i: int, x: torch.Tensor) -> None:
+        if self.tap is not None and self.tap.wants(i, "layer_out"):
+            self.tap.write(i, "layer_out", x)
+
+    def _gated_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+        KL, ws, cfg = self.KL, self.ws, self.cfg
         layers = self.w.layers
-        x, h = ws.x[:T], ws.h[:T]
         if self.static_moe and T <= ws.static_rows[-1] and ws.static_plans:
             self.M.fill_(ws.route_cnt, 0)
         KL.embed_norm(b.token_ids[:T], self.w.embed, x, layers[0].norm, h, cfg.width, cfg.norm_eps)
-        prof = self.prof
         for i, lw in enumerate(layers):
             mx = lw.mixer
             ffn = None
@@ -461,37 +534,68 @@ class LayeredCuda:
                 self.side_stream.wait_stream(main)
                 with torch.cuda.stream(self.side_stream):
                     ffn = self._moe(i, lw, h, T)
-            if prof is not None:
-                prof.mark(i, "proj")
-            proj = self._view(ws.proj, T, mx.w_in.shape[0])
-            K.gemm(h, mx.w_in, out=proj)
-            if prof is not None:
-                prof.mark(i, "mixer")
-            mixer = self._latent if isinstance(lw.spec.mixer, LatentMixer) else self._delta
-            a = mixer(i, lw, proj, b, T)
-            if prof is not None:
-                prof.mark(i, "mixer.out")
-            K.gemm(a, mx.w_o, out=ws.mix[:T])
+            proj = self._mix(i, lw, h, b, T)
             if ffn is not None:
                 torch.cuda.current_stream().wait_stream(self.side_stream)
-            if prof is not None:
-                prof.mark(i, "tail")
+            if self.prof is not None:
+                self.prof.mark(i, "tail")
             nxt = layers[i + 1].norm if i + 1 < len(layers) else self.w.final_norm
             KL.gated_residual_norm(
                 x, nxt, h, cfg.width, cfg.norm_eps, mix=ws.mix[:T], gate1=proj[:, mx.off["rg1"]:], bias1=lw.rg1_b,
                 ffn=ffn, topk=lw.spec.mlp.top if ffn is not None else 0,
                 gate2=proj[:, mx.off["rg2"]:] if ffn is not None else None, bias2=lw.rg2_b)
-            if self.tap is not None and self.tap.wants(i, "layer_out"):
-                self.tap.write(i, "layer_out", x)
-        if prof is not None:
-            prof.mark(len(layers), None)
-        return h
+            self._tapped(i, x)
+
+    def _output_norm_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+        layers, eps = self.w.layers, cfg.norm_eps
+        single = b.n_seqs == T          # one row per sequence: a row's earlier convolution inputs are all in the state
+        seqs = (b.seq_start, b.state_in, b.state_out, b.n_seqs)
+
+        def fused(i):
+            """Input convolution of layer i inside the kernel that completes its stream rows."""
+            if i >= len(layers) or not single or layers[i].canon is None:
+                return None
+            return layers[i].canon, self.states.canon[i], b.state_in, b.state_out, h
+
+        KL.embed_stream(b.token_ids[:T], self.w.embed, x, cfg.width, positions=b.positions[:T], pos_table=self.w.pos,
+                        canon=fused(0))
+        for i, lw in enumerate(layers):
+            if lw.canon is not None and not single:
+                KL.short_conv(x, lw.canon, self.states.canon[i], h, b.row_seq[:T], *seqs, residual=True)
+            self._mix(i, lw, h, b, T)
+            if self.prof is not None:
+                self.prof.mark(i, "tail")
+            if lw.spec.mlp is None:
+                KL.add_normed(x, ws.mix[:T], lw.norm1, cfg.width, eps, canon=fused(i + 1))
+            else:
+                act, ff = ws.act[:T], self._view(ws.ff, T, lw.w_up.shape[0])
+                KL.add_normed(x, ws.mix[:T], lw.norm1, cfg.width, eps, act=act)
+                K.gemm(act, lw.w_up, out=ff, epilogue=K.EPI_GELU)
+                K.gemm(ff, lw.w_down, out=ws.mix[:T])
+                KL.add_normed(x, ws.mix[:T], lw.norm2, cfg.width, eps, canon=fused(i + 1))
+            self._tapped(i, x)
+
+    # -- whole model ---------------------------------------------------------------------
+    def hidden_states(self, b: DeviceBatch, T: int) -> torch.Tensor:
+        """Runs the layers; `ws.x` holds the residual stream.  Returns the rows the head starts from: normalised ones
+        (`ws.h`) behind parallel gated blocks, the stream itself behind output-norm blocks."""
+        ws = self.ws
+        x, h = ws.x[:T], ws.h[:T]
+        gated = self.cfg.block == PARALLEL_GATED
+        (self._gated_blocks if gated else self._output_norm_blocks)(b, T, x, h)
+        if self.prof is not None:
+            self.prof.mark(len(self.w.layers), None)
+        return h if gated else x
 
     def head(self, h: torch.Tensor, logit_rows: torch.Tensor, L: int):
         """Logits and greedy tokens of `L` rows -> (next_id, next_val, logits), views of the workspace."""
         K, ws = self.K, self.ws
         hn = ws.hn_last[:L]
-        self.M.gather_rows(h, logit_rows[:L], hn)
+        if self.cfg.block == OUTPUT_NORM:
+            self.KL.norm_rows(h, logit_rows[:L], self.w.final_norm, hn, self.cfg.width, self.cfg.norm_eps)
+        else:
+            self.M.gather_rows(h, logit_rows[:L], hn)
         logits = ws.logits[:L]
         K.gemm(hn, self.w.lm_head, out=logits)
         if self.cfg.logit_softcap:

@@ -99,7 +99,8 @@ class DeltaArgs(C.Structure):
     _fields_ = [
         ("proj", C.c_void_p), ("ldp", C.c_longlong),
         ("off_q", C.c_int), ("off_k", C.c_int), ("off_v", C.c_int), ("off_b", C.c_int),
-        ("ag", C.c_void_p), ("ldag", C.c_longlong), ("off_gate", C.c_int), ("fp32", C.c_int),
+        ("ag", C.c_void_p), ("ldag", C.c_longlong), ("off_gate", C.c_int),
+        ("off_a", C.c_int), ("off_g", C.c_int), ("gate_silu", C.c_int), ("fp32", C.c_int),
         ("conv", C.c_void_p), ("a_neg", C.c_void_p), ("dt_bias", C.c_void_p), ("norm_w", C.c_void_p),
         ("state", C.c_void_p), ("tail", C.c_void_p), ("row_seq", C.c_void_p), ("seq_start", C.c_void_p),
         ("state_in", C.c_void_p), ("state_out", C.c_void_p),
@@ -108,6 +109,54 @@ class DeltaArgs(C.Structure):
         ("out", C.c_void_p), ("ldo", C.c_longlong), ("status", C.c_void_p),
         ("n_states", C.c_int), ("rows", C.c_int), ("n_seqs", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int),
         ("dim", C.c_int), ("vdim", C.c_int), ("taps", C.c_int), ("eps", C.c_float),
+    ]
+
+
+class StreamArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("ldx", C.c_longlong), ("ids", C.c_void_p), ("positions", C.c_void_p),
+        ("table", C.c_void_p), ("pos_table", C.c_void_p), ("ldt", C.c_longlong), ("vocab", C.c_int), ("max_pos", C.c_int),
+        ("y", C.c_void_p), ("ldy", C.c_longlong), ("norm_w", C.c_void_p), ("norm_b", C.c_void_p), ("rms", C.c_int),
+        ("act", C.c_void_p), ("lda", C.c_longlong), ("conv", C.c_void_p), ("tail", C.c_void_p),
+        ("state_in", C.c_void_p), ("state_out", C.c_void_p), ("taps", C.c_int), ("n_states", C.c_int),
+        ("h", C.c_void_p), ("ldh", C.c_longlong), ("rows", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int),
+        ("fp32", C.c_int), ("eps", C.c_float), ("status", C.c_void_p),
+    ]
+
+
+class ConvArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("ldx", C.c_longlong), ("w", C.c_void_p), ("bias", C.c_void_p), ("tail", C.c_void_p),
+        ("out", C.c_void_p), ("ldo", C.c_longlong), ("row_seq", C.c_void_p), ("seq_start", C.c_void_p),
+        ("state_in", C.c_void_p), ("state_out", C.c_void_p), ("rows", C.c_int), ("channels", C.c_int), ("taps", C.c_int),
+        ("n_states", C.c_int), ("n_seqs", C.c_int), ("x_fp32", C.c_int), ("out_fp32", C.c_int), ("residual", C.c_int),
+        ("silu", C.c_int), ("status", C.c_void_p),
+    ]
+
+
+class ScanArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("ldx", C.c_longlong), ("z", C.c_void_p), ("ldz", C.c_longlong),
+        ("bc", C.c_void_p), ("ldbc", C.c_longlong), ("off_b", C.c_int), ("off_c", C.c_int),
+        ("dt", C.c_void_p), ("lddt", C.c_longlong), ("dt_bias", C.c_void_p), ("a_log2", C.c_void_p), ("d_skip", C.c_void_p),
+        ("states", C.c_void_p), ("seq_start", C.c_void_p), ("state_in", C.c_void_p), ("state_out", C.c_void_p),
+        ("out", C.c_void_p), ("ldo", C.c_longlong), ("rows", C.c_int), ("n_seqs", C.c_int), ("inner", C.c_int),
+        ("state", C.c_int), ("n_states", C.c_int), ("fp32", C.c_int), ("status", C.c_void_p),
+    ]
+
+
+class GqaArgs(C.Structure):
+    _fields_ = [
+        ("q", C.c_void_p), ("ldq", C.c_longlong), ("k", C.c_void_p), ("v", C.c_void_p), ("ldkv", C.c_longlong),
+        ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("cos_t", C.c_void_p), ("sin_t", C.c_void_p),
+        ("max_pos", C.c_int), ("rot_dims", C.c_int), ("positions", C.c_void_p), ("write_slot", C.c_void_p),
+        ("pool", C.c_void_p), ("pool_rows", C.c_longlong), ("pool_ld", C.c_longlong),
+        ("first_pool", C.c_void_p), ("first_off", C.c_longlong), ("v_mix", C.c_float),
+        ("block_table", C.c_void_p), ("row_seq", C.c_void_p), ("row_pos", C.c_void_p),
+        ("num_seqs", C.c_int), ("max_blocks", C.c_int), ("page_size", C.c_int), ("chunk", C.c_int),
+        ("scale", C.c_float), ("eps", C.c_float), ("out", C.c_void_p), ("ldo", C.c_longlong),
+        ("rows", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int),
+        ("vdim", C.c_int), ("vdim_pad", C.c_int), ("fp32", C.c_int), ("status", C.c_void_p),
     ]
 
 

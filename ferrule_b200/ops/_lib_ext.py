@@ -74,6 +74,13 @@ def declare(lib) -> None:
         "fb_latent_attention": ([vp, i, vp], i),
         "fb_delta_decode": ([vp, vp], i),
         "fb_delta_prefill": ([vp, vp], i),
+        # stream_ops.cu, selective_scan.cu, gqa_attention.cu
+        "fb_stream_step": ([vp, vp], i),
+        "fb_norm_rows": ([vp, ll, i, vp, i, vp, vp, i, vp, ll, i, i, f, i, vp, vp], i),
+        "fb_short_conv": ([vp, vp], i),
+        "fb_selective_scan": ([vp, vp], i),
+        "fb_gqa_prep": ([vp, vp], i),
+        "fb_gqa_attention": ([vp, vp], i),
         # v4_ops.cu
         "fb_hc_pre": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, vp], i),
         "fb_hc_pre_split": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, i, vp, vp, vp], i),

@@ -1,4 +1,5 @@
-"""Launchers of the layer-list model kernels (csrc/layered_ops.cu, csrc/delta_rule.cu).
+"""Launchers of the layer-list model kernels (csrc/layered_ops.cu, stream_ops.cu, delta_rule.cu, selective_scan.cu,
+gqa_attention.cu).
 
 Activations are bf16, or fp32 for models that run in full 32 bits: the launcher follows the tensors' dtype.
 """
@@ -10,7 +11,7 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import AttnArgs, DeltaArgs, LayerTailArgs, check, get_lib, ptr, status_tensor, stream_ptr
+from ._lib import AttnArgs, ConvArgs, DeltaArgs, GqaArgs, LayerTailArgs, ScanArgs, StreamArgs, check, get_lib, ptr, status_tensor, stream_ptr
 
 
 def _fp32(t: torch.Tensor) -> int:
@@ -105,7 +106,7 @@ class DeltaScratch:
         self.rows = rows
         self.qn = torch.empty(rows * big(lambda m: m.kv_heads * m.dim), **f32)
         self.kn = torch.empty_like(self.qn)
-        self.decay = torch.empty(rows * big(lambda m: m.heads * m.dim), **f32)
+        self.decay = torch.empty(rows * big(lambda m: m.heads if m.head_decay else m.heads * m.dim), **f32)
         self.v = torch.empty(rows * big(lambda m: m.heads * m.vdim), **f32)
         self.o = torch.empty_like(self.v)
         self.beta = torch.empty(rows * big(lambda m: m.heads), **f32)
@@ -116,19 +117,23 @@ def delta_decode_supported(mixer) -> bool:
     return mixer.vdim <= 128 and mixer.vdim % 4 == 0 and mixer.dim <= 128
 
 
-def delta_rule(proj: torch.Tensor, off, ag: torch.Tensor, img, mixer, eps: float, state: torch.Tensor,
+def delta_rule(proj: torch.Tensor, off, ag: Optional[torch.Tensor], img, mixer, eps: float, state: torch.Tensor,
                tail: torch.Tensor, seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int,
                out: torch.Tensor, *, row_seq: Optional[torch.Tensor] = None, scratch: Optional[DeltaScratch] = None,
                decode: bool = False) -> torch.Tensor:
     """Convolutions, recurrence and gated output norm of a delta mixer over the rows of a packed batch.
-    proj: rows of the layer's input projection, `off` its block offsets; ag: fp32 rows of the second low-rank halves;
+    proj: rows of the layer's input projection, `off` its block offsets; ag: fp32 rows of the second low-rank halves (None:
+    decay and gate pre-activations are blocks `a` and `g` of the projection, one decay per head);
     decode: one row per sequence, a single launch."""
-    assert ag.dtype == torch.float32 and state.dtype == torch.float32 and state.is_contiguous() and tail.is_contiguous()
+    assert (ag is None) == mixer.head_decay and (ag is None or ag.dtype == torch.float32)
+    assert state.dtype == torch.float32 and state.is_contiguous() and tail.is_contiguous()
     assert tail.dtype == proj.dtype == out.dtype
     a = DeltaArgs()
     a.proj, a.ldp = proj.data_ptr(), proj.stride(0)
     a.off_q, a.off_k, a.off_v, a.off_b = off["q"], off["k"], off["v"], off["b"]
-    a.ag, a.ldag, a.off_gate, a.fp32 = ag.data_ptr(), ag.stride(0), img.off_gate, _fp32(proj)
+    a.ag, a.ldag, a.off_gate, a.fp32 = ptr(ag), ag.stride(0) if ag is not None else 0, img.off_gate, _fp32(proj)
+    a.off_a, a.off_g = (off["a"], off["g"]) if ag is None else (-1, -1)
+    a.gate_silu = 1 if mixer.gate == "silu" else 0
     a.conv, a.a_neg, a.dt_bias, a.norm_w = (img.conv.data_ptr(), img.a_neg.data_ptr(), img.dt_bias.data_ptr(),
                                             img.o_norm.data_ptr())
     a.state, a.tail, a.n_states = state.data_ptr(), tail.data_ptr(), state.shape[0]
@@ -148,4 +153,137 @@ def delta_rule(proj: torch.Tensor, off, ag: torch.Tensor, img, mixer, eps: float
     a.beta, a.qk, a.o = scratch.beta.data_ptr(), scratch.qk.data_ptr(), scratch.o.data_ptr()
     check(get_lib(True).fb_delta_prefill(C.byref(a), stream_ptr()), "fb_delta_prefill")
     _lib.LAUNCHES[0] += 2                    # prepare, scan, output
+    return out
+
+
+# ------------------------------------------------------------------ output-norm blocks
+def _canon(a: StreamArgs, conv, tail, state_in, state_out, h) -> None:
+    a.conv, a.taps = conv.data_ptr(), conv.shape[0]
+    a.tail, a.n_states = tail.data_ptr(), tail.shape[0]
+    a.state_in, a.state_out = state_in.data_ptr(), state_out.data_ptr()
+    a.h, a.ldh = h.data_ptr(), h.stride(0)
+    assert tail.is_contiguous() and tail.dtype == torch.float32 and conv.is_contiguous()
+
+
+def _stream(x: torch.Tensor, dim: int, like: torch.Tensor, act: Optional[torch.Tensor], canon) -> StreamArgs:
+    assert x.dtype == torch.float32 and (act is None or act.dtype == like.dtype)
+    a = StreamArgs()
+    a.x, a.ldx, a.rows, a.dim, a.dim_pad, a.fp32 = x.data_ptr(), x.stride(0), x.shape[0], dim, x.shape[1], _fp32(like)
+    a.status = status_tensor(x.device).data_ptr()
+    if act is not None:
+        a.act, a.lda = act.data_ptr(), act.stride(0)
+    if canon is not None:
+        _canon(a, *canon)
+    return a
+
+
+def embed_stream(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, dim: int, *,
+                 positions: Optional[torch.Tensor] = None, pos_table: Optional[torch.Tensor] = None, canon=None) -> None:
+    """x = table[ids] (+ pos_table[positions]).  canon = (filters [taps, width], state plane, state_in, state_out, h): one
+    row per sequence, h = x + conv(x) with the convolution's state."""
+    a = _stream(x, dim, table, None, canon)
+    a.ids, a.table, a.ldt, a.vocab = ids.data_ptr(), table.data_ptr(), table.stride(0), table.shape[0]
+    if pos_table is not None:
+        assert pos_table.dtype == table.dtype and pos_table.stride(0) == table.stride(0)
+        a.positions, a.pos_table, a.max_pos = positions.data_ptr(), pos_table.data_ptr(), pos_table.shape[0]
+    check(get_lib(True).fb_stream_step(C.byref(a), stream_ptr()), "fb_stream_step")
+
+
+def add_normed(x: torch.Tensor, y: torch.Tensor, norm: torch.Tensor, dim: int, eps: float, *,
+               act: Optional[torch.Tensor] = None, canon=None, rms: bool = False) -> None:
+    """x += norm(y); norm: [2, width] weight and bias of a layer norm (rms: [1, width], an RMS norm).  act: the new rows as
+    activations; canon as in `embed_stream`."""
+    a = _stream(x, dim, y, act, canon)
+    a.y, a.ldy, a.eps, a.rms = y.data_ptr(), y.stride(0), eps, 1 if rms else 0
+    a.norm_w, a.norm_b = norm[0].data_ptr(), None if rms else norm[1].data_ptr()
+    check(get_lib(True).fb_stream_step(C.byref(a), stream_ptr()), "fb_stream_step")
+
+
+def norm_rows(x: torch.Tensor, rows: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, dim: int, eps: float,
+              rms: bool = False) -> torch.Tensor:
+    """out[i] = norm(x[rows[i]]) (see `add_normed`)."""
+    assert x.dtype == torch.float32 and rows.dtype == torch.int32 and out.shape[0] == rows.shape[0]
+    check(get_lib(True).fb_norm_rows(x.data_ptr(), x.stride(0), x.shape[0], rows.data_ptr(), rows.shape[0], norm[0].data_ptr(),
+                                     None if rms else norm[1].data_ptr(), 1 if rms else 0, out.data_ptr(), out.stride(0), dim,
+                                     x.shape[1], eps, _fp32(out), status_tensor(x.device).data_ptr(), stream_ptr()),
+          "fb_norm_rows")
+    return out
+
+
+def short_conv(x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, out: torch.Tensor, row_seq: torch.Tensor,
+               seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, *,
+               bias: Optional[torch.Tensor] = None, residual: bool = False, silu: bool = False) -> torch.Tensor:
+    """Causal convolution of packed rows with one filter per channel: x [rows, channels], w fp32 [taps, channels].
+    residual: out = x + conv(x); silu: out = silu(conv(x) + bias)."""
+    assert tail.dtype == x.dtype and tail.is_contiguous() and tail.shape[-1] == w.shape[1] and w.is_contiguous()
+    a = ConvArgs()
+    a.x, a.ldx, a.w, a.bias, a.tail = x.data_ptr(), x.stride(0), w.data_ptr(), ptr(bias), tail.data_ptr()
+    a.out, a.ldo = out.data_ptr(), out.stride(0)
+    a.row_seq, a.seq_start, a.state_in, a.state_out = (row_seq.data_ptr(), seq_start.data_ptr(), state_in.data_ptr(),
+                                                       state_out.data_ptr())
+    a.rows, a.channels, a.taps, a.n_states, a.n_seqs = x.shape[0], w.shape[1], w.shape[0], tail.shape[0], n_seqs
+    a.x_fp32, a.out_fp32, a.residual, a.silu = _fp32(x), _fp32(out), int(residual), int(silu)
+    a.status = status_tensor(x.device).data_ptr()
+    check(get_lib(True).fb_short_conv(C.byref(a), stream_ptr()), "fb_short_conv")
+    return out
+
+
+def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, off_b: int, off_c: int, dt: torch.Tensor, img,
+                   states: torch.Tensor, seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor,
+                   n_seqs: int, out: torch.Tensor) -> torch.Tensor:
+    """(scan + D x) * silu(z) over packed rows; x, z, out [rows, inner], bc rows with B at off_b and C at off_c, dt fp32
+    [rows, inner] without bias; img: a_log2, dt_bias, d_skip."""
+    assert dt.dtype == torch.float32 and states.dtype == torch.float32 and states.is_contiguous()
+    assert x.dtype == z.dtype == bc.dtype == out.dtype
+    a = ScanArgs()
+    a.x, a.ldx, a.z, a.ldz, a.bc, a.ldbc = x.data_ptr(), x.stride(0), z.data_ptr(), z.stride(0), bc.data_ptr(), bc.stride(0)
+    a.off_b, a.off_c, a.dt, a.lddt = off_b, off_c, dt.data_ptr(), dt.stride(0)
+    a.dt_bias, a.a_log2, a.d_skip = img.dt_bias.data_ptr(), img.a_log2.data_ptr(), img.d_skip.data_ptr()
+    a.states, a.n_states, a.state, a.inner = states.data_ptr(), states.shape[0], states.shape[1], states.shape[2]
+    a.seq_start, a.state_in, a.state_out = seq_start.data_ptr(), state_in.data_ptr(), state_out.data_ptr()
+    a.out, a.ldo, a.rows, a.n_seqs, a.fp32 = out.data_ptr(), out.stride(0), x.shape[0], n_seqs, _fp32(x)
+    a.status = status_tensor(x.device).data_ptr()
+    check(get_lib(True).fb_selective_scan(C.byref(a), stream_ptr()), "fb_selective_scan")
+    return out
+
+
+# ------------------------------------------------------------------ grouped-query attention in position chunks
+def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor) -> GqaArgs:
+    a = GqaArgs()
+    assert q.dtype == pool.dtype and pool.is_contiguous()
+    a.q, a.ldq, a.rows, a.fp32 = q.data_ptr(), q.stride(0), q.shape[0], _fp32(q)
+    a.pool, a.pool_ld, a.pool_rows = pool.data_ptr(), pool.shape[-1], pool.numel() // pool.shape[-1]
+    a.heads, a.kv_heads, a.dim, a.vdim, a.dim_pad, a.vdim_pad = (mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim,
+                                                                 mixer.dim_pad, mixer.vdim_pad)
+    a.chunk, a.scale, a.rot_dims = mixer.chunk, mixer.scale, mixer.rot_dims
+    a.status = status_tensor(q.device).data_ptr()
+    return a
+
+
+def gqa_prep(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, mixer, img, rotation, positions: torch.Tensor,
+             write_slot: torch.Tensor, pool: torch.Tensor, eps: float, first_pool: Optional[torch.Tensor] = None,
+             first_off: int = 0) -> None:
+    """Query rows are normalised and rotated in place; keys and values go into the pool rows of their tokens.
+    rotation = (cos, sin) fp32 [positions, rot_dims / 2]; first_pool: the pool of the layer whose values are mixed in, at
+    column first_off."""
+    a = _gqa(q, mixer, pool)
+    assert k.stride(0) == v.stride(0)
+    a.k, a.v, a.ldkv = k.data_ptr(), v.data_ptr(), k.stride(0)
+    a.q_norm, a.k_norm = img.q_norm.data_ptr(), img.k_norm.data_ptr()
+    a.cos_t, a.sin_t, a.max_pos = rotation[0].data_ptr(), rotation[1].data_ptr(), rotation[0].shape[0]
+    a.positions, a.write_slot, a.eps = positions.data_ptr(), write_slot.data_ptr(), eps
+    if first_pool is not None:
+        assert first_pool.shape == pool.shape
+        a.first_pool, a.first_off, a.v_mix = first_pool.data_ptr(), first_off, img.v_mix
+    check(get_lib(True).fb_gqa_prep(C.byref(a), stream_ptr()), "fb_gqa_prep")
+
+
+def gqa_attention(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
+                  row_pos: torch.Tensor, page_size: int, out: torch.Tensor) -> torch.Tensor:
+    """32-bit arithmetic: out [rows, heads * vdim_pad]."""
+    a = _gqa(q, mixer, pool)
+    a.block_table, a.row_seq, a.row_pos = block_table.data_ptr(), row_seq.data_ptr(), row_pos.data_ptr()
+    a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
+    a.out, a.ldo = out.data_ptr(), out.stride(0)
+    check(get_lib(True).fb_gqa_attention(C.byref(a), stream_ptr()), "fb_gqa_attention")
     return out
