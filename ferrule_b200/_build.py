@@ -39,6 +39,8 @@ CUDA_SOURCES = [
     "stream_ops.cu",
     "selective_scan.cu",
     "gqa_attention.cu",
+    "gqa_decode.cu",
+    "gqa_prefill_tc.cu",
     "gemm_f32.cu",
     "ep_moe.cu",
     "expert_table.cu",
@@ -50,7 +52,8 @@ CUDA_SOURCES = [
 # much instead of everything (into a library of its own; the full library is used when it is there).
 COMPONENTS = {
     "layered": ["gemm_tcgen05.cu", "mla_attention.cu", "mla_prefill_tc.cu", "elementwise.cu", "data_movers.cu",
-                "layered_ops.cu", "delta_rule.cu", "gemm_f32.cu", "stream_ops.cu", "selective_scan.cu", "gqa_attention.cu"],
+                "layered_ops.cu", "delta_rule.cu", "gemm_f32.cu", "stream_ops.cu", "selective_scan.cu", "gqa_attention.cu",
+                "gqa_decode.cu", "gqa_prefill_tc.cu"],
 }
 CXX_SOURCES = [
     "host/kv_page_manager.cpp",

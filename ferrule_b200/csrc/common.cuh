@@ -351,8 +351,20 @@ __host__ __device__ constexpr uint32_t umma_idesc(uint32_t m, uint32_t n, uint32
 __device__ __forceinline__ float bf16_round(float x) {
   return __bfloat162float(__float2bfloat16_rn(x));
 }
-// exact GELU
+// Exact (error-function) GELU.  For outputs that are rounded to bf16: the rational approximation of erfc by Hastings
+// (Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26: absolute error below 1.5e-7), written for the tail
+// (1 - erf(|z|)) / 2 so that nothing cancels for negative arguments.
 __device__ __forceinline__ float gelu_f(float x) { return 0.5f * x * (1.f + erff(x * 0.70710678118654752f)); }
+__device__ __forceinline__ float gelu_bf16_f(float x) {
+  const float z = fabsf(x) * 0.70710678118654752f;
+  const float t = __fdividef(1.f, fmaf(0.3275911f, z, 1.f));
+  float q = fmaf(1.061405429f, t, -1.453152027f);
+  q = fmaf(q, t, 1.421413741f);
+  q = fmaf(q, t, -0.284496736f);
+  q = fmaf(q, t, 0.254829592f);
+  const float h = 0.5f * q * t * __expf(-z * z);
+  return x > 0.f ? fmaf(-x, h, x) : x * h;
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -19,6 +19,7 @@
 // over the decayed state.
 #include "act_type.cuh"
 #include "common.cuh"
+#include "f32x2.cuh"
 #include "ferrule_b200.h"
 #include "launch.cuh"
 
@@ -280,26 +281,6 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 // ---------------------------------------------------------------------------------
 constexpr int kScanStep = 16;
 
-// two fp32 lanes in one 64-bit register: one instruction for two multiply-adds, each rounded as the scalar one
-__device__ __forceinline__ uint64_t pack2(float a, float b) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float& a, float& b) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
-}
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
-  return r;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-  uint64_t r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
-  return r;
-}
-
 // HEADG: one decay per head.  The dot products are then taken over the state before the decay and scaled, so that the
 // decay of the state runs beside them instead of ahead of them.
 template <typename T, int RPT, int COLS, bool HEADG>
@@ -317,7 +298,8 @@ delta_scan_kernel(const DeltaParams<T> p) {
   // g [kScanStep] at the end
   constexpr int kBuf = scan_buf<T, RPT, COLS, HEADG>();
   constexpr int kV = (HEADG ? 2 : 3) * kScanStep * DP;          // first float of v
-  const int seq = blockIdx.y;
+  // (a mixed batch lists its decode rows first: the long sequences' CTAs start first and spread over all SMs)
+  const int seq = gridDim.y - 1 - blockIdx.y;
   const int vtiles = (p.vdim + kCols - 1) / kCols;
   const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * kCols;
   const int hk = h / (p.heads / p.kv_heads);

@@ -343,6 +343,12 @@ typedef struct FbGqaArgs {
 } FbGqaArgs;
 int fb_gqa_prep(const FbGqaArgs* args, void* stream);
 int fb_gqa_attention(const FbGqaArgs* args, void* stream);      // dim, vdim <= 512
+// bf16, few rows (gqa_decode.cu): dim, vdim <= 256; the visible keys of a row are divided among `splits` (1, 2, 4, 8) CTAs;
+// early: one row per sequence, keys below a row's own position predate the preceding kernel
+int fb_gqa_decode(const FbGqaArgs* args, int splits, int early, void* stream);
+// bf16 prompts on tcgen05 (gqa_prefill_tc.cu): dim, vdim <= 256, page_size a power of two >= 8; tiles [n_tiles, 4] =
+// sequence, first row, rows (<= tile_positions), position of the first; tile_positions * heads / kv_heads <= 128
+int fb_gqa_prefill_tc(const FbGqaArgs* args, const int* tiles, int n_tiles, int tile_positions, void* stream);
 
 // ---- gated delta rule (see delta_rule.cu) ------------------------------------------------------------------
 typedef struct FbDeltaArgs {

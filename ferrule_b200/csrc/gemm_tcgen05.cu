@@ -413,7 +413,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
-              if (EPI == kEpiGelu) x = gelu_f(x);
+              if (EPI == kEpiGelu) x = gelu_bf16_f(x);
               if (EPI == kEpiScatter && p.row_scale) x *= p.row_scale[row0 + r];
             }
             sb[j * 128 + ch_in_tile] = __float2bfloat16_rn(x);
@@ -452,7 +452,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
-              if (EPI == kEpiGelu) x = gelu_f(x);
+              if (EPI == kEpiGelu) x = p.out_fp32 ? gelu_f(x) : gelu_bf16_f(x);
               long long orow = row0 + r;
               if (EPI == kEpiScatter) {
                 if (p.row_scale) x *= p.row_scale[row0 + r];

@@ -139,6 +139,123 @@ gqa_prep_kernel(const GqaParams<T> p) {
   }
 }
 
+// The same with everything in registers, for rotations whose half is a multiple of 8: an item is a pair of 8-element vectors
+// that turn together, or one vector of the part that is not rotated.  NI items per thread.
+template <typename T, int NI>
+__global__ void __launch_bounds__(256)
+gqa_prep_vec_kernel(const GqaParams<T> p) {
+  pdl_launch_dependents();
+  const int pairs = p.half / 8, per_head = pairs + (p.dim_pad - 2 * p.half) / 8;
+  const int q_items = p.heads * per_head, items = q_items + p.kv_heads * per_head;
+  const int nk = p.kv_heads * p.dim_pad;
+  __shared__ float red[2][32];
+  pdl_wait();
+  const long long r = blockIdx.x;
+  int pos = p.positions[r];
+  const long long slot = p.write_slot[r];
+  float u[NI][8], w[NI][8], ssq = 0.f, ssk = 0.f;
+  int off[NI];                                                       // first element of the item in its matrix row
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    const int i = threadIdx.x + k * 256;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) u[k][j] = w[k][j] = 0.f;
+    off[k] = -1;
+    if (i >= items) continue;
+    const bool is_q = i < q_items;
+    const int n = is_q ? i : i - q_items, v = n % per_head;
+    off[k] = n / per_head * p.dim_pad + (v < pairs ? v * 8 : 2 * p.half + (v - pairs) * 8);
+    const T* src = is_q ? p.q + r * p.ldq : p.k + r * p.ldkv;
+    act_load8(src + off[k], u[k]);
+    if (v < pairs) act_load8(src + off[k] + p.half, w[k]);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(u[k][j], u[k][j], fmaf(w[k][j], w[k][j], ss));
+    (is_q ? ssq : ssk) += ss;
+  }
+  if (pos < 0 || pos >= p.max_pos) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD60, r, pos);
+    pos = 0;
+  }
+  const bool keep = slot >= 0 && slot < p.pool_rows;
+  if (!keep && slot != -1 && threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD61, r, static_cast<uint32_t>(slot));
+  T* row = p.pool + (keep ? slot : 0) * p.pool_ld;
+  // values: one warp per head, independent of the row sums
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (keep) {
+    for (int g = warp; g < p.kv_heads; g += 8) {
+      const T* v = p.v + r * p.ldkv + g * p.vdim_pad;
+      const T* first = p.first_pool ? p.first_pool + slot * p.pool_ld + p.first_off + g * p.vdim_pad : nullptr;
+      float ss = 0.f, x[8], f[8];
+      if (p.vdim_pad <= 256) {
+        const int d = lane * 8;
+        const bool in = d < p.vdim_pad;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = f[j] = 0.f;
+        if (in) act_load8(v + d, x);
+        if (in && first) act_load8(first + d, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) ss = fmaf(x[j], x[j], ss);
+        const float inv = 1.f / sqrtf(warp_sum(ss) / p.vdim + p.eps), own = first ? 1.f - p.v_mix : 1.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = fmaf(p.v_mix, f[j], own * (x[j] * inv));
+        if (in) act_store8(row + nk + g * p.vdim_pad + d, x);
+      } else {
+        for (int d = lane * 8; d < p.vdim_pad; d += 256) {
+          act_load8(v + d, x);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) ss = fmaf(x[j], x[j], ss);
+        }
+        const float inv = 1.f / sqrtf(warp_sum(ss) / p.vdim + p.eps), own = first ? 1.f - p.v_mix : 1.f;
+        for (int d = lane * 8; d < p.vdim_pad; d += 256) {
+          act_load8(v + d, x);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) f[j] = 0.f;
+          if (first) act_load8(first + d, f);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) x[j] = fmaf(p.v_mix, f[j], own * (x[j] * inv));
+          act_store8(row + nk + g * p.vdim_pad + d, x);
+        }
+      }
+    }
+  }
+  ssq = cta_sum(ssq, red[0]);
+  ssk = cta_sum(ssk, red[1]);
+  const float iq = 1.f / sqrtf(ssq / (p.heads * p.dim) + p.eps), ik = 1.f / sqrtf(ssk / (p.kv_heads * p.dim) + p.eps);
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    if (off[k] < 0) continue;
+    const int i = threadIdx.x + k * 256;
+    const bool is_q = i < q_items;
+    if (!is_q && !keep) continue;
+    const int v = (is_q ? i : i - q_items) % per_head;
+    const float inv = is_q ? iq : ik;
+    const float* nw = (is_q ? p.q_norm : p.k_norm) + off[k];
+    T* dst = (is_q ? p.q + r * p.ldq : row) + off[k];
+    float a[8];
+    act_load8(nw, a);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) u[k][j] *= inv * a[j];
+    if (v < pairs) {
+      float c[8], s[8], o[8];
+      act_load8(nw + p.half, a);
+      act_load8(p.cos_t + static_cast<long long>(pos) * p.half + v * 8, c);
+      act_load8(p.sin_t + static_cast<long long>(pos) * p.half + v * 8, s);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        w[k][j] *= inv * a[j];
+        o[j] = fmaf(u[k][j], c[j], -w[k][j] * s[j]);
+      }
+      act_store8(dst, o);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] = fmaf(w[k][j], c[j], u[k][j] * s[j]);
+      act_store8(dst + p.half, o);
+    } else {
+      act_store8(dst, u[k]);
+    }
+  }
+}
+
 // DPL: query / key and value features per lane
 template <typename T, int DPL>
 __global__ void __launch_bounds__(128)
@@ -242,6 +359,15 @@ template <typename T>
 static int run_prep(const FbGqaArgs* a, cudaStream_t s) {
   GqaParams<T> p{};
   fill_gqa(a, p);
+  const int per_head = p.half / 8 + (p.dim_pad - 2 * p.half) / 8, items = (p.heads + p.kv_heads) * per_head;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(a->v) | reinterpret_cast<uintptr_t>(a->first_pool);
+  if (p.half % 8 == 0 && items <= 1024 && (bits & 15) == 0 && a->first_off % 8 == 0) {
+    const dim3 grid(a->rows), block(256);
+    if (items <= 256) launch_pdl(gqa_prep_vec_kernel<T, 1>, grid, block, 0, s, p);
+    else if (items <= 512) launch_pdl(gqa_prep_vec_kernel<T, 2>, grid, block, 0, s, p);
+    else launch_pdl(gqa_prep_vec_kernel<T, 4>, grid, block, 0, s, p);
+    return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  }
   const size_t smem = (static_cast<size_t>(a->heads + a->kv_heads) * a->dim_pad + a->rot_dims) * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
   static bool attr = false;

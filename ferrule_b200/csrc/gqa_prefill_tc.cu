@@ -1,0 +1,396 @@
+// Prefill attention of grouped-query layers inside position chunks on the 5th-generation tensor cores, bf16.
+//
+// CTA = one tile of consecutive query positions of one sequence x the query heads of one key / value head: up to 128
+// (position, head) rows, P = 128 / heads-per-group positions.  Keys are taken in tiles of 64 tokens at absolute positions
+// 64 j, from the first tile that holds a key of the tile's first chunk.
+//
+//   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
+//     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
+//     head's width and rows past the sequence are zeros), two stages each with their own barriers.
+//   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
+//     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
+//     before the current P is waited for.
+//   Softmax (warps 2..5, one row per thread): scores from TMEM, scale, causal and chunk mask, running maximum, exp2, bf16 P
+//     written over the score buffer.  The accumulator is rescaled only when a row's maximum has grown by more than 2^8
+//     since the reference it was scaled by; the sum uses the same reference, so the result is exact up to rounding.
+//
+// A row's result depends on the row and the cache contents, not on which rows share its tile or how a prompt was cut.
+// Every wait is bounded (status word, then teardown with TMEM freed); page ids are range-checked.
+#include "attn_tc.cuh"
+#include "common.cuh"
+#include "ferrule_b200.h"
+#include "launch.cuh"
+
+namespace fb {
+
+constexpr int kGpThreads = 192;
+constexpr int kGpM = 128;
+constexpr int kGpKv = 64;
+constexpr int kGpQBlock = kGpM * 128;         // bytes of a 64-feature block of the query tile
+constexpr int kGpKvBlock = kGpKv * 128;
+
+struct GpParams {
+  const int* tiles;          // [n_tiles, 4] = sequence, first query row, query rows, position of the first
+  const int* block_table;
+  __nv_bfloat16* out;
+  long long ldo;
+  DeviceStatus* status;
+  long long pool_rows;
+  int rows, heads, kv_heads, per;      // per: query heads of a key / value head
+  int positions;             // positions per tile the query box holds
+  int num_seqs, max_blocks, page_size, box_rows, chunk;
+  int dim_pad, vdim_pad, qb, vb;       // qb, vb: 64-feature blocks of a query / key row and of a value row
+  uint32_t tmem_cols;
+  float scale_log2;
+};
+
+__global__ void __launch_bounds__(kGpThreads)
+gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
+                      const __grid_constant__ CUtensorMap map_v, const GpParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int qb = p.qb, vb = p.vb;
+  uint8_t* q_s = smem;
+  uint8_t* k_s = q_s + qb * kGpQBlock;                   // [2][qb] blocks
+  uint8_t* v_s = k_s + 2 * qb * kGpKvBlock;              // [2][vb] blocks
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * vb * kGpKvBlock);
+  uint64_t* q_full = bars + 0;
+  uint64_t* k_full = bars + 1;          // [2]
+  uint64_t* v_full = bars + 3;          // [2]
+  uint64_t* k_free = bars + 5;          // [2]
+  uint64_t* v_free = bars + 7;          // [2]
+  uint64_t* s_full = bars + 9;          // [2]
+  uint64_t* p_full = bars + 11;         // [2]
+  uint64_t* o_done = bars + 13;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
+  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(bars + 15);
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = blockIdx.y;
+  const int4 tile = reinterpret_cast<const int4*>(p.tiles)[blockIdx.x];
+  const int seq = tile.x, row0 = tile.y, nrows = tile.z, pos0 = tile.w;
+  if (seq < 0 || seq >= p.num_seqs || row0 < 0 || nrows <= 0 || nrows > p.positions || row0 + nrows > p.rows || pos0 < 0) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xA80, blockIdx.x, seq);
+    return;
+  }
+  const int kv_len = min(pos0 + nrows, p.max_blocks * p.page_size);
+  const int j0 = pos0 / p.chunk * p.chunk / kGpKv;                       // first token tile
+  const int n_kv = (kv_len + kGpKv - 1) / kGpKv - j0;
+  if (n_kv <= 0) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xA81, blockIdx.x, pos0);
+    return;
+  }
+
+  if (tid == 0) {
+    mbar_init(q_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(k_full + i, 1);
+      mbar_init(v_full + i, 1);
+      mbar_init(k_free + i, 1);
+      mbar_init(v_free + i, 1);
+      mbar_init(s_full + i, 1);
+      mbar_init(p_full + i, 4);
+    }
+    mbar_init(o_done, 1);
+    *abort_flag = 0;
+    fence_barrier_init();
+    tma_prefetch_desc(&map_q);
+    tma_prefetch_desc(&map_k);
+    tma_prefetch_desc(&map_v);
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, p.tmem_cols);
+    tmem_relinquish();
+  }
+  pdl_launch_dependents();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *tmem_slot;
+  const uint32_t col_s = static_cast<uint32_t>(vb * 64);                 // S0, S1 behind the accumulator; P over S
+  pdl_wait();
+
+  if (warp == 0) {
+    // ------------------------------------------------------------------ TMA producer
+    if (lane == 0) {
+      mbar_arrive_expect_tx(q_full, static_cast<uint32_t>(qb * p.positions * p.per * 128));
+      for (int b = 0; b < qb; ++b) tma_load_3d(q_s + b * kGpQBlock, &map_q, q_full, b * 64, g * p.per, row0);
+      const int subs = kGpKv / p.box_rows;
+      const long long n_pages = p.pool_rows / p.page_size;
+      bool ok = true;
+      int armed = 0;                                                     // tiles whose copies were all requested
+      for (int j = 0; j < n_kv && ok; ++j) {
+        const int st = j & 1;
+        int rowc[8];
+        for (int s = 0; s < subs; ++s) {
+          const int t0 = (j0 + j) * kGpKv + s * p.box_rows;
+          int rc = static_cast<int>(p.pool_rows);                        // out of range: the copy fills zeros
+          if (t0 < kv_len) {
+            const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t0 / p.page_size];
+            if (page >= 0 && page < n_pages) rc = page * p.page_size + t0 % p.page_size;
+            else report_status(p.status, kStatusBadIndex, 0xA82, seq, t0);
+          }
+          rowc[s] = rc;
+        }
+        if (j > 1) ok = mbar_wait(k_free + st, ((j - 2) >> 1) & 1, abort_flag, p.status, 0xA90);
+        if (!ok) break;
+        mbar_arrive_expect_tx(k_full + st, static_cast<uint32_t>(qb * kGpKvBlock));
+        for (int s = 0; s < subs; ++s)
+          for (int b = 0; b < qb; ++b)
+            tma_load_3d(k_s + (st * qb + b) * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + st, b * 64, g, rowc[s]);
+        if (j > 1) ok = mbar_wait(v_free + st, ((j - 2) >> 1) & 1, abort_flag, p.status, 0xA91);
+        if (!ok) break;
+        mbar_arrive_expect_tx(v_full + st, static_cast<uint32_t>(vb * kGpKvBlock));
+        for (int s = 0; s < subs; ++s)
+          for (int b = 0; b < vb; ++b)
+            tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rowc[s]);
+        armed = j + 1;
+      }
+      // after an abort: copies of the last two tiles may still be in flight, and the CTA may not exit under them
+      if (*abort_flag) {
+        auto drain = [&](uint64_t* bar, uint32_t parity) {
+          const uint64_t t0 = globaltimer_ns();
+          while (!mbar_try_wait(bar, parity) && globaltimer_ns() - t0 < 2000000ull) {
+          }
+        };
+        drain(q_full, 0);
+        for (int j = armed > 2 ? armed - 2 : 0; j < min(armed + 1, n_kv); ++j) {
+          drain(k_full + (j & 1), (j >> 1) & 1);
+          drain(v_full + (j & 1), (j >> 1) & 1);
+        }
+      }
+    }
+  } else if (warp == 1) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (lane == 0) {
+      const uint32_t q_addr = smem_u32(q_s), k_addr = smem_u32(k_s), v_addr = smem_u32(v_s);
+      constexpr uint32_t idesc_qk = umma_idesc(kGpM, kGpKv, 1, 1);
+      const uint32_t idesc_pv = umma_idesc(kGpM, static_cast<uint32_t>(vb * 64), 1, 1) | (1u << 16);   // B is MN-major
+      const int ksteps = (p.dim_pad + 15) / 16;
+      auto qk = [&](int j) {
+        const uint32_t ks = k_addr + (j & 1) * qb * kGpKvBlock;
+        for (int k = 0; k < ksteps; ++k)
+          umma_bf16(tmem + col_s + (j & 1) * kGpKv, umma_desc_k128(q_addr + (k >> 2) * kGpQBlock + (k & 3) * 32),
+                    umma_desc_k128(ks + (k >> 2) * kGpKvBlock + (k & 3) * 32), idesc_qk, k > 0 ? 1u : 0u);
+        umma_commit(s_full + (j & 1));
+        umma_commit(k_free + (j & 1));
+      };
+      bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 0xAA0);
+      if (ok) ok = mbar_wait(k_full, 0, abort_flag, p.status, 0xAA1);
+      if (ok) {
+        tc_fence_after();
+        qk(0);
+      }
+      for (int j = 0; j < n_kv && ok; ++j) {
+        const uint32_t ph = (j >> 1) & 1;
+        if (j + 1 < n_kv) {
+          // the score buffer of tile j + 1 held P of tile j - 1, whose product was issued before
+          ok = mbar_wait(k_full + ((j + 1) & 1), ((j + 1) >> 1) & 1, abort_flag, p.status, 0xAA2);
+          if (!ok) break;
+          tc_fence_after();
+          qk(j + 1);
+        }
+        ok = mbar_wait(v_full + (j & 1), ph, abort_flag, p.status, 0xAA3);
+        if (ok) ok = mbar_wait(p_full + (j & 1), ph, abort_flag, p.status, 0xAA4);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t vs = v_addr + (j & 1) * vb * kGpKvBlock;
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          umma_bf16_ts(tmem, tmem + col_s + (j & 1) * kGpKv + k * 8, umma_desc_mn128(vs + k * 2048, kGpKvBlock), idesc_pv,
+                       (j > 0 || k > 0) ? 1u : 0u);
+        umma_commit(v_free + (j & 1));
+        if (j + 1 == n_kv) umma_commit(o_done);
+      }
+    }
+  } else {
+    // ------------------------------------------------------------------ softmax + epilogue: one row per thread
+    const int quarter = warp & 3;
+    const int r = quarter * 32 + lane;
+    const int at = r / p.per, head = g * p.per + r - at * p.per;
+    const bool valid = at < nrows;
+    const int pos = pos0 + at;
+    const int hi = valid ? min(pos + 1, kv_len) : 0;
+    const int lo = pos / p.chunk * p.chunk;
+    const uint32_t lane_base = tmem + (static_cast<uint32_t>(quarter * 32) << 16);
+    float m_ref = -INFINITY, l_sum = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_kv; ++j) {
+      const uint32_t s_t = lane_base + col_s + (j & 1) * kGpKv;
+      ok = mbar_wait(s_full + (j & 1), (j >> 1) & 1, abort_flag, p.status, 0xAB0);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      tc_fence_after();
+      uint32_t sv[4][16];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) tmem_ld16(s_t + c * 16, sv[c]);
+      tmem_ld_wait();
+      const int tok0 = (j0 + j) * kGpKv;
+      float mx = -INFINITY;
+      if (__all_sync(0xffffffffu, tok0 >= lo && tok0 + kGpKv <= hi)) {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; ++i) mx = fmaxf(mx, __uint_as_float(sv[c][i]));
+      } else {
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int t = tok0 + c * 16 + i;
+            const float x = (t >= lo && t < hi) ? __uint_as_float(sv[c][i]) : -INFINITY;
+            sv[c][i] = __float_as_uint(x);
+            mx = fmaxf(mx, x);
+          }
+      }
+      mx *= p.scale_log2;                                     // the scale is positive
+      const float m_new = fmaxf(m_ref, mx);
+      if (j == 0) {
+        m_ref = m_new;                                        // nothing accumulated yet
+      } else if (__any_sync(0xffffffffu, m_new > m_ref + 8.f)) {
+        // rescale this warp's 32 accumulator rows: the previous product must have retired
+        ok = mbar_wait(v_free + ((j - 1) & 1), ((j - 1) >> 1) & 1, abort_flag, p.status, 0xAB2);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        tc_fence_after();
+        const float f = (m_new == -INFINITY) ? 1.f : exp2f(m_ref - m_new);
+        m_ref = m_new;
+        l_sum *= f;
+#pragma unroll 1
+        for (int c = 0; c < vb * 4; ++c) {
+          uint32_t ov[16];
+          tmem_ld16(lane_base + c * 16, ov);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * f);
+          tmem_st16(lane_base + c * 16, ov);
+        }
+      }
+      const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
+      float add = 0.f;
+#pragma unroll
+      for (int c = 0; c < 2; ++c) {
+        uint32_t pk[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float p0 = exp2f(fmaf(__uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]), p.scale_log2, -m_use));
+          const float p1 = exp2f(fmaf(__uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]), p.scale_log2, -m_use));
+          add += p0 + p1;
+          pk[i] = pack_bf16x2(p0, p1);
+        }
+        tmem_st16(s_t + c * 16, pk);
+      }
+      l_sum += add;
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(p_full + (j & 1));
+    }
+    if (ok) {
+      ok = mbar_wait(o_done, 0, abort_flag, p.status, 0xAB1);
+      ok = __all_sync(0xffffffffu, ok);
+    }
+    if (ok) {
+      tc_fence_after();
+      const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
+#pragma unroll 1
+      for (int c = 0; c < vb * 4; ++c) {
+        if (c * 16 >= p.vdim_pad) break;
+        uint32_t ov[16];
+        tmem_ld16(lane_base + c * 16, ov);
+        tmem_ld_wait();
+        if (valid) {
+          uint4 w0, w1;
+          w0.x = pack_bf16x2(__uint_as_float(ov[0]) * inv, __uint_as_float(ov[1]) * inv);
+          w0.y = pack_bf16x2(__uint_as_float(ov[2]) * inv, __uint_as_float(ov[3]) * inv);
+          w0.z = pack_bf16x2(__uint_as_float(ov[4]) * inv, __uint_as_float(ov[5]) * inv);
+          w0.w = pack_bf16x2(__uint_as_float(ov[6]) * inv, __uint_as_float(ov[7]) * inv);
+          w1.x = pack_bf16x2(__uint_as_float(ov[8]) * inv, __uint_as_float(ov[9]) * inv);
+          w1.y = pack_bf16x2(__uint_as_float(ov[10]) * inv, __uint_as_float(ov[11]) * inv);
+          w1.z = pack_bf16x2(__uint_as_float(ov[12]) * inv, __uint_as_float(ov[13]) * inv);
+          w1.w = pack_bf16x2(__uint_as_float(ov[14]) * inv, __uint_as_float(ov[15]) * inv);
+          *reinterpret_cast<uint4*>(dst + c * 16) = w0;
+          if (c * 16 + 8 < p.vdim_pad) *reinterpret_cast<uint4*>(dst + c * 16 + 8) = w1;
+        }
+      }
+    }
+  }
+  // ---------------------------------------------------------------------- teardown
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem, p.tmem_cols);
+  }
+}
+
+// bf16 map over [rows][heads][width]: box 64 features x box_heads x box_rows, 128-byte swizzle, zeros outside
+static int gp_map(CUtensorMap* map, const void* base, int width, int heads, uint64_t rows, long long ld, uint32_t box_heads,
+                  uint32_t box_rows) {
+  TcEncodeFn fn = tc_encoder();
+  if (!fn) return FB_ERR_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || width % 8 || ld % 8) return FB_ERR_ALIGN;
+  cuuint64_t dims[3] = {static_cast<cuuint64_t>(width), static_cast<cuuint64_t>(heads), rows};
+  cuuint64_t strides[2] = {static_cast<cuuint64_t>(width) * 2, static_cast<cuuint64_t>(ld) * 2};
+  cuuint32_t box[3] = {64, box_heads, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? FB_OK : FB_ERR_DRIVER;
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_tiles, int tile_positions, void* stream_) {
+  if (!a || !a->q || !a->pool || !a->out || !a->block_table || !tiles || a->fp32) return FB_ERR_SHAPE;
+  if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->kv_heads > 65535 || n_tiles <= 0 ||
+      a->num_seqs <= 0 || a->max_blocks <= 0 || a->chunk <= 0 || !(a->scale > 0.f))
+    return FB_ERR_SHAPE;
+  const int per = a->heads / a->kv_heads;
+  if (tile_positions <= 0 || per * tile_positions > kGpM) return FB_ERR_SHAPE;
+  if (a->page_size < 8 || (a->page_size & (a->page_size - 1)) != 0) return FB_ERR_SHAPE;
+  if (a->dim_pad <= 0 || a->dim_pad > 256 || a->vdim_pad <= 0 || a->vdim_pad > 256) return FB_ERR_LIMIT;
+  if (a->pool_rows <= 0 || a->pool_rows > 0x7fffffffLL || a->pool_rows % a->page_size) return FB_ERR_SHAPE;
+  if (a->pool_ld < static_cast<long long>(a->kv_heads) * (a->dim_pad + a->vdim_pad) ||
+      a->ldq < static_cast<long long>(a->heads) * a->dim_pad || a->ldo < static_cast<long long>(a->heads) * a->vdim_pad)
+    return FB_ERR_SHAPE;
+  if (a->ldo % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15) || (reinterpret_cast<uintptr_t>(tiles) & 15)) return FB_ERR_ALIGN;
+  cudaStream_t stream = static_cast<cudaStream_t>(stream_);
+  GpParams p{};
+  p.box_rows = a->page_size < kGpKv ? a->page_size : kGpKv;
+  CUtensorMap mq, mk, mv;
+  int rc = gp_map(&mq, a->q, a->dim_pad, a->heads, static_cast<uint64_t>(a->rows), a->ldq, per, tile_positions);
+  if (rc != FB_OK) return rc;
+  const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a->pool);
+  rc = gp_map(&mk, pool, a->dim_pad, a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
+  if (rc != FB_OK) return rc;
+  rc = gp_map(&mv, pool + static_cast<long long>(a->kv_heads) * a->dim_pad, a->vdim_pad, a->kv_heads,
+              static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
+  if (rc != FB_OK) return rc;
+  p.tiles = tiles;
+  p.block_table = a->block_table;
+  p.out = static_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo;
+  p.status = static_cast<DeviceStatus*>(a->status);
+  p.pool_rows = a->pool_rows;
+  p.rows = a->rows; p.heads = a->heads; p.kv_heads = a->kv_heads; p.per = per; p.positions = tile_positions;
+  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size; p.chunk = a->chunk;
+  p.dim_pad = a->dim_pad; p.vdim_pad = a->vdim_pad;
+  p.qb = (a->dim_pad + 63) / 64; p.vb = (a->vdim_pad + 63) / 64;
+  p.tmem_cols = p.vb * 64 + 2 * kGpKv <= 256 ? 256 : 512;
+  p.scale_log2 = a->scale * 1.4426950408889634f;
+  const int smem = p.qb * kGpQBlock + 2 * (p.qb + p.vb) * kGpKvBlock + 1024 + 256;
+  static bool attr = false;
+  if (!attr) {
+    const int most = 4 * kGpQBlock + 16 * kGpKvBlock + 1024 + 256;
+    if (cudaFuncSetAttribute(gqa_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  if (launch_pdl(gqa_prefill_tc_kernel, dim3(n_tiles, a->kv_heads), dim3(kGpThreads), smem, stream, mq, mk, mv, p) != cudaSuccess)
+    return FB_ERR_LAUNCH;
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}

@@ -33,6 +33,7 @@
 // bf16_mma.cuh:332-823: 64-token KV tiles, QK / PV on mma.sync).
 #include <cuda.h>
 
+#include "attn_tc.cuh"
 #include "common.cuh"
 #include "ferrule_b200.h"
 #include "launch.cuh"
@@ -71,41 +72,6 @@ struct TcParams {
   const __nv_bfloat16* gate; // optional [rows, ldg]: head output times sigmoid(gate[row][head])
   long long ldg;
 };
-
-__device__ __forceinline__ void umma_bf16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc,
-                                             uint32_t accumulate) {
-  asm volatile(
-      "{\n"
-      ".reg .pred p;\n"
-      "setp.ne.b32 p, %4, 0;\n"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n"
-      "}\n" ::"r"(tmem_d),
-      "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate)
-      : "memory");
-}
-
-__device__ __forceinline__ void tmem_st16(uint32_t taddr, const uint32_t (&r)[16]) {
-  asm volatile(
-      "tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], "
-      "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16};" ::"r"(taddr),
-      "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-      "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15])
-      : "memory");
-}
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-
-// MN-major operand laid out by TMA with the 128-byte swizzle: 64 contiguous elements of the MN dimension per
-// 128-byte row, 8 K-rows per 1024-byte group (stride byte offset), the next 64 MN elements `mn_block_bytes` on
-// (leading byte offset).
-__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr, uint32_t mn_block_bytes) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr & 0x3ffffu) >> 4);
-  d |= static_cast<uint64_t>(mn_block_bytes >> 4) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
-}
 
 template <int BLOCKS>
 __global__ void __launch_bounds__(kTcThreads, 1)
@@ -387,22 +353,6 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 // ---------------------------------------------------------------------------------
 // host side
 // ---------------------------------------------------------------------------------
-typedef CUresult (*TcEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
-                               const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
-                               CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-static TcEncodeFn tc_encoder() {
-  static TcEncodeFn fn = nullptr;
-  if (fn == nullptr) {
-    void* ptr = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess &&
-        q == cudaDriverEntryPointSuccess)
-      fn = reinterpret_cast<TcEncodeFn>(ptr);
-  }
-  return fn;
-}
-
 // bf16 [rows, width] matrix, box 64 features x box_rows rows, 128-byte swizzle, zeros outside
 static int tc_map(CUtensorMap* map, const void* base, int width, uint64_t rows, uint32_t box_rows) {
   TcEncodeFn fn = tc_encoder();

@@ -11,6 +11,7 @@
 // zeros), buffer `state_out[seq]` written (-1: nothing is kept), never the same one.
 #include "act_type.cuh"
 #include "common.cuh"
+#include "f32x2.cuh"
 #include "ferrule_b200.h"
 #include "launch.cuh"
 
@@ -65,26 +66,53 @@ __device__ __forceinline__ float scan_silu(float z) {
   return __fdividef(z, 1.f + __expf(-z));
 }
 
+// SPL states of a lane times one token: S <- exp2(d a) S + u B, returns this lane's share of S . C
+template <typename T, int SPL>
+__device__ __forceinline__ float scan_token(uint64_t (&S)[SPL / 2], const uint64_t (&a2)[SPL / 2], float2 du, const float* b,
+                                            const float* c) {
+  const uint64_t d2 = pack2(du.x, du.x), u2 = pack2(du.y, du.y);
+  uint64_t y = 0;
+#pragma unroll
+  for (int j = 0; j < SPL / 2; ++j) {
+    float e0, e1;
+    unpack2(mul2(d2, a2[j]), e0, e1);
+    S[j] = fma2(pack2(scan_exp2<T>(e0), scan_exp2<T>(e1)), S[j], mul2(u2, *reinterpret_cast<const uint64_t*>(b + 2 * j)));
+    y = fma2(S[j], *reinterpret_cast<const uint64_t*>(c + 2 * j), y);
+  }
+  float y0, y1;
+  unpack2(y, y0, y1);
+  return y0 + y1;
+}
+
 template <typename T, int LPC, int SPL>
 __global__ void __launch_bounds__(kScanThreads)
 selective_scan_kernel(const ScanParams<T> p) {
   constexpr int CH = kScanThreads / LPC, NP = LPC * SPL, TS = kScanTokens;
   constexpr int kPf = TS * CH / kScanThreads;                        // staged (token, channel) pairs per thread
   constexpr int kBc = (2 * TS * NP + kScanThreads - 1) / kScanThreads;
-  __shared__ float s_d[TS][CH], s_x[TS][CH], s_y[TS][CH];
+  static_assert(LPC >= 4 && SPL % 2 == 0, "four tokens share one reduction");
+  __shared__ float2 s_du[TS][CH];                                    // step size, step size times input
+  __shared__ float s_x[TS][CH], s_y[TS][CH];
   __shared__ __align__(16) float s_b[TS][NP], s_c[TS][NP];
   const int tid = threadIdx.x, l = tid % LPC, ch = tid / LPC;
-  const int seq = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
+  // (a mixed batch lists its decode rows first: the long sequences' CTAs start first and spread over all SMs)
+  const int seq = gridDim.y - 1 - blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
   const int sin = p.state_in[seq], sout = p.state_out[seq];
   const bool ok = sin < p.n_states && sout < p.n_states && !(sin >= 0 && sin == sout);
   const bool cin = c < p.inner;
-  float a2[SPL], S[SPL];
+  uint64_t a2[SPL / 2], S[SPL / 2];
 #pragma unroll
-  for (int j = 0; j < SPL; ++j) {
-    const int n = l * SPL + j;
-    const bool in = cin && n < p.state;
-    a2[j] = in ? p.a_log2[static_cast<long long>(n) * p.inner + c] : 0.f;
-    S[j] = in && ok && sin >= 0 ? p.states[(static_cast<long long>(sin) * p.state + n) * p.inner + c] : 0.f;
+  for (int j = 0; j < SPL / 2; ++j) {
+    float av[2], sv[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int n = l * SPL + 2 * j + e;
+      const bool in = cin && n < p.state;
+      av[e] = in ? p.a_log2[static_cast<long long>(n) * p.inner + c] : 0.f;
+      sv[e] = in && ok && sin >= 0 ? p.states[(static_cast<long long>(sin) * p.state + n) * p.inner + c] : 0.f;
+    }
+    a2[j] = pack2(av[0], av[1]);
+    S[j] = pack2(sv[0], sv[1]);
   }
   // staging role of this thread: channel `pc` of tokens pt, pt + 128 / CH, ...
   const int pc = tid % CH, pt = tid / CH;
@@ -110,7 +138,7 @@ selective_scan_kernel(const ScanParams<T> p) {
       fd[k] = fx[k] = fz_next[k] = 0.f;
       if (t < cnt && pin) {
         const long long r = r0 + t0 + t;
-        fd[k] = p.dt[r * p.lddt + c0 + pc];
+        fd[k] = __ldg(p.dt + r * p.lddt + c0 + pc);
         fx[k] = act_load(p.x + r * p.ldx + c0 + pc);
         fz_next[k] = act_load(p.z + r * p.ldz + c0 + pc);
       }
@@ -129,7 +157,8 @@ selective_scan_kernel(const ScanParams<T> p) {
 #pragma unroll
     for (int k = 0; k < kPf; ++k) {
       const int t = pt + k * kStep;
-      s_d[t][pc] = scan_softplus<T>(fd[k] + bias);
+      const float d = t < cnt ? scan_softplus<T>(fd[k] + bias) : 0.f;    // a step of size zero changes nothing
+      s_du[t][pc] = make_float2(d, d * fx[k]);
       s_x[t][pc] = fx[k];
       fz[k] = fz_next[k];
     }
@@ -140,23 +169,29 @@ selective_scan_kernel(const ScanParams<T> p) {
     }
     __syncthreads();
     if (t0 + TS < cnt_all) fetch(t0 + TS);
-    auto token = [&](int t) {
-      const float d = s_d[t][ch], u = d * s_x[t][ch];
-      float y = 0.f;
-#pragma unroll
-      for (int j = 0; j < SPL; ++j) {
-        S[j] = fmaf(scan_exp2<T>(d * a2[j]), S[j], u * s_b[t][l * SPL + j]);
-        y = fmaf(S[j], s_c[t][l * SPL + j], y);
-      }
+    if (cnt == 1) {
+      float y = scan_token<T, SPL>(S, a2, s_du[0][ch], &s_b[0][l * SPL], &s_c[0][l * SPL]);
 #pragma unroll
       for (int o = 1; o < LPC; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      if (l == 0) s_y[t][ch] = y;
-    };
-    if (cnt == TS) {
-#pragma unroll 4
-      for (int t = 0; t < TS; ++t) token(t);
+      if (l == 0) s_y[0][ch] = y;
     } else {
-      for (int t = 0; t < cnt; ++t) token(t);
+#pragma unroll 1
+      for (int t = 0; t < cnt; t += 4) {
+        float y[4];
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          y[q] = scan_token<T, SPL>(S, a2, s_du[t + q][ch], &s_b[t + q][l * SPL], &s_c[t + q][l * SPL]);
+        // four sums over the channel's lanes at once: lane l of the first four ends up with token t + l
+        const bool b0 = l & 1, b1 = l & 2;
+        float k0 = b0 ? y[1] : y[0], k1 = b0 ? y[3] : y[2];
+        k0 += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[1], 1);
+        k1 += __shfl_xor_sync(0xffffffffu, b0 ? y[2] : y[3], 1);
+        float v = b1 ? k1 : k0;
+        v += __shfl_xor_sync(0xffffffffu, b1 ? k0 : k1, 2);
+#pragma unroll
+        for (int o = 4; o < LPC; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+        if (LPC == 4 || l < 4) s_y[t + (l & 3)][ch] = v;
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -165,15 +200,20 @@ selective_scan_kernel(const ScanParams<T> p) {
       if (t < cnt && pin)
         act_store(p.out + (r0 + t0 + t) * p.ldo + c0 + pc, fmaf(skip, s_x[t][pc], s_y[t][pc]) * scan_silu<T>(fz[k]));
     }
-    // the next round overwrites this thread's own s_d / s_x entries, and s_b / s_c, last read before the barrier above;
+    // the next round overwrites this thread's own s_du / s_x entries and s_b / s_c, last read before the barrier above;
     // s_y is written again behind the next barrier
   }
   pdl_launch_dependents();
   if (sout >= 0 && cin) {
 #pragma unroll
-    for (int j = 0; j < SPL; ++j) {
-      const int n = l * SPL + j;
-      if (n < p.state) p.states[(static_cast<long long>(sout) * p.state + n) * p.inner + c] = S[j];
+    for (int j = 0; j < SPL / 2; ++j) {
+      float sv[2];
+      unpack2(S[j], sv[0], sv[1]);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int n = l * SPL + 2 * j + e;
+        if (n < p.state) p.states[(static_cast<long long>(sout) * p.state + n) * p.inner + c] = sv[e];
+      }
     }
   }
 }

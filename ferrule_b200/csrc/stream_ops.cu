@@ -290,6 +290,10 @@ short_conv_kernel(const ConvParams<TI, TO> p) {
     zero8<float>(b);
     if (p.bias) act_load8(p.bias + c, b);
     pdl_wait();
+    int i_[ROWS], n_[ROWS], in_[ROWS], out_[ROWS];
+    bool ok_[ROWS];
+#pragma unroll
+    for (int k = 0; k < ROWS; ++k) ok_[k] = rb + k < p.rows && conv_row(p, rb + k, i_[k], n_[k], in_[k], out_[k]);
     float win[ROWS + KEEP][8];
 #pragma unroll
     for (int t = 0; t < ROWS + KEEP; ++t) {
@@ -299,9 +303,8 @@ short_conv_kernel(const ConvParams<TI, TO> p) {
     }
 #pragma unroll
     for (int k = 0; k < ROWS; ++k) {
-      const int r = rb + k;
-      int i, n, sin, sout;
-      if (r >= p.rows || !conv_row(p, r, i, n, sin, sout)) continue;
+      if (!ok_[k]) continue;
+      const int r = rb + k, i = i_[k], n = n_[k], sin = in_[k], sout = out_[k];
       float acc[8];
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] = b[j];

@@ -47,6 +47,7 @@ class DeviceBatch:
     decode_only: bool = False   # every sequence has exactly one row (a plain decode step)
     tc_tiles: Optional[torch.Tensor] = None     # [cap, 4] int32 tiles of the tensor-core prefill attention kernel
     n_tc_tiles: int = 0
+    tc_positions: int = 0                       # most positions of a tile
     rest_ranges: Optional[list] = None          # (first row, end row) ranges the tiles do not cover
     # models with recurrent state (models/state_pool.py)
     seq_start: Optional[torch.Tensor] = None    # [>= n_seqs + 1] int32 first row of every sequence of the batch

@@ -348,6 +348,7 @@ class LayeredCuda:
         self.fp32 = weights.embed.dtype == torch.float32
         self.decode_rows = decode_rows
         self.attn_splits = attn_splits
+        self.max_seq_len = max_seq_len
         self.split_tokens = max(64, pad_to((max_seq_len + attn_splits - 1) // attn_splits, 64))
         self.ws = LayeredWorkspace(weights, max_rows, max_logit_rows, self.device)
         self.cache_index = {l: i for i, l in enumerate(self.cfg.cache_layers)}
@@ -440,7 +441,18 @@ class LayeredCuda:
         KL.gqa_prep(q, proj[:, mx.off["k"]:], proj[:, mx.off["v"]:], m, mx, self.rotation[m.rot_base, m.rot_dims],
                     b.positions[:T], b.write_slot[:T], pool, cfg.norm_eps, **mixed)
         out = self._view(self.ws.mix_in, T, m.heads * m.vdim_pad)
-        return KL.gqa_attention(q, m, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, out)
+        page = self.pool.page_size
+        if not KL.gqa_tc_group(m, q.dtype, page):
+            return KL.gqa_attention(q, m, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], page, out)
+        ranges = [(0, T)]
+        if b.n_tc_tiles:
+            KL.gqa_prefill_tc(q, m, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, b.tc_positions, page, out)
+            ranges = b.rest_ranges
+        for r0, r1 in ranges:
+            splits = KL.gqa_decode_splits(r1 - r0, m, self.max_seq_len)
+            KL.gqa_decode(q[r0:r1], m, pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], page, out[r0:r1],
+                          splits=splits, decode_only=b.decode_only)
+        return out
 
     def _mamba(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         K, KL, ws = self.K, self.KL, self.ws
@@ -451,7 +463,8 @@ class LayeredCuda:
         KL.short_conv(proj[:, mx.off["x"]:mx.off["x"] + Ip], mx.conv, self.states.tail[layer], x, b.row_seq[:T], *seqs,
                       bias=mx.conv_b, silu=True)
         low = self._view(ws.low, T, mx.w_x.shape[0])
-        K.gemm(x, mx.w_x, out=low)
+        # few output columns: row tiles small enough to fill the GPU
+        K.gemm(x, mx.w_x, out=low, ntok=32 if (T >= 1024 and not self.fp32) else None)
         dt = self._view(ws.dt, T, Ip)
         K.gemm(low[:, :mx.w_dt.shape[1]], mx.w_dt, out=dt)
         out = self._view(ws.mix_in, T, Ip)

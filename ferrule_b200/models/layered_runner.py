@@ -47,6 +47,11 @@ class LayeredRunner(DeepSeekRunner):
 
     def _prefill_tc_heads(self) -> int:
         from ..ops.kernels import prefill_tc_supported
+        if self.cfg.attention_layers:
+            # one tile table for all layers: as many positions as the widest group of query heads leaves room for
+            from ..ops.layered import gqa_tc_group
+            return max(gqa_tc_group(self.cfg.layers[i].mixer, self.w.embed.dtype, self.page_size)
+                       for i in self.cfg.attention_layers)
         heads = {self.cfg.layers[i].mixer.heads for i in self.cfg.latent_layers}
         if len(heads) != 1 or self.w.embed.dtype != torch.bfloat16:
             return 0

@@ -149,6 +149,7 @@ class BatchStaging:
                          self.d_bt, self.d_lrows, R, n_logit)
         if self.n_tiles:
             db.tc_tiles, db.n_tc_tiles, db.rest_ranges = self.d_tiles, self.n_tiles, self.rest_ranges
+            db.tc_positions = 128 // self.tc_heads
         if self.state_slots:
             db.seq_start, db.state_in, db.state_out, db.n_seqs = self.d_start, self.d_state_in, self.d_state_out, self.n_seqs
         return db

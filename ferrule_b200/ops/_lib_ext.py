@@ -81,6 +81,8 @@ def declare(lib) -> None:
         "fb_selective_scan": ([vp, vp], i),
         "fb_gqa_prep": ([vp, vp], i),
         "fb_gqa_attention": ([vp, vp], i),
+        "fb_gqa_decode": ([vp, i, i, vp], i),
+        "fb_gqa_prefill_tc": ([vp, vp, i, i, vp], i),
         # v4_ops.cu
         "fb_hc_pre": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, vp], i),
         "fb_hc_pre_split": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, i, vp, vp, vp], i),

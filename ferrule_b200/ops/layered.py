@@ -278,12 +278,56 @@ def gqa_prep(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, mixer, img, rota
     check(get_lib(True).fb_gqa_prep(C.byref(a), stream_ptr()), "fb_gqa_prep")
 
 
+def _gqa_rows(a: GqaArgs, block_table, row_seq, row_pos, page_size: int, out: torch.Tensor) -> None:
+    if row_seq is not None:
+        a.row_seq, a.row_pos = row_seq.data_ptr(), row_pos.data_ptr()
+    a.block_table, a.num_seqs, a.max_blocks, a.page_size = (block_table.data_ptr(), block_table.shape[0],
+                                                            block_table.shape[1], page_size)
+    a.out, a.ldo = out.data_ptr(), out.stride(0)
+
+
 def gqa_attention(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
                   row_pos: torch.Tensor, page_size: int, out: torch.Tensor) -> torch.Tensor:
     """32-bit arithmetic: out [rows, heads * vdim_pad]."""
     a = _gqa(q, mixer, pool)
-    a.block_table, a.row_seq, a.row_pos = block_table.data_ptr(), row_seq.data_ptr(), row_pos.data_ptr()
-    a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
-    a.out, a.ldo = out.data_ptr(), out.stride(0)
+    _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
     check(get_lib(True).fb_gqa_attention(C.byref(a), stream_ptr()), "fb_gqa_attention")
+    return out
+
+
+def gqa_tc_group(mixer, dtype, page_size: int) -> int:
+    """Query heads per key / value head when the bf16 kernels serve the mixer's prompts, else 0."""
+    per = mixer.heads // mixer.kv_heads
+    ok = (dtype == torch.bfloat16 and max(mixer.dim_pad, mixer.vdim_pad) <= 256 and per <= 128 and mixer.scale > 0
+          and page_size >= 8 and page_size & (page_size - 1) == 0)
+    return per if ok else 0
+
+
+def gqa_decode_splits(rows: int, mixer, max_keys: int) -> int:
+    """CTAs per row: about two per SM over the batch, each with at least 128 keys of the longest row."""
+    ctas = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads + 15) // 16)
+    splits = 1
+    while splits < 8 and ctas * splits * 2 <= 296 and min(mixer.chunk, max_keys) >= splits * 2 * 128:
+        splits *= 2
+    return splits
+
+
+def gqa_decode(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
+               row_pos: torch.Tensor, page_size: int, out: torch.Tensor, splits: int = 1, decode_only: bool = False
+               ) -> torch.Tensor:
+    """Few query rows, bf16.  decode_only: one row per sequence, every key below its position predates the running step."""
+    a = _gqa(q, mixer, pool)
+    _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
+    check(get_lib(True).fb_gqa_decode(C.byref(a), splits, 1 if decode_only else 0, stream_ptr()), "fb_gqa_decode")
+    return out
+
+
+def gqa_prefill_tc(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor, n_tiles: int,
+                   tile_positions: int, page_size: int, out: torch.Tensor) -> torch.Tensor:
+    """Prompt rows on tcgen05, bf16: tiles as `kernels.prefill_tiles` makes them; rows no tile covers are left alone."""
+    a = _gqa(q, mixer, pool)
+    _gqa_rows(a, block_table, None, None, page_size, out)
+    assert tiles.dtype == torch.int32 and tiles.shape[1] == 4 and tiles.is_contiguous() and n_tiles <= tiles.shape[0]
+    check(get_lib(True).fb_gqa_prefill_tc(C.byref(a), tiles.data_ptr(), n_tiles, tile_positions, stream_ptr()),
+          "fb_gqa_prefill_tc")
     return out

@@ -387,6 +387,42 @@ def test_attention_in_chunks(ops, dtype, m, page):
     near(out.view(len(rows), m.heads, -1)[..., :m.vdim], want, dtype)
 
 
+@pytest.mark.parametrize("page,splits,early", [(16, 1, False), (64, 2, False), (8, 4, True), (16, 8, True)])
+@pytest.mark.parametrize("m", [m for m in ATTENTIONS if max(m.dim, m.vdim) <= 256] + [AttentionMixer(40, 2, 64, 64, 0.9, 300, 1.0, 0)],
+                         ids=lambda m: f"{m.heads}x{m.kv_heads}x{m.dim}x{m.vdim}c{m.chunk}")
+def test_attention_of_few_rows(ops, m, page, splits, early):
+    KL = ops[1]
+    pool, table, q, rows, want = attention_case(m, BF, page, [1, 40, 300])
+    out = torch.full((len(rows), m.heads * m.vdim_pad), 7.0, dtype=BF, device="cuda")
+    KL.gqa_decode(q.flatten(1), m, pool, table, i32(*[s for s, _ in rows]), i32(*[p for _, p in rows]), page, out, splits=splits,
+                  decode_only=early)
+    near(out.view(len(rows), m.heads, -1)[..., :m.vdim], want, BF)
+
+
+@pytest.mark.parametrize("page", [8, 16, 64, 128])
+@pytest.mark.parametrize("m", [m for m in ATTENTIONS if max(m.dim, m.vdim) <= 256] + [AttentionMixer(14, 2, 256, 256, 0.9, 90, 1.0, 0)],
+                         ids=lambda m: f"{m.heads}x{m.kv_heads}x{m.dim}x{m.vdim}c{m.chunk}")
+def test_prompt_attention_on_tensor_cores(ops, m, page):
+    """Tiles that start and end anywhere: inside a chunk, at its border, over several chunks; portions that continue."""
+    K, KL = ops
+    parts = ((90, 0), (70, 130), (33, 27), (1, 64))
+    rows = [(s, p0 + i) for s, (n, p0) in enumerate(parts) for i in range(n)]
+    pool, table, q, rows, want = attention_case(m, BF, page, [p0 + n for n, p0 in parts], rows)
+    segs, r0 = [], 0
+    for s, (n, p0) in enumerate(parts):
+        segs.append((s, r0, n, p0))
+        r0 += n
+    out = torch.full((len(rows), m.heads * m.vdim_pad), 7.0, dtype=BF, device="cuda")
+    assert KL.gqa_tc_group(m, BF, page) == m.heads // m.kv_heads
+    for group in {m.heads // m.kv_heads, min(2 * m.heads // m.kv_heads, 128)}:      # also tiles another layer's groups limit
+        tiles, rest = K.prefill_tiles(segs, group, 2)
+        assert rest == [(len(rows) - 1, len(rows))]
+        KL.gqa_prefill_tc(q.flatten(1), m, pool, table, torch.from_numpy(tiles).cuda().contiguous(), len(tiles), 128 // group, page, out)
+        got = out.view(len(rows), m.heads, -1)
+        near(got[:-1, :, :m.vdim], want[:-1], BF)
+        assert (got[-1] == 7.0).all()
+
+
 # ------------------------------------------------------------------ whole models
 _memo = {}
 
