@@ -394,6 +394,14 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
             }
           }
         }
+        if (EPI == kEpiGelu) {
+          // all sixteen without a branch between them: their latencies overlap
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float x = __uint_as_float(v[j]);
+            v[j] = __float_as_uint(p.out_fp32 ? gelu_f(x) : gelu_bf16_f(x));
+          }
+        }
         if (EPI != kEpiAllReduce && p.stage_store) {
           // Swap-AB leaves a thread with one output channel of 16 rows: written directly that is sixteen 2-byte
           // stores per thread, 64 bytes per warp.  Stage the 16 x 128 chunk in shared memory (two buffers, chunk
@@ -413,7 +421,6 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
-              if (EPI == kEpiGelu) x = gelu_bf16_f(x);
               if (EPI == kEpiScatter && p.row_scale) x *= p.row_scale[row0 + r];
             }
             sb[j * 128 + ch_in_tile] = __float2bfloat16_rn(x);
@@ -452,7 +459,6 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 }
                 x = silu_f(x) * up;
               }
-              if (EPI == kEpiGelu) x = p.out_fp32 ? gelu_f(x) : gelu_bf16_f(x);
               long long orow = row0 + r;
               if (EPI == kEpiScatter) {
                 if (p.row_scale) x *= p.row_scale[row0 + r];

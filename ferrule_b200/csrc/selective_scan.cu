@@ -129,26 +129,25 @@ selective_scan_kernel(const ScanParams<T> p) {
     if (tid == 0) report_status(p.status, kStatusBadIndex, 0xD41, seq, r0);
     return;
   }
-  float fd[kPf], fx[kPf], fz[kPf], fz_next[kPf], fbc[kBc];
+  // The loads of the next tokens are unconditional (addresses clamped) and their conversion waits until they are staged:
+  // nothing between the request and the work on the current tokens depends on them.
+  float fd[kPf];
+  T fx[kPf], fz[kPf], fz_next[kPf], fbc[kBc];
+  const int pcc = min(c0 + pc, p.inner - 1);
   auto fetch = [&](int t0) {
     const int cnt = min(TS, cnt_all - t0);
 #pragma unroll
     for (int k = 0; k < kPf; ++k) {
       const int t = pt + k * kStep;
-      fd[k] = fx[k] = fz_next[k] = 0.f;
-      if (t < cnt && pin) {
-        const long long r = r0 + t0 + t;
-        fd[k] = __ldg(p.dt + r * p.lddt + c0 + pc);
-        fx[k] = act_load(p.x + r * p.ldx + c0 + pc);
-        fz_next[k] = act_load(p.z + r * p.ldz + c0 + pc);
-      }
+      const long long r = r0 + t0 + min(t, cnt - 1);
+      fd[k] = __ldg(p.dt + r * p.lddt + pcc);
+      fx[k] = __ldg(p.x + r * p.ldx + pcc);
+      fz_next[k] = __ldg(p.z + r * p.ldz + pcc);
     }
 #pragma unroll
     for (int k = 0; k < kBc; ++k) {
       const int i = tid + k * kScanThreads, t = i / (2 * NP), n = i % (2 * NP), m = n % NP;
-      fbc[k] = 0.f;
-      if (t < cnt && m < p.state)
-        fbc[k] = act_load(p.bc + (r0 + t0 + t) * p.ldbc + (n < NP ? p.off_b : p.off_c) + m);
+      fbc[k] = __ldg(p.bc + (r0 + t0 + min(t, cnt - 1)) * p.ldbc + (n < NP ? p.off_b : p.off_c) + min(m, p.state - 1));
     }
   };
   fetch(0);
@@ -158,14 +157,16 @@ selective_scan_kernel(const ScanParams<T> p) {
     for (int k = 0; k < kPf; ++k) {
       const int t = pt + k * kStep;
       const float d = t < cnt ? scan_softplus<T>(fd[k] + bias) : 0.f;    // a step of size zero changes nothing
-      s_du[t][pc] = make_float2(d, d * fx[k]);
-      s_x[t][pc] = fx[k];
+      const float x = act_load(&fx[k]);
+      s_du[t][pc] = make_float2(d, d * x);
+      s_x[t][pc] = x;
       fz[k] = fz_next[k];
     }
 #pragma unroll
     for (int k = 0; k < kBc; ++k) {
       const int i = tid + k * kScanThreads, t = i / (2 * NP), n = i % (2 * NP);
-      if (t < TS) (n < NP ? s_b[t][n] : s_c[t][n - NP]) = fbc[k];
+      // (padding states have a decay of one and start at zero: their input must be zero)
+      if (t < TS) (n < NP ? s_b[t][n] : s_c[t][n - NP]) = n % NP < p.state ? act_load(&fbc[k]) : 0.f;
     }
     __syncthreads();
     if (t0 + TS < cnt_all) fetch(t0 + TS);
@@ -198,7 +199,7 @@ selective_scan_kernel(const ScanParams<T> p) {
     for (int k = 0; k < kPf; ++k) {
       const int t = pt + k * kStep;
       if (t < cnt && pin)
-        act_store(p.out + (r0 + t0 + t) * p.ldo + c0 + pc, fmaf(skip, s_x[t][pc], s_y[t][pc]) * scan_silu<T>(fz[k]));
+        act_store(p.out + (r0 + t0 + t) * p.ldo + c0 + pc, fmaf(skip, s_x[t][pc], s_y[t][pc]) * scan_silu<T>(act_load(&fz[k])));
     }
     // the next round overwrites this thread's own s_du / s_x entries and s_b / s_c, last read before the barrier above;
     // s_y is written again behind the next barrier

@@ -269,6 +269,32 @@ __device__ __forceinline__ bool conv_row(const ConvParams<TI, TO>& p, int r, int
   return true;
 }
 
+// eight elements as they lie in memory
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<__nv_bfloat16> {
+  uint4 a;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { a = __ldg(reinterpret_cast<const uint4*>(p)); }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&a);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = __bfloat162float(e[j]);
+  }
+};
+template <>
+struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) {
+    a = __ldg(reinterpret_cast<const float4*>(p));
+    b = __ldg(reinterpret_cast<const float4*>(p) + 1);
+  }
+  __device__ __forceinline__ void get(float (&v)[8]) const {
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+  }
+};
+
 // ROWS consecutive rows x 8 channels per thread; KEEP = taps - 1 when it is at most 3 (the inputs of all rows are
 // requested together), -1: any number of taps
 template <typename TI, typename TO, int KEEP, int ROWS, bool RESIDUAL, bool SILU>
@@ -290,16 +316,30 @@ short_conv_kernel(const ConvParams<TI, TO> p) {
     zero8<float>(b);
     if (p.bias) act_load8(p.bias + c, b);
     pdl_wait();
-    int i_[ROWS], n_[ROWS], in_[ROWS], out_[ROWS];
+    // the inputs of all rows and the row tables are requested before anything is waited for (addresses clamped)
+    Raw8<TI> win[ROWS + KEEP];
+#pragma unroll
+    for (int t = 0; t < ROWS + KEEP; ++t) win[t].load(p.x + min(max(rb - KEEP + t, 0), p.rows - 1) * p.ldx + c);
+    int i_[ROWS], n_[ROWS], in_[ROWS], out_[ROWS], seq_[ROWS];
     bool ok_[ROWS];
 #pragma unroll
-    for (int k = 0; k < ROWS; ++k) ok_[k] = rb + k < p.rows && conv_row(p, rb + k, i_[k], n_[k], in_[k], out_[k]);
-    float win[ROWS + KEEP][8];
+    for (int k = 0; k < ROWS; ++k) seq_[k] = p.row_seq[min(rb + k, p.rows - 1)];
 #pragma unroll
-    for (int t = 0; t < ROWS + KEEP; ++t) {
-      const int r = rb - KEEP + t;
-      if (r >= 0 && r < p.rows) act_load8(p.x + r * p.ldx + c, win[t]);
-      else zero8<float>(win[t]);
+    for (int k = 0; k < ROWS; ++k) {
+      const int seq = min(max(seq_[k], 0), p.n_seqs - 1), r0 = p.seq_start[seq];
+      n_[k] = p.seq_start[seq + 1] - r0;
+      i_[k] = rb + k - r0;
+      in_[k] = p.state_in[seq];
+      out_[k] = p.state_out[seq];
+      ok_[k] = rb + k < p.rows;
+    }
+#pragma unroll
+    for (int k = 0; k < ROWS; ++k) {
+      if (!ok_[k]) continue;
+      const int r0 = rb + k - i_[k];
+      ok_[k] = seq_[k] >= 0 && seq_[k] < p.n_seqs && r0 >= 0 && i_[k] >= 0 && i_[k] < n_[k] && r0 + n_[k] <= p.rows &&
+               in_[k] < p.n_states && out_[k] < p.n_states && !(in_[k] >= 0 && in_[k] == out_[k]);
+      if (!ok_[k]) report_status(p.status, kStatusBadIndex, 0xD20, rb + k, seq_[k]);
     }
 #pragma unroll
     for (int k = 0; k < ROWS; ++k) {
@@ -312,8 +352,10 @@ short_conv_kernel(const ConvParams<TI, TO> p) {
       for (int t = 0; t <= KEEP; ++t) {
         const int back = KEEP - t;
         if (back <= i) {
+          float x[8];
+          win[k + t].get(x);
 #pragma unroll
-          for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[t][j], win[k + t][j], acc[j]);
+          for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[t][j], x[j], acc[j]);
         } else if (sin >= 0) {
           float o[8];
           act_load8(p.tail + (static_cast<long long>(sin) * KEEP + i + t) * p.channels + c, o);
@@ -321,8 +363,10 @@ short_conv_kernel(const ConvParams<TI, TO> p) {
           for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[t][j], o[j], acc[j]);
         }
       }
-      if (i == 0 || i >= n - KEEP) conv_tail(p.tail, p.channels, KEEP, c, i, n, sin, sout, win[k + KEEP]);
-      conv_finish<RESIDUAL, SILU, kExact>(win[k + KEEP], acc, p.out + r * p.ldo + c);
+      float x[8];
+      win[k + KEEP].get(x);
+      if (i == 0 || i >= n - KEEP) conv_tail(p.tail, p.channels, KEEP, c, i, n, sin, sout, x);
+      conv_finish<RESIDUAL, SILU, kExact>(x, acc, p.out + r * p.ldo + c);
     }
   } else {
     pdl_wait();

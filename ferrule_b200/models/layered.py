@@ -464,7 +464,7 @@ class LayeredCuda:
                       bias=mx.conv_b, silu=True)
         low = self._view(ws.low, T, mx.w_x.shape[0])
         # few output columns: row tiles small enough to fill the GPU
-        K.gemm(x, mx.w_x, out=low, ntok=32 if (T >= 1024 and not self.fp32) else None)
+        K.gemm(x, mx.w_x, out=low, ntok=64 if (T >= 512 and not self.fp32) else None)
         dt = self._view(ws.dt, T, Ip)
         K.gemm(low[:, :mx.w_dt.shape[1]], mx.w_dt, out=dt)
         out = self._view(ws.mix_in, T, Ip)
