@@ -398,8 +398,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
           // all sixteen without a branch between them: their latencies overlap
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
-            const float x = __uint_as_float(v[j]);
-            v[j] = __float_as_uint(p.out_fp32 ? gelu_f(x) : gelu_bf16_f(x));
+            v[j] = __float_as_uint(gelu_bf16_f(__uint_as_float(v[j])));
           }
         }
         if (EPI != kEpiAllReduce && p.stage_store) {
