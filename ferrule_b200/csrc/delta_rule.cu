@@ -48,7 +48,7 @@ struct DeltaParams {
   const int* seq_start;       // [n_seqs + 1]
   const int* state_in;
   const int* state_out;
-  int rows, n_seqs, heads, kv_heads, dim, vdim, taps;
+  int rows, n_seqs, heads, kv_heads, dim, vdim, taps, long_seqs;
   float *qn, *kn, *v, *decay, *beta, *qk, *o;      // scratch of the prefill form
   T* out;                     // [rows, ldo]
   long long ldo;
@@ -674,6 +674,7 @@ static int fill(const FbDeltaArgs* a, DeltaParams<T>& p) {
   p.row_seq = a->row_seq; p.seq_start = a->seq_start; p.state_in = a->state_in; p.state_out = a->state_out;
   p.rows = a->rows; p.n_seqs = a->n_seqs; p.heads = a->heads; p.kv_heads = a->kv_heads; p.dim = a->dim; p.vdim = a->vdim;
   p.taps = a->taps;
+  p.long_seqs = a->long_seqs;
   p.qn = a->qn; p.kn = a->kn; p.v = a->v; p.decay = a->decay; p.beta = a->beta; p.qk = a->qk; p.o = a->o;
   p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
   p.status = static_cast<DeviceStatus*>(a->status);
@@ -696,14 +697,20 @@ static int run_decode(const FbDeltaArgs* a, cudaStream_t s) {
 
 template <typename T, int RPT, int COLS, bool HEADG>
 static int launch_scan_cols(const DeltaParams<T>& p, cudaStream_t s) {
-  constexpr int smem = 2 * scan_buf<T, RPT, COLS, HEADG>() * static_cast<int>(sizeof(float));
+  constexpr int need = 2 * scan_buf<T, RPT, COLS, HEADG>() * static_cast<int>(sizeof(float));
+  constexpr int whole_sm = 120 * 1024;                 // more than half of an SM's shared memory
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT, COLS, HEADG>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
-        cudaSuccess)
+    if (cudaFuncSetAttribute(delta_scan_kernel<T, RPT, COLS, HEADG>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             need > whole_sm ? need : whole_sm) != cudaSuccess)
       return FB_ERR_LAUNCH;
     attr = true;
   }
+  // A mixed batch: few long sequences among decode rows.  The long ones' CTAs are bound by the latency of a token's chain
+  // and must not share an SM with each other while there are SMs for all of them.
+  const long long tiles = static_cast<long long>(p.heads) * ((p.vdim + 16 * COLS - 1) / (16 * COLS));
+  const bool spread = p.long_seqs > 0 && p.long_seqs < p.n_seqs && p.long_seqs * tiles <= 148;
+  const int smem = spread && need < whole_sm ? whole_sm : need;
   const dim3 grid(p.heads * ((p.vdim + 16 * COLS - 1) / (16 * COLS)), p.n_seqs);
   launch_pdl(delta_scan_kernel<T, RPT, COLS, HEADG>, grid, dim3(128), smem, s, p);
   return launched();
@@ -711,7 +718,7 @@ static int launch_scan_cols(const DeltaParams<T>& p, cudaStream_t s) {
 
 template <typename T, int RPT, bool HEADG>
 static int launch_scan_form(const DeltaParams<T>& p, cudaStream_t s) {
-  const long long per_col = static_cast<long long>(p.heads) * p.n_seqs;
+  const long long per_col = static_cast<long long>(p.heads) * (p.long_seqs > 0 ? p.long_seqs : p.n_seqs);
   auto ctas = [&](int cols) { return per_col * ((p.vdim + 16 * cols - 1) / (16 * cols)); };
   if constexpr (RPT <= 16) {
     if (ctas(4) >= 120 && p.vdim > 32) return launch_scan_cols<T, RPT, 4, HEADG>(p, s);

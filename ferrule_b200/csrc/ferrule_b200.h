@@ -361,6 +361,7 @@ typedef struct FbDeltaArgs {
   int off_a;                // >= 0: one decay per head, pre-activation in projected columns off_a .. (dt_bias: [heads])
   int off_g;                // >= 0: output gate pre-activation in projected columns off_g .. instead of `ag`
   int gate_silu;            // output gate's activation: 0 sigmoid, 1 silu
+  int long_seqs;            // sequences with more than one row, 0: not known (a hint for the scan's CTA placement)
   int fp32;                 // activations (proj, tail, out) are fp32 instead of bf16
   const float* conv;        // [taps, 2 * kv_heads * dim + heads * vdim]
   const float* a_neg;       // [heads] = -exp(A_log)

@@ -3,9 +3,11 @@
 //     d = softplus(dt_c + bias_c);   S[c, n] <- exp(d A[c, n]) S[c, n] + d x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
 //     out_c = y_c * silu(z_c)
 //
-// One kernel serves prompts and decode steps: CTA = (128 / LPC channels) x sequence, LPC lanes share a channel and hold
-// SPL states each in registers.  Tokens are staged sixteen at a time; the next ones are requested before the staged ones
+// Any mix of row counts: CTA = (128 / LPC channels) x sequence, LPC lanes share a channel and hold SPL states each in
+// registers.  Tokens are staged sixteen at a time; the next ones are requested before the staged ones
 // are worked on.  The exponentials do not depend on the state, so a token's chain is one multiply-add per state.
+// Decode steps (one row per sequence): a thread owns a channel, nothing is shared; states are requested before the
+// dependency wait.
 //
 // State of a sequence: fp32 [state, inner], channels innermost.  Buffer `state_in[seq]` is read (-1: a new sequence,
 // zeros), buffer `state_out[seq]` written (-1: nothing is kept), never the same one.
@@ -219,6 +221,54 @@ selective_scan_kernel(const ScanParams<T> p) {
   }
 }
 
+constexpr int kStepStates = 16;      // states requested at a time
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+selective_step_kernel(const ScanParams<T> p) {
+  pdl_launch_dependents();
+  const int seq = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int sin = p.state_in[seq], sout = p.state_out[seq];
+  const bool ok = sin < p.n_states && sout < p.n_states && !(sin >= 0 && sin == sout);
+  const int cc = min(c, p.inner - 1);
+  const float* old = p.states + static_cast<long long>(max(ok ? sin : 0, 0)) * p.state * p.inner + cc;
+  float S[kStepStates], a[kStepStates];
+  auto request = [&](int n0) {
+#pragma unroll
+    for (int j = 0; j < kStepStates; ++j) {
+      const long long n = min(n0 + j, p.state - 1);
+      a[j] = p.a_log2[n * p.inner + cc];
+      S[j] = old[n * p.inner];
+    }
+  };
+  request(0);
+  const float bias = p.dt_bias[cc], skip = p.d_skip[cc];
+  pdl_wait();
+  const int r = p.seq_start[seq];
+  if (!ok || r < 0 || r >= p.rows || p.seq_start[seq + 1] != r + 1) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD42, seq, r);
+    return;
+  }
+  const float x = act_load(p.x + r * p.ldx + cc), z = act_load(p.z + r * p.ldz + cc);
+  const float d = scan_softplus<T>(p.dt[r * p.lddt + cc] + bias), u = d * x;
+  const T* row = p.bc + r * p.ldbc;
+  float* dst = p.states + static_cast<long long>(max(sout, 0)) * p.state * p.inner + cc;
+  float y = 0.f;
+  for (int n0 = 0; n0 < p.state; n0 += kStepStates) {
+    if (n0 > 0) request(n0);
+#pragma unroll
+    for (int j = 0; j < kStepStates; ++j) {
+      const int n = n0 + j;
+      if (n < p.state) {
+        const float s = fmaf(scan_exp2<T>(d * a[j]), sin >= 0 ? S[j] : 0.f, u * act_load(row + p.off_b + n));
+        y = fmaf(s, act_load(row + p.off_c + n), y);
+        if (sout >= 0 && c < p.inner) dst[static_cast<long long>(n) * p.inner] = s;
+      }
+    }
+  }
+  if (c < p.inner) act_store(p.out + r * p.ldo + c, fmaf(skip, x, y) * scan_silu<T>(z));
+}
+
 template <typename T, int LPC, int SPL>
 static int launch_scan_form(const ScanParams<T>& p, cudaStream_t s) {
   constexpr int CH = kScanThreads / LPC;
@@ -237,6 +287,10 @@ static int run_scan(const FbScanArgs* a, cudaStream_t s) {
   p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
   p.rows = a->rows; p.n_seqs = a->n_seqs; p.inner = a->inner; p.state = a->state; p.n_states = a->n_states;
   p.status = static_cast<DeviceStatus*>(a->status);
+  if (p.n_seqs == p.rows) {
+    launch_pdl(selective_step_kernel<T>, dim3((p.inner + 127) / 128, p.n_seqs), dim3(128), 0, s, p);
+    return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  }
   if (p.state <= 8) return launch_scan_form<T, 4, 2>(p, s);
   if (p.state <= 16) return launch_scan_form<T, 4, 4>(p, s);
   if (p.state <= 32) return launch_scan_form<T, 4, 8>(p, s);

@@ -54,6 +54,7 @@ class DeviceBatch:
     state_in: Optional[torch.Tensor] = None     # [>= n_seqs] int32 state index read (-1: a new sequence)
     state_out: Optional[torch.Tensor] = None    # [>= n_seqs] int32 state index written (-1: none)
     n_seqs: int = 0
+    long_seqs: int = 0                          # of them with more than one row (0: not counted)
 
 
 class KvPool:

@@ -427,7 +427,7 @@ class LayeredCuda:
         decode = b.n_seqs == T and KL.delta_decode_supported(m)
         KL.delta_rule(proj, mx.off, ag, mx, m, self.cfg.norm_eps, self.states.state[layer], self.states.tail[layer],
                       b.seq_start, b.state_in, b.state_out, b.n_seqs, out, row_seq=b.row_seq[:T], scratch=ws.delta,
-                      decode=decode)
+                      decode=decode, long_seqs=b.long_seqs)
         return out
 
     def _attention(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:

@@ -88,6 +88,7 @@ class BatchStaging:
             self.np_state_in[:] = -1
             self.np_state_out[:] = -1
             self.n_seqs = seqs
+            self.long_seqs = 0
 
     def fill(self, b: ExecutionBatch, pad_rows: int = 0):
         T = b.rows
@@ -134,6 +135,7 @@ class BatchStaging:
     def fill_states(self, bindings) -> None:
         """(state read, state written) of every sequence of the batch just filled in, and its first rows."""
         n = self.n_seqs
+        self.long_seqs = sum(rows > 1 for _, _, rows in bindings)
         self.np_state_in[:n] = [r for r, _, _ in bindings]
         self.np_state_out[:n] = [w for _, w, _ in bindings]
         self.np_start[0] = 0
@@ -152,6 +154,7 @@ class BatchStaging:
             db.tc_positions = 128 // self.tc_heads
         if self.state_slots:
             db.seq_start, db.state_in, db.state_out, db.n_seqs = self.d_start, self.d_state_in, self.d_state_out, self.n_seqs
+            db.long_seqs = self.long_seqs
         return db
 
 

@@ -100,7 +100,7 @@ class DeltaArgs(C.Structure):
         ("proj", C.c_void_p), ("ldp", C.c_longlong),
         ("off_q", C.c_int), ("off_k", C.c_int), ("off_v", C.c_int), ("off_b", C.c_int),
         ("ag", C.c_void_p), ("ldag", C.c_longlong), ("off_gate", C.c_int),
-        ("off_a", C.c_int), ("off_g", C.c_int), ("gate_silu", C.c_int), ("fp32", C.c_int),
+        ("off_a", C.c_int), ("off_g", C.c_int), ("gate_silu", C.c_int), ("long_seqs", C.c_int), ("fp32", C.c_int),
         ("conv", C.c_void_p), ("a_neg", C.c_void_p), ("dt_bias", C.c_void_p), ("norm_w", C.c_void_p),
         ("state", C.c_void_p), ("tail", C.c_void_p), ("row_seq", C.c_void_p), ("seq_start", C.c_void_p),
         ("state_in", C.c_void_p), ("state_out", C.c_void_p),

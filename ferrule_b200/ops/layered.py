@@ -120,11 +120,11 @@ def delta_decode_supported(mixer) -> bool:
 def delta_rule(proj: torch.Tensor, off, ag: Optional[torch.Tensor], img, mixer, eps: float, state: torch.Tensor,
                tail: torch.Tensor, seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int,
                out: torch.Tensor, *, row_seq: Optional[torch.Tensor] = None, scratch: Optional[DeltaScratch] = None,
-               decode: bool = False) -> torch.Tensor:
+               decode: bool = False, long_seqs: int = 0) -> torch.Tensor:
     """Convolutions, recurrence and gated output norm of a delta mixer over the rows of a packed batch.
     proj: rows of the layer's input projection, `off` its block offsets; ag: fp32 rows of the second low-rank halves (None:
     decay and gate pre-activations are blocks `a` and `g` of the projection, one decay per head);
-    decode: one row per sequence, a single launch."""
+    decode: one row per sequence, a single launch; long_seqs: sequences with more than one row, when known."""
     assert (ag is None) == mixer.head_decay and (ag is None or ag.dtype == torch.float32)
     assert state.dtype == torch.float32 and state.is_contiguous() and tail.is_contiguous()
     assert tail.dtype == proj.dtype == out.dtype
@@ -133,7 +133,7 @@ def delta_rule(proj: torch.Tensor, off, ag: Optional[torch.Tensor], img, mixer, 
     a.off_q, a.off_k, a.off_v, a.off_b = off["q"], off["k"], off["v"], off["b"]
     a.ag, a.ldag, a.off_gate, a.fp32 = ptr(ag), ag.stride(0) if ag is not None else 0, img.off_gate, _fp32(proj)
     a.off_a, a.off_g = (off["a"], off["g"]) if ag is None else (-1, -1)
-    a.gate_silu = 1 if mixer.gate == "silu" else 0
+    a.gate_silu, a.long_seqs = 1 if mixer.gate == "silu" else 0, long_seqs
     a.conv, a.a_neg, a.dt_bias, a.norm_w = (img.conv.data_ptr(), img.a_neg.data_ptr(), img.dt_bias.data_ptr(),
                                             img.o_norm.data_ptr())
     a.state, a.tail, a.n_states = state.data_ptr(), tail.data_ptr(), state.shape[0]

@@ -9,7 +9,8 @@ import numpy as np
 import pytest
 import torch
 
-from ferrule_b200.models.layered_config import AttentionMixer, MambaMixer
+from ferrule_b200.models.layered_config import (OUTPUT_NORM, AttentionMixer, DenseSpec, LayeredConfig, LayerSpec,
+                                                MambaMixer)
 from ferrule_b200.models.layered_runner import LayeredRunner
 from ferrule_b200.models.layered_weights import RandomTensors, pack_weights
 from ferrule_b200.runtime.engine import Engine, EngineConfig, TokenEvent
@@ -481,6 +482,35 @@ def test_portions_of_any_size(sizes, dtype):
         rows.append(eng.replay([ReplayEntry("a", toks[at:at + n], list(range(n)))])[0])
         at += n
     same(np.concatenate(rows), want, dtype)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+@pytest.mark.parametrize("decoded", [False, True])
+@pytest.mark.parametrize("page,chunk", [(8, 24), (64, 50), (16, 16)])
+def test_a_token_is_seen_exactly_inside_its_chunk(page, chunk, decoded, dtype):
+    """One attention layer and no convolution: a changed token changes the logits of its own chunk behind it, no others."""
+    cfg = LayeredConfig(vocab_size=50, width=32, layers=(LayerSpec(AttentionMixer(4, 2, 16, 16, 0.5, chunk, 50.0, 8), DenseSpec(24)),),
+                        norm_eps=1e-5, name="supisun", max_position=200, block=OUTPUT_NORM, canon_taps=1, learned_positions=True)
+    w = pack_weights(cfg, lambda n, t=RandomTensors(cfg, seed=3, dtype=F32, gain=1.5): t(n).to(device="cuda", dtype=dtype))
+    runner = LayeredRunner(w, n_pages=160 // page + 1, page_size=page, max_rows=160, max_seqs=1, max_seq_len=160, full_logit_rows=64)
+    eng = ReplayEngine(runner, EngineConfig(scheduler=SchedulerConfig(1, 1, 160, 160, ctx_size=160), kv_pages=160 // page + 1,
+                                            page_size=page))
+    toks = prompt(cfg, 110, 5)
+
+    def logits(seq):
+        # the head in one portion; the tail decoded token by token, or in a second portion
+        cuts = [(0, 60)] + ([(i, 1) for i in range(60, 110)] if decoded else [(60, 50)])
+        out = [eng.replay([ReplayEntry("a", seq[i:i + n], list(range(n)))], ["a"] if i + n == 110 else [])[0] for i, n in cuts]
+        return np.concatenate(out)
+
+    base = logits(toks)
+    edges = sorted({k * chunk + o for k in range(3) for o in (-1, 0, 1)} | {page - 1, page})
+    for t in (e for e in edges if 0 <= e < 110):
+        seq = list(toks)
+        seq[t] = (seq[t] + 7) % cfg.vocab_size
+        changed = np.abs(logits(seq) - base).max(1) > 1e-3
+        want = np.array([p >= t and p // chunk == t // chunk for p in range(110)])
+        assert not changed[~want].any() and changed[want].mean() > 0.9 and changed[t], t
 
 
 @pytest.mark.parametrize("dtype", [F32, BF])
