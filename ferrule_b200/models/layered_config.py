@@ -474,6 +474,27 @@ def gitozen_latent_lite(n_layers: int = 27) -> LayeredConfig:
     return base.with_(layers=(lat,) * n_layers, name="gitozen-latent-lite")
 
 
+def _gitozen_dense(name: str, width: int, heads: int, dim: int, ff: int, n_layers: int) -> LayeredConfig:
+    """One expert of the given inner width that takes every token: a dense feed-forward.  Sizes beside the supisun-*
+    presets: the same widths, heads, depth and about as many parameters."""
+    lat = LatentMixer(heads=heads, dim=dim, vdim=dim, kv_rank=512, scale=dim ** -0.5)
+    dlt = DeltaMixer(heads=heads, kv_heads=heads, dim=dim, vdim=dim, taps=4, decay_rank=128, gate_rank=128)
+    return LayeredConfig(vocab_size=102400, width=width, layers=tuple(
+        LayerSpec(lat if i % 4 == 3 else dlt, MoeSpec(experts=1, top=1, ff=ff)) for i in range(n_layers)), name=name)
+
+
+def gitozen_dense_small(n_layers: int = 24) -> LayeredConfig:
+    return _gitozen_dense("gitozen-dense-small", 1024, 8, 128, 2048, n_layers)
+
+
+def gitozen_dense_lite(n_layers: int = 27) -> LayeredConfig:
+    return _gitozen_dense("gitozen-dense-lite", 2048, 16, 128, 4608, n_layers)
+
+
+def gitozen_dense_wide(n_layers: int = 32) -> LayeredConfig:
+    return _gitozen_dense("gitozen-dense-wide", 4096, 32, 128, 7680, n_layers)
+
+
 def _supisun(vocab: int, width: int, layers, max_position: int, taps: int = 4, eps: float = 1e-6,
              name: str = "supisun") -> LayeredConfig:
     return LayeredConfig(vocab_size=vocab, width=width, layers=tuple(layers), norm_eps=eps, name=name,
@@ -512,5 +533,7 @@ def supisun_wide(n_layers: int = 32) -> LayeredConfig:
 
 
 PRESETS = {"tiny-gitozen": tiny_gitozen, "gitozen-lite": gitozen_lite, "gitozen-latent-lite": gitozen_latent_lite,
+           "gitozen-dense-small": gitozen_dense_small, "gitozen-dense-lite": gitozen_dense_lite,
+           "gitozen-dense-wide": gitozen_dense_wide,
            "tiny-supisun": tiny_supisun, "supisun-small": supisun_small, "supisun-lite": supisun_lite,
            "supisun-wide": supisun_wide}
