@@ -170,7 +170,7 @@ def main() -> None:
         # instantiated (its weights are not part of the decode step's traffic either way)
         cfg = cfg.with_(n_mtp_layers=0)
     if args.layers:
-        cfg = cfg.with_(layers=cfg.layers[:args.layers]) if layered else cfg.with_(n_layers=args.layers)
+        cfg = cfg.first_layers(args.layers) if layered else cfg.with_(n_layers=args.layers)
     B, P, K, Wm = args.batch, args.prompt_len, args.steps, args.warmup
     page = 64
     margin = 64                      # sequences that finish prefill early decode ahead of the others

@@ -229,10 +229,10 @@ def _expert_plan(args):
 
 
 def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=None):
-    """A layer-list model (Gitozen, Supisun) behind the engine: a checkpoint directory, or a random-init preset."""
+    """A layer-list model (Gitozen, Supisun, Vedadra) behind the engine: a checkpoint directory, or a random-init preset."""
     import torch
 
-    from ..models.layered_config import PRESETS
+    from ..models.layered_config import PRESETS, preset_architecture
     from ..models.layered_weights import random_weights
     from ..models.registry import ARCHITECTURES, RunnerLimits
     from ..runtime.engine import Engine, EngineConfig
@@ -247,7 +247,7 @@ def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=Non
     if getattr(args, "weight_format", "bf16") != "bf16":
         raise SystemExit("--weight-format: layer-list models run bf16 weights")
     args.speculative = False
-    arch = ARCHITECTURES[_architecture(model_dir) if model_dir else ("supisun" if "supisun" in args.preset else "gitozen")]
+    arch = ARCHITECTURES[_architecture(model_dir) if model_dir else preset_architecture(args.preset)]
     dtype = torch.bfloat16 if dev != "cpu" else torch.float32
     if model_dir:
         weights = arch.load(model_dir, dev, dtype, max_layers=getattr(args, "layers", 0))
@@ -255,14 +255,14 @@ def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=Non
     else:
         cfg = PRESETS[args.preset]()
         if getattr(args, "layers", 0):
-            cfg = cfg.with_(layers=tuple(cfg.layers[i % cfg.n_layers] for i in range(args.layers)))
+            cfg = cfg.cycled(args.layers)
         weights = random_weights(cfg, device=dev, dtype=dtype, seed=args.seed)
         name = args.preset
     cfg = weights.cfg
     ctx, pages_per_seq, sched = _engine_sizes(args, cfg.max_position)
     n_pages = args.max_seqs * pages_per_seq + 8
     if args.kv_cache_mb:
-        per_page = max(len(cfg.cache_layers), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
+        per_page = max(len(cfg.cache_runs), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
         n_pages = max(args.kv_cache_mb * (1 << 20) // per_page, pages_per_seq + 1)
     runner = arch.runner(weights, RunnerLimits(n_pages, args.page_size, args.max_batch_tokens, args.max_seqs, ctx), device=dev)
     eng = Engine(runner, EngineConfig(scheduler=sched, kv_pages=n_pages, page_size=args.page_size))
@@ -426,6 +426,7 @@ def cmd_make_fixture(args) -> int:
     from ..io.checkpoint import export_hf
     from ..models import config as C
     from ..models import weights as W
+    from ..models.layered_config import ARCHITECTURES
     if args.family == "v4":
         # DeepSeek-V4 layout: FP8 attention / shared experts, packed FP4 routed experts unless told otherwise
         from ..io.v4_checkpoint import export_v4_hf
@@ -446,13 +447,13 @@ def cmd_make_fixture(args) -> int:
         print(json.dumps({"written": args.out, "family": "deepseek_v4", "layers": cfg.n_layers,
                           "proposal_stages": cfg.n_proposal_stages, "dense_format": dense, "expert_format": expert}))
         return 0
-    if args.family in ("gitozen", "supisun"):
+    if args.family in ARCHITECTURES:
         from ..io.layered_checkpoint import export_layered
         from ..models.layered_config import PRESETS
         from ..models.layered_weights import RandomTensors
         lcfg = PRESETS[args.preset if args.preset in PRESETS else f"tiny-{args.family}"]()
         if args.layers:
-            lcfg = lcfg.with_(layers=tuple(lcfg.layers[i % lcfg.n_layers] for i in range(args.layers)))
+            lcfg = lcfg.cycled(args.layers)
         if args.dense_format != "plain" or args.expert_format != "plain":
             raise SystemExit(f"--family {args.family}: checkpoints are stored in BF16")
         export_layered(lcfg, RandomTensors(lcfg, args.seed, gain=0.0 if args.zeros else 1.0), args.out, args.shard_mb << 20)
@@ -877,6 +878,7 @@ def cmd_expert_stream_smoke(args) -> int:
 
 
 def main(argv: Optional[List[str]] = None) -> int:
+    from ..models.layered_config import ARCHITECTURES as LAYERED
     ap = argparse.ArgumentParser(prog="ferrule_b200")
     sub = ap.add_subparsers(dest="cmd", required=True)
     p = sub.add_parser("info"); p.add_argument("model", nargs="?"); p.add_argument("--model-dir"); p.set_defaults(fn=cmd_info)
@@ -887,9 +889,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--zeros", action="store_true"); p.add_argument("--shard-mb", type=int, default=1024)
     p.add_argument("--dense-format", default="plain", choices=["plain", "fp8_block"])
     p.add_argument("--expert-format", default="plain", choices=["plain", "fp8_block", "mxfp4"])
-    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", "gitozen", "supisun"],
+    p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", *LAYERED],
                    help="v4: a DeepSeek-V4 directory (tiny shape; FP8 dense + packed FP4 experts unless --plain); "
-                        "gitozen, supisun: a layer-list directory (--preset tiny-<family> unless another of its presets is named)")
+                        "gitozen, supisun, vedadra: a layer-list directory (--preset tiny-<family> unless another of its presets is named)")
     p.add_argument("--plain", action="store_true", help="--family v4: keep every linear in BF16")
     p.add_argument("--proposal-stages", type=int, default=0,
                    help="--family v4: also write this many `mtp.*` proposal stages with their prediction heads")

@@ -1,4 +1,4 @@
-"""Checkpoint directories of layer-list models (Gitozen, Supisun): `config.json` with one entry per layer, and safetensors
+"""Checkpoint directories of layer-list models (Gitozen, Supisun, Vedadra): `config.json` with one entry per layer, and safetensors
 files whose tensors are named `embed`, `pos`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.rg1`, `final.norm`, `head`
 (`LayeredConfig.tensor_shapes` lists them).  Linear weights are stored [out, in] in BF16."""
 from __future__ import annotations
@@ -37,7 +37,7 @@ def load_layered(directory, device="cpu", dtype=torch.bfloat16, max_layers: int 
     ck = ShardedCheckpoint(directory)
     cfg = from_layer_list(directory)
     if max_layers:
-        cfg = cfg.with_(layers=cfg.layers[:max_layers])
+        cfg = cfg.first_layers(max_layers)
     cfg = bind_config(cfg, ck)
     for name, shape in cfg.tensor_shapes().items():
         if not ck.has(name):

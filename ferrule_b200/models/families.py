@@ -4,7 +4,7 @@ Roles tell the loader what a tensor is (attention projection, norm, router, rout
 weight, scale, MTP part ...) independent of the naming scheme.  Families: DeepSeek (HuggingFace
 V2/V3 names: `model.layers.N.self_attn.q_a_proj.weight`), DeepSeek-V4 (the reference's flat names:
 `layers.N.attn.wq_a.weight`, `ffn.experts.E.w1.weight`, `mtp.M.*`), Gitozen (layer-list names:
-`lN.mix.q`, `lN.mlp.eE.gate`), Supisun (the same scheme), Qwen3 and generic Llama-style.  The DeepSeek families and
+`lN.mix.q`, `lN.mlp.eE.gate`), Supisun and Vedadra (the same scheme), Qwen3 and generic Llama-style.  The DeepSeek families and
 the layer-list ones execute; the others
 are classified for inspection.
 
@@ -65,6 +65,8 @@ class TensorRole(Enum):
     INPUT_CONV = "input_conv"
     POSITION = "position"
     VALUE_MIX = "value_mix"
+    HEAD_MIX = "head_mix"
+    MAP_WEIGHT = "map_weight"
     MTP = "mtp"
     SCALE = "scale"
     UNKNOWN = "unknown"
@@ -84,6 +86,7 @@ class Family(Enum):
     DEEPSEEK_V4 = "deepseek_v4"
     GITOZEN = "gitozen"
     SUPISUN = "supisun"
+    VEDADRA = "vedadra"
     QWEN3 = "qwen3"
     LLAMA = "llama"
 
@@ -111,7 +114,10 @@ _LAYERED_MIX = {"q": TensorRole.ATTN_Q, "k": TensorRole.ATTN_K, "v": TensorRole.
                 "norm": TensorRole.DELTA_NORM, "a": TensorRole.DELTA_DECAY, "q.norm": TensorRole.ATTN_Q_NORM,
                 "k.norm": TensorRole.ATTN_KV_NORM, "vmix": TensorRole.VALUE_MIX, "in": TensorRole.SCAN_IN,
                 "conv": TensorRole.SCAN_PARAM, "conv.b": TensorRole.SCAN_PARAM, "x": TensorRole.SCAN_PARAM,
-                "dt": TensorRole.SCAN_PARAM, "dt.b": TensorRole.SCAN_PARAM, "D": TensorRole.SCAN_PARAM}
+                "dt": TensorRole.SCAN_PARAM, "dt.b": TensorRole.SCAN_PARAM, "D": TensorRole.SCAN_PARAM,
+                "q.b": TensorRole.ATTN_Q, "k.b": TensorRole.ATTN_K, "o.b": TensorRole.ATTN_OUT,
+                "talk": TensorRole.HEAD_MIX, "temp": TensorRole.HEAD_MIX, "lq1": TensorRole.MAP_WEIGHT,
+                "lk1": TensorRole.MAP_WEIGHT, "lq2": TensorRole.MAP_WEIGHT, "lk2": TensorRole.MAP_WEIGHT}
 _LAYERED_FFN = {"gate": 0, "up": 1, "down": 2}
 
 
@@ -124,13 +130,13 @@ def _classify_layered(name: str) -> "TensorClass":
     if not m:
         return TensorClass(TensorRole.UNKNOWN)
     layer, rest = int(m.group(1)), m.group(2)
-    if rest in ("norm1", "norm1.b"):
+    if rest in ("norm1", "norm1.b", "norm1b"):
         return TensorClass(TensorRole.ATTN_NORM, layer)
-    if rest in ("norm2", "norm2.b"):
+    if rest in ("norm2", "norm2.b", "norm2b"):
         return TensorClass(TensorRole.FFN_NORM, layer)
     if rest == "canon1":
         return TensorClass(TensorRole.INPUT_CONV, layer)
-    if rest in ("mlp.up", "mlp.down"):
+    if rest in ("mlp.gate", "mlp.up", "mlp.down"):
         return TensorClass(_ffn_role("dense", _LAYERED_FFN[rest[4:]]), layer)
     if re.fullmatch(r"rg[12](\.b)?", rest):
         return TensorClass(TensorRole.RESIDUAL_GATE, layer)
@@ -152,7 +158,7 @@ def _ffn_role(kind: str, idx: int) -> TensorRole:
 
 
 def classify(name: str, family: Family, n_layers: Optional[int] = None) -> TensorClass:
-    if family in (Family.GITOZEN, Family.SUPISUN):
+    if family in (Family.GITOZEN, Family.SUPISUN, Family.VEDADRA):
         return _classify_layered(name)
     is_scale = name.endswith(_SCALE_SUFFIX)
     base = name
@@ -250,6 +256,8 @@ def detect_family(names: Iterable[str], model_type: str = "") -> Family:
     names = list(names)
     if "l0.canon1" in names or model_type.lower() == "supisun":
         return Family.SUPISUN
+    if "l0.norm1b" in names or model_type.lower() == "vedadra":
+        return Family.VEDADRA
     if "l0.norm1" in names or model_type.lower() == "gitozen":
         return Family.GITOZEN
     if any(n.startswith("layers.") and ".attn.wq_a" in n for n in names) or any(n.startswith("mtp.") for n in names):

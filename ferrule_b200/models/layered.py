@@ -14,13 +14,25 @@ Output-norm blocks:
                 x += norm2(ff(x))
     logits = head . norm_final(x)
 
+Sandwich blocks (every norm an RMS norm in groups):
+
+    x = embed[token]
+    per run:    x += embed[token]                                (first layer of every later pass of a loop)
+                x += norm1b(mixer(norm1(x)))
+                x += norm2b(ff(norm2(x)))
+    logits = head . norm_final(x)
+
+A layer that runs several times has a cache plane and a state per run.
+
 * `LayeredReference` - plain PyTorch; the execution path of a CPU runner.
 * `LayeredCuda`      - the sm_100a kernel pipeline, allocation-free over a preallocated workspace, so a decode step can be
   captured in a CUDA graph.  With fp32 weights the same pipeline runs in full 32 bits.
 
 Kernels of a latent layer: input projection (one GEMM for q, latent, gates) -> latent append -> W_uk absorption ->
 attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o.  Of an attention layer: input projection (q, k,
-v) -> norms, rotation, value mixing and cache append in one launch -> attention -> W_o.  Of a delta layer: input projection
+v) -> norms, rotation, value mixing and cache append in one launch -> attention -> W_o.  Of a window layer: input projection
+(q, k, v, gate) -> norms, mixing of the queries across heads and cache append in one launch -> attention (distance bias,
+difference of the two maps, gate inside) -> W_o.  Of a delta layer: input projection
 -> second low-rank halves -> delta rule -> W_o.  Of a selective-scan layer: input projection -> convolution -> W_x -> W_dt
 -> scan (step sizes, skip and output gate inside) -> W_o.
 
@@ -28,7 +40,8 @@ In a parallel gated block the feed-forward branch reads the same h and runs on a
 (+ row reservation) -> grouped SwiGLU GEMM -> grouped scatter GEMM.  One kernel joins both branches: gated residual
 additions, expert reduction, next layer's norm.  In an output-norm block one kernel after each sublayer normalises its
 output, adds it to the stream and leaves the rows the next GEMM reads; in decode steps it also applies the next mixer's
-input convolution, whose earlier inputs are in the state pool then.
+input convolution, whose earlier inputs are in the state pool then.  In a sandwich block the same kernel takes the norm of the
+sublayer's output, the addition, the embedding of a new pass and the next sublayer's input norm.
 """
 from __future__ import annotations
 
@@ -40,8 +53,8 @@ import torch.nn.functional as F
 from ..ops import reference as ref
 from .config import SCORE_SOFTMAX
 from .deepseek import DeviceBatch, KvPool, _pow2_at_least
-from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, AttentionMixer, DeltaMixer, LatentMixer, MambaMixer,
-                             MoeSpec, pad_to)
+from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, SANDWICH_NORM, AttentionMixer, DeltaMixer, LatentMixer, MambaMixer,
+                             MoeSpec, WindowMixer, pad_to)
 from .layered_weights import LayerImage, LayeredWeights, MixerImage
 from .state_pool import RecurrentStatePool
 
@@ -57,7 +70,7 @@ def rotation_frequencies(base: float, dims: int) -> torch.Tensor:
 class LayeredReference:
     def __init__(self, weights: LayeredWeights, pool: KvPool, states: RecurrentStatePool):
         self.w, self.cfg, self.pool, self.states = weights, weights.cfg, pool, states
-        self.cache_index = {l: i for i, l in enumerate(self.cfg.cache_layers)}
+        self.cache_index = {r: i for i, r in enumerate(self.cfg.cache_runs)}
         self.prof = self.tap = None
 
     def _norm(self, x: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
@@ -198,6 +211,44 @@ class LayeredReference:
             out[r] = torch.einsum("ght,tgv->ghv", w, v).reshape(H, vp)
         return out.view(T, H * vp) @ mx.w_o.float().T
 
+    def _window(self, run: int, mx: MixerImage, m: WindowMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        T, o, eps = proj.shape[0], mx.off, self.cfg.norm_eps
+        H, G, M, D, V, dp, vp = m.heads, m.kv_heads, m.maps, m.dim, m.vdim, m.dim_pad, m.vdim_pad
+        part = lambda name, heads, pad: proj[:, o[name]:o[name] + heads * pad]
+        rms = lambda t, n: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / n + eps)
+        q, k = part("q", H * M, dp), part("k", G * M, dp)
+        if m.biases:
+            q, k = q + mx.q_bias, k + mx.k_bias
+        v = k if m.tied_values else part("v", G, vp)
+        q = rms(q.reshape(T, H, M, dp), D) * mx.q_norm
+        row = torch.zeros(T, self.cfg.kv_row_dim)
+        row[:, :m.v_offset] = (rms(k.reshape(T, G * M, dp), D) * mx.k_norm).view(T, -1)
+        row[:, m.v_offset:m.v_offset + G * vp] = v
+        slots = b.write_slot[:T]
+        ok = slots >= 0
+        rows = self.pool.layer(self.cache_index[run]).view(-1, self.cfg.kv_row_dim)
+        rows[slots[ok]] = row[ok].to(rows.dtype)
+        out, ps = torch.zeros(T, H, vp), self.pool.page_size
+        for r in range(T):
+            p, seq = int(b.row_pos[r]), int(b.row_seq[r])
+            first = max(p - m.window + 1, 0)
+            t = torch.cat([torch.arange(min(m.keep_first, first)), torch.arange(first, p + 1)])
+            if t.numel() == 0:
+                continue
+            kv = rows[b.block_table[seq, t // ps].long() * ps + t % ps].float()
+            k = kv[:, :m.v_offset].view(-1, G, M, dp).repeat_interleave(H // G, 1)
+            v = kv[:, m.v_offset:m.v_offset + G * vp].view(-1, G, vp).repeat_interleave(H // G, 1)
+            s = torch.einsum("hmd,thmd->hmt", q[r], k)
+            s = torch.einsum("hg,gmt->hmt", mx.q_mix, s) if m.mix_heads else s * mx.q_mix[:, None, None]
+            if m.distance_bias:
+                s = s - (mx.slopes[:, None] * (p - t))[:, None]
+            a = torch.einsum("hmt,thv->hmv", torch.softmax(s, -1), v)
+            out[r] = a[:, 0] if M == 1 else rms(a[:, 0] - mx.diff_lambda * a[:, 1], V) * (1 - m.diff)
+        if m.gate:
+            out = out * torch.sigmoid(part("g", H, vp).reshape(T, H, vp))
+        y = out.view(T, H * vp) @ mx.w_o.float().T
+        return y + mx.o_bias if m.biases else y
+
     def _mamba(self, layer: int, mx: MixerImage, m: MambaMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
         o, Ip, N = mx.off, m.inner_pad, m.state
         x = F.silu(self._conv(proj[:, o["x"]:o["x"] + Ip], mx.conv, self.states.tail[layer], b) + mx.conv_b)
@@ -217,8 +268,8 @@ class LayeredReference:
 
     def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
         m = lw.spec.mixer
-        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, DeltaMixer: self._delta,
-              MambaMixer: self._mamba}[type(m)]
+        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, WindowMixer: self._window,
+              DeltaMixer: self._delta, MambaMixer: self._mamba}[type(m)]
         return fn(layer, lw.mixer, m, proj, b)
 
     def _gated_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
@@ -243,22 +294,39 @@ class LayeredReference:
             x = x + self._layer_norm(F.gelu(x @ lw.w_up.float().T) @ lw.w_down.float().T, lw.norm2)
         return x
 
+    def _group_norm(self, x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        W, out = self.cfg.width, torch.zeros_like(x)
+        parts = x[:, :W].unflatten(1, (self.cfg.norm_groups, -1))
+        out[:, :W] = (parts * torch.rsqrt(parts.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps)).flatten(1) * w[:W]
+        return out
+
+    def _sandwich_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        norm = self._group_norm
+        x = x + norm(self._mixer(i, lw, norm(x, lw.norm1) @ lw.mixer.w_in.float().T, b), lw.norm1b)
+        if lw.spec.mlp is not None:
+            g, u = (norm(x, lw.norm2) @ lw.w_up.float().T).chunk(2, -1)
+            x = x + norm((F.gelu(g, approximate="tanh") * u) @ lw.w_down.float().T, lw.norm2b)
+        return x
+
     def hidden_states(self, b: DeviceBatch, allreduce=None, start_layer: int = 0, h0=None) -> torch.Tensor:
         """Residual stream after the last layer [rows, width_pad]."""
-        x = self.w.embed[b.token_ids[:b.n_rows].long()].float()
+        x = embedded = self.w.embed[b.token_ids[:b.n_rows].long()].float()
         if self.w.pos is not None:
             x = x + self.w.pos[b.positions[:b.n_rows].long()].float()
-        layer = self._gated_layer if self.cfg.block == PARALLEL_GATED else self._output_norm_layer
-        for i, lw in enumerate(self.w.layers):
+        layer = {PARALLEL_GATED: self._gated_layer, OUTPUT_NORM: self._output_norm_layer,
+                 SANDWICH_NORM: self._sandwich_layer}[self.cfg.block]
+        for i, l in enumerate(self.cfg.runs):
             if self.prof is not None:
                 self.prof.mark(i, "layer")
-            x = layer(i, lw, x, b)
+            if i in self.cfg.pass_starts:
+                x = x + embedded
+            x = layer(i, self.w.layers[l], x, b)
             if self.tap is not None:
                 self.tap.write(i, "layer_out", x)
         return x
 
     def logits_from_hidden(self, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
-        norm = self._norm if self.cfg.block == PARALLEL_GATED else self._layer_norm
+        norm = {PARALLEL_GATED: self._norm, OUTPUT_NORM: self._layer_norm, SANDWICH_NORM: self._group_norm}[self.cfg.block]
         logits = norm(x[b.logit_rows[:b.n_logit].long()], self.w.final_norm) @ self.w.lm_head.float().T
         cap = self.cfg.logit_softcap
         return cap * torch.tanh(logits / cap) if cap else logits
@@ -300,9 +368,13 @@ class LayeredWorkspace:
             self.conv_x = torch.zeros(R * n, **act)
             self.dt = torch.zeros(R * n, **f32)
             self.low = torch.zeros(R * max(l.mixer.w_x.shape[0] for l in w.layers if l.mixer.w_x is not None), **act)
+        window = [cfg.layers[i].mixer for i in cfg.window_layers]
+        if window:
+            self.q_rows = torch.zeros(R * max(m.heads * m.maps * m.key_width for m in window), **act)
         if any(l.w_up is not None for l in w.layers):
-            self.ff = torch.zeros(R * max(l.w_up.shape[0] for l in w.layers if l.w_up is not None), **act)
-            self.act = torch.zeros(R, Wp, **act)
+            self.ff = torch.zeros(R * max(l.w_down.shape[1] for l in w.layers if l.w_up is not None), **act)
+            if cfg.block == OUTPUT_NORM:
+                self.act = torch.zeros(R, Wp, **act)
         moes = [(i, l.mlp) for i, l in enumerate(cfg.layers) if isinstance(l.mlp, MoeSpec)]
         self.plans: Dict[tuple, MoePlan] = {}
         self.static_plans: Dict[tuple, MoePlan] = {}
@@ -351,7 +423,7 @@ class LayeredCuda:
         self.max_seq_len = max_seq_len
         self.split_tokens = max(64, pad_to((max_seq_len + attn_splits - 1) // attn_splits, 64))
         self.ws = LayeredWorkspace(weights, max_rows, max_logit_rows, self.device)
-        self.cache_index = {l: i for i, l in enumerate(self.cfg.cache_layers)}
+        self.cache_index = {r: i for i, r in enumerate(self.cfg.cache_runs)}
         # cosines and sines of every rotation in use, computed in double
         self.rotation: Dict[tuple, tuple] = {}
         for i in self.cfg.attention_layers:
@@ -373,7 +445,7 @@ class LayeredCuda:
                 raise ValueError("delta mixers wider than 256 key channels per head are not supported")
             if isinstance(m, MambaMixer) and m.state > 128:
                 raise ValueError("selective scans with more than 128 states per channel are not supported")
-            if isinstance(m, AttentionMixer) and max(m.dim, m.vdim) > 512:
+            if isinstance(m, (AttentionMixer, WindowMixer)) and max(m.dim, m.vdim) > 512:
                 raise ValueError("attention heads wider than 512 are not supported")
             if isinstance(f, MoeSpec) and (f.experts > 256 or f.top > 32 or f.groups > 32):
                 raise ValueError("the router takes at most 256 experts, top 32, 32 groups")
@@ -440,19 +512,34 @@ class LayeredCuda:
                                                first_off=cfg.layers[first].mixer.v_offset)
         KL.gqa_prep(q, proj[:, mx.off["k"]:], proj[:, mx.off["v"]:], m, mx, self.rotation[m.rot_base, m.rot_dims],
                     b.positions[:T], b.write_slot[:T], pool, cfg.norm_eps, **mixed)
+        return self._attend(q, m, pool, b, T)
+
+    def _attend(self, q: torch.Tensor, m, pool: torch.Tensor, b: DeviceBatch, T: int, gate: Optional[torch.Tensor] = None,
+                **form) -> torch.Tensor:
+        """Attention of query rows over a layer's pool: prompt tiles on tcgen05, the other rows in the decode kernels."""
+        KL = self.KL
         out = self._view(self.ws.mix_in, T, m.heads * m.vdim_pad)
         page = self.pool.page_size
-        if not KL.gqa_tc_group(m, q.dtype, page):
-            return KL.gqa_attention(q, m, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], page, out)
         ranges = [(0, T)]
-        if b.n_tc_tiles:
-            KL.gqa_prefill_tc(q, m, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, b.tc_positions, page, out)
+        if b.n_tc_tiles and KL.gqa_tc_group(m, q.dtype, page):
+            KL.gqa_prefill_tc(q, m, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, b.tc_positions, page, out, gate=gate, **form)
             ranges = b.rest_ranges
         for r0, r1 in ranges:
-            splits = KL.gqa_decode_splits(r1 - r0, m, self.max_seq_len)
-            KL.gqa_decode(q[r0:r1], m, pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], page, out[r0:r1],
-                          splits=splits, decode_only=b.decode_only)
+            rows = dict(gate=None if gate is None else gate[r0:r1], **form)
+            at = (q[r0:r1], m, pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], page, out[r0:r1])
+            if KL.gqa_decode_supported(m, q.dtype, page):
+                KL.gqa_decode(*at, splits=KL.gqa_decode_splits(r1 - r0, m, self.max_seq_len), decode_only=b.decode_only, **rows)
+            else:
+                KL.gqa_attention(*at, **rows)
         return out
+
+    def _window(self, run: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        mx, m = lw.mixer, lw.spec.mixer
+        pool = self.pool.layer(self.cache_index[run])
+        q = self._view(self.ws.q_rows, T, m.heads * m.maps * m.key_width)
+        self.KL.head_prep(proj, mx.off, m, mx, b.write_slot[:T], pool, self.cfg.norm_eps, q)
+        gate = proj[:, mx.off["g"]:] if m.gate else None
+        return self._attend(q, m, pool, b, T, slopes=mx.slopes, gate=gate, diff_lambda=mx.diff_lambda, eps=self.cfg.norm_eps)
 
     def _mamba(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         K, KL, ws = self.K, self.KL, self.ws
@@ -472,8 +559,8 @@ class LayeredCuda:
                                  self.states.state[layer], *seqs, out)
 
     def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
-        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, DeltaMixer: self._delta,
-              MambaMixer: self._mamba}[type(lw.spec.mixer)]
+        fn = {LatentMixer: self._latent, AttentionMixer: self._attention, WindowMixer: self._window,
+              DeltaMixer: self._delta, MambaMixer: self._mamba}[type(lw.spec.mixer)]
         return fn(layer, lw, proj, b, T)
 
     # -- feed-forward ------------------------------------------------------------------------
@@ -589,16 +676,53 @@ class LayeredCuda:
                 KL.add_normed(x, ws.mix[:T], lw.norm2, cfg.width, eps, canon=fused(i + 1))
             self._tapped(i, x)
 
+    def _sandwich_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+        runs, starts = cfg.runs, set(cfg.pass_starts)
+        grouped = dict(dim=cfg.width, eps=cfg.norm_eps, groups=cfg.norm_groups)
+        embedding = dict(ids=b.token_ids[:T], table=self.w.embed)
+        layer = lambda r: self.w.layers[runs[r]]
+
+        def close(r: int, norm: torch.Tensor, bias=None) -> None:
+            """End of run r: its last output norm and residual addition, then what the next run starts with."""
+            nxt = layer(r + 1).norm1 if r + 1 < len(runs) else None
+            again = embedding if r + 1 in starts else {}
+            y = ws.mix[:T]
+            if again and self.tap is not None and self.tap.wants(r, "layer_out"):
+                # the tapped stream is the layer's own: the embedding joins it in a launch of its own
+                KL.sandwich_step(x, out_norm=norm, y=y, bias=bias, **grouped)
+                self._tapped(r, x)
+                KL.sandwich_step(x, in_norm=nxt, act=h, **again, **grouped)
+                return
+            KL.sandwich_step(x, out_norm=norm, y=y, bias=bias, in_norm=nxt, act=h if nxt is not None else None, **again, **grouped)
+            self._tapped(r, x)
+
+        KL.sandwich_step(x, in_norm=layer(0).norm1, act=h, fresh=True, **embedding, **grouped)
+        for r in range(len(runs)):
+            lw = layer(r)
+            self._mix(r, lw, h, b, T)
+            if self.prof is not None:
+                self.prof.mark(r, "tail")
+            if lw.spec.mlp is None:
+                close(r, lw.norm1b, lw.mixer.o_bias)
+                continue
+            ff = self._view(ws.ff, T, lw.w_down.shape[1])
+            KL.sandwich_step(x, out_norm=lw.norm1b, y=ws.mix[:T], bias=lw.mixer.o_bias, in_norm=lw.norm2, act=h, **grouped)
+            K.gemm(h, lw.w_up, out=ff, epilogue=K.EPI_GEGLU)
+            K.gemm(ff, lw.w_down, out=ws.mix[:T])
+            close(r, lw.norm2b)
+
     # -- whole model ---------------------------------------------------------------------
     def hidden_states(self, b: DeviceBatch, T: int) -> torch.Tensor:
         """Runs the layers; `ws.x` holds the residual stream.  Returns the rows the head starts from: normalised ones
-        (`ws.h`) behind parallel gated blocks, the stream itself behind output-norm blocks."""
+        (`ws.h`) behind parallel gated blocks, the stream itself behind the other forms."""
         ws = self.ws
         x, h = ws.x[:T], ws.h[:T]
         gated = self.cfg.block == PARALLEL_GATED
-        (self._gated_blocks if gated else self._output_norm_blocks)(b, T, x, h)
+        {PARALLEL_GATED: self._gated_blocks, OUTPUT_NORM: self._output_norm_blocks,
+         SANDWICH_NORM: self._sandwich_blocks}[self.cfg.block](b, T, x, h)
         if self.prof is not None:
-            self.prof.mark(len(self.w.layers), None)
+            self.prof.mark(len(self.cfg.runs), None)
         return h if gated else x
 
     def head(self, h: torch.Tensor, logit_rows: torch.Tensor, L: int):
@@ -607,6 +731,9 @@ class LayeredCuda:
         hn = ws.hn_last[:L]
         if self.cfg.block == OUTPUT_NORM:
             self.KL.norm_rows(h, logit_rows[:L], self.w.final_norm, hn, self.cfg.width, self.cfg.norm_eps)
+        elif self.cfg.block == SANDWICH_NORM:
+            self.KL.sandwich_rows(h, logit_rows[:L], self.w.final_norm, hn, self.cfg.width, self.cfg.norm_eps,
+                                  self.cfg.norm_groups)
         else:
             self.M.gather_rows(h, logit_rows[:L], hn)
         logits = ws.logits[:L]

@@ -6,6 +6,12 @@
   OUTPUT_NORM     the mixer, then the feed-forward, each reading the stream itself; a norm (layer norm with weight and
                   bias) on the sublayer's output before it is added.  With `canon_taps` the mixer reads the stream plus
                   a short causal convolution of it
+  SANDWICH_NORM   the mixer, then the feed-forward, each between two grouped RMS norms: one on its input, one on its
+                  output before that is added to the stream
+
+`loop` runs a range of layers several times in a row with the same weights: `runs` is the sequence of layers a token
+passes, and every run has its own cache plane and state.  The embedding is added to the stream again before every pass
+but the first.
 
 Mixers:
 
@@ -13,15 +19,19 @@ Mixers:
                   per token (the only thing cached), causal softmax, one output gate per head
   AttentionMixer  grouped-query attention inside position-aligned chunks: query and key norm over the whole
                   projection, partial rotation, value norm, values mixed with those of the first mixing layer
+  WindowMixer     grouped-query attention over a sliding window (and kept first tokens) with query and key norm per head:
+                  optionally projection biases, keys that double as values, a distance bias per head, scores mixed
+                  across heads, an output gate, two score maps whose outputs are subtracted
   DeltaMixer      gated delta rule: short causal convolutions, unit-norm queries and keys, one decay per key channel
                   or per head, a [dim, vdim] state per head, gated per-head output norm
   MambaMixer      selective scan: short causal convolution, per-channel step sizes, an [inner, state] diagonal recurrence
 
-Feed-forward: routed experts (softmax scores, group-limited top-k), dense with GELU, or none.
+Feed-forward: routed experts (softmax scores, group-limited top-k), dense with GELU or gated with tanh GELU, or none.
 
 `from_layer_list` reads the `config.json` of the architectures whose checkpoints are stored this way: Gitozen
-(PARALLEL_GATED; latent attention, delta rule with channel decays, experts) and Supisun (OUTPUT_NORM; chunked attention,
-selective scan, delta rule with head decays, dense feed-forward, learned positions).
+(PARALLEL_GATED; latent attention, delta rule with channel decays, experts), Supisun (OUTPUT_NORM; chunked attention,
+selective scan, delta rule with head decays, dense feed-forward, learned positions) and Vedadra (SANDWICH_NORM; window
+attention with mixed heads, differential window attention, gated dense feed-forward, looped layers).
 """
 from __future__ import annotations
 
@@ -64,6 +74,9 @@ class AttentionMixer:
     v_mix: bool = False
 
     kind = "attention"
+    maps = 1
+    window = keep_first = 0
+    shared_keys = False
 
     @property
     def dim_pad(self) -> int:
@@ -81,6 +94,65 @@ class AttentionMixer:
     @property
     def row_dim(self) -> int:
         return pad_to(self.kv_heads * (self.dim_pad + self.vdim_pad), 8)
+
+    @property
+    def key_width(self) -> int:
+        """Width of a query row as the attention kernels take it."""
+        return self.dim_pad
+
+
+@dataclass(frozen=True)
+class WindowMixer:
+    """Position i sees j <= i with i - j < window or j < keep_first.  `maps` = 2: two query / key pairs per head over the
+    same values; the head's output is rms(a1 - lambda a2) * (1 - diff).  `mix_heads`: score_h <- sum_g T[h, g] score_g."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int
+    keep_first: int = 0
+    maps: int = 1
+    diff: float = 0.0              # maps = 2: base of lambda
+    biases: bool = False           # on the query, key and output projections
+    tied_values: bool = False      # the values are the projected keys (before their norm)
+    head_temps: bool = False       # one factor per head on its scores
+    distance_bias: bool = False    # score_h -= 2^(-8 (h + 1) / heads) (i - j)
+    mix_heads: bool = False
+    gate: bool = False             # output multiplied by sigmoid(W_g h), element by element
+
+    chunk = 0
+
+    @property
+    def kind(self) -> str:
+        return "attention" if self.maps == 1 else "attention_2"
+
+    @property
+    def dim_pad(self) -> int:
+        return pad_to(self.dim, 8)
+
+    @property
+    def vdim_pad(self) -> int:
+        return pad_to(self.vdim, 8)
+
+    @property
+    def shared_keys(self) -> bool:
+        """Every query row meets the keys of all kv heads side by side: sum_g T[h, g] q_g . k_kv(g) is one product of a
+        mixed query with the concatenated keys."""
+        return self.mix_heads
+
+    @property
+    def key_width(self) -> int:
+        return (self.kv_heads if self.shared_keys else self.maps) * self.dim_pad
+
+    @property
+    def v_offset(self) -> int:
+        """First value column of a cache row: [kv_heads][maps][dim_pad] keys | [kv_heads][vdim_pad] values."""
+        return self.kv_heads * self.maps * self.dim_pad
+
+    @property
+    def row_dim(self) -> int:
+        return pad_to(self.v_offset + self.kv_heads * self.vdim_pad, 8)
 
 
 @dataclass(frozen=True)
@@ -135,22 +207,32 @@ class MoeSpec:
 
 @dataclass(frozen=True)
 class DenseSpec:
-    """W_down gelu(W_up x), the exact (error-function) GELU."""
+    """W_down gelu(W_up x), the exact (error-function) GELU; gated: W_down (gelu(W_gate x) * W_up x), the tanh form."""
     ff: int
+    gated: bool = False
 
     experts = top = 0
 
 
-Mixer = Union[LatentMixer, AttentionMixer, DeltaMixer, MambaMixer]
+Mixer = Union[LatentMixer, AttentionMixer, WindowMixer, DeltaMixer, MambaMixer]
 
 PARALLEL_GATED = "parallel_gated"
 OUTPUT_NORM = "output_norm"
+SANDWICH_NORM = "sandwich_norm"
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     mixer: Mixer
     mlp: Union[MoeSpec, DenseSpec, None]
+
+
+@dataclass(frozen=True)
+class Loop:
+    """Layers start .. stop - 1 run `times` times in a row."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass(frozen=True)
@@ -167,6 +249,8 @@ class LayeredConfig:
     block: str = PARALLEL_GATED
     canon_taps: int = 0                 # OUTPUT_NORM: taps of the mixers' input convolution, 0: none
     learned_positions: bool = False     # a table of `max_position` vectors is added to the embedding
+    norm_groups: int = 1                # SANDWICH_NORM: parts of a row with an RMS norm of their own
+    loop: Optional[Loop] = None         # SANDWICH_NORM
 
     n_mtp_layers = 0
     attn_sink = False
@@ -185,6 +269,32 @@ class LayeredConfig:
         return pad_to(self.width, 8)
 
     @property
+    def runs(self) -> Tuple[int, ...]:
+        """Layers in the order a token passes them."""
+        n, l = len(self.layers), self.loop
+        if l is None:
+            return tuple(range(n))
+        return (*range(l.start), *(tuple(range(l.start, l.stop)) * l.times), *range(l.stop, n))
+
+    @property
+    def pass_starts(self) -> Tuple[int, ...]:
+        """Runs that begin a pass of the loop other than the first."""
+        l = self.loop
+        return () if l is None else tuple(l.start + k * (l.stop - l.start) for k in range(1, l.times))
+
+    def first_layers(self, n: int) -> "LayeredConfig":
+        """The same model cut off behind its first `n` layers."""
+        l = self.loop
+        if l is not None:
+            l = Loop(l.start, min(l.stop, n), l.times) if l.start < n else None
+        return replace(self, layers=self.layers[:n], loop=l)
+
+    def cycled(self, n: int) -> "LayeredConfig":
+        """A model of `n` layers that repeats this one's."""
+        whole = replace(self, layers=tuple(self.layers[i % len(self.layers)] for i in range(n)))
+        return whole.first_layers(n)
+
+    @property
     def latent_layers(self) -> Tuple[int, ...]:
         return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, LatentMixer))
 
@@ -197,13 +307,23 @@ class LayeredConfig:
         return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, AttentionMixer))
 
     @property
+    def window_layers(self) -> Tuple[int, ...]:
+        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, WindowMixer))
+
+    @property
     def mamba_layers(self) -> Tuple[int, ...]:
         return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, MambaMixer))
 
     @property
     def cache_layers(self) -> Tuple[int, ...]:
         """Layers with a row per token in the paged pool."""
-        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, (LatentMixer, AttentionMixer)))
+        return tuple(i for i, l in enumerate(self.layers) if isinstance(l.mixer, (LatentMixer, AttentionMixer, WindowMixer)))
+
+    @property
+    def cache_runs(self) -> Tuple[int, ...]:
+        """Runs with a plane of their own in the paged pool, in the order of the planes."""
+        cached = set(self.cache_layers)
+        return tuple(r for r, i in enumerate(self.runs) if i in cached)
 
     @property
     def first_value_layer(self) -> int:
@@ -239,6 +359,9 @@ class LayeredConfig:
             x = p + "mix."
             if gated:
                 out[p + "norm1"] = ()
+            elif self.block == SANDWICH_NORM:
+                names = ("norm1", "norm2", "norm1b", "norm2b") if l.mlp else ("norm1", "norm1b")
+                out.update({p + n: (W,) for n in names})
             else:
                 for n in ("norm1", "norm2")[:2 if l.mlp else 1]:
                     out.update({p + n: (W,), p + n + ".b": (W,)})
@@ -252,6 +375,24 @@ class LayeredConfig:
                 if m.v_mix:
                     out[x + "vmix"] = ()
                 out[x + "o"] = (W, m.heads * m.vdim)
+            elif isinstance(m, WindowMixer):
+                nq, nk, nv = m.heads * m.maps * m.dim, m.kv_heads * m.maps * m.dim, m.kv_heads * m.vdim
+                for name, n in (("q", nq), ("k", nk)) + (() if m.tied_values else (("v", nv),)):
+                    out[x + name] = (n, W)
+                    if m.biases and name != "v":
+                        out[x + name + ".b"] = (n,)
+                out.update({x + "q.norm": (m.dim,), x + "k.norm": (m.dim,)})
+                if m.maps == 2:
+                    out.update({x + n: (m.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
+                if m.mix_heads:
+                    out[x + "talk"] = (m.heads, m.heads)
+                if m.head_temps:
+                    out[x + "temp"] = (m.heads,)
+                if m.gate:
+                    out[x + "g"] = (m.heads * m.vdim, W)
+                out[x + "o"] = (W, m.heads * m.vdim)
+                if m.biases:
+                    out[x + "o.b"] = (W,)
             elif isinstance(m, MambaMixer):
                 out.update({x + "in": (2 * m.inner, W), x + "conv": (m.inner, m.taps), x + "conv.b": (m.inner,),
                             x + "x": (m.dt_rank + 2 * m.state, m.inner), x + "dt": (m.inner, m.dt_rank),
@@ -275,6 +416,8 @@ class LayeredConfig:
                     out.update({q + "gate": (l.mlp.ff, W), q + "up": (l.mlp.ff, W), q + "down": (W, l.mlp.ff)})
                 out[p + "mlp.router"] = (l.mlp.experts, W)
             elif l.mlp:
+                if l.mlp.gated:
+                    out[p + "mlp.gate"] = (l.mlp.ff, W)
                 out.update({p + "mlp.up": (l.mlp.ff, W), p + "mlp.down": (W, l.mlp.ff)})
             if gated:
                 out.update({p + "rg1": (W, W), p + "rg1.b": (W,)})
@@ -284,6 +427,8 @@ class LayeredConfig:
                 out[p + "canon1"] = (W, self.canon_taps)
         if gated:
             out["final.norm"] = ()
+        elif self.block == SANDWICH_NORM:
+            out["final.norm"] = (W,)
         else:
             out.update({"final.norm": (W,), "final.norm.b": (W,)})
         out["head"] = (self.vocab_size, W)
@@ -332,6 +477,19 @@ def _attention(m: dict) -> AttentionMixer:
     return x
 
 
+def _window(m: dict, **form) -> WindowMixer:
+    mask = m["mask"]
+    x = WindowMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), int(mask["size"]),
+                    int(mask.get("keep_first") or 0), diff=float(m.get("diff") or 0.0), **form)
+    _positive(heads=x.heads, kv_heads=x.kv_heads, dim=x.dim, vdim=x.vdim, window=x.window)
+    _grouped(x.heads, x.kv_heads)
+    if x.keep_first < 0:
+        raise ValueError("mask.keep_first must not be negative")
+    if x.tied_values and x.dim != x.vdim:
+        raise ValueError("values that are the keys have the keys' width")
+    return x
+
+
 def _mamba(m: dict) -> MambaMixer:
     x = MambaMixer(int(m["inner"]), int(m["state"]), int(m["dt_rank"]), int(m["conv"]))
     _positive(inner=x.inner, state=x.state, dt_rank=x.dt_rank, conv=x.taps)
@@ -347,26 +505,24 @@ def _delta(m: dict, **form) -> DeltaMixer:
 
 HEAD_DELTA = dict(decay_rank=0, gate_rank=0, head_decay=True, gate="silu")
 
-MIXERS: Dict[str, Callable[[dict], Mixer]] = {
-    "latent_attention": _latent,
-    "channel_delta": _delta,
-    "attention": _attention,
-    "mamba1": _mamba,
-    "delta": lambda m: _delta(m, **HEAD_DELTA),
-}
+TALKING_WINDOW = dict(biases=True, tied_values=True, head_temps=True, distance_bias=True, mix_heads=True, gate=True)
 
 
 @dataclass(frozen=True)
 class Design:
-    """What an architecture's name fixes: its block form, and the mixers and feed-forwards its layers may name."""
+    """What an architecture's name fixes: its block form, the mixers its layers may name (type -> reader) and its
+    feed-forward."""
     name: str
     block: str
-    mixers: Tuple[str, ...]
+    mixers: Dict[str, Callable[[dict], Mixer]]
     feed_forward: str
 
 
-DESIGNS = {d.name: d for d in (Design("Gitozen", PARALLEL_GATED, ("latent_attention", "channel_delta"), "moe"),
-                               Design("Supisun", OUTPUT_NORM, ("attention", "mamba1", "delta"), "dense"))}
+DESIGNS = {d.name: d for d in (
+    Design("Gitozen", PARALLEL_GATED, {"latent_attention": _latent, "channel_delta": _delta}, "moe"),
+    Design("Supisun", OUTPUT_NORM, {"attention": _attention, "mamba1": _mamba, "delta": lambda m: _delta(m, **HEAD_DELTA)}, "dense"),
+    Design("Vedadra", SANDWICH_NORM, {"attention": lambda m: _window(m, **TALKING_WINDOW),
+                                      "attention_2": lambda m: _window(m, maps=2)}, "gated_dense"))}
 
 ARCHITECTURES = tuple(n.lower() for n in DESIGNS)       # registry names of the layer-list architectures
 
@@ -374,10 +530,11 @@ ARCHITECTURES = tuple(n.lower() for n in DESIGNS)       # registry names of the 
 def _mlp(m: Optional[dict], kind: str):
     if m is None:
         return None
-    if m.get("kind", kind) != kind:
+    stored = "dense" if kind == "gated_dense" else kind
+    if m.get("kind", stored) != stored:
         raise ValueError(f"unknown feed-forward kind {m.get('kind')!r}")
-    if kind == "dense":
-        d = DenseSpec(int(m["ff"]))
+    if stored == "dense":
+        d = DenseSpec(int(m["ff"]), kind == "gated_dense")
         _positive(ff=d.ff)
         return d
     r = m["router"]
@@ -386,6 +543,16 @@ def _mlp(m: Optional[dict], kind: str):
     _positive(experts=x.experts, top=x.top, ff=x.ff, groups=x.groups, keep=x.keep)
     if x.experts % x.groups or x.keep > x.groups or x.top > x.experts // x.groups * x.keep:
         raise ValueError("router groups do not fit the expert count")
+    return x
+
+
+def _loop(c: dict, n_layers: int) -> Optional[Loop]:
+    l = c.get("loop")
+    if not l:
+        return None
+    x = Loop(int(l["start"]), int(l["stop"]), int(l["times"]))
+    if not 0 <= x.start < x.stop <= n_layers or x.times < 1:
+        raise ValueError(f"loop {l} does not fit {n_layers} layers")
     return x
 
 
@@ -405,7 +572,7 @@ def from_layer_list(source) -> LayeredConfig:
     for l in c["layers"]:
         if l["type"] not in d.mixers:
             raise ValueError(f"unknown mixer type {l['type']!r}")
-        layers.append(LayerSpec(MIXERS[l["type"]](l["mixer"]), _mlp(l.get("mlp"), d.feed_forward)))
+        layers.append(LayerSpec(d.mixers[l["type"]](l["mixer"]), _mlp(l.get("mlp"), d.feed_forward)))
     if not layers:
         raise ValueError("a model needs at least one layer")
     cfg = LayeredConfig(int(c["vocab"]), int(c["width"]), tuple(layers), float(c["norm"]["eps"]),
@@ -413,6 +580,13 @@ def from_layer_list(source) -> LayeredConfig:
     if d.block == OUTPUT_NORM:
         cfg = cfg.with_(max_position=int(c["max_positions"]), learned_positions=True, canon_taps=int(c["canon"]["taps"]))
         _positive(max_positions=cfg.max_position, taps=cfg.canon_taps)
+    if d.block == SANDWICH_NORM:
+        cfg = cfg.with_(norm_groups=int(c["norm"].get("groups") or 1), loop=_loop(c, len(layers)))
+        _positive(groups=cfg.norm_groups)
+        if cfg.width % cfg.norm_groups:
+            raise ValueError("norm.groups must divide the width")
+    elif c.get("loop"):
+        raise ValueError(f"{arch} layers do not loop")
     _positive(vocab=cfg.vocab_size, width=cfg.width)
     shapes = {(m.kv_heads, m.vdim) for m in (layers[i].mixer for i in cfg.attention_layers) if m.v_mix}
     if len(shapes) > 1:
@@ -430,6 +604,11 @@ def to_layer_list(cfg: LayeredConfig) -> dict:
         elif isinstance(m, AttentionMixer):
             mx = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
                   "mask": {"size": m.chunk}, "rot": {"base": m.rot_base, "dims": m.rot_dims}, "v_mix": m.v_mix}
+        elif isinstance(m, WindowMixer):
+            mx = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                  "mask": {"size": m.window, **({"keep_first": m.keep_first} if m.keep_first else {})}}
+            if m.maps == 2:
+                mx["diff"] = m.diff
         elif isinstance(m, MambaMixer):
             mx = {"inner": m.inner, "state": m.state, "dt_rank": m.dt_rank, "conv": m.taps}
         else:
@@ -445,6 +624,9 @@ def to_layer_list(cfg: LayeredConfig) -> dict:
     out = {"vocab": cfg.vocab_size, "width": cfg.width, "norm": {"eps": cfg.norm_eps}, "layers": layers}
     if cfg.block == OUTPUT_NORM:
         return {"architecture": "Supisun", **out, "max_positions": cfg.max_position, "canon": {"taps": cfg.canon_taps}}
+    if cfg.block == SANDWICH_NORM:
+        out["norm"] = {"eps": cfg.norm_eps, "groups": cfg.norm_groups}
+        return {"architecture": "Vedadra", **out, "loop": asdict(cfg.loop) if cfg.loop else None}
     return {"architecture": "Gitozen", **out, "logit_softcap": cfg.logit_softcap or None}
 
 
@@ -510,6 +692,56 @@ def tiny_supisun() -> LayeredConfig:
     return _supisun(512, 96, (LayerSpec(att, ff), LayerSpec(mam, ff), LayerSpec(dlt, None), LayerSpec(att, ff)), 4096, taps=3)
 
 
+def _supisun_attention_stack(name: str, width: int, heads: int, kv_heads: int, dim: int, ff: int, n_layers: int) -> LayeredConfig:
+    """Chunked attention in every layer and no input convolution: the stack closest to the vedadra-* presets."""
+    att = AttentionMixer(heads, kv_heads, dim, dim, dim ** -0.5, 8192, 500000.0, dim, False)
+    return _supisun(102400, width, (LayerSpec(att, DenseSpec(ff)) for _ in range(n_layers)), 32768, taps=1, name=name)
+
+
+def supisun_attention_small(n_layers: int = 24) -> LayeredConfig:
+    return _supisun_attention_stack("supisun-attention-small", 1024, 8, 4, 128, 4608, n_layers)
+
+
+def supisun_attention_lite(n_layers: int = 27) -> LayeredConfig:
+    return _supisun_attention_stack("supisun-attention-lite", 2048, 16, 4, 128, 9216, n_layers)
+
+
+def supisun_attention_wide(n_layers: int = 32) -> LayeredConfig:
+    return _supisun_attention_stack("supisun-attention-wide", 4096, 32, 4, 128, 18432, n_layers)
+
+
+def tiny_vedadra() -> LayeredConfig:
+    """Small shape for fixtures and the command line: both mixers, grouped heads, a layer without feed-forward, a loop."""
+    att = WindowMixer(heads=6, kv_heads=2, dim=24, vdim=24, scale=0.2, window=20, **TALKING_WINDOW)
+    dif = WindowMixer(heads=4, kv_heads=2, dim=16, vdim=40, scale=0.25, window=36, keep_first=3, maps=2, diff=0.6)
+    ff = DenseSpec(160, True)
+    return LayeredConfig(512, 96, (LayerSpec(dif, ff), LayerSpec(att, ff), LayerSpec(dif, None), LayerSpec(att, ff)), 1e-6,
+                         name="vedadra", block=SANDWICH_NORM, norm_groups=3, loop=Loop(1, 3, 2))
+
+
+def _vedadra_stack(name: str, width: int, heads: int, kv_heads: int, dim: int, ff: int, n_layers: int) -> LayeredConfig:
+    """Layers of a served model's size, `n_layers` runs of which three are a second pass: every third mixer differential,
+    its maps of the other heads' width and half as many heads with values twice as wide."""
+    att = WindowMixer(heads, kv_heads, dim, dim, dim ** -0.5, 1024, **TALKING_WINDOW)
+    dif = WindowMixer(heads // 2, kv_heads, dim, 2 * dim, dim ** -0.5, 4096, keep_first=4, maps=2, diff=0.5)
+    n = n_layers - 3
+    return LayeredConfig(102400, width, tuple(LayerSpec(dif if i % 3 == 2 else att, DenseSpec(ff, True)) for i in range(n)), 1e-6,
+                         name=name, block=SANDWICH_NORM, norm_groups=4, loop=Loop(n // 3, n // 3 + 3, 2))
+
+
+def vedadra_small(n_layers: int = 24) -> LayeredConfig:
+    return _vedadra_stack("vedadra-small", 1024, 8, 4, 128, 3072, n_layers)
+
+
+def vedadra_lite(n_layers: int = 27) -> LayeredConfig:
+    """The widths of DeepSeek-V2-Lite (and of supisun-attention-lite)."""
+    return _vedadra_stack("vedadra-lite", 2048, 16, 4, 128, 6144, n_layers)
+
+
+def vedadra_wide(n_layers: int = 32) -> LayeredConfig:
+    return _vedadra_stack("vedadra-wide", 4096, 32, 4, 128, 12288, n_layers)
+
+
 def _supisun_stack(name: str, width: int, heads: int, kv_heads: int, dim: int, ff: int, n_layers: int) -> LayeredConfig:
     """Layers of a served model's size: out of eight, three attention, three selective-scan and two delta mixers."""
     att = AttentionMixer(heads, kv_heads, dim, dim, dim ** -0.5, 8192, 500000.0, dim, True)
@@ -536,4 +768,12 @@ PRESETS = {"tiny-gitozen": tiny_gitozen, "gitozen-lite": gitozen_lite, "gitozen-
            "gitozen-dense-small": gitozen_dense_small, "gitozen-dense-lite": gitozen_dense_lite,
            "gitozen-dense-wide": gitozen_dense_wide,
            "tiny-supisun": tiny_supisun, "supisun-small": supisun_small, "supisun-lite": supisun_lite,
-           "supisun-wide": supisun_wide}
+           "supisun-wide": supisun_wide, "supisun-attention-small": supisun_attention_small,
+           "supisun-attention-lite": supisun_attention_lite, "supisun-attention-wide": supisun_attention_wide,
+           "tiny-vedadra": tiny_vedadra, "vedadra-small": vedadra_small, "vedadra-lite": vedadra_lite,
+           "vedadra-wide": vedadra_wide}
+
+
+def preset_architecture(preset: str) -> str:
+    """Registry name of the architecture a preset belongs to."""
+    return next(a for a in ARCHITECTURES if a in preset)

@@ -43,15 +43,16 @@ class LayeredRunner(DeepSeekRunner):
     # ------------------------------------------------------------------ parts
     def _make_pool(self, n_pages: int) -> KvPool:
         return KvPool(self.cfg, n_pages, self.page_size, self.device, dtype=self.w.embed.dtype,
-                      n_layers=len(self.cfg.cache_layers))
+                      n_layers=len(self.cfg.cache_runs))
 
     def _prefill_tc_heads(self) -> int:
         from ..ops.kernels import prefill_tc_supported
-        if self.cfg.attention_layers:
+        grouped = self.cfg.attention_layers + self.cfg.window_layers
+        if grouped:
             # one tile table for all layers: as many positions as the widest group of query heads leaves room for
             from ..ops.layered import gqa_tc_group
             return max(gqa_tc_group(self.cfg.layers[i].mixer, self.w.embed.dtype, self.page_size)
-                       for i in self.cfg.attention_layers)
+                       for i in grouped)
         heads = {self.cfg.layers[i].mixer.heads for i in self.cfg.latent_layers}
         if len(heads) != 1 or self.w.embed.dtype != torch.bfloat16:
             return 0

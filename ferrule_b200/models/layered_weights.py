@@ -5,6 +5,7 @@ blocks begin at multiples of 8 columns of its output:
 
   latent layer     q (heads x dim, each head padded to 8) | dkv | head gates
   attention layer  q | k | v, each head padded to 8
+  window layer     q | k | v (unless the keys are the values) | output gate, each head padded to 8
   delta layer      q | k | v | decay low rank | gate low rank | beta      (full projections: decay | gate | beta)
   mamba layer      x | z
 
@@ -19,13 +20,14 @@ Constants that enter norms, gates and recurrences are fp32 tensors; everything e
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Callable, Dict, List, Optional
 
 import torch
 
-from .layered_config import (PARALLEL_GATED, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, LayeredConfig, LayerSpec,
-                             MambaMixer, MoeSpec, pad_to)
+from .layered_config import (PARALLEL_GATED, SANDWICH_NORM, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, LayeredConfig,
+                             LayerSpec, MambaMixer, MoeSpec, WindowMixer, pad_to)
 
 GetTensor = Callable[[str], torch.Tensor]
 
@@ -59,6 +61,13 @@ class MixerImage:
     q_norm: Optional[torch.Tensor] = None    # fp32 [heads * dim_pad]
     k_norm: Optional[torch.Tensor] = None    # fp32 [kv_heads * dim_pad]
     v_mix: float = 0.0                       # share of the first mixing layer's values
+    # window attention (q_norm, k_norm: [dim_pad], shared by the heads)
+    q_bias: Optional[torch.Tensor] = None    # fp32 [heads * maps * dim_pad]
+    k_bias: Optional[torch.Tensor] = None    # fp32 [kv_heads * maps * dim_pad]
+    o_bias: Optional[torch.Tensor] = None    # fp32 [width_pad]
+    q_mix: Optional[torch.Tensor] = None     # fp32 [heads, heads]: factor of head g's raw scores in head h's; not mixed: [heads]
+    slopes: Optional[torch.Tensor] = None    # fp32 [heads]: taken off a score per token of distance
+    diff_lambda: float = 0.0                 # weight of the second map's output
     # mamba (also conv, dt_bias)
     w_x: Optional[torch.Tensor] = None       # [dt | B | C rows, inner_pad], blocks at off_b / off_c
     off_b: int = 0
@@ -84,7 +93,10 @@ class LayerImage:
     norm1: Optional[torch.Tensor] = None     # fp32 [2, width_pad]
     norm2: Optional[torch.Tensor] = None     # fp32 [2, width_pad]
     canon: Optional[torch.Tensor] = None     # fp32 [taps, width_pad]
-    w_up: Optional[torch.Tensor] = None      # [ff_pad, width_pad]
+    # sandwich block: norm weights of the sublayers' inputs (norm1, norm2 [width_pad]) and outputs
+    norm1b: Optional[torch.Tensor] = None    # fp32 [width_pad]
+    norm2b: Optional[torch.Tensor] = None    # fp32 [width_pad]
+    w_up: Optional[torch.Tensor] = None      # [ff_pad, width_pad]; gated: [gate ff_pad | up ff_pad, width_pad]
     w_down: Optional[torch.Tensor] = None    # [width_pad, ff_pad]
 
 
@@ -93,7 +105,7 @@ class LayeredWeights:
     cfg: LayeredConfig
     embed: torch.Tensor                      # [vocab, width_pad]
     layers: List[LayerImage]
-    final_norm: torch.Tensor                 # fp32 [1], output-norm blocks: [2, width_pad]
+    final_norm: torch.Tensor                 # fp32 [1], output-norm blocks: [2, width_pad], sandwich blocks: [width_pad]
     lm_head: torch.Tensor                    # [vocab, width_pad]
     pos: Optional[torch.Tensor] = None       # [max_position, width_pad] learned position vectors
     mtp: list = field(default_factory=list)  # the architecture has no proposal stages
@@ -149,6 +161,39 @@ def _pack_attention(m: AttentionMixer, p: str, get: GetTensor, cfg: LayeredConfi
                       k_norm=norm("k.norm", m.kv_heads), v_mix=float(get(p + "vmix").float()) if m.v_mix else 0.0)
 
 
+def _pack_window(m: WindowMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
+    Wp, dp, vp = cfg.width_pad, m.dim_pad, m.vdim_pad
+    nq, nk = m.heads * m.maps, m.kv_heads * m.maps
+    blocks = [("q", nq, m.dim, dp), ("k", nk, m.dim, dp)]
+    if not m.tied_values:
+        blocks.append(("v", m.kv_heads, m.vdim, vp))
+    if m.gate:
+        blocks.append(("g", m.heads, m.vdim, vp))
+    for name, heads, d, pad in blocks:
+        b.add(name, _pad(get(p + name).view(heads, d, cfg.width), heads, pad, Wp).reshape(heads * pad, Wp))
+    o = _pad(get(p + "o").view(cfg.width, m.heads, m.vdim), Wp, m.heads, vp)
+    bias = lambda name, heads: _pad(get(p + name).float().view(heads, m.dim), heads, dp).reshape(-1).contiguous()
+    norm = lambda name: _pad(get(p + name).float(), dp).contiguous()
+    f64 = lambda name: get(p + name).double()
+    img = MixerImage(None, b.off, o.reshape(Wp, m.heads * vp).contiguous(), q_norm=norm("q.norm"), k_norm=norm("k.norm"))
+    if m.biases:
+        img.q_bias, img.k_bias = bias("q.b", nq), bias("k.b", nk)
+        img.o_bias = _pad(get(p + "o.b").float(), Wp).contiguous()
+    # score_h = sum_g T[h, g] (scale temp_g q_g . k - slope_g distance): everything but q and k is constant
+    scale = torch.full((m.heads,), m.scale, dtype=torch.float64, device=o.device)
+    if m.head_temps:
+        scale = scale * f64("temp")
+    mix = f64("talk") if m.mix_heads else None
+    img.q_mix = (scale if mix is None else mix * scale).float().contiguous()
+    if m.distance_bias:
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / m.heads) for h in range(m.heads)], dtype=torch.float64, device=o.device)
+        img.slopes = (slopes if mix is None else mix @ slopes).float().contiguous()
+    if m.maps == 2:
+        dot = lambda a, c: math.exp(float((f64(a) * f64(c)).sum()))
+        img.diff_lambda = dot("lq1", "lk1") - dot("lq2", "lk2") + m.diff
+    return img
+
+
 def _pack_mamba(m: MambaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
     Ip, LOG2E = m.inner_pad, 1.4426950408889634
     w_in = get(p + "in")
@@ -185,12 +230,14 @@ def _pack_delta(m: DeltaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _B
                       o_norm=get(p + "norm").float().contiguous())
 
 
-_PACK = {LatentMixer: _pack_latent, AttentionMixer: _pack_attention, DeltaMixer: _pack_delta, MambaMixer: _pack_mamba}
+_PACK = {LatentMixer: _pack_latent, AttentionMixer: _pack_attention, WindowMixer: _pack_window, DeltaMixer: _pack_delta,
+         MambaMixer: _pack_mamba}
 
 
 def _pack_dense(s: DenseSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: LayerImage) -> None:
     Wp, fp = cfg.width_pad, pad_to(s.ff, 8)
-    img.w_up = _pad(get(p + "up"), fp, Wp).contiguous()
+    up = _pad(get(p + "up"), fp, Wp)
+    img.w_up = (torch.cat([_pad(get(p + "gate"), fp, Wp), up]) if s.gated else up).contiguous()
     img.w_down = _pad(get(p + "down"), Wp, fp).contiguous()
 
 
@@ -210,8 +257,9 @@ def _pack_moe(s: MoeSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: Layer
 def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
     """`get(name)` returns a checkpoint tensor in the dtype and on the device the model runs with."""
     Wp = cfg.width_pad
-    gated = cfg.block == PARALLEL_GATED
-    norm = lambda name: torch.stack([_pad(get(n).float(), Wp) for n in (name, name + ".b")]).contiguous()
+    gated, sandwich = cfg.block == PARALLEL_GATED, cfg.block == SANDWICH_NORM
+    vec = lambda name: _pad(get(name).float(), Wp).contiguous()
+    norm = lambda name: vec(name) if sandwich else torch.stack([vec(n) for n in (name, name + ".b")]).contiguous()
     layers: List[LayerImage] = []
     for i, spec in enumerate(cfg.layers):
         p = f"l{i}."
@@ -224,6 +272,8 @@ def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
             b.add("rg1", get(p + "rg1"))
         else:
             img.norm1 = norm(p + "norm1")
+        if sandwich:
+            img.norm1b = norm(p + "norm1b")
         if cfg.canon_taps:
             img.canon = _pad(get(p + "canon1").float().view(cfg.width, cfg.canon_taps).t(), cfg.canon_taps, Wp).contiguous()
         if spec.mlp is not None:
@@ -232,6 +282,8 @@ def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
                 img.rg2_b = _pad(get(p + "rg2.b").float(), Wp).contiguous()
             else:
                 img.norm2 = norm(p + "norm2")
+            if sandwich:
+                img.norm2b = norm(p + "norm2b")
             (_pack_moe if isinstance(spec.mlp, MoeSpec) else _pack_dense)(spec.mlp, p + "mlp.", get, cfg, img)
         mx.w_in = b.matrix()
         layers.append(img)
@@ -277,8 +329,14 @@ class RandomTensors:
             t[..., -1] += 0.7
         elif name.endswith("canon1"):
             t = normal(0.0, 0.3)
-        elif name.endswith(("norm1.b", "norm2.b", "final.norm.b", ".conv.b")):
+        elif name.endswith(("norm1.b", "norm2.b", "final.norm.b", ".conv.b", ".q.b", ".k.b", ".o.b")):
             t = normal(0.0, 0.2)
+        elif name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+            t = normal(0.0, 0.1)
+        elif name.endswith(".talk"):
+            t = normal(0.0, 0.3) + torch.eye(shape[0], device=self.device)
+        elif name.endswith(".temp"):
+            t = normal(1.0, 0.3)
         elif name.endswith((".vmix", ".D")):
             t = normal(0.5, 0.2)
         elif name.endswith(("rg1.b", "rg2.b")):

@@ -1,7 +1,7 @@
 """Recurrent-state pool: what a sequence carries from token to token beside its paged cache.
 
-Three kinds of plane: per recurrent layer the fp32 state (a matrix per head of a delta mixer, [inner, state] of a selective
-scan) and the last inputs of the short convolutions, and per layer with an input convolution the last rows of the
+Three kinds of plane: per run of a recurrent layer the fp32 state (a matrix per head of a delta mixer, [inner, state] of a selective
+scan) and the last inputs of the short convolutions, and per run of a layer with an input convolution the last rows of the
 32-bit residual stream it read.  A plane is indexed by slot (the engine's logical sequence slot) and buffer: every slot has `buffers`
 copies and one of them is committed.  A step reads the committed copy and writes the next one, and only the commit of its
 transaction makes that one current - a step that fails or is rolled back leaves nothing to undo.  With decode
@@ -29,8 +29,8 @@ class RecurrentStatePool:
         self.tail: Dict[int, torch.Tensor] = {}
         self.canon: Dict[int, torch.Tensor] = {}
         plane = lambda *shape, dt=torch.float32: torch.zeros(self.n_states, *shape, dtype=dt, device=device)
-        for i, l in enumerate(cfg.layers):
-            m = l.mixer
+        for i, layer in enumerate(cfg.runs):
+            m = cfg.layers[layer].mixer
             if isinstance(m, DeltaMixer):
                 self.state[i] = plane(m.heads, m.dim, m.vdim)
                 self.tail[i] = plane(max(m.taps - 1, 1), m.channels, dt=dtype)

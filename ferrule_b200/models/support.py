@@ -18,13 +18,14 @@ from enum import Enum
 from typing import List, Optional, Tuple
 
 from .config import SCORE_SIGMOID, SCORE_SOFTMAX, ModelConfig
-from .layered_config import PARALLEL_GATED, LayeredConfig, MoeSpec
+from .layered_config import OUTPUT_NORM, PARALLEL_GATED, SANDWICH_NORM, LayeredConfig, MoeSpec
 
 
 class AttentionKind(Enum):
     MLA = "mla"                       # latent KV, weight-absorbed (DeepSeek-V2 / V3)
     HYBRID_SPARSE_MLA = "hybrid_mla"  # single latent head + window + compressed selection (DeepSeek-V4)
     LATENT_DELTA = "latent_delta"     # per layer: latent attention without positions, or gated delta rule (Gitozen)
+    WINDOW_MIXED = "window_mixed"     # per layer: window attention with scores mixed across heads, or differential
     CHUNKED_RECURRENT = "chunked_recurrent"   # per layer: chunked grouped-query attention, selective scan or delta rule
 
 
@@ -129,7 +130,7 @@ class PolicySet:
     speculation: SpeculationPolicy
     tokenizer: TokenizerPolicy
     validation: ValidationPolicy
-    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4" | "gitozen" | "supisun"
+    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4" | "gitozen" | "supisun" | "vedadra"
 
     @staticmethod
     def from_config(cfg, weight_format: str = "bf16", parallelism: Optional[ParallelismPlan] = None,
@@ -138,16 +139,18 @@ class PolicySet:
         par = parallelism or ParallelismPlan()
         if isinstance(cfg, LayeredConfig):
             moes = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeSpec)]
-            gated = cfg.block == PARALLEL_GATED
+            kind, sem = {PARALLEL_GATED: (AttentionKind.LATENT_DELTA, "gitozen"),
+                         OUTPUT_NORM: (AttentionKind.CHUNKED_RECURRENT, "supisun"),
+                         SANDWICH_NORM: (AttentionKind.WINDOW_MIXED, "vedadra")}[cfg.block]
             groups = max(((m.groups, m.keep) for m in moes), default=(1, 1))
-            att = AttentionPolicy(AttentionKind.LATENT_DELTA if gated else AttentionKind.CHUNKED_RECURRENT, cfg.kv_row_dim, cfg.n_heads, False)
+            att = AttentionPolicy(kind, cfg.kv_row_dim, cfg.n_heads, False)
             router = RouterPolicy(RouterKind.NONE if not moes else (RouterKind.SOFTMAX_GROUP_TOPK if groups[0] > 1
                                                                     else RouterKind.SOFTMAX_TOPK), cfg.topk, groups)
             expert = ExpertPolicy(cfg.n_routed_experts, 0, cfg.n_layers - len(moes))
-            planes = ((("latent_kv",) if cfg.latent_layers else ()) + (("kv",) if cfg.attention_layers else ())
+            planes = ((("latent_kv",) if cfg.latent_layers else ()) + (("kv",) if cfg.attention_layers or cfg.window_layers else ())
                       + (("recurrent_state",) if cfg.delta_layers or cfg.mamba_layers else ())
                       + (("input_convolution",) if cfg.canon_taps else ()))
-            spec, sem = SpeculationPolicy(SpeculationMode.NONE, 0), "gitozen" if gated else "supisun"
+            spec = SpeculationPolicy(SpeculationMode.NONE, 0)
         elif not isinstance(cfg, ModelConfig):         # models.v4_model.V4Config
             att = AttentionPolicy(AttentionKind.HYBRID_SPARSE_MLA, cfg.head_dim, cfg.n_heads, True)
             router = RouterPolicy(RouterKind.HASH if cfg.n_hash_layers >= cfg.n_layers else RouterKind.SQRT_SOFTPLUS_TOPK,
@@ -229,7 +232,7 @@ class EnginePlan:
                                              "dequantised at load time)"))
             if par.tensor_parallel > 1 or par.pipeline_parallel > 1:
                 missing.append(MissingPolicy("parallelism", "the V4 runner is single-GPU"))
-        if p.semantics in ("gitozen", "supisun"):
+        if p.semantics in ("gitozen", "supisun", "vedadra"):
             if p.quant.weight_format != "bf16":
                 missing.append(MissingPolicy("quantization", "layer-list models run bf16 (or fp32) weights"))
             if par.tensor_parallel > 1 or par.pipeline_parallel > 1 or par.expert_parallel > 1:
