@@ -40,6 +40,8 @@ CUDA_SOURCES = [
     "selective_scan.cu",
     "gqa_attention.cu",
     "gqa_decode.cu",
+    "gqa_decode_wide.cu",
+    "head_prep.cu",
     "gqa_prefill_tc.cu",
     "gemm_f32.cu",
     "ep_moe.cu",
@@ -53,7 +55,7 @@ CUDA_SOURCES = [
 COMPONENTS = {
     "layered": ["gemm_tcgen05.cu", "mla_attention.cu", "mla_prefill_tc.cu", "elementwise.cu", "data_movers.cu",
                 "layered_ops.cu", "delta_rule.cu", "gemm_f32.cu", "stream_ops.cu", "selective_scan.cu", "gqa_attention.cu",
-                "gqa_decode.cu", "gqa_prefill_tc.cu"],
+                "gqa_decode.cu", "gqa_decode_wide.cu", "gqa_prefill_tc.cu", "head_prep.cu"],
 }
 CXX_SOURCES = [
     "host/kv_page_manager.cpp",

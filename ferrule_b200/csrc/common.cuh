@@ -365,6 +365,13 @@ __device__ __forceinline__ float gelu_bf16_f(float x) {
   const float h = 0.5f * q * t * __expf(-z * z);
   return x > 0.f ? fmaf(-x, h, x) : x * h;
 }
+// The tanh form, 0.5 x (1 + tanh(u)) with u = sqrt(2 / pi) (x + 0.044715 x^3), as x / (1 + exp(-2 u)).
+__device__ __forceinline__ float gelu_tanh_f(float x) {
+  return x / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * x * x, x, x)));
+}
+__device__ __forceinline__ float gelu_tanh_bf16_f(float x) {
+  return __fdividef(x, 1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * x * x, x, x)));
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -42,7 +42,8 @@ typedef struct FbGemmArgs {
   int w_rows_per_group;
   int x_rows;
   int ntok;                 // rows per tile: 16, 32, 64, 128 or 256
-  int epilogue;             // 0 store, 1 swiglu (dual weights), 2 scatter, 3 all-reduce, 4 store gelu(x)
+  int epilogue;             // 0 store, 1 swiglu (dual weights), 2 scatter, 3 all-reduce, 4 store gelu(x),
+                            // 5 gelu(gate) * up, tanh form (dual weights)
   int dual_offset;          // row of the "up" block inside a group (epilogue 1)
   int out_fp32;
   int max_tok_tiles;        // capacity of the tile table (grouped mode)
@@ -260,6 +261,30 @@ typedef struct FbStreamArgs {
   void* status;
 } FbStreamArgs;
 int fb_stream_step(const FbStreamArgs* args, void* stream);
+// rows between the sublayers of a sandwich block, every norm an RMS norm of `groups` equal parts of the row:
+// x (0 when `fresh`) += out_w * norm(y + y_bias) + table[ids]; act = in_w * norm(x)
+typedef struct FbSandwichArgs {
+  float* x;                 // [rows, ldx]
+  long long ldx;
+  const void* y;            // optional [rows, ldy] sublayer output
+  long long ldy;
+  const float* y_bias;      // optional [dim_pad]
+  const float* out_w;       // [dim_pad]
+  const int* ids;           // optional: add table[ids]
+  const void* table;
+  long long ldt;
+  int vocab, fresh;
+  const float* in_w;        // optional [dim_pad]
+  void* act;                // [rows, lda]
+  long long lda;
+  int rows, dim, dim_pad, groups, fp32;
+  float eps;
+  void* status;
+} FbSandwichArgs;
+int fb_sandwich_step(const FbSandwichArgs* args, void* stream);
+// out[i] = w * norm(x[rows_idx[i]]) as activations, the same norm
+int fb_sandwich_rows(const float* x, long long ldx, int x_rows, const int* rows_idx, int n, const float* w, void* out,
+                     long long ldo, int dim, int dim_pad, int groups, float eps, int fp32, void* status, void* stream);
 // out[i] = norm(x[rows_idx[i]]) as activations
 int fb_norm_rows(const float* x, long long ldx, int x_rows, const int* rows_idx, int n, const float* norm_w,
                  const float* norm_b, int rms, void* out, long long ldo, int dim, int dim_pad, float eps, int fp32,
@@ -339,16 +364,53 @@ typedef struct FbGqaArgs {
   void* out;                // [rows, ldo]: heads x vdim_pad
   long long ldo;
   int rows, heads, kv_heads, dim, dim_pad, vdim, vdim_pad, fp32;
+  // the attention kernels (not fb_gqa_prep): q holds heads x maps rows of key_width; a row of kv head g meets the cache
+  // columns from g * key_stride on (stride 0: the keys of all kv heads side by side), values start at v_offset
+  int maps;                 // 2: output of a head = rms(map 1 - diff_lambda * map 2) * diff_scale
+  int key_width, key_stride, v_offset;
+  int window, keep_first;   // chunk 0: position i sees j with i - j < window, or j < keep_first
+  const float* slopes;      // optional [heads]: slopes[h] * (i - j) is taken off the scaled score
+  const void* gate;         // optional [rows, ldg]: output multiplied by sigmoid(gate)
+  long long ldg;
+  float diff_lambda, diff_scale;
   void* status;
 } FbGqaArgs;
 int fb_gqa_prep(const FbGqaArgs* args, void* stream);
-int fb_gqa_attention(const FbGqaArgs* args, void* stream);      // dim, vdim <= 512
-// bf16, few rows (gqa_decode.cu): dim, vdim <= 256; the visible keys of a row are divided among `splits` (1, 2, 4, 8) CTAs;
+int fb_gqa_attention(const FbGqaArgs* args, void* stream);      // vdim <= 512
+// bf16, few rows (gqa_decode.cu): key_width, vdim <= 256, key_stride > 0; the visible keys of a row are divided among `splits` (1, 2, 4, 8) CTAs;
 // early: one row per sequence, keys below a row's own position predate the preceding kernel
 int fb_gqa_decode(const FbGqaArgs* args, int splits, int early, void* stream);
-// bf16 prompts on tcgen05 (gqa_prefill_tc.cu): dim, vdim <= 256, page_size a power of two >= 8; tiles [n_tiles, 4] =
-// sequence, first row, rows (<= tile_positions), position of the first; tile_positions * heads / kv_heads <= 128
+// the same for keys that all heads share (gqa_decode_wide.cu): key_stride 0, one map; fb_gqa_decode_wide_ok: whether
+// cache rows of this shape fit its pipeline
+int fb_gqa_decode_wide(const FbGqaArgs* args, int splits, int early, void* stream);
+int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad);
+// bf16 prompts on tcgen05 (gqa_prefill_tc.cu): vdim <= 256, page_size a power of two >= 8; tiles [n_tiles, 4] =
+// sequence, first row, rows (<= tile_positions), position of the first; tile_positions * maps * heads / kv_heads <= 128
 int fb_gqa_prefill_tc(const FbGqaArgs* args, const int* tiles, int n_tiles, int tile_positions, void* stream);
+
+// ---- queries and keys normalised per head, before window attention (see head_prep.cu) -------------------------
+typedef struct FbHeadPrepArgs {
+  const void* q;            // [rows, ldp] projected rows: heads x maps x dim_pad
+  const void* k;            // kv_heads x maps x dim_pad
+  const void* v;            // kv_heads x vdim_pad; null: the values are the keys before their norm
+  long long ldp;
+  const float* q_bias;      // optional, as wide as q and k
+  const float* k_bias;
+  const float* q_norm;      // [dim_pad], shared by the heads
+  const float* k_norm;
+  const float* q_mix;       // [heads] factors, or [heads, heads]: out row h = sum_g q_mix[h, g] q_g, kv head by kv head
+  int mix;
+  void* q_out;              // [rows, ldqo]: mix: heads x (kv_heads x dim_pad); else heads x maps x (maps x dim_pad), map
+                            // m's query in columns m * dim_pad.., zeros elsewhere
+  long long ldqo;
+  const long long* write_slot;
+  void* pool;               // [pool_rows, pool_ld]: kv_heads x maps x dim_pad keys | kv_heads x vdim_pad values
+  long long pool_rows, pool_ld;
+  int rows, heads, kv_heads, maps, dim, dim_pad, vdim_pad, fp32;
+  float eps;
+  void* status;
+} FbHeadPrepArgs;
+int fb_head_prep(const FbHeadPrepArgs* args, void* stream);
 
 // ---- gated delta rule (see delta_rule.cu) ------------------------------------------------------------------
 typedef struct FbDeltaArgs {

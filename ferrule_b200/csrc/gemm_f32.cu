@@ -1,6 +1,6 @@
 // out = x @ w^T in full 32 bits on the FMA units: the GEMM of models that run in fp32 (no tensor-core mode has 32-bit
 // operands).  Takes the argument block of the tcgen05 GEMM - dense, batched per head, grouped by a MoE row-tile
-// table; store, GELU, SwiGLU and weighted scatter epilogues - with fp32 tensors and pitches in elements.
+// table; store, GELU, SwiGLU, GeGLU and weighted scatter epilogues - with fp32 tensors and pitches in elements.
 //
 // 64 rows x 64 channels per CTA, 256 threads with 4 x 4 outputs each, K in steps of 16 through shared memory.
 #include "common.cuh"
@@ -16,7 +16,7 @@ struct GemmF32Params {
   const float* x;
   float* out;
   long long ldw, w_group_stride, ldx, ldo;
-  int n_out, k, groups, x_rows, ntok, dual_offset, x_group_koff, out_group_coff, batched, gelu;
+  int n_out, k, groups, x_rows, ntok, dual_offset, x_group_koff, out_group_coff, batched, gelu, geglu;
   const int* tile_group;
   const int* tile_row0;
   const int* tile_rows;
@@ -94,7 +94,7 @@ gemm_f32_kernel(const GemmF32Params p) {
       const int n = n0 + tx * 4 + j;
       if (n >= p.n_out) continue;
       float v = acc[i][j];
-      if (DUAL) v = v / (1.f + expf(-v)) * up[i][j];
+      if (DUAL) v = (p.geglu ? gelu_tanh_f(v) : v / (1.f + expf(-v))) * up[i][j];
       if (p.gelu) v = gelu_f(v);
       o[n] = v * sc;
     }
@@ -107,7 +107,7 @@ using namespace fb;
 
 extern "C" int fb_gemm_f32(const FbGemmArgs* a, void* stream) {
   if (!a || !a->w || !a->x || !a->out || a->n_out <= 0 || a->k <= 0 || a->groups <= 0 || a->x_rows <= 0) return FB_ERR_SHAPE;
-  if (a->epilogue < 0 || a->epilogue == 3 || a->epilogue > 4 || a->act_limit != 0.f) return FB_ERR_SHAPE;
+  if (a->epilogue < 0 || a->epilogue == 3 || a->epilogue > 5 || a->act_limit != 0.f) return FB_ERR_SHAPE;
   const bool grouped = a->tile_group != nullptr, batched = !grouped && a->groups > 1;
   if (grouped && (!a->tile_row0 || !a->tile_rows || !a->num_tok_tiles || a->max_tok_tiles <= 0 || a->ntok <= 0))
     return FB_ERR_SHAPE;
@@ -119,6 +119,7 @@ extern "C" int fb_gemm_f32(const FbGemmArgs* a, void* stream) {
   p.dual_offset = a->dual_offset; p.x_group_koff = a->x_group_koff; p.out_group_coff = a->out_group_coff;
   p.batched = batched ? 1 : 0;
   p.gelu = a->epilogue == 4 ? 1 : 0;
+  p.geglu = a->epilogue == 5 ? 1 : 0;
   if (grouped) {
     p.tile_group = a->tile_group; p.tile_row0 = a->tile_row0; p.tile_rows = a->tile_rows; p.num_tiles = a->num_tok_tiles;
   }
@@ -128,7 +129,7 @@ extern "C" int fb_gemm_f32(const FbGemmArgs* a, void* stream) {
   if (row_tiles > 65535 || (batched && a->groups > 65535)) return FB_ERR_LIMIT;
   const dim3 grid((a->n_out + kF32Tile - 1) / kF32Tile, row_tiles, batched ? a->groups : 1);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (a->epilogue == 1) launch_pdl(gemm_f32_kernel<true>, grid, dim3(256), 0, s, p);
+  if (a->epilogue == 1 || a->epilogue == 5) launch_pdl(gemm_f32_kernel<true>, grid, dim3(256), 0, s, p);
   else launch_pdl(gemm_f32_kernel<false>, grid, dim3(256), 0, s, p);
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }

@@ -12,6 +12,7 @@
 //   kEpiStore   : out[row, n]            = acc                      (bf16 or fp32)
 //   kEpiGelu    : out[row, n]            = gelu(acc)                (exact, error-function form)
 //   kEpiSwiGLU  : out[row, n]            = silu(gate) * up          (two weight tiles per k-block)
+//   kEpiGeGLU   : out[row, n]            = gelu(gate) * up          (the same, tanh form)
 //   kEpiScatter : out[dst_row[row], n]   = acc * row_scale[row]     (MoE down projection)
 //   kEpiAllReduce: partial tiles are pushed into every rank's receive buffer over
 //                 NVLink peer stores, then summed in rank order once all have landed
@@ -35,7 +36,7 @@ constexpr int kBlockK = 64;   // bf16 elements per k-block = one 128-byte swizzl
 constexpr int kUmmaK = 16;
 constexpr int kGemmThreads = 192;
 
-enum { kEpiStore = 0, kEpiSwiGLU = 1, kEpiScatter = 2, kEpiAllReduce = 3, kEpiGelu = 4 };
+enum { kEpiStore = 0, kEpiSwiGLU = 1, kEpiScatter = 2, kEpiAllReduce = 3, kEpiGelu = 4, kEpiGeGLU = 5 };
 
 struct GemmParams {
   int n_out;          // output channels per group
@@ -393,6 +394,11 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
                 u[j] = __float_as_uint(__uint_as_float(u[j]) + rp[static_cast<size_t>(NTOK + c0 + j) * 128]);
             }
           }
+        }
+        if (EPI == kEpiGeGLU) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j)
+            v[j] = __float_as_uint(gelu_tanh_bf16_f(__uint_as_float(v[j])) * __uint_as_float(u[j]));
         }
         if (EPI == kEpiGelu) {
           // all sixteen without a branch between them: their latencies overlap
@@ -761,8 +767,8 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   if (a == nullptr || a->w == nullptr || a->x == nullptr || a->out == nullptr) return FB_ERR_SHAPE;
   if (a->n_out <= 0 || a->k <= 0 || a->groups <= 0 || (a->k % 8) != 0) return FB_ERR_SHAPE;
-  if (a->epilogue < 0 || a->epilogue > 4) return FB_ERR_SHAPE;
-  const bool dual = a->epilogue == kEpiSwiGLU;
+  if (a->epilogue < 0 || a->epilogue > kEpiGeGLU) return FB_ERR_SHAPE;
+  const bool dual = a->epilogue == kEpiSwiGLU || a->epilogue == kEpiGeGLU;
   const int ntok = a->ntok;
   if (ntok != 16 && ntok != 32 && ntok != 64 && ntok != 128 && ntok != 256) return FB_ERR_SHAPE;
   if (dual && ntok > 128) return FB_ERR_SHAPE;
@@ -841,6 +847,7 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
     p.peer_wait_ns = a->peer_wait_ns ? a->peer_wait_ns : 3000000000ull;
     return launch_ntok<false, kEpiAllReduce>(ntok, mw, mx, p, max_tiles, grouped, stream);
   }
+  if (a->epilogue == kEpiGeGLU) return launch_ntok<true, kEpiGeGLU>(ntok, mw, mx, p, max_tiles, grouped, stream);
   if (dual) return launch_ntok<true, kEpiSwiGLU>(ntok, mw, mx, p, max_tiles, grouped, stream);
   if (a->epilogue == kEpiScatter) {
     if (a->remap_rank != nullptr) {

@@ -1,16 +1,18 @@
-// Grouped-query attention inside position-aligned chunks, over paged keys and values.
+// Grouped-query attention inside position-aligned chunks or sliding windows (gqa_mask.cuh), over paged keys and values.
 //
-// A query at position i sees the keys floor(i / chunk) * chunk .. i; query head h reads key / value head h / (H / G).  A
-// cache row holds [G][dim_pad] keys | [G][vdim_pad] values (heads padded to multiples of 8, padding is zero).
+// Query head h reads key / value head h / (H / G).  A cache row holds [G][maps][dim_pad] keys | [G][vdim_pad] values (heads
+// padded to multiples of 8, padding is zero).
 //
 //   fb_gqa_prep       everything between the projection and the attention in one launch: query and key RMS norm over the
 //                     whole projection, rotation of the leading dimensions (halves paired), value norm per head, mixing
 //                     with the first mixing layer's values of the token (read from that layer's cache row), cache append
 //   fb_gqa_attention  attention in 32-bit arithmetic, one CTA per (query row, head): models that run in fp32, and head sizes
-//                     the tensor-core kernels do not take
+//                     the tensor-core kernels do not take.  Query rows as wide as the keys they meet (all kv heads' keys
+//                     when scores are mixed across heads), distance bias, difference of two maps, output gate
 #include "act_type.cuh"
 #include "common.cuh"
 #include "ferrule_b200.h"
+#include "gqa_mask.cuh"
 #include "launch.cuh"
 
 namespace fb {
@@ -37,7 +39,13 @@ struct GqaParams {
   const int* block_table;
   const int* row_seq;
   const int* row_pos;
-  int num_seqs, max_blocks, page_size, chunk;
+  int num_seqs, max_blocks, page_size;
+  KeySpan span;
+  int maps, key_width, key_stride, v_offset;
+  const float* slopes;
+  const T* gate;
+  long long ldg;
+  float diff_lambda, diff_scale;
   float scale, eps;
   T* out;
   long long ldo;
@@ -256,14 +264,17 @@ gqa_prep_vec_kernel(const GqaParams<T> p) {
   }
 }
 
-// DPL: query / key and value features per lane
+// CTA = (query row, head); DPL: value features per lane.  A head with two maps attends twice over the same values.
 template <typename T, int DPL>
 __global__ void __launch_bounds__(128)
 gqa_attention_kernel(const GqaParams<T> p) {
   pdl_launch_dependents();
   pdl_wait();
-  __shared__ float sm_m[4], sm_l[4];
+  extern __shared__ float sm[];                 // [key_width] query, [maps][vdim_pad] outputs
+  __shared__ float sm_m[4], sm_l[4], red[32];
   __shared__ float sm_o[4][DPL * 32];
+  float* sq = sm;
+  float* res = sm + p.key_width;
   const int r = blockIdx.x, h = blockIdx.y, g = h / (p.heads / p.kv_heads);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.row_seq[r], pos = p.row_pos[r];
@@ -273,60 +284,82 @@ gqa_attention_kernel(const GqaParams<T> p) {
     len = 0;
   }
   len = min(len, p.max_blocks * p.page_size);
-  const int first = pos >= 0 ? pos / p.chunk * p.chunk : 0;
-  const long long koff = static_cast<long long>(g) * p.dim_pad;
-  const long long voff = static_cast<long long>(p.kv_heads) * p.dim_pad + static_cast<long long>(g) * p.vdim_pad;
-  float q[DPL], o[DPL];
+  const int first = len > 0 ? p.span.first(pos) : 0, kept = len > 0 ? p.span.head(pos) : 0;
+  const int n_keys = kept + max(len - first, 0);
+  const float slope = p.slopes ? p.slopes[h] : 0.f;
+  // with two maps a query row is zero outside its own half
+  const int part = p.key_width / p.maps;
+  const long long voff = p.v_offset + static_cast<long long>(g) * p.vdim_pad;
+  for (int map = 0; map < p.maps; ++map) {
+    const T* qr = p.q + r * p.ldq + (static_cast<long long>(h) * p.maps + map) * p.key_width + map * part;
+    const long long koff = static_cast<long long>(g) * p.key_stride + map * part;
+    __syncthreads();
+    for (int d = threadIdx.x; d < part; d += blockDim.x) sq[d] = act_load(qr + d);
+    __syncthreads();
+    float o[DPL];
 #pragma unroll
-  for (int j = 0; j < DPL; ++j) {
-    const int d = lane + 32 * j;
-    q[j] = d < p.dim ? act_load(p.q + r * p.ldq + static_cast<long long>(h) * p.dim_pad + d) : 0.f;
-    o[j] = 0.f;
-  }
-  float m = -INFINITY, l = 0.f;
-  for (int t = first + warp; t < len; t += 4) {
-    const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
-    const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
-    if (page < 0 || slot >= p.pool_rows) {
-      if (lane == 0) report_status(p.status, kStatusBadIndex, 0xD71, seq, t);
-      continue;
+    for (int j = 0; j < DPL; ++j) o[j] = 0.f;
+    float m = -INFINITY, l = 0.f;
+    for (int i = warp; i < n_keys; i += 4) {
+      const int t = i < kept ? i : first + i - kept;
+      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+      const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
+      if (page < 0 || slot >= p.pool_rows) {
+        if (lane == 0) report_status(p.status, kStatusBadIndex, 0xD71, seq, t);
+        continue;
+      }
+      const T* row = p.pool + slot * p.pool_ld;
+      float s = 0.f, v[DPL];
+#pragma unroll
+      for (int j = 0; j < DPL; ++j) {
+        const int d = lane + 32 * j;
+        v[j] = d < p.vdim ? act_load(row + voff + d) : 0.f;
+      }
+#pragma unroll 4
+      for (int d = lane; d < part; d += 32) s = fmaf(sq[d], act_load(row + koff + d), s);
+      s = fmaf(-slope, static_cast<float>(pos - t), warp_sum(s) * p.scale);
+      if (s > m) {
+        const float a = expf(m - s);
+        m = s;
+        l *= a;
+#pragma unroll
+        for (int j = 0; j < DPL; ++j) o[j] *= a;
+      }
+      const float w = expf(s - m);
+      l += w;
+#pragma unroll
+      for (int j = 0; j < DPL; ++j) o[j] = fmaf(w, v[j], o[j]);
     }
-    const T* row = p.pool + slot * p.pool_ld;
-    float s = 0.f, v[DPL];
+    if (lane == 0) { sm_m[warp] = m; sm_l[warp] = l; }
 #pragma unroll
-    for (int j = 0; j < DPL; ++j) {
-      const int d = lane + 32 * j;
-      s = fmaf(q[j], d < p.dim ? act_load(row + koff + d) : 0.f, s);
-      v[j] = d < p.vdim ? act_load(row + voff + d) : 0.f;
+    for (int j = 0; j < DPL; ++j) sm_o[warp][lane + 32 * j] = o[j];
+    __syncthreads();
+    const float M = fmaxf(fmaxf(sm_m[0], sm_m[1]), fmaxf(sm_m[2], sm_m[3]));
+    float w[4], L = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      w[k] = sm_m[k] == -INFINITY ? 0.f : expf(sm_m[k] - M);
+      L += w[k] * sm_l[k];
     }
-    s = warp_sum(s) * p.scale;
-    if (s > m) {
-      const float a = expf(m - s);
-      m = s;
-      l *= a;
-#pragma unroll
-      for (int j = 0; j < DPL; ++j) o[j] *= a;
+    const float f = L > 0.f ? 1.f / L : 0.f;
+    for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x)
+      res[map * p.vdim_pad + d] =
+          d < p.vdim ? (w[0] * sm_o[0][d] + w[1] * sm_o[1][d] + w[2] * sm_o[2][d] + w[3] * sm_o[3][d]) * f : 0.f;
+  }
+  // every thread finishes the columns it wrote itself
+  float inv = 1.f;
+  if (p.maps == 2) {
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x) {
+      res[d] -= p.diff_lambda * res[p.vdim_pad + d];
+      ss = fmaf(res[d], res[d], ss);
     }
-    const float w = expf(s - m);
-    l += w;
-#pragma unroll
-    for (int j = 0; j < DPL; ++j) o[j] = fmaf(w, v[j], o[j]);
+    inv = p.diff_scale / sqrtf(cta_sum(ss, red) / p.vdim + p.eps);
   }
-  if (lane == 0) { sm_m[warp] = m; sm_l[warp] = l; }
-#pragma unroll
-  for (int j = 0; j < DPL; ++j) sm_o[warp][lane + 32 * j] = o[j];
-  __syncthreads();
-  const float M = fmaxf(fmaxf(sm_m[0], sm_m[1]), fmaxf(sm_m[2], sm_m[3]));
-  float w[4], L = 0.f;
-#pragma unroll
-  for (int k = 0; k < 4; ++k) {
-    w[k] = sm_m[k] == -INFINITY ? 0.f : expf(sm_m[k] - M);
-    L += w[k] * sm_l[k];
-  }
-  const float f = L > 0.f ? 1.f / L : 0.f;
   T* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.vdim_pad;
+  const T* gate = p.gate ? p.gate + r * p.ldg + static_cast<long long>(h) * p.vdim_pad : nullptr;
   for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x)
-    act_store(dst + d, d < p.vdim ? (w[0] * sm_o[0][d] + w[1] * sm_o[1][d] + w[2] * sm_o[2][d] + w[3] * sm_o[3][d]) * f : 0.f);
+    act_store(dst + d, res[d] * inv * (gate ? sigmoid_f(act_load(gate + d)) : 1.f));
 }
 
 template <typename T>
@@ -339,7 +372,11 @@ static void fill_gqa(const FbGqaArgs* a, GqaParams<T>& p) {
   p.pool = static_cast<T*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
   p.first_pool = static_cast<const T*>(a->first_pool); p.first_off = a->first_off; p.v_mix = a->v_mix;
   p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
-  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size; p.chunk = a->chunk;
+  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
+  p.span = {a->chunk, a->window, a->keep_first};
+  p.maps = a->maps; p.key_width = a->key_width; p.key_stride = a->key_stride; p.v_offset = a->v_offset;
+  p.slopes = a->slopes; p.gate = static_cast<const T*>(a->gate); p.ldg = a->ldg;
+  p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale;
   p.scale = a->scale; p.eps = a->eps;
   p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
   p.rows = a->rows; p.heads = a->heads; p.kv_heads = a->kv_heads;
@@ -351,8 +388,7 @@ static bool gqa_sizes_ok(const FbGqaArgs* a) {
   return a && a->q && a->pool && a->rows > 0 && a->heads > 0 && a->heads <= 65535 && a->kv_heads > 0 &&
          a->heads % a->kv_heads == 0 && a->dim > 0 && a->vdim > 0 && a->dim_pad >= a->dim && a->vdim_pad >= a->vdim &&
          a->dim_pad % 8 == 0 && a->vdim_pad % 8 == 0 && a->pool_rows > 0 && a->pool_ld % 8 == 0 &&
-         a->pool_ld >= static_cast<long long>(a->kv_heads) * (a->dim_pad + a->vdim_pad) && a->ldq % 8 == 0 &&
-         a->ldq >= static_cast<long long>(a->heads) * a->dim_pad;
+         a->ldq % 8 == 0;
 }
 
 template <typename T>
@@ -380,17 +416,29 @@ static int run_prep(const FbGqaArgs* a, cudaStream_t s) {
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 
+template <typename T, int DPL>
+static int launch_attention(const GqaParams<T>& p, cudaStream_t s) {
+  const size_t smem = (static_cast<size_t>(p.key_width) + p.maps * p.vdim_pad) * sizeof(float);
+  if (smem > 200 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(gqa_attention_kernel<T, DPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(gqa_attention_kernel<T, DPL>, dim3(p.rows, p.heads), dim3(128), smem, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
 template <typename T>
 static int run_attention(const FbGqaArgs* a, cudaStream_t s) {
   GqaParams<T> p{};
   fill_gqa(a, p);
-  const dim3 grid(a->rows, a->heads);
-  const int d = ((a->dim > a->vdim ? a->dim : a->vdim) + 31) / 32;
-  if (d <= 2) launch_pdl(gqa_attention_kernel<T, 2>, grid, dim3(128), 0, s, p);
-  else if (d <= 4) launch_pdl(gqa_attention_kernel<T, 4>, grid, dim3(128), 0, s, p);
-  else if (d <= 8) launch_pdl(gqa_attention_kernel<T, 8>, grid, dim3(128), 0, s, p);
-  else launch_pdl(gqa_attention_kernel<T, 16>, grid, dim3(128), 0, s, p);
-  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  const int d = (a->vdim + 31) / 32;
+  if (d <= 2) return launch_attention<T, 2>(p, s);
+  if (d <= 4) return launch_attention<T, 4>(p, s);
+  if (d <= 8) return launch_attention<T, 8>(p, s);
+  return launch_attention<T, 16>(p, s);
 }
 
 }  // namespace fb
@@ -399,7 +447,8 @@ using namespace fb;
 
 extern "C" int fb_gqa_prep(const FbGqaArgs* a, void* stream) {
   if (!gqa_sizes_ok(a) || !a->k || !a->v || !a->q_norm || !a->k_norm || !a->positions || !a->write_slot || a->max_pos <= 0 ||
-      a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->dim || (a->rot_dims && (!a->cos_t || !a->sin_t)))
+      a->pool_ld < static_cast<long long>(a->kv_heads) * (a->dim_pad + a->vdim_pad) ||
+      a->ldq < static_cast<long long>(a->heads) * a->dim_pad || a->rot_dims < 0 || a->rot_dims % 2 || a->rot_dims > a->dim || (a->rot_dims && (!a->cos_t || !a->sin_t)))
     return FB_ERR_SHAPE;
   if (a->ldkv % 8 || a->first_off < 0 || a->first_off + static_cast<long long>(a->kv_heads) * a->vdim_pad > a->pool_ld)
     return FB_ERR_SHAPE;
@@ -412,9 +461,9 @@ extern "C" int fb_gqa_prep(const FbGqaArgs* a, void* stream) {
 
 extern "C" int fb_gqa_attention(const FbGqaArgs* a, void* stream) {
   if (!gqa_sizes_ok(a) || !a->out || !a->block_table || !a->row_seq || !a->row_pos || a->num_seqs <= 0 || a->max_blocks <= 0 ||
-      a->page_size <= 0 || a->chunk <= 0 || a->ldo < static_cast<long long>(a->heads) * a->vdim_pad)
+      a->page_size <= 0 || !gqa_form_ok(a))
     return FB_ERR_SHAPE;
-  if (a->dim > 512 || a->vdim > 512) return FB_ERR_LIMIT;
+  if (a->vdim > 512) return FB_ERR_LIMIT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return a->fp32 ? run_attention<float>(a, s) : run_attention<__nv_bfloat16>(a, s);
 }

@@ -1,0 +1,407 @@
+// Window attention of few query rows (decode steps, short portions) whose query rows meet the keys of all kv heads, bf16.
+//
+// Scores that are mixed across heads are products of one wide query row per head with the concatenated keys of a token
+// (head_prep.cu), so a CTA takes all of a token's cache row: keys and values of every kv head lie side by side there and come
+// as one bulk copy per token.  CTA = (query row, split of the visible keys, block of 16 heads), 8 warps; a tile is KT tokens.
+//
+//   scores   warp w multiplies the 16 query rows with 8 of the tile's keys over a share of the features (MMA, partial sums in
+//            shared memory)
+//   softmax  two rows per warp, a key per lane: distance bias, running maximum and sum, probabilities to shared memory
+//   values   warp w accumulates 16-column pieces w, w + 8, ... of the values for all 16 rows; a head keeps the columns of
+//            its own kv head
+//
+// The splits of a row (one thread-block cluster) merge through distributed shared memory; the output gate is applied there.
+// The kernel is bound by the cache stream, a 16-row tile is below the 64-row minimum of tcgen05: warp-level MMA.  In a decode
+// step the first tiles (older than the step) are requested before the dependency wait.  Every wait is bounded.
+#include "act_type.cuh"
+#include "common.cuh"
+#include "ferrule_b200.h"
+#include "gqa_mask.cuh"
+#include "launch.cuh"
+#include "mma_sync.cuh"
+
+namespace fb {
+
+constexpr int kGwThreads = 256;
+constexpr int kGwMaxStages = 8;
+constexpr int kGwSmemLimit = 227 * 1024;
+
+struct GwParams {
+  const __nv_bfloat16* q;
+  long long ldq;
+  const __nv_bfloat16* pool;
+  long long pool_rows, pool_ld;
+  const int* block_table;
+  const int* row_seq;
+  const int* row_pos;
+  int num_seqs, max_blocks, page_size;
+  KeySpan span;
+  float scale_log2;
+  const float* slopes;
+  const __nv_bfloat16* gate;
+  long long ldg;
+  __nv_bfloat16* out;
+  long long ldo;
+  int heads, kv_heads, key_width, vdim_pad;
+  int row_bytes, pitch, stages, head_blocks;       // bytes of a token's keys and values, and of its place in a tile
+  int early;
+  DeviceStatus* status;
+};
+
+// shared memory behind the tiles
+struct GwLayout {
+  int q_pitch, q, part, prob, factor, bars, total;
+  __host__ __device__ GwLayout(int key_width, int tile_bytes, int kt) {
+    q_pitch = (key_width + 15) / 16 * 16 + 8;
+    q = tile_bytes;
+    part = q + 16 * q_pitch * 2;
+    prob = part + (64 / kt) * 16 * (kt + 1) * 4;
+    factor = prob + 16 * (kt + 8) * 2;
+    bars = factor + 48 * 4;
+    total = bars + (kGwMaxStages + 1) * 8;
+  }
+};
+
+// untiled copy of one cache row; both addresses and the size are multiples of 16 bytes
+__device__ __forceinline__ void gw_copy_row(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(reinterpret_cast<uint64_t>(src)), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
+}
+__device__ __forceinline__ void ldsm_x2(uint32_t (&r)[2], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
+}
+
+// NC: 16-column value pieces per warp
+template <int KT, int NC>
+__global__ void __launch_bounds__(kGwThreads)
+gqa_decode_wide_kernel(const GwParams p) {
+  constexpr int kNt = KT / 8, kShares = 8 / kNt;   // 8-key columns of the score tile, feature shares
+  pdl_launch_dependents();
+  extern __shared__ __align__(128) uint8_t gw_sm[];
+  const int tile_bytes = KT * p.pitch;
+  const GwLayout at(p.key_width, p.stages * tile_bytes, KT);
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(gw_sm + at.q);
+  float* part_s = reinterpret_cast<float*>(gw_sm + at.part);               // [kShares][16][KT + 1]
+  __nv_bfloat16* prob_s = reinterpret_cast<__nv_bfloat16*>(gw_sm + at.prob);   // [16][KT + 8]
+  float* f_s = reinterpret_cast<float*>(gw_sm + at.factor);                // [16] rescale factors
+  float* c_m = f_s + 16;
+  float* c_l = c_m + 16;
+  uint64_t* full = reinterpret_cast<uint64_t*>(gw_sm + at.bars);
+  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(full + kGwMaxStages);
+
+  const int r = blockIdx.x, split = blockIdx.y, splits = gridDim.y, h0 = blockIdx.z * 16, nh = min(16, p.heads - h0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
+  const int seq = p.row_seq[r], pos = p.row_pos[r], per = p.heads / p.kv_heads;
+  int lo = 0, hi = 0, first = 0, kept = 0, n_keys = 0;                     // lo, hi: indices into the visible keys
+  if (seq < 0 || seq >= p.num_seqs) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE80, r, seq);
+  } else if (pos >= 0) {
+    first = p.span.first(pos);
+    kept = p.span.head(pos);
+    n_keys = kept + max(min(pos + 1, p.max_blocks * p.page_size) - first, 0);
+    const int tiles = (n_keys + KT - 1) / KT, share = (tiles + splits - 1) / splits;
+    lo = min(split * share * KT, n_keys);
+    hi = min(lo + share * KT, n_keys);
+  }
+  const int n_tiles = (hi - lo + KT - 1) / KT;
+  const long long n_pages = p.pool_rows / p.page_size;
+  auto token = [&](int i) { return i < kept ? i : first + i - kept; };
+  if (tid == 0) {
+    for (int i = 0; i < p.stages; ++i) mbar_init(full + i, 1);
+    *abort_flag = 0;
+    fence_barrier_init();
+  }
+  __syncthreads();
+  // warp 0: a token per lane; places past the last key repeat it (their probability is zero, their values must be finite)
+  auto request = [&](int i) {
+    uint8_t* dst = gw_sm + (i % p.stages) * tile_bytes;
+    uint64_t* bar = full + i % p.stages;
+    long long slot = 0;
+    if (lane < KT) {
+      const int t = token(min(lo + i * KT + lane, hi - 1));
+      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+      if (page >= 0 && page < n_pages) slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
+      else report_status(p.status, kStatusBadIndex, 0xE81, seq, t);
+    }
+    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(KT * p.row_bytes));
+    __syncwarp();
+    if (lane < KT) gw_copy_row(dst + lane * p.pitch, p.pool + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes), bar);
+  };
+  int asked = 0;
+  if (warp == 0 && p.early)
+    // tiles that end below the row's own position: written by earlier steps
+    while (asked < p.stages && asked < n_tiles && lo + (asked + 1) * KT < n_keys) request(asked++);
+  pdl_wait();
+  if (warp == 0)
+    for (; asked < p.stages && asked < n_tiles; ++asked) request(asked);
+  // query rows of this block; rows past the last head and columns past the width are zeros
+  for (int i = tid; i < 16 * (at.q_pitch / 8); i += kGwThreads) {
+    const int row = i / (at.q_pitch / 8), c = (i - row * (at.q_pitch / 8)) * 8;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (row < nh && c < p.key_width)
+      v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.key_width + c);
+    *reinterpret_cast<uint4*>(q_s + row * at.q_pitch + c) = v;
+  }
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, sl[2];           // rows 2 warp, 2 warp + 1
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const int row = 2 * warp + k;
+    sl[k] = p.slopes && row < nh ? p.slopes[h0 + row] * 1.4426950408889634f : 0.f;
+  }
+  float o[NC][2][4];
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
+#pragma unroll
+    for (int n = 0; n < 2; ++n) o[c][n][0] = o[c][n][1] = o[c][n][2] = o[c][n][3] = 0.f;
+  const int ksteps = (p.key_width + 15) / 16, share = (ksteps + kShares - 1) / kShares;
+  const int nt = warp % kNt, part = warp / kNt, k0 = min(part * share, ksteps), k1 = min(k0 + share, ksteps);
+  const uint32_t qa = smem_u32(q_s + (lane & 15) * at.q_pitch + (lane >> 4) * 8);
+  const int vcols = (p.vdim_pad + 15) / 16, n_cols = p.kv_heads * vcols;
+  __syncthreads();
+  int done = 0;
+  for (int i = 0; i < n_tiles; ++i) {
+    const uint8_t* tile = gw_sm + (i % p.stages) * tile_bytes;
+    bool ok = mbar_wait(full + i % p.stages, (i / p.stages) & 1, abort_flag, p.status, 0xE90);
+    if (ok) {
+      float s0[4] = {}, s1[4] = {};
+      const uint32_t ka = smem_u32(tile + (nt * 8 + (lane & 7)) * p.pitch) + (lane >> 3) * 16;
+      int k = k0;
+      for (; k + 1 < k1; k += 2) {
+        uint32_t a0[4], a1[4], b[4];
+        ldsm_x4(b, ka + k * 32);
+        ldsm_x4(a0, qa + k * 32);
+        ldsm_x4(a1, qa + k * 32 + 32);
+        mma_bf16_16816(s0, a0, b[0], b[1]);
+        mma_bf16_16816(s1, a1, b[2], b[3]);
+      }
+      if (k < k1) {
+        uint32_t a0[4], b[2];
+        ldsm_x2(b, smem_u32(tile + (nt * 8 + (lane & 7)) * p.pitch) + ((lane >> 3) & 1) * 16 + k * 32);
+        ldsm_x4(a0, qa + k * 32);
+        mma_bf16_16816(s0, a0, b[0], b[1]);
+      }
+      float* dst = part_s + (part * 16 + g4) * (KT + 1) + nt * 8 + t4 * 2;
+      dst[0] = s0[0] + s1[0];
+      dst[1] = s0[1] + s1[1];
+      dst[8 * (KT + 1)] = s0[2] + s1[2];
+      dst[8 * (KT + 1) + 1] = s0[3] + s1[3];
+    }
+    // also: every warp is done with tile i - 1
+    if (!__syncthreads_and(ok)) break;
+    if (warp == 0 && i > 0 && i - 1 + p.stages < n_tiles) request(i - 1 + p.stages);
+    const int key = lo + i * KT + lane;
+    const bool seen = lane < KT && key < hi;
+    const float dist = static_cast<float>(pos - token(min(key, hi - 1)));
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int row = 2 * warp + k;
+      float x = -INFINITY;
+      if (seen) {
+        float s = 0.f;
+#pragma unroll
+        for (int q = 0; q < kShares; ++q) s += part_s[(q * 16 + row) * (KT + 1) + lane];
+        x = fmaf(-sl[k], dist, s * p.scale_log2);
+      }
+      const float mn = fmaxf(m[k], warp_max(x));                            // finite: a tile has at least one visible key
+      const float f = exp2f(m[k] - mn), w = seen ? exp2f(x - mn) : 0.f;
+      m[k] = mn;
+      l[k] = fmaf(l[k], f, warp_sum(w));
+      if (lane < KT) prob_s[row * (KT + 8) + lane] = __float2bfloat16_rn(w);
+      if (lane == 0) f_s[row] = f;
+    }
+    __syncthreads();
+    const float f0 = f_s[g4], f1 = f_s[g4 + 8];
+    uint32_t pf[KT / 16][4];
+#pragma unroll
+    for (int k = 0; k < KT / 16; ++k) ldsm_x4(pf[k], smem_u32(prob_s + (lane & 15) * (KT + 8) + k * 16 + (lane >> 4) * 8));
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const int col = warp + 8 * c;
+      if (col >= n_cols) break;
+      const int g = col / vcols, d = (col - g * vcols) * 16;
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        o[c][n][0] *= f0;
+        o[c][n][1] *= f0;
+        o[c][n][2] *= f1;
+        o[c][n][3] *= f1;
+      }
+      // matrices (transposed): keys 0-7 / 8-15 x columns 0-7, then columns 8-15
+      const uint32_t va = smem_u32(tile + ((lane >> 3 & 1) * 8 + (lane & 7)) * p.pitch) +
+                          (p.key_width + g * p.vdim_pad + d + (lane >> 4) * 8) * 2;
+#pragma unroll
+      for (int k = 0; k < KT / 16; ++k) {
+        uint32_t b[4];
+        ldsm_x4_t(b, va + k * 16 * p.pitch);
+        mma_bf16_16816(o[c][0], pf[k], b[0], b[1]);
+        mma_bf16_16816(o[c][1], pf[k], b[2], b[3]);
+      }
+    }
+    done = i + 1;
+  }
+  if (done < n_tiles && tid == 0) {
+    // a wait gave up: copies may be in flight, and neither the merge nor the exit may happen under them
+    for (int i = done; i < min(done + p.stages, n_tiles); ++i) {
+      const uint64_t t0 = globaltimer_ns();
+      while (!mbar_try_wait(full + i % p.stages, (i / p.stages) & 1) && globaltimer_ns() - t0 < 2000000ull) {
+      }
+    }
+  }
+  if (lane == 0) {
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      c_m[2 * warp + k] = m[k];
+      c_l[2 * warp + k] = l[k];
+    }
+  }
+  __syncthreads();                                                         // the tiles' memory now holds the outputs
+  const int o_pitch = vcols * 16 + 4;
+  float* o_s = reinterpret_cast<float*>(gw_sm);                            // [16][o_pitch]
+#pragma unroll
+  for (int c = 0; c < NC; ++c) {
+    const int col = warp + 8 * c;
+    if (col >= n_cols) break;
+    const int g = col / vcols, d = (col - g * vcols) * 16 + t4 * 2;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int row = g4 + 8 * half;
+      if (row >= nh || (h0 + row) / per != g) continue;
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        o_s[row * o_pitch + d + n * 8] = o[c][n][2 * half];
+        o_s[row * o_pitch + d + n * 8 + 1] = o[c][n][2 * half + 1];
+      }
+    }
+  }
+  if (splits > 1) cluster_sync_all();
+  else __syncthreads();
+  const int quads = p.vdim_pad / 4;
+  for (int i = tid + split * kGwThreads; i < nh * quads; i += kGwThreads * splits) {
+    const int h = i / quads, d = (i - h * quads) * 4;
+    float mm = -INFINITY, ll = 0.f;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (splits == 1) {
+      ll = c_l[h];
+      a = *reinterpret_cast<const float4*>(o_s + h * o_pitch + d);
+    } else {
+      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + h), s)));
+      for (int s = 0; s < splits; ++s) {
+        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + h), s));
+        const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
+        ll = fmaf(f, ld_cluster_f32(mapa_shared(smem_u32(c_l + h), s)), ll);
+        const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(o_s + h * o_pitch + d), s));
+        a.x = fmaf(f, v.x, a.x);
+        a.y = fmaf(f, v.y, a.y);
+        a.z = fmaf(f, v.z, a.z);
+        a.w = fmaf(f, v.w, a.w);
+      }
+    }
+    const float inv = ll > 0.f ? 1.f / ll : 0.f;
+    a = make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+    const long long col = static_cast<long long>(h0 + h) * p.vdim_pad + d;
+    if (p.gate) {
+      const __nv_bfloat162* z = reinterpret_cast<const __nv_bfloat162*>(p.gate + r * p.ldg + col);
+      const float2 z0 = __bfloat1622float2(z[0]), z1 = __bfloat1622float2(z[1]);
+      a = make_float4(a.x * sigmoid_f(z0.x), a.y * sigmoid_f(z0.y), a.z * sigmoid_f(z1.x), a.w * sigmoid_f(z1.y));
+    }
+    __nv_bfloat16* dst = p.out + r * p.ldo + col;
+    *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a.x, a.y);
+    *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(a.z, a.w);
+  }
+  if (splits > 1) cluster_sync_all();                                      // no CTA leaves while a peer reads its rows
+}
+
+// tile size and stages for a cache row of this shape; 0: it does not fit
+struct GwPlan {
+  int kt, stages, nc;
+};
+static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad) {
+  const int vcols = (vdim_pad + 15) / 16, cols = kv_heads * vcols, pitch = (key_width + kv_heads * vdim_pad) * 2 + 16;
+  const int nc = cols <= 8 ? 1 : cols <= 16 ? 2 : cols <= 32 ? 4 : cols <= 64 ? 8 : 0;
+  for (int kt = 32; kt >= 16 && nc; kt /= 2) {
+    int stages = (kGwSmemLimit - GwLayout(key_width, 0, kt).total) / (kt * pitch);
+    if (stages > kGwMaxStages) stages = kGwMaxStages;
+    // the merged outputs reuse the tiles' memory
+    if (stages >= 2 && stages * kt * pitch >= 16 * (vcols * 16 + 4) * 4) return {kt, stages, nc};
+  }
+  return {0, 0, 0};
+}
+
+template <int KT, int NC>
+static int launch_gw(const GwParams& p, int rows, int splits, cudaStream_t stream) {
+  static bool attr_set = false;
+  if (!attr_set) {
+    if (cudaFuncSetAttribute(gqa_decode_wide_kernel<KT, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGwSmemLimit) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr_set = true;
+  }
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = dim3(rows, splits, p.head_blocks);
+  cfg.blockDim = dim3(kGwThreads);
+  cfg.dynamicSmemBytes = GwLayout(p.key_width, p.stages * KT * p.pitch, KT).total;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = 1;
+  attr[0].val.clusterDim.y = splits;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl_enabled() ? 2 : 1;
+  if (cudaLaunchKernelEx(&cfg, gqa_decode_wide_kernel<KT, NC>, p) != cudaSuccess) return FB_ERR_LAUNCH;
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad) {
+  return key_width > 0 && key_width % 8 == 0 && kv_heads > 0 && vdim_pad > 0 && vdim_pad % 8 == 0 &&
+         gw_plan(key_width, kv_heads, vdim_pad).kt > 0;
+}
+
+extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, void* stream) {
+  if (!a || !a->q || !a->pool || !a->out || !a->block_table || !a->row_seq || !a->row_pos || a->fp32) return FB_ERR_SHAPE;
+  if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->vdim_pad <= 0 || a->vdim_pad % 8 ||
+      a->pool_rows <= 0 || a->pool_ld % 8 || a->num_seqs <= 0 || a->max_blocks <= 0 || a->page_size <= 0)
+    return FB_ERR_SHAPE;
+  if (!gqa_form_ok(a) || a->key_stride != 0 || a->maps != 1 || a->v_offset != a->key_width || a->ldq % 8 || a->ldo % 4 ||
+      a->ldg % 4)
+    return FB_ERR_SHAPE;
+  if (splits != 1 && splits != 2 && splits != 4 && splits != 8) return FB_ERR_SHAPE;
+  const uintptr_t bits = reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->pool) |
+                         reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->gate);
+  if (bits & 15) return FB_ERR_ALIGN;
+  const GwPlan plan = gw_plan(a->key_width, a->kv_heads, a->vdim_pad);
+  if (plan.kt == 0) return FB_ERR_LIMIT;
+  GwParams p{};
+  p.q = static_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq;
+  p.pool = static_cast<const __nv_bfloat16*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
+  p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
+  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
+  p.span = {a->chunk, a->window, a->keep_first};
+  p.scale_log2 = a->scale * 1.4426950408889634f;
+  p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
+  p.out = static_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo;
+  p.heads = a->heads; p.kv_heads = a->kv_heads; p.key_width = a->key_width; p.vdim_pad = a->vdim_pad;
+  p.row_bytes = (a->key_width + a->kv_heads * a->vdim_pad) * 2;
+  p.pitch = p.row_bytes + 16;
+  p.stages = plan.stages;
+  p.head_blocks = (a->heads + 15) / 16;
+  p.early = early;
+  p.status = static_cast<DeviceStatus*>(a->status);
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (plan.kt == 32) {
+    if (plan.nc == 1) return launch_gw<32, 1>(p, a->rows, splits, s);
+    if (plan.nc == 2) return launch_gw<32, 2>(p, a->rows, splits, s);
+    if (plan.nc == 4) return launch_gw<32, 4>(p, a->rows, splits, s);
+    return launch_gw<32, 8>(p, a->rows, splits, s);
+  }
+  if (plan.nc == 1) return launch_gw<16, 1>(p, a->rows, splits, s);
+  if (plan.nc == 2) return launch_gw<16, 2>(p, a->rows, splits, s);
+  if (plan.nc == 4) return launch_gw<16, 4>(p, a->rows, splits, s);
+  return launch_gw<16, 8>(p, a->rows, splits, s);
+}

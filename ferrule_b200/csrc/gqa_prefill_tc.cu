@@ -1,24 +1,31 @@
-// Prefill attention of grouped-query layers inside position chunks on the 5th-generation tensor cores, bf16.
+// Prefill attention of grouped-query layers inside position chunks or sliding windows on the 5th-generation tensor cores,
+// bf16.
 //
-// CTA = one tile of consecutive query positions of one sequence x the query heads of one key / value head: up to 128
-// (position, head) rows, P = 128 / heads-per-group positions.  Keys are taken in tiles of 64 tokens at absolute positions
-// 64 j, from the first tile that holds a key of the tile's first chunk.
+// CTA = one tile of consecutive query positions of one sequence x the query heads of one key / value head (with two score
+// maps per head: both maps' rows): up to 128 (position, row) rows, P = 128 / rows-per-group positions.  Keys are taken in
+// tiles of 64 tokens at absolute positions 64 j: the tiles with kept first tokens, then from the first tile that holds a
+// key of the first position's chunk or window.
 //
 //   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
 //     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
-//     head's width and rows past the sequence are zeros), two stages each with their own barriers.
+//     head's width and rows past the sequence are zeros), two stages each with their own barriers.  Wide keys (those of all
+//     kv heads side by side) come in pieces of `kb` feature blocks, a stage each; query rows that do not fit in shared
+//     memory come with them, piece by piece, for every token tile.
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
 //     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
 //     before the current P is waited for.
-//   Softmax (warps 2..5, one row per thread): scores from TMEM, scale, causal and chunk mask, running maximum, exp2, bf16 P
+//   Softmax (warps 2..5, one row per thread): scores from TMEM, scale, distance bias, mask, running maximum, exp2, bf16 P
 //     written over the score buffer.  The accumulator is rescaled only when a row's maximum has grown by more than 2^8
-//     since the reference it was scaled by; the sum uses the same reference, so the result is exact up to rounding.
+//     since the reference it was scaled by; the sum uses the same reference, so the result is exact up to rounding.  The
+//     difference of a head's two maps is taken between neighbouring lanes, its RMS norm and the output gate on the way out.
 //
 // A row's result depends on the row and the cache contents, not on which rows share its tile or how a prompt was cut.
 // Every wait is bounded (status word, then teardown with TMEM freed); page ids are range-checked.
+#include "act_type.cuh"
 #include "attn_tc.cuh"
 #include "common.cuh"
 #include "ferrule_b200.h"
+#include "gqa_mask.cuh"
 #include "launch.cuh"
 
 namespace fb {
@@ -28,6 +35,7 @@ constexpr int kGpM = 128;
 constexpr int kGpKv = 64;
 constexpr int kGpQBlock = kGpM * 128;         // bytes of a 64-feature block of the query tile
 constexpr int kGpKvBlock = kGpKv * 128;
+constexpr int kGpSmemLimit = 227 * 1024;
 
 struct GpParams {
   const int* tiles;          // [n_tiles, 4] = sequence, first query row, query rows, position of the first
@@ -36,14 +44,25 @@ struct GpParams {
   long long ldo;
   DeviceStatus* status;
   long long pool_rows;
-  int rows, heads, kv_heads, per;      // per: query heads of a key / value head
+  int rows, heads, kv_heads, per;      // per: query rows of a key / value head
   int positions;             // positions per tile the query box holds
-  int num_seqs, max_blocks, page_size, box_rows, chunk;
-  int dim_pad, vdim_pad, qb, vb;       // qb, vb: 64-feature blocks of a query / key row and of a value row
+  int num_seqs, max_blocks, page_size, box_rows;
+  KeySpan span;
+  int key_width, vdim_pad, qb, vb;     // qb, vb: 64-feature blocks of a query / key row and of a value row
+  int kb, pieces, q_resident;          // blocks per key stage, stages per token tile
+  int shared_keys;
   uint32_t tmem_cols;
   float scale_log2;
+  const float* slopes;                 // [heads]
+  const __nv_bfloat16* gate;
+  long long ldg;
+  int maps, vdim;
+  float diff_lambda, diff_scale, eps;
 };
 
+constexpr float kLog2e = 1.4426950408889634f;
+
+template <bool BIAS>
 __global__ void __launch_bounds__(kGpThreads)
 gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, const GpParams p) {
@@ -51,8 +70,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int qb = p.qb, vb = p.vb;
   uint8_t* q_s = smem;
-  uint8_t* k_s = q_s + qb * kGpQBlock;                   // [2][qb] blocks
-  uint8_t* v_s = k_s + 2 * qb * kGpKvBlock;              // [2][vb] blocks
+  uint8_t* k_s = q_s + (p.q_resident ? qb : 2 * p.kb) * kGpQBlock;      // [2][kb] blocks
+  uint8_t* v_s = k_s + 2 * p.kb * kGpKvBlock;            // [2][vb] blocks
   uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * vb * kGpKvBlock);
   uint64_t* q_full = bars + 0;
   uint64_t* k_full = bars + 1;          // [2]
@@ -74,8 +93,10 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     return;
   }
   const int kv_len = min(pos0 + nrows, p.max_blocks * p.page_size);
-  const int j0 = pos0 / p.chunk * p.chunk / kGpKv;                       // first token tile
-  const int n_kv = (kv_len + kGpKv - 1) / kGpKv - j0;
+  const int j0 = p.span.first(pos0) / kGpKv;                             // first token tile of the chunk or window
+  const int n_pre = min((p.span.head(pos0 + nrows - 1) + kGpKv - 1) / kGpKv, j0);      // tiles of kept tokens before it
+  const int n_kv = n_pre + (kv_len + kGpKv - 1) / kGpKv - j0;
+  auto tile_of = [&](int j) { return j < n_pre ? j : j0 + j - n_pre; };
   if (n_kv <= 0) {
     if (tid == 0) report_status(p.status, kStatusBadIndex, 0xA81, blockIdx.x, pos0);
     return;
@@ -113,17 +134,20 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
     if (lane == 0) {
-      mbar_arrive_expect_tx(q_full, static_cast<uint32_t>(qb * p.positions * p.per * 128));
-      for (int b = 0; b < qb; ++b) tma_load_3d(q_s + b * kGpQBlock, &map_q, q_full, b * 64, g * p.per, row0);
-      const int subs = kGpKv / p.box_rows;
+      const uint32_t q_block_tx = static_cast<uint32_t>(p.positions * p.per * 128);
+      if (p.q_resident) {
+        mbar_arrive_expect_tx(q_full, qb * q_block_tx);
+        for (int b = 0; b < qb; ++b) tma_load_3d(q_s + b * kGpQBlock, &map_q, q_full, b * 64, g * p.per, row0);
+      }
+      const int subs = kGpKv / p.box_rows, key_head = p.shared_keys ? 0 : g;
       const long long n_pages = p.pool_rows / p.page_size;
       bool ok = true;
-      int armed = 0;                                                     // tiles whose copies were all requested
+      int k_armed = 0, v_armed = 0;                                      // key stages / value tiles that were requested
       for (int j = 0; j < n_kv && ok; ++j) {
         const int st = j & 1;
         int rowc[8];
         for (int s = 0; s < subs; ++s) {
-          const int t0 = (j0 + j) * kGpKv + s * p.box_rows;
+          const int t0 = tile_of(j) * kGpKv + s * p.box_rows;
           int rc = static_cast<int>(p.pool_rows);                        // out of range: the copy fills zeros
           if (t0 < kv_len) {
             const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t0 / p.page_size];
@@ -132,32 +156,39 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           }
           rowc[s] = rc;
         }
-        if (j > 1) ok = mbar_wait(k_free + st, ((j - 2) >> 1) & 1, abort_flag, p.status, 0xA90);
+        for (int c = 0; c < p.pieces && ok; ++c) {
+          const int i = j * p.pieces + c, ks = i & 1, b0 = c * p.kb, nb = min(p.kb, qb - b0);
+          if (i > 1) ok = mbar_wait(k_free + ks, ((i - 2) >> 1) & 1, abort_flag, p.status, 0xA90);
+          if (!ok) break;
+          mbar_arrive_expect_tx(k_full + ks, nb * (static_cast<uint32_t>(kGpKvBlock) + (p.q_resident ? 0u : q_block_tx)));
+          for (int s = 0; s < subs; ++s)
+            for (int b = 0; b < nb; ++b)
+              tma_load_3d(k_s + (ks * p.kb + b) * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + ks, (b0 + b) * 64, key_head,
+                          rowc[s]);
+          if (!p.q_resident)
+            for (int b = 0; b < nb; ++b)
+              tma_load_3d(q_s + (ks * p.kb + b) * kGpQBlock, &map_q, k_full + ks, (b0 + b) * 64, g * p.per, row0);
+          k_armed = i + 1;
+        }
         if (!ok) break;
-        mbar_arrive_expect_tx(k_full + st, static_cast<uint32_t>(qb * kGpKvBlock));
-        for (int s = 0; s < subs; ++s)
-          for (int b = 0; b < qb; ++b)
-            tma_load_3d(k_s + (st * qb + b) * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + st, b * 64, g, rowc[s]);
         if (j > 1) ok = mbar_wait(v_free + st, ((j - 2) >> 1) & 1, abort_flag, p.status, 0xA91);
         if (!ok) break;
         mbar_arrive_expect_tx(v_full + st, static_cast<uint32_t>(vb * kGpKvBlock));
         for (int s = 0; s < subs; ++s)
           for (int b = 0; b < vb; ++b)
             tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rowc[s]);
-        armed = j + 1;
+        v_armed = j + 1;
       }
-      // after an abort: copies of the last two tiles may still be in flight, and the CTA may not exit under them
+      // after an abort: copies of the last two stages may still be in flight, and the CTA may not exit under them
       if (*abort_flag) {
         auto drain = [&](uint64_t* bar, uint32_t parity) {
           const uint64_t t0 = globaltimer_ns();
           while (!mbar_try_wait(bar, parity) && globaltimer_ns() - t0 < 2000000ull) {
           }
         };
-        drain(q_full, 0);
-        for (int j = armed > 2 ? armed - 2 : 0; j < min(armed + 1, n_kv); ++j) {
-          drain(k_full + (j & 1), (j >> 1) & 1);
-          drain(v_full + (j & 1), (j >> 1) & 1);
-        }
+        if (p.q_resident) drain(q_full, 0);
+        for (int i = max(k_armed - 2, 0); i < k_armed; ++i) drain(k_full + (i & 1), (i >> 1) & 1);
+        for (int j = max(v_armed - 2, 0); j < v_armed; ++j) drain(v_full + (j & 1), (j >> 1) & 1);
       }
     }
   } else if (warp == 1) {
@@ -166,29 +197,35 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       const uint32_t q_addr = smem_u32(q_s), k_addr = smem_u32(k_s), v_addr = smem_u32(v_s);
       constexpr uint32_t idesc_qk = umma_idesc(kGpM, kGpKv, 1, 1);
       const uint32_t idesc_pv = umma_idesc(kGpM, static_cast<uint32_t>(vb * 64), 1, 1) | (1u << 16);   // B is MN-major
-      const int ksteps = (p.dim_pad + 15) / 16;
+      const int ksteps = (p.key_width + 15) / 16;
       auto qk = [&](int j) {
-        const uint32_t ks = k_addr + (j & 1) * qb * kGpKvBlock;
-        for (int k = 0; k < ksteps; ++k)
-          umma_bf16(tmem + col_s + (j & 1) * kGpKv, umma_desc_k128(q_addr + (k >> 2) * kGpQBlock + (k & 3) * 32),
-                    umma_desc_k128(ks + (k >> 2) * kGpKvBlock + (k & 3) * 32), idesc_qk, k > 0 ? 1u : 0u);
-        umma_commit(s_full + (j & 1));
-        umma_commit(k_free + (j & 1));
+        for (int c = 0; c < p.pieces; ++c) {
+          const int i = j * p.pieces + c, st = i & 1, k0 = c * p.kb * 4, k1 = min(k0 + p.kb * 4, ksteps);
+          if (!mbar_wait(k_full + st, (i >> 1) & 1, abort_flag, p.status, 0xAA2)) return false;
+          tc_fence_after();
+          const uint32_t ks = k_addr + st * p.kb * kGpKvBlock;
+          const uint32_t qs = p.q_resident ? q_addr + c * p.kb * kGpQBlock : q_addr + st * p.kb * kGpQBlock;
+          for (int k = k0; k < k1; ++k) {
+            const int kk = k - k0;
+            umma_bf16(tmem + col_s + (j & 1) * kGpKv, umma_desc_k128(qs + (kk >> 2) * kGpQBlock + (kk & 3) * 32),
+                      umma_desc_k128(ks + (kk >> 2) * kGpKvBlock + (kk & 3) * 32), idesc_qk, k > 0 ? 1u : 0u);
+          }
+          if (c + 1 == p.pieces) umma_commit(s_full + (j & 1));
+          umma_commit(k_free + st);
+        }
+        return true;
       };
-      bool ok = mbar_wait(q_full, 0, abort_flag, p.status, 0xAA0);
-      if (ok) ok = mbar_wait(k_full, 0, abort_flag, p.status, 0xAA1);
+      bool ok = !p.q_resident || mbar_wait(q_full, 0, abort_flag, p.status, 0xAA0);
       if (ok) {
         tc_fence_after();
-        qk(0);
+        ok = qk(0);
       }
       for (int j = 0; j < n_kv && ok; ++j) {
         const uint32_t ph = (j >> 1) & 1;
         if (j + 1 < n_kv) {
           // the score buffer of tile j + 1 held P of tile j - 1, whose product was issued before
-          ok = mbar_wait(k_full + ((j + 1) & 1), ((j + 1) >> 1) & 1, abort_flag, p.status, 0xAA2);
+          ok = qk(j + 1);
           if (!ok) break;
-          tc_fence_after();
-          qk(j + 1);
         }
         ok = mbar_wait(v_full + (j & 1), ph, abort_flag, p.status, 0xAA3);
         if (ok) ok = mbar_wait(p_full + (j & 1), ph, abort_flag, p.status, 0xAA4);
@@ -207,11 +244,12 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     // ------------------------------------------------------------------ softmax + epilogue: one row per thread
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;
-    const int at = r / p.per, head = g * p.per + r - at * p.per;
+    const int at = r / p.per, head = (g * p.per + r - at * p.per) / p.maps;
     const bool valid = at < nrows;
     const int pos = pos0 + at;
     const int hi = valid ? min(pos + 1, kv_len) : 0;
-    const int lo = pos / p.chunk * p.chunk;
+    const int lo = p.span.first(pos), keep = p.span.keep;
+    const float slope = BIAS && valid ? p.slopes[head] * kLog2e : 0.f;
     const uint32_t lane_base = tmem + (static_cast<uint32_t>(quarter * 32) << 16);
     float m_ref = -INFINITY, l_sum = 0.f;
     bool ok = true;
@@ -225,9 +263,18 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
       for (int c = 0; c < 4; ++c) tmem_ld16(s_t + c * 16, sv[c]);
       tmem_ld_wait();
-      const int tok0 = (j0 + j) * kGpKv;
+      const int tok0 = tile_of(j) * kGpKv;
       float mx = -INFINITY;
-      if (__all_sync(0xffffffffu, tok0 >= lo && tok0 + kGpKv <= hi)) {
+      if (BIAS) {
+        // the score in base 2 with its distance bias
+        const float b0 = slope * static_cast<float>(tok0 - pos);
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            sv[c][i] = __float_as_uint(fmaf(__uint_as_float(sv[c][i]), p.scale_log2, fmaf(slope, static_cast<float>(c * 16 + i), b0)));
+      }
+      if (__all_sync(0xffffffffu, tok0 + kGpKv <= hi && (tok0 >= lo || tok0 + kGpKv <= keep))) {
 #pragma unroll
         for (int c = 0; c < 4; ++c)
 #pragma unroll
@@ -238,12 +285,12 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const int t = tok0 + c * 16 + i;
-            const float x = (t >= lo && t < hi) ? __uint_as_float(sv[c][i]) : -INFINITY;
+            const float x = ((t >= lo || t < keep) && t < hi) ? __uint_as_float(sv[c][i]) : -INFINITY;
             sv[c][i] = __float_as_uint(x);
             mx = fmaxf(mx, x);
           }
       }
-      mx *= p.scale_log2;                                     // the scale is positive
+      if (!BIAS) mx *= p.scale_log2;                          // the scale is positive
       const float m_new = fmaxf(m_ref, mx);
       if (j == 0) {
         m_ref = m_new;                                        // nothing accumulated yet
@@ -273,8 +320,10 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float p0 = exp2f(fmaf(__uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]), p.scale_log2, -m_use));
-          const float p1 = exp2f(fmaf(__uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]), p.scale_log2, -m_use));
+          const float x0 = __uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]);
+          const float x1 = __uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]);
+          const float p0 = exp2f(BIAS ? x0 - m_use : fmaf(x0, p.scale_log2, -m_use));
+          const float p1 = exp2f(BIAS ? x1 - m_use : fmaf(x1, p.scale_log2, -m_use));
           add += p0 + p1;
           pk[i] = pack_bf16x2(p0, p1);
         }
@@ -293,13 +342,69 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     if (ok) {
       tc_fence_after();
       const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+      const __nv_bfloat16* gate = p.gate ? p.gate + static_cast<long long>(row0 + at) * p.ldg + static_cast<long long>(head) * p.vdim_pad
+                                         : nullptr;
+      if (p.maps == 2) {
+        // rows of a head's two maps are neighbouring lanes: both compute the difference, each writes half of it
+        const bool second = lane & 1;
+        const float own = second ? -p.diff_lambda * inv : inv;
+        float ss = 0.f;
+#pragma unroll 1
+        for (int c = 0; c < vb * 4; ++c) {
+          uint32_t ov[16];
+          tmem_ld16(lane_base + c * 16, ov);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const float x = __uint_as_float(ov[i]) * own, d = x + __shfl_xor_sync(0xffffffffu, x, 1);
+            ss = fmaf(d, d, ss);
+          }
+        }
+        const float f = p.diff_scale / sqrtf(ss / p.vdim + p.eps);
+        __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
+#pragma unroll 1
+        for (int c = 0; c < vb * 4; ++c) {
+          if (c * 16 >= p.vdim_pad) break;
+          uint32_t ov[16];
+          tmem_ld16(lane_base + c * 16, ov);
+          tmem_ld_wait();
+          float d[8];
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const float x = __uint_as_float(ov[i]) * own, y = (x + __shfl_xor_sync(0xffffffffu, x, 1)) * f;
+            if (i < 8) d[i] = y;
+            else if (second) d[i - 8] = y;
+          }
+          const int col = c * 16 + (second ? 8 : 0);
+          if (valid && col < p.vdim_pad) {
+            if (gate) {
+              float z[8];
+              act_load8(gate + col, z);
+#pragma unroll
+              for (int i = 0; i < 8; ++i) d[i] = __fdividef(d[i], 1.f + __expf(-z[i]));
+            }
+            act_store8(dst + col, d);
+          }
+        }
+      }
       __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
 #pragma unroll 1
-      for (int c = 0; c < vb * 4; ++c) {
+      for (int c = 0; c < vb * 4 && p.maps == 1; ++c) {
         if (c * 16 >= p.vdim_pad) break;
         uint32_t ov[16];
         tmem_ld16(lane_base + c * 16, ov);
         tmem_ld_wait();
+        if (valid && gate) {
+#pragma unroll
+          for (int e = 0; e < 16; e += 8) {
+            if (c * 16 + e >= p.vdim_pad) break;
+            float z[8];
+            act_load8(gate + c * 16 + e, z);
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+              ov[e + i] = __float_as_uint(__fdividef(__uint_as_float(ov[e + i]), 1.f + __expf(-z[i])));
+          }
+        }
         if (valid) {
           uint4 w0, w1;
           w0.x = pack_bf16x2(__uint_as_float(ov[0]) * inv, __uint_as_float(ov[1]) * inv);
@@ -345,31 +450,44 @@ static int gp_map(CUtensorMap* map, const void* base, int width, int heads, uint
 
 using namespace fb;
 
+template <bool BIAS>
+static int launch_gp(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const GpParams& p, int n_tiles, int smem,
+                     cudaStream_t stream) {
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(gqa_prefill_tc_kernel<BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGpSmemLimit) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  if (launch_pdl(gqa_prefill_tc_kernel<BIAS>, dim3(n_tiles, p.kv_heads), dim3(kGpThreads), smem, stream, mq, mk, mv, p) != cudaSuccess)
+    return FB_ERR_LAUNCH;
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
 extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_tiles, int tile_positions, void* stream_) {
   if (!a || !a->q || !a->pool || !a->out || !a->block_table || !tiles || a->fp32) return FB_ERR_SHAPE;
   if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->kv_heads > 65535 || n_tiles <= 0 ||
-      a->num_seqs <= 0 || a->max_blocks <= 0 || a->chunk <= 0 || !(a->scale > 0.f))
+      a->num_seqs <= 0 || a->max_blocks <= 0 || !(a->scale > 0.f) || !gqa_form_ok(a))
     return FB_ERR_SHAPE;
-  const int per = a->heads / a->kv_heads;
+  const int per = a->heads / a->kv_heads * a->maps;
   if (tile_positions <= 0 || per * tile_positions > kGpM) return FB_ERR_SHAPE;
   if (a->page_size < 8 || (a->page_size & (a->page_size - 1)) != 0) return FB_ERR_SHAPE;
-  if (a->dim_pad <= 0 || a->dim_pad > 256 || a->vdim_pad <= 0 || a->vdim_pad > 256) return FB_ERR_LIMIT;
+  if (a->vdim_pad <= 0 || a->vdim_pad > 256 || a->vdim_pad % 8) return FB_ERR_LIMIT;
   if (a->pool_rows <= 0 || a->pool_rows > 0x7fffffffLL || a->pool_rows % a->page_size) return FB_ERR_SHAPE;
-  if (a->pool_ld < static_cast<long long>(a->kv_heads) * (a->dim_pad + a->vdim_pad) ||
-      a->ldq < static_cast<long long>(a->heads) * a->dim_pad || a->ldo < static_cast<long long>(a->heads) * a->vdim_pad)
-    return FB_ERR_SHAPE;
-  if (a->ldo % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15) || (reinterpret_cast<uintptr_t>(tiles) & 15)) return FB_ERR_ALIGN;
+  if (a->ldo % 8 || a->ldg % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15) || (reinterpret_cast<uintptr_t>(a->gate) & 15) ||
+      (reinterpret_cast<uintptr_t>(tiles) & 15))
+    return FB_ERR_ALIGN;
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   GpParams p{};
   p.box_rows = a->page_size < kGpKv ? a->page_size : kGpKv;
   CUtensorMap mq, mk, mv;
-  int rc = gp_map(&mq, a->q, a->dim_pad, a->heads, static_cast<uint64_t>(a->rows), a->ldq, per, tile_positions);
+  int rc = gp_map(&mq, a->q, a->key_width, a->heads * a->maps, static_cast<uint64_t>(a->rows), a->ldq, per, tile_positions);
   if (rc != FB_OK) return rc;
   const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a->pool);
-  rc = gp_map(&mk, pool, a->dim_pad, a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
+  p.shared_keys = a->key_stride == 0;
+  rc = gp_map(&mk, pool, a->key_width, p.shared_keys ? 1 : a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
   if (rc != FB_OK) return rc;
-  rc = gp_map(&mv, pool + static_cast<long long>(a->kv_heads) * a->dim_pad, a->vdim_pad, a->kv_heads,
-              static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
+  rc = gp_map(&mv, pool + a->v_offset, a->vdim_pad, a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
   if (rc != FB_OK) return rc;
   p.tiles = tiles;
   p.block_table = a->block_table;
@@ -377,20 +495,26 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   p.status = static_cast<DeviceStatus*>(a->status);
   p.pool_rows = a->pool_rows;
   p.rows = a->rows; p.heads = a->heads; p.kv_heads = a->kv_heads; p.per = per; p.positions = tile_positions;
-  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size; p.chunk = a->chunk;
-  p.dim_pad = a->dim_pad; p.vdim_pad = a->vdim_pad;
-  p.qb = (a->dim_pad + 63) / 64; p.vb = (a->vdim_pad + 63) / 64;
+  p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
+  p.span = {a->chunk, a->window, a->keep_first};
+  p.key_width = a->key_width; p.vdim_pad = a->vdim_pad;
+  p.qb = (a->key_width + 63) / 64; p.vb = (a->vdim_pad + 63) / 64;
   p.tmem_cols = p.vb * 64 + 2 * kGpKv <= 256 ? 256 : 512;
-  p.scale_log2 = a->scale * 1.4426950408889634f;
-  const int smem = p.qb * kGpQBlock + 2 * (p.qb + p.vb) * kGpKvBlock + 1024 + 256;
-  static bool attr = false;
-  if (!attr) {
-    const int most = 4 * kGpQBlock + 16 * kGpKvBlock + 1024 + 256;
-    if (cudaFuncSetAttribute(gqa_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess)
-      return FB_ERR_LAUNCH;
-    attr = true;
+  p.scale_log2 = a->scale * kLog2e;
+  p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
+  p.maps = a->maps; p.vdim = a->vdim;
+  p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale; p.eps = a->eps;
+  // key stages as wide as fit beside the query rows; rows too wide to stay are streamed with the keys
+  int smem = 0;
+  for (int form = 0; form < 6; ++form) {
+    p.q_resident = form < 3;
+    p.kb = p.q_resident ? 4 >> form : 4 >> (form - 3);
+    if (p.kb > p.qb && p.kb > 1 && p.q_resident) p.kb = p.qb;
+    smem = (p.q_resident ? p.qb : 2 * p.kb) * kGpQBlock + 2 * (p.kb + p.vb) * kGpKvBlock + 1024 + 256;
+    if (smem <= kGpSmemLimit) break;
+    smem = 0;
   }
-  if (launch_pdl(gqa_prefill_tc_kernel, dim3(n_tiles, a->kv_heads), dim3(kGpThreads), smem, stream, mq, mk, mv, p) != cudaSuccess)
-    return FB_ERR_LAUNCH;
-  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  if (smem == 0) return FB_ERR_LIMIT;
+  p.pieces = (p.qb + p.kb - 1) / p.kb;
+  return a->slopes ? launch_gp<true>(mq, mk, mv, p, n_tiles, smem, stream) : launch_gp<false>(mq, mk, mv, p, n_tiles, smem, stream);
 }

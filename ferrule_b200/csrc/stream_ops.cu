@@ -1,10 +1,12 @@
-// Row operators of output-norm blocks (32-bit residual stream, a norm on every sublayer's output): embedding with
-// learned positions, norm and residual addition, short causal convolutions over packed sequences.
+// Row operators of output-norm and sandwich blocks (32-bit residual stream, a norm on every sublayer's output): embedding,
+// learned positions, norms and residual addition, short causal convolutions over packed sequences.
 //
 //   fb_stream_step  x = table[id] + pos[p]  or  x += norm(y); also the new rows as activations, and in decode steps (one
 //                   row per sequence) the next mixer's input h = x + conv(x) with the convolution state
 //   fb_short_conv   the convolution over any mix of row counts; its state is the last taps - 1 inputs of a sequence
 //   fb_norm_rows    norm of selected rows (the rows whose logits are wanted)
+//   fb_sandwich_step, fb_sandwich_rows   the same for RMS norms of equal parts of a row, with the norm in front of the next
+//                   sublayer and the embedding that a new pass over looped layers adds
 //
 // State of a convolution: buffer `state_in[seq]` is read (-1: a new sequence, zeros), buffer `state_out[seq]` written
 // (-1: nothing is kept), never the same one.
@@ -192,6 +194,204 @@ norm_rows_kernel(const float* __restrict__ x, long long ldx, int x_rows, const i
 #pragma unroll
     for (int j = 0; j < 8; ++j) o[j] = i + j < dim ? fmaf((v[k][j] - mean) * inv, w[j], b[j]) : 0.f;
     act_store8(out + blockIdx.x * ldo + i, o);
+  }
+}
+
+// ---------------------------------------------------------------------------------
+// RMS norm of `groups` equal parts of a row
+// ---------------------------------------------------------------------------------
+// shared memory of one CTA: sums of squares of 8 elements each (of single ones when a part is no multiple of 8), then the
+// inverse root mean square of every part
+struct GroupScratch {
+  float* sums;
+  float* inv;
+  float (*red)[32];
+};
+
+template <int VPT>
+__device__ __forceinline__ void group_norm(const float (&v)[VPT][8], int dim, int groups, float eps, const GroupScratch& g,
+                                           int turn, float (&out)[VPT][8]) {
+  const int part = dim / groups;
+  if (groups == 1) {
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[k][j], v[k][j], ss);      // columns past `dim` are zero
+    const float f = 1.f / sqrtf(cta_sum(ss, g.red[turn]) / dim + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) out[k][j] = v[k][j] * f;
+    return;
+  }
+  const bool aligned = part % 8 == 0;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+    if (i >= dim) continue;
+    if (aligned) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[k][j], v[k][j], ss);
+      g.sums[i / 8] = ss;
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (i + j < dim) g.sums[i + j] = v[k][j] * v[k][j];
+    }
+  }
+  __syncthreads();
+  const int n = aligned ? part / 8 : part, lane = threadIdx.x & 31;
+  for (int p = threadIdx.x >> 5; p < groups; p += blockDim.x >> 5) {
+    float ss = 0.f;
+    for (int i = lane; i < n; i += 32) ss += g.sums[p * n + i];
+    ss = warp_sum(ss);
+    if (lane == 0) g.inv[p] = 1.f / sqrtf(ss / part + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+    const float f = i < dim ? g.inv[i / part] : 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      out[k][j] = v[k][j] * (aligned || i + j >= dim ? f : g.inv[(i + j) / part]);
+  }
+}
+
+template <typename T>
+struct SandwichParams {
+  float* x;
+  long long ldx;
+  const T* y;
+  long long ldy;
+  const float* y_bias;
+  const float* out_w;
+  const int* ids;
+  const T* table;
+  long long ldt;
+  int vocab, fresh;
+  const float* in_w;
+  T* act;
+  long long lda;
+  int dim, dim_pad, groups, n_sums;
+  float eps;
+  DeviceStatus* status;
+};
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(kRowThreads)
+sandwich_step_kernel(const SandwichParams<T> p) {
+  pdl_launch_dependents();
+  extern __shared__ float group_sm[];
+  __shared__ float red[2][32];
+  const GroupScratch g{group_sm, group_sm + p.n_sums, red};
+  const int r = blockIdx.x;
+  pdl_wait();
+  float v[VPT][8], y[VPT][8];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] = y[k][j] = 0.f;
+    if (i >= p.dim_pad) continue;
+    if (!p.fresh) act_load8(p.x + r * p.ldx + i, v[k]);
+    if (p.y) act_load8(p.y + r * p.ldy + i, y[k]);
+  }
+  if (p.y) {
+    if (p.y_bias) {
+#pragma unroll
+      for (int k = 0; k < VPT; ++k) {
+        const int i = (k * blockDim.x + threadIdx.x) * 8;
+        if (i >= p.dim_pad) continue;
+        float b[8];
+        act_load8(p.y_bias + i, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) y[k][j] += b[j];
+      }
+    }
+    group_norm<VPT>(y, p.dim, p.groups, p.eps, g, 0, y);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      if (i >= p.dim_pad) continue;
+      float w[8];
+      act_load8(p.out_w + i, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] = fmaf(y[k][j], w[j], v[k][j]);
+    }
+  }
+  if (p.ids) {
+    int id = p.ids[r];
+    if (id < 0 || id >= p.vocab) {
+      if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD30, r, id);
+      id = 0;
+    }
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      if (i >= p.dim_pad) continue;
+      float e[8];
+      act_load8(p.table + id * p.ldt + i, e);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] += e[j];
+    }
+  }
+  if (p.y || p.ids) {
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      if (i < p.dim_pad) act_store8(p.x + r * p.ldx + i, v[k]);
+    }
+  }
+  if (!p.act) return;
+  group_norm<VPT>(v, p.dim, p.groups, p.eps, g, 1, v);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+    if (i >= p.dim_pad) continue;
+    float w[8];
+    act_load8(p.in_w + i, w);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] *= w[j];
+    act_store8(p.act + r * p.lda + i, v[k]);
+  }
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(kRowThreads)
+sandwich_rows_kernel(const float* __restrict__ x, long long ldx, int x_rows, const int* __restrict__ rows_idx,
+                     const float* __restrict__ w_in, T* __restrict__ out, long long ldo, int dim, int dim_pad, int groups,
+                     int n_sums, float eps, DeviceStatus* st) {
+  pdl_launch_dependents();
+  extern __shared__ float group_sm[];
+  __shared__ float red[2][32];
+  const GroupScratch g{group_sm, group_sm + n_sums, red};
+  pdl_wait();
+  int r = rows_idx[blockIdx.x];
+  if (r < 0 || r >= x_rows) {
+    if (threadIdx.x == 0) report_status(st, kStatusBadIndex, 0xD31, blockIdx.x, r);
+    r = 0;
+  }
+  float v[VPT][8];
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
+    if (i < dim_pad) act_load8(x + r * ldx + i, v[k]);
+  }
+  group_norm<VPT>(v, dim, groups, eps, g, 0, v);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (k * blockDim.x + threadIdx.x) * 8;
+    if (i >= dim_pad) continue;
+    float w[8];
+    act_load8(w_in + i, w);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] *= w[j];
+    act_store8(out + blockIdx.x * ldo + i, v[k]);
   }
 }
 
@@ -480,6 +680,95 @@ extern "C" int fb_norm_rows(const float* x, long long ldx, int x_rows, const int
   return fp32 ? launch_norm_rows<float>(x, ldx, x_rows, rows_idx, n, norm_w, norm_b, rms, out, ldo, dim, dim_pad, eps, status, s)
               : launch_norm_rows<__nv_bfloat16>(x, ldx, x_rows, rows_idx, n, norm_w, norm_b, rms, out, ldo, dim, dim_pad, eps,
                                                 status, s);
+}
+
+// floats of sums in shared memory (and one inverse per part behind them)
+static int group_sums(int dim, int groups) { return groups == 1 ? 0 : dim / groups % 8 ? dim : dim / 8; }
+
+template <typename T, int VPT>
+static int launch_sandwich(const SandwichParams<T>& p, int rows, cudaStream_t s) {
+  const size_t smem = (p.n_sums + p.groups) * sizeof(float);
+  if (smem > 160 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (smem > 40 * 1024 && !attr) {
+    if (cudaFuncSetAttribute(sandwich_step_kernel<T, VPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(sandwich_step_kernel<T, VPT>, dim3(rows), dim3(row_threads(p.dim_pad)), smem, s, p);
+  return ok_launch();
+}
+
+template <typename T>
+static int run_sandwich(const FbSandwichArgs* a, cudaStream_t s) {
+  SandwichParams<T> p{};
+  p.x = a->x; p.ldx = a->ldx;
+  p.y = static_cast<const T*>(a->y); p.ldy = a->ldy; p.y_bias = a->y_bias; p.out_w = a->out_w;
+  p.ids = a->ids; p.table = static_cast<const T*>(a->table); p.ldt = a->ldt; p.vocab = a->vocab; p.fresh = a->fresh;
+  p.in_w = a->in_w; p.act = static_cast<T*>(a->act); p.lda = a->lda;
+  p.dim = a->dim; p.dim_pad = a->dim_pad; p.groups = a->groups; p.n_sums = group_sums(a->dim, a->groups); p.eps = a->eps;
+  p.status = static_cast<DeviceStatus*>(a->status);
+  switch (row_vpt(a->dim_pad)) {
+    case 1: return launch_sandwich<T, 1>(p, a->rows, s);
+    case 2: return launch_sandwich<T, 2>(p, a->rows, s);
+    case 4: return launch_sandwich<T, 4>(p, a->rows, s);
+    case 8: return launch_sandwich<T, 8>(p, a->rows, s);
+    default: return FB_ERR_LIMIT;
+  }
+}
+
+extern "C" int fb_sandwich_step(const FbSandwichArgs* a, void* stream) {
+  if (!a || !a->x || a->rows <= 0 || a->dim <= 0 || a->dim_pad < a->dim || a->dim_pad % 8 || a->ldx < a->dim_pad || a->ldx % 8 ||
+      a->groups <= 0 || a->dim % a->groups)
+    return FB_ERR_SHAPE;
+  if (a->y && (!a->out_w || a->ldy < a->dim_pad || a->ldy % 8)) return FB_ERR_SHAPE;
+  if (a->ids && (!a->table || a->ldt < a->dim_pad || a->ldt % 8 || a->vocab <= 0)) return FB_ERR_SHAPE;
+  if (!a->act != !a->in_w || (a->act && (a->lda < a->dim_pad || a->lda % 8))) return FB_ERR_SHAPE;
+  if (!aligned16(a->x) || !aligned16(a->y) || !aligned16(a->y_bias) || !aligned16(a->out_w) || !aligned16(a->table) ||
+      !aligned16(a->in_w) || !aligned16(a->act))
+    return FB_ERR_ALIGN;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return a->fp32 ? run_sandwich<float>(a, s) : run_sandwich<__nv_bfloat16>(a, s);
+}
+
+template <typename T, int VPT>
+static int launch_sandwich_rows(const float* x, long long ldx, int x_rows, const int* idx, int n, const float* w, void* out,
+                                long long ldo, int dim, int dim_pad, int groups, float eps, void* status, cudaStream_t s) {
+  const int n_sums = group_sums(dim, groups);
+  const size_t smem = (n_sums + groups) * sizeof(float);
+  if (smem > 160 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (smem > 40 * 1024 && !attr) {
+    if (cudaFuncSetAttribute(sandwich_rows_kernel<T, VPT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(sandwich_rows_kernel<T, VPT>, dim3(n), dim3(row_threads(dim_pad)), smem, s, x, ldx, x_rows, idx, w,
+             static_cast<T*>(out), ldo, dim, dim_pad, groups, n_sums, eps, static_cast<DeviceStatus*>(status));
+  return ok_launch();
+}
+
+template <typename T>
+static int run_sandwich_rows(const float* x, long long ldx, int x_rows, const int* idx, int n, const float* w, void* out,
+                             long long ldo, int dim, int dim_pad, int groups, float eps, void* status, cudaStream_t s) {
+  switch (row_vpt(dim_pad)) {
+    case 1: return launch_sandwich_rows<T, 1>(x, ldx, x_rows, idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s);
+    case 2: return launch_sandwich_rows<T, 2>(x, ldx, x_rows, idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s);
+    case 4: return launch_sandwich_rows<T, 4>(x, ldx, x_rows, idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s);
+    case 8: return launch_sandwich_rows<T, 8>(x, ldx, x_rows, idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s);
+    default: return FB_ERR_LIMIT;
+  }
+}
+
+extern "C" int fb_sandwich_rows(const float* x, long long ldx, int x_rows, const int* rows_idx, int n, const float* w, void* out,
+                                long long ldo, int dim, int dim_pad, int groups, float eps, int fp32, void* status, void* stream) {
+  if (!x || !rows_idx || !w || !out || n <= 0 || x_rows <= 0 || dim <= 0 || dim_pad < dim || dim_pad % 8 || ldx < dim_pad ||
+      ldo < dim_pad || ldx % 8 || ldo % 8 || groups <= 0 || dim % groups)
+    return FB_ERR_SHAPE;
+  if (!aligned16(x) || !aligned16(w) || !aligned16(out)) return FB_ERR_ALIGN;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return fp32 ? run_sandwich_rows<float>(x, ldx, x_rows, rows_idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s)
+              : run_sandwich_rows<__nv_bfloat16>(x, ldx, x_rows, rows_idx, n, w, out, ldo, dim, dim_pad, groups, eps, status, s);
 }
 
 template <typename TI, typename TO, int KEEP, int ROWS>

@@ -76,7 +76,7 @@ class AttentionMixer:
     kind = "attention"
     maps = 1
     window = keep_first = 0
-    shared_keys = False
+    shared_keys = scaled_queries = False
 
     @property
     def dim_pad(self) -> int:
@@ -122,6 +122,7 @@ class WindowMixer:
     gate: bool = False             # output multiplied by sigmoid(W_g h), element by element
 
     chunk = 0
+    scaled_queries = True          # the scale is part of the queries the attention kernels read
 
     @property
     def kind(self) -> str:

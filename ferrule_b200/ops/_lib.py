@@ -156,7 +156,31 @@ class GqaArgs(C.Structure):
         ("num_seqs", C.c_int), ("max_blocks", C.c_int), ("page_size", C.c_int), ("chunk", C.c_int),
         ("scale", C.c_float), ("eps", C.c_float), ("out", C.c_void_p), ("ldo", C.c_longlong),
         ("rows", C.c_int), ("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int),
-        ("vdim", C.c_int), ("vdim_pad", C.c_int), ("fp32", C.c_int), ("status", C.c_void_p),
+        ("vdim", C.c_int), ("vdim_pad", C.c_int), ("fp32", C.c_int), ("maps", C.c_int), ("key_width", C.c_int),
+        ("key_stride", C.c_int), ("v_offset", C.c_int), ("window", C.c_int), ("keep_first", C.c_int),
+        ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ldg", C.c_longlong), ("diff_lambda", C.c_float),
+        ("diff_scale", C.c_float), ("status", C.c_void_p),
+    ]
+
+
+class SandwichArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("ldx", C.c_longlong), ("y", C.c_void_p), ("ldy", C.c_longlong), ("y_bias", C.c_void_p),
+        ("out_w", C.c_void_p), ("ids", C.c_void_p), ("table", C.c_void_p), ("ldt", C.c_longlong), ("vocab", C.c_int),
+        ("fresh", C.c_int), ("in_w", C.c_void_p), ("act", C.c_void_p), ("lda", C.c_longlong), ("rows", C.c_int),
+        ("dim", C.c_int), ("dim_pad", C.c_int), ("groups", C.c_int), ("fp32", C.c_int), ("eps", C.c_float),
+        ("status", C.c_void_p),
+    ]
+
+
+class HeadPrepArgs(C.Structure):
+    _fields_ = [
+        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ldp", C.c_longlong), ("q_bias", C.c_void_p),
+        ("k_bias", C.c_void_p), ("q_norm", C.c_void_p), ("k_norm", C.c_void_p), ("q_mix", C.c_void_p), ("mix", C.c_int),
+        ("q_out", C.c_void_p), ("ldqo", C.c_longlong), ("write_slot", C.c_void_p), ("pool", C.c_void_p),
+        ("pool_rows", C.c_longlong), ("pool_ld", C.c_longlong), ("rows", C.c_int), ("heads", C.c_int),
+        ("kv_heads", C.c_int), ("maps", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int),
+        ("fp32", C.c_int), ("eps", C.c_float), ("status", C.c_void_p),
     ]
 
 

@@ -74,7 +74,7 @@ def declare(lib) -> None:
         "fb_latent_attention": ([vp, i, vp], i),
         "fb_delta_decode": ([vp, vp], i),
         "fb_delta_prefill": ([vp, vp], i),
-        # stream_ops.cu, selective_scan.cu, gqa_attention.cu
+        # stream_ops.cu, selective_scan.cu, gqa_*.cu, head_prep.cu
         "fb_stream_step": ([vp, vp], i),
         "fb_norm_rows": ([vp, ll, i, vp, i, vp, vp, i, vp, ll, i, i, f, i, vp, vp], i),
         "fb_short_conv": ([vp, vp], i),
@@ -82,7 +82,12 @@ def declare(lib) -> None:
         "fb_gqa_prep": ([vp, vp], i),
         "fb_gqa_attention": ([vp, vp], i),
         "fb_gqa_decode": ([vp, i, i, vp], i),
+        "fb_gqa_decode_wide": ([vp, i, i, vp], i),
+        "fb_gqa_decode_wide_ok": ([i, i, i], i),
         "fb_gqa_prefill_tc": ([vp, vp, i, i, vp], i),
+        "fb_head_prep": ([vp, vp], i),
+        "fb_sandwich_step": ([vp, vp], i),
+        "fb_sandwich_rows": ([vp, ll, i, vp, i, vp, vp, ll, i, i, i, f, i, vp, vp], i),
         # v4_ops.cu
         "fb_hc_pre": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, vp], i),
         "fb_hc_pre_split": ([vp, vp, vp, vp, vp, i, vp, i, i, i, i, f, f, i, i, vp, vp, vp], i),

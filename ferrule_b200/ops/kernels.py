@@ -20,7 +20,7 @@ import torch
 from . import _lib
 from ._lib import AttnArgs, GemmArgs, check, get_lib, ptr, status_tensor, stream_ptr
 
-EPI_STORE, EPI_SWIGLU, EPI_SCATTER, EPI_ALLREDUCE, EPI_GELU = 0, 1, 2, 3, 4
+EPI_STORE, EPI_SWIGLU, EPI_SCATTER, EPI_ALLREDUCE, EPI_GELU, EPI_GEGLU = 0, 1, 2, 3, 4, 5
 
 
 def pick_ntok(rows: int, dual: bool = False) -> int:
@@ -77,7 +77,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
 
     x [rows, K] bf16 (row stride arbitrary multiple of 8), w [N, K] or [groups, N, K] bf16.
     plan        : grouped mode, x rows are in expert-major order.
-    epilogue    : EPI_STORE | EPI_GELU | EPI_SWIGLU (w rows = [gate block | up block]) | EPI_SCATTER |
+    epilogue    : EPI_STORE | EPI_GELU | EPI_SWIGLU, EPI_GEGLU (w rows = [gate block | up block]) | EPI_SCATTER |
                   EPI_ALLREDUCE (comm = a parallel.symm.AllReduceChannel).
     x_group_koff: batched mode (groups > 1 without a plan): group g reads x[:, g*koff : g*koff+K]
                   and writes out[:, g*out_group_coff : +N].
@@ -91,7 +91,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     w, groups, w_rows, wk, ldw, gstride = _w3(w)
     K = wk if k is None else k
     rows = x.shape[0]
-    dual = epilogue == EPI_SWIGLU
+    dual = epilogue in (EPI_SWIGLU, EPI_GEGLU)
     if n_out is None:
         n_out = w_rows // 2 if dual else w_rows
     if dual and dual_offset == 0:

@@ -1,17 +1,19 @@
 """Launchers of the layer-list model kernels (csrc/layered_ops.cu, stream_ops.cu, delta_rule.cu, selective_scan.cu,
-gqa_attention.cu).
+gqa_*.cu, head_prep.cu).
 
 Activations are bf16, or fp32 for models that run in full 32 bits: the launcher follows the tensors' dtype.
 """
 from __future__ import annotations
 
 import ctypes as C
+import functools
 from typing import Optional
 
 import torch
 
 from . import _lib
-from ._lib import AttnArgs, ConvArgs, DeltaArgs, GqaArgs, LayerTailArgs, ScanArgs, StreamArgs, check, get_lib, ptr, status_tensor, stream_ptr
+from ._lib import (AttnArgs, ConvArgs, DeltaArgs, GqaArgs, HeadPrepArgs, LayerTailArgs, SandwichArgs, ScanArgs, StreamArgs, check,
+                   get_lib, ptr, status_tensor, stream_ptr)
 
 
 def _fp32(t: torch.Tensor) -> int:
@@ -210,6 +212,39 @@ def norm_rows(x: torch.Tensor, rows: torch.Tensor, norm: torch.Tensor, out: torc
     return out
 
 
+def sandwich_step(x: torch.Tensor, *, dim: int, eps: float, groups: int, y: Optional[torch.Tensor] = None,
+                  bias: Optional[torch.Tensor] = None, out_norm: Optional[torch.Tensor] = None,
+                  ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, fresh: bool = False,
+                  in_norm: Optional[torch.Tensor] = None, act: Optional[torch.Tensor] = None) -> None:
+    """x (zeros when `fresh`) += norm(y + bias) * out_norm + table[ids]; act = norm(x) * in_norm.  Every norm divides each of
+    `groups` equal parts of a row by its own root mean square."""
+    a = SandwichArgs()
+    assert x.dtype == torch.float32 and dim % groups == 0 and (act is None) == (in_norm is None)
+    like = next(t for t in (y, table, act) if t is not None)
+    a.x, a.ldx, a.rows, a.dim, a.dim_pad, a.groups, a.eps, a.fp32 = (x.data_ptr(), x.stride(0), x.shape[0], dim, x.shape[1],
+                                                                     groups, eps, _fp32(like))
+    if y is not None:
+        a.y, a.ldy, a.out_w, a.y_bias = y.data_ptr(), y.stride(0), out_norm.data_ptr(), ptr(bias)
+    if ids is not None:
+        assert table.dtype == like.dtype
+        a.ids, a.table, a.ldt, a.vocab = ids.data_ptr(), table.data_ptr(), table.stride(0), table.shape[0]
+    if act is not None:
+        assert act.dtype == like.dtype
+        a.in_w, a.act, a.lda = in_norm.data_ptr(), act.data_ptr(), act.stride(0)
+    a.fresh, a.status = int(fresh), status_tensor(x.device).data_ptr()
+    check(get_lib(True).fb_sandwich_step(C.byref(a), stream_ptr()), "fb_sandwich_step")
+
+
+def sandwich_rows(x: torch.Tensor, rows: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, dim: int, eps: float,
+                  groups: int) -> torch.Tensor:
+    """out[i] = norm(x[rows[i]]) (see `sandwich_step`)."""
+    assert x.dtype == torch.float32 and rows.dtype == torch.int32 and out.shape[0] == rows.shape[0] and dim % groups == 0
+    check(get_lib(True).fb_sandwich_rows(x.data_ptr(), x.stride(0), x.shape[0], rows.data_ptr(), rows.shape[0],
+                                         norm.data_ptr(), out.data_ptr(), out.stride(0), dim, x.shape[1], groups, eps,
+                                         _fp32(out), status_tensor(x.device).data_ptr(), stream_ptr()), "fb_sandwich_rows")
+    return out
+
+
 def short_conv(x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, out: torch.Tensor, row_seq: torch.Tensor,
                seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, *,
                bias: Optional[torch.Tensor] = None, residual: bool = False, silu: bool = False) -> torch.Tensor:
@@ -247,17 +282,50 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, off_b: in
     return out
 
 
-# ------------------------------------------------------------------ grouped-query attention in position chunks
-def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor) -> GqaArgs:
+# ------------------------------------------------------------------ grouped-query attention in chunks and windows
+def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor, slopes: Optional[torch.Tensor] = None,
+         gate: Optional[torch.Tensor] = None, diff_lambda: float = 0.0, eps: float = 0.0) -> GqaArgs:
     a = GqaArgs()
     assert q.dtype == pool.dtype and pool.is_contiguous()
     a.q, a.ldq, a.rows, a.fp32 = q.data_ptr(), q.stride(0), q.shape[0], _fp32(q)
     a.pool, a.pool_ld, a.pool_rows = pool.data_ptr(), pool.shape[-1], pool.numel() // pool.shape[-1]
     a.heads, a.kv_heads, a.dim, a.vdim, a.dim_pad, a.vdim_pad = (mixer.heads, mixer.kv_heads, mixer.dim, mixer.vdim,
                                                                  mixer.dim_pad, mixer.vdim_pad)
-    a.chunk, a.scale, a.rot_dims = mixer.chunk, mixer.scale, mixer.rot_dims
+    a.chunk, a.window, a.keep_first = mixer.chunk, mixer.window, mixer.keep_first
+    a.maps, a.key_width, a.v_offset = mixer.maps, mixer.key_width, mixer.v_offset
+    a.key_stride = 0 if mixer.shared_keys else mixer.key_width
+    a.slopes, a.eps, a.diff_lambda = ptr(slopes), eps, diff_lambda
+    a.diff_scale = 1.0 - mixer.diff if mixer.maps == 2 else 1.0
+    if gate is not None:
+        assert gate.dtype == q.dtype
+        a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
     a.status = status_tensor(q.device).data_ptr()
     return a
+
+
+def _scaled(a: GqaArgs, mixer) -> GqaArgs:
+    """Scale of the products q . k: queries that `head_prep` wrote carry theirs."""
+    a.scale = 1.0 if mixer.scaled_queries else mixer.scale
+    return a
+
+
+def head_prep(proj: torch.Tensor, off, mixer, img, write_slot: torch.Tensor, pool: torch.Tensor, eps: float,
+              q_out: torch.Tensor) -> None:
+    """Between the projection and window attention: biases, query and key norm per head, factors and mixing of the queries
+    across heads (into q_out), cache append of keys and values."""
+    assert proj.dtype == pool.dtype == q_out.dtype and pool.is_contiguous() and write_slot.dtype == torch.int64
+    a = HeadPrepArgs()
+    item = proj.element_size()
+    at = lambda name: proj.data_ptr() + off[name] * item
+    a.q, a.k, a.v, a.ldp = at("q"), at("k"), None if mixer.tied_values else at("v"), proj.stride(0)
+    a.q_bias, a.k_bias, a.q_norm, a.k_norm = ptr(img.q_bias), ptr(img.k_bias), img.q_norm.data_ptr(), img.k_norm.data_ptr()
+    a.q_mix, a.mix, a.q_out, a.ldqo = img.q_mix.data_ptr(), int(mixer.mix_heads), q_out.data_ptr(), q_out.stride(0)
+    a.write_slot, a.pool, a.pool_ld, a.pool_rows = (write_slot.data_ptr(), pool.data_ptr(), pool.shape[-1],
+                                                    pool.numel() // pool.shape[-1])
+    a.rows, a.heads, a.kv_heads, a.maps, a.dim, a.dim_pad, a.vdim_pad = (proj.shape[0], mixer.heads, mixer.kv_heads, mixer.maps,
+                                                                         mixer.dim, mixer.dim_pad, mixer.vdim_pad)
+    a.fp32, a.eps, a.status = _fp32(proj), eps, status_tensor(proj.device).data_ptr()
+    check(get_lib(True).fb_head_prep(C.byref(a), stream_ptr()), "fb_head_prep")
 
 
 def gqa_prep(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, mixer, img, rotation, positions: torch.Tensor,
@@ -266,12 +334,13 @@ def gqa_prep(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, mixer, img, rota
     """Query rows are normalised and rotated in place; keys and values go into the pool rows of their tokens.
     rotation = (cos, sin) fp32 [positions, rot_dims / 2]; first_pool: the pool of the layer whose values are mixed in, at
     column first_off."""
-    a = _gqa(q, mixer, pool)
+    a = _scaled(_gqa(q, mixer, pool), mixer)
     assert k.stride(0) == v.stride(0)
     a.k, a.v, a.ldkv = k.data_ptr(), v.data_ptr(), k.stride(0)
     a.q_norm, a.k_norm = img.q_norm.data_ptr(), img.k_norm.data_ptr()
     a.cos_t, a.sin_t, a.max_pos = rotation[0].data_ptr(), rotation[1].data_ptr(), rotation[0].shape[0]
     a.positions, a.write_slot, a.eps = positions.data_ptr(), write_slot.data_ptr(), eps
+    a.rot_dims = mixer.rot_dims
     if first_pool is not None:
         assert first_pool.shape == pool.shape
         a.first_pool, a.first_off, a.v_mix = first_pool.data_ptr(), first_off, img.v_mix
@@ -287,45 +356,62 @@ def _gqa_rows(a: GqaArgs, block_table, row_seq, row_pos, page_size: int, out: to
 
 
 def gqa_attention(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
-                  row_pos: torch.Tensor, page_size: int, out: torch.Tensor) -> torch.Tensor:
-    """32-bit arithmetic: out [rows, heads * vdim_pad]."""
-    a = _gqa(q, mixer, pool)
+                  row_pos: torch.Tensor, page_size: int, out: torch.Tensor, **form) -> torch.Tensor:
+    """32-bit arithmetic: out [rows, heads * vdim_pad].  form: slopes, gate, diff_lambda, eps of a window mixer."""
+    a = _scaled(_gqa(q, mixer, pool, **form), mixer)
     _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
     check(get_lib(True).fb_gqa_attention(C.byref(a), stream_ptr()), "fb_gqa_attention")
     return out
 
 
 def gqa_tc_group(mixer, dtype, page_size: int) -> int:
-    """Query heads per key / value head when the bf16 kernels serve the mixer's prompts, else 0."""
-    per = mixer.heads // mixer.kv_heads
-    ok = (dtype == torch.bfloat16 and max(mixer.dim_pad, mixer.vdim_pad) <= 256 and per <= 128 and mixer.scale > 0
+    """Query rows per key / value head when the bf16 prompt kernel serves the mixer, else 0."""
+    per = mixer.heads // mixer.kv_heads * mixer.maps
+    ok = (dtype == torch.bfloat16 and mixer.vdim_pad <= 256 and per <= 128
+          and (mixer.shared_keys or mixer.key_width <= 256) and (mixer.scaled_queries or mixer.scale > 0)
           and page_size >= 8 and page_size & (page_size - 1) == 0)
     return per if ok else 0
 
 
+@functools.lru_cache(maxsize=None)
+def gqa_decode_supported(mixer, dtype, page_size: int) -> bool:
+    """Whether the bf16 kernels for few rows serve the mixer."""
+    if dtype != torch.bfloat16:
+        return False
+    if mixer.shared_keys:
+        return bool(get_lib(True).fb_gqa_decode_wide_ok(mixer.key_width, mixer.kv_heads, mixer.vdim_pad))
+    return max(mixer.key_width, mixer.vdim_pad) <= 256
+
+
 def gqa_decode_splits(rows: int, mixer, max_keys: int) -> int:
-    """CTAs per row: about two per SM over the batch, each with at least 128 keys of the longest row."""
-    ctas = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads + 15) // 16)
+    """CTAs per row: about two per SM over the batch (one where a CTA takes all kv heads), each with at least 128 (64) keys of
+    the longest row."""
+    if mixer.shared_keys:
+        ctas, fill, least = rows * ((mixer.heads + 15) // 16), 148, 64
+    else:
+        ctas, fill, least = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads * mixer.maps + 15) // 16), 296, 128
+    visible = mixer.chunk or mixer.window + mixer.keep_first
     splits = 1
-    while splits < 8 and ctas * splits * 2 <= 296 and min(mixer.chunk, max_keys) >= splits * 2 * 128:
+    while splits < 8 and ctas * splits * 2 <= fill and min(visible, max_keys) >= splits * 2 * least:
         splits *= 2
     return splits
 
 
 def gqa_decode(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
-               row_pos: torch.Tensor, page_size: int, out: torch.Tensor, splits: int = 1, decode_only: bool = False
+               row_pos: torch.Tensor, page_size: int, out: torch.Tensor, splits: int = 1, decode_only: bool = False, **form
                ) -> torch.Tensor:
     """Few query rows, bf16.  decode_only: one row per sequence, every key below its position predates the running step."""
-    a = _gqa(q, mixer, pool)
+    a = _scaled(_gqa(q, mixer, pool, **form), mixer)
     _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
-    check(get_lib(True).fb_gqa_decode(C.byref(a), splits, 1 if decode_only else 0, stream_ptr()), "fb_gqa_decode")
+    name = "fb_gqa_decode_wide" if mixer.shared_keys else "fb_gqa_decode"
+    check(getattr(get_lib(True), name)(C.byref(a), splits, 1 if decode_only else 0, stream_ptr()), name)
     return out
 
 
 def gqa_prefill_tc(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor, n_tiles: int,
-                   tile_positions: int, page_size: int, out: torch.Tensor) -> torch.Tensor:
+                   tile_positions: int, page_size: int, out: torch.Tensor, **form) -> torch.Tensor:
     """Prompt rows on tcgen05, bf16: tiles as `kernels.prefill_tiles` makes them; rows no tile covers are left alone."""
-    a = _gqa(q, mixer, pool)
+    a = _scaled(_gqa(q, mixer, pool, **form), mixer)
     _gqa_rows(a, block_table, None, None, page_size, out)
     assert tiles.dtype == torch.int32 and tiles.shape[1] == 4 and tiles.is_contiguous() and n_tiles <= tiles.shape[0]
     check(get_lib(True).fb_gqa_prefill_tc(C.byref(a), tiles.data_ptr(), n_tiles, tile_positions, stream_ptr()),
