@@ -351,6 +351,12 @@ __host__ __device__ constexpr uint32_t umma_idesc(uint32_t m, uint32_t n, uint32
 __device__ __forceinline__ float bf16_round(float x) {
   return __bfloat162float(__float2bfloat16_rn(x));
 }
+// 2^x, results below the smallest normal number flushed to zero
+__device__ __forceinline__ float exp2_ftz(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 // Exact (error-function) GELU.  For outputs that are rounded to bf16: the rational approximation of erfc by Hastings
 // (Abramowitz and Stegun, Handbook of Mathematical Functions, 7.1.26: absolute error below 1.5e-7), written for the tail
 // (1 - erf(|z|)) / 2 so that nothing cancels for negative arguments.

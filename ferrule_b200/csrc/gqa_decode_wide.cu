@@ -2,10 +2,11 @@
 //
 // Scores that are mixed across heads are products of one wide query row per head with the concatenated keys of a token
 // (head_prep.cu), so a CTA takes all of a token's cache row: keys and values of every kv head lie side by side there and come
-// as one bulk copy per token.  CTA = (query row, split of the visible keys, block of 16 heads), 8 warps; a tile is KT tokens.
+// as one bulk copy per token.  CTA = (query row, split of the visible keys, block of 16 heads); a tile is KT tokens.
 //
-//   scores   warp w multiplies the 16 query rows with 8 of the tile's keys over a share of the features (MMA, partial sums in
-//            shared memory)
+//   copies   warp 8 looks up a token per lane and keeps all stages requested
+//   scores   warp w of 8 multiplies the 16 query rows with 8 of the tile's keys over a share of the features (MMA, partial
+//            sums in shared memory); query fragments stay in registers when their share is at most 16 steps
 //   softmax  two rows per warp, a key per lane: distance bias, running maximum and sum, probabilities to shared memory
 //   values   warp w accumulates 16-column pieces w, w + 8, ... of the values for all 16 rows; a head keeps the columns of
 //            its own kv head
@@ -22,7 +23,7 @@
 
 namespace fb {
 
-constexpr int kGwThreads = 256;
+constexpr int kGwThreads = 256;      // of the 8 computing warps
 constexpr int kGwMaxStages = 8;
 constexpr int kGwSmemLimit = 227 * 1024;
 
@@ -58,7 +59,7 @@ struct GwLayout {
     prob = part + (64 / kt) * 16 * (kt + 1) * 4;
     factor = prob + 16 * (kt + 8) * 2;
     bars = factor + 48 * 4;
-    total = bars + (kGwMaxStages + 1) * 8;
+    total = bars + (2 * kGwMaxStages + 1) * 8;
   }
 };
 
@@ -72,9 +73,11 @@ __device__ __forceinline__ void ldsm_x2(uint32_t (&r)[2], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr));
 }
 
-// NC: 16-column value pieces per warp
-template <int KT, int NC>
-__global__ void __launch_bounds__(kGwThreads)
+__device__ __forceinline__ void gw_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kGwThreads) : "memory"); }
+
+// NC: 16-column value pieces per warp; KQ: query fragments in registers (steps of 16 features per share), 0: in shared memory
+template <int KT, int NC, int KQ>
+__global__ void __launch_bounds__(kGwThreads + 32)
 gqa_decode_wide_kernel(const GwParams p) {
   constexpr int kNt = KT / 8, kShares = 8 / kNt;   // 8-key columns of the score tile, feature shares
   pdl_launch_dependents();
@@ -88,7 +91,8 @@ gqa_decode_wide_kernel(const GwParams p) {
   float* c_m = f_s + 16;
   float* c_l = c_m + 16;
   uint64_t* full = reinterpret_cast<uint64_t*>(gw_sm + at.bars);
-  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(full + kGwMaxStages);
+  uint64_t* empty = full + kGwMaxStages;
+  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(empty + kGwMaxStages);
 
   const int r = blockIdx.x, split = blockIdx.y, splits = gridDim.y, h0 = blockIdx.z * 16, nh = min(16, p.heads - h0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
@@ -105,154 +109,213 @@ gqa_decode_wide_kernel(const GwParams p) {
     hi = min(lo + share * KT, n_keys);
   }
   const int n_tiles = (hi - lo + KT - 1) / KT;
-  const long long n_pages = p.pool_rows / p.page_size;
   auto token = [&](int i) { return i < kept ? i : first + i - kept; };
   if (tid == 0) {
-    for (int i = 0; i < p.stages; ++i) mbar_init(full + i, 1);
+    for (int i = 0; i < p.stages; ++i) {
+      mbar_init(full + i, 1);
+      mbar_init(empty + i, 8);
+    }
     *abort_flag = 0;
     fence_barrier_init();
   }
   __syncthreads();
-  // warp 0: a token per lane; places past the last key repeat it (their probability is zero, their values must be finite)
-  auto request = [&](int i) {
-    uint8_t* dst = gw_sm + (i % p.stages) * tile_bytes;
-    uint64_t* bar = full + i % p.stages;
-    long long slot = 0;
-    if (lane < KT) {
-      const int t = token(min(lo + i * KT + lane, hi - 1));
-      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
-      if (page >= 0 && page < n_pages) slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
-      else report_status(p.status, kStatusBadIndex, 0xE81, seq, t);
-    }
-    if (lane == 0) mbar_arrive_expect_tx(bar, static_cast<uint32_t>(KT * p.row_bytes));
-    __syncwarp();
-    if (lane < KT) gw_copy_row(dst + lane * p.pitch, p.pool + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes), bar);
-  };
-  int asked = 0;
-  if (warp == 0 && p.early)
-    // tiles that end below the row's own position: written by earlier steps
-    while (asked < p.stages && asked < n_tiles && lo + (asked + 1) * KT < n_keys) request(asked++);
-  pdl_wait();
-  if (warp == 0)
-    for (; asked < p.stages && asked < n_tiles; ++asked) request(asked);
-  // query rows of this block; rows past the last head and columns past the width are zeros
-  for (int i = tid; i < 16 * (at.q_pitch / 8); i += kGwThreads) {
-    const int row = i / (at.q_pitch / 8), c = (i - row * (at.q_pitch / 8)) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (row < nh && c < p.key_width)
-      v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.key_width + c);
-    *reinterpret_cast<uint4*>(q_s + row * at.q_pitch + c) = v;
-  }
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, sl[2];           // rows 2 warp, 2 warp + 1
-#pragma unroll
-  for (int k = 0; k < 2; ++k) {
-    const int row = 2 * warp + k;
-    sl[k] = p.slopes && row < nh ? p.slopes[h0 + row] * 1.4426950408889634f : 0.f;
-  }
+  const int vcols = (p.vdim_pad + 15) / 16, n_cols = p.kv_heads * vcols;
   float o[NC][2][4];
 #pragma unroll
   for (int c = 0; c < NC; ++c)
 #pragma unroll
     for (int n = 0; n < 2; ++n) o[c][n][0] = o[c][n][1] = o[c][n][2] = o[c][n][3] = 0.f;
-  const int ksteps = (p.key_width + 15) / 16, share = (ksteps + kShares - 1) / kShares;
-  const int nt = warp % kNt, part = warp / kNt, k0 = min(part * share, ksteps), k1 = min(k0 + share, ksteps);
-  const uint32_t qa = smem_u32(q_s + (lane & 15) * at.q_pitch + (lane >> 4) * 8);
-  const int vcols = (p.vdim_pad + 15) / 16, n_cols = p.kv_heads * vcols;
-  __syncthreads();
-  int done = 0;
-  for (int i = 0; i < n_tiles; ++i) {
-    const uint8_t* tile = gw_sm + (i % p.stages) * tile_bytes;
-    bool ok = mbar_wait(full + i % p.stages, (i / p.stages) & 1, abort_flag, p.status, 0xE90);
-    if (ok) {
-      float s0[4] = {}, s1[4] = {};
-      const uint32_t ka = smem_u32(tile + (nt * 8 + (lane & 7)) * p.pitch) + (lane >> 3) * 16;
-      int k = k0;
-      for (; k + 1 < k1; k += 2) {
-        uint32_t a0[4], a1[4], b[4];
-        ldsm_x4(b, ka + k * 32);
-        ldsm_x4(a0, qa + k * 32);
-        ldsm_x4(a1, qa + k * 32 + 32);
-        mma_bf16_16816(s0, a0, b[0], b[1]);
-        mma_bf16_16816(s1, a1, b[2], b[3]);
+  if (warp == 8) {
+    // a token per lane; places past the last key repeat it (their probability is zero, their values must be finite)
+    const long long n_pages = p.pool_rows / p.page_size;
+    bool waited = false, ok = true;
+    int asked = 0;
+    for (; asked < n_tiles; ++asked) {
+      const int st = asked % p.stages;
+      // tiles that end below the row's own position were written by earlier steps
+      if (!waited && !(p.early && asked < p.stages && lo + (asked + 1) * KT < n_keys)) {
+        pdl_wait();
+        waited = true;
       }
-      if (k < k1) {
-        uint32_t a0[4], b[2];
-        ldsm_x2(b, smem_u32(tile + (nt * 8 + (lane & 7)) * p.pitch) + ((lane >> 3) & 1) * 16 + k * 32);
-        ldsm_x4(a0, qa + k * 32);
-        mma_bf16_16816(s0, a0, b[0], b[1]);
+      long long slot = 0;
+      if (lane < KT) {
+        const int t = token(min(lo + asked * KT + lane, hi - 1));
+        const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+        if (page >= 0 && page < n_pages) slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
+        else report_status(p.status, kStatusBadIndex, 0xE81, seq, t);
       }
-      float* dst = part_s + (part * 16 + g4) * (KT + 1) + nt * 8 + t4 * 2;
-      dst[0] = s0[0] + s1[0];
-      dst[1] = s0[1] + s1[1];
-      dst[8 * (KT + 1)] = s0[2] + s1[2];
-      dst[8 * (KT + 1) + 1] = s0[3] + s1[3];
+      if (asked >= p.stages) {
+        ok = mbar_wait(empty + st, (asked / p.stages - 1) & 1, abort_flag, p.status, 0xE91);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+      }
+      if (lane == 0) mbar_arrive_expect_tx(full + st, static_cast<uint32_t>(KT * p.row_bytes));
+      __syncwarp();
+      if (lane < KT)
+        gw_copy_row(gw_sm + st * tile_bytes + lane * p.pitch, p.pool + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes),
+                    full + st);
     }
-    // also: every warp is done with tile i - 1
-    if (!__syncthreads_and(ok)) break;
-    if (warp == 0 && i > 0 && i - 1 + p.stages < n_tiles) request(i - 1 + p.stages);
-    const int key = lo + i * KT + lane;
-    const bool seen = lane < KT && key < hi;
-    const float dist = static_cast<float>(pos - token(min(key, hi - 1)));
+    if (!waited) pdl_wait();
+    if (*abort_flag) {
+      // copies may be in flight, and neither the merge nor the exit may happen under them
+      for (int i = max(asked - p.stages, 0); i < asked; ++i) {
+        const uint64_t t0 = globaltimer_ns();
+        while (!mbar_try_wait(full + i % p.stages, (i / p.stages) & 1) && globaltimer_ns() - t0 < 2000000ull) {
+        }
+      }
+    }
+  } else {
+    pdl_wait();
+    // query rows of this block; rows past the last head and columns past the width are zeros
+    for (int i = tid; i < 16 * (at.q_pitch / 8); i += kGwThreads) {
+      const int row = i / (at.q_pitch / 8), c = (i - row * (at.q_pitch / 8)) * 8;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (row < nh && c < p.key_width)
+        v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.key_width + c);
+      *reinterpret_cast<uint4*>(q_s + row * at.q_pitch + c) = v;
+    }
+    float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, sl[2];         // rows 2 warp, 2 warp + 1
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
       const int row = 2 * warp + k;
-      float x = -INFINITY;
-      if (seen) {
-        float s = 0.f;
-#pragma unroll
-        for (int q = 0; q < kShares; ++q) s += part_s[(q * 16 + row) * (KT + 1) + lane];
-        x = fmaf(-sl[k], dist, s * p.scale_log2);
-      }
-      const float mn = fmaxf(m[k], warp_max(x));                            // finite: a tile has at least one visible key
-      const float f = exp2f(m[k] - mn), w = seen ? exp2f(x - mn) : 0.f;
-      m[k] = mn;
-      l[k] = fmaf(l[k], f, warp_sum(w));
-      if (lane < KT) prob_s[row * (KT + 8) + lane] = __float2bfloat16_rn(w);
-      if (lane == 0) f_s[row] = f;
+      sl[k] = p.slopes && row < nh ? p.slopes[h0 + row] * 1.4426950408889634f : 0.f;
     }
-    __syncthreads();
-    const float f0 = f_s[g4], f1 = f_s[g4 + 8];
-    uint32_t pf[KT / 16][4];
+    const int ksteps = (p.key_width + 15) / 16, share = (ksteps + kShares - 1) / kShares;
+    const int nt = warp % kNt, part = warp / kNt, k0 = min(part * share, ksteps), k1 = min(k0 + share, ksteps);
+    const uint32_t qa = smem_u32(q_s + (lane & 15) * at.q_pitch + (lane >> 4) * 8);
+    gw_sync();
+    uint32_t qf[KQ > 0 ? KQ : 1][4];
+    if constexpr (KQ > 0) {
 #pragma unroll
-    for (int k = 0; k < KT / 16; ++k) ldsm_x4(pf[k], smem_u32(prob_s + (lane & 15) * (KT + 8) + k * 16 + (lane >> 4) * 8));
-#pragma unroll
-    for (int c = 0; c < NC; ++c) {
-      const int col = warp + 8 * c;
-      if (col >= n_cols) break;
-      const int g = col / vcols, d = (col - g * vcols) * 16;
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        o[c][n][0] *= f0;
-        o[c][n][1] *= f0;
-        o[c][n][2] *= f1;
-        o[c][n][3] *= f1;
-      }
-      // matrices (transposed): keys 0-7 / 8-15 x columns 0-7, then columns 8-15
-      const uint32_t va = smem_u32(tile + ((lane >> 3 & 1) * 8 + (lane & 7)) * p.pitch) +
-                          (p.key_width + g * p.vdim_pad + d + (lane >> 4) * 8) * 2;
-#pragma unroll
-      for (int k = 0; k < KT / 16; ++k) {
-        uint32_t b[4];
-        ldsm_x4_t(b, va + k * 16 * p.pitch);
-        mma_bf16_16816(o[c][0], pf[k], b[0], b[1]);
-        mma_bf16_16816(o[c][1], pf[k], b[2], b[3]);
+      for (int k = 0; k < KQ; ++k) {
+        qf[k][0] = qf[k][1] = qf[k][2] = qf[k][3] = 0u;
+        if (k0 + k < k1) ldsm_x4(qf[k], qa + (k0 + k) * 32);
       }
     }
-    done = i + 1;
-  }
-  if (done < n_tiles && tid == 0) {
-    // a wait gave up: copies may be in flight, and neither the merge nor the exit may happen under them
-    for (int i = done; i < min(done + p.stages, n_tiles); ++i) {
-      const uint64_t t0 = globaltimer_ns();
-      while (!mbar_try_wait(full + i % p.stages, (i / p.stages) & 1) && globaltimer_ns() - t0 < 2000000ull) {
-      }
-    }
-  }
-  if (lane == 0) {
+    for (int i = 0; i < n_tiles; ++i) {
+      const uint8_t* tile = gw_sm + (i % p.stages) * tile_bytes;
+      // a wait that gives up leaves its mark in the status word; the loop goes on so that the barriers stay in step
+      mbar_wait(full + i % p.stages, (i / p.stages) & 1, abort_flag, p.status, 0xE90);
+      {
+        float s0[4] = {}, s1[4] = {};
+        const uint32_t kr = smem_u32(tile + (nt * 8 + (lane & 7)) * p.pitch) + k0 * 32;
+        const uint32_t ka = kr + (lane >> 3) * 16;                         // two steps of 16 features
+        if constexpr (KQ > 0) {
 #pragma unroll
-    for (int k = 0; k < 2; ++k) {
-      c_m[2 * warp + k] = m[k];
-      c_l[2 * warp + k] = l[k];
+          for (int k = 0; k < KQ; k += 2) {
+            if (k0 + k + 1 < k1) {
+              uint32_t b[4];
+              ldsm_x4(b, ka + k * 32);
+              mma_bf16_16816(s0, qf[k], b[0], b[1]);
+              mma_bf16_16816(s1, qf[k + 1], b[2], b[3]);
+            } else if (k0 + k < k1) {
+              uint32_t b[2];
+              ldsm_x2(b, kr + ((lane >> 3) & 1) * 16 + k * 32);
+              mma_bf16_16816(s0, qf[k], b[0], b[1]);
+            }
+          }
+        } else {
+          int k = 0;
+          for (; k0 + k + 1 < k1; k += 2) {
+            uint32_t a0[4], a1[4], b[4];
+            ldsm_x4(b, ka + k * 32);
+            ldsm_x4(a0, qa + (k0 + k) * 32);
+            ldsm_x4(a1, qa + (k0 + k) * 32 + 32);
+            mma_bf16_16816(s0, a0, b[0], b[1]);
+            mma_bf16_16816(s1, a1, b[2], b[3]);
+          }
+          if (k0 + k < k1) {
+            uint32_t a0[4], b[2];
+            ldsm_x2(b, kr + ((lane >> 3) & 1) * 16 + k * 32);
+            ldsm_x4(a0, qa + (k0 + k) * 32);
+            mma_bf16_16816(s0, a0, b[0], b[1]);
+          }
+        }
+        float* dst = part_s + (part * 16 + g4) * (KT + 1) + nt * 8 + t4 * 2;
+        dst[0] = s0[0] + s1[0];
+        dst[1] = s0[1] + s1[1];
+        dst[8 * (KT + 1)] = s0[2] + s1[2];
+        dst[8 * (KT + 1) + 1] = s0[3] + s1[3];
+      }
+      gw_sync();
+      const int key = lo + i * KT + lane;
+      const bool seen = lane < KT && key < hi;
+      const float dist = static_cast<float>(pos - token(min(key, hi - 1)));
+      float x[2], w[2];
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int row = 2 * warp + k;
+        x[k] = -INFINITY;
+        if (seen) {
+          float s = 0.f;
+#pragma unroll
+          for (int q = 0; q < kShares; ++q) s += part_s[(q * 16 + row) * (KT + 1) + lane];
+          x[k] = fmaf(-sl[k], dist, s * p.scale_log2);
+        }
+      }
+      float mx0 = x[0], mx1 = x[1];
+#pragma unroll
+      for (int d = 16; d > 0; d >>= 1) {
+        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, d));
+        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, d));
+      }
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int row = 2 * warp + k;
+        const float mn = fmaxf(m[k], k == 0 ? mx0 : mx1);                   // finite: a tile has at least one visible key
+        const float f = exp2f(m[k] - mn);
+        w[k] = seen ? exp2f(x[k] - mn) : 0.f;
+        m[k] = mn;
+        l[k] *= f;
+        if (lane < KT) prob_s[row * (KT + 8) + lane] = __float2bfloat16_rn(w[k]);
+        if (lane == 0) f_s[row] = f;
+      }
+      gw_sync();
+      const float f0 = f_s[g4], f1 = f_s[g4 + 8];
+      uint32_t pf[KT / 16][4];
+#pragma unroll
+      for (int k = 0; k < KT / 16; ++k) ldsm_x4(pf[k], smem_u32(prob_s + (lane & 15) * (KT + 8) + k * 16 + (lane >> 4) * 8));
+#pragma unroll
+      for (int c = 0; c < NC; ++c) {
+        const int col = warp + 8 * c;
+        if (col < n_cols) {
+          const int g = col / vcols, d = (col - g * vcols) * 16;
+#pragma unroll
+          for (int n = 0; n < 2; ++n) {
+            o[c][n][0] *= f0;
+            o[c][n][1] *= f0;
+            o[c][n][2] *= f1;
+            o[c][n][3] *= f1;
+          }
+          // matrices (transposed): keys 0-7 / 8-15 x columns 0-7, then columns 8-15
+          const uint32_t va = smem_u32(tile + ((lane >> 3 & 1) * 8 + (lane & 7)) * p.pitch) +
+                              (p.key_width + g * p.vdim_pad + d + (lane >> 4) * 8) * 2;
+#pragma unroll
+          for (int k = 0; k < KT / 16; ++k) {
+            uint32_t b[4];
+            ldsm_x4_t(b, va + k * 16 * p.pitch);
+            mma_bf16_16816(o[c][0], pf[k], b[0], b[1]);
+            mma_bf16_16816(o[c][1], pf[k], b[2], b[3]);
+          }
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(empty + i % p.stages);
+      // the row sums, off the path to the values
+#pragma unroll
+      for (int d = 16; d > 0; d >>= 1) {
+        w[0] += __shfl_xor_sync(0xffffffffu, w[0], d);
+        w[1] += __shfl_xor_sync(0xffffffffu, w[1], d);
+      }
+      l[0] += w[0];
+      l[1] += w[1];
+    }
+    if (lane == 0) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        c_m[2 * warp + k] = m[k];
+        c_l[2 * warp + k] = l[k];
+      }
     }
   }
   __syncthreads();                                                         // the tiles' memory now holds the outputs
@@ -261,7 +324,7 @@ gqa_decode_wide_kernel(const GwParams p) {
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
     const int col = warp + 8 * c;
-    if (col >= n_cols) break;
+    if (col >= n_cols || warp == 8) break;
     const int g = col / vcols, d = (col - g * vcols) * 16 + t4 * 2;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
@@ -277,7 +340,7 @@ gqa_decode_wide_kernel(const GwParams p) {
   if (splits > 1) cluster_sync_all();
   else __syncthreads();
   const int quads = p.vdim_pad / 4;
-  for (int i = tid + split * kGwThreads; i < nh * quads; i += kGwThreads * splits) {
+  for (int i = tid + split * blockDim.x; i < nh * quads; i += blockDim.x * splits) {
     const int h = i / quads, d = (i - h * quads) * 4;
     float mm = -INFINITY, ll = 0.f;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -312,9 +375,9 @@ gqa_decode_wide_kernel(const GwParams p) {
   if (splits > 1) cluster_sync_all();                                      // no CTA leaves while a peer reads its rows
 }
 
-// tile size and stages for a cache row of this shape; 0: it does not fit
+// tile size and stages for a cache row of this shape; kt 0: it does not fit
 struct GwPlan {
-  int kt, stages, nc;
+  int kt, stages, nc, kq;
 };
 static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad) {
   const int vcols = (vdim_pad + 15) / 16, cols = kv_heads * vcols, pitch = (key_width + kv_heads * vdim_pad) * 2 + 16;
@@ -323,22 +386,24 @@ static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad) {
     int stages = (kGwSmemLimit - GwLayout(key_width, 0, kt).total) / (kt * pitch);
     if (stages > kGwMaxStages) stages = kGwMaxStages;
     // the merged outputs reuse the tiles' memory
-    if (stages >= 2 && stages * kt * pitch >= 16 * (vcols * 16 + 4) * 4) return {kt, stages, nc};
+    if (stages < 2 || stages * kt * pitch < 16 * (vcols * 16 + 4) * 4) continue;
+    const int shares = 64 / kt, steps = ((key_width + 15) / 16 + shares - 1) / shares;
+    return {kt, stages, nc, steps <= 4 ? 4 : steps <= 16 ? 16 : 0};
   }
-  return {0, 0, 0};
+  return {0, 0, 0, 0};
 }
 
-template <int KT, int NC>
+template <int KT, int NC, int KQ>
 static int launch_gw(const GwParams& p, int rows, int splits, cudaStream_t stream) {
   static bool attr_set = false;
   if (!attr_set) {
-    if (cudaFuncSetAttribute(gqa_decode_wide_kernel<KT, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGwSmemLimit) != cudaSuccess)
+    if (cudaFuncSetAttribute(gqa_decode_wide_kernel<KT, NC, KQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGwSmemLimit) != cudaSuccess)
       return FB_ERR_LAUNCH;
     attr_set = true;
   }
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = dim3(rows, splits, p.head_blocks);
-  cfg.blockDim = dim3(kGwThreads);
+  cfg.blockDim = dim3(kGwThreads + 32);
   cfg.dynamicSmemBytes = GwLayout(p.key_width, p.stages * KT * p.pitch, KT).total;
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
@@ -350,8 +415,21 @@ static int launch_gw(const GwParams& p, int rows, int splits, cudaStream_t strea
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
   cfg.numAttrs = pdl_enabled() ? 2 : 1;
-  if (cudaLaunchKernelEx(&cfg, gqa_decode_wide_kernel<KT, NC>, p) != cudaSuccess) return FB_ERR_LAUNCH;
+  if (cudaLaunchKernelEx(&cfg, gqa_decode_wide_kernel<KT, NC, KQ>, p) != cudaSuccess) return FB_ERR_LAUNCH;
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+template <int KT, int NC>
+static int launch_gw_steps(const GwParams& p, int kq, int rows, int splits, cudaStream_t s) {
+  if (kq == 4) return launch_gw<KT, NC, 4>(p, rows, splits, s);
+  if (kq == 16) return launch_gw<KT, NC, 16>(p, rows, splits, s);
+  return launch_gw<KT, NC, 0>(p, rows, splits, s);
+}
+template <int KT>
+static int launch_gw_cols(const GwParams& p, const GwPlan& plan, int rows, int splits, cudaStream_t s) {
+  if (plan.nc == 1) return launch_gw_steps<KT, 1>(p, plan.kq, rows, splits, s);
+  if (plan.nc == 2) return launch_gw_steps<KT, 2>(p, plan.kq, rows, splits, s);
+  if (plan.nc == 4) return launch_gw_steps<KT, 4>(p, plan.kq, rows, splits, s);
+  return launch_gw_steps<KT, 8>(p, plan.kq, rows, splits, s);
 }
 
 }  // namespace fb
@@ -394,14 +472,5 @@ extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, voi
   p.early = early;
   p.status = static_cast<DeviceStatus*>(a->status);
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  if (plan.kt == 32) {
-    if (plan.nc == 1) return launch_gw<32, 1>(p, a->rows, splits, s);
-    if (plan.nc == 2) return launch_gw<32, 2>(p, a->rows, splits, s);
-    if (plan.nc == 4) return launch_gw<32, 4>(p, a->rows, splits, s);
-    return launch_gw<32, 8>(p, a->rows, splits, s);
-  }
-  if (plan.nc == 1) return launch_gw<16, 1>(p, a->rows, splits, s);
-  if (plan.nc == 2) return launch_gw<16, 2>(p, a->rows, splits, s);
-  if (plan.nc == 4) return launch_gw<16, 4>(p, a->rows, splits, s);
-  return launch_gw<16, 8>(p, a->rows, splits, s);
+  return plan.kt == 32 ? launch_gw_cols<32>(p, plan, a->rows, splits, s) : launch_gw_cols<16>(p, plan, a->rows, splits, s);
 }

@@ -9,7 +9,7 @@
 //   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
 //     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
 //     head's width and rows past the sequence are zeros), two stages each with their own barriers.  Wide keys (those of all
-//     kv heads side by side) come in pieces of `kb` feature blocks, a stage each; query rows that do not fit in shared
+//     kv heads side by side) come in pieces of `kb` feature blocks, a stage of up to four each; query rows that do not fit in shared
 //     memory come with them, piece by piece, for every token tile.
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
 //     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
@@ -24,6 +24,7 @@
 #include "act_type.cuh"
 #include "attn_tc.cuh"
 #include "common.cuh"
+#include "f32x2.cuh"
 #include "ferrule_b200.h"
 #include "gqa_mask.cuh"
 #include "launch.cuh"
@@ -49,7 +50,7 @@ struct GpParams {
   int num_seqs, max_blocks, page_size, box_rows;
   KeySpan span;
   int key_width, vdim_pad, qb, vb;     // qb, vb: 64-feature blocks of a query / key row and of a value row
-  int kb, pieces, q_resident;          // blocks per key stage, stages per token tile
+  int kb, pieces, ks, q_resident;      // blocks per key stage, stages per token tile, key stages (2 or 4)
   int shared_keys;
   uint32_t tmem_cols;
   float scale_log2;
@@ -70,19 +71,20 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int qb = p.qb, vb = p.vb;
   uint8_t* q_s = smem;
-  uint8_t* k_s = q_s + (p.q_resident ? qb : 2 * p.kb) * kGpQBlock;      // [2][kb] blocks
-  uint8_t* v_s = k_s + 2 * p.kb * kGpKvBlock;            // [2][vb] blocks
+  uint8_t* k_s = q_s + (p.q_resident ? qb : p.ks * p.kb) * kGpQBlock;   // [ks][kb] blocks
+  uint8_t* v_s = k_s + p.ks * p.kb * kGpKvBlock;         // [2][vb] blocks
   uint64_t* bars = reinterpret_cast<uint64_t*>(v_s + 2 * vb * kGpKvBlock);
   uint64_t* q_full = bars + 0;
-  uint64_t* k_full = bars + 1;          // [2]
-  uint64_t* v_full = bars + 3;          // [2]
-  uint64_t* k_free = bars + 5;          // [2]
-  uint64_t* v_free = bars + 7;          // [2]
-  uint64_t* s_full = bars + 9;          // [2]
-  uint64_t* p_full = bars + 11;         // [2]
-  uint64_t* o_done = bars + 13;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
-  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(bars + 15);
+  uint64_t* k_full = bars + 1;          // [4]
+  uint64_t* v_full = bars + 5;          // [2]
+  uint64_t* k_free = bars + 7;          // [4]
+  uint64_t* v_free = bars + 11;         // [2]
+  uint64_t* s_full = bars + 13;         // [2]
+  uint64_t* p_full = bars + 15;         // [2]
+  uint64_t* o_done = bars + 17;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
+  volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(bars + 19);
+  const int k_mask = p.ks - 1, k_shift = p.ks == 4 ? 2 : 1;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = blockIdx.y;
@@ -96,7 +98,11 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   const int j0 = p.span.first(pos0) / kGpKv;                             // first token tile of the chunk or window
   const int n_pre = min((p.span.head(pos0 + nrows - 1) + kGpKv - 1) / kGpKv, j0);      // tiles of kept tokens before it
   const int n_kv = n_pre + (kv_len + kGpKv - 1) / kGpKv - j0;
-  auto tile_of = [&](int j) { return j < n_pre ? j : j0 + j - n_pre; };
+  // with a distance bias the latest keys come first: a row's maximum is then mostly among them
+  auto tile_of = [&](int j) {
+    if (BIAS) j = n_kv - 1 - j;
+    return j < n_pre ? j : j0 + j - n_pre;
+  };
   if (n_kv <= 0) {
     if (tid == 0) report_status(p.status, kStatusBadIndex, 0xA81, blockIdx.x, pos0);
     return;
@@ -104,10 +110,12 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
   if (tid == 0) {
     mbar_init(q_full, 1);
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < 4; ++i) {
       mbar_init(k_full + i, 1);
-      mbar_init(v_full + i, 1);
       mbar_init(k_free + i, 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(v_full + i, 1);
       mbar_init(v_free + i, 1);
       mbar_init(s_full + i, 1);
       mbar_init(p_full + i, 4);
@@ -157,8 +165,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           rowc[s] = rc;
         }
         for (int c = 0; c < p.pieces && ok; ++c) {
-          const int i = j * p.pieces + c, ks = i & 1, b0 = c * p.kb, nb = min(p.kb, qb - b0);
-          if (i > 1) ok = mbar_wait(k_free + ks, ((i - 2) >> 1) & 1, abort_flag, p.status, 0xA90);
+          const int i = j * p.pieces + c, ks = i & k_mask, b0 = c * p.kb, nb = min(p.kb, qb - b0);
+          if (i >= p.ks) ok = mbar_wait(k_free + ks, ((i >> k_shift) - 1) & 1, abort_flag, p.status, 0xA90);
           if (!ok) break;
           mbar_arrive_expect_tx(k_full + ks, nb * (static_cast<uint32_t>(kGpKvBlock) + (p.q_resident ? 0u : q_block_tx)));
           for (int s = 0; s < subs; ++s)
@@ -179,7 +187,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rowc[s]);
         v_armed = j + 1;
       }
-      // after an abort: copies of the last two stages may still be in flight, and the CTA may not exit under them
+      // after an abort: copies of the last stages may still be in flight, and the CTA may not exit under them
       if (*abort_flag) {
         auto drain = [&](uint64_t* bar, uint32_t parity) {
           const uint64_t t0 = globaltimer_ns();
@@ -187,7 +195,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           }
         };
         if (p.q_resident) drain(q_full, 0);
-        for (int i = max(k_armed - 2, 0); i < k_armed; ++i) drain(k_full + (i & 1), (i >> 1) & 1);
+        for (int i = max(k_armed - p.ks, 0); i < k_armed; ++i) drain(k_full + (i & k_mask), (i >> k_shift) & 1);
         for (int j = max(v_armed - 2, 0); j < v_armed; ++j) drain(v_full + (j & 1), (j >> 1) & 1);
       }
     }
@@ -200,16 +208,22 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       const int ksteps = (p.key_width + 15) / 16;
       auto qk = [&](int j) {
         for (int c = 0; c < p.pieces; ++c) {
-          const int i = j * p.pieces + c, st = i & 1, k0 = c * p.kb * 4, k1 = min(k0 + p.kb * 4, ksteps);
-          if (!mbar_wait(k_full + st, (i >> 1) & 1, abort_flag, p.status, 0xAA2)) return false;
+          const int i = j * p.pieces + c, st = i & k_mask, k0 = c * p.kb * 4, k1 = min(k0 + p.kb * 4, ksteps);
+          if (!mbar_wait(k_full + st, (i >> k_shift) & 1, abort_flag, p.status, 0xAA2)) return false;
           tc_fence_after();
           const uint32_t ks = k_addr + st * p.kb * kGpKvBlock;
           const uint32_t qs = p.q_resident ? q_addr + c * p.kb * kGpQBlock : q_addr + st * p.kb * kGpQBlock;
-          for (int k = k0; k < k1; ++k) {
-            const int kk = k - k0;
-            umma_bf16(tmem + col_s + (j & 1) * kGpKv, umma_desc_k128(qs + (kk >> 2) * kGpQBlock + (kk & 3) * 32),
-                      umma_desc_k128(ks + (kk >> 2) * kGpKvBlock + (kk & 3) * 32), idesc_qk, k > 0 ? 1u : 0u);
+          // one thread issues everything: descriptors are advanced (16-byte units), not rebuilt
+          uint64_t dq = umma_desc_k128(qs), dk = umma_desc_k128(ks);
+          const uint32_t d = tmem + col_s + (j & 1) * kGpKv;
+          int k = k0;
+          for (; k + 4 <= k1; k += 4) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) umma_bf16(d, dq + 2 * e, dk + 2 * e, idesc_qk, (k > 0 || e > 0) ? 1u : 0u);
+            dq += kGpQBlock >> 4;
+            dk += kGpKvBlock >> 4;
           }
+          for (int e = 0; k < k1; ++k, ++e) umma_bf16(d, dq + 2 * e, dk + 2 * e, idesc_qk, k > 0 ? 1u : 0u);
           if (c + 1 == p.pieces) umma_commit(s_full + (j & 1));
           umma_commit(k_free + st);
         }
@@ -231,11 +245,10 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (ok) ok = mbar_wait(p_full + (j & 1), ph, abort_flag, p.status, 0xAA4);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t vs = v_addr + (j & 1) * vb * kGpKvBlock;
+        const uint64_t dv = umma_desc_mn128(v_addr + (j & 1) * vb * kGpKvBlock, kGpKvBlock);
 #pragma unroll
         for (int k = 0; k < 4; ++k)
-          umma_bf16_ts(tmem, tmem + col_s + (j & 1) * kGpKv + k * 8, umma_desc_mn128(vs + k * 2048, kGpKvBlock), idesc_pv,
-                       (j > 0 || k > 0) ? 1u : 0u);
+          umma_bf16_ts(tmem, tmem + col_s + (j & 1) * kGpKv + k * 8, dv + k * (2048 >> 4), idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
         umma_commit(v_free + (j & 1));
         if (j + 1 == n_kv) umma_commit(o_done);
       }
@@ -264,32 +277,40 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int c = 0; c < 4; ++c) tmem_ld16(s_t + c * 16, sv[c]);
       tmem_ld_wait();
       const int tok0 = tile_of(j) * kGpKv;
-      float mx = -INFINITY;
+      // one warp per scheduler: four independent chains for the maximum and the sum, packed multiply-adds
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (BIAS) {
         // the score in base 2 with its distance bias
         const float b0 = slope * static_cast<float>(tok0 - pos);
+        const uint64_t sc2 = pack2(p.scale_log2, p.scale_log2), sl2 = pack2(slope, slope), b02 = pack2(b0, b0);
 #pragma unroll
         for (int c = 0; c < 4; ++c)
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            sv[c][i] = __float_as_uint(fmaf(__uint_as_float(sv[c][i]), p.scale_log2, fmaf(slope, static_cast<float>(c * 16 + i), b0)));
+          for (int i = 0; i < 16; i += 2) {
+            const uint64_t bias = fma2(sl2, pack2(static_cast<float>(c * 16 + i), static_cast<float>(c * 16 + i + 1)), b02);
+            float x0, x1;
+            unpack2(fma2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), sc2, bias), x0, x1);
+            sv[c][i] = __float_as_uint(x0);
+            sv[c][i + 1] = __float_as_uint(x1);
+          }
       }
       if (__all_sync(0xffffffffu, tok0 + kGpKv <= hi && (tok0 >= lo || tok0 + kGpKv <= keep))) {
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
+        for (int i = 0; i < 16; ++i)
 #pragma unroll
-          for (int i = 0; i < 16; ++i) mx = fmaxf(mx, __uint_as_float(sv[c][i]));
+          for (int c = 0; c < 4; ++c) mx4[c] = fmaxf(mx4[c], __uint_as_float(sv[c][i]));
       } else {
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
+        for (int i = 0; i < 16; ++i)
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
+          for (int c = 0; c < 4; ++c) {
             const int t = tok0 + c * 16 + i;
             const float x = ((t >= lo || t < keep) && t < hi) ? __uint_as_float(sv[c][i]) : -INFINITY;
             sv[c][i] = __float_as_uint(x);
-            mx = fmaxf(mx, x);
+            mx4[c] = fmaxf(mx4[c], x);
           }
       }
+      float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       if (!BIAS) mx *= p.scale_log2;                          // the scale is positive
       const float m_new = fmaxf(m_ref, mx);
       if (j == 0) {
@@ -314,22 +335,27 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         }
       }
       const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
-      float add = 0.f;
+      const uint64_t scale2 = pack2(p.scale_log2, p.scale_log2), ref2 = pack2(-m_use, -m_use);
+      uint64_t add[4] = {0ull, 0ull, 0ull, 0ull};
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float x0 = __uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]);
-          const float x1 = __uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]);
-          const float p0 = exp2f(BIAS ? x0 - m_use : fmaf(x0, p.scale_log2, -m_use));
-          const float p1 = exp2f(BIAS ? x1 - m_use : fmaf(x1, p.scale_log2, -m_use));
-          add += p0 + p1;
+          const uint64_t x = pack2(__uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]),
+                                   __uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]));
+          float p0, p1;
+          unpack2(BIAS ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
+          p0 = exp2_ftz(p0);
+          p1 = exp2_ftz(p1);
+          add[i & 3] = add2(add[i & 3], pack2(p0, p1));
           pk[i] = pack_bf16x2(p0, p1);
         }
         tmem_st16(s_t + c * 16, pk);
       }
-      l_sum += add;
+      float add_lo, add_hi;
+      unpack2(add2(add2(add[0], add[1]), add2(add[2], add[3])), add_lo, add_hi);
+      l_sum += add_lo + add_hi;
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -388,6 +414,13 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         }
       }
       __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
+      uint4 ahead[2];                                         // the gates of the next 16 columns
+      auto gates = [&](int col) {
+        if (!gate || !valid) return;
+        if (col < p.vdim_pad) ahead[0] = *reinterpret_cast<const uint4*>(gate + col);
+        if (col + 8 < p.vdim_pad) ahead[1] = *reinterpret_cast<const uint4*>(gate + col + 8);
+      };
+      if (p.maps == 1) gates(0);
 #pragma unroll 1
       for (int c = 0; c < vb * 4 && p.maps == 1; ++c) {
         if (c * 16 >= p.vdim_pad) break;
@@ -395,15 +428,12 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         tmem_ld16(lane_base + c * 16, ov);
         tmem_ld_wait();
         if (valid && gate) {
+          const uint4 now[2] = {ahead[0], ahead[1]};
+          gates(c * 16 + 16);
+          const __nv_bfloat16* z = reinterpret_cast<const __nv_bfloat16*>(now);
 #pragma unroll
-          for (int e = 0; e < 16; e += 8) {
-            if (c * 16 + e >= p.vdim_pad) break;
-            float z[8];
-            act_load8(gate + c * 16 + e, z);
-#pragma unroll
-            for (int i = 0; i < 8; ++i)
-              ov[e + i] = __float_as_uint(__fdividef(__uint_as_float(ov[e + i]), 1.f + __expf(-z[i])));
-          }
+          for (int i = 0; i < 16; ++i)
+            ov[i] = __float_as_uint(__fdividef(__uint_as_float(ov[i]), 1.f + __expf(-__bfloat162float(z[i]))));
         }
         if (valid) {
           uint4 w0, w1;
@@ -504,15 +534,14 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.maps = a->maps; p.vdim = a->vdim;
   p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale; p.eps = a->eps;
-  // key stages as wide as fit beside the query rows; rows too wide to stay are streamed with the keys
+  // query rows that stay in shared memory beside the key stages; rows too wide for that are streamed with the keys
   int smem = 0;
-  for (int form = 0; form < 6; ++form) {
-    p.q_resident = form < 3;
-    p.kb = p.q_resident ? 4 >> form : 4 >> (form - 3);
-    if (p.kb > p.qb && p.kb > 1 && p.q_resident) p.kb = p.qb;
-    smem = (p.q_resident ? p.qb : 2 * p.kb) * kGpQBlock + 2 * (p.kb + p.vb) * kGpKvBlock + 1024 + 256;
-    if (smem <= kGpSmemLimit) break;
-    smem = 0;
+  static const int forms[5][3] = {{1, 4, 2}, {1, 2, 4}, {1, 1, 4}, {0, 2, 2}, {0, 1, 2}};      // resident, kb, ks
+  for (int f = p.qb > 4 ? 1 : 0; f < 5 && smem == 0; ++f) {
+    p.q_resident = forms[f][0]; p.kb = forms[f][1]; p.ks = forms[f][2];
+    if (p.kb > p.qb) p.kb = p.qb;
+    smem = (p.q_resident ? p.qb : p.ks * p.kb) * kGpQBlock + (p.ks * p.kb + 2 * p.vb) * kGpKvBlock + 1024 + 256;
+    if (smem > kGpSmemLimit) smem = 0;
   }
   if (smem == 0) return FB_ERR_LIMIT;
   p.pieces = (p.qb + p.kb - 1) / p.kb;

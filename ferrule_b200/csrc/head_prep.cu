@@ -31,12 +31,12 @@ struct HeadPrepParams {
   const long long* write_slot;
   T* pool;
   long long pool_rows, pool_ld;
-  int heads, kv_heads, maps, dim, dim_pad, vdim_pad, mix;
+  int heads, kv_heads, maps, dim, dim_pad, vdim_pad;
   float eps;
   DeviceStatus* status;
 };
 
-template <typename T>
+template <typename T, bool MIX>
 __global__ void __launch_bounds__(kHpThreads)
 head_prep_kernel(const HeadPrepParams<T> p) {
   pdl_launch_dependents();
@@ -47,7 +47,7 @@ head_prep_kernel(const HeadPrepParams<T> p) {
   float* inv = sk + nk * dp;               // [nq + nk]
   float* coef = inv + nq + nk;             // mix: [heads][heads]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = kHpThreads / 32;
-  if (p.mix)
+  if (MIX)
     for (int i = tid; i < p.heads * p.heads; i += kHpThreads) coef[i] = p.q_mix[i];
   pdl_wait();
   const long long r = blockIdx.x, slot = p.write_slot[r];
@@ -96,22 +96,31 @@ head_prep_kernel(const HeadPrepParams<T> p) {
       act_store8(row + h * dp + d, x);
     }
   T* out = p.q_out + r * p.ldqo;
-  if (p.mix) {
-    const int per = p.heads / p.kv_heads, items = p.heads * p.kv_heads * vecs;
+  if constexpr (MIX) {
+    // an item is kHb output heads x one kv head x 8 features: every query vector is read once for all of them
+    constexpr int kHb = 4;
+    const int per = p.heads / p.kv_heads, gv = p.kv_heads * vecs, items = (p.heads + kHb - 1) / kHb * gv;
     for (int i = tid; i < items; i += kHpThreads) {
-      const int hg = i / vecs, d = (i - hg * vecs) * 8, h = hg / p.kv_heads, g0 = (hg - h * p.kv_heads) * per;
-      float acc[8] = {}, w[8];
-      for (int g = g0; g < g0 + per; ++g) {
-        const float f = coef[h * p.heads + g] * inv[g];
+      const int hb = i / gv, c = i - hb * gv, kv = c / vecs, d = (c - kv * vecs) * 8, h0 = hb * kHb;
+      float acc[kHb][8] = {}, w[8];
+      act_load8(p.q_norm + d, w);
+      for (int g = kv * per; g < kv * per + per; ++g) {
         float x[8];
         act_load8(sq + g * dp + d, x);
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[j] = fmaf(f, x[j], acc[j]);
-      }
-      act_load8(p.q_norm + d, w);
+        for (int b = 0; b < kHb; ++b) {
+          const float f = coef[min(h0 + b, p.heads - 1) * p.heads + g] * inv[g];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) acc[j] *= w[j];
-      act_store8(out + static_cast<long long>(i) * 8, acc);
+          for (int j = 0; j < 8; ++j) acc[b][j] = fmaf(f, x[j], acc[b][j]);
+        }
+      }
+#pragma unroll
+      for (int b = 0; b < kHb; ++b) {
+        if (h0 + b >= p.heads) break;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[b][j] *= w[j];
+        act_store8(out + (static_cast<long long>(h0 + b) * gv + c) * 8, acc[b]);
+      }
     }
   } else {
     const int items = nq * p.maps * vecs;
@@ -131,26 +140,26 @@ head_prep_kernel(const HeadPrepParams<T> p) {
   }
 }
 
-template <typename T>
+template <typename T, bool MIX>
 static int run_head_prep(const FbHeadPrepArgs* a, cudaStream_t s) {
   HeadPrepParams<T> p{};
   p.q = static_cast<const T*>(a->q); p.k = static_cast<const T*>(a->k); p.v = static_cast<const T*>(a->v); p.ldp = a->ldp;
-  p.q_bias = a->q_bias; p.k_bias = a->k_bias; p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.q_mix = a->q_mix; p.mix = a->mix;
+  p.q_bias = a->q_bias; p.k_bias = a->k_bias; p.q_norm = a->q_norm; p.k_norm = a->k_norm; p.q_mix = a->q_mix;
   p.q_out = static_cast<T*>(a->q_out); p.ldqo = a->ldqo;
   p.write_slot = a->write_slot; p.pool = static_cast<T*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
   p.heads = a->heads; p.kv_heads = a->kv_heads; p.maps = a->maps;
   p.dim = a->dim; p.dim_pad = a->dim_pad; p.vdim_pad = a->vdim_pad; p.eps = a->eps;
   p.status = static_cast<DeviceStatus*>(a->status);
   const size_t n = static_cast<size_t>(a->heads + a->kv_heads) * a->maps;
-  const size_t smem = (n * a->dim_pad + n + (a->mix ? static_cast<size_t>(a->heads) * a->heads : 0)) * sizeof(float);
+  const size_t smem = (n * a->dim_pad + n + (MIX ? static_cast<size_t>(a->heads) * a->heads : 0)) * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(head_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+    if (cudaFuncSetAttribute(head_prep_kernel<T, MIX>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
       return FB_ERR_LAUNCH;
     attr = true;
   }
-  launch_pdl(head_prep_kernel<T>, dim3(a->rows), dim3(kHpThreads), smem, s, p);
+  launch_pdl(head_prep_kernel<T, MIX>, dim3(a->rows), dim3(kHpThreads), smem, s, p);
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 
@@ -174,5 +183,6 @@ extern "C" int fb_head_prep(const FbHeadPrepArgs* a, void* stream) {
                          reinterpret_cast<uintptr_t>(a->q_norm) | reinterpret_cast<uintptr_t>(a->k_norm);
   if ((bits & 15) || a->ldp % 8 || a->ldqo % 8 || a->pool_ld % 8) return FB_ERR_ALIGN;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
-  return a->fp32 ? run_head_prep<float>(a, s) : run_head_prep<__nv_bfloat16>(a, s);
+  if (a->fp32) return a->mix ? run_head_prep<float, true>(a, s) : run_head_prep<float, false>(a, s);
+  return a->mix ? run_head_prep<__nv_bfloat16, true>(a, s) : run_head_prep<__nv_bfloat16, false>(a, s);
 }

@@ -384,12 +384,13 @@ def gqa_decode_supported(mixer, dtype, page_size: int) -> bool:
 
 
 def gqa_decode_splits(rows: int, mixer, max_keys: int) -> int:
-    """CTAs per row: about two per SM over the batch (one where a CTA takes all kv heads), each with at least 128 (64) keys of
-    the longest row."""
+    """CTAs per row: about two per SM over the batch (one where it takes all kv heads, or wide ones), each with at least 128
+    (64) keys of the longest row."""
     if mixer.shared_keys:
         ctas, fill, least = rows * ((mixer.heads + 15) // 16), 148, 64
     else:
-        ctas, fill, least = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads * mixer.maps + 15) // 16), 296, 128
+        ctas = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads * mixer.maps + 15) // 16)
+        fill, least = 296 if max(mixer.key_width, mixer.vdim_pad) <= 128 else 148, 128
     visible = mixer.chunk or mixer.window + mixer.keep_first
     splits = 1
     while splits < 8 and ctas * splits * 2 <= fill and min(visible, max_keys) >= splits * 2 * least:
