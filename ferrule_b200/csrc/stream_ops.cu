@@ -200,18 +200,41 @@ norm_rows_kernel(const float* __restrict__ x, long long ldx, int x_rows, const i
 // ---------------------------------------------------------------------------------
 // RMS norm of `groups` equal parts of a row
 // ---------------------------------------------------------------------------------
-// shared memory of one CTA: sums of squares of 8 elements each (of single ones when a part is no multiple of 8), then the
-// inverse root mean square of every part
+// Sums of squares meet in shared memory: of a warp's 256 consecutive elements each when parts are multiples of that, else of
+// 8 elements each (of single ones when a part is no multiple of 8), followed by the inverse root mean square of every part.
 struct GroupScratch {
   float* sums;
   float* inv;
-  float (*red)[32];
+  float (*red)[64];
 };
 
 template <int VPT>
 __device__ __forceinline__ void group_norm(const float (&v)[VPT][8], int dim, int groups, float eps, const GroupScratch& g,
                                            int turn, float (&out)[VPT][8]) {
   const int part = dim / groups;
+  if (part % 256 == 0) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8;
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[k][j], v[k][j], ss);
+      ss = warp_sum(ss);
+      if (lane == 0 && i < dim) g.red[turn][i / 256] = ss;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * 8, n = part / 256, first = i < dim ? i / part * n : 0;
+      float ss = 0.f;
+      for (int w = 0; w < n; ++w) ss += g.red[turn][first + w];
+      const float f = 1.f / sqrtf(ss / part + eps);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) out[k][j] = v[k][j] * f;
+    }
+    return;
+  }
   if (groups == 1) {
     float ss = 0.f;
 #pragma unroll
@@ -285,7 +308,7 @@ __global__ void __launch_bounds__(kRowThreads)
 sandwich_step_kernel(const SandwichParams<T> p) {
   pdl_launch_dependents();
   extern __shared__ float group_sm[];
-  __shared__ float red[2][32];
+  __shared__ float red[2][64];
   const GroupScratch g{group_sm, group_sm + p.n_sums, red};
   const int r = blockIdx.x;
   pdl_wait();
@@ -366,7 +389,7 @@ sandwich_rows_kernel(const float* __restrict__ x, long long ldx, int x_rows, con
                      int n_sums, float eps, DeviceStatus* st) {
   pdl_launch_dependents();
   extern __shared__ float group_sm[];
-  __shared__ float red[2][32];
+  __shared__ float red[2][64];
   const GroupScratch g{group_sm, group_sm + n_sums, red};
   pdl_wait();
   int r = rows_idx[blockIdx.x];

@@ -179,7 +179,8 @@ ATTENTIONS = [talking(6, 3, 20, 0.3, 9), talking(1, 1, 64, 0.3, 1, 2), talking(8
               talking(16, 4, 128, 0.3, 64), differential(4, 2, 12, 20, 0.3, 10, 3, 0.4), differential(3, 3, 64, 64, 0.3, 37, 70, 0.8),
               differential(8, 1, 32, 128, 0.3, 96, 0, 0.1), differential(10, 1, 64, 80, 0.3, 1000, 4, 0.5),
               differential(2, 2, 128, 256, 0.3, 1, 1, 0.2)]
-WIDE = [talking(9, 9, 96, 0.3, 40), talking(8, 8, 128, 0.3, 100, 3), talking(4, 2, 200, 0.3, 33)]
+WIDE = [talking(9, 9, 96, 0.3, 40), talking(8, 8, 128, 0.3, 100, 3), talking(40, 2, 72, 0.3, 50), talking(32, 4, 128, 0.3, 60),
+        talking(4, 2, 200, 0.3, 33)]
 
 
 def visible(m, p):
@@ -259,7 +260,7 @@ def test_attention_in_windows(ops, dtype, m, page):
 
 
 @pytest.mark.parametrize("page,splits,early", [(16, 1, False), (64, 2, False), (8, 4, True), (16, 8, True)])
-@pytest.mark.parametrize("m", ATTENTIONS + WIDE[:2], ids=ids_of)
+@pytest.mark.parametrize("m", ATTENTIONS + WIDE, ids=ids_of)
 def test_attention_of_few_rows(ops, m, page, splits, early):
     KL = ops[1]
     assert KL.gqa_decode_supported(m, BF, page)
