@@ -103,8 +103,9 @@ def main() -> None:
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--model", default="deepseek-v2-lite",
                     help="deepseek-v2-lite is the headline configuration; gitozen-lite, gitozen-latent-lite and supisun-lite are "
-                         "layer-list models of the same widths (one GPU), supisun-small and supisun-wide others, and "
-                         "gitozen-dense-small / -lite / -wide have their sizes; they are reported without a baseline")
+                         "layer-list models of the same widths (one GPU), supisun-small and supisun-wide others, "
+                         "gitozen-dense-small / -lite / -wide have their sizes; vedadra-small / -lite / -wide and "
+                         "supisun-attention-small / -lite / -wide of the same sizes; they are reported without a baseline")
     ap.add_argument("--weight-format", default="bf16", choices=["bf16", "fp8_block", "fp8_mxfp4"],
                     help="bf16 is the headline configuration; the FP8 formats are reported with their own dtype")
     ap.add_argument("--shard-as", type=int, default=0,
