@@ -14,10 +14,11 @@
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
 //     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
 //     before the current P is waited for.
-//   Softmax (warps 2..5, one row per thread): scores from TMEM, scale, distance bias, mask, running maximum, exp2, bf16 P
-//     written over the score buffer.  The accumulator is rescaled only when a row's maximum has grown by more than 2^8
-//     since the reference it was scaled by; the sum uses the same reference, so the result is exact up to rounding.  The
-//     difference of a head's two maps is taken between neighbouring lanes, its RMS norm and the output gate on the way out.
+//   Softmax (warps 2..9, two threads per row with half of the tile's columns each): scores from TMEM, scale, distance bias,
+//     mask, running maximum (the halves meet in shared memory), exp2, bf16 P written over the score buffer.  The
+//     accumulator is rescaled only when a row's maximum has grown by more than 2^8 since the reference it was scaled by;
+//     the sum uses the same reference, so the result is exact up to rounding.  The difference of a head's two maps is
+//     taken between neighbouring lanes, its RMS norm and the output gate on the way out.
 //
 // A row's result depends on the row and the cache contents, not on which rows share its tile or how a prompt was cut.
 // Every wait is bounded (status word, then teardown with TMEM freed); page ids are range-checked.
@@ -31,7 +32,7 @@
 
 namespace fb {
 
-constexpr int kGpThreads = 192;
+constexpr int kGpThreads = 320;
 constexpr int kGpM = 128;
 constexpr int kGpKv = 64;
 constexpr int kGpQBlock = kGpM * 128;         // bytes of a 64-feature block of the query tile
@@ -64,7 +65,7 @@ struct GpParams {
 constexpr float kLog2e = 1.4426950408889634f;
 
 template <bool BIAS>
-__global__ void __launch_bounds__(kGpThreads)
+__global__ void __launch_bounds__(kGpThreads, 2)
 gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                       const __grid_constant__ CUtensorMap map_v, const GpParams p) {
   extern __shared__ uint8_t smem_raw[];
@@ -84,6 +85,9 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   uint64_t* o_done = bars + 17;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 18);
   volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(bars + 19);
+  // exchange between the two halves of a row: maxima [tile parity][half][row] (bf16, rounded up), after the loop sums [half][row]
+  __nv_bfloat16* max_x = reinterpret_cast<__nv_bfloat16*>(bars + 20);
+  float* sum_x = reinterpret_cast<float*>(bars + 20);
   const int k_mask = p.ks - 1, k_shift = p.ks == 4 ? 2 : 1;
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -118,7 +122,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       mbar_init(v_full + i, 1);
       mbar_init(v_free + i, 1);
       mbar_init(s_full + i, 1);
-      mbar_init(p_full + i, 4);
+      mbar_init(p_full + i, 8);
     }
     mbar_init(o_done, 1);
     *abort_flag = 0;
@@ -254,8 +258,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
     }
   } else {
-    // ------------------------------------------------------------------ softmax + epilogue: one row per thread
-    const int quarter = warp & 3;
+    // ------------------------------------------------------------------ softmax + epilogue: two threads per row
+    const int quarter = warp & 3, half = (warp - 2) >> 2;
     const int r = quarter * 32 + lane;
     const int at = r / p.per, head = (g * p.per + r - at * p.per) / p.maps;
     const bool valid = at < nrows;
@@ -264,27 +268,28 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int lo = p.span.first(pos), keep = p.span.keep;
     const float slope = BIAS && valid ? p.slopes[head] * kLog2e : 0.f;
     const uint32_t lane_base = tmem + (static_cast<uint32_t>(quarter * 32) << 16);
+    auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory"); };
     float m_ref = -INFINITY, l_sum = 0.f;
     bool ok = true;
     for (int j = 0; j < n_kv; ++j) {
       const uint32_t s_t = lane_base + col_s + (j & 1) * kGpKv;
-      ok = mbar_wait(s_full + (j & 1), (j >> 1) & 1, abort_flag, p.status, 0xAB0);
-      ok = __all_sync(0xffffffffu, ok);
-      if (!ok) break;
+      // a wait that gives up leaves its mark in the status word; the loop goes on so that the barriers stay in step
+      ok = mbar_wait(s_full + (j & 1), (j >> 1) & 1, abort_flag, p.status, 0xAB0) && ok;
+      __syncwarp();
       tc_fence_after();
-      uint32_t sv[4][16];
+      uint32_t sv[2][16];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) tmem_ld16(s_t + c * 16, sv[c]);
+      for (int c = 0; c < 2; ++c) tmem_ld16(s_t + half * 32 + c * 16, sv[c]);
       tmem_ld_wait();
-      const int tok0 = tile_of(j) * kGpKv;
-      // one warp per scheduler: four independent chains for the maximum and the sum, packed multiply-adds
+      const int tok0 = tile_of(j) * kGpKv + half * 32;
+      // four independent chains for the maximum and the sum, packed multiply-adds
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (BIAS) {
         // the score in base 2 with its distance bias
         const float b0 = slope * static_cast<float>(tok0 - pos);
         const uint64_t sc2 = pack2(p.scale_log2, p.scale_log2), sl2 = pack2(slope, slope), b02 = pack2(b0, b0);
 #pragma unroll
-        for (int c = 0; c < 4; ++c)
+        for (int c = 0; c < 2; ++c)
 #pragma unroll
           for (int i = 0; i < 16; i += 2) {
             const uint64_t bias = fma2(sl2, pack2(static_cast<float>(c * 16 + i), static_cast<float>(c * 16 + i + 1)), b02);
@@ -294,38 +299,47 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             sv[c][i + 1] = __float_as_uint(x1);
           }
       }
-      if (__all_sync(0xffffffffu, tok0 + kGpKv <= hi && (tok0 >= lo || tok0 + kGpKv <= keep))) {
+      if (__all_sync(0xffffffffu, tok0 + 32 <= hi && (tok0 >= lo || tok0 + 32 <= keep))) {
 #pragma unroll
         for (int i = 0; i < 16; ++i)
 #pragma unroll
-          for (int c = 0; c < 4; ++c) mx4[c] = fmaxf(mx4[c], __uint_as_float(sv[c][i]));
+          for (int c = 0; c < 2; ++c) mx4[2 * c + (i & 1)] = fmaxf(mx4[2 * c + (i & 1)], __uint_as_float(sv[c][i]));
       } else {
 #pragma unroll
         for (int i = 0; i < 16; ++i)
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < 2; ++c) {
             const int t = tok0 + c * 16 + i;
             const float x = ((t >= lo || t < keep) && t < hi) ? __uint_as_float(sv[c][i]) : -INFINITY;
             sv[c][i] = __float_as_uint(x);
-            mx4[c] = fmaxf(mx4[c], x);
+            mx4[2 * c + (i & 1)] = fmaxf(mx4[2 * c + (i & 1)], x);
           }
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       if (!BIAS) mx *= p.scale_log2;                          // the scale is positive
+      {
+        // both halves see the same two rounded maxima; behind the barrier both have read their scores
+        __nv_bfloat16* slot = max_x + (j & 1) * 256;
+        const __nv_bfloat16 mine = __float2bfloat16_ru(mx);
+        slot[half * 128 + r] = mine;
+        tc_fence_before();
+        pair_sync();
+        tc_fence_after();
+        mx = fmaxf(__bfloat162float(mine), __bfloat162float(slot[(half ^ 1) * 128 + r]));
+      }
       const float m_new = fmaxf(m_ref, mx);
       if (j == 0) {
         m_ref = m_new;                                        // nothing accumulated yet
       } else if (__any_sync(0xffffffffu, m_new > m_ref + 8.f)) {
-        // rescale this warp's 32 accumulator rows: the previous product must have retired
-        ok = mbar_wait(v_free + ((j - 1) & 1), ((j - 1) >> 1) & 1, abort_flag, p.status, 0xAB2);
-        ok = __all_sync(0xffffffffu, ok);
-        if (!ok) break;
+        // rescale this warp's share of 32 accumulator rows: the previous product must have retired
+        ok = mbar_wait(v_free + ((j - 1) & 1), ((j - 1) >> 1) & 1, abort_flag, p.status, 0xAB2) && ok;
+        __syncwarp();
         tc_fence_after();
         const float f = (m_new == -INFINITY) ? 1.f : exp2f(m_ref - m_new);
         m_ref = m_new;
         l_sum *= f;
 #pragma unroll 1
-        for (int c = 0; c < vb * 4; ++c) {
+        for (int c = half; c < vb * 4; c += 2) {
           uint32_t ov[16];
           tmem_ld16(lane_base + c * 16, ov);
           tmem_ld_wait();
@@ -336,117 +350,97 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
       const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
       const uint64_t scale2 = pack2(p.scale_log2, p.scale_log2), ref2 = pack2(-m_use, -m_use);
-      uint64_t add[4] = {0ull, 0ull, 0ull, 0ull};
+      uint64_t add[2] = {0ull, 0ull};
+      uint32_t pk[16];
 #pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        uint32_t pk[16];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const uint64_t x = pack2(__uint_as_float(sv[2 * c + (i >> 3)][(2 * i) & 15]),
-                                   __uint_as_float(sv[2 * c + (i >> 3)][((2 * i) & 15) + 1]));
-          float p0, p1;
-          unpack2(BIAS ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
-          p0 = exp2_ftz(p0);
-          p1 = exp2_ftz(p1);
-          add[i & 3] = add2(add[i & 3], pack2(p0, p1));
-          pk[i] = pack_bf16x2(p0, p1);
-        }
-        tmem_st16(s_t + c * 16, pk);
+      for (int i = 0; i < 16; ++i) {
+        const uint64_t x = pack2(__uint_as_float(sv[i >> 3][(2 * i) & 15]), __uint_as_float(sv[i >> 3][((2 * i) & 15) + 1]));
+        float p0, p1;
+        unpack2(BIAS ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
+        p0 = exp2_ftz(p0);
+        p1 = exp2_ftz(p1);
+        add[i & 1] = add2(add[i & 1], pack2(p0, p1));
+        pk[i] = pack_bf16x2(p0, p1);
       }
+      tmem_st16(s_t + half * 16, pk);
       float add_lo, add_hi;
-      unpack2(add2(add2(add[0], add[1]), add2(add[2], add[3])), add_lo, add_hi);
+      unpack2(add2(add[0], add[1]), add_lo, add_hi);
       l_sum += add_lo + add_hi;
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(p_full + (j & 1));
     }
-    if (ok) {
-      ok = mbar_wait(o_done, 0, abort_flag, p.status, 0xAB1);
-      ok = __all_sync(0xffffffffu, ok);
-    }
-    if (ok) {
-      tc_fence_after();
-      const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-      const __nv_bfloat16* gate = p.gate ? p.gate + static_cast<long long>(row0 + at) * p.ldg + static_cast<long long>(head) * p.vdim_pad
-                                         : nullptr;
-      if (p.maps == 2) {
-        // rows of a head's two maps are neighbouring lanes: both compute the difference, each writes half of it
-        const bool second = lane & 1;
-        const float own = second ? -p.diff_lambda * inv : inv;
-        float ss = 0.f;
-#pragma unroll 1
-        for (int c = 0; c < vb * 4; ++c) {
-          uint32_t ov[16];
-          tmem_ld16(lane_base + c * 16, ov);
-          tmem_ld_wait();
+    ok = mbar_wait(o_done, 0, abort_flag, p.status, 0xAB1) && ok;
+    ok = __all_sync(0xffffffffu, ok);
+    tc_fence_after();
+    pair_sync();                                              // the last maxima are read: their place takes the sums
+    sum_x[half * 128 + r] = l_sum;
+    pair_sync();
+    l_sum += sum_x[(half ^ 1) * 128 + r];
+    const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+    __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
+    const __nv_bfloat16* gate = p.gate ? p.gate + static_cast<long long>(row0 + at) * p.ldg + static_cast<long long>(head) * p.vdim_pad
+                                       : nullptr;
+    const int chunks = (p.vdim_pad + 15) / 16;                // of 16 columns: every second one per half
+    // eight columns of a row: output gate, rounding, store
+    auto finish = [&](float (&d)[8], int col) {
+      if (!valid || !ok || col >= p.vdim_pad) return;
+      if (gate) {
+        float z[8];
+        act_load8(gate + col, z);
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            const float x = __uint_as_float(ov[i]) * own, d = x + __shfl_xor_sync(0xffffffffu, x, 1);
-            ss = fmaf(d, d, ss);
-          }
-        }
-        const float f = p.diff_scale / sqrtf(ss / p.vdim + p.eps);
-        __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
-#pragma unroll 1
-        for (int c = 0; c < vb * 4; ++c) {
-          if (c * 16 >= p.vdim_pad) break;
-          uint32_t ov[16];
-          tmem_ld16(lane_base + c * 16, ov);
-          tmem_ld_wait();
-          float d[8];
-#pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            const float x = __uint_as_float(ov[i]) * own, y = (x + __shfl_xor_sync(0xffffffffu, x, 1)) * f;
-            if (i < 8) d[i] = y;
-            else if (second) d[i - 8] = y;
-          }
-          const int col = c * 16 + (second ? 8 : 0);
-          if (valid && col < p.vdim_pad) {
-            if (gate) {
-              float z[8];
-              act_load8(gate + col, z);
-#pragma unroll
-              for (int i = 0; i < 8; ++i) d[i] = __fdividef(d[i], 1.f + __expf(-z[i]));
-            }
-            act_store8(dst + col, d);
-          }
-        }
+        for (int i = 0; i < 8; ++i) d[i] = __fdividef(d[i], 1.f + __expf(-z[i]));
       }
-      __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
-      uint4 ahead[2];                                         // the gates of the next 16 columns
-      auto gates = [&](int col) {
-        if (!gate || !valid) return;
-        if (col < p.vdim_pad) ahead[0] = *reinterpret_cast<const uint4*>(gate + col);
-        if (col + 8 < p.vdim_pad) ahead[1] = *reinterpret_cast<const uint4*>(gate + col + 8);
-      };
-      if (p.maps == 1) gates(0);
+      act_store8(dst + col, d);
+    };
+    if (p.maps == 2) {
+      // rows of a head's two maps are neighbouring lanes: both compute the difference, each writes half of it
+      const bool second = lane & 1;
+      const float own = second ? -p.diff_lambda * inv : inv;
+      float ss = 0.f;
 #pragma unroll 1
-      for (int c = 0; c < vb * 4 && p.maps == 1; ++c) {
-        if (c * 16 >= p.vdim_pad) break;
+      for (int c = half; c < chunks; c += 2) {
         uint32_t ov[16];
         tmem_ld16(lane_base + c * 16, ov);
         tmem_ld_wait();
-        if (valid && gate) {
-          const uint4 now[2] = {ahead[0], ahead[1]};
-          gates(c * 16 + 16);
-          const __nv_bfloat16* z = reinterpret_cast<const __nv_bfloat16*>(now);
 #pragma unroll
-          for (int i = 0; i < 16; ++i)
-            ov[i] = __float_as_uint(__fdividef(__uint_as_float(ov[i]), 1.f + __expf(-__bfloat162float(z[i]))));
+        for (int i = 0; i < 16; ++i) {
+          const float x = __uint_as_float(ov[i]) * own, d = x + __shfl_xor_sync(0xffffffffu, x, 1);
+          ss = fmaf(d, d, ss);
         }
-        if (valid) {
-          uint4 w0, w1;
-          w0.x = pack_bf16x2(__uint_as_float(ov[0]) * inv, __uint_as_float(ov[1]) * inv);
-          w0.y = pack_bf16x2(__uint_as_float(ov[2]) * inv, __uint_as_float(ov[3]) * inv);
-          w0.z = pack_bf16x2(__uint_as_float(ov[4]) * inv, __uint_as_float(ov[5]) * inv);
-          w0.w = pack_bf16x2(__uint_as_float(ov[6]) * inv, __uint_as_float(ov[7]) * inv);
-          w1.x = pack_bf16x2(__uint_as_float(ov[8]) * inv, __uint_as_float(ov[9]) * inv);
-          w1.y = pack_bf16x2(__uint_as_float(ov[10]) * inv, __uint_as_float(ov[11]) * inv);
-          w1.z = pack_bf16x2(__uint_as_float(ov[12]) * inv, __uint_as_float(ov[13]) * inv);
-          w1.w = pack_bf16x2(__uint_as_float(ov[14]) * inv, __uint_as_float(ov[15]) * inv);
-          *reinterpret_cast<uint4*>(dst + c * 16) = w0;
-          if (c * 16 + 8 < p.vdim_pad) *reinterpret_cast<uint4*>(dst + c * 16 + 8) = w1;
+      }
+      pair_sync();
+      sum_x[half * 128 + r] = ss;
+      pair_sync();
+      ss += sum_x[(half ^ 1) * 128 + r];
+      const float f = p.diff_scale / sqrtf(ss / p.vdim + p.eps);
+#pragma unroll 1
+      for (int c = half; c < chunks; c += 2) {
+        uint32_t ov[16];
+        tmem_ld16(lane_base + c * 16, ov);
+        tmem_ld_wait();
+        float d[8];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float x = __uint_as_float(ov[i]) * own, y = (x + __shfl_xor_sync(0xffffffffu, x, 1)) * f;
+          if (i < 8) d[i] = y;
+          else if (second) d[i - 8] = y;
+        }
+        finish(d, c * 16 + (second ? 8 : 0));
+      }
+    } else {
+#pragma unroll 2
+      for (int c = half; c < chunks; c += 2) {
+        uint32_t ov[16];
+        tmem_ld16(lane_base + c * 16, ov);
+        tmem_ld_wait();
+#pragma unroll
+        for (int e = 0; e < 16; e += 8) {
+          float d[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) d[i] = __uint_as_float(ov[e + i]) * inv;
+          finish(d, c * 16 + e);
         }
       }
     }
@@ -540,7 +534,7 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   for (int f = p.qb > 4 ? 1 : 0; f < 5 && smem == 0; ++f) {
     p.q_resident = forms[f][0]; p.kb = forms[f][1]; p.ks = forms[f][2];
     if (p.kb > p.qb) p.kb = p.qb;
-    smem = (p.q_resident ? p.qb : p.ks * p.kb) * kGpQBlock + (p.ks * p.kb + 2 * p.vb) * kGpKvBlock + 1024 + 256;
+    smem = (p.q_resident ? p.qb : p.ks * p.kb) * kGpQBlock + (p.ks * p.kb + 2 * p.vb) * kGpKvBlock + 1024 + 160 + 1024;
     if (smem > kGpSmemLimit) smem = 0;
   }
   if (smem == 0) return FB_ERR_LIMIT;
