@@ -8,7 +8,8 @@
 //
 //   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
 //     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
-//     head's width and rows past the sequence are zeros), two stages each with their own barriers.  Wide keys (those of all
+//     head's width and rows past the sequence are zeros; one copy for all blocks when the width is a multiple of 64), two
+//     stages each with their own barriers.  Wide keys (those of all
 //     kv heads side by side) come in pieces of `kb` feature blocks, a stage of up to four each; query rows that do not fit in shared
 //     memory come with them, piece by piece, for every token tile.
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
@@ -52,7 +53,7 @@ struct GpParams {
   KeySpan span;
   int key_width, vdim_pad, qb, vb;     // qb, vb: 64-feature blocks of a query / key row and of a value row
   int kb, pieces, ks, q_resident;      // blocks per key stage, stages per token tile, key stages (2 or 4)
-  int shared_keys;
+  int shared_keys, k_whole, v_whole;   // whole: one copy brings all feature blocks of a stage
   uint32_t tmem_cols;
   float scale_log2;
   const float* slopes;                 // [heads]
@@ -145,7 +146,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 
   if (warp == 0) {
     // ------------------------------------------------------------------ TMA producer
-    if (lane == 0) {
+    if (elect_one()) {
       const uint32_t q_block_tx = static_cast<uint32_t>(p.positions * p.per * 128);
       if (p.q_resident) {
         mbar_arrive_expect_tx(q_full, qb * q_block_tx);
@@ -153,30 +154,36 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
       const int subs = kGpKv / p.box_rows, key_head = p.shared_keys ? 0 : g;
       const long long n_pages = p.pool_rows / p.page_size;
+      const int* pages = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+      auto page_of = [&](int t0) { return t0 < kv_len ? pages[t0 / p.page_size] : -1; };
+      auto row_of = [&](int t0, int page) {
+        if (t0 < kv_len && page >= 0 && page < n_pages) return page * p.page_size + t0 % p.page_size;
+        if (t0 < kv_len) report_status(p.status, kStatusBadIndex, 0xA82, seq, t0);
+        return static_cast<int>(p.pool_rows);                            // out of range: the copy fills zeros
+      };
       bool ok = true;
       int k_armed = 0, v_armed = 0;                                      // key stages / value tiles that were requested
+      int next_page = page_of(tile_of(0) * kGpKv);                       // read a tile ahead
       for (int j = 0; j < n_kv && ok; ++j) {
-        const int st = j & 1;
-        int rowc[8];
-        for (int s = 0; s < subs; ++s) {
-          const int t0 = tile_of(j) * kGpKv + s * p.box_rows;
-          int rc = static_cast<int>(p.pool_rows);                        // out of range: the copy fills zeros
-          if (t0 < kv_len) {
-            const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t0 / p.page_size];
-            if (page >= 0 && page < n_pages) rc = page * p.page_size + t0 % p.page_size;
-            else report_status(p.status, kStatusBadIndex, 0xA82, seq, t0);
-          }
-          rowc[s] = rc;
-        }
+        const int st = j & 1, tok = tile_of(j) * kGpKv;
+        const int row = row_of(tok, next_page);                            // of the tile's first box
+        if (j + 1 < n_kv) next_page = page_of(tile_of(j + 1) * kGpKv);
+        auto sub_row = [&](int s) { return s == 0 ? row : row_of(tok + s * p.box_rows, page_of(tok + s * p.box_rows)); };
         for (int c = 0; c < p.pieces && ok; ++c) {
           const int i = j * p.pieces + c, ks = i & k_mask, b0 = c * p.kb, nb = min(p.kb, qb - b0);
           if (i >= p.ks) ok = mbar_wait(k_free + ks, ((i >> k_shift) - 1) & 1, abort_flag, p.status, 0xA90);
           if (!ok) break;
           mbar_arrive_expect_tx(k_full + ks, nb * (static_cast<uint32_t>(kGpKvBlock) + (p.q_resident ? 0u : q_block_tx)));
-          for (int s = 0; s < subs; ++s)
-            for (int b = 0; b < nb; ++b)
-              tma_load_3d(k_s + (ks * p.kb + b) * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + ks, (b0 + b) * 64, key_head,
-                          rowc[s]);
+          uint8_t* dst = k_s + ks * p.kb * kGpKvBlock;
+          if (p.k_whole) {
+            tma_load_4d(dst, &map_k, k_full + ks, 0, row, b0, key_head);
+          } else {
+            for (int s = 0; s < subs; ++s) {
+              const int rc = sub_row(s);
+              for (int b = 0; b < nb; ++b)
+                tma_load_3d(dst + b * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + ks, (b0 + b) * 64, key_head, rc);
+            }
+          }
           if (!p.q_resident)
             for (int b = 0; b < nb; ++b)
               tma_load_3d(q_s + (ks * p.kb + b) * kGpQBlock, &map_q, k_full + ks, (b0 + b) * 64, g * p.per, row0);
@@ -186,9 +193,15 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (j > 1) ok = mbar_wait(v_free + st, ((j - 2) >> 1) & 1, abort_flag, p.status, 0xA91);
         if (!ok) break;
         mbar_arrive_expect_tx(v_full + st, static_cast<uint32_t>(vb * kGpKvBlock));
-        for (int s = 0; s < subs; ++s)
-          for (int b = 0; b < vb; ++b)
-            tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rowc[s]);
+        if (p.v_whole) {
+          tma_load_4d(v_s + st * vb * kGpKvBlock, &map_v, v_full + st, 0, row, 0, g);
+        } else {
+          for (int s = 0; s < subs; ++s) {
+            const int rc = sub_row(s);
+            for (int b = 0; b < vb; ++b)
+              tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rc);
+          }
+        }
         v_armed = j + 1;
       }
       // after an abort: copies of the last stages may still be in flight, and the CTA may not exit under them
@@ -205,7 +218,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     }
   } else if (warp == 1) {
     // ------------------------------------------------------------------ MMA issuer
-    if (lane == 0) {
+    if (elect_one()) {
       const uint32_t q_addr = smem_u32(q_s), k_addr = smem_u32(k_s), v_addr = smem_u32(v_s);
       constexpr uint32_t idesc_qk = umma_idesc(kGpM, kGpKv, 1, 1);
       const uint32_t idesc_pv = umma_idesc(kGpM, static_cast<uint32_t>(vb * 64), 1, 1) | (1u << 16);   // B is MN-major
@@ -470,6 +483,21 @@ static int gp_map(CUtensorMap* map, const void* base, int width, int heads, uint
   return r == CUDA_SUCCESS ? FB_OK : FB_ERR_DRIVER;
 }
 
+// the same with a head's features as blocks of 64 (width % 64 == 0): box 64 features x 64 rows x box_blocks
+static int gp_map_blocks(CUtensorMap* map, const void* base, int width, int heads, uint64_t rows, long long ld, uint32_t box_blocks) {
+  TcEncodeFn fn = tc_encoder();
+  if (!fn) return FB_ERR_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || width % 64 || ld % 8) return FB_ERR_ALIGN;
+  cuuint64_t dims[4] = {64, rows, static_cast<cuuint64_t>(width / 64), static_cast<cuuint64_t>(heads)};
+  cuuint64_t strides[3] = {static_cast<cuuint64_t>(ld) * 2, 128, static_cast<cuuint64_t>(width) * 2};
+  cuuint32_t box[4] = {64, kGpKv, box_blocks, 1};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, estr,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? FB_OK : FB_ERR_DRIVER;
+}
+
 }  // namespace fb
 
 using namespace fb;
@@ -509,10 +537,6 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   if (rc != FB_OK) return rc;
   const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a->pool);
   p.shared_keys = a->key_stride == 0;
-  rc = gp_map(&mk, pool, a->key_width, p.shared_keys ? 1 : a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
-  if (rc != FB_OK) return rc;
-  rc = gp_map(&mv, pool + a->v_offset, a->vdim_pad, a->kv_heads, static_cast<uint64_t>(a->pool_rows), a->pool_ld, 1, p.box_rows);
-  if (rc != FB_OK) return rc;
   p.tiles = tiles;
   p.block_table = a->block_table;
   p.out = static_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo;
@@ -539,5 +563,16 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   }
   if (smem == 0) return FB_ERR_LIMIT;
   p.pieces = (p.qb + p.kb - 1) / p.kb;
+  const int key_heads = p.shared_keys ? 1 : a->kv_heads;
+  const uint64_t pool_rows = static_cast<uint64_t>(a->pool_rows);
+  p.k_whole = p.box_rows == kGpKv && a->key_width % 64 == 0 && p.qb % p.kb == 0;
+  p.v_whole = p.box_rows == kGpKv && a->vdim_pad % 64 == 0;
+  rc = p.k_whole ? gp_map_blocks(&mk, pool, a->key_width, key_heads, pool_rows, a->pool_ld, p.kb)
+                 : gp_map(&mk, pool, a->key_width, key_heads, pool_rows, a->pool_ld, 1, p.box_rows);
+  if (rc != FB_OK) return rc;
+  const __nv_bfloat16* values = pool + a->v_offset;
+  rc = p.v_whole ? gp_map_blocks(&mv, values, a->vdim_pad, a->kv_heads, pool_rows, a->pool_ld, p.vb)
+                 : gp_map(&mv, values, a->vdim_pad, a->kv_heads, pool_rows, a->pool_ld, 1, p.box_rows);
+  if (rc != FB_OK) return rc;
   return a->slopes ? launch_gp<true>(mq, mk, mv, p, n_tiles, smem, stream) : launch_gp<false>(mq, mk, mv, p, n_tiles, smem, stream);
 }
