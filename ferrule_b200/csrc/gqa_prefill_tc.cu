@@ -555,7 +555,7 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   // query rows that stay in shared memory beside the key stages; rows too wide for that are streamed with the keys
   int smem = 0;
   static const int forms[5][3] = {{1, 4, 2}, {1, 2, 4}, {1, 1, 4}, {0, 2, 2}, {0, 1, 2}};      // resident, kb, ks
-  for (int f = p.qb > 4 ? 1 : 0; f < 5 && smem == 0; ++f) {
+  for (int f = 0; f < 5 && smem == 0; ++f) {
     p.q_resident = forms[f][0]; p.kb = forms[f][1]; p.ks = forms[f][2];
     if (p.kb > p.qb) p.kb = p.qb;
     smem = (p.q_resident ? p.qb : p.ks * p.kb) * kGpQBlock + (p.ks * p.kb + 2 * p.vb) * kGpKvBlock + 1024 + 160 + 1024;
