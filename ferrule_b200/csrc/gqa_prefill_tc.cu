@@ -9,9 +9,9 @@
 //   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
 //     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
 //     head's width and rows past the sequence are zeros; one copy for all blocks when the width is a multiple of 64), two
-//     stages each with their own barriers.  Wide keys (those of all
-//     kv heads side by side) come in pieces of `kb` feature blocks, a stage of up to four each; query rows that do not fit in shared
-//     memory come with them, piece by piece, for every token tile.
+//     stages each with their own barriers.  Wide keys (those of all kv heads side by side) come in pieces of `kb` feature
+//     blocks, a stage each (two or four stages); query rows that do not fit in shared memory come with them, piece by piece,
+//     for every token tile.
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
 //     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
 //     before the current P is waited for.
@@ -21,7 +21,8 @@
 //     the sum uses the same reference, so the result is exact up to rounding.  The difference of a head's two maps is
 //     taken between neighbouring lanes, its RMS norm and the output gate on the way out.
 //
-// A row's result depends on the row and the cache contents, not on which rows share its tile or how a prompt was cut.
+// A row's result depends on the row and the cache contents, not on which rows share its tile or how a prompt was cut,
+// beyond the rounding of a rescale that another row of its warp asked for.
 // Every wait is bounded (status word, then teardown with TMEM freed); page ids are range-checked.
 #include "act_type.cuh"
 #include "attn_tc.cuh"
