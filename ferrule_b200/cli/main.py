@@ -229,7 +229,7 @@ def _expert_plan(args):
 
 
 def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=None):
-    """A layer-list model (Gitozen, Supisun, Vedadra) behind the engine: a checkpoint directory, or a random-init preset."""
+    """A layer-list model (Gitozen, Supisun, Vedadra, Vogunex) behind the engine: a checkpoint directory, or a random-init preset."""
     import torch
 
     from ..models.layered_config import PRESETS, preset_architecture
@@ -262,7 +262,7 @@ def _build_layered_engine(args, dev, model_dir: Optional[str] = None, layout=Non
     ctx, pages_per_seq, sched = _engine_sizes(args, cfg.max_position)
     n_pages = args.max_seqs * pages_per_seq + 8
     if args.kv_cache_mb:
-        per_page = max(len(cfg.cache_runs), 1) * args.page_size * cfg.kv_row_dim * weights.embed.element_size()
+        per_page = max(sum(cfg.plane_dim(cfg.runs[r]) for r in cfg.cache_runs), 64) * args.page_size * weights.embed.element_size()
         n_pages = max(args.kv_cache_mb * (1 << 20) // per_page, pages_per_seq + 1)
     runner = arch.runner(weights, RunnerLimits(n_pages, args.page_size, args.max_batch_tokens, args.max_seqs, ctx), device=dev)
     eng = Engine(runner, EngineConfig(scheduler=sched, kv_pages=n_pages, page_size=args.page_size))
@@ -891,7 +891,7 @@ def main(argv: Optional[List[str]] = None) -> int:
     p.add_argument("--expert-format", default="plain", choices=["plain", "fp8_block", "mxfp4"])
     p.add_argument("--family", default="deepseek", choices=["deepseek", "v4", *LAYERED],
                    help="v4: a DeepSeek-V4 directory (tiny shape; FP8 dense + packed FP4 experts unless --plain); "
-                        "gitozen, supisun, vedadra: a layer-list directory (--preset tiny-<family> unless another of its presets is named)")
+                        "gitozen, supisun, vedadra, vogunex: a layer-list directory (--preset tiny-<family> unless another of its presets is named)")
     p.add_argument("--plain", action="store_true", help="--family v4: keep every linear in BF16")
     p.add_argument("--proposal-stages", type=int, default=0,
                    help="--family v4: also write this many `mtp.*` proposal stages with their prediction heads")

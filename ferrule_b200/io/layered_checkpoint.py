@@ -1,4 +1,4 @@
-"""Checkpoint directories of layer-list models (Gitozen, Supisun, Vedadra): `config.json` with one entry per layer, and safetensors
+"""Checkpoint directories of layer-list models (Gitozen, Supisun, Vedadra, Vogunex): `config.json` with one entry per layer, and safetensors
 files whose tensors are named `embed`, `pos`, `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.rg1`, `final.norm`, `head`
 (`LayeredConfig.tensor_shapes` lists them).  Linear weights are stored [out, in] in BF16."""
 from __future__ import annotations

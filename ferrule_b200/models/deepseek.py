@@ -48,6 +48,7 @@ class DeviceBatch:
     tc_tiles: Optional[torch.Tensor] = None     # [cap, 4] int32 tiles of the tensor-core prefill attention kernel
     n_tc_tiles: int = 0
     tc_positions: int = 0                       # most positions of a tile
+    tc_tables: Optional[dict] = None            # rows per position -> (tiles, tiles in use), with several tables
     rest_ranges: Optional[list] = None          # (first row, end row) ranges the tiles do not cover
     # models with recurrent state (models/state_pool.py)
     seq_start: Optional[torch.Tensor] = None    # [>= n_seqs + 1] int32 first row of every sequence of the batch
@@ -58,40 +59,55 @@ class DeviceBatch:
 
 
 class KvPool:
-    """Physical paged latent-KV pool: [layers, pages, page_size, kv_lora + rope] bf16 (fp32 on CPU)."""
+    """Physical paged pool: per layer [pages, page_size, row width] (bf16; fp32 on CPU).  `row_dims`: row width of every
+    layer; layers of one width share a tensor [layers, pages, page_size, width]."""
 
     def __init__(self, cfg: ModelConfig, n_pages: int, page_size: int, device, dtype=torch.bfloat16,
-                 n_layers: Optional[int] = None):
+                 n_layers: Optional[int] = None, row_dims: Optional[list] = None):
         self.cfg, self.n_pages, self.page_size = cfg, n_pages, page_size
-        self.n_layers = cfg.n_layers + cfg.n_mtp_layers if n_layers is None else n_layers
-        self.data = torch.zeros(self.n_layers, n_pages, page_size, cfg.kv_row_dim, dtype=dtype, device=device)
+        if row_dims is None:
+            row_dims = [cfg.kv_row_dim] * (cfg.n_layers + cfg.n_mtp_layers if n_layers is None else n_layers)
+        self.n_layers = len(row_dims)
+        widths = sorted(set(row_dims)) or [cfg.kv_row_dim]
+        self.planes = [torch.zeros(row_dims.count(w), n_pages, page_size, w, dtype=dtype, device=device) for w in widths]
+        self.where = [(widths.index(w), row_dims[:i].count(w)) for i, w in enumerate(row_dims)]
+
+    @property
+    def data(self) -> torch.Tensor:
+        """All layers of a pool whose rows are equally wide."""
+        assert len(self.planes) == 1
+        return self.planes[0]
 
     def layer(self, i: int) -> torch.Tensor:
-        return self.data[i]
+        group, at = self.where[i]
+        return self.planes[group][at]
 
     @property
     def bytes_per_page(self) -> int:
-        return self.n_layers * self.page_size * self.cfg.kv_row_dim * self.data.element_size()
+        return sum(p.shape[0] * p.shape[2] * p.shape[3] * p.element_size() for p in self.planes)
 
     def copy_pages(self, pairs) -> None:
         """Copy whole pages (all layers): pairs = [(src, dst), ...] (copy-on-write)."""
         if not pairs:
             return
-        if self.data.is_cuda:
-            from ..ops import kernels as K
-            K.copy_pages(self.data, torch.tensor(pairs, dtype=torch.int32, device=self.data.device))
-        else:
-            for s, d in pairs:
-                self.data[:, d] = self.data[:, s]
+        for p in self.planes:
+            if p.is_cuda:
+                from ..ops import kernels as K
+                K.copy_pages(p, torch.tensor(pairs, dtype=torch.int32, device=p.device))
+            else:
+                for s, d in pairs:
+                    p[:, d] = p[:, s]
 
-    def snapshot_pages(self, pages) -> torch.Tensor:
-        """Device -> host copy of pages (session preemption)."""
-        idx = torch.tensor(list(pages), dtype=torch.long, device=self.data.device)
-        return self.data[:, idx].to("cpu", copy=True)
+    def snapshot_pages(self, pages):
+        """Device -> host copy of pages (session preemption): one tensor, or one per row width."""
+        idx = torch.tensor(list(pages), dtype=torch.long, device=self.planes[0].device)
+        out = [p[:, idx].to("cpu", copy=True) for p in self.planes]
+        return out[0] if len(out) == 1 else out
 
-    def restore_pages(self, pages, snap: torch.Tensor) -> None:
-        idx = torch.tensor(list(pages), dtype=torch.long, device=self.data.device)
-        self.data[:, idx] = snap.to(self.data.device)
+    def restore_pages(self, pages, snap) -> None:
+        idx = torch.tensor(list(pages), dtype=torch.long, device=self.planes[0].device)
+        for p, s in zip(self.planes, [snap] if isinstance(snap, torch.Tensor) else snap):
+            p[:, idx] = s.to(p.device)
 
 
 # ======================================================================================

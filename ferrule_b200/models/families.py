@@ -4,7 +4,7 @@ Roles tell the loader what a tensor is (attention projection, norm, router, rout
 weight, scale, MTP part ...) independent of the naming scheme.  Families: DeepSeek (HuggingFace
 V2/V3 names: `model.layers.N.self_attn.q_a_proj.weight`), DeepSeek-V4 (the reference's flat names:
 `layers.N.attn.wq_a.weight`, `ffn.experts.E.w1.weight`, `mtp.M.*`), Gitozen (layer-list names:
-`lN.mix.q`, `lN.mlp.eE.gate`), Supisun and Vedadra (the same scheme), Qwen3 and generic Llama-style.  The DeepSeek families and
+`lN.mix.q`, `lN.mlp.eE.gate`), Supisun, Vedadra and Vogunex (the same scheme), Qwen3 and generic Llama-style.  The DeepSeek families and
 the layer-list ones execute; the others
 are classified for inspection.
 
@@ -50,6 +50,7 @@ class TensorRole(Enum):
     SHARED_GATE = "shared_gate"
     SHARED_UP = "shared_up"
     SHARED_DOWN = "shared_down"
+    SHARED_ROUTER = "shared_router"
     DENSE_GATE = "dense_gate"
     DENSE_UP = "dense_up"
     DENSE_DOWN = "dense_down"
@@ -63,6 +64,7 @@ class TensorRole(Enum):
     SCAN_IN = "scan_in"
     SCAN_PARAM = "scan_param"
     INPUT_CONV = "input_conv"
+    TOKEN_SHIFT = "token_shift"
     POSITION = "position"
     VALUE_MIX = "value_mix"
     HEAD_MIX = "head_mix"
@@ -87,6 +89,7 @@ class Family(Enum):
     GITOZEN = "gitozen"
     SUPISUN = "supisun"
     VEDADRA = "vedadra"
+    VOGUNEX = "vogunex"
     QWEN3 = "qwen3"
     LLAMA = "llama"
 
@@ -117,6 +120,7 @@ _LAYERED_MIX = {"q": TensorRole.ATTN_Q, "k": TensorRole.ATTN_K, "v": TensorRole.
                 "dt": TensorRole.SCAN_PARAM, "dt.b": TensorRole.SCAN_PARAM, "D": TensorRole.SCAN_PARAM,
                 "q.b": TensorRole.ATTN_Q, "k.b": TensorRole.ATTN_K, "o.b": TensorRole.ATTN_OUT,
                 "talk": TensorRole.HEAD_MIX, "temp": TensorRole.HEAD_MIX, "lq1": TensorRole.MAP_WEIGHT,
+                "dq": TensorRole.ATTN_Q_A, "dq.norm": TensorRole.ATTN_Q_NORM, "uq": TensorRole.ATTN_Q_B, "v.b": TensorRole.ATTN_V,
                 "lk1": TensorRole.MAP_WEIGHT, "lq2": TensorRole.MAP_WEIGHT, "lk2": TensorRole.MAP_WEIGHT}
 _LAYERED_FFN = {"gate": 0, "up": 1, "down": 2}
 
@@ -136,8 +140,15 @@ def _classify_layered(name: str) -> "TensorClass":
         return TensorClass(TensorRole.FFN_NORM, layer)
     if rest == "canon1":
         return TensorClass(TensorRole.INPUT_CONV, layer)
-    if rest in ("mlp.gate", "mlp.up", "mlp.down"):
-        return TensorClass(_ffn_role("dense", _LAYERED_FFN[rest[4:]]), layer)
+    if rest == "shift":
+        return TensorClass(TensorRole.TOKEN_SHIFT, layer)
+    m2 = re.fullmatch(r"mlp\.(shared\.)?(gate|up|down)(\.b)?", rest)
+    if m2:
+        return TensorClass(_ffn_role("shared" if m2.group(1) else "dense", _LAYERED_FFN[m2.group(2)]), layer)
+    if rest == "mlp.shared.sg":
+        return TensorClass(TensorRole.SHARED_ROUTER, layer)
+    if rest == "mlp.router.b":
+        return TensorClass(TensorRole.ROUTER_BIAS, layer)
     if re.fullmatch(r"rg[12](\.b)?", rest):
         return TensorClass(TensorRole.RESIDUAL_GATE, layer)
     if rest == "mlp.router":
@@ -158,7 +169,7 @@ def _ffn_role(kind: str, idx: int) -> TensorRole:
 
 
 def classify(name: str, family: Family, n_layers: Optional[int] = None) -> TensorClass:
-    if family in (Family.GITOZEN, Family.SUPISUN, Family.VEDADRA):
+    if family in (Family.GITOZEN, Family.SUPISUN, Family.VEDADRA, Family.VOGUNEX):
         return _classify_layered(name)
     is_scale = name.endswith(_SCALE_SUFFIX)
     base = name
@@ -258,6 +269,8 @@ def detect_family(names: Iterable[str], model_type: str = "") -> Family:
         return Family.SUPISUN
     if "l0.norm1b" in names or model_type.lower() == "vedadra":
         return Family.VEDADRA
+    if "l0.shift" in names or model_type.lower() == "vogunex":
+        return Family.VOGUNEX
     if "l0.norm1" in names or model_type.lower() == "gitozen":
         return Family.GITOZEN
     if any(n.startswith("layers.") and ".attn.wq_a" in n for n in names) or any(n.startswith("mtp.") for n in names):

@@ -22,6 +22,13 @@ Sandwich blocks (every norm an RMS norm in groups):
                 x += norm2b(ff(norm2(x)))
     logits = head . norm_final(x)
 
+Pre-norm blocks:
+
+    x = embed[token] * embed_scale
+    per layer:  x += mixer(shift(norm1(x)))                      (shift: h + (h of the previous token - h) * s)
+                x += ff(norm2(x))
+    logits = head . norm_final(x)
+
 A layer that runs several times has a cache plane and a state per run.
 
 * `LayeredReference` - plain PyTorch; the execution path of a CPU runner.
@@ -53,8 +60,8 @@ import torch.nn.functional as F
 from ..ops import reference as ref
 from .config import SCORE_SOFTMAX
 from .deepseek import DeviceBatch, KvPool, _pow2_at_least
-from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, SANDWICH_NORM, AttentionMixer, DeltaMixer, LatentMixer, MambaMixer,
-                             MoeSpec, WindowMixer, pad_to)
+from .layered_config import (OUTPUT_NORM, PARALLEL_GATED, PRE_NORM, SANDWICH_NORM, AttentionMixer, DeltaMixer, LatentMixer,
+                             Mamba2Mixer, MambaMixer, MoeSpec, WindowMixer, pad_to)
 from .layered_weights import LayerImage, LayeredWeights, MixerImage
 from .state_pool import RecurrentStatePool
 
@@ -79,20 +86,46 @@ class LayeredReference:
         return x * inv * g
 
     def _latent(self, layer: int, mx: MixerImage, m: LatentMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
-        T, DL = proj.shape[0], self.cfg.kv_row_dim
+        T, DL, R, eps = proj.shape[0], m.row_dim, m.rot_dim, self.cfg.norm_eps
         o = mx.off
         dp, vp = pad_to(m.dim, 8), pad_to(m.vdim, 8)
-        q = proj[:, o["q"]:o["q"] + m.heads * dp].view(T, m.heads, dp)
+        q_src, q_off = proj, o
+        if m.q_rank:
+            cq = proj[:, o["dq"]:o["dq"] + m.q_rank]
+            cq = cq * torch.rsqrt(cq.pow(2).mean(-1, keepdim=True) + eps) * mx.dq_norm[:m.q_rank]
+            q_src, q_off = cq @ mx.w_uq[:, :m.q_rank].float().T, mx.off_uq
+        q = q_src[:, q_off["q"]:q_off["q"] + m.heads * dp].view(T, m.heads, dp)
         c = proj[:, o["dkv"]:o["dkv"] + m.kv_rank]
-        c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps) * mx.kv_norm[:m.kv_rank]
+        c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * mx.kv_norm[:m.kv_rank]
         pool = self.pool.layer(self.cache_index[layer]).view(-1, DL)
+        row = torch.zeros(T, DL)
+        row[:, :m.kv_rank] = c
+        q_lat = torch.einsum("thk,hnk->thn", q, mx.w_uk_t.float())
+        if R:
+            a = b.positions[:T].double()[:, None] * rotation_frequencies(m.rot_base, R)
+            cs, sn = torch.cos(a).float()[:, None], torch.sin(a).float()[:, None]
+
+            def turn(t):
+                u, w = t[..., 0::2], t[..., 1::2]
+                return torch.stack([u * cs - w * sn, w * cs + u * sn], -1).flatten(-2)
+
+            at = slice(m.rot_offset, m.rot_offset + R)
+            row[:, at] = turn(proj[:, None, o["dkv"] + m.kv_rank:o["dkv"] + m.kv_rank + R])[:, 0]
+            q_lat[:, :, at] = turn(q_src[:, q_off["qr"]:q_off["qr"] + m.heads * R].view(T, m.heads, R))
         slots = b.write_slot[:T]
         ok = slots >= 0
-        pool[slots[ok], :m.kv_rank] = c[ok].to(pool.dtype)
-        pool[slots[ok], m.kv_rank:] = 0
-        q_lat = torch.einsum("thk,hnk->thn", q, mx.w_uk_t.float())
-        lat = ref.mla_paged_attention(q_lat, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, DL,
-                                      m.scale)
+        pool[slots[ok]] = row[ok].to(pool.dtype)
+        if m.window:
+            lat = torch.zeros(T, m.heads, DL)
+            for r in range(T):
+                p, seq, ps = int(b.row_pos[r]), int(b.row_seq[r]), self.pool.page_size
+                t = torch.arange(max(p - m.window + 1, 0), p + 1)
+                if t.numel():
+                    kv = pool[b.block_table[seq, t // ps].long() * ps + t % ps].float()
+                    lat[r] = torch.softmax(q_lat[r] @ kv.T * m.scale, -1) @ kv
+        else:
+            lat = ref.mla_paged_attention(q_lat, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, DL,
+                                          m.scale)
         v = torch.einsum("thn,hvn->thv", lat, mx.w_uv.float())
         gate = torch.sigmoid(proj[:, o["g"]:o["g"] + m.heads])
         return (v * gate[:, :, None]).reshape(T, m.heads * vp) @ mx.w_o.float().T
@@ -139,20 +172,28 @@ class LayeredReference:
                     tail[sout, :keep] = x[-keep:].to(tail.dtype)
         return out @ mx.w_o.float().T
 
+    @staticmethod
+    def _expert(s: MoeSpec, limit: float, x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor) -> torch.Tensor:
+        g, u = (x @ w13.float().T).chunk(2, -1)
+        if limit:
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        return (g * torch.sigmoid(s.alpha * g) * (u + s.shift)) @ w2.float().T
+
     def _moe(self, lw: LayerImage, h: torch.Tensor) -> torch.Tensor:
         s = lw.spec.mlp
-        idx, wts = ref.route(h @ lw.router_w.float().T, s.top, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep,
+        z = h @ lw.router_w.float().T
+        logits = z[:, :s.experts] if lw.router_b is None else z[:, :s.experts] + lw.router_b
+        idx, wts = ref.route(logits, s.top, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep, normalize=s.renormalize,
                              group_top=1)
         out = torch.zeros_like(h)
-        fp = lw.e_w2.shape[2]
         for e in range(s.experts):
             hit = idx == e
             rows = hit.any(-1).nonzero().flatten()
             if rows.numel() == 0:
                 continue
-            y = h[rows] @ lw.e_w13[e].float().T
-            y = (F.silu(y[:, :fp]) * y[:, fp:]) @ lw.e_w2[e].float().T
-            out[rows] += y * (wts * hit)[rows].sum(-1, keepdim=True)
+            out[rows] += self._expert(s, s.limit, h[rows], lw.e_w13[e], lw.e_w2[e]) * (wts * hit)[rows].sum(-1, keepdim=True)
+        if s.shared_ff:
+            out += torch.sigmoid(z[:, s.experts:]) * self._expert(s, s.shared_limit, h, lw.s_w13, lw.s_w2)
         return out
 
     def _conv(self, x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
@@ -217,37 +258,69 @@ class LayeredReference:
         part = lambda name, heads, pad: proj[:, o[name]:o[name] + heads * pad]
         rms = lambda t, n: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / n + eps)
         q, k = part("q", H * M, dp), part("k", G * M, dp)
-        if m.biases:
+        if mx.q_bias is not None:
             q, k = q + mx.q_bias, k + mx.k_bias
         v = k if m.tied_values else part("v", G, vp)
-        q = rms(q.reshape(T, H, M, dp), D) * mx.q_norm
-        row = torch.zeros(T, self.cfg.kv_row_dim)
-        row[:, :m.v_offset] = (rms(k.reshape(T, G * M, dp), D) * mx.k_norm).view(T, -1)
+        q, k = q.reshape(T, H, M, dp), k.reshape(T, G * M, dp)
+        if m.rot_dims:
+            half = m.rot_dims // 2
+            a = b.positions[:T].double()[:, None] * rotation_frequencies(m.rot_base, m.rot_dims)
+            cs, sn = torch.cos(a).float(), torch.sin(a).float()
+
+            def turn(t):
+                u, w = t[..., :half], t[..., half:2 * half]
+                c_, s_ = (x.view(T, *[1] * (t.dim() - 2), half) for x in (cs, sn))
+                return torch.cat([u * c_ - w * s_, w * c_ + u * s_, t[..., 2 * half:]], -1)
+
+            q, k = turn(q), turn(k)
+        q, k = rms(q, D), rms(k, D)
+        if m.norm_weights:
+            q, k = q * mx.q_norm, k * mx.k_norm
+        rows = self.pool.layer(self.cache_index[run])
+        rows = rows.view(-1, rows.shape[-1])
+        row = torch.zeros(T, rows.shape[1])
+        row[:, :m.v_offset] = k.view(T, -1)
         row[:, m.v_offset:m.v_offset + G * vp] = v
         slots = b.write_slot[:T]
         ok = slots >= 0
-        rows = self.pool.layer(self.cache_index[run]).view(-1, self.cfg.kv_row_dim)
         rows[slots[ok]] = row[ok].to(rows.dtype)
         out, ps = torch.zeros(T, H, vp), self.pool.page_size
+        at = lambda seq, t: rows[b.block_table[seq, t // ps].long() * ps + t % ps].float()
+        pooled = None
+        if m.pool:
+            for r in range(T):
+                p, seq = int(b.row_pos[r]), int(b.row_seq[r])
+                if (p + 1) % m.pool == 0 and p >= 0:
+                    self.states.pooled[run][int(b.state_out[seq]) // self.states.buffers, p // m.pool] = (
+                        at(seq, torch.arange(p + 1 - m.pool, p + 1)).mean(0).to(rows.dtype))
         for r in range(T):
             p, seq = int(b.row_pos[r]), int(b.row_seq[r])
             first = max(p - m.window + 1, 0)
             t = torch.cat([torch.arange(min(m.keep_first, first)), torch.arange(first, p + 1)])
             if t.numel() == 0:
                 continue
-            kv = rows[b.block_table[seq, t // ps].long() * ps + t % ps].float()
+            kv = at(seq, t)
+            if m.pool:
+                blocks = max(p - m.window + 1, 0) // m.pool
+                pooled = self.states.pooled[run][int(b.state_out[seq]) // self.states.buffers, :blocks]
+                kv = torch.cat([pooled.float(), kv])
             k = kv[:, :m.v_offset].view(-1, G, M, dp).repeat_interleave(H // G, 1)
             v = kv[:, m.v_offset:m.v_offset + G * vp].view(-1, G, vp).repeat_interleave(H // G, 1)
             s = torch.einsum("hmd,thmd->hmt", q[r], k)
             s = torch.einsum("hg,gmt->hmt", mx.q_mix, s) if m.mix_heads else s * mx.q_mix[:, None, None]
             if m.distance_bias:
                 s = s - (mx.slopes[:, None] * (p - t))[:, None]
-            a = torch.einsum("hmt,thv->hmv", torch.softmax(s, -1), v)
+            if m.softcap:
+                s = m.softcap * torch.tanh(s / m.softcap)
+            s = torch.softmax(s, -1)
+            if m.mix_weights:
+                s = torch.einsum("hg,gmt->hmt", mx.talk, s)
+            a = torch.einsum("hmt,thv->hmv", s, v)
             out[r] = a[:, 0] if M == 1 else rms(a[:, 0] - mx.diff_lambda * a[:, 1], V) * (1 - m.diff)
         if m.gate:
             out = out * torch.sigmoid(part("g", H, vp).reshape(T, H, vp))
         y = out.view(T, H * vp) @ mx.w_o.float().T
-        return y + mx.o_bias if m.biases else y
+        return y if mx.o_bias is None else y + mx.o_bias
 
     def _mamba(self, layer: int, mx: MixerImage, m: MambaMixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
         o, Ip, N = mx.off, m.inner_pad, m.state
@@ -266,10 +339,30 @@ class LayeredReference:
                 state[sout] = S
         return (y * F.silu(proj[:, o["z"]:o["z"] + Ip])) @ mx.w_o.float().T
 
+    def _mamba2(self, layer: int, mx: MixerImage, m: Mamba2Mixer, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        o, H, V, N, G, I, T = mx.off, m.heads, m.vdim, m.state, m.groups, m.inner, proj.shape[0]
+        xbc = F.silu(self._conv(proj[:, :m.channels], mx.conv, self.states.tail[layer], b) + mx.conv_b)
+        x = xbc[:, :I].view(T, H, V)
+        B, C = (xbc[:, at:at + G * N].view(T, G, N).repeat_interleave(H // G, 1) for at in (mx.off_b, mx.off_c))
+        dt = F.softplus(proj[:, o["dt"]:o["dt"] + H] + mx.dt_bias)
+        decay = torch.exp(mx.a_neg * dt)
+        state, y = self.states.state[layer], torch.zeros(T, m.inner_pad)
+        for s in range(b.n_seqs):
+            sin, sout = int(b.state_in[s]), int(b.state_out[s])
+            S = state[sin].clone() if sin >= 0 else torch.zeros(H, N, V)
+            for r in range(int(b.seq_start[s]), int(b.seq_start[s + 1])):
+                S = decay[r][:, None, None] * S + B[r][:, :, None] * (dt[r][:, None] * x[r])[:, None]
+                y[r, :I] = (torch.einsum("hn,hnv->hv", C[r], S) + mx.d_skip[:, None] * x[r]).flatten()
+            if sout >= 0:
+                state[sout] = S
+        y = (y * F.silu(proj[:, o["z"]:o["z"] + m.inner_pad]))[:, :I].view(T, m.norm_groups, -1)
+        y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + self.cfg.norm_eps)).view(T, I) * mx.o_norm[:I]
+        return y @ mx.w_o[:, :I].float().T
+
     def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
         m = lw.spec.mixer
         fn = {LatentMixer: self._latent, AttentionMixer: self._attention, WindowMixer: self._window,
-              DeltaMixer: self._delta, MambaMixer: self._mamba}[type(m)]
+              DeltaMixer: self._delta, MambaMixer: self._mamba, Mamba2Mixer: self._mamba2}[type(m)]
         return fn(layer, lw.mixer, m, proj, b)
 
     def _gated_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
@@ -308,13 +401,43 @@ class LayeredReference:
             x = x + norm((F.gelu(g, approximate="tanh") * u) @ lw.w_down.float().T, lw.norm2b)
         return x
 
+    def _shift(self, h: torch.Tensor, s: torch.Tensor, plane: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        """Rows moved towards their sequence's previous row, which the state plane holds for the first one."""
+        before = torch.zeros_like(h)
+        for q in range(b.n_seqs):
+            r0, r1 = int(b.seq_start[q]), int(b.seq_start[q + 1])
+            sin, sout = int(b.state_in[q]), int(b.state_out[q])
+            if sin >= 0:
+                before[r0] = plane[sin]
+            before[r0 + 1:r1] = h[r0:r1 - 1]
+            if sout >= 0:
+                plane[sout] = h[r1 - 1]
+        return h + (before - h) * s
+
+    def _pre_norm_layer(self, i: int, lw: LayerImage, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
+        mx = lw.mixer
+        h = self._norm(x, lw.norm1)
+        if lw.shift is not None:
+            h = self._shift(h, lw.shift, self.states.shift[i], b)
+        proj = h @ mx.w_in.float().T
+        x = x + self._mixer(i, lw, proj if mx.b_in is None else proj + mx.b_in, b)
+        if isinstance(lw.spec.mlp, MoeSpec):
+            x = x + self._moe(lw, self._norm(x, lw.norm2))
+        elif lw.spec.mlp is not None:
+            u = self._norm(x, lw.norm2) @ lw.w_up.float().T
+            y = F.gelu(u if lw.up_b is None else u + lw.up_b) @ lw.w_down.float().T
+            x = x + (y if lw.down_b is None else y + lw.down_b)
+        return x
+
     def hidden_states(self, b: DeviceBatch, allreduce=None, start_layer: int = 0, h0=None) -> torch.Tensor:
         """Residual stream after the last layer [rows, width_pad]."""
         x = embedded = self.w.embed[b.token_ids[:b.n_rows].long()].float()
+        if self.cfg.embed_scale != 1.0:
+            x = x * self.cfg.embed_scale
         if self.w.pos is not None:
             x = x + self.w.pos[b.positions[:b.n_rows].long()].float()
         layer = {PARALLEL_GATED: self._gated_layer, OUTPUT_NORM: self._output_norm_layer,
-                 SANDWICH_NORM: self._sandwich_layer}[self.cfg.block]
+                 SANDWICH_NORM: self._sandwich_layer, PRE_NORM: self._pre_norm_layer}[self.cfg.block]
         for i, l in enumerate(self.cfg.runs):
             if self.prof is not None:
                 self.prof.mark(i, "layer")
@@ -326,7 +449,8 @@ class LayeredReference:
         return x
 
     def logits_from_hidden(self, x: torch.Tensor, b: DeviceBatch) -> torch.Tensor:
-        norm = {PARALLEL_GATED: self._norm, OUTPUT_NORM: self._layer_norm, SANDWICH_NORM: self._group_norm}[self.cfg.block]
+        norm = {PARALLEL_GATED: self._norm, OUTPUT_NORM: self._layer_norm, SANDWICH_NORM: self._group_norm,
+                PRE_NORM: self._norm}[self.cfg.block]
         logits = norm(x[b.logit_rows[:b.n_logit].long()], self.w.final_norm) @ self.w.lm_head.float().T
         cap = self.cfg.logit_softcap
         return cap * torch.tanh(logits / cap) if cap else logits

@@ -32,7 +32,7 @@ class LayeredRunner(DeepSeekRunner):
                  max_seq_len: int = 4096, device=None, use_graphs: bool = True, attn_splits: int = 8, lookahead: bool = True,
                  full_logit_rows: int = 0):
         self.states = RecurrentStatePool(weights.cfg, max_seqs, weights.embed.device, weights.embed.dtype,
-                                         buffers=3 if lookahead else 2)
+                                         buffers=3 if lookahead else 2, max_tokens=max_seq_len)
         self.full_logit_rows = full_logit_rows          # logit rows per head pass of batches that ask for whole rows
         self.seq_state: Dict[int, SequenceStateCore] = {}
         self._binds: Dict[int, List[tuple]] = {}
@@ -43,21 +43,17 @@ class LayeredRunner(DeepSeekRunner):
     # ------------------------------------------------------------------ parts
     def _make_pool(self, n_pages: int) -> KvPool:
         return KvPool(self.cfg, n_pages, self.page_size, self.device, dtype=self.w.embed.dtype,
-                      n_layers=len(self.cfg.cache_runs))
+                      row_dims=[self.cfg.plane_dim(self.cfg.runs[r]) for r in self.cfg.cache_runs])
 
-    def _prefill_tc_heads(self) -> int:
-        from ..ops.kernels import prefill_tc_supported
-        grouped = self.cfg.attention_layers + self.cfg.window_layers
-        if grouped:
-            # one tile table for all layers: as many positions as the widest group of query heads leaves room for
-            from ..ops.layered import gqa_tc_group
-            return max(gqa_tc_group(self.cfg.layers[i].mixer, self.w.embed.dtype, self.page_size)
-                       for i in grouped)
-        heads = {self.cfg.layers[i].mixer.heads for i in self.cfg.latent_layers}
-        if len(heads) != 1 or self.w.embed.dtype != torch.bfloat16:
-            return 0
-        n = heads.pop()
-        return n if prefill_tc_supported(n, self.cfg.kv_row_dim, 0, self.page_size) else 0
+    def _prefill_tc_heads(self) -> tuple:
+        """Rows per position of the tile tables: one for all grouped-query layers (as many positions as the widest group of
+        query heads leaves room for), one for every head count of the latent layers."""
+        from ..ops.layered import gqa_tc_group, latent_tc_group
+        mixer = lambda i: self.cfg.layers[i].mixer
+        grouped = [gqa_tc_group(mixer(i), self.w.embed.dtype, self.page_size)
+                   for i in self.cfg.attention_layers + self.cfg.window_layers]
+        latent = {latent_tc_group(mixer(i), self.w.embed.dtype, self.page_size) for i in self.cfg.latent_layers}
+        return tuple(sorted({max(grouped, default=0), *latent} - {0}))
 
     def _make_staging(self, rows: int, seqs: int, prefill: bool = False) -> BatchStaging:
         return BatchStaging(rows, seqs, self.max_blocks, self.device,
@@ -81,8 +77,13 @@ class LayeredRunner(DeepSeekRunner):
                                      supports_provisional=False, supports_full_logits=True)
 
     def kv_schema(self) -> KvLayoutSchema:
-        return KvLayoutSchema((KvPlaneDescriptor("latent_kv" if self.cfg.latent_layers else "kv", self.cfg.kv_row_dim, self.pool.n_layers),), self.page_size,
-                              self.max_seq_len)
+        layer = lambda i: self.cfg.runs[self.cfg.cache_runs[i]]
+        kinds = {}
+        for i in range(self.pool.n_layers):
+            key = ("latent_kv" if layer(i) in self.cfg.latent_layers else "kv", self.cfg.plane_dim(layer(i)))
+            kinds[key] = kinds.get(key, 0) + 1
+        planes = tuple(KvPlaneDescriptor(name, width, n) for (name, width), n in sorted(kinds.items(), reverse=True))
+        return KvLayoutSchema(planes or (KvPlaneDescriptor("kv", self.cfg.kv_row_dim, 0),), self.page_size, self.max_seq_len)
 
     def prepare_batch(self, txn_id: int, batch: ExecutionBatch) -> None:
         for s in batch.sequences:

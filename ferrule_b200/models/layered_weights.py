@@ -3,13 +3,15 @@
 Every linear that reads the mixer's input is one row block of a single matrix `w_in`, so a layer starts with one GEMM;
 blocks begin at multiples of 8 columns of its output:
 
-  latent layer     q (heads x dim, each head padded to 8) | dkv | head gates
+  latent layer     q (heads x dim, each head padded to 8) | rotated q (heads x rot_dim) | dkv | head gates; queries with a
+                   latent of their own: dq | dkv | head gates, and q | rotated q are row blocks of `w_uq`
   attention layer  q | k | v, each head padded to 8
   window layer     q | k | v (unless the keys are the values) | output gate, each head padded to 8
   delta layer      q | k | v | decay low rank | gate low rank | beta      (full projections: decay | gate | beta)
   mamba layer      x | z
+  mamba2 layer     x | B | C | z | dt
 
-followed, in parallel gated blocks, by residual gate 1 | residual gate 2.
+(`b_in`: biases of the projection, added by the GEMM) followed, in parallel gated blocks, by residual gate 1 | residual gate 2.
 
 The second halves of the delta layer's two low-rank projections are one block-diagonal matrix `w_ag` (fp32 output:
 decay pre-activations and output-gate pre-activations).  Keys and values of a latent layer are absorbed: `w_uk_t` maps a
@@ -26,8 +28,8 @@ from typing import Callable, Dict, List, Optional
 
 import torch
 
-from .layered_config import (PARALLEL_GATED, SANDWICH_NORM, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer, LayeredConfig,
-                             LayerSpec, MambaMixer, MoeSpec, WindowMixer, pad_to)
+from .layered_config import (PARALLEL_GATED, PRE_NORM, SANDWICH_NORM, AttentionMixer, DeltaMixer, DenseSpec, LatentMixer,
+                             LayeredConfig, LayerSpec, Mamba2Mixer, MambaMixer, MoeSpec, WindowMixer, pad_to)
 
 GetTensor = Callable[[str], torch.Tensor]
 
@@ -46,10 +48,14 @@ class MixerImage:
     w_in: torch.Tensor                       # [sum of blocks, width_pad]
     off: Dict[str, int]                      # block name -> first output column
     w_o: torch.Tensor                        # [width_pad, inputs]
+    b_in: Optional[torch.Tensor] = None      # fp32, one per row of w_in
     # latent attention
     w_uk_t: Optional[torch.Tensor] = None    # [heads, row_dim, dim_pad]
     w_uv: Optional[torch.Tensor] = None      # [heads, vdim_pad, row_dim]
     kv_norm: Optional[torch.Tensor] = None   # fp32 [row_dim]
+    w_uq: Optional[torch.Tensor] = None      # [heads * dim_pad | heads * rot_dim, q_rank padded to 8]
+    off_uq: Dict[str, int] = field(default_factory=dict)     # its blocks: q, qr
+    dq_norm: Optional[torch.Tensor] = None   # fp32 [q_rank padded to 8]
     # delta rule
     w_ag: Optional[torch.Tensor] = None      # [heads * dim | heads * vdim, low ranks]
     off_gate: int = 0
@@ -68,6 +74,7 @@ class MixerImage:
     q_mix: Optional[torch.Tensor] = None     # fp32 [heads, heads]: factor of head g's raw scores in head h's; not mixed: [heads]
     slopes: Optional[torch.Tensor] = None    # fp32 [heads]: taken off a score per token of distance
     diff_lambda: float = 0.0                 # weight of the second map's output
+    talk: Optional[torch.Tensor] = None      # fp32 [heads, heads]: share of head g's softmax weights in head h's
     # mamba (also conv, dt_bias)
     w_x: Optional[torch.Tensor] = None       # [dt | B | C rows, inner_pad], blocks at off_b / off_c
     off_b: int = 0
@@ -75,7 +82,8 @@ class MixerImage:
     w_dt: Optional[torch.Tensor] = None      # [inner_pad, dt_rank padded to 8]
     conv_b: Optional[torch.Tensor] = None    # fp32 [inner_pad]
     a_log2: Optional[torch.Tensor] = None    # fp32 [state, inner_pad] = -exp(A_log) * log2(e)
-    d_skip: Optional[torch.Tensor] = None    # fp32 [inner_pad]
+    d_skip: Optional[torch.Tensor] = None    # fp32 [inner_pad] (mamba2: [heads])
+    # mamba2: conv [taps, channels], conv_b [channels], dt_bias, a_neg [heads], o_norm [inner_pad]
 
 
 @dataclass
@@ -98,6 +106,14 @@ class LayerImage:
     norm2b: Optional[torch.Tensor] = None    # fp32 [width_pad]
     w_up: Optional[torch.Tensor] = None      # [ff_pad, width_pad]; gated: [gate ff_pad | up ff_pad, width_pad]
     w_down: Optional[torch.Tensor] = None    # [width_pad, ff_pad]
+    up_b: Optional[torch.Tensor] = None      # fp32 [ff_pad]
+    down_b: Optional[torch.Tensor] = None    # fp32 [width_pad]
+    # pre-norm block: norm1, norm2 [width_pad]; share of the previous token in the mixer's input
+    shift: Optional[torch.Tensor] = None     # fp32 [width_pad]
+    # experts, also: router_w has one row more with a shared expert (its gate)
+    router_b: Optional[torch.Tensor] = None  # fp32 [experts]
+    s_w13: Optional[torch.Tensor] = None     # shared expert [2 * ff_pad, width_pad]
+    s_w2: Optional[torch.Tensor] = None      # [width_pad, ff_pad]
 
 
 @dataclass
@@ -105,7 +121,7 @@ class LayeredWeights:
     cfg: LayeredConfig
     embed: torch.Tensor                      # [vocab, width_pad]
     layers: List[LayerImage]
-    final_norm: torch.Tensor                 # fp32 [1], output-norm blocks: [2, width_pad], sandwich blocks: [width_pad]
+    final_norm: torch.Tensor                 # fp32 [1], output-norm blocks: [2, width_pad], sandwich and pre-norm blocks: [width_pad]
     lm_head: torch.Tensor                    # [vocab, width_pad]
     pos: Optional[torch.Tensor] = None       # [max_position, width_pad] learned position vectors
     mtp: list = field(default_factory=list)  # the architecture has no proposal stages
@@ -114,7 +130,7 @@ class LayeredWeights:
     def nbytes(self) -> int:
         total = sum(t.numel() * t.element_size() for t in (self.embed, self.final_norm, self.lm_head)
                     + (() if self.pos is None else (self.pos,)))
-        for l in self.layers:
+        for l in {id(l): l for l in self.layers}.values():       # (layers may share an image)
             for holder in (l, l.mixer):
                 total += sum(t.numel() * t.element_size() for t in vars(holder).values() if isinstance(t, torch.Tensor))
         return total
@@ -124,31 +140,50 @@ class _Blocks:
     """Stacks row blocks, each starting at a multiple of 8."""
 
     def __init__(self, cols: int):
-        self.cols, self.rows, self.off, self.parts = cols, 0, {}, []
+        self.cols, self.rows, self.off, self.parts, self.biases = cols, 0, {}, [], {}
 
-    def add(self, name: str, w: torch.Tensor) -> None:
+    def add(self, name: str, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> None:
         n = pad_to(w.shape[0], 8)
         self.off[name] = self.rows
         self.parts.append(_pad(w, n, self.cols))
+        if bias is not None:
+            self.biases[self.rows] = bias
         self.rows += n
 
     def matrix(self) -> torch.Tensor:
         return torch.cat(self.parts, 0).contiguous()
 
+    def bias(self) -> Optional[torch.Tensor]:
+        if not self.biases:
+            return None
+        out = torch.zeros(self.rows, dtype=torch.float32, device=self.parts[0].device)
+        for at, b in self.biases.items():
+            out[at:at + b.shape[0]] = b.float()
+        return out
+
 
 def _pack_latent(m: LatentMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
-    Wp, DL = cfg.width_pad, cfg.kv_row_dim
+    Wp, DL = cfg.width_pad, m.row_dim
     dp, vp = pad_to(m.dim, 8), pad_to(m.vdim, 8)
-    q = _pad(get(p + "q").view(m.heads, m.dim, cfg.width), m.heads, dp, Wp)
-    b.add("q", q.reshape(m.heads * dp, Wp))
+    w_q = get(p + ("uq" if m.q_rank else "q")).view(m.heads, m.dim + m.rot_dim, -1)
+    src = _Blocks(pad_to(m.q_rank, 8)) if m.q_rank else b
+    src.add("q", _pad(w_q[:, :m.dim], m.heads, dp, src.cols).reshape(m.heads * dp, src.cols))
+    if m.rot_dim:
+        src.add("qr", _pad(w_q[:, m.dim:], m.heads, m.rot_dim, src.cols).reshape(m.heads * m.rot_dim, src.cols))
+    if m.q_rank:
+        b.add("dq", get(p + "dq"))
     b.add("dkv", get(p + "dkv"))
     b.add("g", get(p + "g"))
     uk = get(p + "uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2)
     uv = get(p + "uv").view(m.heads, m.vdim, m.kv_rank)
     o = _pad(get(p + "o").view(cfg.width, m.heads, m.vdim), Wp, m.heads, vp)
-    return MixerImage(None, b.off, o.reshape(Wp, m.heads * vp).contiguous(),
-                      w_uk_t=_pad(uk, m.heads, DL, dp).contiguous(), w_uv=_pad(uv, m.heads, vp, DL).contiguous(),
-                      kv_norm=_pad(get(p + "dkv.norm").float(), DL).contiguous())
+    img = MixerImage(None, b.off, o.reshape(Wp, m.heads * vp).contiguous(),
+                     w_uk_t=_pad(uk, m.heads, DL, dp).contiguous(), w_uv=_pad(uv, m.heads, vp, DL).contiguous(),
+                     kv_norm=_pad(get(p + "dkv.norm").float(), DL).contiguous())
+    if m.q_rank:
+        img.w_uq, img.off_uq = src.matrix(), src.off
+        img.dq_norm = _pad(get(p + "dq.norm").float(), src.cols).contiguous()
+    return img
 
 
 def _pack_attention(m: AttentionMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
@@ -169,15 +204,20 @@ def _pack_window(m: WindowMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: 
         blocks.append(("v", m.kv_heads, m.vdim, vp))
     if m.gate:
         blocks.append(("g", m.heads, m.vdim, vp))
+    bias = lambda name, heads, d, pad: _pad(get(p + name + ".b").float().view(heads, d), heads, pad).reshape(-1).contiguous()
+    in_gemm = "v" in m.biases          # the projection adds them all
     for name, heads, d, pad in blocks:
-        b.add(name, _pad(get(p + name).view(heads, d, cfg.width), heads, pad, Wp).reshape(heads * pad, Wp))
+        b.add(name, _pad(get(p + name).view(heads, d, cfg.width), heads, pad, Wp).reshape(heads * pad, Wp),
+              bias(name, heads, d, pad) if in_gemm and name in m.biases else None)
     o = _pad(get(p + "o").view(cfg.width, m.heads, m.vdim), Wp, m.heads, vp)
-    bias = lambda name, heads: _pad(get(p + name).float().view(heads, m.dim), heads, dp).reshape(-1).contiguous()
-    norm = lambda name: _pad(get(p + name).float(), dp).contiguous()
+    norm = lambda name: _pad(get(p + name).float(), dp).contiguous() if m.norm_weights else None
     f64 = lambda name: get(p + name).double()
     img = MixerImage(None, b.off, o.reshape(Wp, m.heads * vp).contiguous(), q_norm=norm("q.norm"), k_norm=norm("k.norm"))
-    if m.biases:
-        img.q_bias, img.k_bias = bias("q.b", nq), bias("k.b", nk)
+    if not in_gemm and "q" in m.biases:
+        img.q_bias, img.k_bias = bias("q", nq, m.dim, dp), bias("k", nk, m.dim, dp)
+    if m.mix_weights:
+        img.talk = get(p + "talk").float().contiguous()
+    if "o" in m.biases:
         img.o_bias = _pad(get(p + "o.b").float(), Wp).contiguous()
     # score_h = sum_g T[h, g] (scale temp_g q_g . k - slope_g distance): everything but q and k is constant
     scale = torch.full((m.heads,), m.scale, dtype=torch.float64, device=o.device)
@@ -211,6 +251,23 @@ def _pack_mamba(m: MambaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _B
                       dt_bias=vec("dt.b"), d_skip=vec("D"), a_log2=_pad(a.float().t(), m.state, Ip).contiguous())
 
 
+def _pack_mamba2(m: Mamba2Mixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
+    bc = m.groups * m.state
+    z, x, B, C, dt = get(p + "in").split([m.inner, m.inner, bc, bc, m.heads])
+    for name, w in (("x", x), ("B", B), ("C", C), ("z", z), ("dt", dt)):
+        b.add(name, w)
+    assert b.off["z"] == m.channels
+
+    def channels(t):        # x | B | C, padded as the projection's blocks
+        return torch.cat([_pad(c, pad_to(c.shape[0], 8), *c.shape[1:]) for c in t.float().split([m.inner, bc, bc])])
+
+    vec = lambda name: get(p + name).float().contiguous()
+    return MixerImage(None, b.off, _pad(get(p + "o"), cfg.width_pad, m.inner_pad).contiguous(), off_b=b.off["B"],
+                      off_c=b.off["C"], conv=channels(get(p + "conv").view(-1, m.taps)).t().contiguous(),
+                      conv_b=channels(get(p + "conv.b")).contiguous(), dt_bias=vec("dt_bias"), d_skip=vec("D"),
+                      a_neg=-torch.exp(get(p + "A_log").double()).float(), o_norm=_pad(vec("norm"), m.inner_pad).contiguous())
+
+
 def _pack_delta(m: DeltaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _Blocks) -> MixerImage:
     Wp = cfg.width_pad
     nk, nv, nd = m.kv_heads * m.dim, m.heads * m.vdim, m.heads * m.dim
@@ -231,7 +288,7 @@ def _pack_delta(m: DeltaMixer, p: str, get: GetTensor, cfg: LayeredConfig, b: _B
 
 
 _PACK = {LatentMixer: _pack_latent, AttentionMixer: _pack_attention, WindowMixer: _pack_window, DeltaMixer: _pack_delta,
-         MambaMixer: _pack_mamba}
+         MambaMixer: _pack_mamba, Mamba2Mixer: _pack_mamba2}
 
 
 def _pack_dense(s: DenseSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: LayerImage) -> None:
@@ -239,11 +296,20 @@ def _pack_dense(s: DenseSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: L
     up = _pad(get(p + "up"), fp, Wp)
     img.w_up = (torch.cat([_pad(get(p + "gate"), fp, Wp), up]) if s.gated else up).contiguous()
     img.w_down = _pad(get(p + "down"), Wp, fp).contiguous()
+    if s.biases:
+        img.up_b, img.down_b = _pad(get(p + "up.b").float(), fp).contiguous(), _pad(get(p + "down.b").float(), Wp).contiguous()
 
 
 def _pack_moe(s: MoeSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: LayerImage) -> None:
     Wp, fp = cfg.width_pad, pad_to(s.ff, 8)
-    img.router_w = _pad(get(p + "router"), s.experts, Wp).contiguous()
+    router = [get(p + "router")] + ([get(p + "shared.sg")] if s.shared_ff else [])
+    img.router_w = _pad(torch.cat(router), s.experts + len(router) - 1, Wp).contiguous()
+    if s.router_bias:
+        img.router_b = get(p + "router.b").float().contiguous()
+    if s.shared_ff:
+        sp, q = pad_to(s.shared_ff, 8), p + "shared."
+        img.s_w13 = torch.cat([_pad(get(q + "gate"), sp, Wp), _pad(get(q + "up"), sp, Wp)]).contiguous()
+        img.s_w2 = _pad(get(q + "down"), Wp, sp).contiguous()
     like = img.router_w
     img.e_w13 = torch.zeros(s.experts, 2 * fp, Wp, dtype=like.dtype, device=like.device)
     img.e_w2 = torch.zeros(s.experts, Wp, fp, dtype=like.dtype, device=like.device)
@@ -257,15 +323,19 @@ def _pack_moe(s: MoeSpec, p: str, get: GetTensor, cfg: LayeredConfig, img: Layer
 def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
     """`get(name)` returns a checkpoint tensor in the dtype and on the device the model runs with."""
     Wp = cfg.width_pad
-    gated, sandwich = cfg.block == PARALLEL_GATED, cfg.block == SANDWICH_NORM
+    gated, sandwich, pre = (cfg.block == k for k in (PARALLEL_GATED, SANDWICH_NORM, PRE_NORM))
     vec = lambda name: _pad(get(name).float(), Wp).contiguous()
-    norm = lambda name: vec(name) if sandwich else torch.stack([vec(n) for n in (name, name + ".b")]).contiguous()
+    norm = lambda name: vec(name) if sandwich or pre else torch.stack([vec(n) for n in (name, name + ".b")]).contiguous()
     layers: List[LayerImage] = []
+    owners: Dict[int, LayerImage] = {}
     for i, spec in enumerate(cfg.layers):
-        p = f"l{i}."
+        if cfg.owner(i) in owners:
+            layers.append(owners[cfg.owner(i)])
+            continue
+        p = f"l{cfg.owner(i)}."
         b = _Blocks(Wp)
         mx = _PACK[type(spec.mixer)](spec.mixer, p + "mix.", get, cfg, b)
-        img = LayerImage(spec, mx)
+        img = owners[cfg.owner(i)] = LayerImage(spec, mx)
         if gated:
             img.norm = get(p + "norm1").float().reshape(1).contiguous()
             img.rg1_b = _pad(get(p + "rg1.b").float(), Wp).contiguous()
@@ -274,6 +344,8 @@ def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
             img.norm1 = norm(p + "norm1")
         if sandwich:
             img.norm1b = norm(p + "norm1b")
+        if cfg.token_shift:
+            img.shift = vec(p + "shift")
         if cfg.canon_taps:
             img.canon = _pad(get(p + "canon1").float().view(cfg.width, cfg.canon_taps).t(), cfg.canon_taps, Wp).contiguous()
         if spec.mlp is not None:
@@ -285,7 +357,7 @@ def pack_weights(cfg: LayeredConfig, get: GetTensor) -> LayeredWeights:
             if sandwich:
                 img.norm2b = norm(p + "norm2b")
             (_pack_moe if isinstance(spec.mlp, MoeSpec) else _pack_dense)(spec.mlp, p + "mlp.", get, cfg, img)
-        mx.w_in = b.matrix()
+        mx.w_in, mx.b_in = b.matrix(), b.bias()
         layers.append(img)
     final = get("final.norm").float().reshape(1).contiguous() if gated else norm("final.norm")
     pos = _pad(get("pos"), cfg.max_position, Wp).contiguous() if cfg.learned_positions else None
@@ -329,12 +401,15 @@ class RandomTensors:
             t[..., -1] += 0.7
         elif name.endswith("canon1"):
             t = normal(0.0, 0.3)
-        elif name.endswith(("norm1.b", "norm2.b", "final.norm.b", ".conv.b", ".q.b", ".k.b", ".o.b")):
+        elif name.endswith(("norm1.b", "norm2.b", "final.norm.b", ".conv.b", ".q.b", ".k.b", ".v.b", ".o.b", ".up.b", ".down.b",
+                            ".router.b")):
             t = normal(0.0, 0.2)
         elif name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
             t = normal(0.0, 0.1)
         elif name.endswith(".talk"):
             t = normal(0.0, 0.3) + torch.eye(shape[0], device=self.device)
+        elif name.endswith(".shift"):
+            t = normal(0.4, 0.3)
         elif name.endswith(".temp"):
             t = normal(1.0, 0.3)
         elif name.endswith((".vmix", ".D")):

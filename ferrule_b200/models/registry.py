@@ -75,6 +75,8 @@ ARCHITECTURES: Dict[str, Architecture] = {a.name: a for a in (
                  (torch.bfloat16, torch.float32), "layered"),
     Architecture("vedadra", lambda c: c.get("architecture") == "Vedadra", _load_layered, _run_layered,
                  (torch.bfloat16, torch.float32), "layered"),
+    Architecture("vogunex", lambda c: c.get("architecture") == "Vogunex", _load_layered, _run_layered,
+                 (torch.bfloat16, torch.float32), "layered"),
     Architecture("deepseek_v4", lambda c: c.get("model_type") == "deepseek_v4", _load_v4, _run_v4),
     # every other HuggingFace-style config.json is read as a DeepSeek-V2 / V3 model, whose loader checks it
     Architecture("deepseek", lambda c: "architecture" not in c, _load_deepseek, _run_deepseek),

@@ -36,7 +36,7 @@ class BatchStaging:
     Layout (int32 words): write_slot (int64, 2R) | token_ids R | positions R | row_seq R | row_pos R |
     logit_rows R | block_table S*MB | prefill attention tiles 4*TC (only with tc_heads).
 
-    tc_heads > 0: sequences that bring at least `tc_min_rows` query rows are cut into the 128-row tiles of the
+    tc_heads > 0 (or several such numbers: a tile table for each, with the same rows left over): sequences that bring at least `tc_min_rows` query rows are cut into the 128-row tiles of the
     tensor-core prefill attention kernel (128 / tc_heads positions x all heads); the other rows - decode rows,
     verification rows, short chunk tails - stay with the row-tile kernel, whose split boundaries make a
     verification row bit-equal to the decode row of the same position.
@@ -46,12 +46,16 @@ class BatchStaging:
     two from its state pool (`fill_states`).
     """
 
-    def __init__(self, rows: int, seqs: int, max_blocks: int, device, tc_heads: int = 0, tc_min_rows: int = 16,
+    def __init__(self, rows: int, seqs: int, max_blocks: int, device, tc_heads=0, tc_min_rows: int = 16,
                  state_slots: bool = False):
         self.rows, self.seqs, self.max_blocks = rows, seqs, max_blocks
         R = rows
-        self.tc_heads, self.tc_min_rows = tc_heads, tc_min_rows
-        self.tile_cap = (R // (128 // tc_heads) + seqs + 1) if tc_heads else 0
+        self.tc_forms = tuple(h for h in ((tc_heads,) if isinstance(tc_heads, int) else tc_heads) if h)
+        self.tc_heads, self.tc_min_rows = max(self.tc_forms, default=0), tc_min_rows
+        caps = [R // (128 // h) + seqs + 1 for h in self.tc_forms]
+        self.tile_cap = sum(caps)
+        self.tile_first = [sum(caps[:i]) for i in range(len(caps))]       # of every table
+        self.n_form_tiles = [0] * len(caps)
         self.tile_off = (7 * R + seqs * max_blocks + 3) // 4 * 4          # 16-byte aligned
         self.state_slots = state_slots
         self.state_off = self.tile_off + 4 * self.tile_cap
@@ -125,11 +129,16 @@ class BatchStaging:
         self.n_tiles, self.rest_ranges = 0, None
         if self.tc_heads and n != T and any(s.query_len >= self.tc_min_rows for s in seqs):
             from ..ops.kernels import prefill_tiles
-            tiles, rest = prefill_tiles([(i, s.query_start, s.query_len, int(b.positions[s.query_start]))
-                                         for i, s in enumerate(seqs)], self.tc_heads, self.tc_min_rows)
-            if len(tiles) <= self.tile_cap:
-                self.np_tiles[:len(tiles)] = tiles
-                self.n_tiles, self.rest_ranges = len(tiles), rest
+            segments = [(i, s.query_start, s.query_len, int(b.positions[s.query_start])) for i, s in enumerate(seqs)]
+            for f, heads in enumerate(self.tc_forms):
+                tiles, rest = prefill_tiles(segments, heads, self.tc_min_rows)
+                at, end = self.tile_first[f], (self.tile_first + [self.tile_cap])[f + 1]
+                if len(tiles) > end - at:
+                    self.n_tiles, self.rest_ranges = 0, None
+                    break
+                self.np_tiles[at:at + len(tiles)] = tiles
+                self.n_form_tiles[f] = len(tiles)
+                self.n_tiles, self.rest_ranges = self.n_tiles + len(tiles), rest
         return T, R, lrows
 
     def fill_states(self, bindings) -> None:
@@ -150,8 +159,9 @@ class BatchStaging:
         db = DeviceBatch(self.d_ids[:R], self.d_pos[:R], self.d_slot[:R], self.d_seq[:R], self.d_rpos[:R],
                          self.d_bt, self.d_lrows, R, n_logit)
         if self.n_tiles:
-            db.tc_tiles, db.n_tc_tiles, db.rest_ranges = self.d_tiles, self.n_tiles, self.rest_ranges
-            db.tc_positions = 128 // self.tc_heads
+            db.tc_tables = {h: (self.d_tiles[at:], n) for h, at, n in zip(self.tc_forms, self.tile_first, self.n_form_tiles)}
+            db.tc_tiles, db.n_tc_tiles = db.tc_tables[self.tc_heads]
+            db.rest_ranges, db.tc_positions = self.rest_ranges, 128 // self.tc_heads
         if self.state_slots:
             db.seq_start, db.state_in, db.state_out, db.n_seqs = self.d_start, self.d_state_in, self.d_state_out, self.n_seqs
             db.long_seqs = self.long_seqs
@@ -752,7 +762,7 @@ class DeepSeekRunner(ModelRunner):
         d = dict(vars(self.stats))
         d["graphs"] = sorted(self.graphs)
         d["weights_bytes"] = self.w.nbytes()
-        d["kv_pool_bytes"] = self.pool.data.numel() * self.pool.data.element_size()
+        d["kv_pool_bytes"] = self.pool.bytes_per_page * self.pool.n_pages
         if self.arena is not None:
             d["expert_arena"] = dict(vars(self.arena.stats))
             d["expert_telemetry"] = self.telemetry.snapshot()

@@ -1,14 +1,18 @@
 """Recurrent-state pool: what a sequence carries from token to token beside its paged cache.
 
-Three kinds of plane: per run of a recurrent layer the fp32 state (a matrix per head of a delta mixer, [inner, state] of a selective
+Kinds of plane: per run of a recurrent layer the fp32 state (a matrix per head of a delta mixer, [inner, state] of a selective
 scan) and the last inputs of the short convolutions, and per run of a layer with an input convolution the last rows of the
-32-bit residual stream it read.  A plane is indexed by slot (the engine's logical sequence slot) and buffer: every slot has `buffers`
+32-bit residual stream it read, or of a token shift the last normalised row.  Such a plane is indexed by slot (the engine's logical sequence slot) and buffer: every slot has `buffers`
 copies and one of them is committed.  A step reads the committed copy and writes the next one, and only the commit of its
 transaction makes that one current - a step that fails or is rolled back leaves nothing to undo.  With decode
 look-ahead a step may already run before its predecessor has been published, so three buffers are in rotation: the
 committed one, the one the unpublished step wrote, the one the step launched ahead writes.
 
 A sequence starts from zeros: its first step reads index -1 and no memory has to be cleared.
+
+Layers that see mean keys and values of whole blocks of tokens keep them here too: `pooled[run]` holds per slot one cache row for
+every block a sequence can have, in order.  A row is written by the step that appends its block's last token, and again
+whenever that token is appended again; a query only sees blocks whose last token is older.  So there is one buffer.
 """
 from __future__ import annotations
 
@@ -16,11 +20,12 @@ from typing import Dict, List, Tuple
 
 import torch
 
-from .layered_config import DeltaMixer, LayeredConfig, MambaMixer
+from .layered_config import DeltaMixer, LayeredConfig, Mamba2Mixer, MambaMixer
 
 
 class RecurrentStatePool:
-    def __init__(self, cfg: LayeredConfig, n_slots: int, device, dtype=torch.bfloat16, buffers: int = 3):
+    def __init__(self, cfg: LayeredConfig, n_slots: int, device, dtype=torch.bfloat16, buffers: int = 3,
+                 max_tokens: int = 0):
         if buffers < 2:
             raise ValueError("a slot needs at least two buffers")
         self.n_slots, self.buffers = n_slots, buffers
@@ -28,6 +33,8 @@ class RecurrentStatePool:
         self.state: Dict[int, torch.Tensor] = {}
         self.tail: Dict[int, torch.Tensor] = {}
         self.canon: Dict[int, torch.Tensor] = {}
+        self.shift: Dict[int, torch.Tensor] = {}
+        self.pooled: Dict[int, torch.Tensor] = {}
         plane = lambda *shape, dt=torch.float32: torch.zeros(self.n_states, *shape, dtype=dt, device=device)
         for i, layer in enumerate(cfg.runs):
             m = cfg.layers[layer].mixer
@@ -37,13 +44,21 @@ class RecurrentStatePool:
             elif isinstance(m, MambaMixer):
                 self.state[i] = plane(m.state, m.inner_pad)
                 self.tail[i] = plane(max(m.taps - 1, 1), m.inner_pad, dt=dtype)
+            elif isinstance(m, Mamba2Mixer):
+                self.state[i] = plane(m.heads, m.state, m.vdim)
+                self.tail[i] = plane(max(m.taps - 1, 1), m.channels, dt=dtype)
+            elif getattr(m, "pool", 0):
+                self.pooled[i] = torch.zeros(n_slots, max_tokens // m.pool + 1, cfg.plane_dim(layer), dtype=dtype, device=device)
+            if cfg.token_shift:
+                self.shift[i] = plane(cfg.width_pad)
             if cfg.canon_taps:
                 self.canon[i] = plane(max(cfg.canon_taps - 1, 1), cfg.width_pad)
         self.current: List[int] = [-1] * n_slots         # committed buffer of every slot, -1: none yet
 
     @property
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.state, self.tail, self.canon) for t in d.values())
+        return sum(t.numel() * t.element_size() for d in (self.state, self.tail, self.canon, self.shift, self.pooled)
+                   for t in d.values())
 
     def bind(self, slot: int, fresh: bool, ahead: bool = False) -> Tuple[int, int]:
         """(state index to read, state index to write) of the slot's next step.  `fresh`: the sequence starts with

@@ -18,7 +18,7 @@ from enum import Enum
 from typing import List, Optional, Tuple
 
 from .config import SCORE_SIGMOID, SCORE_SOFTMAX, ModelConfig
-from .layered_config import OUTPUT_NORM, PARALLEL_GATED, SANDWICH_NORM, LayeredConfig, MoeSpec
+from .layered_config import OUTPUT_NORM, PARALLEL_GATED, PRE_NORM, SANDWICH_NORM, LayeredConfig, MoeSpec
 
 
 class AttentionKind(Enum):
@@ -26,6 +26,7 @@ class AttentionKind(Enum):
     HYBRID_SPARSE_MLA = "hybrid_mla"  # single latent head + window + compressed selection (DeepSeek-V4)
     LATENT_DELTA = "latent_delta"     # per layer: latent attention without positions, or gated delta rule (Gitozen)
     WINDOW_MIXED = "window_mixed"     # per layer: window attention with scores mixed across heads, or differential
+    POOLED_WINDOW = "pooled_window"   # per layer: window attention with pooled blocks, latent attention, or head-decay scan
     CHUNKED_RECURRENT = "chunked_recurrent"   # per layer: chunked grouped-query attention, selective scan or delta rule
 
 
@@ -130,7 +131,7 @@ class PolicySet:
     speculation: SpeculationPolicy
     tokenizer: TokenizerPolicy
     validation: ValidationPolicy
-    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4" | "gitozen" | "supisun" | "vedadra"
+    semantics: str                    # "deepseek-v2" | "deepseek-v3" | "deepseek-v4" | "gitozen" | "supisun" | "vedadra" | "vogunex"
 
     @staticmethod
     def from_config(cfg, weight_format: str = "bf16", parallelism: Optional[ParallelismPlan] = None,
@@ -141,14 +142,17 @@ class PolicySet:
             moes = [l.mlp for l in cfg.layers if isinstance(l.mlp, MoeSpec)]
             kind, sem = {PARALLEL_GATED: (AttentionKind.LATENT_DELTA, "gitozen"),
                          OUTPUT_NORM: (AttentionKind.CHUNKED_RECURRENT, "supisun"),
-                         SANDWICH_NORM: (AttentionKind.WINDOW_MIXED, "vedadra")}[cfg.block]
+                         SANDWICH_NORM: (AttentionKind.WINDOW_MIXED, "vedadra"),
+                         PRE_NORM: (AttentionKind.POOLED_WINDOW, "vogunex")}[cfg.block]
             groups = max(((m.groups, m.keep) for m in moes), default=(1, 1))
             att = AttentionPolicy(kind, cfg.kv_row_dim, cfg.n_heads, False)
             router = RouterPolicy(RouterKind.NONE if not moes else (RouterKind.SOFTMAX_GROUP_TOPK if groups[0] > 1
                                                                     else RouterKind.SOFTMAX_TOPK), cfg.topk, groups)
-            expert = ExpertPolicy(cfg.n_routed_experts, 0, cfg.n_layers - len(moes))
+            expert = ExpertPolicy(cfg.n_routed_experts, int(any(m.shared_ff for m in moes)), cfg.n_layers - len(moes))
             planes = ((("latent_kv",) if cfg.latent_layers else ()) + (("kv",) if cfg.attention_layers or cfg.window_layers else ())
-                      + (("recurrent_state",) if cfg.delta_layers or cfg.mamba_layers else ())
+                      + (("recurrent_state",) if cfg.delta_layers or cfg.mamba_layers or cfg.mamba2_layers else ())
+                      + (("pooled_kv",) if any(cfg.layers[i].mixer.pool for i in cfg.window_layers) else ())
+                      + (("token_shift",) if cfg.token_shift else ())
                       + (("input_convolution",) if cfg.canon_taps else ()))
             spec = SpeculationPolicy(SpeculationMode.NONE, 0)
         elif not isinstance(cfg, ModelConfig):         # models.v4_model.V4Config
@@ -232,7 +236,7 @@ class EnginePlan:
                                              "dequantised at load time)"))
             if par.tensor_parallel > 1 or par.pipeline_parallel > 1:
                 missing.append(MissingPolicy("parallelism", "the V4 runner is single-GPU"))
-        if p.semantics in ("gitozen", "supisun", "vedadra"):
+        if p.semantics in ("gitozen", "supisun", "vedadra", "vogunex"):
             if p.quant.weight_format != "bf16":
                 missing.append(MissingPolicy("quantization", "layer-list models run bf16 (or fp32) weights"))
             if par.tensor_parallel > 1 or par.pipeline_parallel > 1 or par.expert_parallel > 1:

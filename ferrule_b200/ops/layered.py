@@ -373,6 +373,13 @@ def gqa_tc_group(mixer, dtype, page_size: int) -> int:
     return per if ok else 0
 
 
+def latent_tc_group(mixer, dtype, page_size: int) -> int:
+    """Query rows per position when the bf16 prompt kernel serves the latent mixer, else 0."""
+    from .kernels import prefill_tc_supported
+    ok = dtype == torch.bfloat16 and prefill_tc_supported(mixer.heads, mixer.value_dim, mixer.row_dim - mixer.value_dim, page_size)
+    return mixer.heads if ok else 0
+
+
 @functools.lru_cache(maxsize=None)
 def gqa_decode_supported(mixer, dtype, page_size: int) -> bool:
     """Whether the bf16 kernels for few rows serve the mixer."""
