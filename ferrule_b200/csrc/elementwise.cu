@@ -212,7 +212,7 @@ __device__ __forceinline__ void route_one_token(const float* lr, int warp, int l
                                                 const int* __restrict__ token_ids, int experts, int topk,
                                                 int score_fn, int n_groups, int topk_groups, int normalize,
                                                 float route_scale, int* __restrict__ out_idx,
-                                                float* __restrict__ out_w) {
+                                                float* __restrict__ out_w, const float* __restrict__ logit_bias = nullptr) {
   constexpr int kPer = 8;
   float score[kPer];   // the value weights are taken from
   float select[kPer];  // the value top-k is taken on (score + bias)
@@ -221,7 +221,7 @@ __device__ __forceinline__ void route_one_token(const float* lr, int warp, int l
 #pragma unroll
   for (int j = 0; j < kPer; ++j) {
     const int e = lane + 32 * j;
-    score[j] = e < experts ? lr[e] : -INFINITY;
+    score[j] = e < experts ? lr[e] + (logit_bias ? logit_bias[e] : 0.f) : -INFINITY;
     mx = fmaxf(mx, score[j]);
   }
   if (score_fn == kScoreSoftmax) {
@@ -353,14 +353,14 @@ router_topk_kernel(const float* __restrict__ logits, long long ldl, const float*
                    const long long* __restrict__ hash_table, const int* __restrict__ token_ids,
                    int rows, int experts, int topk, int score_fn, int n_groups, int topk_groups,
                    int normalize, float route_scale, int* __restrict__ out_idx,
-                   float* __restrict__ out_w) {
+                   float* __restrict__ out_w, const float* __restrict__ logit_bias) {
   pdl_launch_dependents();
   pdl_wait();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
   if (warp >= rows) return;
   route_one_token(logits + warp * ldl, warp, lane, bias, hash_table, token_ids, experts, topk, score_fn,
-                  n_groups, topk_groups, normalize, route_scale, out_idx, out_w);
+                  n_groups, topk_groups, normalize, route_scale, out_idx, out_w, logit_bias);
 }
 
 // ---------------------------------------------------------------------------------
@@ -752,6 +752,14 @@ struct QuantRows {
   int s_cols;
 };
 
+// Optional: a bias on the logits, and products of the row with further rows of `w` behind the experts' (the gate of a shared
+// expert), written as they are.
+struct RouterExtra {
+  const float* logit_bias;  // [experts]
+  float* extra;             // [rows, n_extra]
+  int n_extra;
+};
+
 __global__ void __launch_bounds__(1024)
 router_append_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const __nv_bfloat16* __restrict__ w,
                      int hidden, const float* __restrict__ bias, const long long* __restrict__ hash_table,
@@ -760,10 +768,11 @@ router_append_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const _
                      float* __restrict__ out_w, int e_lo, int e_hi, int slot_rows, int dst_slots,
                      int* __restrict__ cnt, int* __restrict__ src_token, int* __restrict__ dst_row,
                      float* __restrict__ row_scale, __nv_bfloat16* __restrict__ xg, long long ldxg, DeviceStatus* st,
-                     NormPrologue np, QuantRows qr) {
+                     NormPrologue np, QuantRows qr, RouterExtra ex) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float xs[];            // hidden floats, then `experts` logits, then (norm prologue) hidden bf16
+  extern __shared__ float xs[];            // hidden floats, then logits, then (norm prologue) hidden bf16
+  const int products = experts + ex.n_extra;
   float* logits = xs + hidden;
   __shared__ int rlist[32];
   __shared__ float red[8];
@@ -775,7 +784,7 @@ router_append_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const _
     // ---- residual add + RMSNorm of this token's row, with the element -> thread mapping, the rounding points and
     // the reduction order of add_rmsnorm_kernel (256 threads x 8 elements, 8 warp sums combined by one warp), so
     // the result is bit-equal to running that kernel first.  x = residual stream, np.delta = the sublayer output. ----
-    __nv_bfloat16* xb = reinterpret_cast<__nv_bfloat16*>(logits + experts);
+    __nv_bfloat16* xb = reinterpret_cast<__nv_bfloat16*>(logits + products);
     const __nv_bfloat16* dr = np.delta ? np.delta + t * np.ldd : nullptr;
     float ss = 0.f;
     if (threadIdx.x < 256) {
@@ -834,9 +843,9 @@ router_append_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const _
     }
   }
   __syncthreads();
-  for (int e = warp; e < experts; e += 2 * nwarps) {
+  for (int e = warp; e < products; e += 2 * nwarps) {
     const int e2 = e + nwarps;
-    const bool two = e2 < experts;
+    const bool two = e2 < products;
     const __nv_bfloat16* wr = w + static_cast<size_t>(e) * hidden;
     const __nv_bfloat16* wr2 = w + static_cast<size_t>(two ? e2 : e) * hidden;
     float acc = 0.f, acc2 = 0.f;
@@ -862,7 +871,8 @@ router_append_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, const _
   __syncthreads();
   if (warp == 0) {
     route_one_token(logits, t, lane, bias, hash_table, token_ids, experts, topk, score_fn, n_groups,
-                    topk_groups, normalize, route_scale, out_idx, out_w);
+                    topk_groups, normalize, route_scale, out_idx, out_w, ex.logit_bias);
+    if (lane < ex.n_extra) ex.extra[static_cast<long long>(t) * ex.n_extra + lane] = logits[experts + lane];
     __syncwarp();
     if (lane < topk) {
       const int e = out_idx[t * topk + lane];
@@ -1309,14 +1319,14 @@ extern "C" int fb_router_topk(const float* logits, long long ldl, const float* b
                               const long long* hash_table, const int* token_ids, int rows,
                               int experts, int topk, int score_fn, int n_groups, int topk_groups,
                               int normalize, float route_scale, int* out_idx, float* out_w,
-                              void* stream) {
+                              const float* logit_bias, void* stream) {
   if (rows <= 0 || experts <= 0 || experts > 256 || topk <= 0 || topk > 32 || topk > experts)
     return FB_ERR_SHAPE;
   if (n_groups > 32 || (n_groups > 1 && experts % n_groups != 0)) return FB_ERR_SHAPE;
   const int blocks = (rows + 3) / 4;
   launch_pdl(router_topk_kernel, dim3(blocks), dim3(128), 0, static_cast<cudaStream_t>(stream), 
       logits, ldl, bias, hash_table, token_ids, rows, experts, topk, score_fn, n_groups,
-      topk_groups, normalize, route_scale, out_idx, out_w);
+      topk_groups, normalize, route_scale, out_idx, out_w, logit_bias);
   return FB_CHECK_LAUNCH();
 }
 
@@ -1395,7 +1405,7 @@ extern "C" int fb_norm_router_append(const void* x, long long ldx, const void* d
                             nullptr, 0, nullptr, 0, nullptr, 0, nullptr, 0, 0, status, stream);
 }
 
-extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delta, long long ldd,
+static int run_router_append(const void* x, long long ldx, const void* delta, long long ldd,
                                   const void* norm_w, void* res_out, long long ldr, void* norm_out, long long ldn,
                                   float eps, const void* w, int hidden, const float* bias,
                                   const long long* hash_table, const int* token_ids, int rows, int experts,
@@ -1404,9 +1414,11 @@ extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delt
                                   int slot_rows, int dst_slots, int* cnt, int* src_token, int* dst_row,
                                   float* row_scale, void* xg, long long ldxg, const void* q_src, long long ldq,
                                   const void* s_src, long long lds, void* xg_q, long long ldxgq, void* xg_s,
-                                  long long ldxgs, int s_cols, void* status, void* stream) {
+                                  long long ldxgs, int s_cols, const RouterExtra& ex, void* status,
+                             void* stream) {
   if (rows <= 0 || experts <= 0 || experts > 256 || topk <= 0 || topk > 32 || topk > experts) return FB_ERR_SHAPE;
   if (hidden % 8 != 0 || hidden > 8192 || (ldx % 8) != 0 || (ldxg % 8) != 0) return FB_ERR_SHAPE;
+  if (ex.n_extra < 0 || ex.n_extra > 32 || (ex.n_extra > 0 && !ex.extra)) return FB_ERR_SHAPE;
   if (slot_rows < rows || e_hi <= e_lo || !cnt || !src_token || !dst_row || !row_scale) return FB_ERR_SHAPE;
   if (q_src == nullptr && !xg) return FB_ERR_SHAPE;
   if (q_src != nullptr && (!s_src || !xg_q || !xg_s || s_cols <= 0 || (ldq % 16) != 0 || (ldxgq % 16) != 0 ||
@@ -1418,7 +1430,7 @@ extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delt
     return FB_ERR_SHAPE;
   const NormPrologue np{static_cast<const __nv_bfloat16*>(delta), ldd, static_cast<const __nv_bfloat16*>(norm_w),
                         static_cast<__nv_bfloat16*>(res_out), ldr, static_cast<__nv_bfloat16*>(norm_out), ldn, eps};
-  const size_t smem = (static_cast<size_t>(hidden) + experts) * sizeof(float) +
+  const size_t smem = (static_cast<size_t>(hidden) + experts + ex.n_extra) * sizeof(float) +
                       (norm_w ? static_cast<size_t>(hidden) * 2 : 0);
   static bool attr_done = false;
   if (!attr_done) {
@@ -1429,8 +1441,35 @@ extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delt
              static_cast<const __nv_bfloat16*>(x), ldx, static_cast<const __nv_bfloat16*>(w), hidden, bias, hash_table,
              token_ids, rows, experts, topk, score_fn, n_groups, topk_groups, normalize, route_scale, out_idx, out_w,
              e_lo, e_hi, slot_rows, dst_slots, cnt, src_token, dst_row, row_scale, static_cast<__nv_bfloat16*>(xg), ldxg,
-             static_cast<DeviceStatus*>(status), np, qr);
+             static_cast<DeviceStatus*>(status), np, qr, ex);
   return FB_CHECK_LAUNCH();
+}
+
+extern "C" int fb_router_append_q(const void* x, long long ldx, const void* delta, long long ldd,
+                                  const void* norm_w, void* res_out, long long ldr, void* norm_out, long long ldn,
+                                  float eps, const void* w, int hidden, const float* bias,
+                                  const long long* hash_table, const int* token_ids, int rows, int experts,
+                                  int topk, int score_fn, int n_groups, int topk_groups, int normalize,
+                                  float route_scale, int* out_idx, float* out_w, int e_lo, int e_hi,
+                                  int slot_rows, int dst_slots, int* cnt, int* src_token, int* dst_row,
+                                  float* row_scale, void* xg, long long ldxg, const void* q_src, long long ldq,
+                                  const void* s_src, long long lds, void* xg_q, long long ldxgq, void* xg_s,
+                                  long long ldxgs, int s_cols, void* status, void* stream) {
+  return run_router_append(x, ldx, delta, ldd, norm_w, res_out, ldr, norm_out, ldn, eps, w, hidden, bias, hash_table, token_ids,
+                           rows, experts, topk, score_fn, n_groups, topk_groups, normalize, route_scale, out_idx, out_w, e_lo,
+                           e_hi, slot_rows, dst_slots, cnt, src_token, dst_row, row_scale, xg, ldxg, q_src, ldq, s_src, lds,
+                           xg_q, ldxgq, xg_s, ldxgs, s_cols, RouterExtra{nullptr, nullptr, 0}, status, stream);
+}
+
+extern "C" int fb_router_append_extra(const void* x, long long ldx, const void* w, int hidden, const float* logit_bias,
+                                      float* extra, int n_extra, int rows, int experts, int topk, int score_fn, int n_groups,
+                                      int topk_groups, int normalize, float route_scale, int* out_idx, float* out_w, int e_lo,
+                                      int e_hi, int slot_rows, int dst_slots, int* cnt, int* src_token, int* dst_row,
+                                      float* row_scale, void* xg, long long ldxg, void* status, void* stream) {
+  return run_router_append(x, ldx, nullptr, 0, nullptr, nullptr, 0, nullptr, 0, 0.f, w, hidden, nullptr, nullptr, nullptr, rows,
+                           experts, topk, score_fn, n_groups, topk_groups, normalize, route_scale, out_idx, out_w, e_lo, e_hi,
+                           slot_rows, dst_slots, cnt, src_token, dst_row, row_scale, xg, ldxg, nullptr, 0, nullptr, 0, nullptr,
+                           0, nullptr, 0, 0, RouterExtra{logit_bias, extra, n_extra}, status, stream);
 }
 
 extern "C" int fb_l2_prefetch(const void* ptr, long long bytes, void* stream) {

@@ -75,11 +75,14 @@ typedef struct FbGemmArgs {
                             //   is bumped once per call when all of this rank's rows are stored
   void* mc_recv;            // epilogue 3, optional: multicast (NVLS) address of the ranks' receive buffers; partials
                             //   are then broadcast with one multimem store instead of one store per peer
+  const float* bias;        // optional [n_out]: added in epilogues 0 and 4 (one group)
+  float act_alpha;          // epilogue 1: gate * sigmoid(alpha gate) * (up + shift); alpha 0 means 1
+  float act_shift;
 } FbGemmArgs;
 
 int fb_gemm_bf16(const FbGemmArgs* args, void* stream);
 
-// fp32 tensors, full 32-bit arithmetic (FMA units); same argument block (epilogues 0..2 and 4, act_limit 0, no collectives)
+// fp32 tensors, full 32-bit arithmetic (FMA units); same argument block (epilogues 0..2, 4 and 5, no collectives)
 int fb_gemm_f32(const FbGemmArgs* args, void* stream);
 
 // ---- block-scaled FP8 GEMM ---------------------------------------------------------------
@@ -155,6 +158,7 @@ typedef struct FbAttnArgs {
                             // KV rows below row_pos were written before the running step began (plain decode)
   const void* gate;         // optional [rows, ldg] (element type of q): head h's output is multiplied by sigmoid(gate[row][h])
   long long ldg;
+  int window;               // > 0: a row sees its last `window` tokens only; splits divide what the row of a tile sees
 } FbAttnArgs;
 
 int fb_mla_attention(const FbAttnArgs* args, void* stream);
@@ -186,6 +190,7 @@ typedef struct FbPrefillAttnArgs {
   float softmax_scale;
   const void* gate;         // optional bf16 [rows, ldg]: head h's output is multiplied by sigmoid(gate[row][h])
   long long ldg;
+  int window;               // > 0: a row sees its last `window` tokens only
 } FbPrefillAttnArgs;
 
 int fb_mla_prefill_tc(const FbPrefillAttnArgs* args, void* stream);
@@ -228,6 +233,29 @@ int fb_gated_residual_norm(const FbLayerTailArgs* args, void* stream);
 int fb_latent_append(const void* src, long long lds, int rank, int row_dim, const float* norm_w, float eps,
                      const long long* write_slot, void* pool, long long pool_rows, int rows, int fp32, void* status,
                      void* stream);
+// latent layers with a query latent or rotated parts: the query latent normalised in place, the cache row of every token
+typedef struct FbLatentPrepArgs {
+  void* cq;                 // [rows, ldp] query latent, normalised in place (null: none)
+  const void* ckv;          // [rows, ldp] `rank` latent features, then `rot` of the key part
+  long long ldp;
+  int rank_q, rank, rot, row_dim, rot_off, rows;
+  const float* q_w;         // [rank_q]
+  const float* kv_w;        // [rank]
+  const float* cos_t;       // [max_pos, rot / 2]
+  const float* sin_t;
+  int max_pos, fp32;
+  const int* positions;
+  const long long* write_slot;
+  void* pool;               // [pool_rows, row_dim]: latent | turned part at rot_off | zeros
+  long long pool_rows;
+  float eps;
+  void* status;
+} FbLatentPrepArgs;
+int fb_latent_prep(const FbLatentPrepArgs* args, void* stream);
+// q[row, h, rot_off ..] = turned src[row, h * rot ..]
+int fb_latent_turn(const void* src, long long lds, int heads, int rot, const float* cos_t, const float* sin_t, int max_pos,
+                   const int* positions, void* q, long long ldq, int row_dim, int rot_off, int rows, int fp32, void* status,
+                   void* stream);
 int fb_softcap(float* logits, long long ldl, int rows, int vocab, float cap, void* stream);
 int fb_state_rotate(int* state_in, int* state_out, int n, int buffers, void* stream);
 
@@ -337,6 +365,65 @@ typedef struct FbScanArgs {
 } FbScanArgs;
 int fb_selective_scan(const FbScanArgs* args, void* stream);    // state <= 128, inner % 8 == 0
 
+// ---- pre-norm blocks (see pre_norm.cu) --------------------------------------------------------------------------
+typedef struct FbPreNormArgs {
+  const float* x;           // [rows, ldx] stream before the step (unused with ids)
+  float* x_out;             // [rows, ldx] after it; another buffer than x when a shift sees rows of this batch
+  long long ldx;
+  const int* ids;           // optional: x = table[ids] * scale
+  const void* table;
+  long long ldt;
+  int vocab;
+  float scale;
+  const void* y;            // optional [rows, ldy]: added to x
+  long long ldy;
+  const void* ffn;          // optional [rows * slots, ldf]: the first `topk` rows of every token are added
+  long long ldf;
+  int slots, topk;
+  const void* shared;       // optional, with ffn: [rows, lds], added times sigmoid(shared_gate[row * ldsg])
+  long long lds;
+  const float* shared_gate;
+  long long ldsg;
+  const float* norm_w;      // [dim_pad]
+  void* act;                // optional [rows, lda]: x / rms(x) * norm_w, shifted
+  long long lda;
+  const float* shift;       // optional [dim_pad]: share of the previous token's normalised row
+  float* plane;             // [n_states, dim_pad] last normalised row of every sequence
+  const int* row_seq;
+  const int* seq_start;
+  const int* state_in;
+  const int* state_out;
+  int n_states, n_seqs;
+  int rows, dim, dim_pad, fp32;
+  float eps;
+  void* status;
+} FbPreNormArgs;
+int fb_pre_norm_step(const FbPreNormArgs* args, void* stream);
+int fb_group_norm_rows(const void* x, long long ldx, const float* norm_w, void* out, long long ldo, int rows, int dim, int dim_pad,
+                       int groups, float eps, int fp32, void* stream);
+
+// ---- scan with one decay per head (see head_scan.cu) --------------------------------------------------------------
+typedef struct FbHeadScanArgs {
+  const void* xbc;          // [rows, ldx] convolved inputs: x (heads x vdim) at 0, B (groups x state) at off_b, C at off_c
+  long long ldx;
+  int off_b, off_c;
+  const void* dt;           // [rows, ldp] step size pre-activation per head, without bias
+  const void* z;            // [rows, ldp] output gate pre-activation: heads x vdim
+  long long ldp;
+  const float* dt_bias;     // [heads]
+  const float* a_neg;       // [heads] decay rates (negative)
+  const float* d_skip;      // [heads]
+  float* states;            // [n_states, heads, state, vdim]
+  const int* seq_start;
+  const int* state_in;
+  const int* state_out;
+  void* out;                // [rows, ldo]: (scan + D x) * silu(z); columns past heads x vdim are zero
+  long long ldo;
+  int rows, n_seqs, heads, vdim, state, groups, n_states, fp32;
+  void* status;
+} FbHeadScanArgs;
+int fb_head_scan(const FbHeadScanArgs* args, void* stream);     // state <= 256
+
 // ---- grouped-query attention in position chunks (see gqa_attention.cu) -----------------------------------------
 typedef struct FbGqaArgs {
   void* q;                  // [rows, ldq]: heads x dim_pad; `fb_gqa_prep` normalises and rotates it in place
@@ -373,6 +460,18 @@ typedef struct FbGqaArgs {
   const void* gate;         // optional [rows, ldg]: output multiplied by sigmoid(gate)
   long long ldg;
   float diff_lambda, diff_scale;
+  // values of a query row of kv head g: `value_width` columns from v_offset + g * value_stride on (stride 0: the values of all
+  // kv heads side by side for every row); out then holds heads x value_width columns
+  int value_width, value_stride;
+  float softcap;            // > 0: score <- softcap tanh(score / softcap)
+  // blocks of `pool_tokens` tokens that lie wholly before a row's window are seen as one cache row each (see gqa_mask.cuh):
+  // row b of sequence s is pooled[(slot_of[s] / slot_div) * pooled_stride + b]
+  const void* pooled;       // [pooled_rows, pool_ld], element type of pool
+  long long pooled_rows;
+  int pool_tokens, pooled_stride, slot_div;
+  const int* slot_of;
+  const float* talk;        // fb_gqa_decode_wide with value_stride 0: out_h = sum_g talk[h, g] (output of head g on the values
+                            // of h's kv head), and out holds heads x vdim_pad columns
   void* status;
 } FbGqaArgs;
 int fb_gqa_prep(const FbGqaArgs* args, void* stream);
@@ -383,7 +482,25 @@ int fb_gqa_decode(const FbGqaArgs* args, int splits, int early, void* stream);
 // the same for keys that all heads share (gqa_decode_wide.cu): key_stride 0, one map; fb_gqa_decode_wide_ok: whether
 // cache rows of this shape fit its pipeline
 int fb_gqa_decode_wide(const FbGqaArgs* args, int splits, int early, void* stream);
-int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad);
+int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads);
+// out[row, h] = sum_g talk[h, g] o[row, g, columns of h's kv head]: o rows hold heads x kv_heads x vdim_pad columns
+int fb_value_mix(const void* o, long long ldv, const float* talk, void* out, long long ldo, int rows, int heads, int kv_heads,
+                 int vdim_pad, int fp32, void* stream);
+// mean cache rows of the blocks of `pool_tokens` tokens that end with a row of this batch: pooled as in FbGqaArgs, `width`
+// columns of the pool's rows
+typedef struct FbPoolArgs {
+  const void* pool;         // [pool_rows, pool_ld]
+  long long pool_rows, pool_ld;
+  void* pooled;             // [pooled_rows, pool_ld]
+  long long pooled_rows;
+  const int* positions;     // [rows], -1: none
+  const int* row_seq;
+  const int* block_table;
+  const int* slot_of;
+  int rows, width, num_seqs, max_blocks, page_size, pool_tokens, pooled_stride, slot_div, fp32;
+  void* status;
+} FbPoolArgs;
+int fb_pool_blocks(const FbPoolArgs* args, void* stream);
 // bf16 prompts on tcgen05 (gqa_prefill_tc.cu): vdim <= 256, page_size a power of two >= 8; tiles [n_tiles, 4] =
 // sequence, first row, rows (<= tile_positions), position of the first; tile_positions * maps * heads / kv_heads <= 128
 int fb_gqa_prefill_tc(const FbGqaArgs* args, const int* tiles, int n_tiles, int tile_positions, void* stream);
@@ -409,6 +526,12 @@ typedef struct FbHeadPrepArgs {
   int rows, heads, kv_heads, maps, dim, dim_pad, vdim_pad, fp32;
   float eps;
   void* status;
+  // optional: rotation of the leading 2 * half dimensions of a head (halves paired); q_norm / k_norm may be null (weights of one)
+  const float* cos_t;       // [max_pos, half]
+  const float* sin_t;
+  const int* positions;
+  int half, max_pos;
+  const FbPoolArgs* blocks; // optional, one row per sequence: also the mean rows of the blocks that end with this step's rows
 } FbHeadPrepArgs;
 int fb_head_prep(const FbHeadPrepArgs* args, void* stream);
 
@@ -469,7 +592,7 @@ int fb_mla_prep(const void* q, long long ldq, int q_head_dim, const void* ckv, l
 int fb_router_topk(const float* logits, long long ldl, const float* bias,
                    const long long* hash_table, const int* token_ids, int rows, int experts,
                    int topk, int score_fn, int n_groups, int topk_groups, int normalize,
-                   float route_scale, int* out_idx, float* out_w, void* stream);
+                   float route_scale, int* out_idx, float* out_w, const float* logit_bias, void* stream);
 int fb_moe_plan(const int* topk_idx, const float* topk_w, int routes, int topk, int e_lo, int e_hi,
                 int ntok, int dst_slots, int* src_token, int* dst_row, float* row_scale, int* tile_group,
                 int* tile_row0, int* tile_rows, int max_tiles, int* counts, int* meta, void* status,
@@ -493,6 +616,13 @@ int fb_router_append(const void* x, long long ldx, const void* w, int hidden, co
                      int n_groups, int topk_groups, int normalize, float route_scale, int* out_idx, float* out_w,
                      int e_lo, int e_hi, int slot_rows, int dst_slots, int* cnt, int* src_token, int* dst_row,
                      float* row_scale, void* xg, long long ldxg, void* status, void* stream);
+// the same with a bias on the logits, and `n_extra` (<= 32) further rows of w behind the experts' whose products with the row
+// are written to extra [rows, n_extra] as they are
+int fb_router_append_extra(const void* x, long long ldx, const void* w, int hidden, const float* logit_bias, float* extra,
+                           int n_extra, int rows, int experts, int topk, int score_fn, int n_groups, int topk_groups,
+                           int normalize, float route_scale, int* out_idx, float* out_w, int e_lo, int e_hi, int slot_rows,
+                           int dst_slots, int* cnt, int* src_token, int* dst_row, float* row_scale, void* xg, long long ldxg,
+                           void* status, void* stream);
 // the same with a prologue: row = bf16(x + delta) (delta may be null) -> res_out, RMSNorm(row) * norm_w -> norm_out
 // and into the router, bit-equal to fb_add_rmsnorm followed by fb_router_append (norm_w null: no prologue)
 int fb_norm_router_append(const void* x, long long ldx, const void* delta, long long ldd, const void* norm_w,

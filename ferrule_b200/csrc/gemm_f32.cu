@@ -1,6 +1,6 @@
 // out = x @ w^T in full 32 bits on the FMA units: the GEMM of models that run in fp32 (no tensor-core mode has 32-bit
 // operands).  Takes the argument block of the tcgen05 GEMM - dense, batched per head, grouped by a MoE row-tile
-// table; store, GELU, SwiGLU, GeGLU and weighted scatter epilogues - with fp32 tensors and pitches in elements.
+// table; store and GELU (with bias), SwiGLU (clamped, scaled, shifted), GeGLU and weighted scatter epilogues - with fp32 tensors and pitches in elements.
 //
 // 64 rows x 64 channels per CTA, 256 threads with 4 x 4 outputs each, K in steps of 16 through shared memory.
 #include "common.cuh"
@@ -17,6 +17,8 @@ struct GemmF32Params {
   float* out;
   long long ldw, w_group_stride, ldx, ldo;
   int n_out, k, groups, x_rows, ntok, dual_offset, x_group_koff, out_group_coff, batched, gelu, geglu;
+  float limit, alpha, shift;
+  const float* bias;
   const int* tile_group;
   const int* tile_row0;
   const int* tile_rows;
@@ -94,7 +96,15 @@ gemm_f32_kernel(const GemmF32Params p) {
       const int n = n0 + tx * 4 + j;
       if (n >= p.n_out) continue;
       float v = acc[i][j];
-      if (DUAL) v = (p.geglu ? gelu_tanh_f(v) : v / (1.f + expf(-v))) * up[i][j];
+      if (DUAL) {
+        float u = up[i][j];
+        if (p.limit > 0.f) {
+          v = fminf(v, p.limit);
+          u = fminf(fmaxf(u, -p.limit), p.limit);
+        }
+        v = (p.geglu ? gelu_tanh_f(v) : v / (1.f + expf(-p.alpha * v))) * (u + p.shift);
+      }
+      if (p.bias) v += p.bias[n];
       if (p.gelu) v = gelu_f(v);
       o[n] = v * sc;
     }
@@ -107,7 +117,7 @@ using namespace fb;
 
 extern "C" int fb_gemm_f32(const FbGemmArgs* a, void* stream) {
   if (!a || !a->w || !a->x || !a->out || a->n_out <= 0 || a->k <= 0 || a->groups <= 0 || a->x_rows <= 0) return FB_ERR_SHAPE;
-  if (a->epilogue < 0 || a->epilogue == 3 || a->epilogue > 5 || a->act_limit != 0.f) return FB_ERR_SHAPE;
+  if (a->epilogue < 0 || a->epilogue == 3 || a->epilogue > 5) return FB_ERR_SHAPE;
   const bool grouped = a->tile_group != nullptr, batched = !grouped && a->groups > 1;
   if (grouped && (!a->tile_row0 || !a->tile_rows || !a->num_tok_tiles || a->max_tok_tiles <= 0 || a->ntok <= 0))
     return FB_ERR_SHAPE;
@@ -118,6 +128,11 @@ extern "C" int fb_gemm_f32(const FbGemmArgs* a, void* stream) {
   p.n_out = a->n_out; p.k = a->k; p.groups = a->groups; p.x_rows = a->x_rows; p.ntok = a->ntok;
   p.dual_offset = a->dual_offset; p.x_group_koff = a->x_group_koff; p.out_group_coff = a->out_group_coff;
   p.batched = batched ? 1 : 0;
+  if (a->bias && (grouped || batched || (a->epilogue != 0 && a->epilogue != 4))) return FB_ERR_SHAPE;
+  p.limit = a->epilogue == 1 ? a->act_limit : 0.f;
+  p.alpha = a->act_alpha == 0.f ? 1.f : a->act_alpha;
+  p.shift = a->act_shift;
+  p.bias = a->bias;
   p.gelu = a->epilogue == 4 ? 1 : 0;
   p.geglu = a->epilogue == 5 ? 1 : 0;
   if (grouped) {

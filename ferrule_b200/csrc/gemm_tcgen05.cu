@@ -9,9 +9,10 @@
 // arrive by TMA into 128-byte-swizzled shared memory, one thread issues
 // tcgen05.mma, four warps drain TMEM and run the fused epilogue:
 //
-//   kEpiStore   : out[row, n]            = acc                      (bf16 or fp32)
-//   kEpiGelu    : out[row, n]            = gelu(acc)                (exact, error-function form)
-//   kEpiSwiGLU  : out[row, n]            = silu(gate) * up          (two weight tiles per k-block)
+//   kEpiStore   : out[row, n]            = acc + bias[n]            (bf16 or fp32; the bias is optional)
+//   kEpiGelu    : out[row, n]            = gelu(acc + bias[n])      (exact, error-function form)
+//   kEpiSwiGLU  : out[row, n]            = silu(gate) * up          (two weight tiles per k-block; optionally clamped inputs,
+//                                          gate * sigmoid(alpha gate) * (up + shift))
 //   kEpiGeGLU   : out[row, n]            = gelu(gate) * up          (the same, tanh form)
 //   kEpiScatter : out[dst_row[row], n]   = acc * row_scale[row]     (MoE down projection)
 //   kEpiAllReduce: partial tiles are pushed into every rank's receive buffer over
@@ -62,6 +63,8 @@ struct GemmParams {
   const int* dst_row;
   const float* row_scale;
   float act_limit;  // SwiGLU clamp (0 = none)
+  float act_alpha, act_shift;
+  const float* bias;         // [n_out], store and GELU
   DeviceStatus* status;
   // fused all-reduce
   int rank;
@@ -98,6 +101,15 @@ struct GemmCfg {
   static_assert(kStages >= 2, "not enough shared memory for a pipeline");
 };
 
+// gate * sigmoid(alpha gate) * (up + shift), both inputs clamped first when a limit is given
+__device__ __forceinline__ float gated_unit(const GemmParams& p, float x, float up) {
+  if (p.act_limit > 0.f) {
+    x = fminf(x, p.act_limit);
+    up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
+  }
+  return x / (1.f + __expf(-p.act_alpha * x)) * (up + p.act_shift);
+}
+
 struct TileInfo {
   int g, row0, rows, nt;
 };
@@ -129,7 +141,6 @@ __device__ __forceinline__ bool tile_empty(const GemmParams& p, int t) {
   return p.tile_group != nullptr && p.tile_rows[t / p.n_tiles] <= 0;
 }
 
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
 
 template <int NTOK, bool DUAL, int EPI>
 __global__ void __launch_bounds__(kGemmThreads, 1)
@@ -337,6 +348,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
       const int row0 = ti.row0, rows = ti.rows;
       const int n = ti.nt * kTileN + ch_in_tile;
       const bool n_ok = n < p.n_out;
+      const float bias_n = (EPI == kEpiStore || EPI == kEpiGelu) && p.bias && n_ok ? p.bias[n] : 0.f;
       const long long ocol = (p.batched ? static_cast<long long>(ti.g) * p.out_group_coff : 0) + n;
       ok = mbar_wait(&acc_full[a], aph, abort_flag, p.status, 0x300);
       if (!ok) break;
@@ -395,6 +407,10 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
             }
           }
         }
+        if ((EPI == kEpiStore || EPI == kEpiGelu) && p.bias) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) v[j] = __float_as_uint(__uint_as_float(v[j]) + bias_n);
+        }
         if (EPI == kEpiGeGLU) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
@@ -418,14 +434,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
             float x = 0.f;
             if (r < rows) {
               x = __uint_as_float(v[j]);
-              if (EPI == kEpiSwiGLU) {
-                float up = __uint_as_float(u[j]);
-                if (p.act_limit > 0.f) {
-                  x = fminf(x, p.act_limit);
-                  up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
-                }
-                x = silu_f(x) * up;
-              }
+              if (EPI == kEpiSwiGLU) x = gated_unit(p, x, __uint_as_float(u[j]));
               if (EPI == kEpiScatter && p.row_scale) x *= p.row_scale[row0 + r];
             }
             sb[j * 128 + ch_in_tile] = __float2bfloat16_rn(x);
@@ -456,14 +465,7 @@ gemm_swapab_kernel(const __grid_constant__ CUtensorMap tmap_w,
             const int r = c0 + j;
             if (r < rows) {
               float x = __uint_as_float(v[j]);
-              if (EPI == kEpiSwiGLU) {
-                float up = __uint_as_float(u[j]);
-                if (p.act_limit > 0.f) {
-                  x = fminf(x, p.act_limit);
-                  up = fminf(fmaxf(up, -p.act_limit), p.act_limit);
-                }
-                x = silu_f(x) * up;
-              }
+              if (EPI == kEpiSwiGLU) x = gated_unit(p, x, __uint_as_float(u[j]));
               long long orow = row0 + r;
               if (EPI == kEpiScatter) {
                 if (p.row_scale) x *= p.row_scale[row0 + r];
@@ -778,6 +780,7 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
   const bool batched = !grouped && a->groups > 1;
   if (batched && (a->epilogue != kEpiStore || a->x_group_koff % 8 != 0)) return FB_ERR_SHAPE;
   if (a->x_rows <= 0) return FB_ERR_SHAPE;
+  if (a->bias && (batched || grouped || (a->epilogue != kEpiStore && a->epilogue != kEpiGelu))) return FB_ERR_SHAPE;
 
   CUtensorMap mw, mx;
   const uint64_t w_rows = static_cast<uint64_t>(a->w_rows_per_group);
@@ -819,6 +822,9 @@ extern "C" int fb_gemm_bf16(const FbGemmArgs* a, void* stream_) {
   p.dst_row = a->dst_row;
   p.row_scale = a->row_scale;
   p.act_limit = a->act_limit;
+  p.act_alpha = a->act_alpha == 0.f ? 1.f : a->act_alpha;
+  p.act_shift = a->act_shift;
+  p.bias = a->bias;
   p.status = static_cast<DeviceStatus*>(a->status);
   const int tok_tiles = grouped ? a->max_tok_tiles
                                 : ((a->x_rows + ntok - 1) / ntok) * (batched ? a->groups : 1);

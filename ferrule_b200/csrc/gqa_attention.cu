@@ -6,9 +6,11 @@
 //   fb_gqa_prep       everything between the projection and the attention in one launch: query and key RMS norm over the
 //                     whole projection, rotation of the leading dimensions (halves paired), value norm per head, mixing
 //                     with the first mixing layer's values of the token (read from that layer's cache row), cache append
+//   fb_value_mix      outputs of every head on the values of every kv head -> outputs whose softmax weights are mixed across heads
 //   fb_gqa_attention  attention in 32-bit arithmetic, one CTA per (query row, head): models that run in fp32, and head sizes
 //                     the tensor-core kernels do not take.  Query rows as wide as the keys they meet (all kv heads' keys
-//                     when scores are mixed across heads), distance bias, difference of two maps, output gate
+//                     when scores are mixed across heads), distance bias, soft cap, mean rows of the blocks before the window,
+//                     values of all kv heads for every query row, difference of two maps, output gate
 #include "act_type.cuh"
 #include "common.cuh"
 #include "ferrule_b200.h"
@@ -41,7 +43,9 @@ struct GqaParams {
   const int* row_pos;
   int num_seqs, max_blocks, page_size;
   KeySpan span;
-  int maps, key_width, key_stride, v_offset;
+  int maps, key_width, key_stride, v_offset, value_width, value_stride, value_slice;
+  float softcap;
+  PooledRows<T> pooled;
   const float* slopes;
   const T* gate;
   long long ldg;
@@ -264,13 +268,13 @@ gqa_prep_vec_kernel(const GqaParams<T> p) {
   }
 }
 
-// CTA = (query row, head); DPL: value features per lane.  A head with two maps attends twice over the same values.
+// CTA = (query row, head, slice of the value columns); DPL: value features per lane.  A head with two maps attends twice over the same values.
 template <typename T, int DPL>
 __global__ void __launch_bounds__(128)
 gqa_attention_kernel(const GqaParams<T> p) {
   pdl_launch_dependents();
   pdl_wait();
-  extern __shared__ float sm[];                 // [key_width] query, [maps][vdim_pad] outputs
+  extern __shared__ float sm[];                 // [key_width] query, [maps][columns] outputs
   __shared__ float sm_m[4], sm_l[4], red[32];
   __shared__ float sm_o[4][DPL * 32];
   float* sq = sm;
@@ -288,8 +292,10 @@ gqa_attention_kernel(const GqaParams<T> p) {
   const int n_keys = kept + max(len - first, 0);
   const float slope = p.slopes ? p.slopes[h] : 0.f;
   // with two maps a query row is zero outside its own half
-  const int part = p.key_width / p.maps;
-  const long long voff = p.v_offset + static_cast<long long>(g) * p.vdim_pad;
+  const int part = p.key_width / p.maps, col0 = blockIdx.z * p.value_slice, cols = min(p.value_slice, p.value_width - col0);
+  const long long voff = p.v_offset + static_cast<long long>(g) * p.value_stride + col0;
+  const long long mean_row = kept > 0 && p.span.pool > 0 ? p.pooled.first(seq) : -1;
+  if (kept > 0 && p.span.pool > 0 && mean_row < 0 && threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xD72, r, seq);
   for (int map = 0; map < p.maps; ++map) {
     const T* qr = p.q + r * p.ldq + (static_cast<long long>(h) * p.maps + map) * p.key_width + map * part;
     const long long koff = static_cast<long long>(g) * p.key_stride + map * part;
@@ -302,22 +308,30 @@ gqa_attention_kernel(const GqaParams<T> p) {
     float m = -INFINITY, l = 0.f;
     for (int i = warp; i < n_keys; i += 4) {
       const int t = i < kept ? i : first + i - kept;
-      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
-      const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
-      if (page < 0 || slot >= p.pool_rows) {
-        if (lane == 0) report_status(p.status, kStatusBadIndex, 0xD71, seq, t);
-        continue;
+      const T* row;
+      if (i < kept && p.span.pool > 0) {
+        if (mean_row < 0) continue;
+        row = p.pooled.base + (mean_row + i) * p.pool_ld;
+      } else {
+        const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+        const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
+        if (page < 0 || slot >= p.pool_rows) {
+          if (lane == 0) report_status(p.status, kStatusBadIndex, 0xD71, seq, t);
+          continue;
+        }
+        row = p.pool + slot * p.pool_ld;
       }
-      const T* row = p.pool + slot * p.pool_ld;
       float s = 0.f, v[DPL];
 #pragma unroll
       for (int j = 0; j < DPL; ++j) {
         const int d = lane + 32 * j;
-        v[j] = d < p.vdim ? act_load(row + voff + d) : 0.f;
+        v[j] = d < cols ? act_load(row + voff + d) : 0.f;
       }
 #pragma unroll 4
       for (int d = lane; d < part; d += 32) s = fmaf(sq[d], act_load(row + koff + d), s);
-      s = fmaf(-slope, static_cast<float>(pos - t), warp_sum(s) * p.scale);
+      s = warp_sum(s) * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      s = fmaf(-slope, static_cast<float>(pos - t), s);
       if (s > m) {
         const float a = expf(m - s);
         m = s;
@@ -342,24 +356,73 @@ gqa_attention_kernel(const GqaParams<T> p) {
       L += w[k] * sm_l[k];
     }
     const float f = L > 0.f ? 1.f / L : 0.f;
-    for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x)
-      res[map * p.vdim_pad + d] =
-          d < p.vdim ? (w[0] * sm_o[0][d] + w[1] * sm_o[1][d] + w[2] * sm_o[2][d] + w[3] * sm_o[3][d]) * f : 0.f;
+    for (int d = threadIdx.x; d < cols; d += blockDim.x)
+      res[map * cols + d] =
+          (w[0] * sm_o[0][d] + w[1] * sm_o[1][d] + w[2] * sm_o[2][d] + w[3] * sm_o[3][d]) * f;
   }
   // every thread finishes the columns it wrote itself
   float inv = 1.f;
   if (p.maps == 2) {
     float ss = 0.f;
-    for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x) {
-      res[d] -= p.diff_lambda * res[p.vdim_pad + d];
+    for (int d = threadIdx.x; d < cols; d += blockDim.x) {
+      res[d] -= p.diff_lambda * res[cols + d];
       ss = fmaf(res[d], res[d], ss);
     }
     inv = p.diff_scale / sqrtf(cta_sum(ss, red) / p.vdim + p.eps);
   }
-  T* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.vdim_pad;
-  const T* gate = p.gate ? p.gate + r * p.ldg + static_cast<long long>(h) * p.vdim_pad : nullptr;
-  for (int d = threadIdx.x; d < p.vdim_pad; d += blockDim.x)
+  T* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.value_width + col0;
+  const T* gate = p.gate ? p.gate + r * p.ldg + static_cast<long long>(h) * p.vdim_pad + col0 : nullptr;
+  for (int d = threadIdx.x; d < cols; d += blockDim.x)
     act_store(dst + d, res[d] * inv * (gate ? sigmoid_f(act_load(gate + d)) : 1.f));
+}
+
+// CTA = (row, kv head): outputs of all heads on the values of one kv head -> mixed outputs of that kv head's own heads
+template <typename T>
+__global__ void __launch_bounds__(128)
+value_mix_kernel(const T* __restrict__ o, long long ldv, const float* __restrict__ talk, T* __restrict__ out, long long ldo,
+                 int heads, int kv_heads, int vp) {
+  pdl_launch_dependents();
+  extern __shared__ float vm_sm[];               // [heads][vp] outputs, [per][heads] shares
+  const int per = heads / kv_heads, c = blockIdx.y, vecs = vp / 8;
+  const long long r = blockIdx.x;
+  float* share = vm_sm + heads * vp;
+  for (int i = threadIdx.x; i < per * heads; i += blockDim.x) share[i] = talk[c * per * heads + i];
+  pdl_wait();
+  for (int i = threadIdx.x; i < heads * vecs; i += blockDim.x) {
+    const int g = i / vecs, d = (i - g * vecs) * 8;
+    float x[8];
+    act_load8(o + r * ldv + (static_cast<long long>(g) * kv_heads + c) * vp + d, x);
+    act_store8(vm_sm + g * vp + d, x);
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < per * vecs; i += blockDim.x) {
+    const int h = i / vecs, d = (i - h * vecs) * 8;
+    float acc[8] = {};
+    for (int g = 0; g < heads; ++g) {
+      float x[8];
+      act_load8(vm_sm + g * vp + d, x);
+      const float w = share[h * heads + g];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, x[j], acc[j]);
+    }
+    act_store8(out + r * ldo + static_cast<long long>(c * per + h) * vp + d, acc);
+  }
+}
+
+template <typename T>
+static int launch_value_mix(const void* o, long long ldv, const float* talk, void* out, long long ldo, int rows, int heads,
+                            int kv_heads, int vp, cudaStream_t s) {
+  const size_t smem = (static_cast<size_t>(heads) * vp + static_cast<size_t>(heads / kv_heads) * heads) * sizeof(float);
+  if (smem > 200 * 1024) return FB_ERR_LIMIT;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(value_mix_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return FB_ERR_LAUNCH;
+    attr = true;
+  }
+  launch_pdl(value_mix_kernel<T>, dim3(rows, kv_heads), dim3(128), smem, s, static_cast<const T*>(o), ldv, talk,
+             static_cast<T*>(out), ldo, heads, kv_heads, vp);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 
 template <typename T>
@@ -373,7 +436,9 @@ static void fill_gqa(const FbGqaArgs* a, GqaParams<T>& p) {
   p.first_pool = static_cast<const T*>(a->first_pool); p.first_off = a->first_off; p.v_mix = a->v_mix;
   p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
   p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
-  p.span = {a->chunk, a->window, a->keep_first};
+  p.span = key_span(a);
+  p.pooled = pooled_rows<T>(a);
+  p.value_width = a->value_width; p.value_stride = a->value_stride; p.softcap = a->softcap;
   p.maps = a->maps; p.key_width = a->key_width; p.key_stride = a->key_stride; p.v_offset = a->v_offset;
   p.slopes = a->slopes; p.gate = static_cast<const T*>(a->gate); p.ldg = a->ldg;
   p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale;
@@ -417,8 +482,11 @@ static int run_prep(const FbGqaArgs* a, cudaStream_t s) {
 }
 
 template <typename T, int DPL>
-static int launch_attention(const GqaParams<T>& p, cudaStream_t s) {
-  const size_t smem = (static_cast<size_t>(p.key_width) + p.maps * p.vdim_pad) * sizeof(float);
+static int launch_attention(GqaParams<T>& p, cudaStream_t s) {
+  p.value_slice = min(p.value_width, DPL * 32);
+  const int slices = (p.value_width + p.value_slice - 1) / p.value_slice;
+  if (slices > 1 && p.maps != 1) return FB_ERR_LIMIT;
+  const size_t smem = (static_cast<size_t>(p.key_width) + p.maps * p.value_slice) * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
   static bool attr = false;
   if (!attr) {
@@ -426,7 +494,7 @@ static int launch_attention(const GqaParams<T>& p, cudaStream_t s) {
       return FB_ERR_LAUNCH;
     attr = true;
   }
-  launch_pdl(gqa_attention_kernel<T, DPL>, dim3(p.rows, p.heads), dim3(128), smem, s, p);
+  launch_pdl(gqa_attention_kernel<T, DPL>, dim3(p.rows, p.heads, slices), dim3(128), smem, s, p);
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 
@@ -434,7 +502,7 @@ template <typename T>
 static int run_attention(const FbGqaArgs* a, cudaStream_t s) {
   GqaParams<T> p{};
   fill_gqa(a, p);
-  const int d = (a->vdim + 31) / 32;
+  const int d = (a->value_width + 31) / 32;
   if (d <= 2) return launch_attention<T, 2>(p, s);
   if (d <= 4) return launch_attention<T, 4>(p, s);
   if (d <= 8) return launch_attention<T, 8>(p, s);
@@ -461,9 +529,20 @@ extern "C" int fb_gqa_prep(const FbGqaArgs* a, void* stream) {
 
 extern "C" int fb_gqa_attention(const FbGqaArgs* a, void* stream) {
   if (!gqa_sizes_ok(a) || !a->out || !a->block_table || !a->row_seq || !a->row_pos || a->num_seqs <= 0 || a->max_blocks <= 0 ||
-      a->page_size <= 0 || !gqa_form_ok(a))
+      a->page_size <= 0 || !gqa_form_ok(a) || a->talk || a->value_width > 16384)
     return FB_ERR_SHAPE;
-  if (a->vdim > 512) return FB_ERR_LIMIT;
+  if (a->maps == 2 && a->vdim > 512) return FB_ERR_LIMIT;
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   return a->fp32 ? run_attention<float>(a, s) : run_attention<__nv_bfloat16>(a, s);
+}
+
+extern "C" int fb_value_mix(const void* o, long long ldv, const float* talk, void* out, long long ldo, int rows, int heads,
+                            int kv_heads, int vdim_pad, int fp32, void* stream) {
+  if (!o || !talk || !out || rows <= 0 || heads <= 0 || kv_heads <= 0 || heads % kv_heads || kv_heads > 65535 || vdim_pad <= 0 ||
+      vdim_pad % 8 || ldv < static_cast<long long>(heads) * kv_heads * vdim_pad || ldo < static_cast<long long>(heads) * vdim_pad)
+    return FB_ERR_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(o) & 15) || (reinterpret_cast<uintptr_t>(out) & 15) || ldv % 8 || ldo % 8) return FB_ERR_ALIGN;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return fp32 ? launch_value_mix<float>(o, ldv, talk, out, ldo, rows, heads, kv_heads, vdim_pad, s)
+              : launch_value_mix<__nv_bfloat16>(o, ldv, talk, out, ldo, rows, heads, kv_heads, vdim_pad, s);
 }

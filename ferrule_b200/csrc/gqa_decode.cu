@@ -395,7 +395,7 @@ extern "C" int fb_gqa_decode(const FbGqaArgs* a, int splits, int early, void* st
   if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->vdim_pad <= 0 || a->vdim_pad % 8 ||
       a->pool_rows <= 0 || a->pool_ld % 8 || a->num_seqs <= 0 || a->max_blocks <= 0 || a->page_size <= 0)
     return FB_ERR_SHAPE;
-  if (!gqa_form_ok(a) || a->key_stride == 0 || a->ldq % 8 || a->ldo % 4 || a->ldg % 4) return FB_ERR_SHAPE;
+  if (!gqa_form_ok(a) || !gqa_plain_form(a) || a->key_stride == 0 || a->ldq % 8 || a->ldo % 4 || a->ldg % 4) return FB_ERR_SHAPE;
   if (splits != 1 && splits != 2 && splits != 4 && splits != 8) return FB_ERR_SHAPE;
   const uintptr_t bits = reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->pool) |
                          reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->gate);
@@ -405,7 +405,7 @@ extern "C" int fb_gqa_decode(const FbGqaArgs* a, int splits, int early, void* st
   p.pool = static_cast<const __nv_bfloat16*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
   p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
   p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
-  p.span = {a->chunk, a->window, a->keep_first};
+  p.span = key_span(a);
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.maps = a->maps; p.v_offset = a->v_offset; p.vdim = a->vdim;
   p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale; p.eps = a->eps;

@@ -1,17 +1,21 @@
-// Window attention of few query rows (decode steps, short portions) whose query rows meet the keys of all kv heads, bf16.
+// Window attention of few query rows (decode steps, short portions) whose query rows meet the keys or the values of all kv heads,
+// bf16.
 //
 // Scores that are mixed across heads are products of one wide query row per head with the concatenated keys of a token
 // (head_prep.cu), so a CTA takes all of a token's cache row: keys and values of every kv head lie side by side there and come
-// as one bulk copy per token.  CTA = (query row, split of the visible keys, block of 16 heads); a tile is KT tokens.
+// as one bulk copy per token.  Softmax weights that are mixed across heads need every head's weights on the values of every kv
+// head: the same rows, queries as wide as one kv head's keys (zero in the other kv heads' columns), and the outputs are mixed
+// when the splits have met.  Mean rows of the blocks before the window (gqa_mask.cuh) are keys like any other.  CTA = (query row, split of the visible keys, block of 16 heads); a tile is KT tokens.
 //
 //   copies   warp 8 looks up a token per lane and keeps all stages requested
 //   scores   warp w of 8 multiplies the 16 query rows with 8 of the tile's keys over a share of the features (MMA, partial
 //            sums in shared memory); query fragments stay in registers when their share is at most 16 steps
 //   softmax  two rows per warp, a key per lane: distance bias, running maximum and sum, probabilities to shared memory
 //   values   warp w accumulates 16-column pieces w, w + 8, ... of the values for all 16 rows; a head keeps the columns of
-//            its own kv head
+//            its own kv head (mixed weights: all of them)
 //
-// The splits of a row (one thread-block cluster) merge through distributed shared memory; the output gate is applied there.
+// The splits of a row (one thread-block cluster; with mixed weights the row's head blocks too) merge through distributed shared
+// memory; the output gate is applied there.
 // The kernel is bound by the cache stream, a 16-row tile is below the 64-row minimum of tcgen05: warp-level MMA.  In a decode
 // step the first tiles (older than the step) are requested before the dependency wait.  Every wait is bounded.
 #include "act_type.cuh"
@@ -44,6 +48,10 @@ struct GwParams {
   __nv_bfloat16* out;
   long long ldo;
   int heads, kv_heads, key_width, vdim_pad;
+  int own_keys;                                    // > 0: a query row is this wide and meets the keys of its kv head
+  float cap_log2, cap_in;                          // soft cap: score2 <- cap_log2 tanh(raw * cap_in / 2); 0: none
+  PooledRows<__nv_bfloat16> pooled;
+  const float* talk;
   int row_bytes, pitch, stages, head_blocks;       // bytes of a token's keys and values, and of its place in a tile
   int early;
   DeviceStatus* status;
@@ -98,11 +106,19 @@ gqa_decode_wide_kernel(const GwParams p) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g4 = lane >> 2, t4 = lane & 3;
   const int seq = p.row_seq[r], pos = p.row_pos[r], per = p.heads / p.kv_heads;
   int lo = 0, hi = 0, first = 0, kept = 0, n_keys = 0;                     // lo, hi: indices into the visible keys
+  long long mean_row = 0;
   if (seq < 0 || seq >= p.num_seqs) {
     if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE80, r, seq);
   } else if (pos >= 0) {
     first = p.span.first(pos);
     kept = p.span.head(pos);
+    if (p.span.pool > 0 && kept > 0) {
+      mean_row = p.pooled.first(seq);
+      if (mean_row < 0 || kept > p.pooled.stride) {
+        if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE82, r, seq);
+        kept = 0;
+      }
+    }
     n_keys = kept + max(min(pos + 1, p.max_blocks * p.page_size) - first, 0);
     const int tiles = (n_keys + KT - 1) / KT, share = (tiles + splits - 1) / splits;
     lo = min(split * share * KT, n_keys);
@@ -138,8 +154,13 @@ gqa_decode_wide_kernel(const GwParams p) {
         waited = true;
       }
       long long slot = 0;
-      if (lane < KT) {
-        const int t = token(min(lo + asked * KT + lane, hi - 1));
+      const __nv_bfloat16* rows = p.pool;
+      const int key = min(lo + asked * KT + lane, hi - 1);
+      if (lane < KT && p.span.pool > 0 && key < kept) {
+        rows = p.pooled.base;
+        slot = mean_row + key;
+      } else if (lane < KT) {
+        const int t = token(key);
         const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
         if (page >= 0 && page < n_pages) slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
         else report_status(p.status, kStatusBadIndex, 0xE81, seq, t);
@@ -152,7 +173,7 @@ gqa_decode_wide_kernel(const GwParams p) {
       if (lane == 0) mbar_arrive_expect_tx(full + st, static_cast<uint32_t>(KT * p.row_bytes));
       __syncwarp();
       if (lane < KT)
-        gw_copy_row(gw_sm + st * tile_bytes + lane * p.pitch, p.pool + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes),
+        gw_copy_row(gw_sm + st * tile_bytes + lane * p.pitch, rows + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes),
                     full + st);
     }
     if (!waited) pdl_wait();
@@ -170,8 +191,13 @@ gqa_decode_wide_kernel(const GwParams p) {
     for (int i = tid; i < 16 * (at.q_pitch / 8); i += kGwThreads) {
       const int row = i / (at.q_pitch / 8), c = (i - row * (at.q_pitch / 8)) * 8;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (row < nh && c < p.key_width)
+      if (p.own_keys > 0) {
+        const int e = c - (h0 + row) / per * p.own_keys;
+        if (row < nh && e >= 0 && e < p.own_keys)
+          v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.own_keys + e);
+      } else if (row < nh && c < p.key_width) {
         v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.key_width + c);
+      }
       *reinterpret_cast<uint4*>(q_s + row * at.q_pitch + c) = v;
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f}, sl[2];         // rows 2 warp, 2 warp + 1
@@ -250,7 +276,10 @@ gqa_decode_wide_kernel(const GwParams p) {
           float s = 0.f;
 #pragma unroll
           for (int q = 0; q < kShares; ++q) s += part_s[(q * 16 + row) * (KT + 1) + lane];
-          x[k] = fmaf(-sl[k], dist, s * p.scale_log2);
+          // tanh as 1 - 2 / (exp(2 x) + 1)
+          if (p.cap_log2 > 0.f) s = fmaf(p.cap_log2, -2.f * __fdividef(1.f, exp2f(s * p.cap_in) + 1.f), p.cap_log2);
+          else s *= p.scale_log2;
+          x[k] = fmaf(-sl[k], dist, s);
         }
       }
       float mx0 = x[0], mx1 = x[1];
@@ -319,7 +348,7 @@ gqa_decode_wide_kernel(const GwParams p) {
     }
   }
   __syncthreads();                                                         // the tiles' memory now holds the outputs
-  const int o_pitch = vcols * 16 + 4;
+  const int o_pitch = (p.talk ? n_cols : vcols) * 16 + 4;
   float* o_s = reinterpret_cast<float*>(gw_sm);                            // [16][o_pitch]
 #pragma unroll
   for (int c = 0; c < NC; ++c) {
@@ -329,31 +358,35 @@ gqa_decode_wide_kernel(const GwParams p) {
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
       const int row = g4 + 8 * half;
-      if (row >= nh || (h0 + row) / per != g) continue;
+      if (row >= nh || (!p.talk && (h0 + row) / per != g)) continue;
+      const int at = row * o_pitch + (p.talk ? g * vcols * 16 : 0) + d;
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
-        o_s[row * o_pitch + d + n * 8] = o[c][n][2 * half];
-        o_s[row * o_pitch + d + n * 8 + 1] = o[c][n][2 * half + 1];
+        o_s[at + n * 8] = o[c][n][2 * half];
+        o_s[at + n * 8 + 1] = o[c][n][2 * half + 1];
       }
     }
   }
-  if (splits > 1) cluster_sync_all();
+  const bool cluster = splits > 1 || (p.talk && p.head_blocks > 1);
+  if (cluster) cluster_sync_all();
   else __syncthreads();
-  const int quads = p.vdim_pad / 4;
-  for (int i = tid + split * blockDim.x; i < nh * quads; i += blockDim.x * splits) {
-    const int h = i / quads, d = (i - h * quads) * 4;
+  // rank of the CTA with split s of head block z in this cluster
+  auto peer = [&](int s, int z) { return static_cast<uint32_t>(s + z * splits); };
+  // columns d .. d + 3 of a row's normalised output over all splits
+  auto merged = [&](int row, int d) {
+    const int z = p.talk ? static_cast<int>(blockIdx.z) : 0;
     float mm = -INFINITY, ll = 0.f;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
     if (splits == 1) {
-      ll = c_l[h];
-      a = *reinterpret_cast<const float4*>(o_s + h * o_pitch + d);
+      ll = c_l[row];
+      a = *reinterpret_cast<const float4*>(o_s + row * o_pitch + d);
     } else {
-      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + h), s)));
+      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + row), peer(s, z))));
       for (int s = 0; s < splits; ++s) {
-        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + h), s));
+        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + row), peer(s, z)));
         const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
-        ll = fmaf(f, ld_cluster_f32(mapa_shared(smem_u32(c_l + h), s)), ll);
-        const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(o_s + h * o_pitch + d), s));
+        ll = fmaf(f, ld_cluster_f32(mapa_shared(smem_u32(c_l + row), peer(s, z))), ll);
+        const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(o_s + row * o_pitch + d), peer(s, z)));
         a.x = fmaf(f, v.x, a.x);
         a.y = fmaf(f, v.y, a.y);
         a.z = fmaf(f, v.z, a.z);
@@ -361,7 +394,47 @@ gqa_decode_wide_kernel(const GwParams p) {
       }
     }
     const float inv = ll > 0.f ? 1.f / ll : 0.f;
-    a = make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+    return make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+  };
+  const int quads = p.vdim_pad / 4;
+  if (p.talk) {
+    // This CTA's share of the columns: merged in place (peers read other columns of this CTA), then heads are mixed.
+    const int all = n_cols * 4, share = (all + splits - 1) / splits, q0 = min(split * share, all), q1 = min(q0 + share, all);
+    for (int i = tid; i < nh * (q1 - q0); i += blockDim.x) {
+      const int row = i / (q1 - q0), d = (q0 + i - row * (q1 - q0)) * 4;
+      *reinterpret_cast<float4*>(o_s + row * o_pitch + d) = merged(row, d);
+    }
+    if (p.head_blocks > 1) cluster_sync_all();
+    else __syncthreads();
+    for (int i = tid; i < per * (q1 - q0); i += blockDim.x) {
+      const int j = i / (q1 - q0), at = (q0 + i - j * (q1 - q0)) * 4, g = at / (vcols * 16), d = at - g * vcols * 16;
+      const int h = g * per + j;
+      if (d >= p.vdim_pad || h < h0 || h >= h0 + nh) continue;
+      const float* t = p.talk + static_cast<long long>(h) * p.heads;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int z = 0; z < p.head_blocks; ++z) {
+        const int n = min(16, p.heads - z * 16);
+        for (int row = 0; row < n; ++row) {
+          const float* src = o_s + row * o_pitch + at;
+          const float4 v = z == static_cast<int>(blockIdx.z) ? *reinterpret_cast<const float4*>(src)
+                                                               : ld_cluster_f32x4(mapa_shared(smem_u32(src), peer(split, z)));
+          const float w = t[z * 16 + row];
+          a.x = fmaf(w, v.x, a.x);
+          a.y = fmaf(w, v.y, a.y);
+          a.z = fmaf(w, v.z, a.z);
+          a.w = fmaf(w, v.w, a.w);
+        }
+      }
+      __nv_bfloat16* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.vdim_pad + d;
+      *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a.x, a.y);
+      *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(a.z, a.w);
+    }
+    if (cluster) cluster_sync_all();                                       // no CTA leaves while a peer reads its rows
+    return;
+  }
+  for (int i = tid + split * blockDim.x; i < nh * quads; i += blockDim.x * splits) {
+    const int h = i / quads, d = (i - h * quads) * 4;
+    float4 a = merged(h, d);
     const long long col = static_cast<long long>(h0 + h) * p.vdim_pad + d;
     if (p.gate) {
       const __nv_bfloat162* z = reinterpret_cast<const __nv_bfloat162*>(p.gate + r * p.ldg + col);
@@ -372,21 +445,21 @@ gqa_decode_wide_kernel(const GwParams p) {
     *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(a.x, a.y);
     *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(a.z, a.w);
   }
-  if (splits > 1) cluster_sync_all();                                      // no CTA leaves while a peer reads its rows
+  if (cluster) cluster_sync_all();                                         // no CTA leaves while a peer reads its rows
 }
 
 // tile size and stages for a cache row of this shape; kt 0: it does not fit
 struct GwPlan {
   int kt, stages, nc, kq;
 };
-static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad) {
+static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad, bool shared_values) {
   const int vcols = (vdim_pad + 15) / 16, cols = kv_heads * vcols, pitch = (key_width + kv_heads * vdim_pad) * 2 + 16;
   const int nc = cols <= 8 ? 1 : cols <= 16 ? 2 : cols <= 32 ? 4 : cols <= 64 ? 8 : 0;
   for (int kt = 32; kt >= 16 && nc; kt /= 2) {
     int stages = (kGwSmemLimit - GwLayout(key_width, 0, kt).total) / (kt * pitch);
     if (stages > kGwMaxStages) stages = kGwMaxStages;
     // the merged outputs reuse the tiles' memory
-    if (stages < 2 || stages * kt * pitch < 16 * (vcols * 16 + 4) * 4) continue;
+    if (stages < 2 || stages * kt * pitch < 16 * ((shared_values ? cols : vcols) * 16 + 4) * 4) continue;
     const int shares = 64 / kt, steps = ((key_width + 15) / 16 + shares - 1) / shares;
     return {kt, stages, nc, steps <= 4 ? 4 : steps <= 16 ? 16 : 0};
   }
@@ -410,7 +483,7 @@ static int launch_gw(const GwParams& p, int rows, int splits, cudaStream_t strea
   attr[0].id = cudaLaunchAttributeClusterDimension;
   attr[0].val.clusterDim.x = 1;
   attr[0].val.clusterDim.y = splits;
-  attr[0].val.clusterDim.z = 1;
+  attr[0].val.clusterDim.z = p.talk ? p.head_blocks : 1;
   attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   attr[1].val.programmaticStreamSerializationAllowed = 1;
   cfg.attrs = attr;
@@ -436,9 +509,10 @@ static int launch_gw_cols(const GwParams& p, const GwPlan& plan, int rows, int s
 
 using namespace fb;
 
-extern "C" int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad) {
+extern "C" int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads) {
+  if (shared_values && (heads + 15) / 16 > 8) return 0;       // the row's head blocks form one cluster
   return key_width > 0 && key_width % 8 == 0 && kv_heads > 0 && vdim_pad > 0 && vdim_pad % 8 == 0 &&
-         gw_plan(key_width, kv_heads, vdim_pad).kt > 0;
+         gw_plan(key_width, kv_heads, vdim_pad, shared_values != 0).kt > 0;
 }
 
 extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, void* stream) {
@@ -446,26 +520,39 @@ extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, voi
   if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->vdim_pad <= 0 || a->vdim_pad % 8 ||
       a->pool_rows <= 0 || a->pool_ld % 8 || a->num_seqs <= 0 || a->max_blocks <= 0 || a->page_size <= 0)
     return FB_ERR_SHAPE;
-  if (!gqa_form_ok(a) || a->key_stride != 0 || a->maps != 1 || a->v_offset != a->key_width || a->ldq % 8 || a->ldo % 4 ||
-      a->ldg % 4)
+  // the keys, the values, or both are shared by all query rows
+  const bool shared_values = a->value_stride == 0;
+  const long long key_width = a->key_stride ? static_cast<long long>(a->kv_heads) * a->key_width : a->key_width;
+  if (!gqa_form_ok(a) || a->maps != 1 || (a->key_stride != 0 && !shared_values) || key_width > 16384 ||
+      a->v_offset != key_width || a->ldq % 8 || a->ldo % 4 || a->ldg % 4 || shared_values != (a->talk != nullptr) ||
+      (shared_values && a->gate))
     return FB_ERR_SHAPE;
+  if (shared_values && (a->heads + 15) / 16 * splits > 8) return FB_ERR_LIMIT;
   if (splits != 1 && splits != 2 && splits != 4 && splits != 8) return FB_ERR_SHAPE;
   const uintptr_t bits = reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->pool) |
-                         reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->gate);
+                         reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->gate) |
+                         reinterpret_cast<uintptr_t>(a->pooled);
   if (bits & 15) return FB_ERR_ALIGN;
-  const GwPlan plan = gw_plan(a->key_width, a->kv_heads, a->vdim_pad);
+  const GwPlan plan = gw_plan(static_cast<int>(key_width), a->kv_heads, a->vdim_pad, shared_values);
   if (plan.kt == 0) return FB_ERR_LIMIT;
   GwParams p{};
   p.q = static_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq;
   p.pool = static_cast<const __nv_bfloat16*>(a->pool); p.pool_rows = a->pool_rows; p.pool_ld = a->pool_ld;
   p.block_table = a->block_table; p.row_seq = a->row_seq; p.row_pos = a->row_pos;
   p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
-  p.span = {a->chunk, a->window, a->keep_first};
+  p.span = key_span(a);
+  p.pooled = pooled_rows<__nv_bfloat16>(a);
+  p.talk = a->talk;
+  p.own_keys = a->key_stride ? a->key_width : 0;
   p.scale_log2 = a->scale * 1.4426950408889634f;
+  if (a->softcap > 0.f) {
+    p.cap_log2 = a->softcap * 1.4426950408889634f;
+    p.cap_in = 2.f * p.scale_log2 / a->softcap;
+  }
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.out = static_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo;
-  p.heads = a->heads; p.kv_heads = a->kv_heads; p.key_width = a->key_width; p.vdim_pad = a->vdim_pad;
-  p.row_bytes = (a->key_width + a->kv_heads * a->vdim_pad) * 2;
+  p.heads = a->heads; p.kv_heads = a->kv_heads; p.key_width = static_cast<int>(key_width); p.vdim_pad = a->vdim_pad;
+  p.row_bytes = (p.key_width + a->kv_heads * a->vdim_pad) * 2;
   p.pitch = p.row_bytes + 16;
   p.stages = plan.stages;
   p.head_blocks = (a->heads + 15) / 16;

@@ -3,8 +3,9 @@
 //
 // CTA = one tile of consecutive query positions of one sequence x the query heads of one key / value head (with two score
 // maps per head: both maps' rows): up to 128 (position, row) rows, P = 128 / rows-per-group positions.  Keys are taken in
-// tiles of 64 tokens at absolute positions 64 j: the tiles with kept first tokens, then from the first tile that holds a
-// key of the first position's chunk or window.
+// tiles of 64 tokens at absolute positions 64 j: the tiles with kept first tokens (or tiles of 64 mean rows of the blocks before
+// the window, gqa_mask.cuh), then from the first tile that holds a key of the first position's chunk or window.  Query rows that
+// meet the values of all kv heads take them in slices of up to 256 columns, a CTA each.
 //
 //   TMA producer (warp 0): the query rows once (boxes of 64 features x group x P), then per token tile the feature blocks of
 //     the keys and of the values straight from the paged pool (box = 64 features x min(page, 64) rows; features past the
@@ -15,7 +16,7 @@
 //   MMA issuer (warp 1): S[128 x 64] = Q K^T, both operands K-major in shared memory, double buffered in TMEM; O[128 x DV]
 //     += P V with P in TMEM as the A operand and the value tile read as an MN-major B operand.  The next tile's S is issued
 //     before the current P is waited for.
-//   Softmax (warps 2..9, two threads per row with half of the tile's columns each): scores from TMEM, scale, distance bias,
+//   Softmax (warps 2..9, two threads per row with half of the tile's columns each): scores from TMEM, scale, distance bias or soft cap,
 //     mask, running maximum (the halves meet in shared memory), exp2, bf16 P written over the score buffer.  The
 //     accumulator is rescaled only when a row's maximum has grown by more than 2^8 since the reference it was scaled by;
 //     the sum uses the same reference, so the result is exact up to rounding.  The difference of a head's two maps is
@@ -52,7 +53,10 @@ struct GpParams {
   int positions;             // positions per tile the query box holds
   int num_seqs, max_blocks, page_size, box_rows;
   KeySpan span;
-  int key_width, vdim_pad, qb, vb;     // qb, vb: 64-feature blocks of a query / key row and of a value row
+  int key_width, value_width, qb, vb;  // qb, vb: 64-feature blocks of a query / key row and of a slice of a value row
+  int shared_values;
+  PooledRows<__nv_bfloat16> pooled;
+  float cap_log2, cap_in;              // soft cap: score2 = cap_log2 tanh(raw * cap_in / 2)
   int kb, pieces, ks, q_resident;      // blocks per key stage, stages per token tile, key stages (2 or 4)
   int shared_keys, k_whole, v_whole;   // whole: one copy brings all feature blocks of a stage
   uint32_t tmem_cols;
@@ -65,11 +69,20 @@ struct GpParams {
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
+enum { kGpPlain = 0, kGpBias = 1, kGpCap = 2 };       // what happens to the scores before the softmax
 
-template <bool BIAS>
+__device__ __forceinline__ float rcp_ftz(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int FORM>
 __global__ void __launch_bounds__(kGpThreads, 2)
 gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                      const __grid_constant__ CUtensorMap map_v, const GpParams p) {
+                      const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_pk,
+                      const __grid_constant__ CUtensorMap map_pv, const GpParams p) {
+  constexpr bool BIAS = FORM == kGpBias, READY = FORM != kGpPlain;      // READY: scores are scaled (base 2) before the mask
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int qb = p.qb, vb = p.vb;
@@ -102,7 +115,10 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
   }
   const int kv_len = min(pos0 + nrows, p.max_blocks * p.page_size);
   const int j0 = p.span.first(pos0) / kGpKv;                             // first token tile of the chunk or window
-  const int n_pre = min((p.span.head(pos0 + nrows - 1) + kGpKv - 1) / kGpKv, j0);      // tiles of kept tokens before it
+  int n_pre = (p.span.head(pos0 + nrows - 1) + kGpKv - 1) / kGpKv;       // tiles of mean rows, or of kept tokens before it
+  if (p.span.pool == 0) n_pre = min(n_pre, j0);
+  auto is_mean = [&](int j) { return p.span.pool > 0 && j < n_pre; };
+  const int slice = blockIdx.z;
   const int n_kv = n_pre + (kv_len + kGpKv - 1) / kGpKv - j0;
   // with a distance bias the latest keys come first: a row's maximum is then mostly among them
   auto tile_of = [&](int j) {
@@ -153,7 +169,16 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         mbar_arrive_expect_tx(q_full, qb * q_block_tx);
         for (int b = 0; b < qb; ++b) tma_load_3d(q_s + b * kGpQBlock, &map_q, q_full, b * 64, g * p.per, row0);
       }
-      const int subs = kGpKv / p.box_rows, key_head = p.shared_keys ? 0 : g;
+      const int subs = kGpKv / p.box_rows, key_head = p.shared_keys ? 0 : g, value_head = p.shared_values ? 0 : g;
+      const int vblock0 = slice * vb;
+      long long mean_row = 0;
+      if (is_mean(0)) {
+        mean_row = p.pooled.first(seq);
+        if (mean_row < 0) {
+          report_status(p.status, kStatusBadIndex, 0xA83, seq, pos0);
+          mean_row = p.pooled.rows;                                      // out of range: the copies fill zeros
+        }
+      }
       const long long n_pages = p.pool_rows / p.page_size;
       const int* pages = p.block_table + static_cast<long long>(seq) * p.max_blocks;
       auto page_of = [&](int t0) { return t0 < kv_len ? pages[t0 / p.page_size] : -1; };
@@ -164,12 +189,18 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       };
       bool ok = true;
       int k_armed = 0, v_armed = 0;                                      // key stages / value tiles that were requested
-      int next_page = page_of(tile_of(0) * kGpKv);                       // read a tile ahead
+      int next_page = is_mean(0) ? -1 : page_of(tile_of(0) * kGpKv);     // read a tile ahead
       for (int j = 0; j < n_kv && ok; ++j) {
         const int st = j & 1, tok = tile_of(j) * kGpKv;
-        const int row = row_of(tok, next_page);                            // of the tile's first box
-        if (j + 1 < n_kv) next_page = page_of(tile_of(j + 1) * kGpKv);
-        auto sub_row = [&](int s) { return s == 0 ? row : row_of(tok + s * p.box_rows, page_of(tok + s * p.box_rows)); };
+        const bool mean = is_mean(j);
+        const int row = mean ? static_cast<int>(min(mean_row + tok, p.pooled.rows)) : row_of(tok, next_page);   // of its first box
+        if (j + 1 < n_kv && !is_mean(j + 1)) next_page = page_of(tile_of(j + 1) * kGpKv);
+        auto sub_row = [&](int s) {
+          if (mean) return row + s * p.box_rows;
+          return s == 0 ? row : row_of(tok + s * p.box_rows, page_of(tok + s * p.box_rows));
+        };
+        const CUtensorMap* mk = mean ? &map_pk : &map_k;
+        const CUtensorMap* mv = mean ? &map_pv : &map_v;
         for (int c = 0; c < p.pieces && ok; ++c) {
           const int i = j * p.pieces + c, ks = i & k_mask, b0 = c * p.kb, nb = min(p.kb, qb - b0);
           if (i >= p.ks) ok = mbar_wait(k_free + ks, ((i >> k_shift) - 1) & 1, abort_flag, p.status, 0xA90);
@@ -177,12 +208,12 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           mbar_arrive_expect_tx(k_full + ks, nb * (static_cast<uint32_t>(kGpKvBlock) + (p.q_resident ? 0u : q_block_tx)));
           uint8_t* dst = k_s + ks * p.kb * kGpKvBlock;
           if (p.k_whole) {
-            tma_load_4d(dst, &map_k, k_full + ks, 0, row, b0, key_head);
+            tma_load_4d(dst, mk, k_full + ks, 0, row, b0, key_head);
           } else {
             for (int s = 0; s < subs; ++s) {
               const int rc = sub_row(s);
               for (int b = 0; b < nb; ++b)
-                tma_load_3d(dst + b * kGpKvBlock + s * p.box_rows * 128, &map_k, k_full + ks, (b0 + b) * 64, key_head, rc);
+                tma_load_3d(dst + b * kGpKvBlock + s * p.box_rows * 128, mk, k_full + ks, (b0 + b) * 64, key_head, rc);
             }
           }
           if (!p.q_resident)
@@ -195,12 +226,13 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         if (!ok) break;
         mbar_arrive_expect_tx(v_full + st, static_cast<uint32_t>(vb * kGpKvBlock));
         if (p.v_whole) {
-          tma_load_4d(v_s + st * vb * kGpKvBlock, &map_v, v_full + st, 0, row, 0, g);
+          tma_load_4d(v_s + st * vb * kGpKvBlock, mv, v_full + st, 0, row, vblock0, value_head);
         } else {
           for (int s = 0; s < subs; ++s) {
             const int rc = sub_row(s);
             for (int b = 0; b < vb; ++b)
-              tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, &map_v, v_full + st, b * 64, g, rc);
+              tma_load_3d(v_s + (st * vb + b) * kGpKvBlock + s * p.box_rows * 128, mv, v_full + st, (vblock0 + b) * 64,
+                          value_head, rc);
           }
         }
         v_armed = j + 1;
@@ -278,8 +310,8 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int at = r / p.per, head = (g * p.per + r - at * p.per) / p.maps;
     const bool valid = at < nrows;
     const int pos = pos0 + at;
-    const int hi = valid ? min(pos + 1, kv_len) : 0;
-    const int lo = p.span.first(pos), keep = p.span.keep;
+    const int hi_tok = valid ? min(pos + 1, kv_len) : 0;
+    const int lo_tok = p.span.first(pos), keep = p.span.keep, n_mean = valid && p.span.pool > 0 ? p.span.head(pos) : 0;
     const float slope = BIAS && valid ? p.slopes[head] * kLog2e : 0.f;
     const uint32_t lane_base = tmem + (static_cast<uint32_t>(quarter * 32) << 16);
     auto pair_sync = [&]() { asm volatile("bar.sync %0, 64;" ::"r"(quarter + 1) : "memory"); };
@@ -296,6 +328,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int c = 0; c < 2; ++c) tmem_ld16(s_t + half * 32 + c * 16, sv[c]);
       tmem_ld_wait();
       const int tok0 = tile_of(j) * kGpKv + half * 32;
+      const int lo = is_mean(j) ? 0 : lo_tok, hi = is_mean(j) ? n_mean : hi_tok;
       // four independent chains for the maximum and the sum, packed multiply-adds
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (BIAS) {
@@ -312,6 +345,14 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             sv[c][i] = __float_as_uint(x0);
             sv[c][i + 1] = __float_as_uint(x1);
           }
+      }
+      if (FORM == kGpCap) {
+        // tanh as 1 - 2 / (exp(2 x) + 1)
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            sv[c][i] = __float_as_uint(fmaf(-2.f * p.cap_log2, rcp_ftz(exp2_ftz(__uint_as_float(sv[c][i]) * p.cap_in) + 1.f), p.cap_log2));
       }
       if (__all_sync(0xffffffffu, tok0 + 32 <= hi && (tok0 >= lo || tok0 + 32 <= keep))) {
 #pragma unroll
@@ -330,7 +371,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
           }
       }
       float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      if (!BIAS) mx *= p.scale_log2;                          // the scale is positive
+      if (!READY) mx *= p.scale_log2;                         // the scale is positive
       {
         // both halves see the same two rounded maxima; behind the barrier both have read their scores
         __nv_bfloat16* slot = max_x + (j & 1) * 256;
@@ -370,7 +411,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int i = 0; i < 16; ++i) {
         const uint64_t x = pack2(__uint_as_float(sv[i >> 3][(2 * i) & 15]), __uint_as_float(sv[i >> 3][((2 * i) & 15) + 1]));
         float p0, p1;
-        unpack2(BIAS ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
+        unpack2(READY ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
         p0 = exp2_ftz(p0);
         p1 = exp2_ftz(p1);
         add[i & 1] = add2(add[i & 1], pack2(p0, p1));
@@ -393,13 +434,15 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     pair_sync();
     l_sum += sum_x[(half ^ 1) * 128 + r];
     const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
-    __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.vdim_pad;
-    const __nv_bfloat16* gate = p.gate ? p.gate + static_cast<long long>(row0 + at) * p.ldg + static_cast<long long>(head) * p.vdim_pad
+    __nv_bfloat16* dst = p.out + static_cast<long long>(row0 + at) * p.ldo + static_cast<long long>(head) * p.value_width +
+                         slice * vb * 64;
+    const __nv_bfloat16* gate = p.gate ? p.gate + static_cast<long long>(row0 + at) * p.ldg + static_cast<long long>(head) * p.value_width
                                        : nullptr;
-    const int chunks = (p.vdim_pad + 15) / 16;                // of 16 columns: every second one per half
+    const int cols = min(vb * 64, p.value_width - slice * vb * 64);
+    const int chunks = (cols + 15) / 16;                // of 16 columns: every second one per half
     // eight columns of a row: output gate, rounding, store
     auto finish = [&](float (&d)[8], int col) {
-      if (!valid || !ok || col >= p.vdim_pad) return;
+      if (!valid || !ok || col >= cols) return;
       if (gate) {
         float z[8];
         act_load8(gate + col, z);
@@ -503,16 +546,16 @@ static int gp_map_blocks(CUtensorMap* map, const void* base, int width, int head
 
 using namespace fb;
 
-template <bool BIAS>
-static int launch_gp(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const GpParams& p, int n_tiles, int smem,
-                     cudaStream_t stream) {
+template <int FORM>
+static int launch_gp(const CUtensorMap (&m)[5], const GpParams& p, int n_tiles, int slices, int smem, cudaStream_t stream) {
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(gqa_prefill_tc_kernel<BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGpSmemLimit) != cudaSuccess)
+    if (cudaFuncSetAttribute(gqa_prefill_tc_kernel<FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, kGpSmemLimit) != cudaSuccess)
       return FB_ERR_LAUNCH;
     attr = true;
   }
-  if (launch_pdl(gqa_prefill_tc_kernel<BIAS>, dim3(n_tiles, p.kv_heads), dim3(kGpThreads), smem, stream, mq, mk, mv, p) != cudaSuccess)
+  if (launch_pdl(gqa_prefill_tc_kernel<FORM>, dim3(n_tiles, p.kv_heads, slices), dim3(kGpThreads), smem, stream, m[0], m[1],
+                 m[2], m[3], m[4], p) != cudaSuccess)
     return FB_ERR_LAUNCH;
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
@@ -520,12 +563,15 @@ static int launch_gp(const CUtensorMap& mq, const CUtensorMap& mk, const CUtenso
 extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_tiles, int tile_positions, void* stream_) {
   if (!a || !a->q || !a->pool || !a->out || !a->block_table || !tiles || a->fp32) return FB_ERR_SHAPE;
   if (a->rows <= 0 || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->kv_heads > 65535 || n_tiles <= 0 ||
-      a->num_seqs <= 0 || a->max_blocks <= 0 || !(a->scale > 0.f) || !gqa_form_ok(a))
+      a->num_seqs <= 0 || a->max_blocks <= 0 || !(a->scale > 0.f) || !gqa_form_ok(a) || a->talk ||
+      (a->softcap > 0.f && a->slopes))
     return FB_ERR_SHAPE;
   const int per = a->heads / a->kv_heads * a->maps;
   if (tile_positions <= 0 || per * tile_positions > kGpM) return FB_ERR_SHAPE;
   if (a->page_size < 8 || (a->page_size & (a->page_size - 1)) != 0) return FB_ERR_SHAPE;
-  if (a->vdim_pad <= 0 || a->vdim_pad > 256 || a->vdim_pad % 8) return FB_ERR_LIMIT;
+  if (a->vdim_pad <= 0 || a->vdim_pad % 8 || (a->value_stride != 0 && a->vdim_pad > 256) || (a->value_stride == 0 && a->gate))
+    return FB_ERR_LIMIT;
+  if (a->pooled && (a->pooled_rows > 0x7fffffffLL || (reinterpret_cast<uintptr_t>(a->pooled) & 15))) return FB_ERR_SHAPE;
   if (a->pool_rows <= 0 || a->pool_rows > 0x7fffffffLL || a->pool_rows % a->page_size) return FB_ERR_SHAPE;
   if (a->ldo % 8 || a->ldg % 8 || (reinterpret_cast<uintptr_t>(a->out) & 15) || (reinterpret_cast<uintptr_t>(a->gate) & 15) ||
       (reinterpret_cast<uintptr_t>(tiles) & 15))
@@ -533,8 +579,8 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   cudaStream_t stream = static_cast<cudaStream_t>(stream_);
   GpParams p{};
   p.box_rows = a->page_size < kGpKv ? a->page_size : kGpKv;
-  CUtensorMap mq, mk, mv;
-  int rc = gp_map(&mq, a->q, a->key_width, a->heads * a->maps, static_cast<uint64_t>(a->rows), a->ldq, per, tile_positions);
+  CUtensorMap maps[5];
+  int rc = gp_map(&maps[0], a->q, a->key_width, a->heads * a->maps, static_cast<uint64_t>(a->rows), a->ldq, per, tile_positions);
   if (rc != FB_OK) return rc;
   const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a->pool);
   p.shared_keys = a->key_stride == 0;
@@ -545,11 +591,19 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   p.pool_rows = a->pool_rows;
   p.rows = a->rows; p.heads = a->heads; p.kv_heads = a->kv_heads; p.per = per; p.positions = tile_positions;
   p.num_seqs = a->num_seqs; p.max_blocks = a->max_blocks; p.page_size = a->page_size;
-  p.span = {a->chunk, a->window, a->keep_first};
-  p.key_width = a->key_width; p.vdim_pad = a->vdim_pad;
-  p.qb = (a->key_width + 63) / 64; p.vb = (a->vdim_pad + 63) / 64;
+  p.span = key_span(a);
+  p.pooled = pooled_rows<__nv_bfloat16>(a);
+  p.key_width = a->key_width; p.value_width = a->value_width;
+  p.shared_values = a->value_stride == 0;
+  const int value_blocks = (a->value_width + 63) / 64, slices = (value_blocks + 3) / 4;
+  if (slices > 65535) return FB_ERR_LIMIT;
+  p.qb = (a->key_width + 63) / 64; p.vb = (value_blocks + slices - 1) / slices;
   p.tmem_cols = p.vb * 64 + 2 * kGpKv <= 256 ? 256 : 512;
   p.scale_log2 = a->scale * kLog2e;
+  if (a->softcap > 0.f) {
+    p.cap_log2 = a->softcap * kLog2e;
+    p.cap_in = 2.f * p.scale_log2 / a->softcap;
+  }
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.maps = a->maps; p.vdim = a->vdim;
   p.diff_lambda = a->diff_lambda; p.diff_scale = a->diff_scale; p.eps = a->eps;
@@ -564,16 +618,22 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   }
   if (smem == 0) return FB_ERR_LIMIT;
   p.pieces = (p.qb + p.kb - 1) / p.kb;
-  const int key_heads = p.shared_keys ? 1 : a->kv_heads;
-  const uint64_t pool_rows = static_cast<uint64_t>(a->pool_rows);
+  const int key_heads = p.shared_keys ? 1 : a->kv_heads, value_heads = p.shared_values ? 1 : a->kv_heads;
   p.k_whole = p.box_rows == kGpKv && a->key_width % 64 == 0 && p.qb % p.kb == 0;
-  p.v_whole = p.box_rows == kGpKv && a->vdim_pad % 64 == 0;
-  rc = p.k_whole ? gp_map_blocks(&mk, pool, a->key_width, key_heads, pool_rows, a->pool_ld, p.kb)
-                 : gp_map(&mk, pool, a->key_width, key_heads, pool_rows, a->pool_ld, 1, p.box_rows);
-  if (rc != FB_OK) return rc;
-  const __nv_bfloat16* values = pool + a->v_offset;
-  rc = p.v_whole ? gp_map_blocks(&mv, values, a->vdim_pad, a->kv_heads, pool_rows, a->pool_ld, p.vb)
-                 : gp_map(&mv, values, a->vdim_pad, a->kv_heads, pool_rows, a->pool_ld, 1, p.box_rows);
-  if (rc != FB_OK) return rc;
-  return a->slopes ? launch_gp<true>(mq, mk, mv, p, n_tiles, smem, stream) : launch_gp<false>(mq, mk, mv, p, n_tiles, smem, stream);
+  p.v_whole = p.box_rows == kGpKv && a->value_width % 64 == 0;
+  for (int i = 0; i < 2; ++i) {
+    // the paged pool, and the mean rows (without any, the pool again)
+    const bool mean = i == 1 && a->pooled;
+    const __nv_bfloat16* base = mean ? p.pooled.base : pool;
+    const uint64_t rows = static_cast<uint64_t>(mean ? a->pooled_rows : a->pool_rows);
+    rc = p.k_whole ? gp_map_blocks(&maps[1 + 2 * i], base, a->key_width, key_heads, rows, a->pool_ld, p.kb)
+                   : gp_map(&maps[1 + 2 * i], base, a->key_width, key_heads, rows, a->pool_ld, 1, p.box_rows);
+    if (rc != FB_OK) return rc;
+    rc = p.v_whole ? gp_map_blocks(&maps[2 + 2 * i], base + a->v_offset, a->value_width, value_heads, rows, a->pool_ld, p.vb)
+                   : gp_map(&maps[2 + 2 * i], base + a->v_offset, a->value_width, value_heads, rows, a->pool_ld, 1, p.box_rows);
+    if (rc != FB_OK) return rc;
+  }
+  if (a->slopes) return launch_gp<kGpBias>(maps, p, n_tiles, slices, smem, stream);
+  if (a->softcap > 0.f) return launch_gp<kGpCap>(maps, p, n_tiles, slices, smem, stream);
+  return launch_gp<kGpPlain>(maps, p, n_tiles, slices, smem, stream);
 }

@@ -1,5 +1,6 @@
-// Everything between the input projection and window attention in one launch: biases, query and key RMS norm per head, the
-// factors of the scores, mixing of scores across heads, cache append.
+// Everything between the input projection and window attention in one launch: biases, rotation, query and key RMS norm per head,
+// the factors of the scores, mixing of scores across heads, cache append; in decode steps also the mean rows of the blocks of
+// tokens that this step completes (fb_pool_blocks: the same for any batch, in a launch of its own).
 //
 // score_h = sum_g M[h, g] q_g . k_kv(g) is linear in the queries, so heads are mixed here: row h of the output holds, side by
 // side for every kv head, the sum of M[h, g] q_g over the heads g of that kv head, and meets the concatenated keys of all kv
@@ -14,6 +15,61 @@
 namespace fb {
 
 constexpr int kHpThreads = 256;
+
+template <typename T>
+struct PoolParams {
+  const T* pool;
+  long long pool_rows, pool_ld;
+  T* pooled;
+  long long pooled_rows;
+  const int* positions;
+  const int* row_seq;
+  const int* block_table;
+  const int* slot_of;
+  int rows, width, num_seqs, max_blocks, page_size, pool_tokens, pooled_stride, slot_div;
+  DeviceStatus* status;
+};
+
+// the mean cache row of the block that ends with batch row r, if one does: eight columns per thread
+template <typename T>
+__device__ __forceinline__ void pool_block(const PoolParams<T>& p, int r) {
+  const int pos = p.positions[r], P = p.pool_tokens;
+  if (pos < 0 || (pos + 1) % P) return;
+  const int seq = p.row_seq[r], b = pos / P;
+  const int slot = seq >= 0 && seq < p.num_seqs ? p.slot_of[seq] : -1;
+  if (slot < 0) return;                                          // a row of no sequence
+  const long long dst = static_cast<long long>(slot / p.slot_div) * p.pooled_stride + b;
+  if (b >= p.pooled_stride || dst >= p.pooled_rows || pos >= p.max_blocks * p.page_size) {
+    if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xE30, r, pos);
+    return;
+  }
+  for (int c = threadIdx.x * 8; c < p.width; c += blockDim.x * 8) {
+    float sum[8] = {};
+    for (int t = pos + 1 - P; t <= pos; ++t) {
+      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
+      const long long row = static_cast<long long>(page) * p.page_size + t % p.page_size;
+      if (page < 0 || row >= p.pool_rows) {
+        report_status(p.status, kStatusBadIndex, 0xE31, seq, t);
+        continue;
+      }
+      float x[8];
+      act_load8(p.pool + row * p.pool_ld + c, x);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sum[j] += x[j];
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) sum[j] /= P;
+    act_store8(p.pooled + dst * p.pool_ld + c, sum);
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+pool_blocks_kernel(const PoolParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  pool_block(p, blockIdx.x);
+}
 
 template <typename T>
 struct HeadPrepParams {
@@ -33,8 +89,24 @@ struct HeadPrepParams {
   long long pool_rows, pool_ld;
   int heads, kv_heads, maps, dim, dim_pad, vdim_pad;
   float eps;
+  const float* cos_t;
+  const float* sin_t;
+  const int* positions;
+  int half, max_pos;
+  PoolParams<T> blocks;
   DeviceStatus* status;
 };
+
+// eight features of a head from d0 on, rotated: feature d turns with d + half
+__device__ __forceinline__ void turned8(const float* x, int d0, int half, const float* cs, const float* sn, float (&o)[8]) {
+#pragma unroll
+  for (int j = 0; j < 8; ++j) {
+    const int d = d0 + j;
+    if (d < half) o[j] = x[d] * cs[d] - x[d + half] * sn[d];
+    else if (d < 2 * half) o[j] = x[d] * cs[d - half] + x[d - half] * sn[d - half];
+    else o[j] = x[d];
+  }
+}
 
 template <typename T, bool MIX>
 __global__ void __launch_bounds__(kHpThreads)
@@ -45,7 +117,9 @@ head_prep_kernel(const HeadPrepParams<T> p) {
   float* sq = hp_sm;                       // [nq][dim_pad]
   float* sk = sq + nq * dp;                // [nk][dim_pad]
   float* inv = sk + nk * dp;               // [nq + nk]
-  float* coef = inv + nq + nk;             // mix: [heads][heads]
+  float* coef = inv + nq + nk;             // mix: [heads][heads]; else cosines and sines
+  float* cs = coef;
+  float* sn = cs + p.half;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = kHpThreads / 32;
   if (MIX)
     for (int i = tid; i < p.heads * p.heads; i += kHpThreads) coef[i] = p.q_mix[i];
@@ -53,6 +127,17 @@ head_prep_kernel(const HeadPrepParams<T> p) {
   const long long r = blockIdx.x, slot = p.write_slot[r];
   const bool keep = slot >= 0 && slot < p.pool_rows;
   if (!keep && slot != -1 && tid == 0) report_status(p.status, kStatusBadIndex, 0xE20, r, static_cast<uint32_t>(slot));
+  if (p.half) {
+    int pos = p.positions[r];
+    if (pos < 0 || pos >= p.max_pos) {
+      if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE21, r, pos);
+      pos = 0;
+    }
+    for (int i = tid; i < p.half; i += kHpThreads) {
+      cs[i] = p.cos_t[static_cast<long long>(pos) * p.half + i];
+      sn[i] = p.sin_t[static_cast<long long>(pos) * p.half + i];
+    }
+  }
   T* row = p.pool + (keep ? slot : 0) * p.pool_ld;
   T* vrow = row + nk * dp;
   for (int i = tid; i < (nq + nk) * vecs; i += kHpThreads) {
@@ -84,15 +169,19 @@ head_prep_kernel(const HeadPrepParams<T> p) {
     if (lane == 0) inv[h] = 1.f / sqrtf(ss / p.dim + p.eps);
   }
   __syncthreads();
+  auto weighted = [&](float (&x)[8], const float* norm, int d, float f) {
+    float w[8];
+    if (norm) act_load8(norm + d, w);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] *= norm ? f * w[j] : f;
+  };
   if (keep)
     for (int i = tid; i < nk * vecs; i += kHpThreads) {
       const int h = i / vecs, d = (i - h * vecs) * 8;
-      float x[8], w[8];
-      act_load8(sk + h * dp + d, x);
-      act_load8(p.k_norm + d, w);
-      const float f = inv[nq + h];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) x[j] *= f * w[j];
+      float x[8];
+      if (p.half) turned8(sk + h * dp, d, p.half, cs, sn, x);        // (turning keeps the root mean square)
+      else act_load8(sk + h * dp + d, x);
+      weighted(x, p.k_norm, d, inv[nq + h]);
       act_store8(row + h * dp + d, x);
     }
   T* out = p.q_out + r * p.ldqo;
@@ -128,16 +217,30 @@ head_prep_kernel(const HeadPrepParams<T> p) {
       const int c = i / vecs, d = (i - c * vecs) * 8, h = c / p.maps;
       float x[8] = {};
       if (c - h * p.maps == h % p.maps) {
-        float w[8];
-        act_load8(sq + h * dp + d, x);
-        act_load8(p.q_norm + d, w);
-        const float f = inv[h] * p.q_mix[h / p.maps];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) x[j] *= f * w[j];
+        if (p.half) turned8(sq + h * dp, d, p.half, cs, sn, x);
+        else act_load8(sq + h * dp + d, x);
+        weighted(x, p.q_norm, d, inv[h] * p.q_mix[h / p.maps]);
       }
       act_store8(out + static_cast<long long>(i) * 8, x);
     }
+    if (p.blocks.pooled && keep) {
+      __syncthreads();                     // this step's own cache row is complete
+      pool_block(p.blocks, static_cast<int>(r));
+    }
   }
+}
+
+template <typename T>
+static PoolParams<T> pool_params(const FbPoolArgs* a) {
+  return {static_cast<const T*>(a->pool), a->pool_rows, a->pool_ld, static_cast<T*>(a->pooled), a->pooled_rows, a->positions,
+          a->row_seq, a->block_table, a->slot_of, a->rows, a->width, a->num_seqs, a->max_blocks, a->page_size, a->pool_tokens,
+          a->pooled_stride, a->slot_div, static_cast<DeviceStatus*>(a->status)};
+}
+static bool pool_args_ok(const FbPoolArgs* a) {
+  return a->pool && a->pooled && a->positions && a->row_seq && a->block_table && a->slot_of && a->rows > 0 && a->pool_rows > 0 &&
+         a->pooled_rows > 0 && a->width > 0 && a->width % 8 == 0 && a->width <= a->pool_ld && a->pool_ld % 8 == 0 &&
+         a->num_seqs > 0 && a->max_blocks > 0 && a->page_size > 0 && a->pool_tokens > 0 && a->pooled_stride > 0 &&
+         a->slot_div > 0 && !(reinterpret_cast<uintptr_t>(a->pool) & 15) && !(reinterpret_cast<uintptr_t>(a->pooled) & 15);
 }
 
 template <typename T, bool MIX>
@@ -150,8 +253,10 @@ static int run_head_prep(const FbHeadPrepArgs* a, cudaStream_t s) {
   p.heads = a->heads; p.kv_heads = a->kv_heads; p.maps = a->maps;
   p.dim = a->dim; p.dim_pad = a->dim_pad; p.vdim_pad = a->vdim_pad; p.eps = a->eps;
   p.status = static_cast<DeviceStatus*>(a->status);
+  p.cos_t = a->cos_t; p.sin_t = a->sin_t; p.positions = a->positions; p.half = a->half; p.max_pos = a->max_pos;
+  if (a->blocks) p.blocks = pool_params<T>(a->blocks);
   const size_t n = static_cast<size_t>(a->heads + a->kv_heads) * a->maps;
-  const size_t smem = (n * a->dim_pad + n + (MIX ? static_cast<size_t>(a->heads) * a->heads : 0)) * sizeof(float);
+  const size_t smem = (n * a->dim_pad + n + (MIX ? static_cast<size_t>(a->heads) * a->heads : 2 * a->half)) * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
   static bool attr = false;
   if (!attr) {
@@ -168,11 +273,16 @@ static int run_head_prep(const FbHeadPrepArgs* a, cudaStream_t s) {
 using namespace fb;
 
 extern "C" int fb_head_prep(const FbHeadPrepArgs* a, void* stream) {
-  if (!a || !a->q || !a->k || !a->q_norm || !a->k_norm || !a->q_mix || !a->q_out || !a->write_slot || !a->pool || a->rows <= 0 ||
+  if (!a || !a->q || !a->k || (a->mix && (!a->q_norm || !a->k_norm)) || !a->q_mix || !a->q_out || !a->write_slot || !a->pool || a->rows <= 0 ||
       a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || (a->maps != 1 && a->maps != 2) || (a->mix && a->maps != 1) ||
       a->dim <= 0 || a->dim_pad < a->dim || a->dim_pad % 8 || a->vdim_pad <= 0 || a->vdim_pad % 8 || a->pool_rows <= 0)
     return FB_ERR_SHAPE;
   if (!a->v && (a->maps != 1 || a->vdim_pad != a->dim_pad)) return FB_ERR_SHAPE;
+  if (a->half < 0 || (a->half && (a->mix || 2 * a->half > a->dim || !a->cos_t || !a->sin_t || !a->positions || a->max_pos <= 0)))
+    return FB_ERR_SHAPE;
+  if (a->blocks && (a->mix || !pool_args_ok(a->blocks) || a->blocks->rows != a->rows || a->blocks->fp32 != a->fp32 ||
+                    a->blocks->pool != a->pool))
+    return FB_ERR_SHAPE;
   const long long kw = static_cast<long long>(a->mix ? a->kv_heads : a->maps) * a->dim_pad;
   if (a->ldqo < a->heads * a->maps * kw || a->ldp < static_cast<long long>(a->heads) * a->maps * a->dim_pad ||
       a->pool_ld < static_cast<long long>(a->kv_heads) * (a->maps * a->dim_pad + a->vdim_pad))
@@ -185,4 +295,12 @@ extern "C" int fb_head_prep(const FbHeadPrepArgs* a, void* stream) {
   cudaStream_t s = static_cast<cudaStream_t>(stream);
   if (a->fp32) return a->mix ? run_head_prep<float, true>(a, s) : run_head_prep<float, false>(a, s);
   return a->mix ? run_head_prep<__nv_bfloat16, true>(a, s) : run_head_prep<__nv_bfloat16, false>(a, s);
+}
+
+extern "C" int fb_pool_blocks(const FbPoolArgs* a, void* stream) {
+  if (!a || !pool_args_ok(a)) return FB_ERR_SHAPE;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  if (a->fp32) launch_pdl(pool_blocks_kernel<float>, dim3(a->rows), dim3(128), 0, s, pool_params<float>(a));
+  else launch_pdl(pool_blocks_kernel<__nv_bfloat16>, dim3(a->rows), dim3(128), 0, s, pool_params<__nv_bfloat16>(a));
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }

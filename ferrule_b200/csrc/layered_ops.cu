@@ -164,6 +164,101 @@ latent_append_kernel(const T* __restrict__ src, long long lds, int rank, int row
   for (int i = lane; i < row_dim; i += 32) act_store(d + i, i < rank ? act_load(s + i) * inv * norm_w[i] : 0.f);
 }
 
+// ---------------------------------------------------------------------------------
+// Latent layers with rotated parts: one CTA per token normalises the query latent in place (when the layer has one) and
+// appends [normalised latent | turned key part | zeros] to the cache; neighbouring dimensions turn together.
+// fb_latent_turn writes the turned query parts into the query rows of the attention, after the latent product.
+// ---------------------------------------------------------------------------------
+template <typename T>
+struct LatentPrepParams {
+  T* cq;                    // [rows, ldp]: rank_q wide, normalised in place; null: none
+  const T* ckv;             // [rows, ldp]: rank, then rot
+  long long ldp;
+  int rank_q, rank, rot, row_dim, rot_off;
+  const float* q_w;
+  const float* kv_w;
+  const float* cos_t;       // [max_pos, rot / 2]
+  const float* sin_t;
+  int max_pos;
+  const int* positions;
+  const long long* write_slot;
+  T* pool;
+  long long pool_rows;
+  float eps;
+  DeviceStatus* status;
+};
+
+__device__ __forceinline__ int checked_pos(int pos, int max_pos, int r, DeviceStatus* st) {
+  if (pos >= 0 && pos < max_pos) return pos;
+  if (threadIdx.x == 0) report_status(st, kStatusBadIndex, 0xB30, r, pos);
+  return 0;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(const LatentPrepParams<T> p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[2][32];
+  const long long r = blockIdx.x, slot = p.write_slot[r];
+  const int pos = p.rot ? checked_pos(p.positions[r], p.max_pos, blockIdx.x, p.status) : 0;
+  const bool keep = slot >= 0 && slot < p.pool_rows;
+  if (!keep && slot != -1 && threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xB31, r, static_cast<uint32_t>(slot));
+  T* q = p.cq ? p.cq + r * p.ldp : nullptr;
+  const T* c = p.ckv + r * p.ldp;
+  float sq = 0.f, sc = 0.f;
+  if (q)
+    for (int i = threadIdx.x; i < p.rank_q; i += blockDim.x) {
+      const float v = act_load(q + i);
+      sq = fmaf(v, v, sq);
+    }
+  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) {
+    const float v = act_load(c + i);
+    sc = fmaf(v, v, sc);
+  }
+  sq = cta_sum(sq, red[0]);
+  sc = cta_sum(sc, red[1]);
+  if (q) {
+    const float f = 1.f / sqrtf(sq / p.rank_q + p.eps);
+    for (int i = threadIdx.x; i < p.rank_q; i += blockDim.x) act_store(q + i, act_load(q + i) * f * p.q_w[i]);
+  }
+  if (!keep) return;
+  const float f = 1.f / sqrtf(sc / p.rank + p.eps);
+  T* d = p.pool + slot * p.row_dim;
+  const int half = p.rot / 2;
+  for (int i = threadIdx.x; i < p.row_dim; i += blockDim.x) {
+    const int e = i - p.rot_off;
+    if (i < p.rank) {
+      act_store(d + i, act_load(c + i) * f * p.kv_w[i]);
+    } else if (e >= 0 && e < p.rot) {
+      const float cs = p.cos_t[static_cast<long long>(pos) * half + e / 2], sn = p.sin_t[static_cast<long long>(pos) * half + e / 2];
+      const float own = act_load(c + p.rank + e), other = act_load(c + p.rank + (e ^ 1));
+      act_store(d + i, e & 1 ? own * cs + other * sn : own * cs - other * sn);
+    } else {
+      act_store(d + i, 0.f);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_turn_kernel(const T* __restrict__ src, long long lds, int heads, int rot, const float* __restrict__ cos_t,
+                   const float* __restrict__ sin_t, int max_pos, const int* __restrict__ positions, T* __restrict__ q,
+                   long long ldq, int row_dim, int rot_off, DeviceStatus* st) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long r = blockIdx.x;
+  const int pos = checked_pos(positions[r], max_pos, blockIdx.x, st), half = rot / 2;
+  for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
+    const int h = i / half, e = i - h * half;
+    const float cs = cos_t[static_cast<long long>(pos) * half + e], sn = sin_t[static_cast<long long>(pos) * half + e];
+    const float u = act_load(src + r * lds + h * rot + 2 * e), v = act_load(src + r * lds + h * rot + 2 * e + 1);
+    T* d = q + r * ldq + static_cast<long long>(h) * row_dim + rot_off + 2 * e;
+    act_store(d, u * cs - v * sn);
+    act_store(d + 1, v * cs + u * sn);
+  }
+}
+
 // logits <- cap * tanh(logits / cap)
 __global__ void __launch_bounds__(256)
 softcap_kernel(float* __restrict__ logits, long long ldl, int vocab, float cap) {
@@ -202,7 +297,7 @@ struct LatentParams {
   int max_blocks, page_size, num_seqs;
   const int* row_seq;
   const int* row_pos;
-  int heads, dl;
+  int heads, dl, window;
   float scale;
   const T* gate;            // optional [rows, ldg]: output of head h is multiplied by sigmoid(gate[row][h])
   long long ldg;
@@ -235,7 +330,8 @@ latent_attention_kernel(const LatentParams<T> p) {
     o[j] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int t = warp; t < len; t += 4) {
+  const int first = p.window > 0 && len > p.window ? len - p.window : 0;
+  for (int t = first + warp; t < len; t += 4) {
     const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
     const long long slot = static_cast<long long>(page) * p.page_size + t % p.page_size;
     if (page < 0 || slot >= p.pool_rows) {
@@ -362,6 +458,41 @@ extern "C" int fb_latent_append(const void* src, long long lds, int rank, int ro
   return ok_launch();
 }
 
+template <typename T>
+static int launch_latent_prep(const FbLatentPrepArgs* a, cudaStream_t s) {
+  LatentPrepParams<T> p{static_cast<T*>(a->cq), static_cast<const T*>(a->ckv), a->ldp, a->rank_q, a->rank, a->rot, a->row_dim,
+                        a->rot_off, a->q_w, a->kv_w, a->cos_t, a->sin_t, a->max_pos, a->positions, a->write_slot,
+                        static_cast<T*>(a->pool), a->pool_rows, a->eps, static_cast<DeviceStatus*>(a->status)};
+  launch_pdl(latent_prep_kernel<T>, dim3(a->rows), dim3(256), 0, s, p);
+  return ok_launch();
+}
+
+extern "C" int fb_latent_prep(const FbLatentPrepArgs* a, void* stream) {
+  if (!a || !a->ckv || !a->kv_w || !a->write_slot || !a->pool || a->rows <= 0 || a->rank <= 0 || a->rot < 0 || a->rot % 2 ||
+      a->row_dim < a->rank || (a->cq && (a->rank_q <= 0 || !a->q_w)) || a->pool_rows <= 0 ||
+      (a->rot && (a->rot_off < a->rank || a->rot_off + a->rot > a->row_dim || !a->cos_t || !a->sin_t || !a->positions || a->max_pos <= 0)))
+    return FB_ERR_SHAPE;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  return a->fp32 ? launch_latent_prep<float>(a, s) : launch_latent_prep<__nv_bfloat16>(a, s);
+}
+
+extern "C" int fb_latent_turn(const void* src, long long lds, int heads, int rot, const float* cos_t, const float* sin_t, int max_pos,
+                              const int* positions, void* q, long long ldq, int row_dim, int rot_off, int rows, int fp32,
+                              void* status, void* stream) {
+  if (!src || !cos_t || !sin_t || !positions || !q || rows <= 0 || heads <= 0 || rot <= 0 || rot % 2 || max_pos <= 0 ||
+      rot_off < 0 || rot_off + rot > row_dim || ldq < static_cast<long long>(heads) * row_dim || lds < static_cast<long long>(heads) * rot)
+    return FB_ERR_SHAPE;
+  cudaStream_t s = static_cast<cudaStream_t>(stream);
+  DeviceStatus* st = static_cast<DeviceStatus*>(status);
+  if (fp32)
+    launch_pdl(latent_turn_kernel<float>, dim3(rows), dim3(256), 0, s, static_cast<const float*>(src), lds, heads, rot, cos_t, sin_t,
+               max_pos, positions, static_cast<float*>(q), ldq, row_dim, rot_off, st);
+  else
+    launch_pdl(latent_turn_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, static_cast<const __nv_bfloat16*>(src), lds, heads,
+               rot, cos_t, sin_t, max_pos, positions, static_cast<__nv_bfloat16*>(q), ldq, row_dim, rot_off, st);
+  return ok_launch();
+}
+
 extern "C" int fb_softcap(float* logits, long long ldl, int rows, int vocab, float cap, void* stream) {
   if (!logits || rows <= 0 || rows > 65535 || vocab <= 0 || !(cap > 0.f)) return FB_ERR_SHAPE;
   int bx = (vocab + 1023) / 1024;
@@ -383,7 +514,7 @@ static int launch_latent(const FbAttnArgs* a, cudaStream_t s) {
   p.kv = static_cast<const T*>(a->kv); p.pool_rows = a->pool_rows;
   p.block_table = a->block_table; p.max_blocks = a->max_blocks; p.page_size = a->page_size; p.num_seqs = a->num_seqs;
   p.row_seq = a->row_seq; p.row_pos = a->row_pos;
-  p.heads = a->heads; p.dl = a->kv_lora; p.scale = a->softmax_scale;
+  p.heads = a->heads; p.dl = a->kv_lora; p.window = a->window; p.scale = a->softmax_scale;
   p.gate = static_cast<const T*>(a->gate); p.ldg = a->ldg;
   p.out = static_cast<T*>(a->out); p.ldo = a->ldo;
   p.status = static_cast<DeviceStatus*>(a->status);
@@ -399,7 +530,7 @@ static int launch_latent(const FbAttnArgs* a, cudaStream_t s) {
 
 extern "C" int fb_latent_attention(const FbAttnArgs* a, int fp32, void* stream) {
   if (!a || !a->q || !a->kv || !a->out || !a->block_table || !a->row_seq || !a->row_pos) return FB_ERR_SHAPE;
-  if (a->rows <= 0 || a->heads <= 0 || a->heads > 65535 || a->kv_lora <= 0 || a->kv_lora > 1024 || a->rope_dim != 0 ||
+  if (a->rows <= 0 || a->heads <= 0 || a->heads > 65535 || a->kv_lora <= 0 || a->kv_lora > 1024 || a->rope_dim != 0 || a->window < 0 ||
       a->page_size <= 0 || a->max_blocks <= 0 || a->num_seqs <= 0 || a->pool_rows <= 0 || (a->gate && a->ldg < a->heads))
     return FB_ERR_SHAPE;
   cudaStream_t s = static_cast<cudaStream_t>(stream);

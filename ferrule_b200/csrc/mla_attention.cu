@@ -62,6 +62,7 @@ struct AttnParams {
                             // the dependency wait
   const __nv_bfloat16* gate;  // optional [rows, ldg]: head output times sigmoid(gate[row][head])
   long long ldg;
+  int window;               // > 0: a row sees its last `window` tokens only
   unsigned long long* trace;  // optional: CTA (0,0,0) writes globaltimer stamps of its milestones
 };
 
@@ -133,6 +134,9 @@ mla_attention_kernel(const AttnParams p) {
   const bool tracing = p.trace != nullptr && blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0 && tid == 0;
   int stamp = 0;
   if (tracing) p.trace[stamp++] = globaltimer_ns();      // entry (dependency wait passed)
+  // first token of a row's window; a tile starts at the 64-token boundary below its first row's
+  auto first_of = [&](int pos) { return p.window > 0 && pos >= p.window ? pos - p.window + 1 : 0; };
+  auto tile_base = [&](int pos) { return first_of(pos) / kKvTile * kKvTile; };
 
   if (tid == 0) {
     mbar_init(bar, kKvTile);
@@ -149,8 +153,8 @@ mla_attention_kernel(const AttnParams p) {
     const int seq0 = p.row_seq[qrow0];
     const int pos0 = p.row_pos[qrow0];
     if (seq0 >= 0 && seq0 < p.num_seqs && tid < kKvTile) {
-      const int tok = blockIdx.y * p.split_tokens + tid;
-      const int lim = min(min(pos0, p.max_blocks * p.page_size), (blockIdx.y + 1) * p.split_tokens);
+      const int base0 = tile_base(pos0), tok = base0 + blockIdx.y * p.split_tokens + tid;
+      const int lim = min(min(pos0, p.max_blocks * p.page_size), base0 + (blockIdx.y + 1) * p.split_tokens);
       if (tok < lim) {                     // strictly below the row's own position: written by an earlier step
         const int page = p.block_table[static_cast<long long>(seq0) * p.max_blocks + tok / p.page_size];
         const long long slot = static_cast<long long>(page) * p.page_size + tok % p.page_size;
@@ -200,11 +204,16 @@ mla_attention_kernel(const AttnParams p) {
 
   if (tracing) p.trace[14] = globaltimer_ns() + (kv_len_max == -12345);
   // per-thread row limits (rows g and g+8 of the tile)
-  int kvlen_lo = 0, kvlen_hi = 0;
+  int kvlen_lo = 0, kvlen_hi = 0, kvfirst_lo = 0, kvfirst_hi = 0, base = 0;
   {
     const int qr_lo = qrow0 + g / Hb, qr_hi = qrow0 + (g + 8) / Hb;
     if (seq_ok && qr_lo < p.rows && g / Hb < G) kvlen_lo = by_selection ? p.sel_width : p.row_pos[qr_lo] + 1;
     if (seq_ok && qr_hi < p.rows && (g + 8) / Hb < G) kvlen_hi = by_selection ? p.sel_width : p.row_pos[qr_hi] + 1;
+    if (p.window > 0 && !by_selection) {
+      kvfirst_lo = first_of(kvlen_lo - 1);
+      kvfirst_hi = first_of(kvlen_hi - 1);
+      base = tile_base(p.row_pos[qrow0]);                // rows of a tile are in the order of their positions
+    }
   }
   if (tracing) p.trace[15] = globaltimer_ns() + (kvlen_lo + kvlen_hi == -12345);
 #pragma unroll
@@ -216,7 +225,7 @@ mla_attention_kernel(const AttnParams p) {
   __syncthreads();
   if (tracing) p.trace[stamp++] = globaltimer_ns();      // query tile staged
 
-  const int kv_begin = split * p.split_tokens;
+  const int kv_begin = base + split * p.split_tokens;
   const int kv_end = min(kv_len_max, kv_begin + p.split_tokens);
 
   float o_acc[kNT][4];
@@ -297,10 +306,10 @@ mla_attention_kernel(const AttnParams p) {
       // an explicit selection masks its -1 entries (their rows were zero-filled above)
       const bool v0 = !by_selection || (tok0 < p.sel_width && sel[tok0] >= 0);
       const bool v1 = !by_selection || (tok1 < p.sel_width && sel[tok1] >= 0);
-      s0[j] = (v0 && tok0 < kvlen_lo) ? s0[j] * p.scale_log2 : -INFINITY;
-      s0[2 + j] = (v0 && tok0 < kvlen_hi) ? s0[2 + j] * p.scale_log2 : -INFINITY;
-      s1[j] = (v1 && tok1 < kvlen_lo) ? s1[j] * p.scale_log2 : -INFINITY;
-      s1[2 + j] = (v1 && tok1 < kvlen_hi) ? s1[2 + j] * p.scale_log2 : -INFINITY;
+      s0[j] = (v0 && tok0 < kvlen_lo && tok0 >= kvfirst_lo) ? s0[j] * p.scale_log2 : -INFINITY;
+      s0[2 + j] = (v0 && tok0 < kvlen_hi && tok0 >= kvfirst_hi) ? s0[2 + j] * p.scale_log2 : -INFINITY;
+      s1[j] = (v1 && tok1 < kvlen_lo && tok1 >= kvfirst_lo) ? s1[j] * p.scale_log2 : -INFINITY;
+      s1[2 + j] = (v1 && tok1 < kvlen_hi && tok1 >= kvfirst_hi) ? s1[2 + j] * p.scale_log2 : -INFINITY;
       tmax_lo = fmaxf(tmax_lo, fmaxf(s0[j], s1[j]));
       tmax_hi = fmaxf(tmax_hi, fmaxf(s0[2 + j], s1[2 + j]));
     }
@@ -709,6 +718,8 @@ extern "C" int fb_mla_attention(const FbAttnArgs* a, void* stream_) {
   p.sel_width = a->sel_width;
   p.status = static_cast<DeviceStatus*>(a->status);
   p.trace = static_cast<unsigned long long*>(a->trace);
+  if (a->window < 0 || (a->window > 0 && a->selection)) return FB_ERR_SHAPE;
+  p.window = a->window;
   p.gate = static_cast<const __nv_bfloat16*>(a->gate);
   p.ldg = a->ldg;
   p.prefetch_old = (a->decode_only && a->group_rows == 1 && a->selection == nullptr) ? 1 : 0;

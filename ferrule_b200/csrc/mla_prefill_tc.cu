@@ -69,6 +69,7 @@ struct TcParams {
   int page_size;
   int box_rows;              // min(page_size, 64)
   float scale_log2;
+  int window;                // > 0: a row sees its last `window` tokens only
   const __nv_bfloat16* gate; // optional [rows, ldg]: head output times sigmoid(gate[row][head])
   long long ldg;
 };
@@ -105,7 +106,13 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     return;
   }
   const int kv_len = min(pos0 + nrows, p.max_blocks * p.page_size);     // tokens 0 .. kv_len-1 are read
-  const int n_kv_tiles = (kv_len + kTcKv - 1) / kTcKv;
+  auto first_of = [&](int pos) { return p.window > 0 && pos >= p.window ? pos - p.window + 1 : 0; };
+  const int j0 = first_of(pos0) / kTcKv;                                // first tile with a token the first row sees
+  const int n_kv_tiles = (kv_len + kTcKv - 1) / kTcKv - j0;
+  if (n_kv_tiles <= 0) {
+    if (tid == 0) report_status(p.status, kStatusBadIndex, 0xA02, blockIdx.x, pos0);
+    return;
+  }
 
   if (tid == 0) {
     mbar_init(q_full, 1);
@@ -148,7 +155,7 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int j = 0; j < n_kv_tiles && ok; ++j) {
         int rowc[8];
         for (int s = 0; s < subs; ++s) {
-          const int t0 = j * kTcKv + s * p.box_rows;
+          const int t0 = (j0 + j) * kTcKv + s * p.box_rows;
           int rc = static_cast<int>(p.pool_rows);              // out of range: the copy fills zeros
           if (t0 < kv_len) {
             const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t0 / p.page_size];
@@ -240,7 +247,7 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
     const int r = quarter * 32 + lane;
     const int g = r / H, head = r - g * H;
     const bool valid = g < nrows;
-    const int kvlen_row = valid ? min(pos0 + g + 1, kv_len) : 0;
+    const int kvlen_row = valid ? min(pos0 + g + 1, kv_len) : 0, kvfirst_row = first_of(pos0 + g);
     const uint32_t lane_base = tmem + (static_cast<uint32_t>(quarter * 32) << 16);
     float m_ref = -INFINITY, l_sum = 0.f;
     bool ok = true;
@@ -254,13 +261,14 @@ mla_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int c = 0; c < 4; ++c) tmem_ld16(lane_base + kColS + (j & 1) * kTcKv + c * 16, sv[c]);
       tmem_ld_wait();
       float mx = -INFINITY;
-      const int tok0 = j * kTcKv;
+      const int tok0 = (j0 + j) * kTcKv;
 #pragma unroll
       for (int c = 0; c < 4; ++c)
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           float x = __uint_as_float(sv[c][i]) * p.scale_log2;
-          x = (tok0 + c * 16 + i < kvlen_row) ? x : -INFINITY;
+          const int t = tok0 + c * 16 + i;
+          x = (t < kvlen_row && t >= kvfirst_row) ? x : -INFINITY;
           sv[c][i] = __float_as_uint(x);
           mx = fmaxf(mx, x);
         }
@@ -418,6 +426,8 @@ extern "C" int fb_mla_prefill_tc(const FbPrefillAttnArgs* a, void* stream_) {
   p.box_rows = box_rows;
   p.scale_log2 = a->softmax_scale * 1.4426950408889634f;
   if (a->gate && a->ldg < a->heads) return FB_ERR_SHAPE;
+  if (a->window < 0) return FB_ERR_SHAPE;
+  p.window = a->window;
   p.gate = static_cast<const __nv_bfloat16*>(a->gate);
   p.ldg = a->ldg;
   return a->rope_dim ? launch_tc<9>(mq, mkv, p, stream) : launch_tc<8>(mq, mkv, p, stream);

@@ -36,19 +36,24 @@ A layer that runs several times has a cache plane and a state per run.
   captured in a CUDA graph.  With fp32 weights the same pipeline runs in full 32 bits.
 
 Kernels of a latent layer: input projection (one GEMM for q, latent, gates) -> latent append -> W_uk absorption ->
-attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o.  Of an attention layer: input projection (q, k,
+attention over the latent pool (head gate in its epilogue) -> W_uv -> W_o; with a query latent the append also normalises it
+and W_uq follows, with rotated parts their queries join behind the absorption.  Of an attention layer: input projection (q, k,
 v) -> norms, rotation, value mixing and cache append in one launch -> attention -> W_o.  Of a window layer: input projection
 (q, k, v, gate) -> norms, mixing of the queries across heads and cache append in one launch -> attention (distance bias,
-difference of the two maps, gate inside) -> W_o.  Of a delta layer: input projection
--> second low-rank halves -> delta rule -> W_o.  Of a selective-scan layer: input projection -> convolution -> W_x -> W_dt
--> scan (step sizes, skip and output gate inside) -> W_o.
+difference of the two maps, soft cap, gate inside) -> W_o; with pooled blocks their mean rows are written in front of the
+attention (in decode steps by the append), and outputs whose softmax weights are mixed across heads are mixed behind the prompt
+attention (in decode steps inside).  Of a delta layer: input projection -> second low-rank halves -> delta rule -> W_o.  Of a selective-scan layer: input projection -> convolution -> W_x -> W_dt
+-> scan (step sizes, skip and output gate inside) -> W_o.  Of a head-decay scan: input projection -> convolution -> scan (step
+sizes, skip and output gate inside) -> group norm -> W_o.
 
 In a parallel gated block the feed-forward branch reads the same h and runs on a second stream beside the mixer: router
 (+ row reservation) -> grouped SwiGLU GEMM -> grouped scatter GEMM.  One kernel joins both branches: gated residual
 additions, expert reduction, next layer's norm.  In an output-norm block one kernel after each sublayer normalises its
 output, adds it to the stream and leaves the rows the next GEMM reads; in decode steps it also applies the next mixer's
 input convolution, whose earlier inputs are in the state pool then.  In a sandwich block the same kernel takes the norm of the
-sublayer's output, the addition, the embedding of a new pass and the next sublayer's input norm.
+sublayer's output, the addition, the embedding of a new pass and the next sublayer's input norm.  In a pre-norm block it adds
+the output (a token's expert rows and its gated shared expert), takes the next norm and the token shift; when rows have their
+predecessors in the same batch it writes the stream to a second buffer.
 """
 from __future__ import annotations
 
@@ -470,9 +475,11 @@ class LayeredWorkspace:
         act = dict(dtype=dt, device=device)
         f32 = dict(dtype=torch.float32, device=device)
         i32 = dict(dtype=torch.int32, device=device)
-        R, Wp, DL = max_rows, cfg.width_pad, cfg.kv_row_dim
+        R, Wp = max_rows, cfg.width_pad
         self.max_rows, self.max_logit_rows = R, max_logit_rows
         self.x = torch.zeros(R, Wp, **f32)
+        if cfg.token_shift:
+            self.x_next = torch.zeros(R, Wp, **f32)
         self.h = torch.zeros(R, Wp, **act)
         self.proj = torch.zeros(R * max(l.mixer.w_in.shape[0] for l in w.layers), **act)
         self.mix_in = torch.zeros(R * max(l.mixer.w_o.shape[1] for l in w.layers), **act)
@@ -480,9 +487,10 @@ class LayeredWorkspace:
         latent, delta, mamba = ([cfg.layers[i].mixer for i in ids] for ids in (cfg.latent_layers, cfg.delta_layers,
                                                                                cfg.mamba_layers))
         if latent:
-            n = max(m.heads for m in latent) * DL
+            n = max(m.heads * m.row_dim for m in latent)
             self.q_lat = torch.zeros(R * n, **act)
             self.o_lat = torch.zeros(R * n, **act)
+            self.uq = torch.zeros(R * max((l.mixer.w_uq.shape[0] for l in w.layers if l.mixer.w_uq is not None), default=0), **act)
         if delta:
             low = [l.mixer.w_ag for l in w.layers if l.mixer.w_ag is not None]
             self.ag = torch.zeros(R * max((t.shape[0] for t in low), default=0), **f32)
@@ -492,9 +500,15 @@ class LayeredWorkspace:
             self.conv_x = torch.zeros(R * n, **act)
             self.dt = torch.zeros(R * n, **f32)
             self.low = torch.zeros(R * max(l.mixer.w_x.shape[0] for l in w.layers if l.mixer.w_x is not None), **act)
+        head_scan = [cfg.layers[i].mixer for i in cfg.mamba2_layers]
+        if head_scan:
+            self.conv_x = torch.zeros(R * max([m.channels for m in head_scan] + [m.inner_pad for m in mamba]), **act)
         window = [cfg.layers[i].mixer for i in cfg.window_layers]
         if window:
-            self.q_rows = torch.zeros(R * max(m.heads * m.maps * m.key_width for m in window), **act)
+            # (queries that are neither mixed nor split into maps stay in the projection's rows)
+            self.q_rows = torch.zeros(R * max((m.heads * m.maps * m.key_width for m in window if m.shared_keys or m.maps > 1),
+                                              default=0), **act)
+            self.o_all = torch.zeros(R * max((m.heads * m.value_width for m in window if m.shared_values), default=0), **act)
         if any(l.w_up is not None for l in w.layers):
             self.ff = torch.zeros(R * max(l.w_down.shape[1] for l in w.layers if l.w_up is not None), **act)
             if cfg.block == OUTPUT_NORM:
@@ -505,7 +519,12 @@ class LayeredWorkspace:
         self.static_rows = (16, 32, 64)
         if moes:
             kmax, emax = max(s.top for _, s in moes), max(s.experts for _, s in moes)
-            self.router_logits = torch.zeros(R * emax, **f32)
+            self.router_logits = torch.zeros(R * (emax + 1), **f32)
+            sff = [l.s_w2.shape[1] for l in w.layers if l.s_w2 is not None]
+            if sff:
+                self.shared_mid = torch.zeros(R * max(sff), **act)
+                self.shared_out = torch.zeros(R, Wp, **act)
+                self.shared_gate = torch.zeros(R, 1, **f32)
             self.topk_idx = torch.zeros(R * kmax, **i32)
             self.topk_w = torch.zeros(R * kmax, **f32)
             xrows = max(R * kmax, emax * self.static_rows[-1])
@@ -545,19 +564,18 @@ class LayeredCuda:
         self.decode_rows = decode_rows
         self.attn_splits = attn_splits
         self.max_seq_len = max_seq_len
-        self.split_tokens = max(64, pad_to((max_seq_len + attn_splits - 1) // attn_splits, 64))
         self.ws = LayeredWorkspace(weights, max_rows, max_logit_rows, self.device)
         self.cache_index = {r: i for i, r in enumerate(self.cfg.cache_runs)}
+        self.gqa_table = max((KL.gqa_tc_group(self.cfg.layers[i].mixer, weights.embed.dtype, pool.page_size)
+                              for i in self.cfg.attention_layers + self.cfg.window_layers), default=0)
         # cosines and sines of every rotation in use, computed in double
         self.rotation: Dict[tuple, tuple] = {}
-        for i in self.cfg.attention_layers:
-            m = self.cfg.layers[i].mixer
-            if (m.rot_base, m.rot_dims) not in self.rotation:
+        for l in self.cfg.layers:
+            base, dims = self._rotation_key(l.mixer)
+            if dims and (base, dims) not in self.rotation:
                 a = (torch.arange(min(max_seq_len, self.cfg.max_position), dtype=torch.float64)[:, None]
-                     * rotation_frequencies(m.rot_base, m.rot_dims))
-                self.rotation[m.rot_base, m.rot_dims] = tuple(f(a).float().to(self.device) for f in (torch.cos, torch.sin))
-        # the tensor-core attention kernels take latents up to 512 features
-        self.mma_attention = not self.fp32 and self.cfg.kv_row_dim <= 512
+                     * rotation_frequencies(base, dims))
+                self.rotation[base, dims] = tuple(f(a).float().to(self.device) for f in (torch.cos, torch.sin))
         self.static_moe = not self.fp32 and self.cfg.width_pad <= 8192
         self.side_stream = torch.cuda.Stream(device=self.device)      # the feed-forward runs beside the mixer
         self.launches = 0
@@ -569,10 +587,17 @@ class LayeredCuda:
                 raise ValueError("delta mixers wider than 256 key channels per head are not supported")
             if isinstance(m, MambaMixer) and m.state > 128:
                 raise ValueError("selective scans with more than 128 states per channel are not supported")
+            if isinstance(m, Mamba2Mixer) and (m.state > 256 or m.vdim > 1024):
+                raise ValueError("head-decay scans with more than 256 states or 1024 columns per head are not supported")
             if isinstance(m, (AttentionMixer, WindowMixer)) and max(m.dim, m.vdim) > 512:
                 raise ValueError("attention heads wider than 512 are not supported")
             if isinstance(f, MoeSpec) and (f.experts > 256 or f.top > 32 or f.groups > 32):
                 raise ValueError("the router takes at most 256 experts, top 32, 32 groups")
+
+    @staticmethod
+    def _rotation_key(m) -> tuple:
+        dims = m.rot_dim if isinstance(m, LatentMixer) else getattr(m, "rot_dims", 0)
+        return (m.rot_base, dims) if dims else (0.0, 0)
 
     @staticmethod
     def _view(buf: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
@@ -582,33 +607,50 @@ class LayeredCuda:
     def _latent(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
         mx, m = lw.mixer, lw.spec.mixer
-        DL, dp, vp = cfg.kv_row_dim, pad_to(m.dim, 8), pad_to(m.vdim, 8)
+        DL, dp, vp = m.row_dim, pad_to(m.dim, 8), pad_to(m.vdim, 8)
         pool = self.pool.layer(self.cache_index[layer])
-        KL.latent_append(proj[:, mx.off["dkv"]:], m.kv_rank, mx.kv_norm, cfg.norm_eps, b.write_slot[:T], pool)
-        q = proj[:, mx.off["q"]:mx.off["q"] + m.heads * dp]
+        rotation = self.rotation.get(self._rotation_key(m))
+        q_src, q_off = proj, mx.off
+        if m.q_rank or m.rot_dim:
+            KL.latent_prep(proj, mx.off, m, mx, rotation, b.positions[:T], b.write_slot[:T], pool, cfg.norm_eps)
+        else:
+            KL.latent_append(proj[:, mx.off["dkv"]:], m.kv_rank, mx.kv_norm, cfg.norm_eps, b.write_slot[:T], pool)
+        if m.q_rank:
+            q_src, q_off = self._view(ws.uq, T, mx.w_uq.shape[0]), mx.off_uq
+            K.gemm(proj[:, mx.off["dq"]:mx.off["dq"] + mx.w_uq.shape[1]], mx.w_uq, out=q_src)
+        q = q_src[:, q_off["q"]:q_off["q"] + m.heads * dp]
         q_lat = self._view(ws.q_lat, T, m.heads * DL)
         K.gemm(q, mx.w_uk_t, out=q_lat, x_group_koff=dp, out_group_coff=DL, k=dp)
-        o_lat = self._view(ws.o_lat, T, m.heads * DL)
-        q3, o3 = q_lat.view(T, m.heads, DL), o_lat.view(T, m.heads, DL)
+        q3 = q_lat.view(T, m.heads, DL)
+        if m.rot_dim:
+            KL.latent_turn(q_src[:, q_off["qr"]:q_off["qr"] + m.heads * m.rot_dim], m, rotation, b.positions[:T], q3)
         gate = proj[:, mx.off["g"]:]
-        if not self.mma_attention:
+        # the tensor-core attention kernels take values up to 512 features
+        mma = not self.fp32 and m.value_dim <= 512
+        D = m.value_dim if mma else DL
+        o_lat = self._view(ws.o_lat, T, m.heads * D)
+        o3 = o_lat.view(T, m.heads, D)
+        if not mma:
             KL.latent_attention(q3, pool, b.block_table, b.row_seq[:T], b.row_pos[:T], self.pool.page_size, m.scale, o3,
-                                gate=gate)
+                                gate=gate, window=m.window)
         else:
-            ranges = [(0, T)]
-            if b.n_tc_tiles:
+            ranges, rope = [(0, T)], DL - D
+            tiles = b.tc_tables.get(KL.latent_tc_group(m, q3.dtype, self.pool.page_size)) if b.n_tc_tiles else None
+            if tiles:
                 # sequences with many rows: 128-row tiles on tcgen05; the other rows keep the row-tile kernel
-                K.mla_prefill_tc(q3, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, self.pool.page_size, DL, 0, m.scale,
-                                 o3, gate=gate)
+                K.mla_prefill_tc(q3, pool, b.block_table, *tiles, self.pool.page_size, D, rope, m.scale, o3, gate=gate,
+                                 window=m.window)
                 ranges = b.rest_ranges
+            span = min(self.max_seq_len, m.window + 64) if m.window else self.max_seq_len
+            split_tokens = max(64, pad_to((span + self.attn_splits - 1) // self.attn_splits, 64))
             for r0, r1 in ranges:
                 split = self.attn_splits > 1 and r1 - r0 <= 4 * self.decode_rows
-                K.mla_attention(q3[r0:r1], pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], self.pool.page_size, DL,
-                                0, m.scale, o3[r0:r1], splits=self.attn_splits if split else 1,
-                                split_tokens=self.split_tokens if split else (1 << 30) // 64 * 64,
-                                decode_only=b.decode_only, gate=gate[r0:r1])
+                K.mla_attention(q3[r0:r1], pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], self.pool.page_size, D,
+                                rope, m.scale, o3[r0:r1], splits=self.attn_splits if split else 1,
+                                split_tokens=split_tokens if split else (1 << 29), decode_only=b.decode_only,
+                                gate=gate[r0:r1], window=m.window)
         out = self._view(ws.mix_in, T, m.heads * vp)
-        K.gemm(o_lat, mx.w_uv, out=out, x_group_koff=DL, out_group_coff=vp)
+        K.gemm(o_lat, mx.w_uv, out=out, x_group_koff=D, out_group_coff=vp, k=D)
         return out
 
     def _delta(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
@@ -639,31 +681,53 @@ class LayeredCuda:
         return self._attend(q, m, pool, b, T)
 
     def _attend(self, q: torch.Tensor, m, pool: torch.Tensor, b: DeviceBatch, T: int, gate: Optional[torch.Tensor] = None,
-                **form) -> torch.Tensor:
-        """Attention of query rows over a layer's pool: prompt tiles on tcgen05, the other rows in the decode kernels."""
+                talk: Optional[torch.Tensor] = None, **form) -> torch.Tensor:
+        """Attention of query rows over a layer's pool: prompt tiles on tcgen05, the other rows in the decode kernels.  With
+        `talk` the rows of both get mixed softmax weights."""
         KL = self.KL
         out = self._view(self.ws.mix_in, T, m.heads * m.vdim_pad)
         page = self.pool.page_size
         ranges = [(0, T)]
+        few = KL.gqa_decode_supported(m, q.dtype, page)
+        o = out if talk is None else self._view(self.ws.o_all, T, m.heads * m.value_width)
         if b.n_tc_tiles and KL.gqa_tc_group(m, q.dtype, page):
-            KL.gqa_prefill_tc(q, m, pool, b.block_table, b.tc_tiles, b.n_tc_tiles, b.tc_positions, page, out, gate=gate, **form)
+            KL.gqa_prefill_tc(q, m, pool, b.block_table, *b.tc_tables[self.gqa_table], 128 // self.gqa_table, page, o, gate=gate,
+                              **form)
             ranges = b.rest_ranges
-        for r0, r1 in ranges:
-            rows = dict(gate=None if gate is None else gate[r0:r1], **form)
-            at = (q[r0:r1], m, pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], page, out[r0:r1])
-            if KL.gqa_decode_supported(m, q.dtype, page):
-                KL.gqa_decode(*at, splits=KL.gqa_decode_splits(r1 - r0, m, self.max_seq_len), decode_only=b.decode_only, **rows)
-            else:
-                KL.gqa_attention(*at, **rows)
+        at = lambda r0, r1, o: (q[r0:r1], m, pool, b.block_table, b.row_seq[r0:r1], b.row_pos[r0:r1], page, o[r0:r1])
+        rows = lambda r0, r1: dict(gate=None if gate is None else gate[r0:r1], **form)
+        if not few:
+            for r0, r1 in ranges:
+                KL.gqa_attention(*at(r0, r1, o), **rows(r0, r1))
+        if talk is not None and (not few or ranges != [(0, T)]):
+            KL.value_mix(o, talk, m, out)
+        if few:
+            mixed = {} if talk is None else dict(talk=talk)
+            for r0, r1 in ranges:
+                KL.gqa_decode(*at(r0, r1, out), splits=KL.gqa_decode_splits(r1 - r0, m, self.max_seq_len),
+                              decode_only=b.decode_only, **rows(r0, r1), **mixed)
         return out
 
     def _window(self, run: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
-        mx, m = lw.mixer, lw.spec.mixer
+        KL, mx, m = self.KL, lw.mixer, lw.spec.mixer
         pool = self.pool.layer(self.cache_index[run])
-        q = self._view(self.ws.q_rows, T, m.heads * m.maps * m.key_width)
-        self.KL.head_prep(proj, mx.off, m, mx, b.write_slot[:T], pool, self.cfg.norm_eps, q)
+        form: dict = {}
+        blocks = None
+        if m.pool:
+            form["mean"] = (self.states.pooled[run], self.states.buffers, b.state_out)
+            blocks = (form["mean"], b.positions[:T], b.row_seq[:T], b.block_table, self.pool.page_size)
+        if m.shared_keys or m.maps > 1:
+            q = self._view(self.ws.q_rows, T, m.heads * m.maps * m.key_width)
+        else:
+            q = proj[:, mx.off["q"]:mx.off["q"] + m.heads * m.dim_pad]
+        single = b.n_seqs == T
+        KL.head_prep(proj, mx.off, m, mx, b.write_slot[:T], pool, self.cfg.norm_eps, q, self.rotation.get(self._rotation_key(m)),
+                     b.positions[:T], blocks if single else None)
+        if blocks is not None and not single:
+            KL.pool_blocks(m, pool, *blocks)
         gate = proj[:, mx.off["g"]:] if m.gate else None
-        return self._attend(q, m, pool, b, T, slopes=mx.slopes, gate=gate, diff_lambda=mx.diff_lambda, eps=self.cfg.norm_eps)
+        return self._attend(q, m, pool, b, T, slopes=mx.slopes, gate=gate, talk=mx.talk, diff_lambda=mx.diff_lambda,
+                            eps=self.cfg.norm_eps, **form)
 
     def _mamba(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         K, KL, ws = self.K, self.KL, self.ws
@@ -682,14 +746,31 @@ class LayeredCuda:
         return KL.selective_scan(x, proj[:, mx.off["z"]:mx.off["z"] + Ip], low, mx.off_b, mx.off_c, dt, mx,
                                  self.states.state[layer], *seqs, out)
 
+    def _mamba2(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
+        KL, ws = self.KL, self.ws
+        mx, m = lw.mixer, lw.spec.mixer
+        seqs = (b.seq_start, b.state_in, b.state_out, b.n_seqs)
+        xbc = self._view(ws.conv_x, T, m.channels)
+        KL.short_conv(proj[:, :m.channels], mx.conv, self.states.tail[layer], xbc, b.row_seq[:T], *seqs, bias=mx.conv_b, silu=True)
+        out = self._view(ws.mix_in, T, m.inner_pad)
+        KL.head_scan(xbc, proj, mx.off, m, mx, self.states.state[layer], *seqs, out)
+        return KL.group_norm_rows(out, mx.o_norm, out, m.inner, m.norm_groups, self.cfg.norm_eps)
+
     def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:
         fn = {LatentMixer: self._latent, AttentionMixer: self._attention, WindowMixer: self._window,
-              DeltaMixer: self._delta, MambaMixer: self._mamba}[type(lw.spec.mixer)]
+              DeltaMixer: self._delta, MambaMixer: self._mamba, Mamba2Mixer: self._mamba2}[type(lw.spec.mixer)]
         return fn(layer, lw, proj, b, T)
 
     # -- feed-forward ------------------------------------------------------------------------
-    def _moe(self, layer: int, lw: LayerImage, h: torch.Tensor, T: int) -> torch.Tensor:
-        """Routed experts -> [T, top, width_pad] weighted expert rows."""
+    def _shared_expert(self, lw: LayerImage, h: torch.Tensor, T: int) -> torch.Tensor:
+        K, ws, s = self.K, self.ws, lw.spec.mlp
+        mid = self._view(ws.shared_mid, T, lw.s_w2.shape[1])
+        K.gemm(h, lw.s_w13, out=mid, epilogue=K.EPI_SWIGLU, act_limit=s.shared_limit, act_alpha=s.alpha, act_shift=s.shift)
+        return K.gemm(mid, lw.s_w2, out=ws.shared_out[:T])
+
+    def _moe(self, layer: int, lw: LayerImage, h: torch.Tensor, T: int, gate: Optional[list] = None) -> torch.Tensor:
+        """Routed experts -> [T, top, width_pad] weighted expert rows.  With a shared expert the pre-activation of its gate is
+        put into `gate`: fp32 [T, 1]."""
         K, ws, s = self.K, self.ws, lw.spec.mlp
         k, E, Wp = s.top, s.experts, self.cfg.width_pad
         fp = lw.e_w2.shape[2]
@@ -698,15 +779,21 @@ class LayeredCuda:
         static = next((nt for nt in ws.static_rows if T <= nt), 0) if self.static_moe else 0
         if static:
             plan = ws.static_plans[layer, static]
+            extra = ws.shared_gate[:T] if s.shared_ff else None
             K.router_append(h, lw.router_w, k, SCORE_SOFTMAX, plan, 0, E, idx, wts, ws.xg, n_groups=s.groups,
-                            topk_groups=s.keep, group_top=1, dst_slots=k)
+                            topk_groups=s.keep, group_top=1, dst_slots=k, normalize=s.renormalize, logit_bias=lw.router_b,
+                            extra=extra)
+            if extra is not None:
+                gate.append(extra)
             rows = plan.cap_rows
             scatter_plan = plan
         else:
-            logits = self._view(ws.router_logits, T, E)
-            K.gemm(h, lw.router_w, out=logits, ntok=32 if (T >= 1024 and not self.fp32) else None)
-            K.router_topk(logits, k, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep, group_top=1, out_idx=idx,
-                          out_w=wts)
+            products = self._view(ws.router_logits, T, lw.router_w.shape[0])
+            K.gemm(h, lw.router_w, out=products, ntok=32 if (T >= 1024 and not self.fp32) else None)
+            if s.shared_ff:
+                gate.append(products[:, E:])
+            K.router_topk(products[:, :E], k, SCORE_SOFTMAX, n_groups=s.groups, topk_groups=s.keep, group_top=1, out_idx=idx,
+                          out_w=wts, normalize=s.renormalize, logit_bias=lw.router_b)
             ntok = _pow2_at_least(2 * T * k / E, 16, 128)
             plan = ws.plans[E, k, ntok]
             K.moe_plan(idx, wts, plan, 0, E, dst_slots=k)
@@ -720,7 +807,8 @@ class LayeredCuda:
                 # prefill-sized expert loads: the scatter GEMM keeps one accumulator and takes 256-row tiles
                 scatter_plan = ws.plans[E, k, 256] = K.moe_retile(plan, 256, ws.plans[E, k, 256])
         hmid = self._view(ws.hmid, rows, fp)
-        K.gemm(ws.xg[:rows], lw.e_w13, out=hmid, epilogue=K.EPI_SWIGLU, plan=plan)
+        K.gemm(ws.xg[:rows], lw.e_w13, out=hmid, epilogue=K.EPI_SWIGLU, plan=plan, act_limit=s.limit, act_alpha=s.alpha,
+               act_shift=s.shift)
         K.gemm(hmid, lw.e_w2, out=route_out, epilogue=K.EPI_SCATTER, plan=scatter_plan, scatter_rows=T * k)
         return route_out.view(T, k, Wp)
 
@@ -731,7 +819,7 @@ class LayeredCuda:
         if prof is not None:
             prof.mark(i, "proj")
         proj = self._view(ws.proj, T, mx.w_in.shape[0])
-        K.gemm(h, mx.w_in, out=proj)
+        K.gemm(h, mx.w_in, out=proj, bias=mx.b_in)
         if prof is not None:
             prof.mark(i, "mixer")
         a = self._mixer(i, lw, proj, b, T)
@@ -744,7 +832,7 @@ class LayeredCuda:
         if self.tap is not None and self.tap.wants(i, "layer_out"):
             self.tap.write(i, "layer_out", x)
 
-    def _gated_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+    def _gated_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
         KL, ws, cfg = self.KL, self.ws, self.cfg
         layers = self.w.layers
         if self.static_moe and T <= ws.static_rows[-1] and ws.static_plans:
@@ -769,8 +857,9 @@ class LayeredCuda:
                 ffn=ffn, topk=lw.spec.mlp.top if ffn is not None else 0,
                 gate2=proj[:, mx.off["rg2"]:] if ffn is not None else None, bias2=lw.rg2_b)
             self._tapped(i, x)
+        return x
 
-    def _output_norm_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+    def _output_norm_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
         K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
         layers, eps = self.w.layers, cfg.norm_eps
         single = b.n_seqs == T          # one row per sequence: a row's earlier convolution inputs are all in the state
@@ -799,8 +888,9 @@ class LayeredCuda:
                 K.gemm(ff, lw.w_down, out=ws.mix[:T])
                 KL.add_normed(x, ws.mix[:T], lw.norm2, cfg.width, eps, canon=fused(i + 1))
             self._tapped(i, x)
+        return x
 
-    def _sandwich_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> None:
+    def _sandwich_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
         K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
         runs, starts = cfg.runs, set(cfg.pass_starts)
         grouped = dict(dim=cfg.width, eps=cfg.norm_eps, groups=cfg.norm_groups)
@@ -835,16 +925,68 @@ class LayeredCuda:
             K.gemm(h, lw.w_up, out=ff, epilogue=K.EPI_GEGLU)
             K.gemm(ff, lw.w_down, out=ws.mix[:T])
             close(r, lw.norm2b)
+        return x
+
+    def _pre_norm_blocks(self, b: DeviceBatch, T: int, x: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+        """Returns the buffer that holds the final stream."""
+        K, KL, ws, cfg = self.K, self.KL, self.ws, self.cfg
+        layers = self.w.layers
+        row = dict(dim=cfg.width, eps=cfg.norm_eps, like=h)
+        seqs = (b.row_seq[:T], b.seq_start, b.state_in, b.state_out, b.n_seqs)
+        swap = cfg.token_shift and b.n_seqs != T         # a shift that sees rows of this batch leaves the old stream alone
+        if self.static_moe and T <= ws.static_rows[-1] and ws.static_plans:
+            self.M.fill_(ws.route_cnt, 0)
+
+        def entry(i: int) -> dict:
+            """What layer i's mixer reads."""
+            if i >= len(layers):
+                return {}
+            lw = layers[i]
+            shift = {} if lw.shift is None else dict(shift=lw.shift, plane=self.states.shift[i], seqs=seqs)
+            return dict(norm=lw.norm1, act=h, **shift)
+
+        KL.pre_norm_step(None, x, ids=b.token_ids[:T], table=self.w.embed, scale=cfg.embed_scale, **entry(0), **row)
+        other = ws.x_next[:T] if swap else x
+        for i, lw in enumerate(layers):
+            self._mix(i, lw, h, b, T)
+            if self.prof is not None:
+                self.prof.mark(i, "tail")
+            left = dict(y=ws.mix[:T])
+            if lw.spec.mlp is not None:
+                KL.pre_norm_step(x, x, norm=lw.norm2, act=h, **left, **row)
+                if isinstance(lw.spec.mlp, MoeSpec):
+                    left = self._routed(i, lw, h, T)
+                else:
+                    ff = self._view(ws.ff, T, lw.w_up.shape[0])
+                    K.gemm(h, lw.w_up, out=ff, epilogue=K.EPI_GELU, bias=lw.up_b)
+                    K.gemm(ff, lw.w_down, out=ws.mix[:T], bias=lw.down_b)
+            KL.pre_norm_step(x, other, **left, **entry(i + 1), **row)
+            x, other = other, x
+            self._tapped(i, x)
+        return x
+
+    def _routed(self, i: int, lw: LayerImage, h: torch.Tensor, T: int) -> dict:
+        """Expert rows of a layer, with the shared expert computed beside them."""
+        s, gate = lw.spec.mlp, []
+        if not s.shared_ff:
+            return dict(ffn=self._moe(i, lw, h, T), topk=s.top)
+        main = torch.cuda.current_stream()
+        self.side_stream.wait_stream(main)
+        with torch.cuda.stream(self.side_stream):
+            shared = self._shared_expert(lw, h, T)
+        ffn = self._moe(i, lw, h, T, gate)
+        main.wait_stream(self.side_stream)
+        return dict(ffn=ffn, topk=s.top, shared=shared, shared_gate=gate[0])
 
     # -- whole model ---------------------------------------------------------------------
     def hidden_states(self, b: DeviceBatch, T: int) -> torch.Tensor:
-        """Runs the layers; `ws.x` holds the residual stream.  Returns the rows the head starts from: normalised ones
+        """Runs the layers.  Returns the rows the head starts from: normalised ones
         (`ws.h`) behind parallel gated blocks, the stream itself behind the other forms."""
         ws = self.ws
         x, h = ws.x[:T], ws.h[:T]
         gated = self.cfg.block == PARALLEL_GATED
-        {PARALLEL_GATED: self._gated_blocks, OUTPUT_NORM: self._output_norm_blocks,
-         SANDWICH_NORM: self._sandwich_blocks}[self.cfg.block](b, T, x, h)
+        x = {PARALLEL_GATED: self._gated_blocks, OUTPUT_NORM: self._output_norm_blocks, SANDWICH_NORM: self._sandwich_blocks,
+             PRE_NORM: self._pre_norm_blocks}[self.cfg.block](b, T, x, h)
         if self.prof is not None:
             self.prof.mark(len(self.cfg.runs), None)
         return h if gated else x
@@ -853,7 +995,9 @@ class LayeredCuda:
         """Logits and greedy tokens of `L` rows -> (next_id, next_val, logits), views of the workspace."""
         K, ws = self.K, self.ws
         hn = ws.hn_last[:L]
-        if self.cfg.block == OUTPUT_NORM:
+        if self.cfg.block == PRE_NORM:
+            self.KL.norm_rows(h, logit_rows[:L], self.w.final_norm[None], hn, self.cfg.width, self.cfg.norm_eps, rms=True)
+        elif self.cfg.block == OUTPUT_NORM:
             self.KL.norm_rows(h, logit_rows[:L], self.w.final_norm, hn, self.cfg.width, self.cfg.norm_eps)
         elif self.cfg.block == SANDWICH_NORM:
             self.KL.sandwich_rows(h, logit_rows[:L], self.w.final_norm, hn, self.cfg.width, self.cfg.norm_eps,

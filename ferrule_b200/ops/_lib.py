@@ -52,6 +52,7 @@ class GemmArgs(C.Structure):
         ("peer_wait_ns", C.c_ulonglong), ("status", C.c_void_p), ("trace", C.c_void_p),
         ("ar_payload_bf16", C.c_int),
         ("remap_rank", C.c_void_p), ("remap_row", C.c_void_p), ("mc_recv", C.c_void_p),
+        ("bias", C.c_void_p), ("act_alpha", C.c_float), ("act_shift", C.c_float),
     ]
 
 
@@ -68,7 +69,7 @@ class AttnArgs(C.Structure):
         ("softmax_scale", C.c_float), ("merge_ctr", C.c_void_p),
         ("selection", C.c_void_p), ("sel_width", C.c_int), ("trace", C.c_void_p),
         ("decode_only", C.c_int),
-        ("gate", C.c_void_p), ("ldg", C.c_longlong),
+        ("gate", C.c_void_p), ("ldg", C.c_longlong), ("window", C.c_int),
     ]
 
 
@@ -79,7 +80,7 @@ class PrefillAttnArgs(C.Structure):
         ("ldq", C.c_longlong), ("ldo", C.c_longlong), ("pool_rows", C.c_longlong),
         ("n_tiles", C.c_int), ("rows", C.c_int), ("heads", C.c_int), ("kv_lora", C.c_int), ("rope_dim", C.c_int),
         ("num_seqs", C.c_int), ("max_blocks", C.c_int), ("page_size", C.c_int), ("softmax_scale", C.c_float),
-        ("gate", C.c_void_p), ("ldg", C.c_longlong),
+        ("gate", C.c_void_p), ("ldg", C.c_longlong), ("window", C.c_int),
     ]
 
 
@@ -159,7 +160,9 @@ class GqaArgs(C.Structure):
         ("vdim", C.c_int), ("vdim_pad", C.c_int), ("fp32", C.c_int), ("maps", C.c_int), ("key_width", C.c_int),
         ("key_stride", C.c_int), ("v_offset", C.c_int), ("window", C.c_int), ("keep_first", C.c_int),
         ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ldg", C.c_longlong), ("diff_lambda", C.c_float),
-        ("diff_scale", C.c_float), ("status", C.c_void_p),
+        ("diff_scale", C.c_float), ("value_width", C.c_int), ("value_stride", C.c_int), ("softcap", C.c_float),
+        ("pooled", C.c_void_p), ("pooled_rows", C.c_longlong), ("pool_tokens", C.c_int), ("pooled_stride", C.c_int),
+        ("slot_div", C.c_int), ("slot_of", C.c_void_p), ("talk", C.c_void_p), ("status", C.c_void_p),
     ]
 
 
@@ -173,6 +176,50 @@ class SandwichArgs(C.Structure):
     ]
 
 
+class PreNormArgs(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("x_out", C.c_void_p), ("ldx", C.c_longlong), ("ids", C.c_void_p), ("table", C.c_void_p),
+        ("ldt", C.c_longlong), ("vocab", C.c_int), ("scale", C.c_float), ("y", C.c_void_p), ("ldy", C.c_longlong),
+        ("ffn", C.c_void_p), ("ldf", C.c_longlong), ("slots", C.c_int), ("topk", C.c_int), ("shared", C.c_void_p),
+        ("lds", C.c_longlong), ("shared_gate", C.c_void_p), ("ldsg", C.c_longlong), ("norm_w", C.c_void_p),
+        ("act", C.c_void_p), ("lda", C.c_longlong), ("shift", C.c_void_p), ("plane", C.c_void_p), ("row_seq", C.c_void_p),
+        ("seq_start", C.c_void_p), ("state_in", C.c_void_p), ("state_out", C.c_void_p), ("n_states", C.c_int),
+        ("n_seqs", C.c_int), ("rows", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int), ("fp32", C.c_int),
+        ("eps", C.c_float), ("status", C.c_void_p),
+    ]
+
+
+class HeadScanArgs(C.Structure):
+    _fields_ = [
+        ("xbc", C.c_void_p), ("ldx", C.c_longlong), ("off_b", C.c_int), ("off_c", C.c_int), ("dt", C.c_void_p),
+        ("z", C.c_void_p), ("ldp", C.c_longlong), ("dt_bias", C.c_void_p), ("a_neg", C.c_void_p), ("d_skip", C.c_void_p),
+        ("states", C.c_void_p), ("seq_start", C.c_void_p), ("state_in", C.c_void_p), ("state_out", C.c_void_p),
+        ("out", C.c_void_p), ("ldo", C.c_longlong), ("rows", C.c_int), ("n_seqs", C.c_int), ("heads", C.c_int),
+        ("vdim", C.c_int), ("state", C.c_int), ("groups", C.c_int), ("n_states", C.c_int), ("fp32", C.c_int),
+        ("status", C.c_void_p),
+    ]
+
+
+class LatentPrepArgs(C.Structure):
+    _fields_ = [
+        ("cq", C.c_void_p), ("ckv", C.c_void_p), ("ldp", C.c_longlong), ("rank_q", C.c_int), ("rank", C.c_int),
+        ("rot", C.c_int), ("row_dim", C.c_int), ("rot_off", C.c_int), ("rows", C.c_int), ("q_w", C.c_void_p),
+        ("kv_w", C.c_void_p), ("cos_t", C.c_void_p), ("sin_t", C.c_void_p), ("max_pos", C.c_int), ("fp32", C.c_int),
+        ("positions", C.c_void_p), ("write_slot", C.c_void_p), ("pool", C.c_void_p), ("pool_rows", C.c_longlong),
+        ("eps", C.c_float), ("status", C.c_void_p),
+    ]
+
+
+class PoolArgs(C.Structure):
+    _fields_ = [
+        ("pool", C.c_void_p), ("pool_rows", C.c_longlong), ("pool_ld", C.c_longlong), ("pooled", C.c_void_p),
+        ("pooled_rows", C.c_longlong), ("positions", C.c_void_p), ("row_seq", C.c_void_p), ("block_table", C.c_void_p),
+        ("slot_of", C.c_void_p), ("rows", C.c_int), ("width", C.c_int), ("num_seqs", C.c_int), ("max_blocks", C.c_int),
+        ("page_size", C.c_int), ("pool_tokens", C.c_int), ("pooled_stride", C.c_int), ("slot_div", C.c_int),
+        ("fp32", C.c_int), ("status", C.c_void_p),
+    ]
+
+
 class HeadPrepArgs(C.Structure):
     _fields_ = [
         ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ldp", C.c_longlong), ("q_bias", C.c_void_p),
@@ -180,7 +227,8 @@ class HeadPrepArgs(C.Structure):
         ("q_out", C.c_void_p), ("ldqo", C.c_longlong), ("write_slot", C.c_void_p), ("pool", C.c_void_p),
         ("pool_rows", C.c_longlong), ("pool_ld", C.c_longlong), ("rows", C.c_int), ("heads", C.c_int),
         ("kv_heads", C.c_int), ("maps", C.c_int), ("dim", C.c_int), ("dim_pad", C.c_int), ("vdim_pad", C.c_int),
-        ("fp32", C.c_int), ("eps", C.c_float), ("status", C.c_void_p),
+        ("fp32", C.c_int), ("eps", C.c_float), ("status", C.c_void_p), ("cos_t", C.c_void_p), ("sin_t", C.c_void_p),
+        ("positions", C.c_void_p), ("half", C.c_int), ("max_pos", C.c_int), ("blocks", C.POINTER(PoolArgs)),
     ]
 
 
@@ -210,7 +258,7 @@ def _declare(lib: C.CDLL) -> None:
     lib.fb_add_rmsnorm.argtypes = [vp, ll, vp, ll, vp, vp, ll, vp, ll, i, i, f, vp]
     lib.fb_mla_prep.argtypes = [vp, ll, i, vp, ll, i, i, i, vp, f, vp, vp, i, vp, vp, vp, ll, vp,
                                 ll, i, vp, vp]
-    lib.fb_router_topk.argtypes = [vp, ll, vp, vp, vp, i, i, i, i, i, i, i, f, vp, vp, vp]
+    lib.fb_router_topk.argtypes = [vp, ll, vp, vp, vp, i, i, i, i, i, i, i, f, vp, vp, vp, vp]
     lib.fb_moe_plan.argtypes = [vp, vp, i, i, i, i, i, i, vp, vp, vp, vp, vp, vp, i, vp, vp, vp, vp]
     lib.fb_gather_rows.argtypes = [vp, ll, vp, vp, vp, ll, i, i, i, vp, vp]
     lib.fb_moe_reduce.argtypes = [vp, i, i, vp, i, i, vp, ll, vp, ll, vp, ll, i, i, i, vp]

@@ -38,6 +38,8 @@ def declare(lib) -> None:
                               vp, vp], i),
         "fb_norm_router_append": ([vp, ll, vp, ll, vp, vp, ll, vp, ll, f, vp, i, vp, vp, vp, i, i, i, i, i, i, i, f, vp, vp,
                                    i, i, i, i, vp, vp, vp, vp, vp, ll, vp, vp], i),
+        "fb_router_append_extra": ([vp, ll, vp, i, vp, vp, i, i, i, i, i, i, i, i, f, vp, vp, i, i, i, i, vp, vp, vp, vp, vp, ll,
+                                    vp, vp], i),
         "fb_router_append_q": ([vp, ll, vp, ll, vp, vp, ll, vp, ll, f, vp, i, vp, vp, vp, i, i, i, i, i, i, i, f, vp, vp,
                                 i, i, i, i, vp, vp, vp, vp, vp, ll, vp, ll, vp, ll, vp, ll, vp, ll, i, vp, vp], i),
         "fb_moe_reduce_norm": ([vp, i, i, vp, i, i, vp, ll, vp, ll, i, i, vp, vp, ll, f, vp], i),
@@ -83,7 +85,14 @@ def declare(lib) -> None:
         "fb_gqa_attention": ([vp, vp], i),
         "fb_gqa_decode": ([vp, i, i, vp], i),
         "fb_gqa_decode_wide": ([vp, i, i, vp], i),
-        "fb_gqa_decode_wide_ok": ([i, i, i], i),
+        "fb_gqa_decode_wide_ok": ([i, i, i, i, i], i),
+        "fb_value_mix": ([vp, ll, vp, vp, ll, i, i, i, i, i, vp], i),
+        "fb_pool_blocks": ([vp, vp], i),
+        "fb_pre_norm_step": ([vp, vp], i),
+        "fb_group_norm_rows": ([vp, ll, vp, vp, ll, i, i, i, i, f, i, vp], i),
+        "fb_head_scan": ([vp, vp], i),
+        "fb_latent_prep": ([vp, vp], i),
+        "fb_latent_turn": ([vp, ll, i, i, vp, vp, i, vp, vp, ll, i, i, i, i, vp, vp], i),
         "fb_gqa_prefill_tc": ([vp, vp, i, i, vp], i),
         "fb_head_prep": ([vp, vp], i),
         "fb_sandwich_step": ([vp, vp], i),

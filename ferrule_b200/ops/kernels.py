@@ -72,13 +72,17 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
          use_row_scale: bool = True, act_limit: float = 0.0, ntok: Optional[int] = None,
          x_group_koff: int = 0, out_group_coff: int = 0, k: Optional[int] = None,
          comm=None, residual: Optional[torch.Tensor] = None, split_k: int = 0,
-         trace: Optional[torch.Tensor] = None, ep_combine=None) -> torch.Tensor:
+         trace: Optional[torch.Tensor] = None, ep_combine=None, bias: Optional[torch.Tensor] = None,
+         act_alpha: float = 1.0, act_shift: float = 0.0) -> torch.Tensor:
     """out = x @ w^T on the tcgen05 path (bf16 operands), or in full 32 bits on the FMA units (fp32 operands).
 
     x [rows, K] bf16 (row stride arbitrary multiple of 8), w [N, K] or [groups, N, K] bf16.
     plan        : grouped mode, x rows are in expert-major order.
     epilogue    : EPI_STORE | EPI_GELU | EPI_SWIGLU, EPI_GEGLU (w rows = [gate block | up block]) | EPI_SCATTER |
                   EPI_ALLREDUCE (comm = a parallel.symm.AllReduceChannel).
+    bias        : fp32 [n_out], added in EPI_STORE and EPI_GELU.
+    act_limit, act_alpha, act_shift: EPI_SWIGLU is gate * sigmoid(alpha gate) * (up + shift), with gate <= limit and
+                  |up| <= limit when a limit is given.
     x_group_koff: batched mode (groups > 1 without a plan): group g reads x[:, g*koff : g*koff+K]
                   and writes out[:, g*out_group_coff : +N].
     ep_combine  : EPI_SCATTER only, (rank, world, peer buffers, peer flags, ctr, remap_rank, remap_row, pitch):
@@ -111,7 +115,10 @@ def gemm(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     a.x_rows, a.ntok, a.epilogue, a.dual_offset = rows, ntok, epilogue, dual_offset
     a.out_fp32 = 1 if out.dtype == torch.float32 else 0
     a.x_group_koff, a.out_group_coff = x_group_koff, out_group_coff
-    a.act_limit = act_limit
+    a.act_limit, a.act_alpha, a.act_shift = act_limit, act_alpha, act_shift
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.numel() >= n_out and bias.is_contiguous()
+        a.bias = bias.data_ptr()
     a.force_split = split_k
     a.trace = ptr(trace)
     if plan is not None:
@@ -211,8 +218,9 @@ def router_topk(logits: torch.Tensor, topk: int, score_fn: int, bias: Optional[t
                 n_groups: int = 1, topk_groups: int = 1, normalize: bool = False,
                 route_scale: float = 1.0, hash_table: Optional[torch.Tensor] = None,
                 token_ids: Optional[torch.Tensor] = None, out_idx: Optional[torch.Tensor] = None,
-                out_w: Optional[torch.Tensor] = None, group_top: int = 2):
-    """group_top: a group's score is the sum of its two best selection values (2) or its best one (1)."""
+                out_w: Optional[torch.Tensor] = None, group_top: int = 2, logit_bias: Optional[torch.Tensor] = None):
+    """group_top: a group's score is the sum of its two best selection values (2) or its best one (1).  bias: added to the
+    scores for the selection; logit_bias: added to the logits."""
     lib = get_lib(True)
     rows, experts = logits.shape
     assert logits.dtype == torch.float32
@@ -223,7 +231,7 @@ def router_topk(logits: torch.Tensor, topk: int, score_fn: int, bias: Optional[t
     check(lib.fb_router_topk(logits.data_ptr(), logits.stride(0), ptr(bias), ptr(hash_table),
                              ptr(token_ids), rows, experts, topk, score_fn, n_groups, topk_groups,
                              _norm_bits(normalize, group_top), route_scale, out_idx.data_ptr(), out_w.data_ptr(),
-                             stream_ptr()), "fb_router_topk")
+                             ptr(logit_bias), stream_ptr()), "fb_router_topk")
     return out_idx, out_w
 
 
@@ -385,12 +393,15 @@ def router_append(x: torch.Tensor, w: torch.Tensor, topk: int, score_fn: int, pl
                   token_ids: Optional[torch.Tensor] = None, dst_slots: int = 0,
                   norm_w: Optional[torch.Tensor] = None, eps: float = 0.0, delta: Optional[torch.Tensor] = None,
                   res_out: Optional[torch.Tensor] = None, norm_out: Optional[torch.Tensor] = None,
-                  quant_rows=None, group_top: int = 2) -> None:
+                  quant_rows=None, group_top: int = 2, logit_bias: Optional[torch.Tensor] = None,
+                  extra: Optional[torch.Tensor] = None) -> None:
     """Router + top-k + row reservation in a static plan + activation gather, one launch (one CTA per token).
     `plan.counts` must be zero on entry.  With `norm_w` the kernel first forms the row itself: `x` is then the
     residual stream, res_out = bf16(x + delta), norm_out = RMSNorm(res_out) * norm_w (bit-equal to `add_rmsnorm`),
     and the router reads that normalised row.  `quant_rows` = (codes [rows, hidden] u8, scales [rows, c] u8,
-    xg codes, xg scales): the gathered rows are the token's quantised codes and scale bytes (`xg` is unused)."""
+    xg codes, xg scales): the gathered rows are the token's quantised codes and scale bytes (`xg` is unused).
+    `logit_bias` is added to the logits; `extra` [rows, n] fp32 receives the products with the last n rows of `w`, which
+    belong to no expert."""
     lib = get_lib(True)
     rows, hidden = x.shape
     assert rows <= plan.ntok and w.is_contiguous()
@@ -411,6 +422,17 @@ def router_append(x: torch.Tensor, w: torch.Tensor, topk: int, score_fn: int, pl
                                      status_tensor(x.device).data_ptr(), stream_ptr()), "fb_router_append_q")
         return
     assert xg.shape[0] >= plan.cap_rows and xg.shape[1] == hidden
+    if logit_bias is not None or extra is not None:
+        assert bias is None and hash_table is None and norm_w is None
+        n = 0 if extra is None else extra.shape[1]
+        assert n == 0 or (extra.is_contiguous() and extra.dtype == torch.float32)
+        check(lib.fb_router_append_extra(x.data_ptr(), x.stride(0), w.data_ptr(), hidden, ptr(logit_bias), ptr(extra), n, rows,
+                                         w.shape[0] - n, topk, score_fn, n_groups, topk_groups, _norm_bits(normalize, group_top),
+                                         route_scale, out_idx.data_ptr(), out_w.data_ptr(), e_lo, e_hi, plan.ntok, dst_slots,
+                                         plan.counts.data_ptr(), plan.src_token.data_ptr(), plan.dst_row.data_ptr(),
+                                         plan.row_scale.data_ptr(), xg.data_ptr(), xg.stride(0),
+                                         status_tensor(x.device).data_ptr(), stream_ptr()), "fb_router_append_extra")
+        return
     check(lib.fb_norm_router_append(x.data_ptr(), x.stride(0), ptr(delta), delta.stride(0) if delta is not None else 0,
                                     ptr(norm_w), ptr(res_out), res_out.stride(0) if res_out is not None else 0,
                                     ptr(norm_out), norm_out.stride(0) if norm_out is not None else 0, eps,
@@ -493,7 +515,7 @@ def prefill_tc_supported(heads: int, kv_lora: int, rope_dim: int, page_size: int
 
 def mla_prefill_tc(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Tensor, tiles: torch.Tensor,
                    n_tiles: int, page_size: int, kv_lora: int, rope_dim: int, scale: float, out: torch.Tensor,
-                   sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
     """Prefill attention on tcgen05: q [rows, heads, 512 + rope_dim] bf16 contiguous, tiles [>= n_tiles, 4] int32 on the
     device (see `prefill_tiles`); rows that no tile covers are left untouched in `out` [rows, heads, 512]."""
     lib = get_lib(True)
@@ -507,7 +529,7 @@ def mla_prefill_tc(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.T
     a.pool_rows = kv_layer.numel() // D
     a.n_tiles, a.rows, a.heads, a.kv_lora, a.rope_dim = n_tiles, rows, heads, kv_lora, rope_dim
     a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
-    a.softmax_scale = scale
+    a.softmax_scale, a.window = scale, window
     if gate is not None:
         a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
     check(lib.fb_mla_prefill_tc(C.byref(a), stream_ptr()), "fb_mla_prefill_tc")
@@ -520,11 +542,13 @@ def mla_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Te
                   split_tokens: int = 1 << 20, ws: Optional[AttnWorkspace] = None,
                   sink: Optional[torch.Tensor] = None, group_rows: int = 1,
                   trace: Optional[torch.Tensor] = None, decode_only: bool = False,
-                  gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  gate: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
     """q [rows, heads, D] bf16; kv_layer [..., D] bf16 (any leading shape, contiguous rows).
     decode_only: one query row per sequence, and every KV row below its position predates the running step
     (the kernel then requests its first KV tile before waiting for the preceding kernel).
-    gate: bf16 [rows, >= heads], the output of a head is multiplied by the sigmoid of its entry."""
+    gate: bf16 [rows, >= heads], the output of a head is multiplied by the sigmoid of its entry.
+    window > 0: a row sees its last `window` tokens only; the splits together cover `split_tokens` each from the 64-token
+    boundary below a tile's first visible token on."""
     lib = get_lib(True)
     rows, heads, D = q.shape
     assert D == kv_lora + rope_dim and q.stride(2) == 1 and q.stride(1) == D
@@ -542,7 +566,7 @@ def mla_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Te
     a.rows, a.heads, a.kv_lora, a.rope_dim = rows, heads, kv_lora, rope_dim
     a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
     a.group_rows, a.splits, a.split_tokens = group_rows, splits, split_tokens
-    a.softmax_scale = scale
+    a.softmax_scale, a.window = scale, window
     a.trace = ptr(trace)
     a.decode_only = 1 if (decode_only and group_rows == 1) else 0
     if gate is not None:

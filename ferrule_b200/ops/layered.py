@@ -1,5 +1,5 @@
 """Launchers of the layer-list model kernels (csrc/layered_ops.cu, stream_ops.cu, delta_rule.cu, selective_scan.cu,
-gqa_*.cu, head_prep.cu).
+gqa_*.cu, head_prep.cu, pre_norm.cu, head_scan.cu).
 
 Activations are bf16, or fp32 for models that run in full 32 bits: the launcher follows the tensors' dtype.
 """
@@ -12,8 +12,8 @@ from typing import Optional
 import torch
 
 from . import _lib
-from ._lib import (AttnArgs, ConvArgs, DeltaArgs, GqaArgs, HeadPrepArgs, LayerTailArgs, SandwichArgs, ScanArgs, StreamArgs, check,
-                   get_lib, ptr, status_tensor, stream_ptr)
+from ._lib import (AttnArgs, ConvArgs, DeltaArgs, GqaArgs, HeadPrepArgs, HeadScanArgs, LatentPrepArgs, LayerTailArgs, PoolArgs,
+                   PreNormArgs, SandwichArgs, ScanArgs, StreamArgs, check, get_lib, ptr, status_tensor, stream_ptr)
 
 
 def _fp32(t: torch.Tensor) -> int:
@@ -81,8 +81,9 @@ def state_rotate(state_in: torch.Tensor, state_out: torch.Tensor, buffers: int) 
 
 def latent_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
                      row_pos: torch.Tensor, page_size: int, scale: float, out: torch.Tensor,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Causal attention over a latent cache in 32-bit arithmetic: q / out [rows, heads, row_dim]."""
+                     gate: Optional[torch.Tensor] = None, window: int = 0) -> torch.Tensor:
+    """Causal attention over a latent cache in 32-bit arithmetic: q / out [rows, heads, row_dim].  window > 0: the last
+    `window` tokens of a row only."""
     rows, heads, D = q.shape
     assert q.stride(1) == D and out.stride(1) == D and kv_layer.shape[-1] == D and kv_layer.dtype == q.dtype
     a = AttnArgs()
@@ -92,11 +93,42 @@ def latent_attention(q: torch.Tensor, kv_layer: torch.Tensor, block_table: torch
     a.ldq, a.ldo, a.pool_rows = q.stride(0), out.stride(0), kv_layer.numel() // D
     a.rows, a.heads, a.kv_lora = rows, heads, D
     a.num_seqs, a.max_blocks, a.page_size = block_table.shape[0], block_table.shape[1], page_size
-    a.softmax_scale = scale
+    a.softmax_scale, a.window = scale, window
     if gate is not None:
         a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
     check(get_lib(True).fb_latent_attention(C.byref(a), _fp32(q), stream_ptr()), "fb_latent_attention")
     return out
+
+
+def latent_prep(proj: torch.Tensor, off, mixer, img, rotation, positions: torch.Tensor, write_slot: torch.Tensor,
+                pool_layer: torch.Tensor, eps: float) -> None:
+    """Latent layers with a query latent or a rotated part: the query latent (block `dq` of the projection) is normalised in
+    place, the cache row of every token is [RMSNorm(latent) | turned key part | zeros].  rotation = (cos, sin) fp32
+    [positions, rot_dim / 2]."""
+    a = LatentPrepArgs()
+    item, DL = proj.element_size(), pool_layer.shape[-1]
+    assert pool_layer.is_contiguous() and pool_layer.dtype == proj.dtype and DL == mixer.row_dim and write_slot.dtype == torch.int64
+    if mixer.q_rank:
+        a.cq, a.rank_q, a.q_w = proj.data_ptr() + off["dq"] * item, mixer.q_rank, img.dq_norm.data_ptr()
+    a.ckv, a.ldp = proj.data_ptr() + off["dkv"] * item, proj.stride(0)
+    a.rank, a.rot, a.row_dim, a.rot_off, a.rows = mixer.kv_rank, mixer.rot_dim, DL, mixer.rot_offset, proj.shape[0]
+    a.kv_w, a.fp32, a.eps = img.kv_norm.data_ptr(), _fp32(proj), eps
+    if mixer.rot_dim:
+        a.cos_t, a.sin_t, a.max_pos = rotation[0].data_ptr(), rotation[1].data_ptr(), rotation[0].shape[0]
+        a.positions = positions.data_ptr()
+    a.write_slot, a.pool, a.pool_rows = write_slot.data_ptr(), pool_layer.data_ptr(), pool_layer.numel() // DL
+    a.status = status_tensor(proj.device).data_ptr()
+    check(get_lib(True).fb_latent_prep(C.byref(a), stream_ptr()), "fb_latent_prep")
+
+
+def latent_turn(src: torch.Tensor, mixer, rotation, positions: torch.Tensor, q: torch.Tensor) -> None:
+    """Rotated query parts (src [rows, heads * rot_dim]) into their columns of the query rows q [rows, heads, row_dim]."""
+    rows, heads, DL = q.shape
+    assert src.dtype == q.dtype and q.stride(1) == DL and src.stride(1) == 1
+    check(get_lib(True).fb_latent_turn(src.data_ptr(), src.stride(0), heads, mixer.rot_dim, rotation[0].data_ptr(),
+                                       rotation[1].data_ptr(), rotation[0].shape[0], positions.data_ptr(), q.data_ptr(),
+                                       q.stride(0), DL, mixer.rot_offset, rows, _fp32(q), status_tensor(q.device).data_ptr(),
+                                       stream_ptr()), "fb_latent_turn")
 
 
 class DeltaScratch:
@@ -245,6 +277,68 @@ def sandwich_rows(x: torch.Tensor, rows: torch.Tensor, norm: torch.Tensor, out: 
     return out
 
 
+def pre_norm_step(x: Optional[torch.Tensor], x_out: torch.Tensor, *, dim: int, eps: float, like: torch.Tensor,
+                  ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, scale: float = 1.0,
+                  y: Optional[torch.Tensor] = None, ffn: Optional[torch.Tensor] = None, topk: int = 0,
+                  shared: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None,
+                  norm: Optional[torch.Tensor] = None, act: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None,
+                  plane: Optional[torch.Tensor] = None, seqs=None) -> None:
+    """x_out = (x, or table[ids] * scale) + y + the first `topk` of a token's ffn rows [rows, slots, width] + sigmoid(shared_gate)
+    shared; act = RMSNorm(x_out) * norm, with `shift` moved towards the previous token's row.  plane: the shift's state;
+    seqs = (row_seq, seq_start, state_in, state_out, n_seqs).  `like` has the activations' dtype."""
+    a = PreNormArgs()
+    assert x_out.dtype == torch.float32 and (x is None or (x.dtype == torch.float32 and x.stride(0) == x_out.stride(0)))
+    assert all(t is None or t.dtype == like.dtype for t in (table, y, ffn, shared, act))
+    a.x, a.x_out, a.ldx = ptr(x), x_out.data_ptr(), x_out.stride(0)
+    if ids is not None:
+        a.ids, a.table, a.ldt, a.vocab, a.scale = ids.data_ptr(), table.data_ptr(), table.stride(0), table.shape[0], scale
+    if y is not None:
+        a.y, a.ldy = y.data_ptr(), y.stride(0)
+    if ffn is not None:
+        assert ffn.dim() == 3 and ffn.is_contiguous() and topk <= ffn.shape[1]
+        a.ffn, a.ldf, a.slots, a.topk = ffn.data_ptr(), ffn.stride(1), ffn.shape[1], topk
+    if shared is not None:
+        assert shared_gate.dtype == torch.float32
+        a.shared, a.lds, a.shared_gate, a.ldsg = shared.data_ptr(), shared.stride(0), shared_gate.data_ptr(), shared_gate.stride(0)
+    if act is not None:
+        a.norm_w, a.act, a.lda = norm.data_ptr(), act.data_ptr(), act.stride(0)
+    if shift is not None:
+        assert plane.dtype == torch.float32 and plane.is_contiguous() and plane.shape[1] == x_out.shape[1]
+        a.shift, a.plane, a.n_states = shift.data_ptr(), plane.data_ptr(), plane.shape[0]
+        a.row_seq, a.seq_start, a.state_in, a.state_out = (t.data_ptr() for t in seqs[:4])
+        a.n_seqs = seqs[4]
+    a.rows, a.dim, a.dim_pad, a.fp32, a.eps = x_out.shape[0], dim, x_out.shape[1], _fp32(like), eps
+    a.status = status_tensor(x_out.device).data_ptr()
+    check(get_lib(True).fb_pre_norm_step(C.byref(a), stream_ptr()), "fb_pre_norm_step")
+
+
+def group_norm_rows(x: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, dim: int, groups: int, eps: float) -> torch.Tensor:
+    """out = x with each of `groups` equal parts of a row divided by its root mean square, times norm (in place allowed)."""
+    assert x.dtype == out.dtype and x.shape == out.shape
+    check(get_lib(True).fb_group_norm_rows(x.data_ptr(), x.stride(0), norm.data_ptr(), out.data_ptr(), out.stride(0), x.shape[0],
+                                           dim, x.shape[1], groups, eps, _fp32(x), stream_ptr()), "fb_group_norm_rows")
+    return out
+
+
+def head_scan(xbc: torch.Tensor, proj: torch.Tensor, off, mixer, img, states: torch.Tensor, seq_start: torch.Tensor,
+              state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, out: torch.Tensor) -> torch.Tensor:
+    """(scan + D x) * silu(z) of a head-decay scan over packed rows: xbc the convolved x | B | C, z and dt blocks of the
+    projection."""
+    assert states.dtype == torch.float32 and states.is_contiguous() and xbc.dtype == proj.dtype == out.dtype
+    a = HeadScanArgs()
+    item = proj.element_size()
+    a.xbc, a.ldx, a.off_b, a.off_c = xbc.data_ptr(), xbc.stride(0), img.off_b, img.off_c
+    a.dt, a.z, a.ldp = proj.data_ptr() + off["dt"] * item, proj.data_ptr() + off["z"] * item, proj.stride(0)
+    a.dt_bias, a.a_neg, a.d_skip = img.dt_bias.data_ptr(), img.a_neg.data_ptr(), img.d_skip.data_ptr()
+    a.states, a.n_states = states.data_ptr(), states.shape[0]
+    a.seq_start, a.state_in, a.state_out = seq_start.data_ptr(), state_in.data_ptr(), state_out.data_ptr()
+    a.out, a.ldo, a.rows, a.n_seqs, a.fp32 = out.data_ptr(), out.stride(0), xbc.shape[0], n_seqs, _fp32(xbc)
+    a.heads, a.vdim, a.state, a.groups = mixer.heads, mixer.vdim, mixer.state, mixer.groups
+    a.status = status_tensor(xbc.device).data_ptr()
+    check(get_lib(True).fb_head_scan(C.byref(a), stream_ptr()), "fb_head_scan")
+    return out
+
+
 def short_conv(x: torch.Tensor, w: torch.Tensor, tail: torch.Tensor, out: torch.Tensor, row_seq: torch.Tensor,
                seq_start: torch.Tensor, state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, *,
                bias: Optional[torch.Tensor] = None, residual: bool = False, silu: bool = False) -> torch.Tensor:
@@ -284,7 +378,8 @@ def selective_scan(x: torch.Tensor, z: torch.Tensor, bc: torch.Tensor, off_b: in
 
 # ------------------------------------------------------------------ grouped-query attention in chunks and windows
 def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor, slopes: Optional[torch.Tensor] = None,
-         gate: Optional[torch.Tensor] = None, diff_lambda: float = 0.0, eps: float = 0.0) -> GqaArgs:
+         gate: Optional[torch.Tensor] = None, diff_lambda: float = 0.0, eps: float = 0.0, mean=None,
+         talk: Optional[torch.Tensor] = None) -> GqaArgs:
     a = GqaArgs()
     assert q.dtype == pool.dtype and pool.is_contiguous()
     a.q, a.ldq, a.rows, a.fp32 = q.data_ptr(), q.stride(0), q.shape[0], _fp32(q)
@@ -296,6 +391,13 @@ def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor, slopes: Optional[torch.Tens
     a.key_stride = 0 if mixer.shared_keys else mixer.key_width
     a.slopes, a.eps, a.diff_lambda = ptr(slopes), eps, diff_lambda
     a.diff_scale = 1.0 - mixer.diff if mixer.maps == 2 else 1.0
+    a.value_width, a.value_stride = mixer.value_width, 0 if mixer.shared_values else mixer.vdim_pad
+    a.softcap, a.talk = mixer.softcap, ptr(talk)
+    if mean is not None:
+        rows, a.slot_div, slots = mean
+        assert rows.dtype == q.dtype and rows.is_contiguous() and rows.shape[2] == pool.shape[-1]
+        a.pooled, a.pooled_rows, a.pooled_stride, a.pool_tokens = rows.data_ptr(), rows.shape[0] * rows.shape[1], rows.shape[1], mixer.pool
+        a.slot_of = slots.data_ptr()
     if gate is not None:
         assert gate.dtype == q.dtype
         a.gate, a.ldg = gate.data_ptr(), gate.stride(0)
@@ -309,16 +411,46 @@ def _scaled(a: GqaArgs, mixer) -> GqaArgs:
     return a
 
 
+def _pool_args(mixer, pool: torch.Tensor, mean, positions, row_seq, block_table, page_size: int) -> PoolArgs:
+    rows, div, slots = mean
+    a = PoolArgs()
+    assert rows.dtype == pool.dtype and rows.is_contiguous() and pool.is_contiguous() and rows.shape[2] == pool.shape[-1]
+    a.pool, a.pool_ld, a.pool_rows = pool.data_ptr(), pool.shape[-1], pool.numel() // pool.shape[-1]
+    a.pooled, a.pooled_rows, a.pooled_stride, a.slot_div = rows.data_ptr(), rows.shape[0] * rows.shape[1], rows.shape[1], div
+    a.positions, a.row_seq, a.block_table, a.slot_of = (positions.data_ptr(), row_seq.data_ptr(), block_table.data_ptr(),
+                                                        slots.data_ptr())
+    a.rows, a.width, a.num_seqs, a.max_blocks = positions.shape[0], mixer.row_dim, block_table.shape[0], block_table.shape[1]
+    a.page_size, a.pool_tokens, a.fp32 = page_size, mixer.pool, _fp32(pool)
+    a.status = status_tensor(pool.device).data_ptr()
+    return a
+
+
+def pool_blocks(mixer, pool: torch.Tensor, mean, positions: torch.Tensor, row_seq: torch.Tensor, block_table: torch.Tensor,
+                page_size: int) -> None:
+    """Mean cache rows of the blocks that end with rows of this batch, whose cache rows are written.  mean = (rows [slots,
+    blocks, row width], divisor, slot numbers): sequence s owns rows[slots[s] // divisor]."""
+    a = _pool_args(mixer, pool, mean, positions, row_seq, block_table, page_size)
+    check(get_lib(True).fb_pool_blocks(C.byref(a), stream_ptr()), "fb_pool_blocks")
+
+
 def head_prep(proj: torch.Tensor, off, mixer, img, write_slot: torch.Tensor, pool: torch.Tensor, eps: float,
-              q_out: torch.Tensor) -> None:
-    """Between the projection and window attention: biases, query and key norm per head, factors and mixing of the queries
-    across heads (into q_out), cache append of keys and values."""
+              q_out: torch.Tensor, rotation=None, positions: Optional[torch.Tensor] = None, blocks=None) -> None:
+    """Between the projection and window attention: biases, rotation, query and key norm per head, factors and mixing of the
+    queries across heads (into q_out, which may be the projection's own queries), cache append of keys and values.  blocks
+    (one row per sequence) = the further arguments of `pool_blocks`."""
     assert proj.dtype == pool.dtype == q_out.dtype and pool.is_contiguous() and write_slot.dtype == torch.int64
     a = HeadPrepArgs()
     item = proj.element_size()
     at = lambda name: proj.data_ptr() + off[name] * item
     a.q, a.k, a.v, a.ldp = at("q"), at("k"), None if mixer.tied_values else at("v"), proj.stride(0)
-    a.q_bias, a.k_bias, a.q_norm, a.k_norm = ptr(img.q_bias), ptr(img.k_bias), img.q_norm.data_ptr(), img.k_norm.data_ptr()
+    a.q_bias, a.k_bias, a.q_norm, a.k_norm = ptr(img.q_bias), ptr(img.k_bias), ptr(img.q_norm), ptr(img.k_norm)
+    if mixer.rot_dims:
+        a.cos_t, a.sin_t, a.max_pos, a.half = (rotation[0].data_ptr(), rotation[1].data_ptr(), rotation[0].shape[0],
+                                               mixer.rot_dims // 2)
+        a.positions = positions.data_ptr()
+    if blocks is not None:
+        pool_args = _pool_args(mixer, pool, *blocks)
+        a.blocks = C.pointer(pool_args)
     a.q_mix, a.mix, a.q_out, a.ldqo = img.q_mix.data_ptr(), int(mixer.mix_heads), q_out.data_ptr(), q_out.stride(0)
     a.write_slot, a.pool, a.pool_ld, a.pool_rows = (write_slot.data_ptr(), pool.data_ptr(), pool.shape[-1],
                                                     pool.numel() // pool.shape[-1])
@@ -357,17 +489,25 @@ def _gqa_rows(a: GqaArgs, block_table, row_seq, row_pos, page_size: int, out: to
 
 def gqa_attention(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Tensor, row_seq: torch.Tensor,
                   row_pos: torch.Tensor, page_size: int, out: torch.Tensor, **form) -> torch.Tensor:
-    """32-bit arithmetic: out [rows, heads * vdim_pad].  form: slopes, gate, diff_lambda, eps of a window mixer."""
+    """32-bit arithmetic: out [rows, heads * value_width].  form: slopes, gate, diff_lambda, eps, mean of a window mixer."""
     a = _scaled(_gqa(q, mixer, pool, **form), mixer)
     _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
     check(get_lib(True).fb_gqa_attention(C.byref(a), stream_ptr()), "fb_gqa_attention")
     return out
 
 
+def value_mix(o: torch.Tensor, talk: torch.Tensor, mixer, out: torch.Tensor) -> torch.Tensor:
+    """Outputs of every head on the values of every kv head (o [rows, heads * value_width]) -> those of mixed softmax weights."""
+    assert o.dtype == out.dtype and talk.dtype == torch.float32 and talk.is_contiguous() and mixer.shared_values
+    check(get_lib(True).fb_value_mix(o.data_ptr(), o.stride(0), talk.data_ptr(), out.data_ptr(), out.stride(0), o.shape[0],
+                                     mixer.heads, mixer.kv_heads, mixer.vdim_pad, _fp32(o), stream_ptr()), "fb_value_mix")
+    return out
+
+
 def gqa_tc_group(mixer, dtype, page_size: int) -> int:
     """Query rows per key / value head when the bf16 prompt kernel serves the mixer, else 0."""
     per = mixer.heads // mixer.kv_heads * mixer.maps
-    ok = (dtype == torch.bfloat16 and mixer.vdim_pad <= 256 and per <= 128
+    ok = (dtype == torch.bfloat16 and (mixer.vdim_pad <= 256 or mixer.shared_values) and per <= 128
           and (mixer.shared_keys or mixer.key_width <= 256) and (mixer.scaled_queries or mixer.scale > 0)
           and page_size >= 8 and page_size & (page_size - 1) == 0)
     return per if ok else 0
@@ -385,22 +525,29 @@ def gqa_decode_supported(mixer, dtype, page_size: int) -> bool:
     """Whether the bf16 kernels for few rows serve the mixer."""
     if dtype != torch.bfloat16:
         return False
-    if mixer.shared_keys:
-        return bool(get_lib(True).fb_gqa_decode_wide_ok(mixer.key_width, mixer.kv_heads, mixer.vdim_pad))
+    if mixer.shared_keys or mixer.shared_values:
+        width = mixer.key_width if mixer.shared_keys else mixer.kv_heads * mixer.key_width
+        return bool(get_lib(True).fb_gqa_decode_wide_ok(width, mixer.kv_heads, mixer.vdim_pad, mixer.shared_values, mixer.heads))
+    if mixer.pool or mixer.softcap:
+        return False
     return max(mixer.key_width, mixer.vdim_pad) <= 256
 
 
 def gqa_decode_splits(rows: int, mixer, max_keys: int) -> int:
     """CTAs per row: about two per SM over the batch (one where it takes all kv heads, or wide ones), each with at least 128
     (64) keys of the longest row."""
-    if mixer.shared_keys:
+    most, visible = 8, mixer.chunk or mixer.window + mixer.keep_first
+    if mixer.pool:
+        visible += max(max_keys - mixer.window, 0) // mixer.pool
+    if mixer.shared_keys or mixer.shared_values:
         ctas, fill, least = rows * ((mixer.heads + 15) // 16), 148, 64
+        if mixer.shared_values:
+            most = 8 // ((mixer.heads + 15) // 16)         # a row's head blocks belong to its cluster
     else:
         ctas = rows * mixer.kv_heads * ((mixer.heads // mixer.kv_heads * mixer.maps + 15) // 16)
         fill, least = 296 if max(mixer.key_width, mixer.vdim_pad) <= 128 else 148, 128
-    visible = mixer.chunk or mixer.window + mixer.keep_first
     splits = 1
-    while splits < 8 and ctas * splits * 2 <= fill and min(visible, max_keys) >= splits * 2 * least:
+    while splits * 2 <= most and ctas * splits * 2 <= fill and min(visible, max_keys) >= splits * 2 * least:
         splits *= 2
     return splits
 
@@ -411,7 +558,7 @@ def gqa_decode(q: torch.Tensor, mixer, pool: torch.Tensor, block_table: torch.Te
     """Few query rows, bf16.  decode_only: one row per sequence, every key below its position predates the running step."""
     a = _scaled(_gqa(q, mixer, pool, **form), mixer)
     _gqa_rows(a, block_table, row_seq, row_pos, page_size, out)
-    name = "fb_gqa_decode_wide" if mixer.shared_keys else "fb_gqa_decode"
+    name = "fb_gqa_decode_wide" if mixer.shared_keys or mixer.shared_values else "fb_gqa_decode"
     check(getattr(get_lib(True), name)(C.byref(a), splits, 1 if decode_only else 0, stream_ptr()), name)
     return out
 
