@@ -39,6 +39,7 @@ CUDA_SOURCES = [
     "stream_ops.cu",
     "selective_scan.cu",
     "head_scan.cu",
+    "head_scan_chunk.cu",
     "pre_norm.cu",
     "gqa_attention.cu",
     "gqa_decode.cu",
@@ -57,7 +58,8 @@ CUDA_SOURCES = [
 COMPONENTS = {
     "layered": ["gemm_tcgen05.cu", "mla_attention.cu", "mla_prefill_tc.cu", "elementwise.cu", "data_movers.cu",
                 "layered_ops.cu", "delta_rule.cu", "gemm_f32.cu", "stream_ops.cu", "selective_scan.cu", "gqa_attention.cu",
-                "gqa_decode.cu", "gqa_decode_wide.cu", "gqa_prefill_tc.cu", "head_prep.cu", "head_scan.cu", "pre_norm.cu"],
+                "gqa_decode.cu", "gqa_decode_wide.cu", "gqa_prefill_tc.cu", "head_prep.cu", "head_scan.cu", "head_scan_chunk.cu",
+                "pre_norm.cu"],
 }
 CXX_SOURCES = [
     "host/kv_page_manager.cpp",

@@ -420,6 +420,8 @@ typedef struct FbHeadScanArgs {
   void* out;                // [rows, ldo]: (scan + D x) * silu(z); columns past heads x vdim are zero
   long long ldo;
   int rows, n_seqs, heads, vdim, state, groups, n_states, fp32;
+  int long_seqs;            // sequences with more than one row, when known (0: not counted)
+  int by_token;             // prompts token by token instead of in chunks
   void* status;
 } FbHeadScanArgs;
 int fb_head_scan(const FbHeadScanArgs* args, void* stream);     // state <= 256

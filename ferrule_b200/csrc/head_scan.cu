@@ -4,9 +4,10 @@
 //
 // B, C and x have passed the short convolution.  Step sizes, decays, state and sums are fp32.
 //
-// Any mix of row counts: CTA = (columns of a head, head, sequence).  LPC lanes share VPL columns and hold SPL state rows of each in
+// Prompts of bf16 models take the chunked form (head_scan_chunk.cu) where the sizes allow it.  Token by token, any mix of row
+// counts: CTA = (columns of a head, head, sequence).  LPC lanes share VPL columns and hold SPL state rows of each in
 // registers; sixteen tokens are staged at a time and the next ones requested before the staged ones are worked on.
-// Decode steps (one row per sequence): CTA = (head, sequence), the state streams through registers once; its first part is
+// Sequences with one row (decode steps, and the single rows beside chunked prompts): CTA = (head, sequence), the state streams through registers once; its first part is
 // requested before the dependency wait.
 //
 // State of a sequence: fp32 [heads, state, vdim].  Buffer `state_in[seq]` is read (-1: a new sequence, zeros), buffer
@@ -15,6 +16,7 @@
 #include "common.cuh"
 #include "f32x2.cuh"
 #include "ferrule_b200.h"
+#include "head_scan.cuh"
 #include "launch.cuh"
 #include "scan_math.cuh"
 
@@ -23,34 +25,6 @@ namespace fb {
 constexpr int kHsThreads = 128;
 constexpr int kHsTokens = 16;
 constexpr int kHsRows = 8, kHsCols = 4;       // state rows and columns of a lane
-
-template <typename T>
-struct HeadScanParams {
-  const T* xbc;
-  long long ldx;
-  int off_b, off_c;
-  const T* dt;
-  const T* z;
-  long long ldp;
-  const float* dt_bias;
-  const float* a_neg;
-  const float* d_skip;
-  float* states;
-  const int* seq_start;
-  const int* state_in;
-  const int* state_out;
-  T* out;
-  long long ldo;
-  int rows, n_seqs, heads, vdim, state, groups, n_states, out_cols;
-  DeviceStatus* status;
-};
-
-template <typename T>
-__device__ __forceinline__ bool scan_bind(const HeadScanParams<T>& p, int seq, int& sin, int& sout) {
-  sin = p.state_in[seq];
-  sout = p.state_out[seq];
-  return sin < p.n_states && sout < p.n_states && !(sin >= 0 && sin == sout);
-}
 
 template <typename T, int LPC>
 __global__ void __launch_bounds__(kHsThreads)
@@ -225,12 +199,13 @@ template <typename T>
 __global__ void __launch_bounds__(kHsStepThreads)
 head_scan_step_kernel(const HeadScanParams<T> p) {
   pdl_launch_dependents();
-  extern __shared__ float hs_sm[];                       // [state] B, [state] C, [vdim] x, [row groups][quads * 4] partial sums
+  extern __shared__ __align__(16) float hs_sm[];                       // [state] B, [state] C, [vdim] x, [row groups][quads * 4] partial sums
   const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, group = h / (p.heads / p.groups);
   const int quads = (p.vdim + 3) / 4, lanes = min(quads, kHsStepThreads), n_groups = kHsStepThreads / lanes;
+  const int n_pad = (p.state + 3) / 4 * 4;               // 16-byte alignment of what follows
   float* s_b = hs_sm;
-  float* s_c = s_b + p.state;
-  float* s_x = s_c + p.state;
+  float* s_c = s_b + n_pad;
+  float* s_x = s_c + n_pad;
   float* s_y = s_x + (p.vdim + 3) / 4 * 4;
   int sin, sout;
   const bool ok = scan_bind(p, seq, sin, sout);
@@ -251,6 +226,7 @@ head_scan_step_kernel(const HeadScanParams<T> p) {
   const float bias = p.dt_bias[h], rate = p.a_neg[h] * 1.4426950408889634f, skip = p.d_skip[h];
   pdl_wait();
   const int r = p.seq_start[seq];
+  if (ok && r >= 0 && p.seq_start[seq + 1] > r + 1 && p.skip_single) return;     // beside a chunked launch: not a single row
   if (!ok || r < 0 || r >= p.rows || p.seq_start[seq + 1] != r + 1) {
     if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE52, seq, r);
     return;
@@ -312,6 +288,15 @@ static int launch_head_scan(const HeadScanParams<T>& p, cudaStream_t s) {
 }
 
 template <typename T>
+static int launch_step(const HeadScanParams<T>& p, cudaStream_t s) {
+  const int quads = (p.vdim + 3) / 4, lanes = quads < kHsStepThreads ? quads : kHsStepThreads;
+  const size_t smem = (2 * static_cast<size_t>((p.state + 3) / 4 * 4) + quads * 4 + static_cast<size_t>(kHsStepThreads / lanes) * quads * 4) * sizeof(float);
+  if (smem > 48 * 1024) return FB_ERR_LIMIT;
+  launch_pdl(head_scan_step_kernel<T>, dim3(p.heads, p.n_seqs), dim3(kHsStepThreads), smem, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+}
+
+template <typename T>
 static int run_head_scan(const FbHeadScanArgs* a, cudaStream_t s) {
   HeadScanParams<T> p{};
   p.xbc = static_cast<const T*>(a->xbc); p.ldx = a->ldx; p.off_b = a->off_b; p.off_c = a->off_c;
@@ -323,12 +308,16 @@ static int run_head_scan(const FbHeadScanArgs* a, cudaStream_t s) {
   p.n_states = a->n_states;
   p.out_cols = (a->heads * a->vdim + 7) / 8 * 8;
   p.status = static_cast<DeviceStatus*>(a->status);
-  if (p.n_seqs == p.rows) {
-    const int quads = (p.vdim + 3) / 4, lanes = quads < kHsStepThreads ? quads : kHsStepThreads;
-    const size_t smem = (2 * static_cast<size_t>(p.state) + quads * 4 + static_cast<size_t>(kHsStepThreads / lanes) * quads * 4) * sizeof(float);
-    if (smem > 48 * 1024) return FB_ERR_LIMIT;
-    launch_pdl(head_scan_step_kernel<T>, dim3(p.heads, p.n_seqs), dim3(kHsStepThreads), smem, s, p);
-    return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  if (p.n_seqs == p.rows) return launch_step<T>(p, s);
+  if constexpr (sizeof(T) == 2) {
+    if (!a->by_token && head_scan_chunk_ok(p.vdim, p.state, p.groups)) {
+      p.skip_single = a->long_seqs != p.n_seqs;
+      if (p.skip_single) {
+        const int rc = launch_step<T>(p, s);
+        if (rc != FB_OK) return rc;
+      }
+      return run_head_scan_chunk(p, s);
+    }
   }
   if (p.state <= 32) return launch_head_scan<T, 4>(p, s);
   if (p.state <= 64) return launch_head_scan<T, 8>(p, s);

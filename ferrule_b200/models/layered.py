@@ -753,7 +753,7 @@ class LayeredCuda:
         xbc = self._view(ws.conv_x, T, m.channels)
         KL.short_conv(proj[:, :m.channels], mx.conv, self.states.tail[layer], xbc, b.row_seq[:T], *seqs, bias=mx.conv_b, silu=True)
         out = self._view(ws.mix_in, T, m.inner_pad)
-        KL.head_scan(xbc, proj, mx.off, m, mx, self.states.state[layer], *seqs, out)
+        KL.head_scan(xbc, proj, mx.off, m, mx, self.states.state[layer], *seqs, out, long_seqs=b.long_seqs)
         return KL.group_norm_rows(out, mx.o_norm, out, m.inner, m.norm_groups, self.cfg.norm_eps)
 
     def _mixer(self, layer: int, lw: LayerImage, proj: torch.Tensor, b: DeviceBatch, T: int) -> torch.Tensor:

@@ -196,7 +196,7 @@ class HeadScanArgs(C.Structure):
         ("states", C.c_void_p), ("seq_start", C.c_void_p), ("state_in", C.c_void_p), ("state_out", C.c_void_p),
         ("out", C.c_void_p), ("ldo", C.c_longlong), ("rows", C.c_int), ("n_seqs", C.c_int), ("heads", C.c_int),
         ("vdim", C.c_int), ("state", C.c_int), ("groups", C.c_int), ("n_states", C.c_int), ("fp32", C.c_int),
-        ("status", C.c_void_p),
+        ("long_seqs", C.c_int), ("by_token", C.c_int), ("status", C.c_void_p),
     ]
 
 

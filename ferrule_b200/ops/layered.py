@@ -321,9 +321,10 @@ def group_norm_rows(x: torch.Tensor, norm: torch.Tensor, out: torch.Tensor, dim:
 
 
 def head_scan(xbc: torch.Tensor, proj: torch.Tensor, off, mixer, img, states: torch.Tensor, seq_start: torch.Tensor,
-              state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, out: torch.Tensor) -> torch.Tensor:
+              state_in: torch.Tensor, state_out: torch.Tensor, n_seqs: int, out: torch.Tensor, long_seqs: int = 0,
+              by_token: bool = False) -> torch.Tensor:
     """(scan + D x) * silu(z) of a head-decay scan over packed rows: xbc the convolved x | B | C, z and dt blocks of the
-    projection."""
+    projection; long_seqs: sequences with more than one row, when known; by_token: prompts not in chunks."""
     assert states.dtype == torch.float32 and states.is_contiguous() and xbc.dtype == proj.dtype == out.dtype
     a = HeadScanArgs()
     item = proj.element_size()
@@ -333,6 +334,7 @@ def head_scan(xbc: torch.Tensor, proj: torch.Tensor, off, mixer, img, states: to
     a.states, a.n_states = states.data_ptr(), states.shape[0]
     a.seq_start, a.state_in, a.state_out = seq_start.data_ptr(), state_in.data_ptr(), state_out.data_ptr()
     a.out, a.ldo, a.rows, a.n_seqs, a.fp32 = out.data_ptr(), out.stride(0), xbc.shape[0], n_seqs, _fp32(xbc)
+    a.long_seqs, a.by_token = long_seqs, int(by_token)
     a.heads, a.vdim, a.state, a.groups = mixer.heads, mixer.vdim, mixer.state, mixer.groups
     a.status = status_tensor(xbc.device).data_ptr()
     check(get_lib(True).fb_head_scan(C.byref(a), stream_ptr()), "fb_head_scan")
