@@ -466,6 +466,7 @@ typedef struct FbGqaArgs {
   // kv heads side by side for every row); out then holds heads x value_width columns
   int value_width, value_stride;
   float softcap;            // > 0: score <- softcap tanh(score / softcap)
+  float score_bound;        // > 0: no scaled score is larger before the cap
   // blocks of `pool_tokens` tokens that lie wholly before a row's window are seen as one cache row each (see gqa_mask.cuh):
   // row b of sequence s is pooled[(slot_of[s] / slot_div) * pooled_stride + b]
   const void* pooled;       // [pooled_rows, pool_ld], element type of pool

@@ -376,43 +376,49 @@ gqa_attention_kernel(const GqaParams<T> p) {
     act_store(dst + d, res[d] * inv * (gate ? sigmoid_f(act_load(gate + d)) : 1.f));
 }
 
-// CTA = (row, kv head): outputs of all heads on the values of one kv head -> mixed outputs of that kv head's own heads
+// outputs of all heads on the values of one kv head -> mixed outputs of that kv head's own heads.  A thread takes 8 columns of a
+// row and kv head, for up to kVmHeads of its heads at a time.
+constexpr int kVmThreads = 256, kVmHeads = 4;
+
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kVmThreads)
 value_mix_kernel(const T* __restrict__ o, long long ldv, const float* __restrict__ talk, T* __restrict__ out, long long ldo,
-                 int heads, int kv_heads, int vp) {
+                 int rows, int heads, int kv_heads, int vp) {
   pdl_launch_dependents();
-  extern __shared__ float vm_sm[];               // [heads][vp] outputs, [per][heads] shares
-  const int per = heads / kv_heads, c = blockIdx.y, vecs = vp / 8;
-  const long long r = blockIdx.x;
-  float* share = vm_sm + heads * vp;
-  for (int i = threadIdx.x; i < per * heads; i += blockDim.x) share[i] = talk[c * per * heads + i];
-  pdl_wait();
-  for (int i = threadIdx.x; i < heads * vecs; i += blockDim.x) {
-    const int g = i / vecs, d = (i - g * vecs) * 8;
-    float x[8];
-    act_load8(o + r * ldv + (static_cast<long long>(g) * kv_heads + c) * vp + d, x);
-    act_store8(vm_sm + g * vp + d, x);
-  }
+  extern __shared__ float share[];               // [heads of the output][heads]
+  const int per = heads / kv_heads, vecs = vp / 8, blocks = (per + kVmHeads - 1) / kVmHeads;
+  for (int i = threadIdx.x; i < heads * heads; i += kVmThreads) share[i] = talk[i];
   __syncthreads();
-  for (int i = threadIdx.x; i < per * vecs; i += blockDim.x) {
-    const int h = i / vecs, d = (i - h * vecs) * 8;
-    float acc[8] = {};
+  pdl_wait();
+  const long long total = static_cast<long long>(rows) * kv_heads * vecs * blocks;
+  for (long long i = static_cast<long long>(blockIdx.x) * kVmThreads + threadIdx.x; i < total;
+       i += static_cast<long long>(gridDim.x) * kVmThreads) {
+    // neighbouring threads: columns, then kv heads, then blocks of heads, then rows
+    const long long t = i / vecs, u = t / kv_heads, r = u / blocks;
+    const int d = static_cast<int>(i - t * vecs) * 8, c = static_cast<int>(t - u * kv_heads), j0 = static_cast<int>(u - r * blocks) * kVmHeads;
+    const T* src = o + r * ldv + c * vp + d;
+    float acc[kVmHeads][8] = {};
+#pragma unroll 8
     for (int g = 0; g < heads; ++g) {
       float x[8];
-      act_load8(vm_sm + g * vp + d, x);
-      const float w = share[h * heads + g];
+      act_load8(src + static_cast<long long>(g) * kv_heads * vp, x);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) acc[j] = fmaf(w, x[j], acc[j]);
+      for (int h = 0; h < kVmHeads; ++h) {
+        const float w = share[(c * per + min(j0 + h, per - 1)) * heads + g];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[h][j] = fmaf(w, x[j], acc[h][j]);
+      }
     }
-    act_store8(out + r * ldo + static_cast<long long>(c * per + h) * vp + d, acc);
+#pragma unroll
+    for (int h = 0; h < kVmHeads; ++h)
+      if (j0 + h < per) act_store8(out + r * ldo + static_cast<long long>(c * per + j0 + h) * vp + d, acc[h]);
   }
 }
 
 template <typename T>
 static int launch_value_mix(const void* o, long long ldv, const float* talk, void* out, long long ldo, int rows, int heads,
                             int kv_heads, int vp, cudaStream_t s) {
-  const size_t smem = (static_cast<size_t>(heads) * vp + static_cast<size_t>(heads / kv_heads) * heads) * sizeof(float);
+  const size_t smem = static_cast<size_t>(heads) * heads * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;
   static bool attr = false;
   if (!attr) {
@@ -420,8 +426,10 @@ static int launch_value_mix(const void* o, long long ldv, const float* talk, voi
       return FB_ERR_LAUNCH;
     attr = true;
   }
-  launch_pdl(value_mix_kernel<T>, dim3(rows, kv_heads), dim3(128), smem, s, static_cast<const T*>(o), ldv, talk,
-             static_cast<T*>(out), ldo, heads, kv_heads, vp);
+  const int blocks = (heads / kv_heads + kVmHeads - 1) / kVmHeads;
+  const long long total = static_cast<long long>(rows) * kv_heads * (vp / 8) * blocks, ctas = (total + kVmThreads - 1) / kVmThreads;
+  launch_pdl(value_mix_kernel<T>, dim3(static_cast<unsigned>(ctas < 148 * 16 ? ctas : 148 * 16)), dim3(kVmThreads), smem, s,
+             static_cast<const T*>(o), ldv, talk, static_cast<T*>(out), ldo, rows, heads, kv_heads, vp);
   return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 

@@ -57,6 +57,7 @@ struct GpParams {
   int shared_values;
   PooledRows<__nv_bfloat16> pooled;
   float cap_log2, cap_in;              // soft cap: score2 = cap_log2 tanh(raw * cap_in / 2)
+  float cap_poly[6];                   // kGpBounded: coefficients of score2 in powers of (raw * cap_in / 2)^2, times that
   int kb, pieces, ks, q_resident;      // blocks per key stage, stages per token tile, key stages (2 or 4)
   int shared_keys, k_whole, v_whole;   // whole: one copy brings all feature blocks of a stage
   uint32_t tmem_cols;
@@ -69,7 +70,15 @@ struct GpParams {
 };
 
 constexpr float kLog2e = 1.4426950408889634f;
-enum { kGpPlain = 0, kGpBias = 1, kGpCap = 2 };       // what happens to the scores before the softmax
+// What happens to the scores before the softmax.  kGpBounded: a soft cap where the caller bounds the score by 0.7 of the cap:
+// tanh is then a polynomial (below), and as capped scores cannot leave [-cap, cap] no maximum is taken.
+enum { kGpPlain = 0, kGpBias = 1, kGpCap = 2, kGpBounded = 3 };
+constexpr float kGpMaxCap = 40.f;                      // exp(cap) times a long sum fits fp32 without a reference
+
+// tanh(u) = u p(u^2) for |u| <= 0.7: p interpolates tanh(sqrt(w)) / sqrt(w) at the six Chebyshev nodes of [0, 0.49]
+// (error below 1e-8, in fp32 below 1e-7)
+constexpr float kTanhPoly[6] = {1.f, -0.33333128690719604f, 0.13328377902507782f, -0.053523916751146317f, 0.02001960761845112f,
+                                -0.005084393545985222f};
 
 __device__ __forceinline__ float rcp_ftz(float x) {
   float y;
@@ -298,7 +307,7 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const uint64_t dv = umma_desc_mn128(v_addr + (j & 1) * vb * kGpKvBlock, kGpKvBlock);
 #pragma unroll
         for (int k = 0; k < 4; ++k)
-          umma_bf16_ts(tmem, tmem + col_s + (j & 1) * kGpKv + k * 8, dv + k * (2048 >> 4), idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
+          umma_bf16_ts(tmem, tmem + col_s + (j & 1) * kGpKv + (k >> 1) * 32 + (k & 1) * 8, dv + k * (2048 >> 4), idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
         umma_commit(v_free + (j & 1));
         if (j + 1 == n_kv) umma_commit(o_done);
       }
@@ -348,11 +357,31 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       }
       if (FORM == kGpCap) {
         // tanh as 1 - 2 / (exp(2 x) + 1)
+        const float cap_in2 = p.cap_in * kLog2e;
 #pragma unroll
         for (int c = 0; c < 2; ++c)
 #pragma unroll
           for (int i = 0; i < 16; ++i)
-            sv[c][i] = __float_as_uint(fmaf(-2.f * p.cap_log2, rcp_ftz(exp2_ftz(__uint_as_float(sv[c][i]) * p.cap_in) + 1.f), p.cap_log2));
+            sv[c][i] = __float_as_uint(fmaf(-2.f * p.cap_log2, rcp_ftz(exp2_ftz(__uint_as_float(sv[c][i]) * cap_in2) + 1.f), p.cap_log2));
+      }
+      if (FORM == kGpBounded) {
+        const uint64_t in2 = pack2(0.5f * p.cap_in, 0.5f * p.cap_in);
+        uint64_t c2[6];
+#pragma unroll
+        for (int e = 0; e < 6; ++e) c2[e] = pack2(p.cap_poly[e], p.cap_poly[e]);
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+          for (int i = 0; i < 16; i += 2) {
+            const uint64_t u = mul2(pack2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), in2), w = mul2(u, u);
+            uint64_t y = c2[5];
+#pragma unroll
+            for (int e = 4; e >= 0; --e) y = fma2(y, w, c2[e]);
+            float x0, x1;
+            unpack2(mul2(u, y), x0, x1);
+            sv[c][i] = __float_as_uint(x0);
+            sv[c][i + 1] = __float_as_uint(x1);
+          }
       }
       if (__all_sync(0xffffffffu, tok0 + 32 <= hi && (tok0 >= lo || tok0 + 32 <= keep))) {
 #pragma unroll
@@ -370,37 +399,39 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
             mx4[2 * c + (i & 1)] = fmaxf(mx4[2 * c + (i & 1)], x);
           }
       }
-      float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-      if (!READY) mx *= p.scale_log2;                         // the scale is positive
-      {
-        // both halves see the same two rounded maxima; behind the barrier both have read their scores
-        __nv_bfloat16* slot = max_x + (j & 1) * 256;
-        const __nv_bfloat16 mine = __float2bfloat16_ru(mx);
-        slot[half * 128 + r] = mine;
-        tc_fence_before();
-        pair_sync();
-        tc_fence_after();
-        mx = fmaxf(__bfloat162float(mine), __bfloat162float(slot[(half ^ 1) * 128 + r]));
-      }
-      const float m_new = fmaxf(m_ref, mx);
-      if (j == 0) {
-        m_ref = m_new;                                        // nothing accumulated yet
-      } else if (__any_sync(0xffffffffu, m_new > m_ref + 8.f)) {
-        // rescale this warp's share of 32 accumulator rows: the previous product must have retired
-        ok = mbar_wait(v_free + ((j - 1) & 1), ((j - 1) >> 1) & 1, abort_flag, p.status, 0xAB2) && ok;
-        __syncwarp();
-        tc_fence_after();
-        const float f = (m_new == -INFINITY) ? 1.f : exp2f(m_ref - m_new);
-        m_ref = m_new;
-        l_sum *= f;
+      if constexpr (FORM != kGpBounded) {
+        float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
+        if (!READY) mx *= p.scale_log2;                         // the scale is positive
+        {
+          // both halves see the same two rounded maxima; behind the barrier both have read their scores
+          __nv_bfloat16* slot = max_x + (j & 1) * 256;
+          const __nv_bfloat16 mine = __float2bfloat16_ru(mx);
+          slot[half * 128 + r] = mine;
+          tc_fence_before();
+          pair_sync();
+          tc_fence_after();
+          mx = fmaxf(__bfloat162float(mine), __bfloat162float(slot[(half ^ 1) * 128 + r]));
+        }
+        const float m_new = fmaxf(m_ref, mx);
+        if (j == 0) {
+          m_ref = m_new;                                        // nothing accumulated yet
+        } else if (__any_sync(0xffffffffu, m_new > m_ref + 8.f)) {
+          // rescale this warp's share of 32 accumulator rows: the previous product must have retired
+          ok = mbar_wait(v_free + ((j - 1) & 1), ((j - 1) >> 1) & 1, abort_flag, p.status, 0xAB2) && ok;
+          __syncwarp();
+          tc_fence_after();
+          const float f = (m_new == -INFINITY) ? 1.f : exp2f(m_ref - m_new);
+          m_ref = m_new;
+          l_sum *= f;
 #pragma unroll 1
-        for (int c = half; c < vb * 4; c += 2) {
-          uint32_t ov[16];
-          tmem_ld16(lane_base + c * 16, ov);
-          tmem_ld_wait();
+          for (int c = half; c < vb * 4; c += 2) {
+            uint32_t ov[16];
+            tmem_ld16(lane_base + c * 16, ov);
+            tmem_ld_wait();
 #pragma unroll
-          for (int i = 0; i < 16; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * f);
-          tmem_st16(lane_base + c * 16, ov);
+            for (int i = 0; i < 16; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * f);
+            tmem_st16(lane_base + c * 16, ov);
+          }
         }
       }
       const float m_use = (m_ref == -INFINITY) ? 0.f : m_ref;
@@ -411,13 +442,13 @@ gqa_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
       for (int i = 0; i < 16; ++i) {
         const uint64_t x = pack2(__uint_as_float(sv[i >> 3][(2 * i) & 15]), __uint_as_float(sv[i >> 3][((2 * i) & 15) + 1]));
         float p0, p1;
-        unpack2(READY ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
+        unpack2(FORM == kGpBounded ? x : READY ? add2(x, ref2) : fma2(x, scale2, ref2), p0, p1);
         p0 = exp2_ftz(p0);
         p1 = exp2_ftz(p1);
         add[i & 1] = add2(add[i & 1], pack2(p0, p1));
         pk[i] = pack_bf16x2(p0, p1);
       }
-      tmem_st16(s_t + half * 16, pk);
+      tmem_st16(s_t + half * 32, pk);                         // over this half's own scores
       float add_lo, add_hi;
       unpack2(add2(add[0], add[1]), add_lo, add_hi);
       l_sum += add_lo + add_hi;
@@ -602,7 +633,8 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
   p.scale_log2 = a->scale * kLog2e;
   if (a->softcap > 0.f) {
     p.cap_log2 = a->softcap * kLog2e;
-    p.cap_in = 2.f * p.scale_log2 / a->softcap;
+    p.cap_in = 2.f * a->scale / a->softcap;
+    for (int e = 0; e < 6; ++e) p.cap_poly[e] = p.cap_log2 * kTanhPoly[e];
   }
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.maps = a->maps; p.vdim = a->vdim;
@@ -634,6 +666,8 @@ extern "C" int fb_gqa_prefill_tc(const FbGqaArgs* a, const int* tiles, int n_til
     if (rc != FB_OK) return rc;
   }
   if (a->slopes) return launch_gp<kGpBias>(maps, p, n_tiles, slices, smem, stream);
+  if (a->softcap > 0.f && a->softcap <= kGpMaxCap && a->score_bound > 0.f && a->score_bound <= 0.7f * a->softcap)
+    return launch_gp<kGpBounded>(maps, p, n_tiles, slices, smem, stream);
   if (a->softcap > 0.f) return launch_gp<kGpCap>(maps, p, n_tiles, slices, smem, stream);
   return launch_gp<kGpPlain>(maps, p, n_tiles, slices, smem, stream);
 }

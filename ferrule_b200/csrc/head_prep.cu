@@ -30,6 +30,8 @@ struct PoolParams {
   DeviceStatus* status;
 };
 
+constexpr int kPoolBatch = 8;
+
 // the mean cache row of the block that ends with batch row r, if one does: eight columns per thread
 template <typename T>
 __device__ __forceinline__ void pool_block(const PoolParams<T>& p, int r) {
@@ -43,19 +45,30 @@ __device__ __forceinline__ void pool_block(const PoolParams<T>& p, int r) {
     if (threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xE30, r, pos);
     return;
   }
+  const int* pages = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+  const int t0 = pos + 1 - P;
   for (int c = threadIdx.x * 8; c < p.width; c += blockDim.x * 8) {
     float sum[8] = {};
-    for (int t = pos + 1 - P; t <= pos; ++t) {
-      const int page = p.block_table[static_cast<long long>(seq) * p.max_blocks + t / p.page_size];
-      const long long row = static_cast<long long>(page) * p.page_size + t % p.page_size;
-      if (page < 0 || row >= p.pool_rows) {
-        report_status(p.status, kStatusBadIndex, 0xE31, seq, t);
-        continue;
-      }
-      float x[8];
-      act_load8(p.pool + row * p.pool_ld + c, x);
+    for (int k = 0; k < P; k += kPoolBatch) {
+      // the rows of a batch are requested together (past the block's end: its last row again, not counted)
+      Raw8<T> raw[kPoolBatch];
+      bool ok[kPoolBatch];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) sum[j] += x[j];
+      for (int e = 0; e < kPoolBatch; ++e) {
+        const int t = min(t0 + k + e, pos), page = pages[t / p.page_size];
+        const long long row = static_cast<long long>(page) * p.page_size + t % p.page_size;
+        ok[e] = page >= 0 && row < p.pool_rows;
+        raw[e].load_written(p.pool + (ok[e] ? row : 0) * p.pool_ld + c);
+      }
+#pragma unroll
+      for (int e = 0; e < kPoolBatch; ++e) {
+        if (!ok[e]) report_status(p.status, kStatusBadIndex, 0xE31, seq, t0 + k + e);
+        const float w = ok[e] && k + e < P ? 1.f : 0.f;
+        float x[8];
+        raw[e].get(x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sum[j] = fmaf(w, x[j], sum[j]);
+      }
     }
 #pragma unroll
     for (int j = 0; j < 8; ++j) sum[j] /= P;
@@ -230,6 +243,97 @@ head_prep_kernel(const HeadPrepParams<T> p) {
   }
 }
 
+// The same without mixing, one map per head and rotations whose half is a multiple of 8, in registers: LPH lanes share a head, a lane
+// holds a pair of 8-element vectors that turn together, or one vector of the part that is not rotated.
+template <typename T, int LPH>
+__global__ void __launch_bounds__(kHpThreads)
+head_turn_kernel(const HeadPrepParams<T> p) {
+  pdl_launch_dependents();
+  const int pairs = p.half / 8, per_head = pairs + (p.dim_pad - 2 * p.half) / 8, heads = p.heads + p.kv_heads;
+  const int tid = threadIdx.x, v = tid % LPH;
+  const bool pair = v < pairs;
+  const int at = pair ? v * 8 : 2 * p.half + (v - pairs) * 8;                // first feature of this lane's vector
+  pdl_wait();
+  const long long r = blockIdx.x, slot = p.write_slot[r];
+  const bool keep = slot >= 0 && slot < p.pool_rows;
+  if (!keep && slot != -1 && tid == 0) report_status(p.status, kStatusBadIndex, 0xE22, r, static_cast<uint32_t>(slot));
+  T* row = p.pool + (keep ? slot : 0) * p.pool_ld;
+  float c[8] = {}, s[8] = {};
+  if (p.half) {
+    int pos = p.positions[r];
+    if (pos < 0 || pos >= p.max_pos) {
+      if (tid == 0) report_status(p.status, kStatusBadIndex, 0xE21, r, pos);
+      pos = 0;
+    }
+    if (pair) {
+      act_load8(p.cos_t + static_cast<long long>(pos) * p.half + at, c);
+      act_load8(p.sin_t + static_cast<long long>(pos) * p.half + at, s);
+    }
+  }
+  constexpr int kStep = kHpThreads / LPH;
+  for (int h0 = 0; h0 < heads; h0 += kStep) {
+    const int h = h0 + tid / LPH, hk = h - p.heads;
+    const bool is_q = hk < 0, in = h < heads && v < per_head;
+    const T* src = is_q ? p.q + r * p.ldp + h * p.dim_pad : p.k + r * p.ldp + hk * p.dim_pad;
+    const float* bias = is_q ? p.q_bias : p.k_bias;
+    const float* norm = is_q ? p.q_norm : p.k_norm;
+    float u[8] = {}, w[8] = {}, b[8];
+    if (in) {
+      act_load8(src + at, u);
+      if (pair) act_load8(src + at + p.half, w);
+      if (bias) {
+        bias += (is_q ? h : hk) * p.dim_pad + at;
+        act_load8(bias, b);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) u[j] += b[j];
+        if (pair) {
+          act_load8(bias + p.half, b);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) w[j] += b[j];
+        }
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(u[j], u[j], fmaf(w[j], w[j], ss));
+#pragma unroll
+    for (int o = 1; o < LPH; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!in || (!is_q && !keep)) continue;
+    const float f = 1.f / sqrtf(ss / p.dim + p.eps) * (is_q ? p.q_mix[h] : 1.f);
+    T* dst = (is_q ? p.q_out + r * p.ldqo + h * p.dim_pad : row + hk * p.dim_pad) + at;
+    float o[8], n[8];
+    // the norm's weights belong to the features behind the turn
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = (pair ? fmaf(u[j], c[j], -w[j] * s[j]) : u[j]) * f;
+    if (norm) {
+      act_load8(norm + at, n);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] *= n[j];
+    }
+    act_store8(dst, o);
+    if (!pair) continue;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = fmaf(w[j], c[j], u[j] * s[j]) * f;
+    if (norm) {
+      act_load8(norm + at + p.half, n);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] *= n[j];
+    }
+    act_store8(dst + p.half, o);
+  }
+  if (!keep) return;
+  T* vrow = row + p.kv_heads * p.dim_pad;
+  for (int e = tid * 8; e < p.kv_heads * p.vdim_pad; e += kHpThreads * 8) {
+    float x[8];
+    act_load8(p.v + r * p.ldp + e, x);
+    act_store8(vrow + e, x);
+  }
+  if (p.blocks.pooled) {
+    __syncthreads();                       // this step's own cache row is complete
+    pool_block(p.blocks, static_cast<int>(r));
+  }
+}
+
 template <typename T>
 static PoolParams<T> pool_params(const FbPoolArgs* a) {
   return {static_cast<const T*>(a->pool), a->pool_rows, a->pool_ld, static_cast<T*>(a->pooled), a->pooled_rows, a->positions,
@@ -255,6 +359,15 @@ static int run_head_prep(const FbHeadPrepArgs* a, cudaStream_t s) {
   p.status = static_cast<DeviceStatus*>(a->status);
   p.cos_t = a->cos_t; p.sin_t = a->sin_t; p.positions = a->positions; p.half = a->half; p.max_pos = a->max_pos;
   if (a->blocks) p.blocks = pool_params<T>(a->blocks);
+  const int lanes = a->half / 8 + (a->dim_pad - 2 * a->half) / 8;
+  if (!MIX && a->maps == 1 && a->v && a->half % 8 == 0 && lanes <= 32) {
+    const dim3 grid(a->rows), block(kHpThreads);
+    if (lanes <= 4) launch_pdl(head_turn_kernel<T, 4>, grid, block, 0, s, p);
+    else if (lanes <= 8) launch_pdl(head_turn_kernel<T, 8>, grid, block, 0, s, p);
+    else if (lanes <= 16) launch_pdl(head_turn_kernel<T, 16>, grid, block, 0, s, p);
+    else launch_pdl(head_turn_kernel<T, 32>, grid, block, 0, s, p);
+    return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+  }
   const size_t n = static_cast<size_t>(a->heads + a->kv_heads) * a->maps;
   const size_t smem = (n * a->dim_pad + n + (MIX ? static_cast<size_t>(a->heads) * a->heads : 2 * a->half)) * sizeof(float);
   if (smem > 200 * 1024) return FB_ERR_LIMIT;

@@ -194,7 +194,9 @@ __device__ __forceinline__ int checked_pos(int pos, int max_pos, int r, DeviceSt
   return 0;
 }
 
-template <typename T>
+constexpr int kLpVecs = 2;
+
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(const LatentPrepParams<T> p) {
   pdl_launch_dependents();
@@ -206,7 +208,66 @@ latent_prep_kernel(const LatentPrepParams<T> p) {
   if (!keep && slot != -1 && threadIdx.x == 0) report_status(p.status, kStatusBadIndex, 0xB31, r, static_cast<uint32_t>(slot));
   T* q = p.cq ? p.cq + r * p.ldp : nullptr;
   const T* c = p.ckv + r * p.ldp;
+  T* d = p.pool + (keep ? slot : 0) * p.row_dim;
+  const int half = p.rot / 2;
   float sq = 0.f, sc = 0.f;
+  if constexpr (VEC) {
+    // widths are multiples of 8: a thread holds up to kLpVecs vectors of the query latent and one of everything else
+    float x[kLpVecs][8], y[8], o[8];
+#pragma unroll
+    for (int k = 0; k < kLpVecs; ++k) {
+      const int i = (k * 256 + threadIdx.x) * 8;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[k][j] = 0.f;
+      if (q && i < p.rank_q) act_load8(q + i, x[k]);
+    }
+    const int i = threadIdx.x * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) y[j] = 0.f;
+    if (i < p.rank + p.rot) act_load8(c + i, y);
+#pragma unroll
+    for (int k = 0; k < kLpVecs; ++k)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sq = fmaf(x[k][j], x[k][j], sq);
+    if (i < p.rank)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) sc = fmaf(y[j], y[j], sc);
+    sq = cta_sum(sq, red[0]);
+    sc = cta_sum(sc, red[1]);
+    const float fq = q ? 1.f / sqrtf(sq / p.rank_q + p.eps) : 0.f, fc = 1.f / sqrtf(sc / p.rank + p.eps);
+#pragma unroll
+    for (int k = 0; k < kLpVecs; ++k) {
+      const int e = (k * 256 + threadIdx.x) * 8;
+      if (!q || e >= p.rank_q) continue;
+      act_load8(p.q_w + e, o);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] *= x[k][j] * fq;
+      act_store8(q + e, o);
+    }
+    if (!keep) return;
+    if (i < p.rank) {
+      act_load8(p.kv_w + i, o);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o[j] *= y[j] * fc;
+      act_store8(d + i, o);
+    } else if (i < p.rank + p.rot) {
+      const long long t = static_cast<long long>(pos) * half + (i - p.rank) / 2;
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        const float cs = p.cos_t[t + j / 2], sn = p.sin_t[t + j / 2];
+        o[j] = y[j] * cs - y[j + 1] * sn;
+        o[j + 1] = y[j + 1] * cs + y[j] * sn;
+      }
+      act_store8(d + p.rot_off + i - p.rank, o);
+    }
+    // padding columns
+#pragma unroll
+    for (int j = 0; j < 8; ++j) o[j] = 0.f;
+    const int gap = p.rot_off - p.rank, end = p.rot_off + p.rot;
+    if (p.rot && i < gap) act_store8(d + p.rank + i, o);
+    if (end + i < p.row_dim) act_store8(d + end + i, o);
+    return;
+  }
   if (q)
     for (int i = threadIdx.x; i < p.rank_q; i += blockDim.x) {
       const float v = act_load(q + i);
@@ -224,8 +285,6 @@ latent_prep_kernel(const LatentPrepParams<T> p) {
   }
   if (!keep) return;
   const float f = 1.f / sqrtf(sc / p.rank + p.eps);
-  T* d = p.pool + slot * p.row_dim;
-  const int half = p.rot / 2;
   for (int i = threadIdx.x; i < p.row_dim; i += blockDim.x) {
     const int e = i - p.rot_off;
     if (i < p.rank) {
@@ -463,7 +522,12 @@ static int launch_latent_prep(const FbLatentPrepArgs* a, cudaStream_t s) {
   LatentPrepParams<T> p{static_cast<T*>(a->cq), static_cast<const T*>(a->ckv), a->ldp, a->rank_q, a->rank, a->rot, a->row_dim,
                         a->rot_off, a->q_w, a->kv_w, a->cos_t, a->sin_t, a->max_pos, a->positions, a->write_slot,
                         static_cast<T*>(a->pool), a->pool_rows, a->eps, static_cast<DeviceStatus*>(a->status)};
-  launch_pdl(latent_prep_kernel<T>, dim3(a->rows), dim3(256), 0, s, p);
+  const bool vec = a->rank % 8 == 0 && a->rot % 8 == 0 && a->rot_off % 8 == 0 && a->row_dim % 8 == 0 && a->ldp % 8 == 0 &&
+                   a->rank + a->rot <= 2048 && a->row_dim <= 2048 &&
+                   (!a->cq || (a->rank_q % 8 == 0 && a->rank_q <= kLpVecs * 2048)) && aligned16(a->cq) && aligned16(a->ckv) &&
+                   aligned16(a->q_w) && aligned16(a->kv_w) && aligned16(a->pool);
+  if (vec) launch_pdl(latent_prep_kernel<T, true>, dim3(a->rows), dim3(256), 0, s, p);
+  else launch_pdl(latent_prep_kernel<T, false>, dim3(a->rows), dim3(256), 0, s, p);
   return ok_launch();
 }
 

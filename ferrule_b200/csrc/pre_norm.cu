@@ -17,7 +17,7 @@
 
 namespace fb {
 
-constexpr int kShiftRows = 8;
+constexpr int kShiftRows = 4;
 
 template <typename T>
 struct PreNormParams {

@@ -405,32 +405,6 @@ __device__ __forceinline__ bool conv_row(const ConvParams<TI, TO>& p, int r, int
   return true;
 }
 
-// eight elements as they lie in memory
-template <typename T>
-struct Raw8;
-template <>
-struct Raw8<__nv_bfloat16> {
-  uint4 a;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { a = __ldg(reinterpret_cast<const uint4*>(p)); }
-  __device__ __forceinline__ void get(float (&v)[8]) const {
-    const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&a);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = __bfloat162float(e[j]);
-  }
-};
-template <>
-struct Raw8<float> {
-  float4 a, b;
-  __device__ __forceinline__ void load(const float* p) {
-    a = __ldg(reinterpret_cast<const float4*>(p));
-    b = __ldg(reinterpret_cast<const float4*>(p) + 1);
-  }
-  __device__ __forceinline__ void get(float (&v)[8]) const {
-    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
-    v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-  }
-};
-
 // ROWS consecutive rows x 8 channels per thread; KEEP = taps - 1 when it is at most 3 (the inputs of all rows are
 // requested together), -1: any number of taps
 template <typename TI, typename TO, int KEEP, int ROWS, bool RESIDUAL, bool SILU>

@@ -104,7 +104,7 @@ class AttentionMixer:
     kind = "attention"
     maps = 1
     window = keep_first = pool = 0
-    softcap = 0.0
+    softcap = score_bound = 0.0
     shared_keys = shared_values = scaled_queries = False
 
     @property
@@ -180,6 +180,12 @@ class WindowMixer:
         """Every query row meets the keys of all kv heads side by side: sum_g T[h, g] q_g . k_kv(g) is one product of a
         mixed query with the concatenated keys."""
         return self.mix_heads
+
+    @property
+    def score_bound(self) -> float:
+        """No scaled score is larger (0: unknown): without norm weights queries and keys have the length sqrt(dim), means of
+        keys are not longer.  (Rounding them to bf16 adds at most a hundredth.)"""
+        return 0.0 if self.norm_weights or self.mix_heads else 1.01 * self.dim * abs(self.scale)
 
     @property
     def shared_values(self) -> bool:

@@ -161,7 +161,7 @@ class GqaArgs(C.Structure):
         ("key_stride", C.c_int), ("v_offset", C.c_int), ("window", C.c_int), ("keep_first", C.c_int),
         ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ldg", C.c_longlong), ("diff_lambda", C.c_float),
         ("diff_scale", C.c_float), ("value_width", C.c_int), ("value_stride", C.c_int), ("softcap", C.c_float),
-        ("pooled", C.c_void_p), ("pooled_rows", C.c_longlong), ("pool_tokens", C.c_int), ("pooled_stride", C.c_int),
+        ("score_bound", C.c_float), ("pooled", C.c_void_p), ("pooled_rows", C.c_longlong), ("pool_tokens", C.c_int), ("pooled_stride", C.c_int),
         ("slot_div", C.c_int), ("slot_of", C.c_void_p), ("talk", C.c_void_p), ("status", C.c_void_p),
     ]
 

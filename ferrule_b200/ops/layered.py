@@ -394,7 +394,7 @@ def _gqa(q: torch.Tensor, mixer, pool: torch.Tensor, slopes: Optional[torch.Tens
     a.slopes, a.eps, a.diff_lambda = ptr(slopes), eps, diff_lambda
     a.diff_scale = 1.0 - mixer.diff if mixer.maps == 2 else 1.0
     a.value_width, a.value_stride = mixer.value_width, 0 if mixer.shared_values else mixer.vdim_pad
-    a.softcap, a.talk = mixer.softcap, ptr(talk)
+    a.softcap, a.score_bound, a.talk = mixer.softcap, mixer.score_bound, ptr(talk)
     if mean is not None:
         rows, a.slot_div, slots = mean
         assert rows.dtype == q.dtype and rows.is_contiguous() and rows.shape[2] == pool.shape[-1]

@@ -271,7 +271,8 @@ def test_mean_rows_of_blocks(ops, dtype, page, P):
 # ------------------------------------------------------------------ attention with pooled blocks and mixed weights
 ATTENTIONS = [pooled(6, 3, 20, 12, 0.3, 9, 4), pooled(1, 1, 64, 40, 0.3, 1, 1), pooled(8, 2, 128, 128, 0.3, 70, 16),
               pooled(20, 4, 40, 16, 0.3, 130, 7), pooled(16, 4, 128, 128, 0.3, 64, 5, softcap=30.0), pooled(6, 2, 64, 80, 0.3, 17, 40),
-              pooled(40, 2, 24, 64, 0.3, 33, 3), pooled(4, 4, 72, 136, 0.3, 20, 64, softcap=0.0), pooled(3, 3, 16, 200, 0.3, 300, 2)]
+              pooled(40, 2, 24, 64, 0.3, 33, 3), pooled(4, 4, 72, 136, 0.3, 20, 64, softcap=0.0), pooled(3, 3, 16, 200, 0.3, 300, 2),
+              pooled(12, 3, 48, 48, 0.2, 100, 16, softcap=20.0)]
 
 
 def attention_case(m, dtype, page, lens, rows=None, seed=0):
@@ -292,7 +293,10 @@ def attention_case(m, dtype, page, lens, rows=None, seed=0):
                                 | {n - 1}) if 0 <= p < n]
     H, G, D, V, dp, vp = m.heads, m.kv_heads, m.dim, m.vdim, m.dim_pad, m.vdim_pad
     pool = torch.zeros(sum(per) + 3, page, m.row_dim + 8, dtype=dtype, device="cuda")
-    pool[..., :G * dp].unflatten(2, (G, dp))[..., :D] = rnd(*pool.shape[:2], G, D, dtype=dtype)
+    # a kernel may rely on a bound of the scores that the norms of queries and keys give: such mixers get normalised ones
+    bounded = 0 < m.score_bound <= 0.7 * m.softcap
+    keys = rnd(*pool.shape[:2], G, D)
+    pool[..., :G * dp].unflatten(2, (G, dp))[..., :D] = (VO.rms(keys, 0.0) if bounded else keys).to(dtype)
     pool[..., m.v_offset:m.v_offset + G * vp].unflatten(2, (G, vp))[..., :V] = rnd(*pool.shape[:2], G, V, dtype=dtype, seed=1)
     flat, img = dbl(pool).flatten(0, 1), Img(m)
     slot = lambda s, t: int(table[s, t // page]) * page + t % page
@@ -316,6 +320,8 @@ def attention_case(m, dtype, page, lens, rows=None, seed=0):
                 kv = h // (H // G)
                 t = t[kv * dp:kv * dp + D]
                 q[i, h] = t * (8.0 / float(t.norm() ** 2))
+        if bounded:
+            q[i] *= D ** 0.5 * m.scale / q[i].norm(dim=-1, keepdim=True)
         qi = q[i].to(dtype).double()
         kv = torch.cat([means[n - 1 - s, :blocks], flat[[slot(s, t) for t in range(lo, p + 1)]]])
         w = []
