@@ -245,7 +245,7 @@ head_prep_kernel(const HeadPrepParams<T> p) {
 
 // The same without mixing, one map per head and rotations whose half is a multiple of 8, in registers: LPH lanes share a head, a lane
 // holds a pair of 8-element vectors that turn together, or one vector of the part that is not rotated.
-template <typename T, int LPH>
+template <typename T, int LPH, bool BLOCKS>
 __global__ void __launch_bounds__(kHpThreads)
 head_turn_kernel(const HeadPrepParams<T> p) {
   pdl_launch_dependents();
@@ -328,10 +328,17 @@ head_turn_kernel(const HeadPrepParams<T> p) {
     act_load8(p.v + r * p.ldp + e, x);
     act_store8(vrow + e, x);
   }
-  if (p.blocks.pooled) {
+  if constexpr (BLOCKS) {
     __syncthreads();                       // this step's own cache row is complete
     pool_block(p.blocks, static_cast<int>(r));
   }
+}
+
+template <typename T, int LPH>
+static int launch_head_turn(const HeadPrepParams<T>& p, int rows, cudaStream_t s) {
+  if (p.blocks.pooled) launch_pdl(head_turn_kernel<T, LPH, true>, dim3(rows), dim3(kHpThreads), 0, s, p);
+  else launch_pdl(head_turn_kernel<T, LPH, false>, dim3(rows), dim3(kHpThreads), 0, s, p);
+  return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
 }
 
 template <typename T>
@@ -361,12 +368,10 @@ static int run_head_prep(const FbHeadPrepArgs* a, cudaStream_t s) {
   if (a->blocks) p.blocks = pool_params<T>(a->blocks);
   const int lanes = a->half / 8 + (a->dim_pad - 2 * a->half) / 8;
   if (!MIX && a->maps == 1 && a->v && a->half % 8 == 0 && lanes <= 32) {
-    const dim3 grid(a->rows), block(kHpThreads);
-    if (lanes <= 4) launch_pdl(head_turn_kernel<T, 4>, grid, block, 0, s, p);
-    else if (lanes <= 8) launch_pdl(head_turn_kernel<T, 8>, grid, block, 0, s, p);
-    else if (lanes <= 16) launch_pdl(head_turn_kernel<T, 16>, grid, block, 0, s, p);
-    else launch_pdl(head_turn_kernel<T, 32>, grid, block, 0, s, p);
-    return cudaGetLastError() == cudaSuccess ? FB_OK : FB_ERR_LAUNCH;
+    if (lanes <= 4) return launch_head_turn<T, 4>(p, a->rows, s);
+    if (lanes <= 8) return launch_head_turn<T, 8>(p, a->rows, s);
+    if (lanes <= 16) return launch_head_turn<T, 16>(p, a->rows, s);
+    return launch_head_turn<T, 32>(p, a->rows, s);
   }
   const size_t n = static_cast<size_t>(a->heads + a->kv_heads) * a->maps;
   const size_t smem = (n * a->dim_pad + n + (MIX ? static_cast<size_t>(a->heads) * a->heads : 2 * a->half)) * sizeof(float);
