@@ -482,10 +482,10 @@ int fb_gqa_attention(const FbGqaArgs* args, void* stream);      // vdim <= 512
 // bf16, few rows (gqa_decode.cu): key_width, vdim <= 256, key_stride > 0; the visible keys of a row are divided among `splits` (1, 2, 4, 8) CTAs;
 // early: one row per sequence, keys below a row's own position predate the preceding kernel
 int fb_gqa_decode(const FbGqaArgs* args, int splits, int early, void* stream);
-// the same for keys that all heads share (gqa_decode_wide.cu): key_stride 0, one map; fb_gqa_decode_wide_ok: whether
-// cache rows of this shape fit its pipeline
+// the same for keys (key_stride 0) or values (value_stride 0, with talk) that all heads share (gqa_decode_wide.cu), one map;
+// fb_gqa_decode_wide_ok: whether cache rows of this shape fit its pipeline (key_width of a query row; own_keys: key_stride > 0)
 int fb_gqa_decode_wide(const FbGqaArgs* args, int splits, int early, void* stream);
-int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads);
+int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads, int own_keys);
 // out[row, h] = sum_g talk[h, g] o[row, g, columns of h's kv head]: o rows hold heads x kv_heads x vdim_pad columns
 int fb_value_mix(const void* o, long long ldv, const float* talk, void* out, long long ldo, int rows, int heads, int kv_heads,
                  int vdim_pad, int fp32, void* stream);

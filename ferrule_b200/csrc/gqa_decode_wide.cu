@@ -4,8 +4,8 @@
 // Scores that are mixed across heads are products of one wide query row per head with the concatenated keys of a token
 // (head_prep.cu), so a CTA takes all of a token's cache row: keys and values of every kv head lie side by side there and come
 // as one bulk copy per token.  Softmax weights that are mixed across heads need every head's weights on the values of every kv
-// head: the same rows, queries as wide as one kv head's keys (zero in the other kv heads' columns), and the outputs are mixed
-// when the splits have met.  Mean rows of the blocks before the window (gqa_mask.cuh) are keys like any other.  CTA = (query row, split of the visible keys, block of 16 heads); a tile is KT tokens.
+// head: the keys of the CTA's own kv heads (a query is zero in the others' columns) and all values, and every CTA mixes its outputs
+// before the cluster adds them up.  Mean rows of the blocks before the window (gqa_mask.cuh) are keys like any other.  CTA = (query row, split of the visible keys, block of 16 heads); a tile is KT tokens.
 //
 //   copies   warp 8 looks up a token per lane and keeps all stages requested
 //   scores   warp w of 8 multiplies the 16 query rows with 8 of the tile's keys over a share of the features (MMA, partial
@@ -48,7 +48,9 @@ struct GwParams {
   __nv_bfloat16* out;
   long long ldo;
   int heads, kv_heads, key_width, vdim_pad;
-  int own_keys;                                    // > 0: a query row is this wide and meets the keys of its kv head
+  int own_keys;                                    // > 0: a query row is this wide and meets the keys of its kv head; key_width
+                                                   //   is then that of the most kv heads a block of 16 heads has
+  int v_offset;                                    // first value column of a cache row in memory
   float cap_log2, cap_in;                          // soft cap: score2 <- cap_log2 tanh(raw * cap_in / 2); 0: none
   PooledRows<__nv_bfloat16> pooled;
   const float* talk;
@@ -59,14 +61,15 @@ struct GwParams {
 
 // shared memory behind the tiles
 struct GwLayout {
-  int q_pitch, q, part, prob, factor, bars, total;
-  __host__ __device__ GwLayout(int key_width, int tile_bytes, int kt) {
+  int q_pitch, q, part, prob, factor, talk, bars, total;
+  __host__ __device__ GwLayout(int key_width, int tile_bytes, int kt, int talk_heads) {
     q_pitch = (key_width + 15) / 16 * 16 + 8;
     q = tile_bytes;
     part = q + 16 * q_pitch * 2;
     prob = part + (64 / kt) * 16 * (kt + 1) * 4;
     factor = prob + 16 * (kt + 8) * 2;
-    bars = factor + 48 * 4;
+    talk = factor + 48 * 4;
+    bars = talk + talk_heads * 16 * 4;
     total = bars + (2 * kGwMaxStages + 1) * 8;
   }
 };
@@ -91,13 +94,14 @@ gqa_decode_wide_kernel(const GwParams p) {
   pdl_launch_dependents();
   extern __shared__ __align__(128) uint8_t gw_sm[];
   const int tile_bytes = KT * p.pitch;
-  const GwLayout at(p.key_width, p.stages * tile_bytes, KT);
+  const GwLayout at(p.key_width, p.stages * tile_bytes, KT, p.talk ? p.heads : 0);
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(gw_sm + at.q);
   float* part_s = reinterpret_cast<float*>(gw_sm + at.part);               // [kShares][16][KT + 1]
   __nv_bfloat16* prob_s = reinterpret_cast<__nv_bfloat16*>(gw_sm + at.prob);   // [16][KT + 8]
   float* f_s = reinterpret_cast<float*>(gw_sm + at.factor);                // [16] rescale factors
   float* c_m = f_s + 16;
   float* c_l = c_m + 16;
+  float* talk_s = reinterpret_cast<float*>(gw_sm + at.talk);                // [heads][16]: shares of this block's heads
   uint64_t* full = reinterpret_cast<uint64_t*>(gw_sm + at.bars);
   uint64_t* empty = full + kGwMaxStages;
   volatile uint32_t* abort_flag = reinterpret_cast<volatile uint32_t*>(empty + kGwMaxStages);
@@ -125,7 +129,13 @@ gqa_decode_wide_kernel(const GwParams p) {
     hi = min(lo + share * KT, n_keys);
   }
   const int n_tiles = (hi - lo + KT - 1) / KT;
+  // columns of this block's keys
+  const int g0 = p.own_keys > 0 ? h0 / per : 0;
+  const int width = p.own_keys > 0 ? ((h0 + nh - 1) / per - g0 + 1) * p.own_keys : p.key_width;
   auto token = [&](int i) { return i < kept ? i : first + i - kept; };
+  if (p.talk)
+    for (int i = tid; i < p.heads * 16; i += blockDim.x)
+      talk_s[i] = (i & 15) < nh ? p.talk[static_cast<long long>(i >> 4) * p.heads + h0 + (i & 15)] : 0.f;
   if (tid == 0) {
     for (int i = 0; i < p.stages; ++i) {
       mbar_init(full + i, 1);
@@ -170,11 +180,21 @@ gqa_decode_wide_kernel(const GwParams p) {
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
       }
-      if (lane == 0) mbar_arrive_expect_tx(full + st, static_cast<uint32_t>(KT * p.row_bytes));
+      // fewer keys than there is room for: whole k-steps (queries are zero in the columns that follow, values have to be finite)
+      const uint32_t key_bytes = (width < p.key_width ? (width + 15) / 16 * 16 : width) * 2;
+      const uint32_t value_bytes = p.row_bytes - p.key_width * 2;
+      if (lane == 0) mbar_arrive_expect_tx(full + st, KT * (key_bytes + value_bytes));
       __syncwarp();
-      if (lane < KT)
-        gw_copy_row(gw_sm + st * tile_bytes + lane * p.pitch, rows + slot * p.pool_ld, static_cast<uint32_t>(p.row_bytes),
-                    full + st);
+      if (lane < KT) {
+        uint8_t* dst = gw_sm + st * tile_bytes + lane * p.pitch;
+        const __nv_bfloat16* src = rows + slot * p.pool_ld;
+        if (width == p.v_offset) {
+          gw_copy_row(dst, src, key_bytes + value_bytes, full + st);
+        } else {
+          gw_copy_row(dst, src + g0 * p.own_keys, key_bytes, full + st);
+          gw_copy_row(dst + p.key_width * 2, src + p.v_offset, value_bytes, full + st);
+        }
+      }
     }
     if (!waited) pdl_wait();
     if (*abort_flag) {
@@ -192,7 +212,7 @@ gqa_decode_wide_kernel(const GwParams p) {
       const int row = i / (at.q_pitch / 8), c = (i - row * (at.q_pitch / 8)) * 8;
       uint4 v = make_uint4(0u, 0u, 0u, 0u);
       if (p.own_keys > 0) {
-        const int e = c - (h0 + row) / per * p.own_keys;
+        const int e = c - ((h0 + row) / per - g0) * p.own_keys;
         if (row < nh && e >= 0 && e < p.own_keys)
           v = *reinterpret_cast<const uint4*>(p.q + r * p.ldq + static_cast<long long>(h0 + row) * p.own_keys + e);
       } else if (row < nh && c < p.key_width) {
@@ -206,7 +226,7 @@ gqa_decode_wide_kernel(const GwParams p) {
       const int row = 2 * warp + k;
       sl[k] = p.slopes && row < nh ? p.slopes[h0 + row] * 1.4426950408889634f : 0.f;
     }
-    const int ksteps = (p.key_width + 15) / 16, share = (ksteps + kShares - 1) / kShares;
+    const int ksteps = (width + 15) / 16, share = (ksteps + kShares - 1) / kShares;
     const int nt = warp % kNt, part = warp / kNt, k0 = min(part * share, ksteps), k1 = min(k0 + share, ksteps);
     const uint32_t qa = smem_u32(q_s + (lane & 15) * at.q_pitch + (lane >> 4) * 8);
     gw_sync();
@@ -370,59 +390,55 @@ gqa_decode_wide_kernel(const GwParams p) {
   const bool cluster = splits > 1 || (p.talk && p.head_blocks > 1);
   if (cluster) cluster_sync_all();
   else __syncthreads();
-  // rank of the CTA with split s of head block z in this cluster
-  auto peer = [&](int s, int z) { return static_cast<uint32_t>(s + z * splits); };
-  // columns d .. d + 3 of a row's normalised output over all splits
-  auto merged = [&](int row, int d) {
-    const int z = p.talk ? static_cast<int>(blockIdx.z) : 0;
-    float mm = -INFINITY, ll = 0.f;
-    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (splits == 1) {
-      ll = c_l[row];
-      a = *reinterpret_cast<const float4*>(o_s + row * o_pitch + d);
-    } else {
-      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + row), peer(s, z))));
-      for (int s = 0; s < splits; ++s) {
-        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + row), peer(s, z)));
-        const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
-        ll = fmaf(f, ld_cluster_f32(mapa_shared(smem_u32(c_l + row), peer(s, z))), ll);
-        const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(o_s + row * o_pitch + d), peer(s, z)));
-        a.x = fmaf(f, v.x, a.x);
-        a.y = fmaf(f, v.y, a.y);
-        a.z = fmaf(f, v.z, a.z);
-        a.w = fmaf(f, v.w, a.w);
-      }
-    }
-    const float inv = ll > 0.f ? 1.f / ll : 0.f;
-    return make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
-  };
   const int quads = p.vdim_pad / 4;
   if (p.talk) {
-    // This CTA's share of the columns: merged in place (peers read other columns of this CTA), then heads are mixed.
-    const int all = n_cols * 4, share = (all + splits - 1) / splits, q0 = min(split * share, all), q1 = min(q0 + share, all);
-    for (int i = tid; i < nh * (q1 - q0); i += blockDim.x) {
-      const int row = i / (q1 - q0), d = (q0 + i - row * (q1 - q0)) * 4;
-      *reinterpret_cast<float4*>(o_s + row * o_pitch + d) = merged(row, d);
+    // Mixing is linear, so every CTA mixes what it has - its rows and its keys, weighted as the whole row's softmax says - and
+    // the cluster adds these up.
+    const int z = static_cast<int>(blockIdx.z), all = n_cols * 4, ctas = splits * p.head_blocks;
+    if (tid < 16 && splits > 1) {
+      float mm = -INFINITY, ll = 0.f;
+      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + tid), s + z * splits)));
+      for (int s = 0; s < splits; ++s) {
+        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + tid), s + z * splits));
+        ll = fmaf(ms == -INFINITY ? 0.f : exp2f(ms - mm), ld_cluster_f32(mapa_shared(smem_u32(c_l + tid), s + z * splits)), ll);
+      }
+      f_s[tid] = c_m[tid] == -INFINITY || !(ll > 0.f) ? 0.f : exp2f(c_m[tid] - mm) / ll;
+    } else if (tid < 16) {
+      f_s[tid] = c_l[tid] > 0.f ? 1.f / c_l[tid] : 0.f;
     }
-    if (p.head_blocks > 1) cluster_sync_all();
-    else __syncthreads();
-    for (int i = tid; i < per * (q1 - q0); i += blockDim.x) {
-      const int j = i / (q1 - q0), at = (q0 + i - j * (q1 - q0)) * 4, g = at / (vcols * 16), d = at - g * vcols * 16;
-      const int h = g * per + j;
-      if (d >= p.vdim_pad || h < h0 || h >= h0 + nh) continue;
-      const float* t = p.talk + static_cast<long long>(h) * p.heads;
+    __syncthreads();
+    for (int i = tid; i < p.heads * 16; i += blockDim.x) talk_s[i] *= (i & 15) < nh ? f_s[i & 15] : 0.f;
+    __syncthreads();
+    float* mix_s = o_s + 16 * o_pitch;                                     // [per][all columns]
+    for (int i = tid; i < per * all; i += blockDim.x) {
+      const int j = i / all, col = (i - j * all) * 4, h = col / (vcols * 16) * per + j;
+      const float* t = talk_s + h * 16;
       float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int z = 0; z < p.head_blocks; ++z) {
-        const int n = min(16, p.heads - z * 16);
-        for (int row = 0; row < n; ++row) {
-          const float* src = o_s + row * o_pitch + at;
-          const float4 v = z == static_cast<int>(blockIdx.z) ? *reinterpret_cast<const float4*>(src)
-                                                               : ld_cluster_f32x4(mapa_shared(smem_u32(src), peer(split, z)));
-          const float w = t[z * 16 + row];
-          a.x = fmaf(w, v.x, a.x);
-          a.y = fmaf(w, v.y, a.y);
-          a.z = fmaf(w, v.z, a.z);
-          a.w = fmaf(w, v.w, a.w);
+      for (int row = 0; row < nh; ++row) {
+        const float4 v = *reinterpret_cast<const float4*>(o_s + row * o_pitch + col);
+        const float w = t[row];
+        a.x = fmaf(w, v.x, a.x);
+        a.y = fmaf(w, v.y, a.y);
+        a.z = fmaf(w, v.z, a.z);
+        a.w = fmaf(w, v.w, a.w);
+      }
+      *reinterpret_cast<float4*>(mix_s + j * all * 4 + col) = a;
+    }
+    if (cluster) cluster_sync_all();
+    else __syncthreads();
+    for (int i = tid + (split + z * splits) * blockDim.x; i < p.heads * quads; i += blockDim.x * ctas) {
+      const int h = i / quads, d = (i - h * quads) * 4, c = h / per;
+      const float* src = mix_s + (h - c * per) * all * 4 + c * vcols * 16 + d;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (!cluster) {
+        a = *reinterpret_cast<const float4*>(src);
+      } else {
+        for (int k = 0; k < ctas; ++k) {
+          const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(src), k));
+          a.x += v.x;
+          a.y += v.y;
+          a.z += v.z;
+          a.w += v.w;
         }
       }
       __nv_bfloat16* dst = p.out + r * p.ldo + static_cast<long long>(h) * p.vdim_pad + d;
@@ -432,6 +448,29 @@ gqa_decode_wide_kernel(const GwParams p) {
     if (cluster) cluster_sync_all();                                       // no CTA leaves while a peer reads its rows
     return;
   }
+  // columns d .. d + 3 of a row's normalised output over all splits
+  auto merged = [&](int row, int d) {
+    float mm = -INFINITY, ll = 0.f;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (splits == 1) {
+      ll = c_l[row];
+      a = *reinterpret_cast<const float4*>(o_s + row * o_pitch + d);
+    } else {
+      for (int s = 0; s < splits; ++s) mm = fmaxf(mm, ld_cluster_f32(mapa_shared(smem_u32(c_m + row), s)));
+      for (int s = 0; s < splits; ++s) {
+        const float ms = ld_cluster_f32(mapa_shared(smem_u32(c_m + row), s));
+        const float f = ms == -INFINITY ? 0.f : exp2f(ms - mm);
+        ll = fmaf(f, ld_cluster_f32(mapa_shared(smem_u32(c_l + row), s)), ll);
+        const float4 v = ld_cluster_f32x4(mapa_shared(smem_u32(o_s + row * o_pitch + d), s));
+        a.x = fmaf(f, v.x, a.x);
+        a.y = fmaf(f, v.y, a.y);
+        a.z = fmaf(f, v.z, a.z);
+        a.w = fmaf(f, v.w, a.w);
+      }
+    }
+    const float inv = ll > 0.f ? 1.f / ll : 0.f;
+    return make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+  };
   for (int i = tid + split * blockDim.x; i < nh * quads; i += blockDim.x * splits) {
     const int h = i / quads, d = (i - h * quads) * 4;
     float4 a = merged(h, d);
@@ -452,14 +491,15 @@ gqa_decode_wide_kernel(const GwParams p) {
 struct GwPlan {
   int kt, stages, nc, kq;
 };
-static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad, bool shared_values) {
+static GwPlan gw_plan(int key_width, int kv_heads, int vdim_pad, bool shared_values, int heads) {
   const int vcols = (vdim_pad + 15) / 16, cols = kv_heads * vcols, pitch = (key_width + kv_heads * vdim_pad) * 2 + 16;
   const int nc = cols <= 8 ? 1 : cols <= 16 ? 2 : cols <= 32 ? 4 : cols <= 64 ? 8 : 0;
   for (int kt = 32; kt >= 16 && nc; kt /= 2) {
-    int stages = (kGwSmemLimit - GwLayout(key_width, 0, kt).total) / (kt * pitch);
+    int stages = (kGwSmemLimit - GwLayout(key_width, 0, kt, shared_values ? heads : 0).total) / (kt * pitch);
     if (stages > kGwMaxStages) stages = kGwMaxStages;
-    // the merged outputs reuse the tiles' memory
-    if (stages < 2 || stages * kt * pitch < 16 * ((shared_values ? cols : vcols) * 16 + 4) * 4) continue;
+    // the outputs reuse the tiles' memory: with shared values all columns, and the mixed ones of every head
+    const long long outputs = 16LL * ((shared_values ? cols : vcols) * 16 + 4) * 4 + (shared_values ? 64LL * heads * vcols : 0);
+    if (stages < 2 || stages * kt * pitch < outputs) continue;
     const int shares = 64 / kt, steps = ((key_width + 15) / 16 + shares - 1) / shares;
     return {kt, stages, nc, steps <= 4 ? 4 : steps <= 16 ? 16 : 0};
   }
@@ -477,7 +517,7 @@ static int launch_gw(const GwParams& p, int rows, int splits, cudaStream_t strea
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = dim3(rows, splits, p.head_blocks);
   cfg.blockDim = dim3(kGwThreads + 32);
-  cfg.dynamicSmemBytes = GwLayout(p.key_width, p.stages * KT * p.pitch, KT).total;
+  cfg.dynamicSmemBytes = GwLayout(p.key_width, p.stages * KT * p.pitch, KT, p.talk ? p.heads : 0).total;
   cfg.stream = stream;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -509,10 +549,23 @@ static int launch_gw_cols(const GwParams& p, const GwPlan& plan, int rows, int s
 
 using namespace fb;
 
-extern "C" int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads) {
+// key columns of a CTA: of the most kv heads that a block of 16 heads has, when query rows meet their own kv head's keys
+static int gw_key_width(int key_width, int own_keys, int heads, int kv_heads) {
+  if (!own_keys) return key_width;
+  int most = 0;
+  for (int h0 = 0, per = heads / kv_heads; h0 < heads; h0 += 16) {
+    const int last = (h0 + 16 < heads ? h0 + 16 : heads) - 1, n = last / per - h0 / per + 1;
+    if (n > most) most = n;
+  }
+  return most * key_width;
+}
+
+extern "C" int fb_gqa_decode_wide_ok(int key_width, int kv_heads, int vdim_pad, int shared_values, int heads, int own_keys) {
+  if (kv_heads <= 0 || heads <= 0 || heads % kv_heads) return 0;
   if (shared_values && (heads + 15) / 16 > 8) return 0;       // the row's head blocks form one cluster
+  key_width = gw_key_width(key_width, own_keys, heads, kv_heads);
   return key_width > 0 && key_width % 8 == 0 && kv_heads > 0 && vdim_pad > 0 && vdim_pad % 8 == 0 &&
-         gw_plan(key_width, kv_heads, vdim_pad, shared_values != 0).kt > 0;
+         gw_plan(key_width, kv_heads, vdim_pad, shared_values != 0, heads).kt > 0;
 }
 
 extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, void* stream) {
@@ -533,7 +586,8 @@ extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, voi
                          reinterpret_cast<uintptr_t>(a->out) | reinterpret_cast<uintptr_t>(a->gate) |
                          reinterpret_cast<uintptr_t>(a->pooled);
   if (bits & 15) return FB_ERR_ALIGN;
-  const GwPlan plan = gw_plan(static_cast<int>(key_width), a->kv_heads, a->vdim_pad, shared_values);
+  const int cta_width = gw_key_width(a->key_width, a->key_stride, a->heads, a->kv_heads);
+  const GwPlan plan = gw_plan(cta_width, a->kv_heads, a->vdim_pad, shared_values, a->heads);
   if (plan.kt == 0) return FB_ERR_LIMIT;
   GwParams p{};
   p.q = static_cast<const __nv_bfloat16*>(a->q); p.ldq = a->ldq;
@@ -551,7 +605,7 @@ extern "C" int fb_gqa_decode_wide(const FbGqaArgs* a, int splits, int early, voi
   }
   p.slopes = a->slopes; p.gate = static_cast<const __nv_bfloat16*>(a->gate); p.ldg = a->ldg;
   p.out = static_cast<__nv_bfloat16*>(a->out); p.ldo = a->ldo;
-  p.heads = a->heads; p.kv_heads = a->kv_heads; p.key_width = static_cast<int>(key_width); p.vdim_pad = a->vdim_pad;
+  p.heads = a->heads; p.kv_heads = a->kv_heads; p.key_width = cta_width; p.v_offset = a->v_offset; p.vdim_pad = a->vdim_pad;
   p.row_bytes = (p.key_width + a->kv_heads * a->vdim_pad) * 2;
   p.pitch = p.row_bytes + 16;
   p.stages = plan.stages;

@@ -85,7 +85,7 @@ def declare(lib) -> None:
         "fb_gqa_attention": ([vp, vp], i),
         "fb_gqa_decode": ([vp, i, i, vp], i),
         "fb_gqa_decode_wide": ([vp, i, i, vp], i),
-        "fb_gqa_decode_wide_ok": ([i, i, i, i, i], i),
+        "fb_gqa_decode_wide_ok": ([i, i, i, i, i, i], i),
         "fb_value_mix": ([vp, ll, vp, vp, ll, i, i, i, i, i, vp], i),
         "fb_pool_blocks": ([vp, vp], i),
         "fb_pre_norm_step": ([vp, vp], i),

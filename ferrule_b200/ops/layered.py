@@ -528,8 +528,8 @@ def gqa_decode_supported(mixer, dtype, page_size: int) -> bool:
     if dtype != torch.bfloat16:
         return False
     if mixer.shared_keys or mixer.shared_values:
-        width = mixer.key_width if mixer.shared_keys else mixer.kv_heads * mixer.key_width
-        return bool(get_lib(True).fb_gqa_decode_wide_ok(width, mixer.kv_heads, mixer.vdim_pad, mixer.shared_values, mixer.heads))
+        return bool(get_lib(True).fb_gqa_decode_wide_ok(mixer.key_width, mixer.kv_heads, mixer.vdim_pad, mixer.shared_values,
+                                                        mixer.heads, not mixer.shared_keys))
     if mixer.pool or mixer.softcap:
         return False
     return max(mixer.key_width, mixer.vdim_pad) <= 256
