@@ -105,7 +105,8 @@ def main() -> None:
                     help="deepseek-v2-lite is the headline configuration; gitozen-lite, gitozen-latent-lite and supisun-lite are "
                          "layer-list models of the same widths (one GPU), supisun-small and supisun-wide others, "
                          "gitozen-dense-small / -lite / -wide have their sizes; vedadra-small / -lite / -wide and "
-                         "supisun-attention-small / -lite / -wide of the same sizes; they are reported without a baseline")
+                         "supisun-attention-small / -lite / -wide of the same sizes; vogunex-small / -lite / -wide have supisun's "
+                         "sizes, vogunex-moe-lite gitozen-lite's; they are reported without a baseline")
     ap.add_argument("--weight-format", default="bf16", choices=["bf16", "fp8_block", "fp8_mxfp4"],
                     help="bf16 is the headline configuration; the FP8 formats are reported with their own dtype")
     ap.add_argument("--shard-as", type=int, default=0,

@@ -7,8 +7,8 @@
 // Prompts of bf16 models take the chunked form (head_scan_chunk.cu) where the sizes allow it.  Token by token, any mix of row
 // counts: CTA = (columns of a head, head, sequence).  LPC lanes share VPL columns and hold SPL state rows of each in
 // registers; sixteen tokens are staged at a time and the next ones requested before the staged ones are worked on.
-// Sequences with one row (decode steps, and the single rows beside chunked prompts): CTA = (head, sequence), the state streams through registers once; its first part is
-// requested before the dependency wait.
+// Sequences with one row (decode steps, and the single rows beside chunked prompts): CTA = (head, sequence), the
+// state streams through registers once; its first part is requested before the dependency wait.
 //
 // State of a sequence: fp32 [heads, state, vdim].  Buffer `state_in[seq]` is read (-1: a new sequence, zeros), buffer
 // `state_out[seq]` written (-1: nothing is kept), never the same one.

@@ -11,8 +11,9 @@
 // CTA = (64 columns of a head, head, sequence), four warps with 16 columns each.  A warp keeps the transposed state of its
 // columns as MMA accumulators: their layout is that of the B operand of C S.  Per chunk: the warps compute the masked and
 // decayed products P of C and B together (16 rows each, two bf16 parts in shared memory), then every warp its columns of y and
-// of the state.  L is summed in double and kept as two floats: behind a strong decay it is large, its differences may be small.  The next chunk's rows are copied while this one is worked on.  A 64-token chunk of a head is too small for the
-// 128-row tiles of tcgen05, and the accumulators feed the next product from registers: warp-level MMA.
+// of the state.  L is summed in double and kept as two floats: behind a strong decay it is large, its differences may be small.  The
+// next chunk's rows are copied while this one is worked on.  A 64-token chunk of a head is too small for the 128-row tiles of
+// tcgen05, and the accumulators feed the next product from registers: warp-level MMA.
 #include "act_type.cuh"
 #include "common.cuh"
 #include "head_scan.cuh"
